@@ -49,6 +49,89 @@ void zse_gemm_w4_dec_set_tuning(int min_steps, int max_split);
 int zse_gemm_f16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, const void* bias, void* out, int M,
                  int N, int K, int ldo, int epilogue, int k_split, void* status, void* stream);
 int zse_gemm_f16_splits(int M, int N, int K, int k_split);
+// the same kernel on bfloat16 weights and activations (epilogue 0: bfloat16 store, 2: fp32 planes)
+int zse_gemm_bf16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, void* out, int M, int N, int K, int ldo,
+                  int epilogue, int k_split, void* status, void* stream);
+
+// ---- gemm_tile.cu -------------------------------------------------------------------------------------------
+// dtype of the functions below: 1 = bfloat16, 2 = float.
+typedef struct ZseTileGemm {
+  const void* a;            // [M, K], row stride lda, batch stride a_batch
+  int64_t lda, a_batch;
+  const void* b;            // element (n, k) at n * ldb_n + k * ldb_k, batch stride b_batch, expert stride b_group
+  int64_t ldb_n, ldb_k, b_batch, b_group;
+  void* out;                // row stride ldo, batch stride o_batch; row m goes to out_rows[m] or m * out_row_mul + add
+  int64_t ldo, o_batch;
+  int32_t M, N, K, epilogue;   // 0 store, 1 fp32 store, 2 gelu(row_scale * acc), 3 acc * sigmoid(gate)
+  const float* row_scale;
+  const int32_t* out_rows;
+  int32_t out_row_mul, out_row_add;
+  const void* gate;
+  int64_t ldg, gate_batch;
+  const void* tiles;        // grouped: MoeTile table and its length on the device (tiles of 64 rows)
+  const int32_t* n_tiles;
+} ZseTileGemm;
+int zse_gemm_tile(int dtype, const ZseTileGemm* a, int batch, int max_tiles, void* stream);
+
+int zse_apply_repetition_penalty_f32(void* logits, int ld, const void* rows_i32, const void* tokens_i32,
+                                     const void* counts_i32, int n, const void* penalty_f32, int V, void* stream);
+
+// ---- rows.cu ------------------------------------------------------------------------------------------------
+int zse_embedding_typed(int dtype, const void* table, const void* ids, void* out_f32, int M, int H, int vocab,
+                        float scale, void* status, void* stream);
+// residual += planes [n_planes][M][H] + slots [M][n_slots][H]; out = RMSNorm(residual) * weight
+int zse_add_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes, const void* slots,
+                 int n_slots, const void* weight, void* out, int M, int H, float eps, void* stream);
+// fp32 logits in place: cap * tanh(scale * x / cap) (cap 0: scale * x)
+int zse_logits_finish(void* logits, int ld, int M, int V, float scale, float cap, void* stream);
+int zse_argmax_f32(const void* logits, int ld, void* out_i32, int M, int V, void* stream);
+
+// ---- latent.cu ----------------------------------------------------------------------------------------------
+typedef struct ZseRowCache {
+  void* rows;               // one layer's cached rows [blocks][block_size][row], blocks block_stride elements apart
+  int64_t block_stride;
+  int32_t block_size, row;
+  const void* tables;       // block tables [sequences][max_blocks]
+  int32_t max_blocks;
+} ZseRowCache;
+typedef struct ZseChunks {  // sequences [first, last) of a packed pass
+  const void *cu_q, *q_pos0, *ctx_off;
+  int32_t first, last, window;
+} ZseChunks;
+int zse_latent_mma_ok(int heads, int dim, int rot, int vdim, int kv_rank, int row);
+int zse_latent_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, int M, const ZseRowCache* c,
+                    const void* positions, const void* slots, const void* freqs, const void* norm_w, int heads, int dim,
+                    int rot, int rot_dims, int kv_rank, int latent_col, int gate_col, int gate_w, float eps,
+                    void* stream);
+int zse_latent_attn(int dtype, const void* q_lat, const ZseRowCache* c, const void* row_seq, const void* positions,
+                    void* o_lat, void* scratch, int M, int heads, int used, int kv_rank, int window, float scale,
+                    int num_splits, int tensor_cores, void* stream);
+int zse_latent_absorb(const void* inp, int ld, const void* uk, void* q_lat, int M, int heads, int dim, int rot,
+                      int kv_rank, int row, void* stream);
+int zse_latent_unabsorb(const void* o_lat, const void* uv, const void* gate, int ldg, void* out, int ldo, int M,
+                        int heads, int vdim, int kv_rank, void* stream);
+int zse_latent_gather(const ZseRowCache* c, const ZseChunks* g, int rows, int kv_rank, int rot, void* c_out,
+                      void* kr_out, void* stream);
+int zse_latent_chunk(const void* inp, int ld, const void* kvx, int ldkv, int v_col, const void* kr_ctx,
+                     const ZseRowCache* c, const ZseChunks* g, int max_q, void* out, int ldo, const void* gate, int heads,
+                     int dim, int rot, int vdim, float scale, void* stream);
+
+// ---- moe.cu -------------------------------------------------------------------------------------------------
+int zse_moe_tile_rows(int M, int E, int top);
+// router logits (fp32 planes) -> chosen experts, sorted rows, tile table; `counts` [E] must be zero and is zero afterwards
+int zse_moe_route(int dtype, const void* planes, int n_planes, int M, int E, int top, int tile_rows, const void* x, int H,
+                  int out_per_token, void* counts, void* slot_expert, void* slot_rank, void* slot_score,
+                  void* first_row, void* tiles, void* n_tiles, void* xs, void* row_score, void* out_rows, void* stream);
+typedef struct ZseMoeGemm {
+  const void *routed_w, *routed_x;
+  void* routed_out;
+  const void *shared_w, *shared_x;
+  void* shared_out;
+  const void *row_score, *out_rows, *tiles, *n_tiles;
+  int32_t routed_n, routed_k, routed_ldo, shared_n, shared_k, shared_ldo, shared_mul, shared_add, shared_x_rows;
+} ZseMoeGemm;
+int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int tile_rows, int max_tiles, int epilogue,
+                 void* status, void* stream);
 
 // ---- repack.cu ----------------------------------------------------------------------------------------------
 // Row-major INT4 [N, K/2] + scales/zeros [N, K/128] -> tiled chunks.  interleave_rows > 0 builds a fused gate/up

@@ -1,4 +1,4 @@
-// Dense fp16-weight linear layers on the 5th-generation tensor cores (lm_head, tensors the INT4 kernel does not
+// Dense fp16- and bfloat16-weight linear layers on the 5th-generation tensor cores (lm_head, tensors the INT4 kernel does not
 // take, int8 models expanded at load).
 //
 //   Y[t, n] = sum_k X[t, k] * W[n, k]          X fp16 [M, K] row-major, W fp16 [N, K] row-major
@@ -13,6 +13,7 @@
 #include <unordered_map>
 
 #include "gemm_common.cuh"
+#include "typed.cuh"
 
 namespace zse {
 
@@ -28,7 +29,7 @@ struct PipeBars {
 // ---- epilogue shared by both kernels ---------------------------------------------------------------
 // Warps 2..9: quarter q = warp % 4 owns TMEM lanes [32q, 32q+32); half ch = (warp-2)/4 owns the columns
 // [ch*NT/2, (ch+1)*NT/2) (for NT == 16 only ch == 0 works).
-template <int NT, int EPI>
+template <int NT, int EPI, bool BF16>
 __device__ __forceinline__ void epilogue(const GemmArgs& a, uint32_t tmem_acc, int warp, int lane, float* stage_smem,
                                          bool valid) {
   const int q = warp & 3;
@@ -94,7 +95,9 @@ __device__ __forceinline__ void epilogue(const GemmArgs& a, uint32_t tmem_acc, i
       const int t = t0 + col0 + c + i;
       if (t < a.M && n_ok) {
         const float v = __uint_as_float(r[i]);
-        if (EPI == kEpiF16) {
+        if (EPI == kEpiF16 && BF16) {
+          reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n] = __float2bfloat16_rn(v);
+        } else if (EPI == kEpiF16) {
           reinterpret_cast<__half*>(a.out)[size_t(t) * a.ldo + n] = __float2half_rn(clamp_f16(v + bias));
         } else {
           reinterpret_cast<float*>(a.out)[(size_t(blockIdx.z) * a.M + t) * a.ldo + n] = v;
@@ -117,7 +120,7 @@ struct F16Cfg {
   static constexpr int kMinBlocks = NT <= 64 ? 2 : 1;
 };
 
-template <int NT, int EPI>
+template <int NT, int EPI, bool BF16>
 __global__ void __launch_bounds__(kGemmThreads, F16Cfg<NT>::kMinBlocks)
 gemm_f16_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x,
                 const GemmArgs a) {
@@ -176,7 +179,7 @@ gemm_f16_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constan
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      constexpr uint32_t idesc = make_idesc_f16(kTileN, NT);
+      constexpr uint32_t idesc = make_idesc_f16(kTileN, NT, BF16 ? 1 : 0);
       for (int it = 0; it < n_iter; ++it) {
         const int s = it % S;
         if (!mbar_wait(&bars->full[s], (it / S) & 1, abort_flag, a.status, 12, it)) break;
@@ -193,7 +196,7 @@ gemm_f16_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constan
   } else {
     const bool ok = mbar_wait(&bars->acc_ready, 0, abort_flag, a.status, 15, 0);
     tc_fence_after_sync();
-    epilogue<NT, EPI>(a, tmem, warp, lane, reinterpret_cast<float*>(smem), ok);
+    epilogue<NT, EPI, BF16>(a, tmem, warp, lane, reinterpret_cast<float*>(smem), ok);
   }
   tc_fence_before_sync();
   __syncthreads();
@@ -261,9 +264,9 @@ int get_tmap(const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows, C
   return 0;
 }
 
-template <int NT, int EPI>
+template <int NT, int EPI, bool BF16>
 static int launch_f16(const CUtensorMap& tw, const CUtensorMap& tx, const GemmArgs& a, dim3 grid, cudaStream_t st) {
-  auto kern = gemm_f16_kernel<NT, EPI>;
+  auto kern = gemm_f16_kernel<NT, EPI, BF16>;
   static bool attr_done[kMaxDevices] = {};
   const int dev_slot = current_device_slot();
   if (!attr_done[dev_slot]) {
@@ -281,8 +284,9 @@ static int launch_f16(const CUtensorMap& tw, const CUtensorMap& tx, const GemmAr
 
 using namespace zse;
 
-extern "C" int zse_gemm_f16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, const void* bias, void* out,
-                            int M, int N, int K, int ldo, int epilogue, int k_split, void* status, void* stream) {
+template <bool BF16>
+static int gemm_16bit(const void* w, int w_rows_cap, const void* x, int x_rows_cap, const void* bias, void* out, int M,
+                      int N, int K, int ldo, int epilogue, int k_split, void* status, void* stream) {
   if (M <= 0) return 0;
   if (K % 8 != 0 || N <= 0 || epilogue == kEpiSwiGLU) return ZSE_ERR_SHAPE;
   if (epilogue != kEpiPartialF32) k_split = 1;
@@ -300,11 +304,21 @@ extern "C" int zse_gemm_f16(const void* w, int w_rows_cap, const void* x, int x_
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   int rc = ZSE_ERR_SHAPE;
   if (epilogue == kEpiF16) {
-    ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiF16>(tw, tx, a, grid, st)))
+    ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiF16, BF16>(tw, tx, a, grid, st)))
   } else {
-    ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiPartialF32>(tw, tx, a, grid, st)))
+    ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiPartialF32, BF16>(tw, tx, a, grid, st)))
   }
   return rc;
+}
+
+extern "C" int zse_gemm_f16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, const void* bias, void* out,
+                            int M, int N, int K, int ldo, int epilogue, int k_split, void* status, void* stream) {
+  return gemm_16bit<false>(w, w_rows_cap, x, x_rows_cap, bias, out, M, N, K, ldo, epilogue, k_split, status, stream);
+}
+
+extern "C" int zse_gemm_bf16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, void* out, int M, int N, int K,
+                             int ldo, int epilogue, int k_split, void* status, void* stream) {
+  return gemm_16bit<true>(w, w_rows_cap, x, x_rows_cap, nullptr, out, M, N, K, ldo, epilogue, k_split, status, stream);
 }
 
 extern "C" int zse_gemm_f16_splits(int M, int N, int K, int k_split) {

@@ -254,7 +254,13 @@ sample_kernel(const __half* __restrict__ logits, int ld, int* __restrict__ out, 
 }
 
 // logit <- logit / f (positive) or logit * f (negative), f = penalty^(1 + log2(count))
-__global__ void repetition_penalty_kernel(__half* __restrict__ logits, int ld, const int* __restrict__ rows,
+__device__ __forceinline__ float logit_value(__half v) { return __half2float(v); }
+__device__ __forceinline__ float logit_value(float v) { return v; }
+__device__ __forceinline__ void set_logit(__half* p, float v) { *p = __float2half_rn(v); }
+__device__ __forceinline__ void set_logit(float* p, float v) { *p = v; }
+
+template <typename L>
+__global__ void repetition_penalty_kernel(L* __restrict__ logits, int ld, const int* __restrict__ rows,
                                           const int* __restrict__ tokens, const int* __restrict__ counts, int n,
                                           const float* __restrict__ penalty, int V) {
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
@@ -263,9 +269,9 @@ __global__ void repetition_penalty_kernel(__half* __restrict__ logits, int ld, c
   const float pen = penalty[r];
   if (c <= 0 || pen == 1.f || t < 0 || t >= V) return;
   const float f = powf(pen, 1.f + log2f(float(c)));
-  __half* p = logits + size_t(r) * ld + t;
-  const float v = __half2float(*p);
-  *p = __float2half_rn(v > 0.f ? v / f : v * f);
+  L* p = logits + size_t(r) * ld + t;
+  const float v = logit_value(*p);
+  set_logit(p, v > 0.f ? v / f : v * f);
 }
 
 }  // namespace zse
@@ -293,8 +299,17 @@ extern "C" int zse_sample(const void* logits, int ld, void* out, int M, int V, c
 extern "C" int zse_apply_repetition_penalty(void* logits, int ld, const void* rows, const void* tokens,
                                             const void* counts, int n, const void* penalty, int V, void* stream) {
   if (n <= 0) return 0;
-  repetition_penalty_kernel<<<(n + 255) / 256, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
+  repetition_penalty_kernel<__half><<<(n + 255) / 256, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
       reinterpret_cast<__half*>(logits), ld, reinterpret_cast<const int*>(rows), reinterpret_cast<const int*>(tokens),
+      reinterpret_cast<const int*>(counts), n, reinterpret_cast<const float*>(penalty), V);
+  return cudaGetLastError() == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+}
+
+extern "C" int zse_apply_repetition_penalty_f32(void* logits, int ld, const void* rows, const void* tokens,
+                                                const void* counts, int n, const void* penalty, int V, void* stream) {
+  if (n <= 0) return 0;
+  repetition_penalty_kernel<float><<<(n + 255) / 256, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
+      reinterpret_cast<float*>(logits), ld, reinterpret_cast<const int*>(rows), reinterpret_cast<const int*>(tokens),
       reinterpret_cast<const int*>(counts), n, reinterpret_cast<const float*>(penalty), V);
   return cudaGetLastError() == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }

@@ -2,7 +2,8 @@
 
 The slab is a single fp16 tensor ``[layers, blocks, 2 (K,V), kv_heads, block_size, head_dim]``: per layer every
 block's K (and V) for one kv head is a contiguous ``block_size*head_dim`` run, which is what the attention kernels
-stream.  Bookkeeping (free list, reference counts for shared/forked blocks) is host-side, as in
+stream.  Models that cache one latent row per token instead of K and V use the same pool with ``planes=1`` and one kv
+head, at the width of their activations.  Bookkeeping (free list, reference counts for shared/forked blocks) is host-side, as in
 zse-engine/zse_engine/cache/block_pool.py:18-282; with ``device=None`` the pool only does bookkeeping, which is
 how the CPU tests and the scheduler simulations use it.
 """
@@ -39,13 +40,14 @@ class Block:
 
 class BlockPool:
     def __init__(self, num_blocks: int, block_size_tokens: int, num_layers: int, num_kv_heads: int, head_dim: int,
-                 device=None, dtype=torch.float16):
+                 device=None, dtype=torch.float16, planes: int = 2):
         if num_blocks <= 0:
             raise ValueError("the KV budget is smaller than one block")
         self._num_blocks = num_blocks
         self._block_size = block_size_tokens
-        self._shape = (num_layers, num_blocks, 2, num_kv_heads, block_size_tokens, head_dim)
-        self._bytes_per_token = num_layers * 2 * num_kv_heads * head_dim * 2
+        self._shape = (num_layers, num_blocks, planes, num_kv_heads, block_size_tokens, head_dim)
+        self._itemsize = torch.empty(0, dtype=dtype).element_size()
+        self._bytes_per_token = num_layers * planes * num_kv_heads * head_dim * self._itemsize
         self._free: Deque[int] = deque(range(num_blocks))
         self._blocks: Dict[int, Block] = {}
         self.slab: Optional[torch.Tensor] = None
@@ -55,9 +57,11 @@ class BlockPool:
 
     @classmethod
     def from_budget(cls, budget_bytes: int, block_size_tokens: int, num_layers: int, num_kv_heads: int,
-                    head_dim: int, device=None) -> "BlockPool":
-        block_bytes = block_size_tokens * num_layers * 2 * num_kv_heads * head_dim * 2
-        return cls(budget_bytes // block_bytes, block_size_tokens, num_layers, num_kv_heads, head_dim, device)
+                    head_dim: int, device=None, dtype=torch.float16, planes: int = 2) -> "BlockPool":
+        block_bytes = (block_size_tokens * num_layers * planes * num_kv_heads * head_dim
+                       * torch.empty(0, dtype=dtype).element_size())
+        return cls(budget_bytes // block_bytes, block_size_tokens, num_layers, num_kv_heads, head_dim, device, dtype,
+                   planes)
 
     # ---- facts ----------------------------------------------------------------------------------------
     @property
@@ -99,8 +103,8 @@ class BlockPool:
     # ---- addresses (zse-engine/zse_engine/cache/block_pool.py:163-258, for this pool's layer-major slab) -------
     @property
     def layer_block_bytes(self) -> int:
-        _, _, two, kvh, bs, hd = self._shape
-        return two * kvh * bs * hd * 2
+        _, _, planes, kvh, bs, hd = self._shape
+        return planes * kvh * bs * hd * self._itemsize
 
     @property
     def is_uniform_kv(self) -> bool:
@@ -129,7 +133,7 @@ class BlockPool:
         return self.gpu_ptr_for_block_layer(block, 0)
 
     def gpu_ptr_for_kv(self, block: Block, layer: int, is_value: bool) -> int:
-        return self.gpu_ptr_for_block_layer(block, layer) + (self.layer_block_bytes // 2 if is_value else 0)
+        return self.gpu_ptr_for_block_layer(block, layer) + (self.layer_block_bytes // 2 if is_value and self._shape[2] == 2 else 0)
 
     # ---- alloc / free ---------------------------------------------------------------------------------
     def alloc(self, seq_id: Optional[int] = None) -> Block:

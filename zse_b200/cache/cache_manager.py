@@ -16,6 +16,7 @@ from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence, Set
 
 import numpy as np
+import torch
 
 from ..format.config import ModelConfig
 from .attention_metadata import AttentionMetadata
@@ -55,7 +56,7 @@ class CacheStats:
 class KVCacheManager:
     def __init__(self, config: ModelConfig, device=None, budget_bytes: int = 0, block_size: int = 0,
                  eviction_policy: str = "smart", enable_dedup: bool = True, num_kv_heads: Optional[int] = None,
-                 num_blocks: int = 0):
+                 num_blocks: int = 0, dtype=None):
         self._config = config
         self._lock = threading.RLock()
         self._block_size = block_size if block_size > 0 else self._auto_block_size(config)
@@ -63,16 +64,18 @@ class KVCacheManager:
             raise ValueError("block_size must be a multiple of 16")
         # local kv heads under tensor parallelism; rows of the widest layer when layers differ (Gemma-4)
         nkv, pool_hd = config.kv_pool_dims(num_kv_heads)
+        kind = dict(planes=config.kv_planes, dtype=dtype or torch.float16)
         if num_blocks > 0:
-            self._pool = BlockPool(num_blocks, self._block_size, config.num_layers, nkv, pool_hd, device)
+            self._pool = BlockPool(num_blocks, self._block_size, config.num_layers, nkv, pool_hd, device, **kind)
         else:
             if budget_bytes <= 0:
                 raise ValueError("either budget_bytes or num_blocks is required")
             self._pool = BlockPool.from_budget(budget_bytes, self._block_size, config.num_layers, nkv,
-                                               pool_hd, device)
-        # a uniform window (Mistral) lets old blocks go; models that mix local and global layers keep everything and
-        # apply the window inside attention
-        self._windowed = bool(config.sliding_window and config.sliding_window > 0 and not config.layer_types)
+                                               pool_hd, device, **kind)
+        # a window that bounds every layer (Mistral) lets old blocks go; models that mix local and global layers keep
+        # everything and apply the window inside attention
+        self._window = config.cache_window
+        self._windowed = self._window > 0
         self._page_table = PageTable(self._pool)
         self._evictor = Evictor(eviction_policy)
         self._dedup = BlockDedup(self._pool) if enable_dedup else None
@@ -85,6 +88,8 @@ class KVCacheManager:
     @staticmethod
     def _auto_block_size(config: ModelConfig) -> int:
         """<= 4096 context: 16; <= 32768: 32; longer: 64; halved (not below 16) for heavy GQA (kv/heads <= 1/4)."""
+        if config.is_latent:                 # one narrow row per token: 64 rows are one attention tile
+            return 64
         base = 16 if config.max_seq_len <= 4096 else 32 if config.max_seq_len <= 32768 else 64
         if config.num_kv_heads / config.num_heads <= 0.25 and base > 16:
             base //= 2
@@ -170,6 +175,8 @@ class KVCacheManager:
             if cur + num_new_tokens > self._config.max_seq_len:
                 raise ValueError(f"extending sequence {seq_id} to {cur + num_new_tokens} tokens exceeds max_seq_len "
                                  f"{self._config.max_seq_len}")
+            if self._windowed:
+                self._trim_sliding_window(seq_id, cur)
             need = self._page_table.blocks_needed(seq_id, num_new_tokens)
             if need > self._pool.num_free and not self._evict_locked(need):
                 raise RuntimeError(f"cannot extend sequence {seq_id}: need {need} KV blocks, "
@@ -178,8 +185,6 @@ class KVCacheManager:
             if new_ids:
                 e = self._page_table.get_entry(seq_id)
                 self._track_blocks(e, max(0, len(e.blocks) - len(new_ids) - 1))
-            if self._windowed:
-                self._trim_sliding_window(seq_id)
 
     def _track_blocks(self, e, first_idx: int) -> None:
         """Tells the evictor about blocks ``first_idx..`` of a sequence (new, shared or copied ones)."""
@@ -201,8 +206,9 @@ class KVCacheManager:
         with self._lock:
             for i, sid in enumerate(seq_ids):
                 e = self._page_table.get_entry_or_none(sid)
-                if e is not None and not windowed:
-                    n = e.num_tokens
+                n = e.num_tokens if e is not None else 0
+                # (the step that moves the window's start over a block border gives a block back: ordinary path)
+                if e is not None and (not windowed or (n + 1 - self._window) % bs):
                     fill = n % bs
                     if fill and n < limit and e.blocks:
                         tail = e.blocks[-1]
@@ -303,12 +309,14 @@ class KVCacheManager:
                 return True
         return self._pool.num_free >= blocks_needed
 
-    def _trim_sliding_window(self, seq_id: int) -> None:
+    def _trim_sliding_window(self, seq_id: int, first_new: int) -> None:
+        """Gives back the blocks no token from position ``first_new`` on can see: that token itself still sees the
+        ``window - 1`` before it, however many more are appended with it."""
         e = self._page_table.get_entry_or_none(seq_id)
-        window = self._config.sliding_window
-        if e is None or e.num_tokens <= window:
+        keep_from = first_new + 1 - self._window
+        if e is None or keep_from <= 0:
             return
-        for idx in range((e.num_tokens - window) // self._block_size):
+        for idx in range(min(keep_from // self._block_size, len(e.blocks))):
             if idx not in e.evicted_indices:
                 self._evictor.remove_block(e.blocks[idx].block_id, seq_id)
                 self._page_table.evict_block(seq_id, idx)

@@ -44,6 +44,8 @@ class EngineConfig:
     eviction_policy: str = "smart"
     enable_prefix_cache: bool = True
     int4_layout: Optional[str] = None     # override for files that do not record their INT4 layout
+    dtype: Optional[str] = None           # "bfloat16" | "float32" for the models that offer both; None = the model's own
+    logits_rows: int = 0                  # most logits rows one pass may be asked for (0 = one per sequence, at least 64)
     device: Optional[str] = None          # "cpu" forces the torch path
     quiet: bool = True
 

@@ -25,7 +25,7 @@ import torch
 
 from .cache.cache_manager import KVCacheManager
 from .config import EngineConfig
-from .format.loader import ZSELoader
+from .format.directory import open_model
 from .models.decoder import DecoderModel
 from .runtime.runner import ModelRunner
 from .runtime.vram import VRAMAllocator
@@ -94,13 +94,14 @@ class ZStreamerEngine:
         self.device = torch.device(f"cuda:{cfg.device_index}" if on_gpu else "cpu")
         if on_gpu:
             torch.cuda.set_device(self.device)
-        self._loader = ZSELoader(model_path, int4_layout=cfg.int4_layout)
+        self._loader = open_model(model_path, int4_layout=cfg.int4_layout)
         self._config = self._loader.config
         self._tokenizer = self._loader.tokenizer
         self.init_times["open"] = time.monotonic() - t0
 
         t1 = time.monotonic()
-        self._model = DecoderModel.from_loader(self._loader, self.device, tp_size=cfg.tp_size, rank=tp_rank)
+        self._model = DecoderModel.from_loader(self._loader, self.device, tp_size=cfg.tp_size, rank=tp_rank,
+                                               dtype=cfg.dtype)
         self._model.comm = comm
         if on_gpu:
             torch.cuda.synchronize(self.device)
@@ -109,7 +110,8 @@ class ZStreamerEngine:
 
         t2 = time.monotonic()
         mc = self._config
-        self._max_seq_len = min(cfg.max_seq_len or mc.max_seq_len, mc.max_seq_len, 32768)
+        self._max_seq_len = min(cfg.max_seq_len or 32768, mc.max_seq_len)
+        act = self._model.act_dtype
         block_size = cfg.block_size or KVCacheManager._auto_block_size(mc)
         nkv_local = self._model.plan.num_kv_heads
         if cfg.kv_blocks > 0:
@@ -118,16 +120,17 @@ class ZStreamerEngine:
             scratch_est = cfg.max_batch_tokens * (mc.hidden_size * 40 + mc.intermediate_size * 2) + (256 << 20)
             plan = VRAMAllocator.for_device(self.device).plan_allocation(
                 mc, 0, scratch_est, block_size, self._max_seq_len, cfg.max_batch_seqs, cfg.tp_size, cfg.kv_fraction)
-            blocks = plan.kv_blocks
+            blocks = max(1, plan.kv_blocks * 2 // act.itemsize)       # the plan counts 16-bit elements
             self.vram_plan = plan
         else:
             blocks = max(64, (cfg.max_batch_seqs * min(self._max_seq_len, 2048)) // block_size)
         self._kv_cache = KVCacheManager(mc, self.device, block_size=block_size, num_blocks=blocks,
                                         eviction_policy=cfg.eviction_policy, enable_dedup=cfg.enable_prefix_cache,
-                                        num_kv_heads=nkv_local)
+                                        num_kv_heads=nkv_local, dtype=act)
         self._runner = ModelRunner(self._model, self._kv_cache, max_batch_seqs=cfg.max_batch_seqs,
                                    max_tokens_per_pass=max(cfg.max_batch_tokens, cfg.prefill_chunk_size or 0),
-                                   max_seq_len=self._max_seq_len, use_graphs=cfg.use_cuda_graphs)
+                                   max_seq_len=self._max_seq_len, use_graphs=cfg.use_cuda_graphs,
+                                   logits_rows=cfg.logits_rows)
         from .lora.manager import LoRAManager
         self._lora_manager = LoRAManager(self._model, self.device)
         self._budget = MemoryBudget(blocks, block_size, cfg.headroom_ratio)

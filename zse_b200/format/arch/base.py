@@ -41,9 +41,10 @@ def detect_architecture(hf_config: dict) -> str:
         for needle, arch in _DETECT:
             if needle in low:
                 return arch
-    mt = str(hf_config.get("model_type", "")).lower()
-    if mt in _REGISTRY:
-        return mt
+    for key in ("model_type", "architecture"):
+        name = str(hf_config.get(key, "")).lower()
+        if name in _REGISTRY:
+            return name
     raise ValueError(f"cannot detect the architecture (architectures={hf_config.get('architectures')}, "
                      f"model_type={hf_config.get('model_type')})")
 
@@ -71,6 +72,8 @@ class ArchAdapter:
     LAYER_TENSORS = ("self_attn.q_proj.weight", "self_attn.k_proj.weight", "self_attn.v_proj.weight",
                      "self_attn.o_proj.weight", "mlp.gate_proj.weight", "mlp.up_proj.weight",
                      "mlp.down_proj.weight", "input_layernorm.weight", "post_attention_layernorm.weight")
+    #: width of tensors that are not quantised
+    STORED_DTYPE = "float16"
 
     def config_from_hf(self, hf_config: dict) -> ModelConfig:
         hf = hf_config

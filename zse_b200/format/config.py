@@ -49,6 +49,60 @@ class LayerSpec:
     qk_norm: bool            # per-head RMSNorm of q and k (learned weight) and of v (no weight)
 
 
+def _up8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+@dataclass(frozen=True)
+class LatentSpec:
+    """Attention over a shared low-rank latent: a token caches its normed latent (``kv_rank``) and one rotated key part
+    (``rot_dim``) that all heads share; a head's key and value are linear images of the latent."""
+    heads: int
+    dim: int                 # query/key dimensions of a head that carry no position
+    rot_dim: int             # ... and those that are rotated
+    vdim: int
+    kv_rank: int
+    window: int              # a position sees itself and the window - 1 before it; 0 = everything before it
+    scale: float
+    rot_dims: int            # leading dimensions of the rot_dim part that rotate (pairs 2i, 2i + 1)
+    rot_base: float
+    gated: bool = True       # heads are multiplied by sigmoid(W_g h) before the output projection
+
+    @property
+    def qk_dim(self) -> int:
+        return self.dim + self.rot_dim
+
+    # columns of the fused input projection [q | latent, rotated key | gate]; every section starts on 8 elements
+    @property
+    def latent_col(self) -> int:
+        return _up8(self.heads * self.qk_dim)
+
+    @property
+    def gate_col(self) -> int:
+        return self.latent_col + _up8(self.kv_rank + self.rot_dim)
+
+    @property
+    def in_width(self) -> int:
+        return self.gate_col + (_up8(self.heads * self.vdim) if self.gated else 0)
+
+    @property
+    def row(self) -> int:
+        """Elements of a cached token: [latent | rotated key part], padded to 16 bytes of a 16-bit type."""
+        return _up8(self.kv_rank + self.rot_dim)
+
+
+@dataclass(frozen=True)
+class MoESpec:
+    """Routed feed-forward: ``top`` of ``experts`` per token, chosen and weighted by ``score``; the weight scales the
+    expert's INPUT.  ``shared_ff`` > 0 adds an expert that every token uses."""
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0
+    score: str = "sigmoid"
+    activation: str = "gelu"     # exact (erf) gelu
+
+
 @dataclass
 class ModelConfig:
     arch: str = "llama"
@@ -77,6 +131,12 @@ class ModelConfig:
     query_pre_attn_scalar: Optional[float] = None
     attention_k_eq_v: bool = False
     embed_scale: bool = False
+    # designs that describe every layer on its own (None = not applicable): ``design_layers[i]`` is the layer's entry of
+    # the model's config.json ({"type", "mixer", "mlp"}), ``weight_dtype`` the width its weights are stored in
+    design_layers: Optional[List[Dict[str, Any]]] = None
+    embed_multiplier: Optional[float] = None
+    logit_scale: Optional[float] = None
+    weight_dtype: Optional[str] = None
     multimodal: Optional[Dict[str, Any]] = None
     quant: QuantConfig = field(default_factory=QuantConfig)
 
@@ -123,13 +183,46 @@ class ModelConfig:
 
     @property
     def kv_cache_bytes_per_token(self) -> int:
-        """fp16 K and V of one token in one layer (of the widest layer when layers differ)."""
+        """What one token keeps in one layer, in 16-bit elements (of the widest layer when layers differ)."""
         n, d = self.kv_pool_dims()
-        return 2 * n * d * 2
+        return self.kv_planes * n * d * 2
+
+    @property
+    def kv_planes(self) -> int:
+        """Rows a token has per layer and kv head: K and V, or one latent row that serves as both."""
+        return 1 if self.is_latent else 2
 
     @property
     def total_kv_cache_bytes_per_token(self) -> int:
         return self.kv_cache_bytes_per_token * self.num_layers
+
+    # ---- designs whose layers are listed one by one ----------------------------------------------------
+    @property
+    def is_latent(self) -> bool:
+        return self.design_layers is not None
+
+    def latent_spec(self, i: int) -> LatentSpec:
+        m = self.design_layers[i]["mixer"]
+        rot = m.get("rot") or {}
+        return LatentSpec(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]),
+                          int((m.get("mask") or {}).get("size") or 0), float(m["scale"]),
+                          int(rot.get("dims", m["rot_dim"])), float(rot.get("base", 10000.0)))
+
+    def moe_spec(self, i: int) -> Optional[MoESpec]:
+        m = self.design_layers[i].get("mlp")
+        if m is None:
+            return None
+        return MoESpec(int(m["router"]["experts"]), int(m["router"]["top"]), int(m["expert"]["ff"]),
+                       int((m.get("shared") or {}).get("ff") or 0))
+
+    @property
+    def cache_window(self) -> int:
+        """Tokens that some layer still sees: blocks that fell out of every layer's window may be given back.  0 when a
+        layer keeps everything (models that mix local and global layers apply the window inside attention)."""
+        if self.is_latent:
+            w = [self.latent_spec(i).window for i in range(self.num_layers)]
+            return max(w) if w and min(w) > 0 else 0
+        return int(self.sliding_window) if (self.sliding_window or 0) > 0 and not self.layer_types else 0
 
     # ---- per-layer attention geometry (Gemma-family models mix layer kinds) -----------------------
     @property
@@ -172,6 +265,8 @@ class ModelConfig:
         """(kv_heads, head_dim) the KV pool is allocated with; ``num_kv_heads`` = this rank's share of
         ``self.num_kv_heads`` under tensor parallelism.  Models whose layers differ get rows of the widest layer
         (``1 x max(kv_heads * head_dim)`` of the local heads); each layer lays its heads out inside that row."""
+        if self.is_latent:
+            return 1, max(self.latent_spec(i).row for i in range(self.num_layers))
         local = num_kv_heads or self.num_kv_heads
         tp = max(1, self.num_kv_heads // max(1, local))
         specs = {(s.num_kv_heads, s.head_dim) for s in (self.layer_spec(i) for i in range(self.num_layers))}
@@ -180,6 +275,15 @@ class ModelConfig:
         return 1, max(max(1, n // tp) * d for n, d in specs)
 
     def linear_param_count(self) -> int:
+        if self.is_latent:
+            n = 0
+            for i in range(self.num_layers):
+                a, m = self.latent_spec(i), self.moe_spec(i)
+                n += self.hidden_size * (a.heads * (a.qk_dim + 2 * a.vdim) + a.kv_rank + a.rot_dim)
+                n += a.heads * (a.dim + a.vdim) * a.kv_rank
+                if m is not None:
+                    n += self.hidden_size * (m.experts + 2 * m.experts * m.ff + 2 * m.shared_ff)
+            return n
         per_layer = (self.hidden_size * self.q_dim + 2 * self.hidden_size * self.kv_dim
                      + self.q_dim * self.hidden_size + 3 * self.hidden_size * self.intermediate_size)
         return per_layer * self.num_layers

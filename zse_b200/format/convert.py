@@ -55,6 +55,12 @@ def _to_f32(raw, dtype: str) -> np.ndarray:
     return arr.astype(np.float32)
 
 
+def round_bf16(v: np.ndarray) -> np.ndarray:
+    """fp32 -> bfloat16 bit patterns, nearest even (finite values)."""
+    u = np.ascontiguousarray(v, dtype=np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
 def read_safetensors_tensor(path: str, info: dict, data_base: int):
     raw, dtype, shape = read_safetensors_tensor_raw(path, info, data_base)
     return _to_f32(raw, dtype), shape
@@ -181,6 +187,8 @@ def convert_hf_to_zse(model_dir: str, output_path: str,
         hf = json.load(f)
     adapter = get_adapter(arch_override or detect_architecture(hf))
     cfg = adapter.config_from_hf(hf)
+    if adapter.STORED_DTYPE != "float16":       # served at the width of its checkpoint, never quantised
+        quant_method, quant_bits = int(QuantMethod.NONE), 16
     cfg.quant.method, cfg.quant.bits, cfg.quant.group_size = quant_method, quant_bits, group_size
     for warning in adapter.validate_config(cfg):
         if not quiet:
@@ -237,6 +245,10 @@ def convert_hf_to_zse(model_dir: str, output_path: str,
                     writer.add_weight_raw_int8(name, shape, res[0], res[1], group_size)
                 else:
                     writer.add_weight_raw(name, shape, res[0], res[1], res[2], group_size)
+            elif not floating and adapter.STORED_DTYPE != "float16":
+                writer.add_weight_raw_int32(name, shape, values.astype(np.int32))
+            elif adapter.STORED_DTYPE == "bfloat16":
+                writer.add_weight_raw_bf16(name, shape, round_bf16(values))
             else:
                 writer.add_weight_raw_fp16(name, shape, values.astype(np.float16))
             del values

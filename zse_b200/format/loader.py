@@ -26,6 +26,8 @@ from .weight_index import WeightEntry, WeightIndex
 
 
 class ZSELoader:
+    streamable = True            # the weights are one contiguous section (runtime/weight_stream.py)
+
     def __init__(self, path: str, int4_layout: Optional[str] = None, verify_crc: bool = True):
         self._path = path
         self._fd = None
@@ -149,6 +151,10 @@ class ZSELoader:
         mv = self._span(entry.data_offset, entry.data_nbytes)
         if entry.dtype == "float16":
             return np.frombuffer(mv, dtype=np.float16).reshape(entry.shape)
+        if entry.dtype == "bfloat16":        # numpy has no bfloat16: the bit patterns
+            return np.frombuffer(mv, dtype=np.uint16).reshape(entry.shape)
+        if entry.dtype == "int32":
+            return np.frombuffer(mv, dtype=np.int32).reshape(entry.shape)
         if entry.dtype == "int8":
             return np.frombuffer(mv, dtype=np.int8)
         return np.frombuffer(mv, dtype=np.uint8)
@@ -168,8 +174,10 @@ class ZSELoader:
 
     def get_weight_as_float(self, entry: WeightEntry) -> np.ndarray:
         """Dequantised fp32 tensor of shape ``entry.shape`` (verification / CPU oracle)."""
-        if entry.dtype == "float16":
+        if entry.dtype in ("float16", "int32"):
             return self.view_data(entry).astype(np.float32)
+        if entry.dtype == "bfloat16":
+            return (self.view_data(entry).astype(np.uint32) << 16).view(np.float32)
         if entry.dtype == "int4":
             flat = dequantize_int4_arrays(self.int4_rowmajor(entry), self.view_scales(entry),
                                           self.view_zeros(entry), entry.num_elements, entry.group_size)

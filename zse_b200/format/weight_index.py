@@ -20,7 +20,7 @@ _KEYS = ("name", "shape", "dtype", "quant_method", "group_size", "data_offset", 
 class WeightEntry:
     name: str
     shape: Tuple[int, ...]
-    dtype: str                       # "int4" | "int8" | "float16"
+    dtype: str                       # "int4" | "int8" | "float16" | "bfloat16" | "int32"
     quant_method: int = int(QuantMethod.NONE)
     group_size: int = 128
     data_offset: int = 0

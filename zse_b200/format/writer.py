@@ -103,6 +103,15 @@ class ZSEWriter:
         ((d, dn),) = self._append(fp16_data)
         self._weight_index.add(WeightEntry(name, tuple(shape), "float16", int(QuantMethod.NONE), 128, d, dn))
 
+    def add_weight_raw_bf16(self, name, shape, bits) -> None:
+        """``bits``: bfloat16 values as 16-bit patterns."""
+        ((d, dn),) = self._append(bits)
+        self._weight_index.add(WeightEntry(name, tuple(shape), "bfloat16", int(QuantMethod.NONE), 128, d, dn))
+
+    def add_weight_raw_int32(self, name, shape, values) -> None:
+        ((d, dn),) = self._append(values)
+        self._weight_index.add(WeightEntry(name, tuple(shape), "int32", int(QuantMethod.NONE), 128, d, dn))
+
     def add_weight_raw_int8(self, name, shape, packed_data, scales_data, group_size: int = 128) -> None:
         (d, dn), (s, sn) = self._append(packed_data, scales_data)
         self._weight_index.add(WeightEntry(name, tuple(shape), "int8", int(QuantMethod.INT8_SYM), group_size,

@@ -28,7 +28,7 @@ from ..ops import reference as ref
 from ..ops.backend import LinearWeight, TorchOps, make_ops, np_to_dev
 from ..parallel.shard_plan import ShardPlan, make_plan
 
-SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "phi3", "gemma2", "gemma4")
+SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "phi3", "gemma2", "gemma4", "ruralorn")
 
 
 def _entry_part(loader: ZSELoader, name: str, rows=None, cols=None, mirror=None) -> dict:
@@ -96,8 +96,25 @@ class StepBuffers:
 
     def __init__(self, c: ModelConfig, plan: ShardPlan, device, max_tokens: int, max_seqs: int, max_blocks: int,
                  max_planes: int, logits_rows: int, attn_splits: int):
-        f16, f32, i32, i64 = torch.float16, torch.float32, torch.int32, torch.int64
+        f16, f32 = torch.float16, torch.float32
         H = c.hidden_size
+        z = lambda *s, dt: torch.zeros(*s, dtype=dt, device=device)
+        self._common(device, H, plan.vocab_size, max_tokens, max_seqs, max_blocks, logits_rows, attn_splits)
+        self.qkv = z(max_tokens, plan.q_dim + 2 * plan.kv_dim, dt=f16)
+        self.attn_out = z(max_tokens, plan.q_dim, dt=f16)
+        # decode-sized passes take QKV as fp32 split-K planes (summed, biased and rotated by the RoPE kernel)
+        self.qkv_plane_rows = min(max_tokens, 256)
+        self.qkv_planes = z(8, self.qkv_plane_rows, plan.q_dim + 2 * plan.kv_dim, dt=f32)
+        self.act = z(max_tokens, plan.inter_size, dt=f16)
+        self.partials = z(max_planes, max_tokens, H, dt=f32)
+        self.attn_scratch = z(max(1, max_seqs * plan.num_heads * attn_splits * (c.head_dim + 2)), dt=f32)
+        self.lora_tmp = z(max_tokens, 64, dt=f32)
+
+    def _common(self, device, H: int, vocab: int, max_tokens: int, max_seqs: int, max_blocks: int, logits_rows: int,
+                attn_splits: int, act=torch.float16, logits=torch.float16) -> None:
+        """What the runner stages and reads, whatever the layers look like.  ``act`` / ``logits``: the model's activation
+        and logits types."""
+        f32, i32, i64 = torch.float32, torch.int32, torch.int64
         z = lambda *s, dt: torch.zeros(*s, dtype=dt, device=device)
         self.max_tokens, self.max_seqs, self.max_blocks = max_tokens, max_seqs, max_blocks
         self.ids = z(max_tokens, dt=i32)
@@ -109,19 +126,11 @@ class StepBuffers:
         self.q_pos0 = z(max_seqs, dt=i32)
         self.logit_rows = z(logits_rows, dt=i64)
         self.residual = z(max_tokens, H, dt=f32)
-        self.xnorm = z(max_tokens, H, dt=f16)
-        self.qkv = z(max_tokens, plan.q_dim + 2 * plan.kv_dim, dt=f16)
-        self.attn_out = z(max_tokens, plan.q_dim, dt=f16)
-        # decode-sized passes take QKV as fp32 split-K planes (summed, biased and rotated by the RoPE kernel)
-        self.qkv_plane_rows = min(max_tokens, 256)
-        self.qkv_planes = z(8, self.qkv_plane_rows, plan.q_dim + 2 * plan.kv_dim, dt=f32)
-        self.act = z(max_tokens, plan.inter_size, dt=f16)
-        self.partials = z(max_planes, max_tokens, H, dt=f32)
-        self.xsel = z(logits_rows, H, dt=f16)
-        self.logits = z(logits_rows, plan.vocab_size, dt=f16)
+        self.xnorm = z(max_tokens, H, dt=act)
+        self.xsel = z(logits_rows, H, dt=act)
+        self.logits = z(logits_rows, vocab, dt=logits)
         self.out_tokens = z(logits_rows, dt=i32)
         self.attn_splits = attn_splits
-        self.attn_scratch = z(max(1, max_seqs * plan.num_heads * attn_splits * (c.head_dim + 2)), dt=f32)
         # sampling parameters per logits row
         self.temperature = torch.ones(logits_rows, dtype=f32, device=device)
         self.top_k = z(logits_rows, dt=i32)
@@ -129,13 +138,15 @@ class StepBuffers:
         self.seeds = z(logits_rows, dt=i64)
         # LoRA routing
         self.adapter_ids = torch.full((max_tokens,), -1, dtype=i32, device=device)
-        self.lora_tmp = z(max_tokens, 64, dt=f32)
 
     def nbytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in vars(self).values() if isinstance(t, torch.Tensor))
 
 
 class DecoderModel:
+    act_dtype = torch.float16       # activations, and the rows of the KV cache
+    mixed_passes = False            # prompt chunks and decoding sequences may share one packed pass
+
     def __init__(self, config: ModelConfig, plan: ShardPlan, ops: TorchOps):
         self.config, self.plan, self.ops = config, plan, ops
         self.device = ops.device
@@ -157,7 +168,8 @@ class DecoderModel:
     # ---- loading --------------------------------------------------------------------------------------
     @classmethod
     def from_loader(cls, loader: ZSELoader, device="cpu", tp_size: int = 1, rank: int = 0, ops=None,
-                    progress=None) -> "DecoderModel":
+                    progress=None, dtype: Optional[str] = None) -> "DecoderModel":
+        """``dtype``: "bfloat16" or "float32" for the models that offer both; None = what the model is served in."""
         c = loader.config
         if c.arch not in SUPPORTED_ARCHS:
             raise NotImplementedError(f"architecture '{c.arch}' has a converter but no runtime here yet "
@@ -166,9 +178,17 @@ class DecoderModel:
         if c.is_gemma and cls is DecoderModel:
             from .gemma import GemmaDecoderModel
             cls = GemmaDecoderModel
+        elif c.is_latent and cls is DecoderModel:
+            from .latent_moe import LatentMoEModel
+            cls = LatentMoEModel
         m = cls(c, plan, ops or make_ops(device))
+        m.set_dtype(dtype)
         m._load(loader, progress)
         return m
+
+    def set_dtype(self, dtype: Optional[str]) -> None:
+        if dtype not in (None, "float16"):
+            raise ValueError(f"'{self.config.arch}' runs in float16, not {dtype}")
 
     def _load(self, loader: ZSELoader, progress=None) -> None:
         c, p, ops, dev = self.config, self.plan, self.ops, self.device
@@ -266,6 +286,22 @@ class DecoderModel:
                      and L.down.bias is None and L.gate_up.swiglu for L in self.layers) and not self.config.is_gemma
             self._sp_ok_cache = ok
         return ok
+
+    # ---- what the runner asks about a packed pass --------------------------------------------------------
+    def pass_order(self, items) -> Optional[List[int]]:
+        """Order in which a pass lays out its sequences (None: as given)."""
+        return None
+
+    def stage_prefill(self, b: StepBuffers, spans) -> None:
+        """Called while a packed pass is staged; ``spans[s] = (start, tokens)`` in the pass's order."""
+
+    def attention_span(self, max_len: int) -> int:
+        """Cached tokens a decoding sequence of ``max_len`` tokens attends to."""
+        return max_len
+
+    def attention_ctas(self) -> int:
+        """CTAs one decoding sequence brings to the attention kernel before its keys are split."""
+        return self.plan.num_kv_heads
 
     # ---- forward --------------------------------------------------------------------------------------
     def _add_norm(self, b: StepBuffers, planes: int, weight: torch.Tensor, M: int, add=None) -> None:

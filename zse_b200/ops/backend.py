@@ -67,7 +67,10 @@ class TorchOps:
 
     # ---- ops ------------------------------------------------------------------------------------------
     def linear(self, w: LinearWeight, x, M, out, x_cap=None, gather=None):
-        out[:M, : w.N] = ref.linear(x[:M], w.data, w.bias)
+        if out.dtype != torch.float16:
+            out[:M, : w.N] = x[:M].float() @ w.data.T
+        else:
+            out[:M, : w.N] = ref.linear(x[:M], w.data, w.bias)
 
     def linear_swiglu(self, w: LinearWeight, x, M, out, x_cap=None, gelu=False, gather=None):
         y = x[:M].float() @ w.data.T
@@ -119,6 +122,99 @@ class TorchOps:
         out[:total_q, : nh * hd] = ref.attn_prefill(qkv[:total_q, : nh * hd], kv_layer, block_tables[:num_seqs],
                                                     cu_q[: num_seqs + 1], q_pos0[:num_seqs], nh, nkv, hd, block_size,
                                                     scale, softcap, window)
+
+    # ---- latent attention and routed feed-forward -----------------------------------------------------
+    # (activations and cache at the model's own width: bfloat16 or fp32)
+    def dense(self, t: torch.Tensor, dtype) -> torch.Tensor:
+        """Weights of the ops below, as this back end keeps them."""
+        return t.to(self.device, torch.float32)
+
+    def dense_linear(self, w: torch.Tensor) -> LinearWeight:
+        """``w`` [N, K] as ``dense`` returned it."""
+        kind = {torch.bfloat16: "bf16", torch.float32: "f32"}[w.dtype] if self.name == "cuda" else "ref"
+        return LinearWeight(kind, w.shape[0], w.shape[1], w, None, False, w.numel() * w.element_size())
+
+    def linear_f32(self, w: LinearWeight, x, M, out):
+        """out [M, N] fp32, one plane."""
+        out[:M, : w.N] = x[:M].float() @ w.data.T
+
+    def add_norm(self, residual, partials, n_partials, slots, weight, out, M, eps):
+        """residual += the planes' sum + the sum over a row's ``slots`` [M, n, H]; out = RMSNorm(residual) * weight."""
+        H = residual.shape[1]
+        if n_partials:
+            residual[:M] += partials.view(-1)[: n_partials * M * H].view(n_partials, M, H).sum(0)
+        if slots is not None:
+            residual[:M] += slots[:M].float().sum(1)
+        out[:M] = ref.rmsnorm_f32(residual[:M], weight, eps)
+
+    def latent_prep(self, inp, planes, n_planes, rows, positions, slots, freqs, norm_w, spec, eps, M):
+        if n_planes:
+            ld = inp.shape[1]
+            inp[:M] = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
+        ref.latent_prep(inp[:M], rows, positions[:M], slots[:M], freqs, norm_w, spec, eps)
+
+    def latent_attn(self, inp, L, rows, block_tables, row_seq, positions, q_lat, o_lat, out, M, spec, scratch, num_splits):
+        """Rows [0, M) attend to the cached rows themselves: queries go through W_uk, results through W_uv and the gate.
+        Row t belongs to sequence ``row_seq[t]`` (None: t)."""
+        H, vd = spec.heads, spec.vdim
+        q = ref.latent_absorb(inp[:M], L.uk, spec).to(inp.dtype)
+        o = torch.zeros(M, H, spec.kv_rank, dtype=inp.dtype, device=inp.device)
+        for t in range(M):
+            s = t if row_seq is None else int(row_seq[t])
+            o[t] = ref.latent_attn_token(q[t], rows, block_tables[s], int(positions[t]), spec)
+        y = torch.einsum("thc,hvc->thv", o.float(), L.uv.view(H, vd, spec.kv_rank)).reshape(M, H * vd)
+        self._gate(y, inp[:M], out[:M], spec)
+
+    def latent_attn_chunks(self, inp, L, rows, block_tables, cu_q, q_pos0, ctx_off, group, ctx, out, spec):
+        """Rows of the sequences ``group.first .. group.last - 1`` attend to keys and values expanded from the cached rows
+        their windows reach; ``ctx``: scratch (c, kr, kvx), ``ctx_off[s]``: sequence s's first row in it."""
+        bs = rows.shape[1]
+        kr, r = spec.kv_rank, spec.rot_dim
+        for s in range(group.first, group.last):
+            a, e, p0 = int(cu_q[s]), int(cu_q[s + 1]), int(q_pos0[s])
+            lo = max(0, p0 + 1 - spec.window) if spec.window > 0 else 0
+            pos = torch.arange(lo, p0 + e - a, device=rows.device)
+            blk = block_tables[s][pos // bs].long()
+            got = rows[blk.clamp_min(0), pos % bs]
+            c = got[:, :kr].contiguous()
+            kvx = (c.float() @ L.ukv.data.T).to(inp.dtype)
+            y = ref.latent_attn_chunk(inp[a:e], c, got[:, kr: kr + r], blk >= 0, kvx,
+                                      torch.arange(p0, p0 + e - a, device=rows.device), pos, spec)
+            self._gate(y.reshape(e - a, -1), inp[a:e], out[a:e], spec)
+
+    @staticmethod
+    def _gate(y, inp, out, spec):
+        w = spec.heads * spec.vdim
+        if spec.gated:
+            y = y * torch.sigmoid(inp[:, spec.gate_col: spec.gate_col + w].float())
+        out[:, :w] = y
+
+    def moe(self, L, x, M, ws):
+        """The routed feed-forward of rows [0, M): returns ``slots`` [M, top (+1), H], to be summed."""
+        m, H = L.moe, x.shape[1]
+        xs = x[:M].float()
+        ids, w = ref.route_top(xs @ L.router.data.T, m.top)
+        slots = torch.zeros(M, m.top + (m.shared_ff > 0), H, dtype=torch.float32, device=x.device)
+        up, down = L.up.view(m.experts, m.ff, H), L.down.view(m.experts, H, m.ff)
+        for e in torch.unique(ids).tolist():
+            t, k = torch.where(ids == e)
+            act = ref.gelu_exact(w[t, k, None] * (xs[t] @ up[e].T)).to(x.dtype)
+            slots[t, k] = act.float() @ down[e].T
+        if m.shared_ff:
+            slots[:, m.top] = ref.gelu_exact(xs @ L.shared_up.T).to(x.dtype).float() @ L.shared_down.T
+        return slots
+
+    def latent_expands(self, spec, dtype) -> bool:
+        """Whether long chunks of such a layer take ``latent_attn_chunks``."""
+        return True
+
+    def moe_workspace(self, specs, H: int, max_tokens: int, dtype):
+        return None
+
+    def logits_finish(self, logits, M, scale, cap):
+        """logits <- cap * tanh(scale * logits / cap) in place (cap 0: only scaled)."""
+        z = logits[:M] * scale
+        logits[:M] = cap * torch.tanh(z / cap) if cap > 0 else z
 
     # ---- Gemma-family ops ---------------------------------------------------------------------------
     def headnorm_rope_kv_write(self, qkv, kv_layer, positions, slots, freqs, q_norm_w, k_norm_w, norm_v, k_is_v, eps,
@@ -183,6 +279,35 @@ def _dense_f32(p: dict, group_size: int, device) -> torch.Tensor:
                             _np_to_dev(p["zeros"], device), shape, group_size)
 
 
+def _dp(t: Optional[torch.Tensor]) -> Optional[int]:
+    return None if t is None else t.data_ptr()
+
+
+class MoeWorkspace:
+    """Device tables and activations of the routed feed-forward, shared by all layers of a model."""
+    F32_ROWS = 1024
+
+    def __init__(self, specs, H: int, max_tokens: int, dtype, device):
+        z = lambda n, dt: torch.zeros(max(1, n), dtype=dt, device=device)
+        i32, f32 = torch.int32, torch.float32
+        E, top = max(s.experts for s in specs), max(s.top for s in specs)
+        slots = max_tokens * top
+        per = max(s.top + (s.shared_ff > 0) for s in specs)
+        self.counts, self.first_row, self.n_tiles = z(E, i32), z(E, i32), z(1, i32)
+        self.slot_expert, self.slot_rank, self.slot_score = z(slots, i32), z(slots, i32), z(slots, f32)
+        self.row_score, self.out_rows = z(slots, f32), z(slots, i32)
+        self.tiles = z((E + slots // 16 + 1) * 4, i32)
+        self.xs = z(slots * H, dtype)
+        self.act = z(max_tokens * max(s.top * s.ff for s in specs), dtype)
+        self.act_shared = z(max_tokens * max(s.shared_ff for s in specs), dtype)
+        self.y = z(max(min(max_tokens, self.F32_ROWS) * 4, max_tokens * dtype.itemsize) * per * H, torch.uint8)
+        # router logits: split-K planes of decode-sized passes, one plane otherwise
+        rows = min(max_tokens, 256)
+        self.router = z(max(8 * rows, max_tokens) * E, f32)
+        self.plane_rows = rows
+        self.router_views = {s.experts: self.router[: 8 * rows * s.experts].view(8, rows * s.experts) for s in specs}
+
+
 class CudaOps(TorchOps):
     name = "cuda"
 
@@ -204,6 +329,8 @@ class CudaOps(TorchOps):
         self.int8_resident = env.flag("ZSE_W8_RESIDENT")
         self._w8_scratch = None
         self._norm_ctx = None
+        self._logits16 = None
+        self._no_tables = torch.zeros(1, 1, dtype=torch.int32, device=self.device)
         self.attn_prefill_tc = env.flag("ZSE_ATTN_PREFILL_TC")
 
     def _w8_dense(self, w: "LinearWeight") -> torch.Tensor:
@@ -315,6 +442,8 @@ class CudaOps(TorchOps):
                                self.status.ptr)
         elif w.kind == "w4t":
             self.n.gemm_w4(w.data, x, cap, w.bias, out, M, w.N, w.K, out.stride(0), EPI_F16, 0, self.status.ptr)
+        elif w.kind in ("bf16", "f32"):
+            self._typed_linear(w, x, M, out, out.stride(0), EPI_F16, 1, cap)
         else:
             self.n.gemm_f16(w.data, w.N, x, cap, w.bias, out, M, w.N, w.K, out.stride(0), EPI_F16, 1, self.status.ptr)
 
@@ -380,12 +509,126 @@ class CudaOps(TorchOps):
             return planes
         ks = self.pick_k_split(w, M) if k_split is None else k_split
         ks = min(ks, partials.shape[0])
+        if w.kind in ("bf16", "f32"):
+            return self._typed_linear(w, x, M, partials, w.N, EPI_PARTIAL, ks, cap)
         planes = self.n.gemm_f16_splits(M, w.N, w.K, ks)
         self.n.gemm_f16(w.data, w.N, x, cap, None, partials, M, w.N, w.K, partials.stride(1), EPI_PARTIAL, ks,
                         self.status.ptr)
         return planes
 
+    # ---- bfloat16 / float layers ------------------------------------------------------------------------
+    def _typed_linear(self, w, x, M, out, ldo, epilogue, k_split, cap) -> int:
+        """Store (EPI_F16: in the activations' type) or fp32 planes; returns how many planes.  The tensor-core kernel
+        takes bfloat16 rows of whole 16-byte pieces, everything else the general kernel (one plane)."""
+        if w.kind == "bf16" and w.K % 8 == 0:
+            planes = self.n.gemm_f16_splits(M, w.N, w.K, k_split) if epilogue == EPI_PARTIAL else 1
+            self.n.gemm_bf16(w.data, w.N, x, cap, out, M, w.N, w.K, ldo, epilogue, k_split, self.status.ptr)
+            return planes
+        self.n.gemm_tile(w.data.dtype, x, x.stride(0), w.data, (w.K, 1), out, ldo, M, w.N, w.K,
+                         self.n.TILE_STORE if epilogue == EPI_F16 else self.n.TILE_F32)
+        return 1
+
+    def dense(self, t: torch.Tensor, dtype) -> torch.Tensor:
+        return t.to(self.device, dtype)
+
+    def linear_f32(self, w, x, M, out):
+        self._typed_linear(w, x, M, out, out.stride(0), EPI_PARTIAL, 1, x.shape[0])
+
+    def add_norm(self, residual, partials, n_partials, slots, weight, out, M, eps):
+        self.n.add_norm(residual, partials, n_partials, slots, 0 if slots is None else slots.shape[1], weight, out, M,
+                        residual.shape[1], float(eps))
+
+    def logits_finish(self, logits, M, scale, cap):
+        self.n.logits_finish(logits, M, scale, cap)
+
+    def latent_expands(self, spec, dtype) -> bool:
+        return dtype == torch.bfloat16 and self.n.latent_mma_ok(spec)
+
+    def latent_prep(self, inp, planes, n_planes, rows, positions, slots, freqs, norm_w, spec, eps, M):
+        rc = self.n.row_cache(rows, self._no_tables)
+        self.n.latent_prep(inp, planes, n_planes, M, rc, positions, slots, freqs, norm_w, spec, eps)
+
+    @staticmethod
+    def _gate_ptr(inp, spec):
+        return inp.data_ptr() + spec.gate_col * inp.element_size() if spec.gated else None
+
+    def latent_attn(self, inp, L, rows, block_tables, row_seq, positions, q_lat, o_lat, out, M, spec, scratch, num_splits):
+        n, H, d, r, kr, vd = self.n, spec.heads, spec.dim, spec.rot_dim, spec.kv_rank, spec.vdim
+        rc = n.row_cache(rows, block_tables)
+        if self.latent_expands(spec, inp.dtype):
+            if num_splits > 1 and scratch.numel() < M * num_splits * H * (kr + 2):
+                num_splits = 1
+            n.latent_absorb(inp, L.uk, q_lat, M, spec)
+            n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, True)
+            n.latent_unabsorb(o_lat, L.uv, self._gate_ptr(inp, spec), inp.stride(0), out, M, spec)
+            return
+        ql = q_lat[: M * H * spec.row].view(M, H, spec.row)
+        n.gemm_tile(inp.dtype, inp, inp.stride(0), L.uk, (1, kr), ql, H * spec.row, M, kr, d, batch=H, a_batch=d + r,
+                    b_batch=d * kr, o_batch=spec.row)
+        ql[:, :, kr: kr + r].copy_(inp[:M, : H * (d + r)].view(M, H, d + r)[:, :, d:])
+        n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, 1, False)
+        gate = inp[:, spec.gate_col:] if spec.gated else None
+        n.gemm_tile(inp.dtype, o_lat, H * kr, L.uv, (kr, 1), out, out.stride(0), M, vd, kr,
+                    n.TILE_GATE if spec.gated else n.TILE_STORE, batch=H, a_batch=kr, b_batch=vd * kr, o_batch=vd,
+                    gate=gate, ldg=inp.stride(0), gate_batch=vd)
+
+    def latent_attn_chunks(self, inp, L, rows, block_tables, cu_q, q_pos0, ctx_off, group, ctx, out, spec):
+        n = self.n
+        c, kr, kvx = ctx
+        rc = n.row_cache(rows, block_tables)
+        ch = n.Chunks(cu_q.data_ptr(), q_pos0.data_ptr(), ctx_off.data_ptr(), group.first, group.last, spec.window)
+        n.latent_gather(rc, ch, group.rows, spec, c, kr)
+        cap = c.numel() // spec.kv_rank
+        n.gemm_bf16(L.ukv.data, L.ukv.N, c, cap, kvx, group.rows, L.ukv.N, L.ukv.K, L.ukv.N, EPI_F16, 1, self.status.ptr)
+        v_col = (spec.heads * spec.dim + 7) // 8 * 8
+        n.latent_chunk(inp, kvx, L.ukv.N, v_col, kr, rc, ch, group.max_q, out, self._gate_ptr(inp, spec), spec)
+
+    def moe_workspace(self, specs, H: int, max_tokens: int, dtype):
+        return MoeWorkspace(specs, H, max_tokens, dtype, self.device) if specs else None
+
+    def moe(self, L, x, M, ws):
+        n, m, H = self.n, L.moe, x.shape[1]
+        dt = x.dtype
+        per = m.top + (m.shared_ff > 0)
+        planes = self.linear_partial(L.router, x, M, ws.router_views[m.experts],
+                                     None if M <= ws.plane_rows else 1)
+        slots = M * m.top
+        # result rows in fp32 while they are few, in the activations' type for long passes
+        y_dt = torch.float32 if M <= ws.F32_ROWS else dt
+        y = ws.y[: M * per * H * y_dt.itemsize].view(y_dt).view(M, per, H)
+        if dt == torch.bfloat16 and H % 8 == 0 and m.ff % 8 == 0 and m.shared_ff % 8 == 0:
+            tile = n.moe_tile_rows(M, m.experts, m.top)
+            max_tiles = min(slots, m.experts + slots // tile)
+            n.moe_route(ws.router, planes, M, m.experts, m.top, tile, x, H, per, ws)
+            g = n.MoeGemm(L.up.data_ptr(), ws.xs.data_ptr(), ws.act.data_ptr(), _dp(L.shared_up), x.data_ptr(),
+                          ws.act_shared.data_ptr(), ws.row_score.data_ptr(), None, ws.tiles.data_ptr(),
+                          ws.n_tiles.data_ptr(), m.ff, H, m.ff, m.shared_ff, H, m.shared_ff, 1, 0, x.shape[0])
+            n.moe_gemm(g, M, m.experts, ws.xs.numel() // H, tile, max_tiles, 0, self.status.ptr)
+            g = n.MoeGemm(L.down.data_ptr(), ws.act.data_ptr(), y.data_ptr(), _dp(L.shared_down),
+                          ws.act_shared.data_ptr(), y.data_ptr(), None, ws.out_rows.data_ptr(), ws.tiles.data_ptr(),
+                          ws.n_tiles.data_ptr(), H, m.ff, H, H if m.shared_ff else 0, m.shared_ff, H, per, m.top,
+                          ws.act_shared.numel() // max(1, m.shared_ff))
+            n.moe_gemm(g, M, m.experts, ws.act.numel() // m.ff, tile, max_tiles, 2 if y_dt == torch.float32 else 1,
+                       self.status.ptr)
+            return y
+        max_tiles = min(slots, m.experts + slots // 64)
+        n.moe_route(ws.router, planes, M, m.experts, m.top, 64, x, H, per, ws)
+        store = n.TILE_F32 if y_dt == torch.float32 else n.TILE_STORE
+        group = dict(tiles=ws.tiles, n_tiles=ws.n_tiles, max_tiles=max_tiles)
+        n.gemm_tile(dt, ws.xs, H, L.up, (H, 1), ws.act, m.ff, slots, m.ff, H, n.TILE_GELU, row_scale=ws.row_score,
+                    b_group=m.ff * H, **group)
+        n.gemm_tile(dt, ws.act, m.ff, L.down, (m.ff, 1), y, H, slots, H, m.ff, store, out_rows=ws.out_rows,
+                    b_group=m.ff * H, **group)
+        if m.shared_ff:
+            n.gemm_tile(dt, x, H, L.shared_up, (H, 1), ws.act_shared, m.shared_ff, M, m.shared_ff, H, n.TILE_GELU)
+            n.gemm_tile(dt, ws.act_shared, m.shared_ff, L.shared_down, (m.shared_ff, 1), y, H, M, H, m.shared_ff, store,
+                        out_row=(per, m.top))
+        return y
+
     def embedding(self, table, ids, out, M, scale=1.0):
+        if table.dtype != torch.float16:
+            self.n.embedding_typed(table, ids, out, M, table.shape[1], table.shape[0], float(scale), self.status.ptr)
+            return
         self.n.embedding(table, ids, out, M, table.shape[1], table.shape[0], float(scale), self.status.ptr)
 
     def add_rmsnorm(self, residual, partials, n_partials, add_f16, weight, out, M, eps):
@@ -458,12 +701,29 @@ class CudaOps(TorchOps):
         self.n.softcap(logits, M, logits.shape[1], cap)
 
     def argmax(self, logits, out, M):
+        if logits.dtype == torch.float32:
+            self.n.argmax_f32(logits, logits.stride(0), out, M, logits.shape[1])
+            return
         self.n.argmax(logits, logits.stride(0), out, M, logits.shape[1])
 
+    def _half_logits(self, logits, M):
+        """fp16 copy of fp32 logits for the sampling kernel, whose cut-offs work on 16-bit keys."""
+        h = self._logits16
+        if h is None or h.shape[0] < logits.shape[0] or h.shape[1] != logits.shape[1]:
+            h = self._logits16 = torch.empty(logits.shape, dtype=torch.float16, device=self.device)
+        h[:M].copy_(logits[:M])
+        return h
+
     def sample(self, logits, out, M, temperature, top_k, top_p, seeds, step):
+        if logits.dtype == torch.float32:
+            logits = self._half_logits(logits, M)
         self.n.sample(logits, logits.stride(0), out, M, logits.shape[1], temperature, top_k, top_p, seeds, int(step))
 
     def apply_repetition_penalty(self, logits, rows, tokens, counts, n, penalty):
+        if logits.dtype == torch.float32:
+            self.n.apply_repetition_penalty_f32(logits, logits.stride(0), rows, tokens, counts, n, penalty,
+                                                logits.shape[1])
+            return
         self.n.apply_repetition_penalty(logits, logits.stride(0), rows, tokens, counts, n, penalty, logits.shape[1])
 
     def lora_apply(self, x, a_table, b_table, ids, scales, y, M, K, N, rank, tmp=None, y_col0=0):

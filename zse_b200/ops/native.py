@@ -8,7 +8,7 @@ from __future__ import annotations
 
 import ctypes
 import os
-from ctypes import c_char_p, c_float, c_int, c_int64, c_uint64, c_void_p, POINTER, c_uint32
+from ctypes import c_char_p, c_float, c_int, c_int32, c_int64, c_uint64, c_void_p, POINTER, Structure, byref, c_uint32
 from typing import Optional
 
 import torch
@@ -25,6 +25,33 @@ class NativeError(RuntimeError):
 
 class DeviceStatusError(RuntimeError):
     """A kernel reported a failure through the status word (bounded wait ran out, bad index, ...)."""
+
+
+# mirrors of the structs in csrc/api.h
+class TileGemm(Structure):
+    _fields_ = [("a", c_void_p), ("lda", c_int64), ("a_batch", c_int64), ("b", c_void_p), ("ldb_n", c_int64),
+                ("ldb_k", c_int64), ("b_batch", c_int64), ("b_group", c_int64), ("out", c_void_p), ("ldo", c_int64),
+                ("o_batch", c_int64), ("M", c_int32), ("N", c_int32), ("K", c_int32), ("epilogue", c_int32),
+                ("row_scale", c_void_p), ("out_rows", c_void_p), ("out_row_mul", c_int32), ("out_row_add", c_int32),
+                ("gate", c_void_p), ("ldg", c_int64), ("gate_batch", c_int64), ("tiles", c_void_p),
+                ("n_tiles", c_void_p)]
+
+
+class RowCache(Structure):
+    _fields_ = [("rows", c_void_p), ("block_stride", c_int64), ("block_size", c_int32), ("row", c_int32),
+                ("tables", c_void_p), ("max_blocks", c_int32)]
+
+
+class Chunks(Structure):
+    _fields_ = [("cu_q", c_void_p), ("q_pos0", c_void_p), ("ctx_off", c_void_p), ("first", c_int32), ("last", c_int32),
+                ("window", c_int32)]
+
+
+class MoeGemm(Structure):
+    _fields_ = [(n, c_void_p) for n in ("routed_w", "routed_x", "routed_out", "shared_w", "shared_x", "shared_out",
+                                        "row_score", "out_rows", "tiles", "n_tiles")] + \
+               [(n, c_int32) for n in ("routed_n", "routed_k", "routed_ldo", "shared_n", "shared_k", "shared_ldo",
+                                       "shared_mul", "shared_add", "shared_x_rows")]
 
 
 _lib: Optional[ctypes.CDLL] = None
@@ -91,6 +118,8 @@ _SIGS = {
                            c_void_p]),
     "zse_apply_repetition_penalty": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                              c_void_p]),
+    "zse_apply_repetition_penalty_f32": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                                                 c_void_p]),
     "zse_lora_shrink": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
     "zse_attn_prefill_tc": (c_int, [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                     c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p]),
@@ -132,6 +161,27 @@ _SIGS = {
     "zse_tp_sum_add_rmsnorm_emulated": (c_int, [c_void_p, POINTER(c_uint64), c_void_p, POINTER(c_uint64), c_int,
                                                 c_float, c_int, c_int, c_void_p, c_void_p]),
     "zse_tp_ctx_set_gather": (c_int, [c_void_p, c_int, c_int, POINTER(c_uint64), POINTER(c_uint64)]),
+    "zse_gemm_bf16": (c_int, [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                              c_void_p, c_void_p]),
+    "zse_gemm_tile": (c_int, [c_int, POINTER(TileGemm), c_int, c_int, c_void_p]),
+    "zse_embedding_typed": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p]),
+    "zse_add_norm": (c_int, [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                             c_float, c_void_p]),
+    "zse_logits_finish": (c_int, [c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p]),
+    "zse_argmax_f32": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p]),
+    "zse_latent_mma_ok": (c_int, [c_int] * 6),
+    "zse_latent_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_int, POINTER(RowCache), c_void_p, c_void_p,
+                                c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_void_p]),
+    "zse_latent_attn": (c_int, [c_int, c_void_p, POINTER(RowCache), c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                c_int, c_int, c_int, c_float, c_int, c_int, c_void_p]),
+    "zse_latent_absorb": (c_int, [c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 6 + [c_void_p]),
+    "zse_latent_unabsorb": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p] + [c_int] * 5 + [c_void_p]),
+    "zse_latent_gather": (c_int, [POINTER(RowCache), POINTER(Chunks), c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
+    "zse_latent_chunk": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, POINTER(RowCache), POINTER(Chunks),
+                                 c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]),
+    "zse_moe_tile_rows": (c_int, [c_int, c_int, c_int]),
+    "zse_moe_route": (c_int, [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int] + [c_void_p] * 11),
+    "zse_moe_gemm": (c_int, [POINTER(MoeGemm), c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
     "zse_read_probe": (c_int, [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p]),
     "zse_tp_gather_rows": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]),
     "zse_tp_gather_rows_emulated": (c_int, [c_void_p, POINTER(c_uint64), c_int, c_int, c_int, c_void_p, c_void_p]),
@@ -422,6 +472,11 @@ def apply_repetition_penalty(logits, ld, rows, tokens, counts, n, penalty, V):
                                             _stream()), "repetition_penalty")
 
 
+def apply_repetition_penalty_f32(logits, ld, rows, tokens, counts, n, penalty, V):
+    _ck(load().zse_apply_repetition_penalty_f32(_p(logits), ld, _p(rows), _p(tokens), _p(counts), n, _p(penalty), V,
+                                                _stream()), "repetition_penalty")
+
+
 def lora_shrink(x, ldx, a, ids, tmp, M, K, rank):
     _ck(load().zse_lora_shrink(_p(x), ldx, _p(a), _p(ids), _p(tmp), M, K, rank, _stream()), "lora_shrink")
 
@@ -433,6 +488,108 @@ def lora_apply(x, ldx, a, b, ids, scales, y, ldy, M, K, N, rank):
 
 def lora_expand(tmp, b, ids, scales, y, ldy, M, N, rank):
     _ck(load().zse_lora_expand(_p(tmp), _p(b), _p(ids), _p(scales), _p(y), ldy, M, N, rank, _stream()), "lora_expand")
+
+
+# ---- bfloat16 / float activations (gemm.cu, gemm_tile.cu, rows.cu, latent.cu, moe.cu) -------------------------------
+_DTYPE = {torch.bfloat16: 1, torch.float32: 2}
+
+
+def gemm_bf16(w, w_rows, x, x_rows_cap, out, M, N, K, ldo, epilogue, k_split, status):
+    _ck(load().zse_gemm_bf16(_p(w), w_rows, _p(x), x_rows_cap, _p(out), M, N, K, ldo, epilogue, k_split, status,
+                             _stream()), "gemm_bf16")
+
+
+TILE_STORE, TILE_F32, TILE_GELU, TILE_GATE = 0, 1, 2, 3
+
+
+def gemm_tile(dtype, a, lda, b, ldb, out, ldo, M, N, K, epilogue=TILE_STORE, batch=1, a_batch=0, b_batch=0, o_batch=0,
+              row_scale=None, out_rows=None, out_row=(1, 0), gate=None, ldg=0, gate_batch=0, tiles=None, n_tiles=None,
+              max_tiles=0, b_group=0):
+    """``ldb``: (stride of n, stride of k) of the second operand; ``out_row``: (mul, add) of the output row."""
+    g = TileGemm(_p(a), lda, a_batch, _p(b), ldb[0], ldb[1], b_batch, b_group, _p(out), ldo, o_batch, M, N, K, epilogue,
+                 _p(row_scale), _p(out_rows), out_row[0], out_row[1], _p(gate), ldg, gate_batch, _p(tiles), _p(n_tiles))
+    _ck(load().zse_gemm_tile(_DTYPE[dtype], byref(g), batch, max_tiles, _stream()), "gemm_tile")
+
+
+def embedding_typed(table, ids, out, M, H, vocab, scale, status):
+    _ck(load().zse_embedding_typed(_DTYPE[table.dtype], _p(table), _p(ids), _p(out), M, H, vocab, scale, status,
+                                   _stream()), "embedding_typed")
+
+
+def add_norm(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps):
+    sd = 0 if slots is None else _DTYPE[slots.dtype]
+    _ck(load().zse_add_norm(_DTYPE[out.dtype], sd, _p(residual), _p(planes), n_planes, _p(slots), n_slots, _p(weight),
+                            _p(out), M, H, eps, _stream()), "add_norm")
+
+
+def logits_finish(logits, M, scale, cap):
+    _ck(load().zse_logits_finish(_p(logits), logits.stride(0), M, logits.shape[1], float(scale), float(cap), _stream()),
+        "logits_finish")
+
+
+def argmax_f32(logits, ld, out, M, V):
+    _ck(load().zse_argmax_f32(_p(logits), ld, _p(out), M, V, _stream()), "argmax_f32")
+
+
+def row_cache(rows, block_tables) -> RowCache:
+    """``rows``: a layer's cached rows [blocks, block_size, row] (blocks may be strided)."""
+    return RowCache(rows.data_ptr(), rows.stride(0), rows.shape[1], rows.shape[2], block_tables.data_ptr(),
+                    block_tables.stride(0))
+
+
+def latent_mma_ok(spec) -> bool:
+    return bool(load().zse_latent_mma_ok(spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank, spec.row))
+
+
+def latent_prep(inp, planes, n_planes, M, rc, positions, slots, freqs, norm_w, spec, eps):
+    gate_w = spec.heads * spec.vdim if spec.gated else 0
+    _ck(load().zse_latent_prep(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, M, byref(rc),
+                               _p(positions), _p(slots), _p(freqs), _p(norm_w), spec.heads, spec.dim, spec.rot_dim,
+                               spec.rot_dims, spec.kv_rank, spec.latent_col, spec.gate_col, gate_w, float(eps),
+                               _stream()), "latent_prep")
+
+
+def latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, tensor_cores):
+    _ck(load().zse_latent_attn(_DTYPE[q_lat.dtype], _p(q_lat), byref(rc), _p(row_seq), _p(positions), _p(o_lat),
+                               _p(scratch), M, spec.heads, spec.kv_rank + spec.rot_dim, spec.kv_rank, spec.window,
+                               float(spec.scale), num_splits, int(tensor_cores), _stream()), "latent_attn",
+        2 if num_splits > 1 else 1)
+
+
+def latent_absorb(inp, uk, q_lat, M, spec):
+    _ck(load().zse_latent_absorb(_p(inp), inp.stride(0), _p(uk), _p(q_lat), M, spec.heads, spec.dim, spec.rot_dim,
+                                 spec.kv_rank, spec.row, _stream()), "latent_absorb")
+
+
+def latent_unabsorb(o_lat, uv, gate, ldg, out, M, spec):
+    _ck(load().zse_latent_unabsorb(_p(o_lat), _p(uv), gate, ldg, _p(out), out.stride(0), M, spec.heads, spec.vdim,
+                                   spec.kv_rank, _stream()), "latent_unabsorb")
+
+
+def latent_gather(rc, chunks, rows, spec, c_out, kr_out):
+    _ck(load().zse_latent_gather(byref(rc), byref(chunks), rows, spec.kv_rank, spec.rot_dim, _p(c_out), _p(kr_out),
+                                 _stream()), "latent_gather")
+
+
+def latent_chunk(inp, kvx, ldkv, v_col, kr_ctx, rc, chunks, max_q, out, gate, spec):
+    _ck(load().zse_latent_chunk(_p(inp), inp.stride(0), _p(kvx), ldkv, v_col, _p(kr_ctx), byref(rc), byref(chunks),
+                                max_q, _p(out), out.stride(0), gate, spec.heads, spec.dim, spec.rot_dim, spec.vdim,
+                                float(spec.scale), _stream()), "latent_chunk")
+
+
+def moe_tile_rows(M, E, top) -> int:
+    return load().zse_moe_tile_rows(M, E, top)
+
+
+def moe_route(planes, n_planes, M, E, top, tile_rows, x, H, out_per_token, ws):
+    _ck(load().zse_moe_route(_DTYPE[x.dtype], _p(planes), n_planes, M, E, top, tile_rows, _p(x), H, out_per_token,
+                             _p(ws.counts), _p(ws.slot_expert), _p(ws.slot_rank), _p(ws.slot_score), _p(ws.first_row),
+                             _p(ws.tiles), _p(ws.n_tiles), _p(ws.xs), _p(ws.row_score), _p(ws.out_rows), _stream()),
+        "moe_route", 3)
+
+
+def moe_gemm(g, M, E, max_rows, tile_rows, max_tiles, epilogue, status):
+    _ck(load().zse_moe_gemm(byref(g), M, E, max_rows, tile_rows, max_tiles, epilogue, status, _stream()), "moe_gemm")
 
 
 def _u64s(vals):

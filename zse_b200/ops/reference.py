@@ -242,3 +242,93 @@ def filtered_probs(logits: torch.Tensor, temperature: float, top_k: int, top_p: 
 def lora_delta(x: torch.Tensor, a: torch.Tensor, b: torch.Tensor, scaling: float) -> torch.Tensor:
     """x [M, K], a [r, K], b [N, r] -> scaling * (x a^T) b^T in fp32."""
     return scaling * ((x.float() @ a.float().T) @ b.float().T)
+
+
+# ---- latent attention (one cached latent row per token) -------------------------------------------------------------
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, freqs: torch.Tensor) -> torch.Tensor:
+    """Interleaved rotation of the leading ``2 * len(freqs)`` of the last dimension: (2i, 2i+1) turn by
+    ``position * freqs[i]``.  ``x`` [T, ..., R] fp32, ``positions`` [T]."""
+    n = 2 * freqs.numel()
+    ang = positions.float().reshape(-1, *([1] * (x.dim() - 1))) * freqs
+    c, s = torch.cos(ang), torch.sin(ang)
+    u, v = x[..., 0:n:2], x[..., 1:n:2]
+    out = x.clone()
+    out[..., 0:n:2] = u * c - v * s
+    out[..., 1:n:2] = v * c + u * s
+    return out
+
+
+def latent_prep(inp: torch.Tensor, cache_rows: torch.Tensor, positions, slots, freqs, norm_w, spec, eps: float) -> None:
+    """Second half of the fused input projection [q | latent, rotated key | gate]: the latent is RMS-normed and joins the
+    rotated key part in the cache, the rotated part of every query head is rotated in place.  ``cache_rows``
+    [blocks, block_size, row]."""
+    H, d, r, kr = spec.heads, spec.dim, spec.rot_dim, spec.kv_rank
+    T, bs = inp.shape[0], cache_rows.shape[1]
+    q = inp[:, : H * (d + r)].float().view(T, H, d + r)
+    lat = inp[:, spec.latent_col: spec.latent_col + kr + r].float()
+    c = lat[:, :kr] * torch.rsqrt(lat[:, :kr].pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
+    row = torch.cat([c, rotate_pairs(lat[:, kr:], positions, freqs)], dim=-1).to(cache_rows.dtype)
+    ok = slots >= 0
+    s = slots[ok]
+    cache_rows[s // bs, s % bs, : kr + r] = row[ok]
+    q[..., d:] = rotate_pairs(q[..., d:], positions, freqs)
+    inp[:, : H * (d + r)] = q.view(T, -1).to(inp.dtype)
+
+
+def latent_absorb(inp: torch.Tensor, uk: torch.Tensor, spec) -> torch.Tensor:
+    """Queries in the space of the cached rows: [T, H, row], the unrotated part multiplied by W_uk."""
+    H, d, r, kr = spec.heads, spec.dim, spec.rot_dim, spec.kv_rank
+    T = inp.shape[0]
+    q = inp[:, : H * (d + r)].float().view(T, H, d + r)
+    out = torch.zeros(T, H, spec.row, device=inp.device)
+    out[..., :kr] = torch.einsum("thd,hdc->thc", q[..., :d], uk.float().view(H, d, kr))
+    out[..., kr: kr + r] = q[..., d:]
+    return out
+
+
+def latent_attn_token(q_lat: torch.Tensor, cache_rows: torch.Tensor, table: torch.Tensor, pos: int, spec) -> torch.Tensor:
+    """One token's heads against the cached rows it sees: [H, kv_rank] fp32.  ``q_lat`` [H, row]."""
+    bs = cache_rows.shape[1]
+    lo = max(0, pos + 1 - spec.window) if spec.window > 0 else 0
+    j = torch.arange(lo, pos + 1, device=cache_rows.device)
+    blk = table[j // bs].long()
+    j, blk = j[blk >= 0], blk[blk >= 0]
+    if j.numel() == 0:
+        return torch.zeros(spec.heads, spec.kv_rank, device=cache_rows.device)
+    rows = cache_rows[blk, j % bs].float()
+    w = torch.softmax(q_lat.float() @ rows.T * spec.scale, dim=-1)
+    return w @ rows[:, : spec.kv_rank]
+
+
+def latent_attn_chunk(inp: torch.Tensor, c_ctx: torch.Tensor, kr_ctx: torch.Tensor, valid: torch.Tensor, kvx: torch.Tensor,
+                      q_pos: torch.Tensor, ctx_pos: torch.Tensor, spec) -> torch.Tensor:
+    """A chunk's heads against expanded keys and values ``kvx`` [C, H*dim (padded) | H*vdim]: [T, H, vdim] fp32."""
+    H, d, r, vd = spec.heads, spec.dim, spec.rot_dim, spec.vdim
+    T, C = inp.shape[0], kvx.shape[0]
+    q = inp[:, : H * (d + r)].float().view(T, H, d + r)
+    v0 = (H * d + 7) // 8 * 8
+    k = kvx[:, : H * d].float().view(C, H, d)
+    v = kvx[:, v0: v0 + H * vd].float().view(C, H, vd)
+    s = torch.einsum("thd,chd->htc", q[..., :d], k) + torch.einsum("thr,cr->htc", q[..., d:], kr_ctx[:, :r].float())
+    dist = q_pos[:, None] - ctx_pos[None, :]
+    see = (dist >= 0) & valid[None, :]
+    if spec.window > 0:
+        see &= dist < spec.window
+    s = (s * spec.scale).masked_fill(~see, float("-inf"))
+    return torch.einsum("htc,chv->thv", torch.softmax(s, dim=-1).nan_to_num(0.0), v)
+
+
+def gelu_exact(x: torch.Tensor) -> torch.Tensor:
+    return 0.5 * x * (1.0 + torch.erf(x * math.sqrt(0.5)))
+
+
+def route_top(logits: torch.Tensor, top: int):
+    """(expert ids [T, top], their sigmoid scores): largest scores first, the lower id on a tie."""
+    s = torch.sigmoid(logits.float())
+    w, e = torch.sort(s, dim=-1, descending=True, stable=True)
+    return e[:, :top], w[:, :top]
+
+
+def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    """x / sqrt(mean(x^2) + eps) * w, fp32 in and out."""
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()

@@ -50,7 +50,7 @@ class ModelRunner:
 
     def __init__(self, model: DecoderModel, cache: KVCacheManager, max_batch_seqs: int = 64,
                  max_tokens_per_pass: int = 2048, max_seq_len: Optional[int] = None, use_graphs: Optional[bool] = None,
-                 attn_splits: Optional[int] = None):
+                 attn_splits: Optional[int] = None, logits_rows: int = 0):
         self.model, self.cache = model, cache
         self.device = model.device
         c = model.config
@@ -63,7 +63,8 @@ class ModelRunner:
         sm = torch.cuda.get_device_properties(self.device).multi_processor_count if on_gpu else 1
         self._sm = sm
         self.max_attn_splits = attn_splits or (16 if on_gpu else 1)
-        logits_rows = max(max_batch_seqs, 64)
+        logits_rows = max(max_batch_seqs, 64, logits_rows)
+        model.cache_block_size = cache.block_size
         self.buf = model.make_buffers(self.max_tokens, max_batch_seqs, self.max_blocks, logits_rows,
                                       max_planes=8, attn_splits=self.max_attn_splits)
         self._graphs: Dict[Tuple[int, int, bool], torch.cuda.CUDAGraph] = {}
@@ -188,22 +189,28 @@ class ModelRunner:
 
     # ---- prefill / chunk / verify -------------------------------------------------------------------------
     def prefill(self, items: Sequence[Tuple[int, Sequence[int], int]], sampling: Optional[Sequence[SamplingRow]] = None,
-                all_logits: bool = False, adapters: Optional[Sequence[int]] = None, select: bool = True):
+                all_logits: bool = False, adapters: Optional[Sequence[int]] = None, select: bool = True,
+                want: Optional[Sequence[Sequence[int]]] = None):
         """``items``: ``(seq_id, chunk_tokens, start_position)``; the cache must already hold blocks for positions
         ``start .. start+len-1`` of each sequence.  Returns the token chosen after each chunk's last token, or (with
-        ``all_logits``) the fp16 logits of every row (device tensor view, valid until the next pass)."""
+        ``all_logits``) the logits of every row (device tensor view, valid until the next pass).  ``want[i]``: places
+        among the tokens of item i whose logits are wanted instead (returned like ``all_logits``)."""
         b, cache = self.buf, self.cache
         S = len(items)
         total = sum(len(t) for _, t, _ in items)
         if S > self.max_batch_seqs or total > self.max_tokens:
             raise ValueError(f"prefill pass of {total} tokens / {S} sequences exceeds the pass limits "
                              f"({self.max_tokens} / {self.max_batch_seqs})")
-        at, max_q, rows = 0, 0, []
+        at, max_q = 0, 0
         self._staging_begin()
         self.h_bt[:S].fill_(-1)
         per_tok_adapter = [] if adapters is not None else None
-        for s, (sid, toks, start) in enumerate(items):
+        order = self.model.pass_order(items) or range(S)
+        first_row = [0] * S
+        for s, i in enumerate(order):
+            sid, toks, start = items[i]
             n = len(toks)
+            first_row[i] = at
             self.h_ids[at:at + n] = torch.as_tensor(list(toks), dtype=torch.int32)
             self.h_pos[at:at + n] = torch.arange(start, start + n, dtype=torch.int32)
             self.h_slots[at:at + n] = torch.from_numpy(cache.slots_for_range(sid, start, n))
@@ -212,11 +219,15 @@ class ModelRunner:
             self.h_cu[s] = at
             self.h_pos0[s] = start
             if per_tok_adapter is not None:
-                per_tok_adapter += [adapters[s]] * n
-            rows += list(range(at, at + n)) if all_logits else [at + n - 1]
+                per_tok_adapter += [adapters[i]] * n
             at += n
             max_q = max(max_q, n)
         self.h_cu[S] = at
+        if want is None:
+            want = [range(len(t)) if all_logits else (len(t) - 1,) for _, t, _ in items]
+        else:
+            all_logits = True
+        rows = [first_row[i] + k for i in range(S) for k in want[i]]
         n_rows = len(rows)
         if n_rows > b.logits.shape[0]:
             raise ValueError(f"{n_rows} logits rows requested, buffer holds {b.logits.shape[0]}")
@@ -226,6 +237,7 @@ class ModelRunner:
                             (b.logit_rows, self.h_rows, n_rows)):
             self._upload(dst, src, n)
         self._stage_adapters(per_tok_adapter, total, total)
+        self.model.stage_prefill(b, [(items[i][2], len(items[i][1])) for i in order])
         greedy = self._stage_sampling(sampling or [GREEDY] * n_rows, n_rows) if select else True
         self._staging_end()
         ev = None
@@ -251,7 +263,8 @@ class ModelRunner:
     def _pick_splits(self, S: int, max_len: int) -> int:
         if self.device.type != "cuda":
             return 1
-        ctas = S * self.model.plan.num_kv_heads
+        ctas = S * self.model.attention_ctas()
+        max_len = self.model.attention_span(max_len)
         want = (2 * self._sm + ctas - 1) // ctas
         by_len = max(1, max_len // 128)              # at least 128 cached tokens per split
         n = int(max(1, min(want, by_len, self.max_attn_splits)))
@@ -398,6 +411,22 @@ class ModelRunner:
             from ..ops import native
             return native.LAUNCHES
         return [0]
+
+    # ---- one batch of anything ------------------------------------------------------------------------------
+    def run_batch(self, items: Sequence[Tuple[int, Sequence[int], int]], want: Sequence[Sequence[int]]) -> torch.Tensor:
+        """Runs the next tokens of every item - portions of prompts beside single decoded tokens - as one batch and
+        returns the logits at ``want[i]`` (places among item i's tokens), item by item: a device tensor view, valid
+        until the next pass.  A batch of single tokens that continue their sequences is a decode step (graphs
+        included); anything else is one packed pass.  ``items`` as for ``prefill``."""
+        if all(len(t) == 1 and start > 0 for _, t, start in items):
+            self.decode([sid for sid, _, _ in items], [t[0] for _, t, _ in items])
+            rows = [i for i, w in enumerate(want) for _ in w]
+            if rows == list(range(len(items))):
+                return self.buf.logits[: len(rows)]
+            return self.buf.logits[torch.tensor(rows, dtype=torch.int64, device=self.device)]
+        out = self.prefill(items, want=want, select=False)
+        self.model.ops.check()
+        return out
 
     # ---- convenience ----------------------------------------------------------------------------------------
     def verify_tokens(self, seq_id: int, tokens: Sequence[int], start_position: int) -> torch.Tensor:

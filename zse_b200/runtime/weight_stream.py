@@ -17,7 +17,8 @@ import numpy as np
 import torch
 from ..utils import env
 
-_DTYPES = {"uint8": torch.uint8, "int8": torch.int8, "float16": torch.float16}
+_DTYPES = {"uint8": torch.uint8, "int8": torch.int8, "float16": torch.float16,
+           "bfloat16": torch.bfloat16, "int32": torch.int32}
 
 
 class DeviceMirror:
@@ -115,7 +116,7 @@ def open_mirror(loader, device, stats: Optional[dict] = None) -> Optional["Devic
     from its streamed path (zse-engine/zse_engine/orchestrator/weight_loader.py:188-199).  With ``ZSE_DEBUG_LOAD=1`` the
     failure is printed with its traceback; ``stats`` receives the throughput or the reason."""
     dev = torch.device(device)
-    if dev.type != "cuda" or not env.flag("ZSE_STREAM_WEIGHTS"):
+    if dev.type != "cuda" or not getattr(loader, "streamable", True) or not env.flag("ZSE_STREAM_WEIGHTS"):
         return None
     try:
         mirror = DeviceMirror(loader, dev)
