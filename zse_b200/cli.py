@@ -1,4 +1,4 @@
-"""``zse`` command line: ``serve | convert | info | version | warm | keys | synth | bench-kernels``.
+"""``zse`` command line: ``serve | convert | info | version | warm | keys | synth | trace-run | bench-kernels``.
 
 Same verbs and flags as zse-engine/zse_engine/cli.py:213-285 (``serve [model] --port --host --admin-key --db-path
 --model-name -q --tp N``; ``convert <hf_dir> <out.zse> --quant int4|int8|fp16 --group-size --arch --no-tokenizer -q``;
@@ -31,7 +31,7 @@ def _cmd_serve(a) -> int:
                                 max_batch_seqs=a.max_batch_seqs, prefill_chunk_size=a.prefill_chunk_size,
                                 speculative_k=a.speculative_k, speculative_mode=a.speculative_mode,
                                 use_cuda_graphs=not a.no_graphs, comm_backend=a.comm, quiet=a.quiet,
-                                device="cpu" if a.cpu else None)
+                                dtype=a.dtype, device="cpu" if a.cpu else None)
     server = ZSEServer(a.model, a.host, a.port, a.admin_key, a.db_path, a.model_name, a.quiet, a.tp_size,
                        engine_config=cfg, require_auth=a.require_auth)
     loop = asyncio.new_event_loop()
@@ -95,8 +95,8 @@ def _cmd_info(a) -> int:
     for line in describe_devices():
         print(line)
     if a.model:
-        from .format.loader import ZSELoader
-        with ZSELoader(a.model) as l:
+        from .format.directory import open_model
+        with open_model(a.model) as l:
             print()
             print(l.summary())
     if getattr(a, "env", False):
@@ -129,8 +129,22 @@ def _cmd_warm(a) -> int:
     if not os.path.exists(a.model):
         print(f"error: model file not found: {a.model}", file=sys.stderr)
         return 1
-    size, done, t0 = os.path.getsize(a.model), 0, time.time()
-    fd = os.open(a.model, os.O_RDONLY)
+    if os.path.isdir(a.model):
+        from .format.convert import find_safetensor_files
+        files = find_safetensor_files(a.model)
+    else:
+        files = [a.model]
+    size, done, t0 = sum(os.path.getsize(f) for f in files), 0, time.time()
+    for path in files:
+        done += _read_through(path)
+    dt = max(time.time() - t0, 1e-6)
+    print(f"warmed {done / 2**30:.2f} GiB of {size / 2**30:.2f} GiB in {dt:.1f}s ({done / 2**30 / dt:.2f} GiB/s)")
+    return 0
+
+
+def _read_through(path: str) -> int:
+    done = 0
+    fd = os.open(path, os.O_RDONLY)
     try:
         if hasattr(os, "posix_fadvise"):
             os.posix_fadvise(fd, 0, 0, os.POSIX_FADV_WILLNEED)
@@ -142,9 +156,7 @@ def _cmd_warm(a) -> int:
             done += n
     finally:
         os.close(fd)
-    dt = max(time.time() - t0, 1e-6)
-    print(f"warmed {done / 2**30:.2f} GiB of {size / 2**30:.2f} GiB in {dt:.1f}s ({done / 2**30 / dt:.2f} GiB/s)")
-    return 0
+    return done
 
 
 def _cmd_keys(a) -> int:
@@ -187,10 +199,16 @@ def _cmd_bench_kernels(a) -> int:
     return 0
 
 
+def _cmd_trace_run(a) -> int:
+    from .trace import main as trace_main
+    argv = ["--model", a.model, "--dtype", a.dtype, "--out", a.out, "--max-tokens", str(a.max_tokens)]
+    return trace_main(argv + (["--device", a.device] if a.device else []))
+
+
 def build_parser() -> argparse.ArgumentParser:
     p = argparse.ArgumentParser(prog="zse", description="Blackwell-native LLM inference engine for .zse models")
     sub = p.add_subparsers(dest="cmd")
-    s = sub.add_parser("serve", help="serve a .zse model over the OpenAI-compatible HTTP API")
+    s = sub.add_parser("serve", help="serve a .zse model or a model directory over the OpenAI-compatible HTTP API")
     s.add_argument("model", nargs="?", default=None)
     s.add_argument("--port", type=int, default=8000)
     s.add_argument("--host", default="0.0.0.0")
@@ -208,6 +226,8 @@ def build_parser() -> argparse.ArgumentParser:
     s.add_argument("--comm", default="fused", choices=["fused", "nccl", "nccl-sp"],
                    help="tensor-parallel collectives: fused in-kernel exchange, NCCL all-reduce, or NCCL with "
                         "sequence-parallel prefill (reduce-scatter / all-gather, residual split by rows)")
+    s.add_argument("--dtype", default=None, choices=["float16", "bfloat16", "float32"],
+                   help="activation type, for the models that offer more than one (default: the model's own)")
     s.add_argument("--require-auth", action="store_true")
     s.add_argument("--cpu", action="store_true", help="run on the CPU reference path")
     s.set_defaults(fn=_cmd_serve)
@@ -252,10 +272,18 @@ def build_parser() -> argparse.ArgumentParser:
     y = sub.add_parser("synth", help="write a random-weight model of a named shape")
     y.add_argument("shape")
     y.add_argument("output")
-    y.add_argument("--quant", default="int4", choices=["int4", "int8", "fp16"])
+    y.add_argument("--quant", default="int4", choices=["int4", "int8", "fp16"],
+                   help="ignored by architectures that are kept in bfloat16")
     y.add_argument("--seed", type=int, default=0)
     y.add_argument("--fast", action="store_true")
     y.set_defaults(fn=_cmd_synth)
+    t = sub.add_parser("trace-run", help="feed token ids from standard input through a model step by step, write logits")
+    t.add_argument("--model", required=True)
+    t.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    t.add_argument("--out", required=True)
+    t.add_argument("--max-tokens", type=int, required=True)
+    t.add_argument("--device", default=None)
+    t.set_defaults(fn=_cmd_trace_run)
     b = sub.add_parser("bench-kernels", help="per-kernel microbenchmarks with roofline fractions")
     b.add_argument("--shape", default="qwen2.5-14b")
     b.add_argument("--tokens", type=int, default=64)

@@ -16,7 +16,34 @@ from .spec import QuantMethod
 from .tokenizer import BPETokenizer, BYTE_ENCODER, SpecialTokens
 from .writer import ZSEWriter
 
+
+
+def ruralorn_design(layers: int, width: int, vocab: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int,
+                    window: int, experts: int, top: int, ff: int, shared_ff: int = 0, rot_base: float = 10000.0,
+                    eps: float = 1e-6, embed_scale: float = 1.0, logit_scale: float = 1.0,
+                    logit_softcap: float = 30.0) -> dict:
+    """A Ruralorn ``config.json`` whose layers are all alike (callers may change single entries)."""
+    def layer() -> dict:
+        mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+        if shared_ff:
+            mlp["shared"] = {"ff": shared_ff}
+        return {"type": "latent_attention", "mlp": mlp,
+                "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+                          "scale": (dim + rot_dim) ** -0.5, "mask": {"size": window},
+                          "rot": {"dims": rot_dim, "base": rot_base}}}
+    return {"architecture": "Ruralorn", "vocab": vocab, "width": width, "norm": {"eps": eps},
+            "embedding": {"scale": embed_scale}, "logit_scale": logit_scale, "logit_softcap": logit_softcap,
+            "layers": [layer() for _ in range(layers)]}
+
+
+# entries with a "design" hold a config.json of that architecture instead of ``ModelConfig`` fields
 SHAPES = {
+    "tiny-ruralorn": dict(arch="ruralorn", design=ruralorn_design(3, 192, 1024, 6, 24, 8, 40, 56, 40, 10, 3, 72, 104)),
+    # layers of the size real models of this kind have, a few of them
+    "ruralorn-2k": dict(arch="ruralorn", design=ruralorn_design(8, 2048, 102400, 16, 128, 64, 128, 512, 4096, 64, 6, 1408,
+                                                                2816)),
+    "ruralorn-4k": dict(arch="ruralorn", design=ruralorn_design(4, 4096, 102400, 32, 128, 64, 128, 512, 4096, 64, 4, 2048,
+                                                                4096)),
     "tiny": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64, intermediate_size=688,
                  vocab_size=1024, rms_norm_eps=1e-6, rope_theta=10000.0, arch="llama", max_seq_len=2048),
     "tiny-aligned": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64,
@@ -71,6 +98,12 @@ SHAPES = {
 
 def shape_config(name: str, quant: str = "int4", **overrides) -> ModelConfig:
     kw = dict(SHAPES[name])
+    if "design" in kw:
+        from .arch import get_adapter
+        c = get_adapter(kw["arch"]).config_from_hf(kw["design"])
+        for k, v in overrides.items():
+            setattr(c, k, v)
+        return c
     kw.update(overrides)
     method = {"int4": QuantMethod.INT4_ASYM, "int8": QuantMethod.INT8_SYM, "fp16": QuantMethod.NONE}[quant]
     bits = {"int4": 4, "int8": 8, "fp16": 16}[quant]
@@ -107,6 +140,43 @@ def layer_weight_shapes(c: ModelConfig, layer: int = 0):
                   ("mlp.down_proj", c.hidden_size, c.intermediate_size)]
 
 
+def latent_tensor_shapes(c: ModelConfig):
+    """(name, shape) of every tensor of a design with latent attention, in file order."""
+    H = c.hidden_size
+    yield "embed", (c.vocab_size, H)
+    for i in range(c.num_layers):
+        p, a, m = f"l{i}.", c.latent_spec(i), c.moe_spec(i)
+        yield p + "norm1", (H,)
+        yield p + "mix.q", (a.heads * a.qk_dim, H)
+        yield p + "mix.dkv", (a.kv_rank + a.rot_dim, H)
+        yield p + "mix.dkv.norm", (a.kv_rank,)
+        yield p + "mix.uk", (a.heads * a.dim, a.kv_rank)
+        yield p + "mix.uv", (a.heads * a.vdim, a.kv_rank)
+        yield p + "mix.g", (a.heads * a.vdim, H)
+        yield p + "mix.o", (H, a.heads * a.vdim)
+        if m is None:
+            continue
+        yield p + "norm2", (H,)
+        yield p + "mlp.router", (m.experts, H)
+        parts = [(f"mlp.e{e}", m.ff) for e in range(m.experts)] + ([("mlp.shared", m.shared_ff)] if m.shared_ff else [])
+        for name, ff in parts:
+            yield f"{p}{name}.up", (ff, H)
+            yield f"{p}{name}.down", (H, ff)
+    yield "final.norm", (H,)
+    yield "head", (c.vocab_size, H)
+
+
+def _random_bf16(rng, shape, fast: bool) -> np.ndarray:
+    """N(0, 1/fan_in) matrices, norm weights around 1, as bfloat16 bit patterns.  ``fast`` repeats one block of values."""
+    from .convert import round_bf16
+    if len(shape) == 1:
+        return round_bf16(1.0 + 0.1 * rng.standard_normal(shape, dtype=np.float32))
+    n = shape[0] * shape[1]
+    block = min(n, 1 << 20) if fast else n
+    bits = round_bf16(rng.standard_normal(block, dtype=np.float32) * shape[1] ** -0.5)
+    return np.resize(bits, n).reshape(shape)
+
+
 def write_random_model(path: str, config: ModelConfig, seed: int = 0, std: float = 0.02, fast: bool = False,
                        with_tokenizer: bool = True, qkv_bias: Optional[bool] = None) -> None:
     rng = np.random.default_rng(seed)
@@ -118,6 +188,11 @@ def write_random_model(path: str, config: ModelConfig, seed: int = 0, std: float
     if with_tokenizer:
         w.set_tokenizer(byte_tokenizer(c.vocab_size).serialize())
     w.begin_weights()
+    if c.is_latent:
+        for name, shape in latent_tensor_shapes(c):
+            w.add_weight_raw_bf16(name, shape, _random_bf16(rng, shape, fast))
+        w.finalize()
+        return
 
     def linear(name, n, k):
         if c.quant.method == QuantMethod.NONE:

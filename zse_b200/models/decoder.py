@@ -145,6 +145,7 @@ class StepBuffers:
 
 class DecoderModel:
     act_dtype = torch.float16       # activations, and the rows of the KV cache
+    kernel_group: Optional[str] = None      # subset of the native library that is enough (ops/build.py); None = all of it
     mixed_passes = False            # prompt chunks and decoding sequences may share one packed pass
 
     def __init__(self, config: ModelConfig, plan: ShardPlan, ops: TorchOps):
@@ -181,7 +182,7 @@ class DecoderModel:
         elif c.is_latent and cls is DecoderModel:
             from .latent_moe import LatentMoEModel
             cls = LatentMoEModel
-        m = cls(c, plan, ops or make_ops(device))
+        m = cls(c, plan, ops or make_ops(device, cls.kernel_group))
         m.set_dtype(dtype)
         m._load(loader, progress)
         return m

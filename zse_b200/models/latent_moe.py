@@ -120,6 +120,7 @@ class LatentStepBuffers(StepBuffers):
 
 class LatentMoEModel(DecoderModel):
     act_dtype = torch.bfloat16
+    kernel_group = "latent"
     mixed_passes = True
 
     def set_dtype(self, dtype: Optional[str]) -> None:

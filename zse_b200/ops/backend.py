@@ -311,12 +311,13 @@ class MoeWorkspace:
 class CudaOps(TorchOps):
     name = "cuda"
 
-    def __init__(self, device="cuda"):
+    def __init__(self, device="cuda", group: Optional[str] = None):
+        """``group``: the kernels the model needs (``build.GROUPS``); None = the whole library."""
         from . import native
         if not torch.cuda.is_available():
             raise RuntimeError("CudaOps needs a CUDA device")
         self.n = native
-        native.load(build_if_missing=True)
+        native.load(build_if_missing=True, group=group, whole=group is None)
         self.device = torch.device(device)
         self.status = native.Status(self.device)
         self.sm_count = torch.cuda.get_device_properties(self.device).multi_processor_count
@@ -738,8 +739,8 @@ class CudaOps(TorchOps):
         self.n.lora_expand(tmp, b_table, ids, scales, yv, y.stride(0), M, N, rank)
 
 
-def make_ops(device) -> TorchOps:
+def make_ops(device, group: Optional[str] = None) -> TorchOps:
     device = torch.device(device)
     if device.type == "cuda":
-        return CudaOps(device)
+        return CudaOps(device, group)
     return TorchOps(device)

@@ -129,14 +129,15 @@ def variant_path(name: str) -> str:
 
 
 def build_variant(name: str, verbose: bool = False) -> str:
-    extra = VARIANTS[name]
+    return _build_named(variant_path(name), sources(), VARIANTS[name], verbose)
+
+
+def _build_named(out: str, srcs: List[str], extra: tuple, verbose: bool) -> str:
     nvcc = nvcc_path()
     os.makedirs(OBJ_DIR, exist_ok=True)
     os.makedirs(OUT_DIR, exist_ok=True)
     hdr = _headers_digest()
-    srcs = sources()
     objs = [_object_for(s, hdr, extra) for s in srcs]
-    out = variant_path(name)
     stamp = out + ".stamp"
     want = "\n".join(os.path.basename(o) for o in objs)
     if os.path.exists(out) and os.path.exists(stamp) and open(stamp).read() == want:
@@ -151,6 +152,21 @@ def build_variant(name: str, verbose: bool = False) -> str:
         f.write(want)
     _prune()
     return out
+
+
+# Subsets of the library: what one kind of model launches, for a checkout in which nothing has been built yet (a model's
+# first start then waits for these sources only).  The ordinary build contains all of them and is preferred.
+GROUPS = {
+    "latent": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "latent.cu", "moe.cu", "sampling.cu"),
+}
+
+
+def group_path(name: str) -> str:
+    return os.path.join(OUT_DIR, f"libzse_b200.{name}.so")
+
+
+def build_group(name: str, verbose: bool = False) -> str:
+    return _build_named(group_path(name), [os.path.join(CSRC, f) for f in GROUPS[name]], (), verbose)
 
 
 def is_built() -> bool:

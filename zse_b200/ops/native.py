@@ -203,22 +203,34 @@ def lib_path() -> str:
     return os.environ.get("ZSE_NATIVE_LIB") or _build.LIB_PATH
 
 
-def load(build_if_missing: bool = True) -> ctypes.CDLL:
-    global _lib
-    if _lib is not None:
+_partial = False         # _lib is a subset of the library (build.GROUPS)
+
+
+def load(build_if_missing: bool = True, group: Optional[str] = None, whole: bool = False) -> ctypes.CDLL:
+    """The native library this process has loaded, or loads now.  ``group``: the caller needs the kernels of that group
+    only (``build.GROUPS``); where the whole library has not been built, the group's own is built and loaded instead.
+    ``whole``: every kernel is needed, a loaded subset is replaced."""
+    global _lib, _partial
+    if _lib is not None and not (whole and _partial):
         return _lib
     path = lib_path()
+    partial = False
     if not os.path.exists(path):
-        if not build_if_missing:
+        if group is not None and build_if_missing:
+            path, partial = _build.group_path(group), True
+            if not os.path.exists(path):
+                _build.build_group(group)
+        elif not build_if_missing:
             raise NativeError(f"{path} is missing: run `python -m zse_b200.ops.build`")
-        _build.build()
+        else:
+            _build.build()
     lib = ctypes.CDLL(path)
     for name, (res, args) in _SIGS.items():
         fn = getattr(lib, name, None)
         if fn is None:
             continue   # optional entry points are looked up by their users
         fn.restype, fn.argtypes = res, args
-    _lib = lib
+    _lib, _partial = lib, partial
     return lib
 
 

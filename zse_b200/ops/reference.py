@@ -264,7 +264,7 @@ def latent_prep(inp: torch.Tensor, cache_rows: torch.Tensor, positions, slots, f
     [blocks, block_size, row]."""
     H, d, r, kr = spec.heads, spec.dim, spec.rot_dim, spec.kv_rank
     T, bs = inp.shape[0], cache_rows.shape[1]
-    q = inp[:, : H * (d + r)].float().view(T, H, d + r)
+    q = inp[:, : H * (d + r)].float().reshape(T, H, d + r).clone()
     lat = inp[:, spec.latent_col: spec.latent_col + kr + r].float()
     c = lat[:, :kr] * torch.rsqrt(lat[:, :kr].pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
     row = torch.cat([c, rotate_pairs(lat[:, kr:], positions, freqs)], dim=-1).to(cache_rows.dtype)

@@ -57,9 +57,9 @@ def _worker(rank: int, world: int, model_path: str, cfg: EngineConfig, port: int
         ctrl = dist.new_group(backend="gloo")          # control plane (objects), separate from the data group
         from ..engine import ZStreamerEngine
         from .comm import make_comm
-        from ..format.loader import ZSELoader
+        from ..format.directory import open_model
         cfg = EngineConfig(**{**cfg.__dict__, "tp_size": world, "device_index": rank, "quiet": True})
-        with ZSELoader(model_path) as l:
+        with open_model(model_path) as l:
             hidden = l.config.hidden_size
         dev = torch.device(f"cuda:{rank}" if on_gpu else "cpu")
         # the plain collective paths also run on gloo; the fused kernels need GPUs
@@ -169,7 +169,7 @@ class TPEngine:
                  quiet: Optional[bool] = None):
         """``config``: an ``EngineConfig``; the reference's third argument is ``quiet`` (zse-engine/zse_engine/
         orchestrator/tp_engine.py:46-63), so a bool given there is taken as that."""
-        from ..format.loader import ZSELoader
+        from ..format.directory import open_model
         if isinstance(config, bool):
             quiet, config = config, None
         self.model_path, self.tp_size = model_path, tp_size
@@ -177,7 +177,7 @@ class TPEngine:
         self.engine_config.tp_size = tp_size
         if quiet is not None:
             self.engine_config.quiet = bool(quiet)
-        with ZSELoader(model_path) as l:
+        with open_model(model_path) as l:
             self._config = l.config
             self._tokenizer = l.tokenizer
         self._max_seq_len = min(self.engine_config.max_seq_len or self._config.max_seq_len, self._config.max_seq_len, 32768)

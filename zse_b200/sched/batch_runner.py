@@ -77,6 +77,7 @@ class BatchRunner:
         self._inflight: Optional[_InFlight] = None
         self.ahead_launches = 0          # decode steps launched before the step ahead of them had been read
         self.ahead_dropped = 0           # ... of which the result had to be thrown away
+        self.mixed_passes = 0            # passes that held prompt chunks beside decoding sequences
         self._runner = runner
         self._cache = runner.cache
         self._sched = scheduler
@@ -96,8 +97,19 @@ class BatchRunner:
             res.preempted_ids.append(r.request_id)
         for r in plan.finished_requests:
             self._finalize(r, res)
-        if plan.prefill_requests:
+        if plan.prefill_requests and plan.decode_requests and self._run_mixed(plan, res):
+            pass
+        elif plan.prefill_requests:
             self._run_prefill(plan, res)
+            self._decode_planned(plan, res)
+        elif plan.decode_requests:
+            self._decode_planned(plan, res)
+        for r in plan.prefill_requests + plan.decode_requests:
+            if r.is_finished:
+                self._finalize(r, res)
+        return res
+
+    def _decode_planned(self, plan: SchedulerOutput, res: StepResult) -> None:
         if plan.decode_requests:
             live = [r for r in plan.decode_requests if not r.is_finished]
             if live:
@@ -105,10 +117,6 @@ class BatchRunner:
                     self._run_speculative(live, res)
                 else:
                     self._run_decode(live, res)
-        for r in plan.prefill_requests + plan.decode_requests:
-            if r.is_finished:
-                self._finalize(r, res)
-        return res
 
     # ---- helpers ----------------------------------------------------------------------------------------
     def _cache_salt(self, r: InferenceRequest) -> int:
@@ -160,7 +168,8 @@ class BatchRunner:
             self.fatal_error = " ".join(f"{type(exc).__name__}: {exc}".split())[:300]
 
     # ---- prefill ----------------------------------------------------------------------------------------
-    def _run_prefill(self, plan: SchedulerOutput, res: StepResult) -> None:
+    def _prefill_items(self, plan: SchedulerOutput, res: StepResult):
+        """(items of the pass, (request, tokens) of each) for the chunks of a step; new sequences get their blocks."""
         items, owners = [], []
         for r, n in zip(plan.prefill_requests, plan.prefill_chunk_sizes):
             if r.is_finished or n <= 0:
@@ -178,6 +187,10 @@ class BatchRunner:
                 owners.append((r, n))
             except Exception as exc:
                 self._fail(r, exc, res)
+        return items, owners
+
+    def _run_prefill(self, plan: SchedulerOutput, res: StepResult) -> None:
+        items, owners = self._prefill_items(plan, res)
         if not items:
             return
         # split into passes that respect the runner's limits
@@ -201,13 +214,64 @@ class BatchRunner:
                     self._fail(r, exc, res)
                 continue
             for (r, n), tok in zip(ows, toks):
-                res.num_prefill_tokens += n
-                resumed = r.num_generated > 0            # re-prefill after preemption: next input is known
-                self._sched.on_prefill_complete(r, n)
-                if r.state == RequestState.DECODING and not resumed:
-                    self._sched.on_token_generated(r, int(tok))
-                    res.new_tokens[r.request_id] = int(tok)
-                    res.tokens_generated += 1
+                self._chunk_done(r, n, int(tok), res)
+
+    def _chunk_done(self, r: InferenceRequest, n: int, tok: int, res: StepResult) -> None:
+        res.num_prefill_tokens += n
+        resumed = r.num_generated > 0            # re-prefill after preemption: next input is known
+        self._sched.on_prefill_complete(r, n)
+        if r.state == RequestState.DECODING and not resumed:
+            self._sched.on_token_generated(r, tok)
+            res.new_tokens[r.request_id] = tok
+            res.tokens_generated += 1
+
+    def _run_mixed(self, plan: SchedulerOutput, res: StepResult) -> bool:
+        """Prompt chunks and decoding sequences of one step in ONE packed pass, for models whose passes hold both at no
+        loss (``DecoderModel.mixed_passes``).  False when the step has to run as two passes: another model, drafts to
+        verify, penalties that need the token history, or more rows than a pass holds."""
+        if not getattr(self._runner.model, "mixed_passes", False) or (self._spec is not None and self._spec.k > 0):
+            return False
+        live = [r for r in plan.decode_requests if not r.is_finished]
+        total = sum(plan.prefill_chunk_sizes) + len(live)
+        if (not live or any(r.params.repetition_penalty != 1.0 for r in live) or total > self._runner.max_tokens
+                or len(live) + len(plan.prefill_requests) > self._runner.max_batch_seqs):
+            return False
+        items, owners = self._prefill_items(plan, res)
+        ready = self._extend(live, res)
+        items += [(r.seq_id, [r.output_tokens[-1]], self._cache.num_tokens(r.seq_id) - 1) for r in ready]
+        if not items:
+            return True
+        try:
+            toks = self._runner.prefill(items, sampling=[_sampling_row(r) for r, _ in owners]
+                                        + [_sampling_row(r) for r in ready])
+        except Exception as exc:
+            for r in [o[0] for o in owners] + ready:
+                self._fail(r, exc, res)
+            return True
+        for (r, n), tok in zip(owners, toks):
+            self._chunk_done(r, n, int(tok), res)
+        for r, tok in zip(ready, toks[len(owners):]):
+            self._sched.on_token_generated(r, int(tok))
+            res.new_tokens[r.request_id] = int(tok)
+        res.num_decode_tokens += len(ready)
+        res.tokens_generated += len(ready)
+        self.mixed_passes += 1
+        return True
+
+    def _extend(self, reqs: List[InferenceRequest], res: StepResult) -> List[InferenceRequest]:
+        """Reserves the next cache slot of each request; those that got one (the others fail)."""
+        # a request that was extended ahead of time (while the previous step ran on the device) is ready as it is
+        todo = [r for r in reqs if not r.pre_extended]
+        errs = dict(zip((id(r) for r in todo), self._cache.extend_batch([r.seq_id for r in todo])))
+        ready = []
+        for r in reqs:
+            exc = None if r.pre_extended else errs[id(r)]
+            r.pre_extended = False
+            if exc is None:
+                ready.append(r)
+            else:
+                self._fail(r, exc, res)
+        return ready
 
     # ---- decode -----------------------------------------------------------------------------------------
     def _run_decode(self, reqs: List[InferenceRequest], res: StepResult) -> None:
@@ -233,17 +297,7 @@ class BatchRunner:
                 self._inflight = fly
                 self._drop_inflight()
         if rows is None:
-            # a request that was extended ahead of time (while the previous step ran on the device) is ready as it is
-            todo = [r for r in reqs if not r.pre_extended]
-            errs = dict(zip((id(r) for r in todo), self._cache.extend_batch([r.seq_id for r in todo])))
-            ready = []
-            for r in reqs:
-                exc = None if r.pre_extended else errs[id(r)]
-                r.pre_extended = False
-                if exc is None:
-                    ready.append(r)
-                else:
-                    self._fail(r, exc, res)
+            ready = self._extend(reqs, res)
             if not ready:
                 return
             pen = None
