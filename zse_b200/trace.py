@@ -62,7 +62,7 @@ class TraceRunner:
         if items:
             logits = runner.run_batch(items, want)
             if any(want):
-                out = logits.float().cpu().numpy()
+                out = np.array(logits.float().cpu().numpy())       # the buffer belongs to the next pass
         for rid in end:
             sid = self._seq.pop(str(rid), None)
             if sid is not None:
