@@ -68,12 +68,15 @@ def parse_args():
                          "0's per-kernel device times to FILE (a diagnostic: not part of any reported number)")
     ap.add_argument("--spec-k", type=int, default=None,
                     help="override the workload's number of draft tokens per step (0: plain decoding of the same requests)")
-    ap.add_argument("--workload", default="batch64", choices=sorted(WORKLOADS),
+    ap.add_argument("--kernels-file", default=None, metavar="FILE",
+                    help="with --workload ruralorn: also time every kernel alone and write the roofline table to FILE")
+    ap.add_argument("--workload", default="batch64", choices=sorted(WORKLOADS) + ["ruralorn"],
                     help="batch64: 64 requests, prompts uniform in [128, 2048] (the headline); single: one request "
                          "with a 512-token prompt on the 7B shape (the case the reference publishes); spec32b: n-gram "
-                         "speculative decoding on the 32B shape; lora72b: 256 requests over 32 adapters on the 72B shape")
+                         "speculative decoding on the 32B shape; lora72b: 256 requests over 32 adapters on the 72B shape; ruralorn: prefill and decode of the "
+                         "latent-attention / routed design at two sizes beside a dense model of equal size (one GPU)")
     a = ap.parse_args()
-    if a.workload != "batch64":
+    if a.workload not in ("batch64", "ruralorn"):
         w = WORKLOADS[a.workload]
         a.model = w["model"] if a.model == MODEL_SHAPE else a.model
         a.requests = w["requests"] if a.requests == NUM_REQUESTS else a.requests
@@ -394,6 +397,28 @@ def run_ours(args):
         watchdog.cancel()
 
 
+def run_designs(args):
+    """bfloat16 Ruralorn shapes beside their dense neighbours (zse_b200/runtime/design_bench.py)."""
+    from zse_b200.runtime import design_bench
+    if int(os.environ.get("WORLD_SIZE", "1")) > 1:
+        raise SystemExit("--workload ruralorn runs on one GPU")
+    sampler = ClockSampler(0)
+    res = design_bench.run(args.steps, args.warmup, kernels_file=args.kernels_file)
+    clocks = sampler.stop()
+    first = res[design_bench.SHAPES[0]]["ruralorn"]
+    print(json.dumps({
+        "metric": "bf16 Ruralorn decode tok/s", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1,
+        "steps": args.steps, "warmup": args.warmup, "ms_per_step": first["decode_ms_per_step"], "higher_is_better": True,
+        "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"model": f"{design_bench.SHAPES[0]} (random weights)", "global_batch": 64,
+                   "seq_len": "3072-token prompts", "parallelism": "tp1",
+                   "l2_policy": "inputs larger than L2: each step streams the weights and the cache"},
+        "e2e": {"value": first["decode_tok_s_e2e"], "unit": "tok/s", "ms_per_step": first["e2e_ms_per_step"],
+                "h2d_bytes_per_step": 64 * (28 + 4 * first["max_blocks"]), "d2h_bytes_per_step": 64 * 4,
+                "api": "ZStreamerEngine.add_request_tokens + ZStreamerEngine.step"},
+        "gpu_launches": first["gpu_launches"], "clocks": clocks, "extra": {"designs": res, "impl": "ours"}}), flush=True)
+
+
 def rerun_once_in_fresh_process(exc: BaseException) -> None:
     """A device fault ends the CUDA context of this process, and with it the measurement.  A single-GPU run repeats
     itself ONCE in a fresh process (the way a serving deployment restarts a worker) and says so in its result line
@@ -414,8 +439,12 @@ def run_reference(args):
 
 if __name__ == "__main__":
     a = parse_args()
-    if a.impl == "reference":
+    if a.impl == "reference" and a.workload == "ruralorn":
+        print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this design"}))
+    elif a.impl == "reference":
         run_reference(a)
+    elif a.workload == "ruralorn":
+        run_designs(a)
     else:
         try:
             run_ours(a)

@@ -599,18 +599,9 @@ class CudaOps(TorchOps):
         y = ws.y[: M * per * H * y_dt.itemsize].view(y_dt).view(M, per, H)
         if dt == torch.bfloat16 and H % 8 == 0 and m.ff % 8 == 0 and m.shared_ff % 8 == 0:
             tile = n.moe_tile_rows(M, m.experts, m.top)
-            max_tiles = min(slots, m.experts + slots // tile)
             n.moe_route(ws.router, planes, M, m.experts, m.top, tile, x, H, per, ws)
-            g = n.MoeGemm(L.up.data_ptr(), ws.xs.data_ptr(), ws.act.data_ptr(), _dp(L.shared_up), x.data_ptr(),
-                          ws.act_shared.data_ptr(), ws.row_score.data_ptr(), None, ws.tiles.data_ptr(),
-                          ws.n_tiles.data_ptr(), m.ff, H, m.ff, m.shared_ff, H, m.shared_ff, 1, 0, x.shape[0])
-            n.moe_gemm(g, M, m.experts, ws.xs.numel() // H, tile, max_tiles, 0, self.status.ptr)
-            g = n.MoeGemm(L.down.data_ptr(), ws.act.data_ptr(), y.data_ptr(), _dp(L.shared_down),
-                          ws.act_shared.data_ptr(), y.data_ptr(), None, ws.out_rows.data_ptr(), ws.tiles.data_ptr(),
-                          ws.n_tiles.data_ptr(), H, m.ff, H, H if m.shared_ff else 0, m.shared_ff, H, per, m.top,
-                          ws.act_shared.numel() // max(1, m.shared_ff))
-            n.moe_gemm(g, M, m.experts, ws.act.numel() // m.ff, tile, max_tiles, 2 if y_dt == torch.float32 else 1,
-                       self.status.ptr)
+            self.moe_product_call(L, x, M, ws, 0)()
+            self.moe_product_call(L, x, M, ws, 2 if y_dt == torch.float32 else 1)()
             return y
         max_tiles = min(slots, m.experts + slots // 64)
         n.moe_route(ws.router, planes, M, m.experts, m.top, 64, x, H, per, ws)
@@ -625,6 +616,26 @@ class CudaOps(TorchOps):
             n.gemm_tile(dt, ws.act_shared, m.shared_ff, L.shared_down, (m.shared_ff, 1), y, H, M, H, m.shared_ff, store,
                         out_row=(per, m.top))
         return y
+
+    def moe_product_call(self, L, x, M, ws, epilogue: int):
+        """The tensor-core launch of one half of the experts (0: up + gelu; 1, 2: down to bfloat16 / fp32 rows), over
+        the tables that ``moe_route`` left in ``ws``."""
+        n, m, H = self.n, L.moe, x.shape[1]
+        tile = n.moe_tile_rows(M, m.experts, m.top)
+        max_tiles = min(M * m.top, m.experts + M * m.top // tile)
+        if epilogue == 0:
+            g = n.MoeGemm(L.up.data_ptr(), ws.xs.data_ptr(), ws.act.data_ptr(), _dp(L.shared_up), x.data_ptr(),
+                          ws.act_shared.data_ptr(), ws.row_score.data_ptr(), None, ws.tiles.data_ptr(),
+                          ws.n_tiles.data_ptr(), m.ff, H, m.ff, m.shared_ff, H, m.shared_ff, 1, 0, x.shape[0])
+            rows = ws.xs.numel() // H
+        else:
+            per = m.top + (m.shared_ff > 0)
+            g = n.MoeGemm(L.down.data_ptr(), ws.act.data_ptr(), ws.y.data_ptr(), _dp(L.shared_down),
+                          ws.act_shared.data_ptr(), ws.y.data_ptr(), None, ws.out_rows.data_ptr(), ws.tiles.data_ptr(),
+                          ws.n_tiles.data_ptr(), H, m.ff, H, H if m.shared_ff else 0, m.shared_ff, H, per, m.top,
+                          ws.act_shared.numel() // max(1, m.shared_ff))
+            rows = ws.act.numel() // m.ff
+        return lambda: n.moe_gemm(g, M, m.experts, rows, tile, max_tiles, epilogue, self.status.ptr)
 
     def embedding(self, table, ids, out, M, scale=1.0):
         if table.dtype != torch.float16:
