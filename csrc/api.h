@@ -105,7 +105,7 @@ int zse_latent_prep(int dtype, void* inp, int ld, const void* planes, int n_plan
                     void* stream);
 int zse_latent_attn(int dtype, const void* q_lat, const ZseRowCache* c, const void* row_seq, const void* positions,
                     void* o_lat, void* scratch, int M, int heads, int used, int kv_rank, int window, float scale,
-                    int num_splits, int tensor_cores, void* stream);
+                    int num_splits, int tensor_cores, void* status, void* stream);
 int zse_latent_absorb(const void* inp, int ld, const void* uk, void* q_lat, int M, int heads, int dim, int rot,
                       int kv_rank, int row, void* stream);
 int zse_latent_unabsorb(const void* o_lat, const void* uv, const void* gate, int ldg, void* out, int ldo, int M,

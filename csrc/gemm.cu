@@ -114,10 +114,10 @@ struct F16Cfg {
   static constexpr int kABytes = kTileN * 128;
   static constexpr int kXBytes = NT * 128;
   static constexpr int kStageBytes = kABytes + kXBytes;
-  static constexpr int kStages = NT <= 64 ? 4 : (NT == 128 ? 6 : 4);
+  static constexpr int kStages = NT <= 64 ? 4 : (NT == 128 ? 6 : 2);
   static constexpr int kTmemCols = NT < 32 ? 32 : NT;
   static constexpr int kSmemBytes = kStages * kStageBytes + 1024 + 256;
-  static constexpr int kMinBlocks = NT <= 64 ? 2 : 1;
+  static constexpr int kMinBlocks = NT <= 64 || NT == 256 ? 2 : 1;
 };
 
 template <int NT, int EPI, bool BF16>

@@ -30,6 +30,10 @@ struct PrepArgs {
   float eps;
 };
 
+// grid (tokens, 1 + pieces): piece 0 does the latent, the others the queries and (with planes) everything else that later
+// kernels read, kPrepCols columns each.
+constexpr int kPrepCols = 1024;
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_planes, int M, T* __restrict__ cache,
@@ -39,7 +43,7 @@ latent_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, np = a.rot_dims / 2;
+  const int t = blockIdx.x, np = a.rot_dims / 2, qk = a.dim + a.rot;
   float* cs = sm;
   float* sn = sm + np;
   float* lat = sn + np;
@@ -55,6 +59,35 @@ latent_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_
   };
   const float pos = float(positions[t]);
   for (int i = threadIdx.x; i < np; i += blockDim.x) sincosf(pos * freqs[i], &sn[i], &cs[i]);
+  if (blockIdx.y > 0) {
+    __syncthreads();
+    const int c0 = (blockIdx.y - 1) * kPrepCols, qw = a.heads * qk;
+    if (n_planes == 0) {                         // in place: one thread per rotated pair
+      const int i1 = min(a.heads * np, c0 + kPrepCols);
+      for (int i = c0 + threadIdx.x; i < i1; i += blockDim.x) {
+        const int h = i / np, j = i % np, c = h * qk + a.dim + 2 * j;
+        const float u = value(c), v = value(c + 1);
+        in[c] = from_f32<T>(u * cs[j] - v * sn[j]);
+        in[c + 1] = from_f32<T>(v * cs[j] + u * sn[j]);
+      }
+      return;
+    }
+#pragma unroll
+    for (int k = 0; k < kPrepCols / 256; ++k) {
+      const int i = c0 + threadIdx.x + k * 256;
+      if (i >= qw + a.gate_w) break;
+      if (i >= qw) {
+        const int c = a.gate_col + i - qw;
+        in[c] = from_f32<T>(value(c));
+        continue;
+      }
+      const int j = i % qk - a.dim;              // place in the rotated part
+      float v = value(i);
+      if (j >= 0 && j < a.rot_dims) v = v * cs[j >> 1] + ((j & 1) ? value(i - 1) : -value(i + 1)) * sn[j >> 1];
+      in[i] = from_f32<T>(v);
+    }
+    return;
+  }
   float ss = 0.f;
   for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) {
     const float v = value(a.latent_col + i);
@@ -67,38 +100,15 @@ latent_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_
   const float total = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
   const float inv = 1.f / sqrtf(total / float(a.kv_rank) + a.eps);
   const long long slot = slots[t];
-  if (slot >= 0) {
-    T* dst = cache + (slot / rc.block_size) * rc.block_stride + (slot % rc.block_size) * rc.row;
-    for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) dst[i] = from_f32<T>(lat[i] * inv * to_f32(norm_w[i]));
-    const int c0 = a.latent_col + a.kv_rank;
-    for (int i = threadIdx.x; i < a.rot / 2; i += blockDim.x) {
-      float u = value(c0 + 2 * i), v = value(c0 + 2 * i + 1);
-      if (i < np) {
-        const float x = u * cs[i] - v * sn[i];
-        v = v * cs[i] + u * sn[i];
-        u = x;
-      }
-      dst[a.kv_rank + 2 * i] = from_f32<T>(u);
-      dst[a.kv_rank + 2 * i + 1] = from_f32<T>(v);
-    }
-    if ((a.rot & 1) && threadIdx.x == 0) dst[a.kv_rank + a.rot - 1] = from_f32<T>(value(c0 + a.rot - 1));
+  if (slot < 0) return;
+  T* dst = cache + (slot / rc.block_size) * rc.block_stride + (slot % rc.block_size) * rc.row;
+  for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) dst[i] = from_f32<T>(lat[i] * inv * to_f32(norm_w[i]));
+  const int r0 = a.latent_col + a.kv_rank;
+  for (int j = threadIdx.x; j < a.rot; j += blockDim.x) {
+    float v = value(r0 + j);
+    if (j < a.rot_dims) v = v * cs[j >> 1] + ((j & 1) ? value(r0 + j - 1) : -value(r0 + j + 1)) * sn[j >> 1];
+    dst[a.kv_rank + j] = from_f32<T>(v);
   }
-  // queries: the rotated part of every head; with planes also everything else that later kernels read
-  const int qk = a.dim + a.rot;
-  for (int i = threadIdx.x; i < a.heads * np; i += blockDim.x) {
-    const int h = i / np, j = i % np, c = h * qk + a.dim + 2 * j;
-    const float u = value(c), v = value(c + 1);
-    in[c] = from_f32<T>(u * cs[j] - v * sn[j]);
-    in[c + 1] = from_f32<T>(v * cs[j] + u * sn[j]);
-  }
-  if (n_planes == 0) return;
-  const int keep = qk - a.rot_dims;              // per head: unrotated columns and the unrotated tail of the rot part
-  for (int i = threadIdx.x; i < a.heads * keep; i += blockDim.x) {
-    const int h = i / keep, j = i % keep;
-    const int c = h * qk + (j < a.dim ? j : j + a.rot_dims);
-    in[c] = from_f32<T>(value(c));
-  }
-  for (int i = threadIdx.x; i < a.gate_w; i += blockDim.x) in[a.gate_col + i] = from_f32<T>(value(a.gate_col + i));
 }
 
 // ---- tokens against the cached rows: any shape, any type ---------------------------------------------------------------
@@ -154,184 +164,246 @@ latent_attn_simple_kernel(const T* __restrict__ q_lat, const T* __restrict__ cac
 }
 
 // ---- tokens against the cached rows: bfloat16 tensor cores ----------------------------------------------------------
-// CTA = (group of 16 * MT heads, token, key split), 8 warps.  Key tiles of 64 rows stream through a two-stage ring in
-// shared memory.  Scores: warp w takes keys 8w .. 8w+7 of the tile for every head.  Values: warp w takes NTW blocks of 8
-// latent columns for every key.  Shared-memory rows are padded by 16 bytes, which makes ldmatrix conflict-free.
+// CTA = (group of 16 * MT heads, token, key split), 8 warps.  Tiles of 64 keys (aligned to 64, so a tile is a whole number
+// of blocks, or part of one) arrive by bulk copies, one per block, in a two-stage ring.  A cached row is an odd number of
+// 16-byte pieces, which makes ldmatrix conflict-free on the rows exactly as they lie in the cache: nothing is rearranged.
+// Scores: warp (kg, g) takes keys 16 kg .. 16 kg + 15 for head tile g (MT = 2), or for half of the row's columns with the
+// halves exchanged through shared memory (MT = 1).  Values: warp w takes NTW blocks of 8 latent columns for every key.
 constexpr int kLatKeys = 64;
 constexpr int kLatWarps = 8;
 
-__host__ __device__ inline int latent_pitch(int row) { return (row + 15) / 16 * 32 + 16; }     // bytes
-inline size_t latent_smem(int mt, int row) {
-  return size_t(16 * mt + 2 * kLatKeys) * latent_pitch(row) + 2 * size_t(16 * mt) * (kLatKeys * 2 + 16) +
-         size_t(2 * kLatWarps * 16 * mt) * 4 + 2 * kLatKeys * 4;
+__host__ __device__ inline int latent_qpitch(int used) { return (used + 15) / 16 * 32 + 16; }     // bytes
+inline size_t latent_smem(int mt, int row, int used) {
+  return size_t(16 * mt) * latent_qpitch(used) + size_t(2 * kLatKeys) * row * 2 + 64 + 2 * size_t(16 * mt) * (kLatKeys * 2 + 16) +
+         size_t(2 * kLatWarps * 16 * mt) * 4 + kLatWarps * 32 * 16 + 2 * kLatKeys * 4 + 64;
 }
 
 template <int MT, int NTW>
 __global__ void __launch_bounds__(kLatWarps * 32)
 latent_attn_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ cache, RowCache rc,
                    const int* __restrict__ row_seq, const int* __restrict__ positions, bf16* __restrict__ o_lat,
-                   float* __restrict__ scratch, int heads, int kv_rank, int window, float scale_log2, int num_splits) {
+                   float* __restrict__ scratch, int heads, int used, int kv_rank, int window, float scale_log2,
+                   int num_splits, Status* status) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int kRows = 16 * MT;
   constexpr int kPPitch = kLatKeys * 2 + 16;
-  const int row = rc.row, pitch = latent_pitch(row), ksteps = (row + 15) / 16, chunks = row / 8;
+  const int row = rc.row, pitch = row * 2, qpitch = latent_qpitch(used), ksteps = (used + 15) / 16, chunks = row / 8;
+  const int stage_bytes = kLatKeys * pitch;
   uint8_t* sq = smem;
-  uint8_t* sk = sq + kRows * pitch;
-  uint8_t* sp = sk + 2 * kLatKeys * pitch;                       // [hi, lo][kRows][kPPitch]
+  uint8_t* sk = sq + kRows * qpitch;                             // two stages, then 64 bytes that the last k step may read
+  uint8_t* sp = sk + 2 * stage_bytes + 64;                       // [hi, lo][kRows][kPPitch]
   float* smax = reinterpret_cast<float*>(sp + 2 * kRows * kPPitch);   // [warps][kRows]
   float* ssum = smax + kLatWarps * kRows;
-  int* valid = reinterpret_cast<int*>(ssum + kLatWarps * kRows);      // [2][kLatKeys]
+  float4* swap = reinterpret_cast<float4*>(ssum + kLatWarps * kRows); // [warps][32]
+  int* valid = reinterpret_cast<int*>(swap + kLatWarps * 32);         // [2][kLatKeys]
+  uint64_t* full = reinterpret_cast<uint64_t*>(valid + 2 * kLatKeys); // [2]
+  int* abort_flag = reinterpret_cast<int*>(full + 2);
   pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kg = warp & 3, g = warp >> 2;
+  if (threadIdx.x == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  // a hole is not copied and its weights are 0: what lies there has to be finite
+  for (int i = threadIdx.x; i < (2 * stage_bytes + 64) / 16; i += blockDim.x)
+    reinterpret_cast<uint4*>(sk)[i] = make_uint4(0, 0, 0, 0);
+  fence_proxy_async_smem();
   pdl_wait();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h0 = blockIdx.x * kRows, t = blockIdx.y, split = blockIdx.z;
   const int nh = min(kRows, heads - h0);
   const int seq = row_seq != nullptr ? row_seq[t] : t, pos = positions[t];
   const int* table = rc.tables + size_t(seq) * rc.max_blocks;
   const int lo = window > 0 ? max(0, pos + 1 - window) : 0;
-  const int n_tiles = (pos + 1 - lo + kLatKeys - 1) / kLatKeys;
+  const int tile0 = lo / kLatKeys, n_tiles = pos / kLatKeys + 1 - tile0;
   const int per = (n_tiles + num_splits - 1) / num_splits;
-  const int k_begin = lo + split * per * kLatKeys;
-  const int k_end = min(pos + 1, k_begin + per * kLatKeys);
-  const int count = k_end > k_begin ? (k_end - k_begin + kLatKeys - 1) / kLatKeys : 0;
-
-  // queries (zero rows beyond the heads, zero columns beyond the row)
-  for (int r = warp; r < kRows; r += kLatWarps) {
+  const int first = tile0 + split * per;
+  const int count = max(0, min(tile0 + n_tiles, first + per) - first);
+  for (int r = warp; r < kRows; r += kLatWarps) {                // queries (zero rows beyond the heads)
     const bf16* src = q_lat + (size_t(t) * heads + h0 + r) * row;
     for (int c = lane; c < ksteps * 2; c += 32)
-      *reinterpret_cast<uint4*>(sq + r * pitch + c * 16) =
-          (r < nh && c < chunks) ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
+      *reinterpret_cast<uint4*>(sq + r * qpitch + c * 16) =
+          r < nh && c < chunks ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
   }
-  if (chunks < ksteps * 2)
-    for (int r = threadIdx.x; r < 2 * kLatKeys; r += blockDim.x)
-      *reinterpret_cast<uint4*>(sk + r * pitch + chunks * 16) = make_uint4(0, 0, 0, 0);
+  __syncthreads();
 
-  auto issue = [&](int i) {
-    if (i < count) {
-      uint8_t* st = sk + (i & 1) * kLatKeys * pitch;
-      const int key0 = k_begin + i * kLatKeys + warp * 8;
-      int blk = -1;
-      if (lane < 8 && key0 + lane < k_end) blk = table[(key0 + lane) / rc.block_size];
-      if (lane < 8) valid[(i & 1) * kLatKeys + warp * 8 + lane] = blk >= 0;
-#pragma unroll
-      for (int r = 0; r < 8; ++r) {
-        const int b = __shfl_sync(0xffffffffu, blk, r);
-        uint8_t* dst = st + (warp * 8 + r) * pitch;
-        if (b >= 0) {
-          const bf16* src = cache + b * rc.block_stride + size_t((key0 + r) % rc.block_size) * row;
-          for (int c = lane; c < chunks; c += 32) cpa16(dst + c * 16, src + c * 8);
-        } else {
-          for (int c = lane; c < chunks; c += 32) *reinterpret_cast<uint4*>(dst + c * 16) = make_uint4(0, 0, 0, 0);
-        }
-      }
+  const int piece = min(rc.block_size, kLatKeys);                // keys of a tile that lie in one block
+  auto issue = [&](int i) {                                      // warp 0
+    const int st = i & 1, key0 = (first + i) * kLatKeys;
+    const int k = lane * piece;                                  // first key of this lane's piece
+    int blk = -1;
+    if (k < kLatKeys && key0 + k <= pos) blk = table[(key0 + k) / rc.block_size];
+    const unsigned have = __ballot_sync(0xffffffffu, blk >= 0);
+    for (int j = lane; j < kLatKeys; j += 32) {
+      const int key = key0 + j;
+      valid[st * kLatKeys + j] = key >= lo && key <= pos && (have >> (j / piece) & 1);
     }
-    cpa_commit();
+    if (lane == 0) mbar_arrive_expect_tx(&full[st], __popc(have) * piece * pitch);
+    __syncwarp();
+    if (blk >= 0)
+      bulk_g2s(sk + st * stage_bytes + k * pitch,
+               cache + blk * rc.block_stride + size_t((key0 + k) % rc.block_size) * row, piece * pitch, &full[st]);
   };
 
   float o[MT][NTW][4];
-  float m[MT][2], l[MT][2];
+  float m[MT][2], l[2] = {0.f, 0.f};
 #pragma unroll
   for (int a = 0; a < MT; ++a) {
     m[a][0] = m[a][1] = -INFINITY;
-    l[a][0] = l[a][1] = 0.f;
 #pragma unroll
     for (int n = 0; n < NTW; ++n) o[a][n][0] = o[a][n][1] = o[a][n][2] = o[a][n][3] = 0.f;
   }
   const int rq = lane >> 2, cq = (lane & 3) * 2;
-  const uint32_t q_addr = smem_u32(sq) + (lane & 15) * pitch + (lane >> 4) * 16;
+  constexpr int kMaxParts = MT == 1 ? kLatWarps : 4;             // warps that share a head tile's keys
+  const int part = MT == 1 ? warp : kg, tile_row = MT == 1 ? 0 : g * 16;
+  const uint32_t q_addr = smem_u32(sq) + (tile_row + (lane & 15)) * qpitch + (lane >> 4) * 16;
   const uint32_t p_addr = smem_u32(sp) + (lane & 15) * kPPitch + (lane >> 4) * 16;
+  const int half_steps = (ksteps + 1) / 2;
+  const int kk0 = MT == 1 ? g * half_steps : 0;
+  const int kk1 = MT == 1 ? min(ksteps, kk0 + half_steps) : ksteps;
+  const int key_w = MT == 1 ? kg * 16 + g * 8 : kg * 16;         // first key this warp weighs
 
-  issue(0);
+  bool ok = true;
+  if (warp == 0 && count > 0) issue(0);
   for (int i = 0; i < count; ++i) {
-    issue(i + 1);
-    cpa_wait<1>();
-    __syncthreads();
-    const uint32_t kbase = smem_u32(sk + (i & 1) * kLatKeys * pitch);
-    // scores of this warp's 8 keys
-    float s[MT][2][4];
-#pragma unroll
-    for (int a = 0; a < MT; ++a)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[a][0][e] = s[a][1][e] = 0.f;
-    const uint32_t k_addr = kbase + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 16;
-#pragma unroll 4
-    for (int kk = 0; kk < ksteps; kk += 2) {
-      uint32_t b[4];
-      ldm_x4(k_addr + kk * 32, b);
-#pragma unroll
-      for (int a = 0; a < MT; ++a) {
-        uint32_t qa[4];
-        ldm_x4(q_addr + a * 16 * pitch + kk * 32, qa);
-        mma_bf16(s[a][0], qa, b[0], b[1]);
-        if (kk + 1 < ksteps) {
-          ldm_x4(q_addr + a * 16 * pitch + kk * 32 + 32, qa);
-          mma_bf16(s[a][1], qa, b[2], b[3]);
+    if (warp == 0 && i + 1 < count) issue(i + 1);
+    ok = mbar_wait(&full[i & 1], (i >> 1) & 1, abort_flag, status, 81, i);
+    ok = __syncthreads_and(ok) != 0;
+    if (!ok) {                                                   // reported; let the copies in flight land
+      if (threadIdx.x == 0)
+        for (int j = i; j < min(count, i + 2); ++j) {
+          SpinClock clock;
+          while (!mbar_try_wait(&full[j & 1], (j >> 1) & 1) && !clock.expired(0xFF)) {
+          }
         }
-      }
+      break;
     }
-    const int key = warp * 8 + cq;
-    const bool ok0 = valid[(i & 1) * kLatKeys + key] != 0, ok1 = valid[(i & 1) * kLatKeys + key + 1] != 0;
+    const uint32_t kbase = smem_u32(sk) + (i & 1) * stage_bytes;
+    float s[2][2][4];                                            // [even, odd step][8 keys]
 #pragma unroll
-    for (int a = 0; a < MT; ++a) {
+    for (int e = 0; e < 4; ++e) s[0][0][e] = s[0][1][e] = s[1][0][e] = s[1][1][e] = 0.f;
+    const uint32_t k_addr = kbase + (kg * 16 + (lane >> 4) * 8 + (lane & 7)) * pitch + (lane >> 3 & 1) * 16;
+    int kk = kk0;
+#pragma unroll 2
+    for (; kk + 1 < kk1; kk += 2) {
+      uint32_t qa[4], qb[4], b[4], c[4];
+      ldm_x4(q_addr + kk * 32, qa);
+      ldm_x4(k_addr + kk * 32, b);
+      ldm_x4(q_addr + kk * 32 + 32, qb);
+      ldm_x4(k_addr + kk * 32 + 32, c);
+      mma_bf16(s[0][0], qa, b[0], b[1]);
+      mma_bf16(s[0][1], qa, b[2], b[3]);
+      mma_bf16(s[1][0], qb, c[0], c[1]);
+      mma_bf16(s[1][1], qb, c[2], c[3]);
+    }
+    if (kk < kk1) {
+      uint32_t qa[4], b[4];
+      ldm_x4(q_addr + kk * 32, qa);
+      ldm_x4(k_addr + kk * 32, b);
+      mma_bf16(s[0][0], qa, b[0], b[1]);
+      mma_bf16(s[0][1], qa, b[2], b[3]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      s[0][0][e] += s[1][0][e];
+      s[0][1][e] += s[1][1][e];
+    }
+    if (MT == 1) {                                               // the other half of the columns of this warp's 8 keys
+      const float* give = g == 0 ? s[0][1] : s[0][0];
+      swap[warp * 32 + lane] = make_float4(give[0], give[1], give[2], give[3]);
+      __syncthreads();
+      const float4 got = swap[(warp ^ 4) * 32 + lane];
+      if (g == 1) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[0][0][e] = s[0][1][e];
+      }
+      s[0][0][0] += got.x;
+      s[0][0][1] += got.y;
+      s[0][0][2] += got.z;
+      s[0][0][3] += got.w;
+    }
+    float x[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int nb = 0; nb < MT; ++nb) {
+      const int* ok_key = valid + (i & 1) * kLatKeys + key_w + nb * 8 + cq;
+      const bool ok0 = ok_key[0] != 0, ok1 = ok_key[1] != 0;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const float v = (s[a][0][e] + s[a][1][e]) * scale_log2;
-        s[a][0][e] = ((e & 1) ? ok1 : ok0) ? v : -INFINITY;
-      }
-      float x0 = fmaxf(s[a][0][0], s[a][0][1]), x1 = fmaxf(s[a][0][2], s[a][0][3]);
-      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1));
-      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
-      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1));
-      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-      if ((lane & 3) == 0) {
-        smax[warp * kRows + a * 16 + rq] = x0;
-        smax[warp * kRows + a * 16 + rq + 8] = x1;
+        s[0][nb][e] = ((e & 1) ? ok1 : ok0) ? s[0][nb][e] * scale_log2 : -INFINITY;
+        x[e >> 1] = fmaxf(x[e >> 1], s[0][nb][e]);
       }
     }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      x[half] = fmaxf(x[half], __shfl_xor_sync(0xffffffffu, x[half], 1));
+      x[half] = fmaxf(x[half], __shfl_xor_sync(0xffffffffu, x[half], 2));
+      if ((lane & 3) == 0) smax[part * kRows + tile_row + rq + half * 8] = x[half];
+    }
     __syncthreads();
+    bool moved = false;
+    float corr[MT][2];
 #pragma unroll
     for (int a = 0; a < MT; ++a) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
-        const int r = a * 16 + rq + half * 8;
         float mn = m[a][half];
 #pragma unroll
-        for (int w = 0; w < kLatWarps; ++w) mn = fmaxf(mn, smax[w * kRows + r]);
+        for (int w = 0; w < kMaxParts; ++w) mn = fmaxf(mn, smax[w * kRows + a * 16 + rq + half * 8]);
         const float base = mn == -INFINITY ? 0.f : mn;
-        const float corr = exp2f(m[a][half] - base);             // 0 when there was nothing before
+        corr[a][half] = exp2f(m[a][half] - base);                // 0 when there was nothing before
+        moved |= mn > m[a][half];
         m[a][half] = mn;
-        const float p0 = exp2f(s[a][0][half * 2] - base), p1 = exp2f(s[a][0][half * 2 + 1] - base);
-        l[a][half] = l[a][half] * corr + p0 + p1;
+      }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int a0 = MT == 1 ? 0 : g;
+      const float mine = MT == 1 ? m[0][half] : (a0 == 0 ? m[0][half] : m[MT - 1][half]);
+      const float base = mine == -INFINITY ? 0.f : mine;
+      l[half] *= MT == 1 ? corr[0][half] : (a0 == 0 ? corr[0][half] : corr[MT - 1][half]);
+      const int r = tile_row + rq + half * 8;
+#pragma unroll
+      for (int nb = 0; nb < MT; ++nb) {
+        const float p0 = exp2f(s[0][nb][half * 2] - base), p1 = exp2f(s[0][nb][half * 2 + 1] - base);
+        l[half] += p0 + p1;
+        const int key = key_w + nb * 8 + cq;
         *reinterpret_cast<uint32_t*>(sp + r * kPPitch + key * 2) = pack_bf16(p0, p1);
         *reinterpret_cast<uint32_t*>(sp + (kRows + r) * kPPitch + key * 2) = pack_bf16_rest(p0, p1);
+      }
+    }
+    if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+      for (int a = 0; a < MT; ++a)
 #pragma unroll
         for (int n = 0; n < NTW; ++n) {
-          o[a][n][half * 2] *= corr;
-          o[a][n][half * 2 + 1] *= corr;
+          o[a][n][0] *= corr[a][0];
+          o[a][n][1] *= corr[a][0];
+          o[a][n][2] *= corr[a][1];
+          o[a][n][3] *= corr[a][1];
         }
-      }
     }
     __syncthreads();
     const int vr = (lane >> 3 & 1) * 8 + (lane & 7), vc = lane >> 4;
 #pragma unroll
-    for (int kk = 0; kk < kLatKeys / 16; ++kk) {
+    for (int kv = 0; kv < kLatKeys / 16; ++kv) {
       uint32_t ph[MT][4], pl[MT][4];
 #pragma unroll
       for (int a = 0; a < MT; ++a) {
-        ldm_x4(p_addr + a * 16 * kPPitch + kk * 32, ph[a]);
-        ldm_x4(p_addr + (kRows + a * 16) * kPPitch + kk * 32, pl[a]);
+        ldm_x4(p_addr + a * 16 * kPPitch + kv * 32, ph[a]);
+        ldm_x4(p_addr + (kRows + a * 16) * kPPitch + kv * 32, pl[a]);
       }
 #pragma unroll
       for (int n = 0; n < NTW; n += 2) {
         const int col = warp * NTW + n;                          // block of 8 columns (warp-uniform bound)
         if (col * 8 < kv_rank) {
           uint32_t v[4];
-          ldm_x4_t(kbase + (kk * 16 + vr) * pitch + (col + vc) * 16, v);
+          ldm_x4_t(kbase + (kv * 16 + vr) * pitch + (col + vc) * 16, v);
 #pragma unroll
           for (int a = 0; a < MT; ++a) {
             mma_bf16(o[a][n], ph[a], v[0], v[1]);
-            mma_bf16(o[a][n], pl[a], v[0], v[1]);
             mma_bf16(o[a][n + 1], ph[a], v[2], v[3]);
+            mma_bf16(o[a][n], pl[a], v[0], v[1]);
             mma_bf16(o[a][n + 1], pl[a], v[2], v[3]);
           }
         }
@@ -339,16 +411,13 @@ latent_attn_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ cach
     }
     __syncthreads();                                             // the stage may be refilled
   }
-  cpa_wait<0>();
+  if (!ok) return;
 #pragma unroll
-  for (int a = 0; a < MT; ++a) {
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      float v = l[a][half];
-      v += __shfl_xor_sync(0xffffffffu, v, 1);
-      v += __shfl_xor_sync(0xffffffffu, v, 2);
-      if ((lane & 3) == 0) ssum[warp * kRows + a * 16 + rq + half * 8] = v;
-    }
+  for (int half = 0; half < 2; ++half) {
+    float v = l[half];
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
+    if ((lane & 3) == 0) ssum[part * kRows + tile_row + rq + half * 8] = v;
   }
   __syncthreads();
 #pragma unroll
@@ -359,25 +428,23 @@ latent_attn_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ cach
       if (r >= nh) continue;
       float L = 0.f;
 #pragma unroll
-      for (int w = 0; w < kLatWarps; ++w) L += ssum[w * kRows + r];
+      for (int w = 0; w < kMaxParts; ++w) L += ssum[w * kRows + r];
       const size_t hh = size_t(t) * heads + h0 + r;
       const float inv = L > 0.f ? 1.f / L : 0.f;
-      float* part = scratch + (hh * num_splits + split) * (kv_rank + 2);
+      float* out = scratch + (hh * num_splits + split) * (kv_rank + 2);
 #pragma unroll
       for (int n = 0; n < NTW; ++n) {
         const int c = (warp * NTW + n) * 8 + cq;
         const float x = o[a][n][half * 2], y = o[a][n][half * 2 + 1];
-        if (num_splits == 1) {
-          if (c < kv_rank) o_lat[hh * kv_rank + c] = from_f32<bf16>(x * inv);
-          if (c + 1 < kv_rank) o_lat[hh * kv_rank + c + 1] = from_f32<bf16>(y * inv);
-        } else {
-          if (c < kv_rank) part[c] = x;
-          if (c + 1 < kv_rank) part[c + 1] = y;
-        }
+        if (c >= kv_rank) continue;                              // kv_rank is a multiple of 8, c + 1 is below it too
+        if (num_splits == 1)
+          *reinterpret_cast<uint32_t*>(o_lat + hh * kv_rank + c) = pack_bf16(x * inv, y * inv);
+        else
+          *reinterpret_cast<float2*>(out + c) = make_float2(x, y);
       }
       if (num_splits > 1 && warp == 0 && (lane & 3) == 0) {
-        part[kv_rank] = m[a][half];
-        part[kv_rank + 1] = L;
+        out[kv_rank] = m[a][half];
+        out[kv_rank + 1] = L;
       }
     }
   }
@@ -561,6 +628,21 @@ inline size_t chunk_smem(int qk, int vdim) {
   return size_t(64 + 2 * kChKeys) * chunk_pitch(qk) + size_t(2 * kChKeys) * chunk_pitch(vdim) + 2 * kChKeys * 4;
 }
 
+// Rows r, r + step, .. of a key tile, one 16-byte column of each; rows past the end are zero.
+__device__ __forceinline__ void copy_rows(uint8_t* dst, int pitch, const bf16* src, int ld, int r, int step, int rows) {
+  dst += r * pitch;
+  src += size_t(r) * ld;
+#pragma unroll 4
+  for (; r < kChKeys; r += step) {
+    if (r < rows)
+      cpa16(dst, src);
+    else
+      *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+    dst += step * pitch;
+    src += size_t(step) * ld;
+  }
+}
+
 template <int DVT>
 __global__ void __launch_bounds__(128)
 latent_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ kvx, int ldkv, int v_col,
@@ -604,19 +686,23 @@ latent_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict
         const int p = key0 + threadIdx.x;
         valid[st * kChKeys + threadIdx.x] = p < k_end && table[p / rc.block_size] >= 0;
       }
-      const int per = qch + vch;
-      for (int j = threadIdx.x; j < kChKeys * per; j += 128) {
-        const int r = j / per, c = j % per;
-        uint8_t* dst = c < qch ? sk + (st * kChKeys + r) * qp + c * 16 : sv + (st * kChKeys + r) * vp + (c - qch) * 16;
-        if (key0 + r < k_end) {
-          const size_t x = size_t(off + key0 + r - lo);
-          const bf16* src = c < dch ? kvx + x * ldkv + size_t(h) * dim + c * 8
-                          : c < qch ? kr_ctx + x * rot_pad + (c - dch) * 8
-                                    : kvx + x * ldkv + v_col + size_t(h) * vdim + (c - qch) * 8;
-          cpa16(dst, src);
-        } else {
-          *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
-        }
+      // a warp takes 16 rows; a lane keeps its 16-byte columns, so its addresses only move by whole rows
+      const int rows = min(kChKeys, k_end - key0);
+      const size_t x0 = size_t(off + key0 - lo);
+      for (int c = lane; c < qch; c += 32) {
+        const bf16* src = c < dch ? kvx + x0 * ldkv + size_t(h) * dim + c * 8 : kr_ctx + x0 * rot_pad + (c - dch) * 8;
+        const int step = c < dch ? ldkv : rot_pad;
+        copy_rows(sk + st * kChKeys * qp + c * 16, qp, src, step, warp, 4, rows);
+      }
+      if (vch <= 16) {                                           // two rows of values per pass
+        const int c = lane & 15;
+        if (c < vch)
+          copy_rows(sv + st * kChKeys * vp + c * 16, vp, kvx + x0 * ldkv + v_col + size_t(h) * vdim + c * 8, ldkv,
+                    warp * 2 + (lane >> 4), 8, rows);
+      } else {
+        for (int c = lane; c < vch; c += 32)
+          copy_rows(sv + st * kChKeys * vp + c * 16, vp, kvx + x0 * ldkv + v_col + size_t(h) * vdim + c * 8, ldkv, warp, 4,
+                    rows);
       }
     }
     cpa_commit();
@@ -744,17 +830,18 @@ int raise_smem(K kern, size_t bytes, size_t* done) {      // `done`: per device,
 
 template <int MT, int NTW>
 int launch_latent(const void* q, const void* cache, const RowCache& rc, const void* row_seq, const void* positions,
-                  void* o, void* scratch, int M, int heads, int kv_rank, int window, float scale, int splits,
-                  cudaStream_t st) {
+                  void* o, void* scratch, int M, int heads, int used, int kv_rank, int window, float scale, int splits,
+                  Status* status, cudaStream_t st) {
   static size_t done[kMaxDevices] = {};
   auto kern = latent_attn_kernel<MT, NTW>;
-  const size_t smem = latent_smem(MT, rc.row);
+  const size_t smem = latent_smem(MT, rc.row, used);
   if (int r = raise_smem(kern, smem, done)) return r;
   dim3 grid((heads + 16 * MT - 1) / (16 * MT), M, splits);
   return launch_pdl(kern, grid, dim3(kLatWarps * 32), smem, st, reinterpret_cast<const bf16*>(q),
                     reinterpret_cast<const bf16*>(cache), rc, reinterpret_cast<const int*>(row_seq),
                     reinterpret_cast<const int*>(positions), reinterpret_cast<bf16*>(o),
-                    reinterpret_cast<float*>(scratch), heads, kv_rank, window, scale * kLog2E, splits) == cudaSuccess
+                    reinterpret_cast<float*>(scratch), heads, used, kv_rank, window, scale * kLog2E, splits,
+                    status) == cudaSuccess
              ? 0
              : ZSE_ERR_LAUNCH;
 }
@@ -781,14 +868,16 @@ extern "C" int zse_latent_prep(int dtype, void* inp, int ld, const void* planes,
   const PrepArgs a{ld, heads, dim, rot, rot_dims, kv_rank, latent_col, gate_col, gate_w, eps};
   const size_t smem = size_t(rot_dims + kv_rank) * sizeof(float);
   if (smem > 48 * 1024) return ZSE_ERR_LIMIT;
+  const int work = n_planes > 0 ? heads * (dim + rot) + gate_w : heads * (rot_dims / 2);
+  const dim3 grid(M, 1 + (work + kPrepCols - 1) / kPrepCols);
   cudaError_t e;
   if (dtype == kBF16)
-    e = launch_pdl(latent_prep_kernel<bf16>, dim3(M), dim3(256), smem, ST(stream), reinterpret_cast<bf16*>(inp),
+    e = launch_pdl(latent_prep_kernel<bf16>, grid, dim3(256), smem, ST(stream), reinterpret_cast<bf16*>(inp),
                    reinterpret_cast<const float*>(planes), n_planes, M, reinterpret_cast<bf16*>(c->rows), row_cache(c),
                    reinterpret_cast<const int*>(positions), reinterpret_cast<const long long*>(slots),
                    reinterpret_cast<const float*>(freqs), reinterpret_cast<const bf16*>(norm_w), a);
   else
-    e = launch_pdl(latent_prep_kernel<float>, dim3(M), dim3(256), smem, ST(stream), reinterpret_cast<float*>(inp),
+    e = launch_pdl(latent_prep_kernel<float>, grid, dim3(256), smem, ST(stream), reinterpret_cast<float*>(inp),
                    reinterpret_cast<const float*>(planes), n_planes, M, reinterpret_cast<float*>(c->rows), row_cache(c),
                    reinterpret_cast<const int*>(positions), reinterpret_cast<const long long*>(slots),
                    reinterpret_cast<const float*>(freqs), reinterpret_cast<const float*>(norm_w), a);
@@ -797,25 +886,27 @@ extern "C" int zse_latent_prep(int dtype, void* inp, int ld, const void* planes,
 
 // 1 when the tensor-core kernels take this shape (bfloat16): per-head products and latent_attn, and the chunk kernel.
 extern "C" int zse_latent_mma_ok(int heads, int dim, int rot, int vdim, int kv_rank, int row) {
-  return dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && kv_rank % 8 == 0 && dim > 0 && kv_rank <= 512 &&
-         vdim <= 256 && heads > 0 && latent_smem(1, row) <= kSmemLimit && chunk_smem(dim + rot, vdim) <= kSmemLimit;
+  return dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && kv_rank % 8 == 0 && dim > 0 && kv_rank <= 512 && row % 16 == 8 &&
+         vdim <= 256 && heads > 0 && latent_smem(1, row, kv_rank + rot) <= kSmemLimit && chunk_smem(dim + rot, vdim) <= kSmemLimit;
 }
 
 extern "C" int zse_latent_attn(int dtype, const void* q_lat, const ZseRowCache* c, const void* row_seq,
                                const void* positions, void* o_lat, void* scratch, int M, int heads, int used,
-                               int kv_rank, int window, float scale, int num_splits, int tensor_cores, void* stream) {
+                               int kv_rank, int window, float scale, int num_splits, int tensor_cores, void* status,
+                               void* stream) {
   if (M <= 0) return 0;
   if (M > 65535 || num_splits < 1) return ZSE_ERR_LIMIT;
   const RowCache rc = row_cache(c);
   cudaStream_t st = ST(stream);
   if (dtype == kBF16 && tensor_cores) {
-    if (rc.row % 8 || kv_rank > 512 || latent_smem(1, rc.row) > kSmemLimit) return ZSE_ERR_SHAPE;
+    if (rc.row % 16 != 8 || kv_rank % 8 || kv_rank > 512 || 64 % min(rc.block_size, 64) ||
+        rc.block_size % min(rc.block_size, 64) || latent_smem(1, rc.row, used) > kSmemLimit) return ZSE_ERR_SHAPE;
     if ((reinterpret_cast<uintptr_t>(c->rows) & 15) || (rc.block_stride & 7)) return ZSE_ERR_ALIGN;
-    const bool two = heads > 16 && latent_smem(2, rc.row) <= kSmemLimit;
+    const bool two = heads > 16 && latent_smem(2, rc.row, used) <= kSmemLimit;
     int r = ZSE_ERR_SHAPE;
 #define ZSE_LAT(MT_, NTW_)                                                                                           \
-  r = launch_latent<MT_, NTW_>(q_lat, c->rows, rc, row_seq, positions, o_lat, scratch, M, heads, kv_rank, window,     \
-                               scale, num_splits, st)
+  r = launch_latent<MT_, NTW_>(q_lat, c->rows, rc, row_seq, positions, o_lat, scratch, M, heads, used, kv_rank,       \
+                               window, scale, num_splits, reinterpret_cast<Status*>(status), st)
     if (kv_rank <= 128) {
       if (two) ZSE_LAT(2, 2); else ZSE_LAT(1, 2);
     } else if (kv_rank <= 256) {

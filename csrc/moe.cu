@@ -167,10 +167,10 @@ struct MoeCfg {
   static constexpr int kABytes = kTileN * 128;
   static constexpr int kXBytes = NT * 128;
   static constexpr int kStageBytes = kABytes + kXBytes;
-  static constexpr int kStages = NT <= 32 ? 5 : (NT == 128 ? 3 : 4);
-  static constexpr int kTmemCols = NT < 32 ? 32 : NT;
-  static constexpr int kSmemBytes = kStages * kStageBytes + 1024 + 256;
-  static constexpr int kMinBlocks = NT <= 128 ? 2 : 1;
+  static constexpr int kStages = NT <= 32 ? 5 : NT == 64 ? 4 : NT == 128 ? 3 : 2;   // two CTAs share an SM:
+  static constexpr int kTmemCols = NT < 32 ? 32 : NT;                               // one computes while the
+  static constexpr int kSmemBytes = kStages * kStageBytes + 1024 + 256;             // other writes its results
+  static constexpr int kMinBlocks = 2;
 };
 struct MoeBars {
   uint64_t full[8], empty[8], acc_ready;

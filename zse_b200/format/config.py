@@ -87,8 +87,11 @@ class LatentSpec:
 
     @property
     def row(self) -> int:
-        """Elements of a cached token: [latent | rotated key part], padded to 16 bytes of a 16-bit type."""
-        return _up8(self.kv_rank + self.rot_dim)
+        """Elements of a cached token: [latent | rotated key part], padded to an odd number of 16-byte pieces (of a
+        16-bit type): consecutive rows then start in different shared-memory banks and can be used where a plain copy
+        puts them."""
+        n = _up8(self.kv_rank + self.rot_dim)
+        return n if n // 8 % 2 else n + 8
 
 
 @dataclass(frozen=True)

@@ -556,18 +556,18 @@ class CudaOps(TorchOps):
     def latent_attn(self, inp, L, rows, block_tables, row_seq, positions, q_lat, o_lat, out, M, spec, scratch, num_splits):
         n, H, d, r, kr, vd = self.n, spec.heads, spec.dim, spec.rot_dim, spec.kv_rank, spec.vdim
         rc = n.row_cache(rows, block_tables)
-        if self.latent_expands(spec, inp.dtype):
+        if self.latent_expands(spec, inp.dtype) and (rows.shape[1] in (16, 32) or rows.shape[1] % 64 == 0):
             if num_splits > 1 and scratch.numel() < M * num_splits * H * (kr + 2):
                 num_splits = 1
             n.latent_absorb(inp, L.uk, q_lat, M, spec)
-            n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, True)
+            n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, True, self.status.ptr)
             n.latent_unabsorb(o_lat, L.uv, self._gate_ptr(inp, spec), inp.stride(0), out, M, spec)
             return
         ql = q_lat[: M * H * spec.row].view(M, H, spec.row)
         n.gemm_tile(inp.dtype, inp, inp.stride(0), L.uk, (1, kr), ql, H * spec.row, M, kr, d, batch=H, a_batch=d + r,
                     b_batch=d * kr, o_batch=spec.row)
         ql[:, :, kr: kr + r].copy_(inp[:M, : H * (d + r)].view(M, H, d + r)[:, :, d:])
-        n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, 1, False)
+        n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, 1, False, self.status.ptr)
         gate = inp[:, spec.gate_col:] if spec.gated else None
         n.gemm_tile(inp.dtype, o_lat, H * kr, L.uv, (kr, 1), out, out.stride(0), M, vd, kr,
                     n.TILE_GATE if spec.gated else n.TILE_STORE, batch=H, a_batch=kr, b_batch=vd * kr, o_batch=vd,

@@ -173,7 +173,7 @@ _SIGS = {
     "zse_latent_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_int, POINTER(RowCache), c_void_p, c_void_p,
                                 c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_void_p]),
     "zse_latent_attn": (c_int, [c_int, c_void_p, POINTER(RowCache), c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                c_int, c_int, c_int, c_float, c_int, c_int, c_void_p]),
+                                c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p]),
     "zse_latent_absorb": (c_int, [c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 6 + [c_void_p]),
     "zse_latent_unabsorb": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p] + [c_int] * 5 + [c_void_p]),
     "zse_latent_gather": (c_int, [POINTER(RowCache), POINTER(Chunks), c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
@@ -561,10 +561,10 @@ def latent_prep(inp, planes, n_planes, M, rc, positions, slots, freqs, norm_w, s
                                _stream()), "latent_prep")
 
 
-def latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, tensor_cores):
+def latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, tensor_cores, status):
     _ck(load().zse_latent_attn(_DTYPE[q_lat.dtype], _p(q_lat), byref(rc), _p(row_seq), _p(positions), _p(o_lat),
                                _p(scratch), M, spec.heads, spec.kv_rank + spec.rot_dim, spec.kv_rank, spec.window,
-                               float(spec.scale), num_splits, int(tensor_cores), _stream()), "latent_attn",
+                               float(spec.scale), num_splits, int(tensor_cores), status, _stream()), "latent_attn",
         2 if num_splits > 1 else 1)
 
 

@@ -197,7 +197,8 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
             add(phase, "queries into the latent", "output projection", lambda: ops.n.latent_absorb(inp, L.uk, ql, M, s),
                 2.0 * (s.heads * s.dim * kr + M * hw + M * s.heads * row), 2.0 * M * s.heads * s.dim * kr)
             add(phase, "latent attention (with merge of splits)", "attention (with merge of splits)",
-                lambda: ops.n.latent_attn(ql, rc, None, positions, ol, scratch, M, s, splits, True),
+                lambda: ops.n.latent_attn(ql, rc, None, positions, ol, scratch, M, s, splits, True,
+                                          ops.status.ptr),
                 2.0 * M * (ctx * row + s.heads * (row + kr)), 2.0 * M * ctx * s.heads * (row + kr))
             lens = ii([ctx] * M)
             add(phase, "attention (with merge of splits)", None,
