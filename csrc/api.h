@@ -93,6 +93,7 @@ typedef struct ZseRowCache {
   int32_t block_size, row;
   const void* tables;       // block tables [sequences][max_blocks]
   int32_t max_blocks;
+  int32_t num_blocks;       // blocks in the pool (0: unknown, the kernels that need a tensor map are not used)
 } ZseRowCache;
 typedef struct ZseChunks {  // sequences [first, last) of a packed pass
   const void *cu_q, *q_pos0, *ctx_off;
@@ -103,6 +104,7 @@ int zse_latent_prep(int dtype, void* inp, int ld, const void* planes, int n_plan
                     const void* positions, const void* slots, const void* freqs, const void* norm_w, int heads, int dim,
                     int rot, int rot_dims, int kv_rank, int latent_col, int gate_col, int gate_w, float eps,
                     void* stream);
+// tensor_cores: 0 the general kernel, 1 tcgen05 where the shape allows (else as 2), 2 mma.sync
 int zse_latent_attn(int dtype, const void* q_lat, const ZseRowCache* c, const void* row_seq, const void* positions,
                     void* o_lat, void* scratch, int M, int heads, int used, int kv_rank, int window, float scale,
                     int num_splits, int tensor_cores, void* status, void* stream);

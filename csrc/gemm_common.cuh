@@ -31,6 +31,11 @@ struct GemmArgs {
 // bounds; cached per (pointer, shape, box).  Defined in gemm.cu.
 int get_tmap(const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows, CUtensorMap* out);
 
+// 16-bit rows in blocks, [blocks][block_size][row] with `block_stride` elements between blocks: box = 64 columns x box_rows
+// rows of one block, 128-byte swizzle, zero fill out of bounds; cached.  Defined in gemm.cu.
+int get_tmap_rows3(const void* ptr, int blocks, int block_size, int row, long long block_stride, int box_rows,
+                   CUtensorMap* out);
+
 // Where a row-parallel GEMM sends its partial output tiles when the tensor-parallel exchange is part of the GEMM
 // (gemm_w4.cu, kEpiPushF16): rank r's tile goes, as fp16, into slot r of EVERY rank's inbox - one multimem.st through
 // the NVSwitch, or one store per peer - and each CTA then adds 1 to the counter `arrive[k][slot][r]` on every rank k.

@@ -2,7 +2,7 @@
 //
 //   latent_prep     second half of the fused input projection: latent norm, rotation, cache write
 //   latent_attn     tokens against the cached rows themselves (queries already multiplied by W_uk): all heads of a group
-//                   share each row, its leading part is the value as well
+//                   share each row, its leading part is the value as well (tcgen05 form: latent_tc.cu)
 //   latent_combine  merges the key splits of a decode step
 //   head_gemm       per-head products around latent_attn: q W_uk before it, o W_uv^T (times the gate) after it
 //   latent_gather   cached rows a chunk's window reaches, in order, for the expansion GEMM
@@ -12,17 +12,10 @@
 // product with the values as two bfloat16 terms (value and remainder), so that they keep 16 bits.  The *_simple kernels
 // run any shape and float.  Cached rows are addressed through the block table; block -1 is a hole whose tokens do not exist.
 #include "api.h"
-#include "typed.cuh"
+#include "latent.cuh"
 
 namespace zse {
 namespace {
-
-struct RowCache {
-  long long block_stride;       // elements between blocks
-  int block_size, row;          // tokens per block, elements per row
-  const int* tables;            // [sequences][max_blocks]
-  int max_blocks;
-};
 
 // ---- prep -----------------------------------------------------------------------------------------------------------
 struct PrepArgs {
@@ -869,15 +862,15 @@ extern "C" int zse_latent_prep(int dtype, void* inp, int ld, const void* planes,
   const size_t smem = size_t(rot_dims + kv_rank) * sizeof(float);
   if (smem > 48 * 1024) return ZSE_ERR_LIMIT;
   const int work = n_planes > 0 ? heads * (dim + rot) + gate_w : heads * (rot_dims / 2);
-  const dim3 grid(M, 1 + (work + kPrepCols - 1) / kPrepCols);
+  const dim3 grid(M, 1 + (work + kPrepCols - 1) / kPrepCols), block(n_planes > 0 ? 256 : 128);
   cudaError_t e;
   if (dtype == kBF16)
-    e = launch_pdl(latent_prep_kernel<bf16>, grid, dim3(256), smem, ST(stream), reinterpret_cast<bf16*>(inp),
+    e = launch_pdl(latent_prep_kernel<bf16>, grid, block, smem, ST(stream), reinterpret_cast<bf16*>(inp),
                    reinterpret_cast<const float*>(planes), n_planes, M, reinterpret_cast<bf16*>(c->rows), row_cache(c),
                    reinterpret_cast<const int*>(positions), reinterpret_cast<const long long*>(slots),
                    reinterpret_cast<const float*>(freqs), reinterpret_cast<const bf16*>(norm_w), a);
   else
-    e = launch_pdl(latent_prep_kernel<float>, grid, dim3(256), smem, ST(stream), reinterpret_cast<float*>(inp),
+    e = launch_pdl(latent_prep_kernel<float>, grid, block, smem, ST(stream), reinterpret_cast<float*>(inp),
                    reinterpret_cast<const float*>(planes), n_planes, M, reinterpret_cast<float*>(c->rows), row_cache(c),
                    reinterpret_cast<const int*>(positions), reinterpret_cast<const long long*>(slots),
                    reinterpret_cast<const float*>(freqs), reinterpret_cast<const float*>(norm_w), a);
@@ -898,6 +891,16 @@ extern "C" int zse_latent_attn(int dtype, const void* q_lat, const ZseRowCache* 
   if (M > 65535 || num_splits < 1) return ZSE_ERR_LIMIT;
   const RowCache rc = row_cache(c);
   cudaStream_t st = ST(stream);
+  if (dtype == kBF16 && tensor_cores == 1 && latent_tc_ok(rc, c->num_blocks, used, kv_rank) &&
+      !((reinterpret_cast<uintptr_t>(c->rows) & 15) || (rc.block_stride & 7))) {
+    const int r = launch_latent_tc(reinterpret_cast<const bf16*>(q_lat), c->rows, rc, c->num_blocks,
+                                   reinterpret_cast<const int*>(row_seq), reinterpret_cast<const int*>(positions),
+                                   reinterpret_cast<bf16*>(o_lat), reinterpret_cast<float*>(scratch), M, heads, used,
+                                   kv_rank, window, scale, num_splits, reinterpret_cast<Status*>(status), st);
+    if (r || num_splits == 1) return r;
+    return launch_pdl(latent_combine_kernel, dim3(heads, M), dim3(128), 0, st, reinterpret_cast<const float*>(scratch),
+                      reinterpret_cast<bf16*>(o_lat), heads, kv_rank, num_splits) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+  }
   if (dtype == kBF16 && tensor_cores) {
     if (rc.row % 16 != 8 || kv_rank % 8 || kv_rank > 512 || 64 % min(rc.block_size, 64) ||
         rc.block_size % min(rc.block_size, 64) || latent_smem(1, rc.row, used) > kSmemLimit) return ZSE_ERR_SHAPE;

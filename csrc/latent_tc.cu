@@ -1,0 +1,402 @@
+// Latent attention of decoding tokens on the 5th-generation tensor cores (bfloat16).
+//
+// CTA = (16 or 32 heads, token, key split).  Every head of the group uses the same cached rows, as keys and as values, so
+// both products put the rows on the wide side of the MMA and the heads on the narrow one:
+//
+//   S^T [keys, heads]      = K [64 keys, row] . Q^T          A = cached rows, K-major;  B = queries
+//   O^T [latent, heads]   += V^T [latent, 64 keys] . P^T     A = the SAME shared-memory tile, MN-major (the latent part of
+//                                                            a row is the value);  B = softmax weights
+//
+// Both accumulators live in TMEM.  A tile of 64 keys is a set of 64-column panels with the 128-byte swizzle, each brought by
+// one TMA box per cache block through the block table.  The MMA's 128 rows are more than the 64 keys of a tile: its upper
+// half multiplies whatever follows the panel in shared memory and is never read.  Roles: a TMA producer, an MMA issuer, four
+// softmax warps.  The products of tile i + 1 with the queries run while tile i is weighed; softmax weights are split into two
+// bfloat16 terms; the running maximum is only moved (and O rescaled) when a score exceeds it by more than 2^8.  Every wait is
+// bounded and reports through the status word.
+#include <mutex>
+#include <unordered_map>
+
+#include "api.h"
+#include "gemm_common.cuh"
+#include "latent.cuh"
+
+namespace zse {
+namespace {
+
+constexpr int kTcKeys = 64;
+constexpr int kTcPanelBytes = kTcKeys * 128;
+constexpr int kTcMaxPanels = 9;                 // rows of up to 576 columns
+constexpr int kTcThreads = 256;                 // warp 0 producer, 1 MMA, 2 TMEM, 4..7 softmax
+constexpr float kTcSlack = 8.f;                 // log2 of how far a score may exceed the reference
+
+struct LatentTcArgs {
+  const bf16* q_lat;
+  RowCache rc;
+  const int *row_seq, *positions;
+  bf16* o_lat;
+  float* scratch;
+  int heads, used, kv_rank, window, num_splits;
+  float scale_log2;
+  Status* status;
+};
+
+struct LatentTcBars {
+  uint64_t full[2], s_ready[2], p_ready[2], pv_done[2];
+  uint32_t tmem_base;
+  int abort_flag;
+};
+
+template <int N>
+struct LatentTcCfg {
+  static constexpr int kSPitch = kTcKeys + 4;   // floats
+  static constexpr int kTmemCols = N == 16 ? 128 : 256;
+  static constexpr int kOCol = 2 * N;           // O^T blocks after the two S^T buffers
+  __host__ __device__ static int q_bytes(int panels) { return panels * N * 128; }
+  __host__ __device__ static size_t smem(int panels) {
+    return 1024 + size_t(2) * panels * kTcPanelBytes + q_bytes(panels) + 4 * N * 128 + size_t(N) * kSPitch * 4 +
+           3 * N * 4 + 64 + sizeof(LatentTcBars);
+  }
+};
+
+__device__ __forceinline__ void tma_load_3d(void* dst, const void* map, int x, int y, int z, uint64_t* bar) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(
+          smem_u32(dst)),
+      "l"(map), "r"(x), "r"(y), "r"(z), "r"(smem_u32(bar))
+      : "memory");
+}
+// MN-major operand, 128-byte swizzle: rows of the K dimension hold 64 MN elements, eight rows per 1024 bytes, the next 64 MN
+// elements one panel on.
+__device__ __forceinline__ uint64_t make_desc_panel_mn(uint32_t smem_addr) {
+  uint64_t d = 0;
+  d |= uint64_t((smem_addr >> 4) & 0x3FFF);
+  d |= uint64_t(kTcPanelBytes >> 4) << 16;
+  d |= uint64_t(1024 >> 4) << 32;
+  d |= uint64_t(1) << 46;
+  d |= uint64_t(2) << 61;
+  return d;
+}
+// Barrier of the softmax warps; true on every thread when `ok` was true on all of them.
+__device__ __forceinline__ bool softmax_agree(bool ok) {
+  uint32_t all;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\t"
+      "barrier.cta.red.and.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+      : "=r"(all)
+      : "r"(uint32_t(ok))
+      : "memory");
+  return all != 0;
+}
+__device__ __forceinline__ bool softmax_any(bool v) { return !softmax_agree(!v); }
+
+// N consecutive 32-bit columns of the thread's TMEM lane
+template <int N>
+__device__ __forceinline__ void tmem_load(uint32_t* r, uint32_t addr) {
+#pragma unroll
+  for (int c = 0; c < N; c += 16) ZSE_TMEM_LD_X16((r + c), addr + c);
+  tc_wait_ld();
+}
+
+template <int N>
+__global__ void __launch_bounds__(kTcThreads, 1)
+latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) {
+  using Cfg = LatentTcCfg<N>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int panels = (a.used + 63) / 64, ksteps = (a.used + 15) / 16, blocks = (a.kv_rank + 127) / 128;
+  const int stage_bytes = panels * kTcPanelBytes;
+  uint8_t* sk = smem;                                            // [2 stages][panels][64 keys][128 bytes]
+  uint8_t* sq = sk + 2 * stage_bytes;                            // [panels][N heads][128 bytes]
+  uint8_t* sp = sq + Cfg::q_bytes(panels);                       // [2][hi, lo][N heads][128 bytes]
+  float* ss = reinterpret_cast<float*>(sp + 4 * N * 128);        // scores [N][kSPitch]
+  float* corr = ss + N * Cfg::kSPitch;                           // [N]
+  float* ref_out = corr + N;                                     // [N] reference, [N] sum
+  LatentTcBars* bars = reinterpret_cast<LatentTcBars*>(
+      (reinterpret_cast<uintptr_t>(ref_out + 2 * N) + 15) & ~uintptr_t(15));
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_launch_dependents();
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&bars->full[i], 1);
+      mbar_init(&bars->s_ready[i], 1);
+      mbar_init(&bars->p_ready[i], 128);
+      mbar_init(&bars->pv_done[i], 1);
+    }
+    bars->abort_flag = 0;
+    mbar_fence_init();
+    prefetch_tmap(&map);
+  }
+  if (warp == 2) {
+    tmem_alloc(&bars->tmem_base, Cfg::kTmemCols);
+    tmem_relinquish();
+  }
+  // a hole is not copied and its weights are 0: what lies there has to be finite
+  for (int i = threadIdx.x; i < 2 * stage_bytes / 16; i += kTcThreads)
+    reinterpret_cast<uint4*>(sk)[i] = make_uint4(0, 0, 0, 0);
+  pdl_wait();
+  const int h0 = blockIdx.x * N, t = blockIdx.y, split = blockIdx.z;
+  const int nh = min(N, a.heads - h0);
+  const int seq = a.row_seq != nullptr ? a.row_seq[t] : t, pos = a.positions[t];
+  const int* table = a.rc.tables + size_t(seq) * a.rc.max_blocks;
+  const int lo = a.window > 0 ? max(0, pos + 1 - a.window) : 0;
+  const int tile0 = lo / kTcKeys, n_tiles = pos / kTcKeys + 1 - tile0;
+  const int per = (n_tiles + a.num_splits - 1) / a.num_splits;
+  const int first = tile0 + split * per;
+  const int count = max(0, min(tile0 + n_tiles, first + per) - first);
+  const int chunks = a.rc.row / 8;
+  for (int i = threadIdx.x; i < N * panels * 8; i += kTcThreads) {       // queries; zero beyond the heads and the row
+    const int h = i / (panels * 8), c = i % (panels * 8);
+    const uint4 v = h < nh && c < chunks
+                        ? reinterpret_cast<const uint4*>(a.q_lat + (size_t(t) * a.heads + h0 + h) * a.rc.row)[c]
+                        : make_uint4(0, 0, 0, 0);
+    *reinterpret_cast<uint4*>(sq + (c >> 3) * N * 128 + h * 128 + (((c & 7) ^ (h & 7)) << 4)) = v;
+  }
+  fence_proxy_async_smem();
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem = bars->tmem_base;
+  volatile int* abort_flag = &bars->abort_flag;
+
+  if (warp == 0) {
+    const int piece = min(a.rc.block_size, kTcKeys);
+    int issued = 0;
+    for (int i = 0; i < count; ++i) {
+      const int st = i & 1, key0 = (first + i) * kTcKeys;
+      const bool go = i < 2 || mbar_wait(&bars->pv_done[st], ((i >> 1) - 1) & 1, abort_flag, a.status, 91, i);
+      if (!__all_sync(0xffffffffu, go)) break;
+      int blk = -1;
+      if (lane * piece < kTcKeys && key0 + lane * piece <= pos) blk = table[(key0 + lane * piece) / a.rc.block_size];
+      const unsigned have = __ballot_sync(0xffffffffu, blk >= 0);
+      if (lane == 0) mbar_arrive_expect_tx(&bars->full[st], __popc(have) * piece * panels * 128);
+      __syncwarp();
+      // lane p brings panel p of every block
+      for (int j = 0; j * piece < kTcKeys; ++j) {
+        const int b = __shfl_sync(0xffffffffu, blk, j);
+        if (b >= 0 && lane < panels)
+          tma_load_3d(sk + st * stage_bytes + lane * kTcPanelBytes + j * piece * 128, &map, lane * 64,
+                      (key0 + j * piece) % a.rc.block_size, b, &bars->full[st]);
+      }
+      issued = i + 1;
+    }
+    if (*abort_flag && lane == 0) {
+      for (int i = max(0, issued - 2); i < issued; ++i) {        // the copies in flight land before the CTA leaves
+        SpinClock clock;
+        while (!mbar_try_wait(&bars->full[i & 1], (i >> 1) & 1) && !clock.expired(0xFF)) {
+        }
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = make_idesc_f16(128, N, 1);
+      constexpr uint32_t idesc_o = make_idesc_f16(128, N, 1) | (1u << 15);          // A is MN-major
+      auto weigh = [&](int i) {                                                     // O^T += V^T P^T of tile i
+        const uint32_t kb = smem_u32(sk) + (i & 1) * stage_bytes, pb = smem_u32(sp) + (i & 1) * 2 * N * 128;
+        for (int b = 0; b < blocks; ++b) {
+#pragma unroll
+          for (int j = 0; j < kTcKeys / 16; ++j) {
+            const uint64_t v = make_desc_panel_mn(kb + 2 * b * kTcPanelBytes + j * 2048);
+            umma_ss(tmem + Cfg::kOCol + b * N, v, make_desc_sw128(pb + j * 32), idesc_o, (i | j) != 0);
+            umma_ss(tmem + Cfg::kOCol + b * N, v, make_desc_sw128(pb + N * 128 + j * 32), idesc_o, 1);
+          }
+        }
+        tc_commit(&bars->pv_done[i & 1]);
+      };
+      bool ok = true;
+      for (int i = 0; i < count && ok; ++i) {
+        ok = mbar_wait(&bars->full[i & 1], (i >> 1) & 1, abort_flag, a.status, 92, i);
+        if (!ok) break;
+        tc_fence_after_sync();
+        const uint32_t kb = smem_u32(sk) + (i & 1) * stage_bytes, qb = smem_u32(sq);
+        for (int kk = 0; kk < ksteps; ++kk)
+          umma_ss(tmem + (i & 1) * N, make_desc_sw128(kb + (kk >> 2) * kTcPanelBytes + (kk & 3) * 32),
+                  make_desc_sw128(qb + (kk >> 2) * N * 128 + (kk & 3) * 32), idesc_s, kk != 0);
+        tc_commit(&bars->s_ready[i & 1]);
+        if (i > 0) {
+          ok = mbar_wait(&bars->p_ready[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, a.status, 93, i);
+          if (!ok) break;
+          tc_fence_after_sync();
+          weigh(i - 1);
+        }
+      }
+      if (ok && count > 0) {
+        const int i = count - 1;
+        if (mbar_wait(&bars->p_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 94, i)) {
+          tc_fence_after_sync();
+          weigh(i);
+        }
+      }
+    }
+  } else if (warp >= 4) {
+    constexpr int kPerHead = 128 / N, kMine = kTcKeys / kPerHead;        // threads per head, keys per thread (8 or 16)
+    const int tid = threadIdx.x - 128, quarter = warp & 3;
+    const int head = tid / kPerHead, sub = tid % kPerHead;
+    const uint32_t lane_base = tmem + (uint32_t(quarter * 32) << 16);
+    float ref = -INFINITY, sum = 0.f;
+    bool ok = true;
+    for (int i = 0; i < count; ++i) {
+      ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 95, i));
+      if (ok && quarter < 2) {                                   // lanes 0..63 of S^T are the tile's keys
+        tc_fence_after_sync();
+        uint32_t r[N];
+        tmem_load<N>(r, lane_base + (i & 1) * N);
+        const int k = quarter * 32 + lane, key = (first + i) * kTcKeys + k;
+        const bool see = key >= lo && key <= pos && table[key / a.rc.block_size] >= 0;
+#pragma unroll
+        for (int h = 0; h < N; ++h)
+          ss[h * Cfg::kSPitch + k] = see ? __uint_as_float(r[h]) * a.scale_log2 : -INFINITY;
+        tc_fence_before_sync();
+      }
+      ok = softmax_agree(ok);
+      if (!ok) break;
+      float s[kMine], mx = -INFINITY;
+#pragma unroll
+      for (int c = 0; c < kMine; c += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(ss + head * Cfg::kSPitch + sub * kMine + c);
+        s[c] = v.x;
+        s[c + 1] = v.y;
+        s[c + 2] = v.z;
+        s[c + 3] = v.w;
+        mx = fmaxf(fmaxf(fmaxf(mx, v.x), fmaxf(v.y, v.z)), v.w);
+      }
+#pragma unroll
+      for (int d = 1; d < kPerHead; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+      const bool move = mx > ref + kTcSlack || (ref == -INFINITY && mx > ref);
+      const float next = move ? mx : ref;
+      const float factor = ref == -INFINITY ? 0.f : exp2f(ref - next);   // 1 when the reference stays
+      ref = next;
+      sum *= factor;
+      if (sub == 0) corr[head] = move ? factor : 1.f;
+      const bool rescale = softmax_any(move) && i > 0;
+      if (rescale) {                                             // O^T so far is relative to the old references
+        ok = mbar_wait(&bars->pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, a.status, 96, i);
+        ok = softmax_agree(ok);
+        if (!ok) break;
+        tc_fence_after_sync();
+        for (int b = 0; b < blocks; ++b) {
+#pragma unroll
+          for (int c = 0; c < N; c += 16) {
+            uint32_t r[16];
+            const uint32_t addr = lane_base + Cfg::kOCol + b * N + c;
+            ZSE_TMEM_LD_X16(r, addr);
+            tc_wait_ld();
+#pragma unroll
+            for (int e = 0; e < 16; ++e) r[e] = __float_as_uint(__uint_as_float(r[e]) * corr[c + e]);
+            ZSE_TMEM_ST_X16(addr, r);
+          }
+        }
+        tc_wait_st();
+        tc_fence_before_sync();
+      } else if (i >= 2) {                                       // the weights of tile i - 2 have been used
+        ok = mbar_wait(&bars->pv_done[i & 1], ((i >> 1) - 1) & 1, abort_flag, a.status, 97, i);
+        ok = softmax_agree(ok);
+        if (!ok) break;
+      }
+      const float base = ref == -INFINITY ? 0.f : ref;
+      uint8_t* p = sp + (i & 1) * 2 * N * 128 + head * 128;
+#pragma unroll
+      for (int c = 0; c < kMine; c += 8) {
+        float w[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          w[e] = exp2f(s[c + e] - base);
+          sum += w[e];
+        }
+        const int chunk = ((sub * kMine + c) >> 3) ^ (head & 7);
+        *reinterpret_cast<uint4*>(p + (chunk << 4)) =
+            make_uint4(pack_bf16(w[0], w[1]), pack_bf16(w[2], w[3]), pack_bf16(w[4], w[5]), pack_bf16(w[6], w[7]));
+        *reinterpret_cast<uint4*>(p + N * 128 + (chunk << 4)) =
+            make_uint4(pack_bf16_rest(w[0], w[1]), pack_bf16_rest(w[2], w[3]), pack_bf16_rest(w[4], w[5]),
+                       pack_bf16_rest(w[6], w[7]));
+      }
+      fence_proxy_async_smem();
+      mbar_arrive(&bars->p_ready[i & 1]);
+    }
+    if (ok && count > 0) {
+      const int i = count - 1;
+      ok = mbar_wait(&bars->pv_done[i & 1], (i >> 1) & 1, abort_flag, a.status, 98, i);
+    }
+#pragma unroll
+    for (int d = 1; d < kPerHead; d <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+    if (sub == 0) {
+      ref_out[head] = ref;
+      ref_out[N + head] = sum;
+    }
+    ok = softmax_agree(ok);
+    if (ok) {
+      tc_fence_after_sync();
+      for (int b = 0; b < blocks; ++b) {
+        uint32_t r[N];
+        if (count > 0) {
+          tmem_load<N>(r, lane_base + Cfg::kOCol + b * N);
+        } else {
+#pragma unroll
+          for (int h = 0; h < N; ++h) r[h] = 0u;
+        }
+        const int c = b * 128 + quarter * 32 + lane;
+        if (c < a.kv_rank) {
+#pragma unroll
+          for (int h = 0; h < N; ++h) {
+            if (h < nh) {
+              const size_t hh = size_t(t) * a.heads + h0 + h;
+              const float v = __uint_as_float(r[h]), L = ref_out[N + h];
+              if (a.num_splits == 1)
+                a.o_lat[hh * a.kv_rank + c] = from_f32<bf16>(L > 0.f ? v / L : 0.f);
+              else
+                a.scratch[(hh * a.num_splits + split) * (a.kv_rank + 2) + c] = v;
+            }
+          }
+        }
+      }
+      if (a.num_splits > 1 && tid < nh) {
+        float* part = a.scratch + ((size_t(t) * a.heads + h0 + tid) * a.num_splits + split) * (a.kv_rank + 2) + a.kv_rank;
+        part[0] = ref_out[tid];
+        part[1] = ref_out[N + tid];
+      }
+      tc_fence_before_sync();
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 2) tmem_dealloc(tmem, Cfg::kTmemCols);
+}
+
+template <int N>
+int launch_tc(const CUtensorMap& map, const LatentTcArgs& a, int M, cudaStream_t st) {
+  const int panels = (a.used + 63) / 64;
+  const size_t smem = LatentTcCfg<N>::smem(panels);
+  static size_t granted[kMaxDevices] = {};
+  const int slot = current_device_slot();
+  auto kern = latent_tc_kernel<N>;
+  if (smem > granted[slot]) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) != cudaSuccess)
+      return ZSE_ERR_LAUNCH;
+    granted[slot] = smem;
+  }
+  return launch_pdl(kern, dim3((a.heads + N - 1) / N, M, a.num_splits), dim3(kTcThreads), smem, st, map, a) == cudaSuccess
+             ? 0
+             : ZSE_ERR_LAUNCH;
+}
+
+}  // namespace
+
+bool latent_tc_ok(const RowCache& rc, int num_blocks, int used, int kv_rank) {
+  const int panels = (used + 63) / 64;
+  return panels <= kTcMaxPanels && kv_rank % 8 == 0 && kv_rank <= 512 && rc.row % 8 == 0 && num_blocks > 0 &&
+         (rc.block_size == 16 || rc.block_size == 32 || rc.block_size % kTcKeys == 0) &&
+         (kv_rank + 127) / 128 * 2 <= panels + 2 && LatentTcCfg<32>::smem(panels) <= 227 * 1024;
+}
+
+int launch_latent_tc(const bf16* q_lat, const void* rows, const RowCache& rc, int num_blocks, const int* row_seq,
+                     const int* positions, bf16* o_lat, float* scratch, int M, int heads, int used, int kv_rank, int window,
+                     float scale, int num_splits, Status* status, cudaStream_t st) {
+  CUtensorMap map;
+  if (int r = get_tmap_rows3(rows, num_blocks, rc.block_size, rc.row, rc.block_stride,
+                             rc.block_size < kTcKeys ? rc.block_size : kTcKeys, &map))
+    return r;
+  LatentTcArgs a{q_lat, rc, row_seq, positions, o_lat, scratch, heads, used, kv_rank, window, num_splits,
+                 scale * kLog2E, status};
+  return heads <= 16 ? launch_tc<16>(map, a, M, st) : launch_tc<32>(map, a, M, st);
+}
+
+}  // namespace zse

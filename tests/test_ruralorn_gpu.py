@@ -122,15 +122,25 @@ class Layer:
         return out, cu
 
 
-@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.fixture
+def form(ops, request):
+    """The tensor-core form of decode attention that the test runs on."""
+    ops.latent_form, old = request.param, ops.latent_form
+    yield request.param
+    ops.latent_form = old
+
+
+@pytest.mark.parametrize("form,dt", [(1, BF), (2, BF), (0, F32)], indirect=["form"])
 @pytest.mark.parametrize("name", list(SPECS))
-def test_tokens_against_cached_rows(ops, name, dt):
-    L = Layer(ops, SPECS[name], dt)
+@pytest.mark.parametrize("bs", [64, 16, 128])
+def test_tokens_against_cached_rows(ops, name, dt, form, bs):
+    L = Layer(ops, SPECS[name], dt, blocks=40 * 64 // bs, bs=bs, width=12 * 64 // bs)
     L.tables[3, 1] = -1                                 # a hole, inside some windows
     seqs, pos = [0, 1, 2, 3, 4, 5, 5, 0], [0, 1, 63, 150, 64, 700, 511, 199]
     want = torch.stack([L.plain(t, s, p) for t, (s, p) in enumerate(zip(seqs, pos))])
     for splits in (1, 2, 8):
         assert rel(L.tokens(ops, seqs, pos, splits), want) < tol(dt), splits
+    ops.check()
 
 
 @pytest.mark.parametrize("name", [n for n in SPECS if n != "general"])
@@ -147,9 +157,10 @@ def test_chunks_against_expanded_rows(ops, name):
             assert rel(out[t], L.plain(t, s, spans[s][0] + i)) < tol(BF), (s, i)
 
 
-@pytest.mark.parametrize("form,dt", [("tokens", BF), ("tokens", F32), ("chunks", BF)])
+@pytest.mark.parametrize("form,dt,what", [(1, BF, "tokens"), (2, BF, "tokens"), (0, F32, "tokens"), (1, BF, "chunks")],
+                         indirect=["form"])
 @pytest.mark.parametrize("name", ["one-group", "two-groups", "wide"])
-def test_one_loud_key_inside_and_outside_the_window(ops, name, dt, form):
+def test_one_loud_key_inside_and_outside_the_window(ops, name, dt, form, what):
     """A key that takes all the weight sits on the last place that is seen, one before it, far away, on block borders, on
     the token itself and on the next one."""
     spec = SPECS[name]
@@ -166,7 +177,7 @@ def test_one_loud_key_inside_and_outside_the_window(ops, name, dt, form):
             loud = torch.cat([lat[H - 1], q[H - 1, d:]])
             L.row_at(0, key)[: kr + r] = (loud * (60 / spec.scale / loud.pow(2).sum())).to(dt)
             want = L.plain(t, 0, pos)
-            if form == "tokens":
+            if what == "tokens":
                 one = Layer.tokens.__get__(L)
                 L.inp[0] = L.inp[t]
                 got = one(ops, [0], [pos], 2)[0]

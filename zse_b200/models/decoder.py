@@ -296,13 +296,14 @@ class DecoderModel:
     def stage_prefill(self, b: StepBuffers, spans) -> None:
         """Called while a packed pass is staged; ``spans[s] = (start, tokens)`` in the pass's order."""
 
-    def attention_span(self, max_len: int) -> int:
-        """Cached tokens a decoding sequence of ``max_len`` tokens attends to."""
-        return max_len
-
-    def attention_ctas(self) -> int:
-        """CTAs one decoding sequence brings to the attention kernel before its keys are split."""
-        return self.plan.num_kv_heads
+    def attention_splits(self, seqs: int, max_len: int, most: int, sms: int) -> int:
+        """Key splits of a decode step over ``seqs`` sequences of up to ``max_len`` tokens (few distinct values: each is
+        a CUDA graph of its own)."""
+        ctas = seqs * self.plan.num_kv_heads
+        want = (2 * sms + ctas - 1) // ctas
+        by_len = max(1, max_len // 128)              # at least 128 cached tokens per split
+        n = int(max(1, min(want, by_len, most)))
+        return 1 << (n.bit_length() - 1)              # powers of two
 
     # ---- forward --------------------------------------------------------------------------------------
     def _add_norm(self, b: StepBuffers, planes: int, weight: torch.Tensor, M: int, add=None) -> None:

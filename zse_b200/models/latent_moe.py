@@ -37,6 +37,20 @@ SHORT_CHUNK = 16            # chunks up to this length read the cached rows dire
 PLANE_ROWS = 256            # passes up to this size take projections as fp32 split-K planes
 
 
+def attention_splits(seqs: int, groups: int, span: int, most: int, sms: int) -> int:
+    """Key splits of a decode step's attention.  One CTA of it fills an SM, so the time goes with the number of waves
+    each split takes; every split also costs its part of the merge.  A split holds at least two tiles of 64 keys."""
+    best, cost = 1, float("inf")
+    for n in (1, 2, 3, 4, 5, 7, 9, 12, 16):
+        if n > most or (n > 1 and span < 128 * n):
+            break
+        waves = (seqs * groups * n + sms - 1) // sms
+        c = waves / n * (1 + 0.015 * n)
+        if c < cost * 0.98:
+            best, cost = n, c
+    return best
+
+
 @dataclass
 class LatentLayer:
     spec: LatentSpec
@@ -220,11 +234,9 @@ class LatentMoEModel(DecoderModel):
             self._row_views[key] = v
         return v
 
-    def attention_span(self, max_len: int) -> int:
-        return min(max_len, self.max_window) if self.max_window else max_len
-
-    def attention_ctas(self) -> int:
-        return max((L.spec.heads + 31) // 32 for L in self.layers)
+    def attention_splits(self, seqs: int, max_len: int, most: int, sms: int) -> int:
+        span = min(max_len, self.max_window) if self.max_window else max_len
+        return attention_splits(seqs, max((L.spec.heads + 31) // 32 for L in self.layers), span, most, sms)
 
     # ---- layout of a packed pass ----------------------------------------------------------------------
     def pass_order(self, items) -> Optional[List[int]]:

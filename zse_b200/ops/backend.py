@@ -301,11 +301,10 @@ class MoeWorkspace:
         self.act = z(max_tokens * max(s.top * s.ff for s in specs), dtype)
         self.act_shared = z(max_tokens * max(s.shared_ff for s in specs), dtype)
         self.y = z(max(min(max_tokens, self.F32_ROWS) * 4, max_tokens * dtype.itemsize) * per * H, torch.uint8)
-        # router logits: split-K planes of decode-sized passes, one plane otherwise
-        rows = min(max_tokens, 256)
-        self.router = z(max(8 * rows, max_tokens) * E, f32)
-        self.plane_rows = rows
-        self.router_views = {s.experts: self.router[: 8 * rows * s.experts].view(8, rows * s.experts) for s in specs}
+        # router logits in split-K planes: few columns, so the reduction is what fills the GPU
+        self.router = z(8 * max_tokens * E, f32)
+        self.router_views = {s.experts: self.router[: 8 * max_tokens * s.experts].view(8, max_tokens * s.experts)
+                             for s in specs}
 
 
 class CudaOps(TorchOps):
@@ -331,6 +330,7 @@ class CudaOps(TorchOps):
         self._w8_scratch = None
         self._norm_ctx = None
         self._logits16 = None
+        self.latent_form = 1           # decode attention over latent rows: 1 tcgen05 (csrc/latent_tc.cu), 2 mma.sync
         self._no_tables = torch.zeros(1, 1, dtype=torch.int32, device=self.device)
         self.attn_prefill_tc = env.flag("ZSE_ATTN_PREFILL_TC")
 
@@ -560,7 +560,8 @@ class CudaOps(TorchOps):
             if num_splits > 1 and scratch.numel() < M * num_splits * H * (kr + 2):
                 num_splits = 1
             n.latent_absorb(inp, L.uk, q_lat, M, spec)
-            n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, True, self.status.ptr)
+            n.latent_attn(q_lat, rc, row_seq, positions, o_lat, scratch, M, spec, num_splits, self.latent_form,
+                          self.status.ptr)
             n.latent_unabsorb(o_lat, L.uv, self._gate_ptr(inp, spec), inp.stride(0), out, M, spec)
             return
         ql = q_lat[: M * H * spec.row].view(M, H, spec.row)
@@ -591,8 +592,7 @@ class CudaOps(TorchOps):
         n, m, H = self.n, L.moe, x.shape[1]
         dt = x.dtype
         per = m.top + (m.shared_ff > 0)
-        planes = self.linear_partial(L.router, x, M, ws.router_views[m.experts],
-                                     None if M <= ws.plane_rows else 1)
+        planes = self.linear_partial(L.router, x, M, ws.router_views[m.experts])
         slots = M * m.top
         # result rows in fp32 while they are few, in the activations' type for long passes
         y_dt = torch.float32 if M <= ws.F32_ROWS else dt

@@ -157,7 +157,7 @@ def _build_named(out: str, srcs: List[str], extra: tuple, verbose: bool) -> str:
 # Subsets of the library: what one kind of model launches, for a checkout in which nothing has been built yet (a model's
 # first start then waits for these sources only).  The ordinary build contains all of them and is preferred.
 GROUPS = {
-    "latent": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "latent.cu", "moe.cu", "sampling.cu"),
+    "latent": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "latent.cu", "latent_tc.cu", "moe.cu", "sampling.cu"),
 }
 
 

@@ -39,7 +39,7 @@ class TileGemm(Structure):
 
 class RowCache(Structure):
     _fields_ = [("rows", c_void_p), ("block_stride", c_int64), ("block_size", c_int32), ("row", c_int32),
-                ("tables", c_void_p), ("max_blocks", c_int32)]
+                ("tables", c_void_p), ("max_blocks", c_int32), ("num_blocks", c_int32)]
 
 
 class Chunks(Structure):
@@ -546,7 +546,7 @@ def argmax_f32(logits, ld, out, M, V):
 def row_cache(rows, block_tables) -> RowCache:
     """``rows``: a layer's cached rows [blocks, block_size, row] (blocks may be strided)."""
     return RowCache(rows.data_ptr(), rows.stride(0), rows.shape[1], rows.shape[2], block_tables.data_ptr(),
-                    block_tables.stride(0))
+                    block_tables.stride(0), rows.shape[0])
 
 
 def latent_mma_ok(spec) -> bool:

@@ -126,7 +126,7 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
                  chunks: int = 4, only=()) -> List[dict]:
     """Kernels of one layer in a decode step of ``seqs`` sequences of ``ctx`` tokens and in a prefill pass of ``chunks``
     chunks; the dense neighbour's like kernel is named in ``like``."""
-    from ..models.latent_moe import ChunkGroup
+    from ..models.latent_moe import ChunkGroup, attention_splits
     from ..ops.backend import CudaOps, LinearWeight
     ops = CudaOps("cuda")
     c = synth.shape_config(shape)
@@ -193,11 +193,11 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
             scratch = torch.zeros(M * 16 * s.heads * (kr + 2), device="cuda")
             fscratch = torch.zeros(M * nh * 16 * (hd + 2), device="cuda")
             rc = ops.n.row_cache(rows, tables)
-            splits = 4 if s.heads <= 32 else 2
+            splits = attention_splits(M, (s.heads + 31) // 32, ctx, 16, ops.sm_count)
             add(phase, "queries into the latent", "output projection", lambda: ops.n.latent_absorb(inp, L.uk, ql, M, s),
                 2.0 * (s.heads * s.dim * kr + M * hw + M * s.heads * row), 2.0 * M * s.heads * s.dim * kr)
             add(phase, "latent attention (with merge of splits)", "attention (with merge of splits)",
-                lambda: ops.n.latent_attn(ql, rc, None, positions, ol, scratch, M, s, splits, True,
+                lambda: ops.n.latent_attn(ql, rc, None, positions, ol, scratch, M, s, splits, 1,
                                           ops.status.ptr),
                 2.0 * M * (ctx * row + s.heads * (row + kr)), 2.0 * M * ctx * s.heads * (row + kr))
             lens = ii([ctx] * M)
@@ -251,7 +251,7 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
         ops.moe(L, x, M, ws)                               # tables for the single kernels below
         tile = ops.n.moe_tile_rows(M, m.experts, m.top)
         add(phase, "router logits", "output projection",
-            lambda: ops.linear_partial(L.router, x, M, ws.router_views[m.experts], None if dec else 1), *mm(m.experts, H))
+            lambda: ops.linear_partial(L.router, x, M, ws.router_views[m.experts]), *mm(m.experts, H))
         add(phase, "routing + sorted rows", "rotation + cache write",
             lambda: ops.n.moe_route(ws.router, 1, M, m.experts, m.top, tile, x, H, per, ws), 4.0 * M * m.top * H)
         add(phase, "feed-forward (all routed kernels)", "gate/up + down projections", lambda: ops.moe(L, x, M, ws),

@@ -263,12 +263,7 @@ class ModelRunner:
     def _pick_splits(self, S: int, max_len: int) -> int:
         if self.device.type != "cuda":
             return 1
-        ctas = S * self.model.attention_ctas()
-        max_len = self.model.attention_span(max_len)
-        want = (2 * self._sm + ctas - 1) // ctas
-        by_len = max(1, max_len // 128)              # at least 128 cached tokens per split
-        n = int(max(1, min(want, by_len, self.max_attn_splits)))
-        return 1 << (n.bit_length() - 1)              # powers of two: few distinct CUDA graphs as sequences grow
+        return self.model.attention_splits(S, max_len, self.max_attn_splits, self._sm)
 
     def _apply_penalties(self, penalties, n_rows: int) -> None:
         """``penalties[i] = (penalty, {token: count})`` for logits row i (zse-engine/zse_engine/orchestrator/
