@@ -9,9 +9,9 @@
 //
 // Both accumulators live in TMEM.  A tile of 64 keys is a set of 64-column panels with the 128-byte swizzle, each brought by
 // one TMA box per cache block through the block table.  The MMA's 128 rows are more than the 64 keys of a tile: its upper
-// half multiplies whatever follows the panel in shared memory and is never read.  Roles: a TMA producer, an MMA issuer, four
-// softmax warps.  The products of tile i + 1 with the queries run while tile i is weighed; softmax weights are split into two
-// bfloat16 terms; the running maximum is only moved (and O rescaled) when a score exceeds it by more than 2^8.  Every wait is
+// half multiplies whatever follows the panel in shared memory and is never read.  Roles: a TMA producer, one MMA issuer
+// per product, four softmax warps.  The products of tile i + 1 with the queries run while tile i is weighed; softmax weights
+// are split into two bfloat16 terms that stand side by side as columns of P^T (their results are added at the end); the running maximum is only moved (and O rescaled) when a score exceeds it by more than 2^8.  Every wait is
 // bounded and reports through the status word.
 #include <mutex>
 #include <unordered_map>
@@ -26,7 +26,7 @@ namespace {
 constexpr int kTcKeys = 64;
 constexpr int kTcPanelBytes = kTcKeys * 128;
 constexpr int kTcMaxPanels = 9;                 // rows of up to 576 columns
-constexpr int kTcThreads = 256;                 // warp 0 producer, 1 MMA, 2 TMEM, 4..7 softmax
+constexpr int kTcThreads = 256;                 // warp 0 producer, 1 and 3 MMA, 2 TMEM, 4..7 softmax
 constexpr float kTcSlack = 8.f;                 // log2 of how far a score may exceed the reference
 
 struct LatentTcArgs {
@@ -49,8 +49,8 @@ struct LatentTcBars {
 template <int N>
 struct LatentTcCfg {
   static constexpr int kSPitch = kTcKeys + 4;   // floats
-  static constexpr int kTmemCols = N == 16 ? 128 : 256;
-  static constexpr int kOCol = 2 * N;           // O^T blocks after the two S^T buffers
+  static constexpr int kTmemCols = N == 16 ? 256 : 512;
+  static constexpr int kOCol = 2 * N;           // O^T blocks [2 terms of P][N] after two S^T buffers
   __host__ __device__ static int q_bytes(int panels) { return panels * N * 128; }
   __host__ __device__ static size_t smem(int panels) {
     return 1024 + size_t(2) * panels * kTcPanelBytes + q_bytes(panels) + 4 * N * 128 + size_t(N) * kSPitch * 4 +
@@ -187,44 +187,35 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
-      constexpr uint32_t idesc_s = make_idesc_f16(128, N, 1);
-      constexpr uint32_t idesc_o = make_idesc_f16(128, N, 1) | (1u << 15);          // A is MN-major
-      auto weigh = [&](int i) {                                                     // O^T += V^T P^T of tile i
-        const uint32_t kb = smem_u32(sk) + (i & 1) * stage_bytes, pb = smem_u32(sp) + (i & 1) * 2 * N * 128;
-        for (int b = 0; b < blocks; ++b) {
-#pragma unroll
-          for (int j = 0; j < kTcKeys / 16; ++j) {
-            const uint64_t v = make_desc_panel_mn(kb + 2 * b * kTcPanelBytes + j * 2048);
-            umma_ss(tmem + Cfg::kOCol + b * N, v, make_desc_sw128(pb + j * 32), idesc_o, (i | j) != 0);
-            umma_ss(tmem + Cfg::kOCol + b * N, v, make_desc_sw128(pb + N * 128 + j * 32), idesc_o, 1);
-          }
-        }
-        tc_commit(&bars->pv_done[i & 1]);
-      };
-      bool ok = true;
-      for (int i = 0; i < count && ok; ++i) {
-        ok = mbar_wait(&bars->full[i & 1], (i >> 1) & 1, abort_flag, a.status, 92, i);
-        if (!ok) break;
+    if (lane == 0) {                                             // S^T = K Q^T
+      constexpr uint32_t idesc = make_idesc_f16(128, N, 1);
+      for (int i = 0; i < count; ++i) {
+        if (!mbar_wait_spin(&bars->full[i & 1], (i >> 1) & 1, abort_flag, a.status, 92, i)) break;
+        // the scores of tile i - 2 have been read
+        if (i >= 2 && !mbar_wait_spin(&bars->p_ready[i & 1], ((i >> 1) - 1) & 1, abort_flag, a.status, 93, i)) break;
         tc_fence_after_sync();
-        const uint32_t kb = smem_u32(sk) + (i & 1) * stage_bytes, qb = smem_u32(sq);
-        for (int kk = 0; kk < ksteps; ++kk)
-          umma_ss(tmem + (i & 1) * N, make_desc_sw128(kb + (kk >> 2) * kTcPanelBytes + (kk & 3) * 32),
-                  make_desc_sw128(qb + (kk >> 2) * N * 128 + (kk & 3) * 32), idesc_s, kk != 0);
+        const uint64_t k = make_desc_sw128(smem_u32(sk) + (i & 1) * stage_bytes), q = make_desc_sw128(smem_u32(sq));
+#pragma unroll 4
+        for (int kk = 0; kk < ksteps; ++kk)                      // addresses are in units of 16 bytes
+          umma_ss(tmem + (i & 1) * N, k + (kk >> 2) * (kTcPanelBytes / 16) + (kk & 3) * 2,
+                  q + (kk >> 2) * (N * 8) + (kk & 3) * 2, idesc, kk != 0);
         tc_commit(&bars->s_ready[i & 1]);
-        if (i > 0) {
-          ok = mbar_wait(&bars->p_ready[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, a.status, 93, i);
-          if (!ok) break;
-          tc_fence_after_sync();
-          weigh(i - 1);
-        }
       }
-      if (ok && count > 0) {
-        const int i = count - 1;
-        if (mbar_wait(&bars->p_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 94, i)) {
-          tc_fence_after_sync();
-          weigh(i);
-        }
+    }
+  } else if (warp == 3) {
+    if (lane == 0) {                                             // O^T += V^T P^T; both terms of P side by side
+      constexpr uint32_t idesc = make_idesc_f16(128, 2 * N, 1) | (1u << 15);            // A is MN-major
+      for (int i = 0; i < count; ++i) {
+        if (!mbar_wait_spin(&bars->p_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 94, i)) break;
+        if (!mbar_wait_spin(&bars->full[i & 1], (i >> 1) & 1, abort_flag, a.status, 99, i)) break;
+        tc_fence_after_sync();
+        const uint64_t v = make_desc_panel_mn(smem_u32(sk) + (i & 1) * stage_bytes),
+                       p = make_desc_sw128(smem_u32(sp) + (i & 1) * 2 * N * 128);
+        for (int b = 0; b < blocks; ++b)
+#pragma unroll
+          for (int j = 0; j < kTcKeys / 16; ++j)
+            umma_ss(tmem + Cfg::kOCol + b * 2 * N, v + b * (kTcPanelBytes / 8) + j * 128, p + j * 2, idesc, (i | j) != 0);
+        tc_commit(&bars->pv_done[i & 1]);
       }
     }
   } else if (warp >= 4) {
@@ -275,13 +266,13 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
         tc_fence_after_sync();
         for (int b = 0; b < blocks; ++b) {
 #pragma unroll
-          for (int c = 0; c < N; c += 16) {
+          for (int c = 0; c < 2 * N; c += 16) {
             uint32_t r[16];
-            const uint32_t addr = lane_base + Cfg::kOCol + b * N + c;
+            const uint32_t addr = lane_base + Cfg::kOCol + b * 2 * N + c;
             ZSE_TMEM_LD_X16(r, addr);
             tc_wait_ld();
 #pragma unroll
-            for (int e = 0; e < 16; ++e) r[e] = __float_as_uint(__uint_as_float(r[e]) * corr[c + e]);
+            for (int e = 0; e < 16; ++e) r[e] = __float_as_uint(__uint_as_float(r[e]) * corr[(c & (N - 1)) + e]);
             ZSE_TMEM_ST_X16(addr, r);
           }
         }
@@ -328,7 +319,11 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
       for (int b = 0; b < blocks; ++b) {
         uint32_t r[N];
         if (count > 0) {
-          tmem_load<N>(r, lane_base + Cfg::kOCol + b * N);
+          uint32_t rest[N];
+          tmem_load<N>(r, lane_base + Cfg::kOCol + b * 2 * N);
+          tmem_load<N>(rest, lane_base + Cfg::kOCol + b * 2 * N + N);
+#pragma unroll
+          for (int h = 0; h < N; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) + __uint_as_float(rest[h]));
         } else {
 #pragma unroll
           for (int h = 0; h < N; ++h) r[h] = 0u;
