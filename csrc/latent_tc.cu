@@ -130,9 +130,6 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
     tmem_alloc(&bars->tmem_base, Cfg::kTmemCols);
     tmem_relinquish();
   }
-  // a hole is not copied and its weights are 0: what lies there has to be finite
-  for (int i = threadIdx.x; i < 2 * stage_bytes / 16; i += kTcThreads)
-    reinterpret_cast<uint4*>(sk)[i] = make_uint4(0, 0, 0, 0);
   pdl_wait();
   const int h0 = blockIdx.x * N, t = blockIdx.y, split = blockIdx.z;
   const int nh = min(N, a.heads - h0);
@@ -143,7 +140,16 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
   const int per = (n_tiles + a.num_splits - 1) / a.num_splits;
   const int first = tile0 + split * per;
   const int count = max(0, min(tile0 + n_tiles, first + per) - first);
-  const int chunks = a.rc.row / 8;
+  const int chunks = a.rc.row / 8, piece = min(a.rc.block_size, kTcKeys);
+  // keys that are not copied (a hole, what follows the newest token) weigh 0, but what lies in their place has to be finite
+  bool missing = false;
+  for (int i = threadIdx.x; i < count * (kTcKeys / piece); i += kTcThreads) {
+    const int key = first * kTcKeys + i * piece;
+    missing |= key > pos || table[key / a.rc.block_size] < 0;
+  }
+  if (__syncthreads_or(missing))
+    for (int i = threadIdx.x; i < 2 * stage_bytes / 16; i += kTcThreads)
+      reinterpret_cast<uint4*>(sk)[i] = make_uint4(0, 0, 0, 0);
   for (int i = threadIdx.x; i < N * panels * 8; i += kTcThreads) {       // queries; zero beyond the heads and the row
     const int h = i / (panels * 8), c = i % (panels * 8);
     const uint4 v = h < nh && c < chunks
@@ -159,14 +165,13 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
   volatile int* abort_flag = &bars->abort_flag;
 
   if (warp == 0) {
-    const int piece = min(a.rc.block_size, kTcKeys);
     int issued = 0;
     for (int i = 0; i < count; ++i) {
       const int st = i & 1, key0 = (first + i) * kTcKeys;
-      const bool go = i < 2 || mbar_wait(&bars->pv_done[st], ((i >> 1) - 1) & 1, abort_flag, a.status, 91, i);
-      if (!__all_sync(0xffffffffu, go)) break;
-      int blk = -1;
+      int blk = -1;                                              // looked up while the stage is still in use
       if (lane * piece < kTcKeys && key0 + lane * piece <= pos) blk = table[(key0 + lane * piece) / a.rc.block_size];
+      const bool go = i < 2 || mbar_wait_spin(&bars->pv_done[st], ((i >> 1) - 1) & 1, abort_flag, a.status, 91, i);
+      if (!__all_sync(0xffffffffu, go)) break;
       const unsigned have = __ballot_sync(0xffffffffu, blk >= 0);
       if (lane == 0) mbar_arrive_expect_tx(&bars->full[st], __popc(have) * piece * panels * 128);
       __syncwarp();
@@ -226,13 +231,13 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
     float ref = -INFINITY, sum = 0.f;
     bool ok = true;
     for (int i = 0; i < count; ++i) {
-      ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 95, i));
+      const int k = quarter * 32 + lane, key = (first + i) * kTcKeys + k;
+      const bool see = quarter < 2 && key >= lo && key <= pos && table[key / a.rc.block_size] >= 0;
+      ok = __all_sync(0xffffffffu, mbar_wait_spin(&bars->s_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 95, i));
       if (ok && quarter < 2) {                                   // lanes 0..63 of S^T are the tile's keys
         tc_fence_after_sync();
         uint32_t r[N];
         tmem_load<N>(r, lane_base + (i & 1) * N);
-        const int k = quarter * 32 + lane, key = (first + i) * kTcKeys + k;
-        const bool see = key >= lo && key <= pos && table[key / a.rc.block_size] >= 0;
 #pragma unroll
         for (int h = 0; h < N; ++h)
           ss[h * Cfg::kSPitch + k] = see ? __uint_as_float(r[h]) * a.scale_log2 : -INFINITY;
@@ -260,7 +265,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
       if (sub == 0) corr[head] = move ? factor : 1.f;
       const bool rescale = softmax_any(move) && i > 0;
       if (rescale) {                                             // O^T so far is relative to the old references
-        ok = mbar_wait(&bars->pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, a.status, 96, i);
+        ok = mbar_wait_spin(&bars->pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, a.status, 96, i);
         ok = softmax_agree(ok);
         if (!ok) break;
         tc_fence_after_sync();
@@ -279,7 +284,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
         tc_wait_st();
         tc_fence_before_sync();
       } else if (i >= 2) {                                       // the weights of tile i - 2 have been used
-        ok = mbar_wait(&bars->pv_done[i & 1], ((i >> 1) - 1) & 1, abort_flag, a.status, 97, i);
+        ok = mbar_wait_spin(&bars->pv_done[i & 1], ((i >> 1) - 1) & 1, abort_flag, a.status, 97, i);
         ok = softmax_agree(ok);
         if (!ok) break;
       }
