@@ -9,8 +9,8 @@
 //
 // Both accumulators live in TMEM.  A tile of 64 keys is a set of 64-column panels with the 128-byte swizzle, each brought by
 // one TMA box per cache block through the block table.  The MMA's 128 rows are more than the 64 keys of a tile: its upper
-// half multiplies whatever follows the panel in shared memory and is never read.  Roles: a TMA producer, one MMA issuer
-// per product, four softmax warps.  The products of tile i + 1 with the queries run while tile i is weighed; softmax weights
+// half multiplies whatever follows the panel in shared memory and is never read.  Roles: a TMA producer, two MMA
+// issuers for the scores (even and odd k steps, added when they are read) and one for the values, four softmax warps.  The products of tile i + 1 with the queries run while tile i is weighed; softmax weights
 // are split into two bfloat16 terms that stand side by side as columns of P^T (their results are added at the end); the running maximum is only moved (and O rescaled) when a score exceeds it by more than 2^8.  Every wait is
 // bounded and reports through the status word.
 #include <mutex>
@@ -26,7 +26,7 @@ namespace {
 constexpr int kTcKeys = 64;
 constexpr int kTcPanelBytes = kTcKeys * 128;
 constexpr int kTcMaxPanels = 9;                 // rows of up to 576 columns
-constexpr int kTcThreads = 256;                 // warp 0 producer, 1 and 3 MMA, 2 TMEM, 4..7 softmax
+constexpr int kTcThreads = 256;                 // warp 0 producer, 1 and 2 scores, 3 values, 4..7 softmax
 constexpr float kTcSlack = 8.f;                 // log2 of how far a score may exceed the reference
 
 struct LatentTcArgs {
@@ -50,7 +50,7 @@ template <int N>
 struct LatentTcCfg {
   static constexpr int kSPitch = kTcKeys + 4;   // floats
   static constexpr int kTmemCols = N == 16 ? 256 : 512;
-  static constexpr int kOCol = 2 * N;           // O^T blocks [2 terms of P][N] after two S^T buffers
+  static constexpr int kOCol = 4 * N;           // O^T blocks [2 terms of P][N] after two S^T buffers of two parts
   __host__ __device__ static int q_bytes(int panels) { return panels * N * 128; }
   __host__ __device__ static size_t smem(int panels) {
     return 1024 + size_t(2) * panels * kTcPanelBytes + q_bytes(panels) + 4 * N * 128 + size_t(N) * kSPitch * 4 +
@@ -118,7 +118,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; ++i) {
       mbar_init(&bars->full[i], 1);
-      mbar_init(&bars->s_ready[i], 1);
+      mbar_init(&bars->s_ready[i], ksteps > 1 ? 2 : 1);
       mbar_init(&bars->p_ready[i], 128);
       mbar_init(&bars->pv_done[i], 1);
     }
@@ -191,19 +191,19 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
         }
       }
     }
-  } else if (warp == 1) {
-    if (lane == 0) {                                             // S^T = K Q^T
+  } else if (warp == 1 || warp == 2) {
+    if (lane == 0) {                                             // S^T = K Q^T, every other k step each
       constexpr uint32_t idesc = make_idesc_f16(128, N, 1);
-      for (int i = 0; i < count; ++i) {
+      for (int i = 0; i < count && warp - 1 < ksteps; ++i) {
         if (!mbar_wait_spin(&bars->full[i & 1], (i >> 1) & 1, abort_flag, a.status, 92, i)) break;
         // the scores of tile i - 2 have been read
         if (i >= 2 && !mbar_wait_spin(&bars->p_ready[i & 1], ((i >> 1) - 1) & 1, abort_flag, a.status, 93, i)) break;
         tc_fence_after_sync();
         const uint64_t k = make_desc_sw128(smem_u32(sk) + (i & 1) * stage_bytes), q = make_desc_sw128(smem_u32(sq));
 #pragma unroll 4
-        for (int kk = 0; kk < ksteps; ++kk)                      // addresses are in units of 16 bytes
-          umma_ss(tmem + (i & 1) * N, k + (kk >> 2) * (kTcPanelBytes / 16) + (kk & 3) * 2,
-                  q + (kk >> 2) * (N * 8) + (kk & 3) * 2, idesc, kk != 0);
+        for (int kk = warp - 1; kk < ksteps; kk += 2)            // addresses are in units of 16 bytes
+          umma_ss(tmem + (i & 1) * 2 * N + (warp - 1) * N, k + (kk >> 2) * (kTcPanelBytes / 16) + (kk & 3) * 2,
+                  q + (kk >> 2) * (N * 8) + (kk & 3) * 2, idesc, kk > 1);
         tc_commit(&bars->s_ready[i & 1]);
       }
     }
@@ -236,8 +236,13 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
       ok = __all_sync(0xffffffffu, mbar_wait_spin(&bars->s_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 95, i));
       if (ok && quarter < 2) {                                   // lanes 0..63 of S^T are the tile's keys
         tc_fence_after_sync();
-        uint32_t r[N];
-        tmem_load<N>(r, lane_base + (i & 1) * N);
+        uint32_t r[N], odd[N];
+        tmem_load<N>(r, lane_base + (i & 1) * 2 * N);
+        if (ksteps > 1) {
+          tmem_load<N>(odd, lane_base + (i & 1) * 2 * N + N);
+#pragma unroll
+          for (int h = 0; h < N; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) + __uint_as_float(odd[h]));
+        }
 #pragma unroll
         for (int h = 0; h < N; ++h)
           ss[h * Cfg::kSPitch + k] = see ? __uint_as_float(r[h]) * a.scale_log2 : -INFINITY;

@@ -38,15 +38,16 @@ PLANE_ROWS = 256            # passes up to this size take projections as fp32 sp
 
 
 def attention_splits(seqs: int, groups: int, span: int, most: int, sms: int) -> int:
-    """Key splits of a decode step's attention.  One CTA of it fills an SM, so the time goes with the number of waves
-    each split takes; every split also costs its part of the merge.  A split holds at least two tiles of 64 keys."""
+    """Key splits of a decode step's attention.  One CTA of it fills an SM, so the time goes with the number of waves; a
+    wave costs its tiles of 64 keys and about four tiles' time to start and end, every split its part of the merge.  A
+    split holds at least two tiles."""
     best, cost = 1, float("inf")
     for n in (1, 2, 3, 4, 5, 7, 9, 12, 16):
         if n > most or (n > 1 and span < 128 * n):
             break
         waves = (seqs * groups * n + sms - 1) // sms
-        c = waves / n * (1 + 0.015 * n)
-        if c < cost * 0.98:
+        c = waves * (span / 64 / n + 4) + 0.5 * n
+        if c < cost:
             best, cost = n, c
     return best
 

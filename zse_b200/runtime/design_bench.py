@@ -304,3 +304,14 @@ def run(steps: int, warmup: int, shapes=SHAPES, kernels_file: Optional[str] = No
                 f.write(f"## {shape}\n\n{markdown(kernel_table(shape))}\n\n")
                 torch.cuda.empty_cache()
     return out
+
+
+if __name__ == "__main__":       # one or a few kernels, for a profiler: --only takes parts of their names
+    import argparse
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--shape", default=SHAPES[0], choices=SHAPES)
+    ap.add_argument("--only", default="")
+    ap.add_argument("--iters", type=int, default=20)
+    a = ap.parse_args()
+    for row in kernel_table(a.shape, iters=a.iters, only=[x for x in a.only.split(",") if x]):
+        print(row)
