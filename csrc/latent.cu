@@ -23,9 +23,11 @@ struct PrepArgs {
   float eps;
 };
 
-// grid (tokens, 1 + pieces): piece 0 does the latent, the others the queries and (with planes) everything else that later
-// kernels read, kPrepCols columns each.
+// With planes: grid (tokens, 1 + pieces): piece 0 does the latent, the others the queries and everything else that later
+// kernels read, kPrepCols columns each.  Without: one CTA per token, warps 0..3 on the latent, the others on the queries,
+// whose rotated parts turn in place.
 constexpr int kPrepCols = 1024;
+constexpr int kPrepLatent = 128;                 // threads on the latent
 
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -52,19 +54,20 @@ latent_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_
   };
   const float pos = float(positions[t]);
   for (int i = threadIdx.x; i < np; i += blockDim.x) sincosf(pos * freqs[i], &sn[i], &cs[i]);
-  if (blockIdx.y > 0) {
-    __syncthreads();
-    const int c0 = (blockIdx.y - 1) * kPrepCols, qw = a.heads * qk;
-    if (n_planes == 0) {                         // in place: one thread per rotated pair
-      const int i1 = min(a.heads * np, c0 + kPrepCols);
-      for (int i = c0 + threadIdx.x; i < i1; i += blockDim.x) {
-        const int h = i / np, j = i % np, c = h * qk + a.dim + 2 * j;
-        const float u = value(c), v = value(c + 1);
-        in[c] = from_f32<T>(u * cs[j] - v * sn[j]);
-        in[c + 1] = from_f32<T>(v * cs[j] + u * sn[j]);
-      }
-      return;
+  __syncthreads();
+  if (n_planes == 0 && threadIdx.x >= kPrepLatent) {             // one thread per rotated pair
+    const int step = blockDim.x - kPrepLatent, total = a.heads * np;
+#pragma unroll 4
+    for (int i = threadIdx.x - kPrepLatent; i < total; i += step) {
+      const int h = i / np, j = i % np, c = h * qk + a.dim + 2 * j;
+      const float u = to_f32(in[c]), v = to_f32(in[c + 1]);
+      in[c] = from_f32<T>(u * cs[j] - v * sn[j]);
+      in[c + 1] = from_f32<T>(v * cs[j] + u * sn[j]);
     }
+    return;
+  }
+  if (blockIdx.y > 0) {
+    const int c0 = (blockIdx.y - 1) * kPrepCols, qw = a.heads * qk;
 #pragma unroll
     for (int k = 0; k < kPrepCols / 256; ++k) {
       const int i = c0 + threadIdx.x + k * 256;
@@ -81,23 +84,25 @@ latent_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_
     }
     return;
   }
+  if (threadIdx.x >= kPrepLatent) return;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) {
+#pragma unroll 4
+  for (int i = threadIdx.x; i < a.kv_rank; i += kPrepLatent) {
     const float v = value(a.latent_col + i);
     lat[i] = v;
     ss += v * v;
   }
   ss = warp_sum(ss);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  const float total = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
+  asm volatile("bar.sync 1, %0;" ::"n"(kPrepLatent) : "memory");
+  const float total = warp_sum((threadIdx.x & 31) < kPrepLatent / 32 ? red[threadIdx.x & 31] : 0.f);
   const float inv = 1.f / sqrtf(total / float(a.kv_rank) + a.eps);
   const long long slot = slots[t];
   if (slot < 0) return;
   T* dst = cache + (slot / rc.block_size) * rc.block_stride + (slot % rc.block_size) * rc.row;
-  for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) dst[i] = from_f32<T>(lat[i] * inv * to_f32(norm_w[i]));
+  for (int i = threadIdx.x; i < a.kv_rank; i += kPrepLatent) dst[i] = from_f32<T>(lat[i] * inv * to_f32(norm_w[i]));
   const int r0 = a.latent_col + a.kv_rank;
-  for (int j = threadIdx.x; j < a.rot; j += blockDim.x) {
+  for (int j = threadIdx.x; j < a.rot; j += kPrepLatent) {
     float v = value(r0 + j);
     if (j < a.rot_dims) v = v * cs[j >> 1] + ((j & 1) ? value(r0 + j - 1) : -value(r0 + j + 1)) * sn[j >> 1];
     dst[a.kv_rank + j] = from_f32<T>(v);
@@ -344,7 +349,7 @@ latent_attn_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ cach
 #pragma unroll
         for (int w = 0; w < kMaxParts; ++w) mn = fmaxf(mn, smax[w * kRows + a * 16 + rq + half * 8]);
         const float base = mn == -INFINITY ? 0.f : mn;
-        corr[a][half] = exp2f(m[a][half] - base);                // 0 when there was nothing before
+        corr[a][half] = ex2(m[a][half] - base);                // 0 when there was nothing before
         moved |= mn > m[a][half];
         m[a][half] = mn;
       }
@@ -358,7 +363,7 @@ latent_attn_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ cach
       const int r = tile_row + rq + half * 8;
 #pragma unroll
       for (int nb = 0; nb < MT; ++nb) {
-        const float p0 = exp2f(s[0][nb][half * 2] - base), p1 = exp2f(s[0][nb][half * 2 + 1] - base);
+        const float p0 = ex2(s[0][nb][half * 2] - base), p1 = ex2(s[0][nb][half * 2 + 1] - base);
         l[half] += p0 + p1;
         const int key = key_w + nb * 8 + cq;
         *reinterpret_cast<uint32_t*>(sp + r * kPPitch + key * 2) = pack_bf16(p0, p1);
@@ -672,12 +677,15 @@ latent_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict
     if (qch < ksteps * 2) *reinterpret_cast<uint4*>(sk + r * qp + qch * 16) = make_uint4(0, 0, 0, 0);
     for (int c = vch; c * 16 < vp; ++c) *reinterpret_cast<uint4*>(sv + r * vp + c * 16) = make_uint4(0, 0, 0, 0);
   }
+  bool whole[2] = {true, true};                  // this thread's key of the stage exists
   auto issue = [&](int i) {
     if (i < count) {
       const int st = i & 1, key0 = k_begin + i * kChKeys;
       if (threadIdx.x < kChKeys) {
         const int p = key0 + threadIdx.x;
-        valid[st * kChKeys + threadIdx.x] = p < k_end && table[p / rc.block_size] >= 0;
+        const bool v = p < k_end && table[p / rc.block_size] >= 0;
+        valid[st * kChKeys + threadIdx.x] = v;
+        if (st == 0) whole[0] = v; else whole[1] = v;
       }
       // a warp takes 16 rows; a lane keeps its 16-byte columns, so its addresses only move by whole rows
       const int rows = min(kChKeys, k_end - key0);
@@ -712,7 +720,7 @@ latent_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict
   for (int i = 0; i < count; ++i) {
     issue(i + 1);
     cpa_wait<1>();
-    __syncthreads();
+    const bool all_there = __syncthreads_and((i & 1) == 0 ? whole[0] : whole[1]) != 0;
     const uint32_t kb = smem_u32(sk + (i & 1) * kChKeys * qp), vb = smem_u32(sv + (i & 1) * kChKeys * vp);
     float sc[8][4];
 #pragma unroll
@@ -731,6 +739,16 @@ latent_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict
     }
     const int key0 = k_begin + i * kChKeys;
     float x[2] = {-INFINITY, -INFINITY};
+    if (all_there && key0 + kChKeys - 1 <= p_first && (g.window <= 0 || p_last - key0 < g.window)) {
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {              // every query sees every key
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sc[n][e] *= scale_log2;
+          x[e >> 1] = fmaxf(x[e >> 1], sc[n][e]);
+        }
+      }
+    } else
 #pragma unroll
     for (int n = 0; n < 8; ++n) {
 #pragma unroll
@@ -748,7 +766,7 @@ latent_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict
       x[half] = fmaxf(x[half], __shfl_xor_sync(0xffffffffu, x[half], 2));
       const float mn = fmaxf(m[half], x[half]);
       base[half] = mn == -INFINITY ? 0.f : mn;
-      const float corr = exp2f(m[half] - base[half]);
+      const float corr = ex2(m[half] - base[half]);
       m[half] = mn;
       l[half] *= corr;
 #pragma unroll
@@ -764,7 +782,7 @@ latent_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict
       for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          p[j][e] = exp2f(sc[2 * kk + j][e] - base[e >> 1]);
+          p[j][e] = ex2(sc[2 * kk + j][e] - base[e >> 1]);
           l[e >> 1] += p[j][e];
         }
       const uint32_t ph[4] = {pack_bf16(p[0][0], p[0][1]), pack_bf16(p[0][2], p[0][3]), pack_bf16(p[1][0], p[1][1]),
@@ -861,8 +879,8 @@ extern "C" int zse_latent_prep(int dtype, void* inp, int ld, const void* planes,
   const PrepArgs a{ld, heads, dim, rot, rot_dims, kv_rank, latent_col, gate_col, gate_w, eps};
   const size_t smem = size_t(rot_dims + kv_rank) * sizeof(float);
   if (smem > 48 * 1024) return ZSE_ERR_LIMIT;
-  const int work = n_planes > 0 ? heads * (dim + rot) + gate_w : heads * (rot_dims / 2);
-  const dim3 grid(M, 1 + (work + kPrepCols - 1) / kPrepCols), block(n_planes > 0 ? 256 : 128);
+  const int work = n_planes > 0 ? heads * (dim + rot) + gate_w : 0;
+  const dim3 grid(M, 1 + (work + kPrepCols - 1) / kPrepCols), block(256);
   cudaError_t e;
   if (dtype == kBF16)
     e = launch_pdl(latent_prep_kernel<bf16>, grid, block, smem, ST(stream), reinterpret_cast<bf16*>(inp),

@@ -300,7 +300,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
         float w[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-          w[e] = exp2f(s[c + e] - base);
+          w[e] = ex2(s[c + e] - base);
           sum += w[e];
         }
         const int chunk = ((sub * kMine + c) >> 3) ^ (head & 7);

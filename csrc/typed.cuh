@@ -21,6 +21,13 @@ __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat1
 __device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float gelu_exact(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
+// 2^x on the special-function unit: softmax weights need no more than its fp32 accuracy, and no range handling around it
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<uint32_t*>(&h);
