@@ -264,36 +264,37 @@ int get_tmap(const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows, C
   return 0;
 }
 
-int get_tmap_rows3(const void* ptr, int blocks, int block_size, int row, long long block_stride, int box_rows,
+int get_tmap_rows3(const void* ptr, int blocks, int block_size, int row, long long block_stride, int box_rows, int panels,
                    CUtensorMap* out) {
-  struct Key {
-    const void* ptr;
-    int blocks, block_size, row, box_rows;
-    long long block_stride;
-  };
-  static std::unordered_map<MapKey, std::pair<Key, CUtensorMap>, MapKeyHash> cache;
+  static std::unordered_map<MapKey, std::pair<long long, CUtensorMap>, MapKeyHash> cache;      // with the block stride
   static std::mutex mu;
-  const MapKey hash{ptr, uint64_t(blocks), uint64_t(block_size) * 65536 + row, uint32_t(box_rows)};
+  const MapKey hash{ptr, uint64_t(blocks), uint64_t(block_size) * 65536 + row, uint32_t(box_rows + panels * 256)};
   std::lock_guard<std::mutex> g(mu);
   auto it = cache.find(hash);
-  if (it != cache.end() && it->second.first.block_stride == block_stride) {
+  if (it != cache.end() && it->second.first == block_stride) {
     *out = it->second.second;
     return 0;
   }
   EncodeTiledFn fn = encode_fn();
   if (fn == nullptr) return ZSE_ERR_DRIVER;
   if ((reinterpret_cast<uintptr_t>(ptr) & 15) || (row * 2) % 16 || (block_stride * 2) % 16) return ZSE_ERR_ALIGN;
-  cuuint64_t dims[3] = {cuuint64_t(row), cuuint64_t(block_size), cuuint64_t(blocks)};
-  cuuint64_t strides[2] = {cuuint64_t(row) * 2, cuuint64_t(block_stride) * 2};
-  cuuint32_t box[3] = {64, cuuint32_t(box_rows), 1};
-  cuuint32_t estr[3] = {1, 1, 1};
+  if (panels * 64 > row) return ZSE_ERR_SHAPE;
+  cuuint64_t dims[4] = {cuuint64_t(row), cuuint64_t(block_size), cuuint64_t(blocks), 1};
+  cuuint64_t strides[3] = {cuuint64_t(row) * 2, cuuint64_t(block_stride) * 2, 0};
+  cuuint32_t box[4] = {64, cuuint32_t(box_rows), 1, 1};
+  cuuint32_t estr[4] = {1, 1, 1, 1};
+  if (panels > 0) {
+    dims[0] = 64, dims[2] = cuuint64_t(panels), dims[3] = cuuint64_t(blocks);
+    strides[1] = 128, strides[2] = cuuint64_t(block_stride) * 2;
+    box[2] = cuuint32_t(panels);
+  }
   CUtensorMap m;
-  if (fn(&m, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
+  if (fn(&m, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, panels > 0 ? 4 : 3, const_cast<void*>(ptr), dims, strides, box, estr,
          CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
          CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
     return ZSE_ERR_DRIVER;
   if (cache.size() > 1024) cache.clear();
-  cache[hash] = {Key{ptr, blocks, block_size, row, box_rows, block_stride}, m};
+  cache[hash] = {block_stride, m};
   *out = m;
   return 0;
 }

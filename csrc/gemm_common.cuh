@@ -32,8 +32,9 @@ struct GemmArgs {
 int get_tmap(const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows, CUtensorMap* out);
 
 // 16-bit rows in blocks, [blocks][block_size][row] with `block_stride` elements between blocks: box = 64 columns x box_rows
-// rows of one block, 128-byte swizzle, zero fill out of bounds; cached.  Defined in gemm.cu.
-int get_tmap_rows3(const void* ptr, int blocks, int block_size, int row, long long block_stride, int box_rows,
+// rows of one block, 128-byte swizzle, zero fill out of bounds; cached.  With panels > 0 a box holds that many neighbouring
+// panels of 64 columns, one after the other (coordinates: column in the panel, row, panel, block).  Defined in gemm.cu.
+int get_tmap_rows3(const void* ptr, int blocks, int block_size, int row, long long block_stride, int box_rows, int panels,
                    CUtensorMap* out);
 
 // Where a row-parallel GEMM sends its partial output tiles when the tensor-parallel exchange is part of the GEMM

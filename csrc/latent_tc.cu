@@ -26,7 +26,7 @@ namespace {
 constexpr int kTcKeys = 64;
 constexpr int kTcPanelBytes = kTcKeys * 128;
 constexpr int kTcMaxPanels = 9;                 // rows of up to 576 columns
-constexpr int kTcThreads = 256;                 // warp 0 producer, 1 and 2 scores, 3 values, 4..7 softmax
+constexpr int kTcThreads = 288;                 // warp 0 producer, 1 and 2 scores, 3 and 8 values, 4..7 softmax
 constexpr float kTcSlack = 8.f;                 // log2 of how far a score may exceed the reference
 
 struct LatentTcArgs {
@@ -37,11 +37,12 @@ struct LatentTcArgs {
   float* scratch;
   int heads, used, kv_rank, window, num_splits;
   float scale_log2;
+  int one_box;                                  // a block's piece of a tile is one TMA box (all panels)
   Status* status;
 };
 
 struct LatentTcBars {
-  uint64_t full[2], s_ready[2], p_ready[2], pv_done[2];
+  uint64_t full[2], s_ready[2], p_ready[2], pv_done[2], q_ready;
   uint32_t tmem_base;
   int abort_flag;
 };
@@ -63,6 +64,13 @@ __device__ __forceinline__ void tma_load_3d(void* dst, const void* map, int x, i
       "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(
           smem_u32(dst)),
       "l"(map), "r"(x), "r"(y), "r"(z), "r"(smem_u32(bar))
+      : "memory");
+}
+__device__ __forceinline__ void tma_load_4d(void* dst, const void* map, int x, int y, int p, int z, uint64_t* bar) {
+  asm volatile(
+      "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5}], [%6];" ::"r"(
+          smem_u32(dst)),
+      "l"(map), "r"(x), "r"(y), "r"(p), "r"(z), "r"(smem_u32(bar))
       : "memory");
 }
 // MN-major operand, 128-byte swizzle: rows of the K dimension hold 64 MN elements, eight rows per 1024 bytes, the next 64 MN
@@ -120,8 +128,9 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
       mbar_init(&bars->full[i], 1);
       mbar_init(&bars->s_ready[i], ksteps > 1 ? 2 : 1);
       mbar_init(&bars->p_ready[i], 128);
-      mbar_init(&bars->pv_done[i], 1);
+      mbar_init(&bars->pv_done[i], blocks > 1 ? 2 : 1);
     }
+    mbar_init(&bars->q_ready, 128);
     bars->abort_flag = 0;
     mbar_fence_init();
     prefetch_tmap(&map);
@@ -130,6 +139,11 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
     tmem_alloc(&bars->tmem_base, Cfg::kTmemCols);
     tmem_relinquish();
   }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem = bars->tmem_base;
+  volatile int* abort_flag = &bars->abort_flag;
   pdl_wait();
   const int h0 = blockIdx.x * N, t = blockIdx.y, split = blockIdx.z;
   const int nh = min(N, a.heads - h0);
@@ -140,31 +154,20 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
   const int per = (n_tiles + a.num_splits - 1) / a.num_splits;
   const int first = tile0 + split * per;
   const int count = max(0, min(tile0 + n_tiles, first + per) - first);
-  const int chunks = a.rc.row / 8, piece = min(a.rc.block_size, kTcKeys);
-  // keys that are not copied (a hole, what follows the newest token) weigh 0, but what lies in their place has to be finite
-  bool missing = false;
-  for (int i = threadIdx.x; i < count * (kTcKeys / piece); i += kTcThreads) {
-    const int key = first * kTcKeys + i * piece;
-    missing |= key > pos || table[key / a.rc.block_size] < 0;
-  }
-  if (__syncthreads_or(missing))
-    for (int i = threadIdx.x; i < 2 * stage_bytes / 16; i += kTcThreads)
-      reinterpret_cast<uint4*>(sk)[i] = make_uint4(0, 0, 0, 0);
-  for (int i = threadIdx.x; i < N * panels * 8; i += kTcThreads) {       // queries; zero beyond the heads and the row
-    const int h = i / (panels * 8), c = i % (panels * 8);
-    const uint4 v = h < nh && c < chunks
-                        ? reinterpret_cast<const uint4*>(a.q_lat + (size_t(t) * a.heads + h0 + h) * a.rc.row)[c]
-                        : make_uint4(0, 0, 0, 0);
-    *reinterpret_cast<uint4*>(sq + (c >> 3) * N * 128 + h * 128 + (((c & 7) ^ (h & 7)) << 4)) = v;
-  }
-  fence_proxy_async_smem();
-  tc_fence_before_sync();
-  __syncthreads();
-  tc_fence_after_sync();
-  const uint32_t tmem = bars->tmem_base;
-  volatile int* abort_flag = &bars->abort_flag;
+  const int piece = min(a.rc.block_size, kTcKeys);
 
   if (warp == 0) {
+    // keys that are not copied (a hole, what follows the newest token) weigh 0, but what lies in their place has to be finite
+    bool missing = false;
+    for (int i = lane; i < count * (kTcKeys / piece); i += 32) {
+      const int key = first * kTcKeys + i * piece;
+      missing |= key > pos || table[key / a.rc.block_size] < 0;
+    }
+    if (__any_sync(0xffffffffu, missing)) {
+      for (int i = lane; i < 2 * stage_bytes / 16; i += 32) reinterpret_cast<uint4*>(sk)[i] = make_uint4(0, 0, 0, 0);
+      fence_proxy_async_smem();
+      __syncwarp();
+    }
     int issued = 0;
     for (int i = 0; i < count; ++i) {
       const int st = i & 1, key0 = (first + i) * kTcKeys;
@@ -175,12 +178,16 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
       const unsigned have = __ballot_sync(0xffffffffu, blk >= 0);
       if (lane == 0) mbar_arrive_expect_tx(&bars->full[st], __popc(have) * piece * panels * 128);
       __syncwarp();
-      // lane p brings panel p of every block
-      for (int j = 0; j * piece < kTcKeys; ++j) {
-        const int b = __shfl_sync(0xffffffffu, blk, j);
-        if (b >= 0 && lane < panels)
-          tma_load_3d(sk + st * stage_bytes + lane * kTcPanelBytes + j * piece * 128, &map, lane * 64,
-                      (key0 + j * piece) % a.rc.block_size, b, &bars->full[st]);
+      if (a.one_box) {                                           // a whole block's tile: lane 0 only (piece = tile)
+        if (blk >= 0)
+          tma_load_4d(sk + st * stage_bytes, &map, 0, key0 % a.rc.block_size, 0, blk, &bars->full[st]);
+      } else {
+        for (int j = 0; j * piece < kTcKeys; ++j) {              // lane p brings panel p of every block
+          const int b = __shfl_sync(0xffffffffu, blk, j);
+          if (b >= 0 && lane < panels)
+            tma_load_3d(sk + st * stage_bytes + lane * kTcPanelBytes + j * piece * 128, &map, lane * 64,
+                        (key0 + j * piece) % a.rc.block_size, b, &bars->full[st]);
+        }
       }
       issued = i + 1;
     }
@@ -194,7 +201,8 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
   } else if (warp == 1 || warp == 2) {
     if (lane == 0) {                                             // S^T = K Q^T, every other k step each
       constexpr uint32_t idesc = make_idesc_f16(128, N, 1);
-      for (int i = 0; i < count && warp - 1 < ksteps; ++i) {
+      const bool go = mbar_wait_spin(&bars->q_ready, 0, abort_flag, a.status, 90, 0);
+      for (int i = 0; go && i < count && warp - 1 < ksteps; ++i) {
         if (!mbar_wait_spin(&bars->full[i & 1], (i >> 1) & 1, abort_flag, a.status, 92, i)) break;
         // the scores of tile i - 2 have been read
         if (i >= 2 && !mbar_wait_spin(&bars->p_ready[i & 1], ((i >> 1) - 1) & 1, abort_flag, a.status, 93, i)) break;
@@ -207,8 +215,9 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
         tc_commit(&bars->s_ready[i & 1]);
       }
     }
-  } else if (warp == 3) {
-    if (lane == 0) {                                             // O^T += V^T P^T; both terms of P side by side
+  } else if (warp == 3 || warp == 8) {
+    const int half = warp == 3 ? 0 : 1;                          // every other block of 128 latent columns
+    if (lane == 0 && half < blocks) {                            // O^T += V^T P^T; both terms of P side by side
       constexpr uint32_t idesc = make_idesc_f16(128, 2 * N, 1) | (1u << 15);            // A is MN-major
       for (int i = 0; i < count; ++i) {
         if (!mbar_wait_spin(&bars->p_ready[i & 1], (i >> 1) & 1, abort_flag, a.status, 94, i)) break;
@@ -216,7 +225,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
         tc_fence_after_sync();
         const uint64_t v = make_desc_panel_mn(smem_u32(sk) + (i & 1) * stage_bytes),
                        p = make_desc_sw128(smem_u32(sp) + (i & 1) * 2 * N * 128);
-        for (int b = 0; b < blocks; ++b)
+        for (int b = half; b < blocks; b += 2)
 #pragma unroll
           for (int j = 0; j < kTcKeys / 16; ++j)
             umma_ss(tmem + Cfg::kOCol + b * 2 * N, v + b * (kTcPanelBytes / 8) + j * 128, p + j * 2, idesc, (i | j) != 0);
@@ -228,6 +237,20 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
     const int tid = threadIdx.x - 128, quarter = warp & 3;
     const int head = tid / kPerHead, sub = tid % kPerHead;
     const uint32_t lane_base = tmem + (uint32_t(quarter * 32) << 16);
+    const int chunks = a.rc.row / 8;
+    for (int h = tid >> 3; h < N; h += 16) {                     // queries; zero beyond the heads and the row
+      const uint4* src = reinterpret_cast<const uint4*>(a.q_lat + (size_t(t) * a.heads + h0 + min(h, nh - 1)) * a.rc.row);
+      const int c0 = tid & 7;
+#pragma unroll
+      for (int p = 0; p < kTcMaxPanels; ++p) {
+        const int c = p * 8 + c0;
+        if (p < panels)
+          *reinterpret_cast<uint4*>(sq + p * N * 128 + h * 128 + ((c0 ^ (h & 7)) << 4)) =
+              h < nh && c < chunks ? src[c] : make_uint4(0, 0, 0, 0);
+      }
+    }
+    fence_proxy_async_smem();
+    mbar_arrive(&bars->q_ready);
     float ref = -INFINITY, sum = 0.f;
     bool ok = true;
     for (int i = 0; i < count; ++i) {
@@ -321,44 +344,48 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentTcArgs a) 
     for (int d = 1; d < kPerHead; d <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
     if (sub == 0) {
       ref_out[head] = ref;
-      ref_out[N + head] = sum;
+      ref_out[N + head] = a.num_splits > 1 ? sum : sum > 0.f ? 1.f / sum : 0.f;
     }
-    ok = softmax_agree(ok);
-    if (ok) {
-      tc_fence_after_sync();
-      for (int b = 0; b < blocks; ++b) {
-        uint32_t r[N];
-        if (count > 0) {
-          uint32_t rest[N];
-          tmem_load<N>(r, lane_base + Cfg::kOCol + b * 2 * N);
-          tmem_load<N>(rest, lane_base + Cfg::kOCol + b * 2 * N + N);
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (*abort_flag == 0 && warp < 8) {            // eight warps write the blocks: two for each quarter of the lanes
+    tc_fence_after_sync();
+    const int quarter = warp & 3;
+    const size_t hh0 = size_t(t) * a.heads + h0;
+    for (int b = warp >> 2; b < blocks; b += 2) {
+      uint32_t r[N];
+      if (count > 0) {
+        uint32_t rest[N];
+        const uint32_t addr = tmem + (uint32_t(quarter * 32) << 16) + Cfg::kOCol + b * 2 * N;
+        tmem_load<N>(r, addr);
+        tmem_load<N>(rest, addr + N);
 #pragma unroll
-          for (int h = 0; h < N; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) + __uint_as_float(rest[h]));
+        for (int h = 0; h < N; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) + __uint_as_float(rest[h]));
+      } else {
+#pragma unroll
+        for (int h = 0; h < N; ++h) r[h] = 0u;
+      }
+      const int c = b * 128 + quarter * 32 + lane;
+      if (c < a.kv_rank) {
+        if (a.num_splits == 1) {
+          bf16* out = a.o_lat + hh0 * a.kv_rank + c;
+#pragma unroll
+          for (int h = 0; h < N; ++h)
+            if (h < nh) out[size_t(h) * a.kv_rank] = from_f32<bf16>(__uint_as_float(r[h]) * ref_out[N + h]);
         } else {
+          const int step = a.num_splits * (a.kv_rank + 2);
+          float* out = a.scratch + (hh0 * a.num_splits + split) * (a.kv_rank + 2) + c;
 #pragma unroll
-          for (int h = 0; h < N; ++h) r[h] = 0u;
-        }
-        const int c = b * 128 + quarter * 32 + lane;
-        if (c < a.kv_rank) {
-#pragma unroll
-          for (int h = 0; h < N; ++h) {
-            if (h < nh) {
-              const size_t hh = size_t(t) * a.heads + h0 + h;
-              const float v = __uint_as_float(r[h]), L = ref_out[N + h];
-              if (a.num_splits == 1)
-                a.o_lat[hh * a.kv_rank + c] = from_f32<bf16>(L > 0.f ? v / L : 0.f);
-              else
-                a.scratch[(hh * a.num_splits + split) * (a.kv_rank + 2) + c] = v;
-            }
-          }
+          for (int h = 0; h < N; ++h)
+            if (h < nh) out[size_t(h) * step] = __uint_as_float(r[h]);
         }
       }
-      if (a.num_splits > 1 && tid < nh) {
-        float* part = a.scratch + ((size_t(t) * a.heads + h0 + tid) * a.num_splits + split) * (a.kv_rank + 2) + a.kv_rank;
-        part[0] = ref_out[tid];
-        part[1] = ref_out[N + tid];
-      }
-      tc_fence_before_sync();
+    }
+    if (a.num_splits > 1 && int(threadIdx.x) < nh) {
+      float* part = a.scratch + ((hh0 + threadIdx.x) * a.num_splits + split) * (a.kv_rank + 2) + a.kv_rank;
+      part[0] = ref_out[threadIdx.x];
+      part[1] = ref_out[N + threadIdx.x];
     }
   }
   tc_fence_before_sync();
@@ -396,11 +423,14 @@ int launch_latent_tc(const bf16* q_lat, const void* rows, const RowCache& rc, in
                      const int* positions, bf16* o_lat, float* scratch, int M, int heads, int used, int kv_rank, int window,
                      float scale, int num_splits, Status* status, cudaStream_t st) {
   CUtensorMap map;
+  // all panels in one box where they are whole (nothing past a row's end is touched) and a tile lies in one block
+  const int panels = (used + 63) / 64;
+  const bool one_box = used % 64 == 0 && rc.block_size % kTcKeys == 0;
   if (int r = get_tmap_rows3(rows, num_blocks, rc.block_size, rc.row, rc.block_stride,
-                             rc.block_size < kTcKeys ? rc.block_size : kTcKeys, &map))
+                             rc.block_size < kTcKeys ? rc.block_size : kTcKeys, one_box ? panels : 0, &map))
     return r;
   LatentTcArgs a{q_lat, rc, row_seq, positions, o_lat, scratch, heads, used, kv_rank, window, num_splits,
-                 scale * kLog2E, status};
+                 scale * kLog2E, one_box, status};
   return heads <= 16 ? launch_tc<16>(map, a, M, st) : launch_tc<32>(map, a, M, st);
 }
 
