@@ -31,7 +31,7 @@ def _cmd_serve(a) -> int:
                                 max_batch_seqs=a.max_batch_seqs, prefill_chunk_size=a.prefill_chunk_size,
                                 speculative_k=a.speculative_k, speculative_mode=a.speculative_mode,
                                 use_cuda_graphs=not a.no_graphs, comm_backend=a.comm, quiet=a.quiet,
-                                dtype=a.dtype, device="cpu" if a.cpu else None)
+                                dtype=getattr(a, "dtype", None), device="cpu" if a.cpu else None)
     server = ZSEServer(a.model, a.host, a.port, a.admin_key, a.db_path, a.model_name, a.quiet, a.tp_size,
                        engine_config=cfg, require_auth=a.require_auth)
     loop = asyncio.new_event_loop()
