@@ -4,14 +4,14 @@
 
 Steps come from standard input, one JSON object a line:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["a"]}
+    {"step": 7, "entries": [{"id": "chat-1", "tokens": [901, 44], "want": [1]}], "end": ["chat-1"]}
 
-``entries`` holds the next tokens of each request and the places among them whose logits are wanted; ``end`` names the
-requests that give back what they hold after the step.  All entries of a step are one batch of the engine's runner
-(``ModelRunner.run_batch``), over the engine's own cache.  The logits of a step are written to ``DIR/<step>.f32`` (little-
-endian fp32, [wanted, vocab]); ``done <step>`` follows on standard output.  Nothing is sampled.
+An entry continues (or starts) a request by its tokens; ``want`` picks the places among them whose logits the caller needs.
+Requests named in ``end`` free their cache blocks once the step has run.  A step is one call of ``ModelRunner.run_batch`` on
+the engine's cache, whatever mixture of prompt portions and single tokens it carries.  Its logits go to ``DIR/<step>.f32``
+(little-endian fp32, one row of the vocabulary per wanted place), then ``done <step>`` is printed.  No token is chosen.
 
-The cache holds ``--max-tokens`` tokens (the most that live requests have at any time, each rounded up to a block).
+``--max-tokens`` sizes the cache: the sum of the live requests' tokens at its peak, each counted in whole blocks of 64.
 """
 from __future__ import annotations
 
