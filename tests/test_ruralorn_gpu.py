@@ -45,6 +45,8 @@ SPECS = {
     "two-groups": LatentSpec(18, 64, 32, 64, 192, 300, 0.12, 32, 1e4),
     "wide": LatentSpec(48, 128, 64, 128, 512, 700, 0.072, 64, 1e4),
     "wide-values": LatentSpec(3, 32, 16, 144, 344, 129, 0.14, 8, 1e4),
+    "long-row": LatentSpec(20, 32, 128, 32, 512, 200, 0.08, 128, 1e4),       # more than the tcgen05 form's nine panels
+    "smallest": LatentSpec(1, 8, 8, 8, 8, 3, 0.3, 8, 1e2),
     "no-window": LatentSpec(4, 16, 16, 24, 128, 0, 0.2, 16, 1e4),
     "general": LatentSpec(3, 10, 6, 7, 22, 50, 0.4, 4, 1e3),
 }
