@@ -24,6 +24,7 @@ from .block_pool import BlockPool
 from .dedup import BlockDedup
 from .evictor import Evictor
 from .page_table import PageTable
+from .state_slots import StateSlots
 
 
 @dataclass
@@ -56,7 +57,8 @@ class CacheStats:
 class KVCacheManager:
     def __init__(self, config: ModelConfig, device=None, budget_bytes: int = 0, block_size: int = 0,
                  eviction_policy: str = "smart", enable_dedup: bool = True, num_kv_heads: Optional[int] = None,
-                 num_blocks: int = 0, dtype=None):
+                 num_blocks: int = 0, dtype=None, state_slots: int = 0):
+        """``state_slots``: sequences that may hold recurrent state at the same time (models that keep any)."""
         self._config = config
         self._lock = threading.RLock()
         self._block_size = block_size if block_size > 0 else self._auto_block_size(config)
@@ -66,16 +68,19 @@ class KVCacheManager:
         nkv, pool_hd = config.kv_pool_dims(num_kv_heads)
         kind = dict(planes=config.kv_planes, dtype=dtype or torch.float16)
         if num_blocks > 0:
-            self._pool = BlockPool(num_blocks, self._block_size, config.num_layers, nkv, pool_hd, device, **kind)
+            self._pool = BlockPool(num_blocks, self._block_size, config.num_cache_layers, nkv, pool_hd, device, **kind)
         else:
             if budget_bytes <= 0:
                 raise ValueError("either budget_bytes or num_blocks is required")
-            self._pool = BlockPool.from_budget(budget_bytes, self._block_size, config.num_layers, nkv,
+            self._pool = BlockPool.from_budget(budget_bytes, self._block_size, config.num_cache_layers, nkv,
                                                pool_hd, device, **kind)
-        # a window that bounds every layer (Mistral) lets old blocks go; models that mix local and global layers keep
-        # everything and apply the window inside attention
-        self._window = config.cache_window
-        self._windowed = self._window > 0
+        # a window or chunk that bounds every layer (Mistral) lets old blocks go; models that mix local and global layers
+        # keep everything and apply the window inside attention
+        self._windowed = config.first_seen(1 << 30) > 0
+        self.states: Optional[StateSlots] = None
+        if config.keeps_state:
+            self.states = StateSlots(state_slots or 64, config.state_floats, device)
+            enable_dedup = False         # a shared prefix has no recurrent state to start from
         self._page_table = PageTable(self._pool)
         self._evictor = Evictor(eviction_policy)
         self._dedup = BlockDedup(self._pool) if enable_dedup else None
@@ -88,7 +93,7 @@ class KVCacheManager:
     @staticmethod
     def _auto_block_size(config: ModelConfig) -> int:
         """<= 4096 context: 16; <= 32768: 32; longer: 64; halved (not below 16) for heavy GQA (kv/heads <= 1/4)."""
-        if config.is_latent:                 # one narrow row per token: 64 rows are one attention tile
+        if config.is_design:                 # 64 rows are one attention tile
             return 64
         base = 16 if config.max_seq_len <= 4096 else 32 if config.max_seq_len <= 32768 else 64
         if config.num_kv_heads / config.num_heads <= 0.25 and base > 16:
@@ -126,6 +131,8 @@ class KVCacheManager:
             if need > self._pool.num_free and not self._evict_locked(need):
                 raise RuntimeError(f"cannot allocate {need} KV blocks for sequence {seq_id}: "
                                    f"{self._pool.num_free} free and eviction did not help")
+            if self.states is not None:
+                self.states.allocate(seq_id)
             e = self._page_table.create_sequence(seq_id)
             for i, bid in enumerate(shared):
                 b = self._pool.get_block(bid)
@@ -207,8 +214,9 @@ class KVCacheManager:
             for i, sid in enumerate(seq_ids):
                 e = self._page_table.get_entry_or_none(sid)
                 n = e.num_tokens if e is not None else 0
-                # (the step that moves the window's start over a block border gives a block back: ordinary path)
-                if e is not None and (not windowed or (n + 1 - self._window) % bs):
+                # (the step that moves the first position seen over a block border gives blocks back: ordinary path)
+                if e is not None and (not windowed or self._config.first_seen(n) // bs
+                                      == self._config.first_seen(max(0, n - 1)) // bs):
                     fill = n % bs
                     if fill and n < limit and e.blocks:
                         tail = e.blocks[-1]
@@ -232,12 +240,16 @@ class KVCacheManager:
                     self._dedup.deregister_block(b.block_id)
             self._evictor.remove_sequence(seq_id)
             self._page_table.remove_sequence(seq_id)
+            if self.states is not None:
+                self.states.free(seq_id)
             for d in (self._prompt_lengths, self._prompt_tokens, self._registered_upto, self._salts):
                 d.pop(seq_id, None)
             self._active.discard(seq_id)
 
     def fork_sequence(self, src_id: int, dst_id: int) -> KVCacheHandle:
         with self._lock:
+            if self.states is not None:
+                self.states.fork(src_id, dst_id)
             e = self._page_table.fork_sequence(src_id, dst_id)
             self._prompt_lengths[dst_id] = self._prompt_lengths.get(src_id, 0)
             self._active.add(dst_id)
@@ -310,10 +322,10 @@ class KVCacheManager:
         return self._pool.num_free >= blocks_needed
 
     def _trim_sliding_window(self, seq_id: int, first_new: int) -> None:
-        """Gives back the blocks no token from position ``first_new`` on can see: that token itself still sees the
-        ``window - 1`` before it, however many more are appended with it."""
+        """Gives back the blocks no token from position ``first_new`` on can see: with a window, that token itself still
+        sees the ``window - 1`` before it, however many more are appended with it."""
         e = self._page_table.get_entry_or_none(seq_id)
-        keep_from = first_new + 1 - self._window
+        keep_from = self._config.first_seen(first_new)
         if e is None or keep_from <= 0:
             return
         for idx in range(min(keep_from // self._block_size, len(e.blocks))):
@@ -329,6 +341,12 @@ class KVCacheManager:
     def block_ids_np(self, seq_id: int):
         with self._lock:
             return self._page_table.block_ids_np(seq_id)
+
+    def stage_states(self, spans, read, write) -> None:
+        """``spans``: (seq_id, start, tokens) of a pass's sequences; fills the rows of ``states`` they read and write."""
+        with self._lock:
+            for s, (sid, start, n) in enumerate(spans):
+                read[s], write[s] = self.states.advance(sid, start, n)
 
     def stage_decode(self, seq_ids, block_tables, seq_lens, positions, slots) -> int:
         """Fills the decode-step arrays (numpy views of the runner's pinned staging buffers) for ``seq_ids`` in one
@@ -441,3 +459,5 @@ class KVCacheManager:
     def destroy(self) -> None:
         with self._lock:
             self._pool.destroy()
+            if self.states is not None:
+                self.states.destroy()

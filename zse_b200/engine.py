@@ -24,6 +24,7 @@ from typing import Callable, Dict, Iterator, List, Optional
 import torch
 
 from .cache.cache_manager import KVCacheManager
+from .cache.state_slots import StateSlots
 from .config import EngineConfig
 from .format.directory import open_model
 from .models.decoder import DecoderModel
@@ -114,10 +115,13 @@ class ZStreamerEngine:
         act = self._model.act_dtype
         block_size = cfg.block_size or KVCacheManager._auto_block_size(mc)
         nkv_local = self._model.plan.num_kv_heads
+        slots = cfg.state_slots or cfg.max_batch_seqs + 1
         if cfg.kv_blocks > 0:
             blocks = cfg.kv_blocks
         elif on_gpu:
             scratch_est = cfg.max_batch_tokens * (mc.hidden_size * 40 + mc.intermediate_size * 2) + (256 << 20)
+            if mc.keeps_state:
+                scratch_est += slots * StateSlots.bytes_per_slot(mc.state_floats)
             plan = VRAMAllocator.for_device(self.device).plan_allocation(
                 mc, 0, scratch_est, block_size, self._max_seq_len, cfg.max_batch_seqs, cfg.tp_size, cfg.kv_fraction)
             blocks = max(1, plan.kv_blocks * 2 // act.itemsize)       # the plan counts 16-bit elements
@@ -126,7 +130,7 @@ class ZStreamerEngine:
             blocks = max(64, (cfg.max_batch_seqs * min(self._max_seq_len, 2048)) // block_size)
         self._kv_cache = KVCacheManager(mc, self.device, block_size=block_size, num_blocks=blocks,
                                         eviction_policy=cfg.eviction_policy, enable_dedup=cfg.enable_prefix_cache,
-                                        num_kv_heads=nkv_local, dtype=act)
+                                        num_kv_heads=nkv_local, dtype=act, state_slots=slots)
         self._runner = ModelRunner(self._model, self._kv_cache, max_batch_seqs=cfg.max_batch_seqs,
                                    max_tokens_per_pass=max(cfg.max_batch_tokens, cfg.prefill_chunk_size or 0),
                                    max_seq_len=self._max_seq_len, use_graphs=cfg.use_cuda_graphs,

@@ -96,14 +96,127 @@ class LatentSpec:
 
 @dataclass(frozen=True)
 class MoESpec:
-    """Routed feed-forward: ``top`` of ``experts`` per token, chosen and weighted by ``score``; the weight scales the
-    expert's INPUT.  ``shared_ff`` > 0 adds an expert that every token uses."""
+    """Routed feed-forward: ``top`` of ``experts`` per token, chosen and weighted by ``score``.  ``shared_ff`` > 0 adds an
+    expert that every token uses."""
     experts: int
     top: int
     ff: int
     shared_ff: int = 0
-    score: str = "sigmoid"
-    activation: str = "gelu"     # exact (erf) gelu
+    score: str = "sigmoid"       # of the router's logits: "sigmoid" (each on its own) or "softmax" (over all experts)
+    activation: str = "gelu"     # exact (erf) gelu, or "clamped_glu": two up products, see ``ops.reference.clamped_glu``
+    weigh: str = "input"         # the weight scales the expert's "input" or "output"
+    normalise: bool = False      # the chosen scores are divided by their sum
+    scale: float = 1.0           # ... and multiplied by this
+    limit: float = 0.0           # clamp of "clamped_glu"
+    shared_limit: float = 0.0
+    shared_gate: bool = False    # the shared expert is multiplied by sigmoid(w . h), one number per token
+
+    @property
+    def gated(self) -> bool:
+        return self.activation == "clamped_glu"
+
+    @property
+    def router_rows(self) -> int:
+        """Columns of the router's product: the experts, and the shared expert's gate behind them."""
+        return self.experts + (1 if self.shared_gate else 0)
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    """Feed-forward of one up product, an activation and one down product."""
+    ff: int
+    activation: str = "relu2"    # the square of relu
+
+
+@dataclass(frozen=True)
+class HeadsSpec:
+    """Attention of ``heads`` query heads over ``kv_heads`` key/value heads whose widths may differ; no rotation."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: int = 0               # > 0: a position sees the positions of its own chunk of this size only
+    window: int = 0              # > 0: a position sees itself and the window - 1 before it
+    kv_from: int = -1            # >= 0: keys and values are those of that layer
+    gated: bool = True           # a head's result is multiplied by sigmoid(w_h . x)
+
+    @property
+    def own_kv(self) -> bool:
+        return self.kv_from < 0
+
+    # columns of the fused input projection [q | k | v | gate]; every section starts on 8 elements
+    @property
+    def k_col(self) -> int:
+        return _up8(self.heads * self.dim)
+
+    @property
+    def v_col(self) -> int:
+        return self.k_col + (_up8(self.kv_heads * self.dim) if self.own_kv else 0)
+
+    @property
+    def gate_col(self) -> int:
+        return self.v_col + (_up8(self.kv_heads * self.vdim) if self.own_kv else 0)
+
+    @property
+    def in_width(self) -> int:
+        return self.gate_col + (_up8(self.heads) if self.gated else 0)
+
+    @property
+    def row(self) -> int:
+        """Elements of a cached token."""
+        return self.kv_heads * (_up8(self.dim) + _up8(self.vdim))
+
+    def first_seen(self, position: int) -> int:
+        """First position that the token at ``position`` sees."""
+        if self.chunk > 0:
+            return position // self.chunk * self.chunk
+        return max(0, position + 1 - self.window) if self.window > 0 else 0
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Recurrent mixer whose heads keep a [dim, vdim] matrix memory, a key sum [dim] and a running maximum of the log
+    gates (mLSTM)."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    # columns of the fused input projection [q | k | v | output gate | input and forget gates]
+    @property
+    def k_col(self) -> int:
+        return _up8(self.heads * self.dim)
+
+    @property
+    def v_col(self) -> int:
+        return 2 * self.k_col
+
+    @property
+    def gate_col(self) -> int:
+        return self.v_col + _up8(self.heads * self.vdim)
+
+    @property
+    def if_col(self) -> int:
+        return self.gate_col + _up8(self.heads * self.vdim)
+
+    @property
+    def in_width(self) -> int:
+        return self.if_col + _up8(2 * self.heads)
+
+    # state of one sequence, in 32-bit elements: memory [heads, dim, vdim], key sum [heads, dim], maximum [heads]; every
+    # part starts on 4 elements
+    @property
+    def sum_at(self) -> int:
+        return (self.heads * self.dim * self.vdim + 3) // 4 * 4
+
+    @property
+    def max_at(self) -> int:
+        return self.sum_at + (self.heads * self.dim + 3) // 4 * 4
+
+    @property
+    def state_floats(self) -> int:
+        return self.max_at + (self.heads + 3) // 4 * 4
 
 
 @dataclass
@@ -138,6 +251,8 @@ class ModelConfig:
     # the model's config.json ({"type", "mixer", "mlp"}), ``weight_dtype`` the width its weights are stored in
     design_layers: Optional[List[Dict[str, Any]]] = None
     embed_multiplier: Optional[float] = None
+    # {"bigram": {"buckets", "mul_prev", "mul_cur"}, "sinusoid_base", "norm"}: what is added to a token's embedding
+    embed_design: Optional[Dict[str, Any]] = None
     logit_scale: Optional[float] = None
     weight_dtype: Optional[str] = None
     multimodal: Optional[Dict[str, Any]] = None
@@ -193,16 +308,83 @@ class ModelConfig:
     @property
     def kv_planes(self) -> int:
         """Rows a token has per layer and kv head: K and V, or one latent row that serves as both."""
-        return 1 if self.is_latent else 2
+        return 1 if self.is_design else 2
 
     @property
     def total_kv_cache_bytes_per_token(self) -> int:
-        return self.kv_cache_bytes_per_token * self.num_layers
+        return self.kv_cache_bytes_per_token * self.num_cache_layers
 
     # ---- designs whose layers are listed one by one ----------------------------------------------------
     @property
-    def is_latent(self) -> bool:
+    def is_design(self) -> bool:
         return self.design_layers is not None
+
+    @property
+    def is_latent(self) -> bool:
+        return self.is_design and any(L["type"] == "latent_attention" for L in self.design_layers)
+
+    @property
+    def is_hybrid(self) -> bool:
+        """Layers of attention over heads and of recurrent mixers, in any order."""
+        return self.is_design and not self.is_latent
+
+    def mixer_spec(self, i: int):
+        """``HeadsSpec`` or ``MatrixMemorySpec`` of layer ``i`` of a hybrid design."""
+        L = self.design_layers[i]
+        m = L["mixer"]
+        if L["type"] == "mlstm":
+            return MatrixMemorySpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+        src = m.get("kv_from")
+        return HeadsSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                         chunk=int((m.get("mask") or {}).get("size") or 0), kv_from=-1 if src is None else int(src))
+
+    def ff_spec(self, i: int):
+        """``DenseSpec``, ``MoESpec`` or None of layer ``i`` of a hybrid design."""
+        m = self.design_layers[i].get("mlp")
+        if m is None:
+            return None
+        if m["kind"] == "dense":
+            return DenseSpec(int(m["ff"]))
+        r, e, s = m["router"], m["expert"], m.get("shared")
+        return MoESpec(int(r["experts"]), int(r["top"]), int(e["ff"]), int(s["ff"]) if s else 0, "softmax",
+                       "clamped_glu", "output", True, float(r.get("scale", 1.0)), float(e["limit"]),
+                       float(s["limit"]) if s else 0.0, bool(s))
+
+    @property
+    def cache_layers(self) -> Dict[int, int]:
+        """Layer -> its layer of the cache pool; layers without keys and values of their own have none."""
+        if not self.is_hybrid:
+            return {i: i for i in range(self.num_layers)}
+        own = [i for i in range(self.num_layers) if isinstance(self.mixer_spec(i), HeadsSpec)
+               and self.mixer_spec(i).own_kv]
+        return {i: n for n, i in enumerate(own)}
+
+    @property
+    def num_cache_layers(self) -> int:
+        return max(1, len(self.cache_layers))
+
+    @property
+    def state_offsets(self) -> Dict[int, int]:
+        """Recurrent layer -> its first element in a sequence's state."""
+        out, at = {}, 0
+        if self.is_hybrid:
+            for i in range(self.num_layers):
+                s = self.mixer_spec(i)
+                if isinstance(s, MatrixMemorySpec):
+                    out[i] = at
+                    at += s.state_floats
+        return out
+
+    @property
+    def state_floats(self) -> int:
+        off = self.state_offsets
+        last = max(off, default=-1)
+        return off[last] + self.mixer_spec(last).state_floats if off else 0
+
+    @property
+    def keeps_state(self) -> bool:
+        """Sequences carry more than their cache blocks from token to token: recurrent layers, or the token before."""
+        return self.is_hybrid and (self.state_floats > 0 or bool((self.embed_design or {}).get("bigram")))
 
     def latent_spec(self, i: int) -> LatentSpec:
         m = self.design_layers[i]["mixer"]
@@ -222,10 +404,23 @@ class ModelConfig:
     def cache_window(self) -> int:
         """Tokens that some layer still sees: blocks that fell out of every layer's window may be given back.  0 when a
         layer keeps everything (models that mix local and global layers apply the window inside attention)."""
+        if self.is_hybrid:
+            return 0
         if self.is_latent:
             w = [self.latent_spec(i).window for i in range(self.num_layers)]
             return max(w) if w and min(w) > 0 else 0
         return int(self.sliding_window) if (self.sliding_window or 0) > 0 and not self.layer_types else 0
+
+    def first_seen(self, position: int) -> int:
+        """First position that some layer still sees from ``position`` (and from any later one): the cache may give back
+        the blocks before it."""
+        if self.is_hybrid:
+            if self.__dict__.get("_masks") is None:
+                self.__dict__["_masks"] = list({(s.chunk, s.window): s for s in (self.mixer_spec(i) for i in range(
+                    self.num_layers)) if isinstance(s, HeadsSpec)}.values())
+            return min((s.first_seen(position) for s in self.__dict__["_masks"]), default=position)
+        w = self.cache_window
+        return max(0, position + 1 - w) if w > 0 else 0
 
     # ---- per-layer attention geometry (Gemma-family models mix layer kinds) -----------------------
     @property
@@ -270,6 +465,8 @@ class ModelConfig:
         (``1 x max(kv_heads * head_dim)`` of the local heads); each layer lays its heads out inside that row."""
         if self.is_latent:
             return 1, max(self.latent_spec(i).row for i in range(self.num_layers))
+        if self.is_hybrid:
+            return 1, max((self.mixer_spec(i).row for i in self.cache_layers), default=8)
         local = num_kv_heads or self.num_kv_heads
         tp = max(1, self.num_kv_heads // max(1, local))
         specs = {(s.num_kv_heads, s.head_dim) for s in (self.layer_spec(i) for i in range(self.num_layers))}
@@ -278,6 +475,16 @@ class ModelConfig:
         return 1, max(max(1, n // tp) * d for n, d in specs)
 
     def linear_param_count(self) -> int:
+        if self.is_hybrid:
+            n = 0
+            for i in range(self.num_layers):
+                a, m = self.mixer_spec(i), self.ff_spec(i)
+                n += self.hidden_size * (a.in_width + a.heads * a.vdim)
+                if isinstance(m, MoESpec):
+                    n += self.hidden_size * (m.router_rows + 3 * m.experts * m.ff + 3 * m.shared_ff)
+                elif m is not None:
+                    n += self.hidden_size * 2 * m.ff
+            return n
         if self.is_latent:
             n = 0
             for i in range(self.num_layers):

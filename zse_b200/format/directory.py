@@ -50,7 +50,7 @@ class DirectoryLoader(ZSELoader):
             self._weight_index.add(WeightEntry(stored, shape, dtype, data_nbytes=n * _WIDTH[dtype]))
             self._source[stored] = src
         missing = [t for t in adapter.expected_tensors(self._config) if t not in self._weight_index] \
-            if self._config.is_latent else []
+            if self._config.is_design else []
         if missing:
             raise ValueError(f"{path}: {len(missing)} tensors are missing, the first is '{missing[0]}'")
         self._tokenizer = None

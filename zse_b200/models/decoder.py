@@ -28,7 +28,7 @@ from ..ops import reference as ref
 from ..ops.backend import LinearWeight, TorchOps, make_ops, np_to_dev
 from ..parallel.shard_plan import ShardPlan, make_plan
 
-SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "phi3", "gemma2", "gemma4", "ruralorn")
+SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "phi3", "gemma2", "gemma4", "ruralorn", "nimelorn")
 
 
 def _entry_part(loader: ZSELoader, name: str, rows=None, cols=None, mirror=None) -> dict:
@@ -157,6 +157,7 @@ class DecoderModel:
         self.lm_head: Optional[LinearWeight] = None
         self.inv_freq: Optional[torch.Tensor] = None
         self.scale = 1.0 / math.sqrt(config.head_dim)
+        self.states = None          # cache.state_slots.StateSlots of the runner's cache (models with recurrent state)
         self.comm = None            # parallel.comm.TPComm when tp_size > 1
         # a uniform sliding window (Mistral, Phi-3): a token sees the last ``window`` positions, itself included; the
         # cache lets blocks that fell out of every window go, attention masks inside the oldest block that is left
@@ -182,6 +183,9 @@ class DecoderModel:
         elif c.is_latent and cls is DecoderModel:
             from .latent_moe import LatentMoEModel
             cls = LatentMoEModel
+        elif c.is_hybrid and cls is DecoderModel:
+            from .hybrid import HybridModel
+            cls = HybridModel
         m = cls(c, plan, ops or make_ops(device, cls.kernel_group))
         m.set_dtype(dtype)
         m._load(loader, progress)

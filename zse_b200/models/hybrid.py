@@ -1,0 +1,286 @@
+"""Decoders whose layers mix attention over heads and recurrent matrix memories, with norms on the sublayers' outputs
+(Nimelorn), over the paged cache and the state slots.
+
+Same pass contract as ``DecoderModel``.  The residual x is fp32; sublayers read x itself (rounded to the activations' type):
+
+    x     = norm(embedding + what the design adds to it)                                       1 kernel
+    y     = mixer(x);  x += norm(y) * w1                                    (sum of the split-K planes, norm, add: 1 kernel)
+    y     = ff(x);     x += norm(y) * w2                                                       (the same kernel)
+    after the last sublayer the same kernel also writes norm(x) * w_final for the head
+
+Attention caches normed keys and values as [kv head][token][dim] tiles of a block; a layer that takes another layer's keys
+and values projects queries only.  Rows that decode, and chunks of at most ``SHORT_CHUNK`` tokens, run a row at a time with
+the keys split over CTAs; longer chunks run in tiles of queries.  A matrix memory does the same: short chunks step through
+the state token by token, with read-out, head norm and output gate in the step's kernel; longer ones run chunkwise, with the
+decays inside a chunk as a lower-triangular matrix.  A packed pass may hold both kinds: short ones are laid out first.
+
+A sequence's recurrent state and its last token live in ``cache.state_slots``; ``state_rows`` names the rows that a pass's
+sequences read and write.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Dict, List, Optional, Union
+
+import torch
+
+from ..format.config import DenseSpec, HeadsSpec, MatrixMemorySpec, MoESpec
+from ..format.loader import ZSELoader
+from ..ops.backend import LinearWeight
+from .decoder import StepBuffers
+from .design import PLANE_ROWS, SHORT_CHUNK, DesignModel
+
+
+@dataclass
+class EmbedDesign:
+    table: torch.Tensor
+    scale: float
+    base: float                             # of the sinusoid
+    norm: torch.Tensor
+    bigram: Optional[torch.Tensor] = None   # [buckets + 1, H]; the last row is that of a sequence's first token
+    buckets: int = 0
+    mul_prev: int = 0
+    mul_cur: int = 0
+    turns: Optional[torch.Tensor] = None    # device form of the sinusoid's frequencies
+
+
+@dataclass
+class HybridLayer:
+    spec: Union[HeadsSpec, MatrixMemorySpec]
+    ff: Union[DenseSpec, MoESpec, None]
+    norm1: torch.Tensor
+    w_in: LinearWeight
+    o: LinearWeight
+    norm2: Optional[torch.Tensor] = None
+    # attention
+    q_norm: Optional[torch.Tensor] = None
+    k_norm: Optional[torch.Tensor] = None
+    cache_layer: int = -1
+    # matrix memory
+    w_if: Optional[LinearWeight] = None     # the rows of w_in that make the gates
+    if_bias: Optional[torch.Tensor] = None  # fp32 [2 * heads]
+    head_norm: Optional[torch.Tensor] = None
+    state_at: int = 0
+    # feed-forward
+    up_w: Optional[LinearWeight] = None
+    down_w: Optional[LinearWeight] = None
+    router: Optional[LinearWeight] = None
+    up: Optional[torch.Tensor] = None
+    down: Optional[torch.Tensor] = None
+    shared_up: Optional[torch.Tensor] = None
+    shared_down: Optional[torch.Tensor] = None
+
+    @property
+    def moe(self) -> Optional[MoESpec]:
+        return self.ff if isinstance(self.ff, MoESpec) else None
+
+
+class PagedHeads:
+    """One layer's cached keys [blocks, kv_heads, block_size, dim] and values inside the pool, whose rows are as wide as the
+    widest layer's; dims are padded to 8."""
+
+    def __init__(self, layer: torch.Tensor, spec: HeadsSpec):
+        # layer: [blocks, 1, 1, block_size, pool row]
+        bs, G = layer.shape[3], spec.kv_heads
+        d, v = (spec.dim + 7) // 8 * 8, (spec.vdim + 7) // 8 * 8
+        self.block_size, self.block_stride = bs, layer.stride(0)
+        self.k = layer.as_strided((layer.shape[0], G, bs, d), (layer.stride(0), bs * d, d, 1), layer.storage_offset())
+        self.v = layer.as_strided((layer.shape[0], G, bs, v), (layer.stride(0), bs * v, v, 1),
+                                  layer.storage_offset() + G * bs * d)
+
+
+class HybridStepBuffers(StepBuffers):
+    def __init__(self, model: "HybridModel", max_tokens: int, max_seqs: int, max_blocks: int, max_planes: int,
+                 logits_rows: int, attn_splits: int):
+        c, dev, act = model.config, model.device, model.act_dtype
+        f32, i32 = torch.float32, torch.int32
+        z = lambda *s, dt: torch.zeros(*s, dtype=dt, device=dev)
+        H = c.hidden_size
+        self._common(dev, H, c.vocab_size, max_tokens, max_seqs, max_blocks, logits_rows, attn_splits, act=act,
+                     logits=f32)
+        specs = [L.spec for L in model.layers]
+        heads = [s for s in specs if isinstance(s, HeadsSpec)]
+        memories = [s for s in specs if isinstance(s, MatrixMemorySpec)]
+        self.plane_rows = min(max_tokens, PLANE_ROWS)
+
+        def views(widths, dt):
+            flat = z(max_tokens * max(widths), dt=dt)
+            return {w: flat[: max_tokens * w].view(max_tokens, w) for w in set(widths)}
+
+        self.in_views = views([s.in_width for s in specs], act)
+        self.out_views = views([s.heads * s.vdim for s in specs], act)
+        planes = z(max_planes * self.plane_rows * max(s.in_width for s in specs), dt=f32)
+        self.in_plane_views = {w: planes[: max_planes * self.plane_rows * w].view(max_planes, self.plane_rows, w)
+                               for w in {s.in_width for s in specs}}
+        # split-K planes of decode-sized passes, one plane of any other
+        partials = z(max(max_planes * self.plane_rows, max_tokens) * H, dt=f32)
+        self.partial_views = (partials[: max_planes * self.plane_rows * H].view(max_planes, self.plane_rows, H),
+                              partials[: max_tokens * H].view(1, max_tokens, H))
+        dense = [L.ff.ff for L in model.layers if isinstance(L.ff, DenseSpec)]
+        self.act_views = views(dense, act) if dense else {}
+        rows_split = min(max_tokens, max(256, max_seqs))      # only decode passes split their keys
+        self.attn_scratch = z(rows_split * attn_splits * max([1] + [s.heads * (s.vdim + 2) for s in heads]), dt=f32)
+        gate_w = max([1] + [2 * s.heads for s in memories])
+        self.gates = z(max_tokens * gate_w, dt=f32)
+        self.gate_planes = z(max_planes, max_tokens * gate_w, dt=f32)
+        self.memory_ws = model.ops.memory_workspace(memories, max_tokens)
+        self.row_seq = z(max_tokens, dt=i32)
+        self.state_rows = torch.full((2, max_seqs), -1, dtype=i32, device=dev)
+        self.h_row_seq = torch.zeros(max_tokens, dtype=i32, pin_memory=dev.type == "cuda")
+        self.short_rows = self.short_seqs = 0     # rows and sequences of the staged pass that run token by token
+        self.moe_ws = model.ops.moe_workspace([L.moe for L in model.layers if L.moe is not None], H, max_tokens, act)
+
+
+class HybridModel(DesignModel):
+    kernel_group = "hybrid"
+
+    # ---- loading --------------------------------------------------------------------------------------
+    def _load(self, loader: ZSELoader, progress=None) -> None:
+        c, ops, dev = self.config, self.ops, self.device
+        r = self._open(loader)
+        H, ex = c.hidden_size, c.embed_design
+        self.embed = r.get("embed")
+        self.embed_design = EmbedDesign(self.embed, float(c.embed_multiplier or 1.0), float(ex["sinusoid_base"]),
+                                        r.get("embed.norm"))
+        if ex.get("bigram"):
+            b, e = ex["bigram"], self.embed_design
+            e.bigram, e.buckets, e.mul_prev, e.mul_cur = r.get("bigram"), b["buckets"], b["mul_prev"], b["mul_cur"]
+        self.norm = r.get("final.norm")
+        for i in range(c.num_layers):
+            p, s, m = f"l{i}.", c.mixer_spec(i), c.ff_spec(i)
+            t = lambda name: r.tensor(p + name)
+            if isinstance(s, MatrixMemorySpec):
+                w = r.stack([(0, t("mix.q")), (s.k_col, t("mix.k")), (s.v_col, t("mix.v")), (s.gate_col, t("mix.g")),
+                             (s.if_col, t("mix.i")), (s.if_col + s.heads, t("mix.f"))], s.in_width, H)
+                L = HybridLayer(s, m, r.get(p + "norm1"), ops.dense_linear(w), r.linear(p + "mix.o"))
+                L.w_if = ops.dense_linear(w[s.if_col: s.if_col + 2 * s.heads])
+                L.if_bias = torch.cat([t("mix.i.b"), t("mix.f.b")]).float().contiguous()
+                L.head_norm, L.state_at = r.get(p + "mix.norm"), c.state_offsets[i]
+            else:
+                parts = [(0, t("mix.q")), (s.gate_col, t("mix.g"))]
+                if s.own_kv:
+                    parts += [(s.k_col, t("mix.k")), (s.v_col, t("mix.v"))]
+                L = HybridLayer(s, m, r.get(p + "norm1"), ops.dense_linear(r.stack(parts, s.in_width, H)),
+                                r.linear(p + "mix.o"), q_norm=r.get(p + "mix.q.norm"))
+                if s.own_kv:
+                    L.k_norm = r.get(p + "mix.k.norm")
+                L.cache_layer = c.cache_layers[i if s.own_kv else s.kv_from]
+            if m is not None:
+                L.norm2 = r.get(p + "norm2")
+            if isinstance(m, DenseSpec):
+                L.up_w, L.down_w = r.linear(p + "mlp.up"), r.linear(p + "mlp.down")
+            elif m is not None:
+                rows = [(0, t("mlp.router"))] + ([(m.experts, t("mlp.shared.sg"))] if m.shared_gate else [])
+                L.router = ops.dense_linear(r.stack(rows, m.router_rows, H))
+                count = lambda w: self._count(w)
+                L.up = count(ops.moe_up([(t(f"mlp.e{e}.gate"), t(f"mlp.e{e}.up")) for e in range(m.experts)],
+                                        self.act_dtype))
+                L.down = r.stack([(e * H, t(f"mlp.e{e}.down")) for e in range(m.experts)], m.experts * H, m.ff)
+                if m.shared_ff:
+                    L.shared_up = count(ops.moe_up([(t("mlp.shared.gate"), t("mlp.shared.up"))], self.act_dtype))
+                    L.shared_down = r.get(p + "mlp.shared.down")
+            self.layers.append(L)
+            if progress:
+                progress(i + 1, c.num_layers)
+        self.lm_head = r.linear("head")
+        r.release()
+        self.heads_specs = [L.spec for L in self.layers if isinstance(L.spec, HeadsSpec)]
+        self._views: Dict[tuple, PagedHeads] = {}
+
+    def _count(self, w: torch.Tensor) -> torch.Tensor:
+        self.weight_bytes += w.numel() * w.element_size()
+        return w
+
+    # ---- buffers --------------------------------------------------------------------------------------
+    def make_buffers(self, max_tokens: int, max_seqs: int, max_blocks: int, logits_rows: Optional[int] = None,
+                     max_planes: int = 8, attn_splits: int = 1) -> HybridStepBuffers:
+        return HybridStepBuffers(self, max_tokens, max_seqs, max_blocks, max_planes, logits_rows or max_seqs, attn_splits)
+
+    def _heads_view(self, kv: torch.Tensor, L: HybridLayer) -> PagedHeads:
+        key = (kv.data_ptr(), L.cache_layer)
+        v = self._views.get(key)
+        if v is None:
+            v = self._views[key] = PagedHeads(kv[L.cache_layer], L.spec)
+        return v
+
+    def attention_splits(self, seqs: int, max_len: int, most: int, sms: int) -> int:
+        if not self.heads_specs:
+            return 1
+        span = max(min(max_len, s.chunk or max_len, s.window or max_len) for s in self.heads_specs)
+        ctas = seqs * min(s.kv_heads * ((s.heads // s.kv_heads + 15) // 16) for s in self.heads_specs)
+        want = (2 * sms + ctas - 1) // ctas
+        n = int(max(1, min(want, span // 128, most)))
+        return 1 << (n.bit_length() - 1)
+
+    # ---- layout of a packed pass ----------------------------------------------------------------------
+    def pass_order(self, items) -> Optional[List[int]]:
+        return sorted(range(len(items)), key=lambda i: len(items[i][1]) > SHORT_CHUNK)
+
+    def stage_prefill(self, b: HybridStepBuffers, spans) -> None:
+        at = b.short_rows = b.short_seqs = 0
+        for s, (_, n) in enumerate(spans):
+            b.h_row_seq[at: at + n] = s
+            at += n
+            if n <= SHORT_CHUNK:
+                b.short_rows, b.short_seqs = at, s + 1
+        b.row_seq[:at].copy_(b.h_row_seq[:at], non_blocking=True)
+
+    # ---- forward --------------------------------------------------------------------------------------
+    def forward(self, b: HybridStepBuffers, kv: torch.Tensor, M: int, mode: str, num_seqs: int, max_q_len: int = 1,
+                n_logit_rows: int = 0, attn_splits: int = 1) -> None:
+        c, ops, eps = self.config, self.ops, self.config.rms_norm_eps
+        decode = mode == "decode"
+        row_seq, cu_q = (None, None) if decode else (b.row_seq, b.cu_q)
+        short = (M, num_seqs) if decode else (b.short_rows, b.short_seqs)
+        planes_ok = M <= b.plane_rows
+        partials = b.partial_views[0 if planes_ok else 1]
+        last_token = self.states.last_token if self.states is not None else None
+        ops.embed_design(self.embed_design, b.ids, b.positions, row_seq, cu_q, b.state_rows, last_token, b.residual,
+                         b.xnorm, M, num_seqs, eps)
+        for li, L in enumerate(self.layers):
+            s = L.spec
+            inp, in_planes, n_in = b.in_views[s.in_width], b.in_plane_views[s.in_width], 0
+            if planes_ok:
+                n_in = ops.linear_partial(L.w_in, b.xnorm, M, in_planes)
+            else:
+                ops.linear(L.w_in, b.xnorm, M, inp)
+            out = b.out_views[s.heads * s.vdim]
+            if isinstance(s, HeadsSpec):
+                view = self._heads_view(kv, L)
+                ops.heads_prep(inp, in_planes, n_in, view, b.slots, L, s, eps, M)
+                rows, seqs = short if ops.heads_expands(s, self.act_dtype) else (M, num_seqs)
+                if rows:
+                    ops.heads_attn(inp, view, b.block_tables, row_seq, b.positions, out, rows, s, b.attn_scratch,
+                                   attn_splits)
+                if seqs < num_seqs:
+                    ops.heads_attn_chunks(inp, view, b.block_tables, b.cu_q, b.q_pos0, b.positions, seqs, num_seqs,
+                                          max_q_len, out, s)
+            else:
+                n_gate = 0
+                if not n_in:
+                    n_gate = ops.linear_partial(L.w_if, b.xnorm, M, b.gate_planes)
+                ops.memory_prep(inp, in_planes, n_in, b.gate_planes, n_gate, b.gates, L, s, M)
+                rows, seqs = short if ops.memory_expands(s, self.act_dtype) else (M, num_seqs)
+                states = self.states.rows
+                if seqs:
+                    ops.memory_tokens(inp, b.gates, states, L.state_at, b.state_rows, cu_q, L, out, seqs, M, s, eps)
+                if seqs < num_seqs:
+                    ops.memory_chunks(inp, b.gates, states, L.state_at, b.state_rows, b.cu_q, L, out, seqs, num_seqs, M,
+                                      s, eps, b.memory_ws)
+            planes = ops.linear_partial(L.o, out, M, partials)
+            last = li + 1 == len(self.layers)
+            ops.post_norm(b.residual, partials, planes, None, L.norm1, self.norm if last and L.ff is None else None,
+                          b.xnorm, M, eps)
+            if L.ff is None:
+                continue
+            slots = None
+            if L.moe is not None:
+                slots, planes = ops.moe(L, b.xnorm, M, b.moe_ws), 0
+            else:
+                act = b.act_views[L.ff.ff]
+                ops.linear_act(L.up_w, b.xnorm, M, act, L.ff.activation)
+                planes = ops.linear_partial(L.down_w, act, M, partials)
+            ops.post_norm(b.residual, partials, planes, slots, L.norm2, self.norm if last else None, b.xnorm, M, eps)
+        if n_logit_rows:
+            torch.index_select(b.xnorm, 0, b.logit_rows[:n_logit_rows], out=b.xsel[:n_logit_rows])
+            ops.linear_f32(self.lm_head, b.xsel, n_logit_rows, b.logits)

@@ -25,16 +25,13 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import List, Optional
 
-import numpy as np
 import torch
 
 from ..format.config import LatentSpec, MoESpec
 from ..format.loader import ZSELoader
 from ..ops.backend import LinearWeight
-from .decoder import DecoderModel, StepBuffers
-
-SHORT_CHUNK = 16            # chunks up to this length read the cached rows directly
-PLANE_ROWS = 256            # passes up to this size take projections as fp32 split-K planes
+from .decoder import StepBuffers
+from .design import PLANE_ROWS, SHORT_CHUNK, DesignModel
 
 
 def attention_splits(seqs: int, groups: int, span: int, most: int, sms: int) -> int:
@@ -133,54 +130,14 @@ class LatentStepBuffers(StepBuffers):
         self.moe_ws = model.ops.moe_workspace([L.moe for L in model.layers if L.moe is not None], H, max_tokens, act)
 
 
-class LatentMoEModel(DecoderModel):
-    act_dtype = torch.bfloat16
+class LatentMoEModel(DesignModel):
     kernel_group = "latent"
-    mixed_passes = True
-
-    def set_dtype(self, dtype: Optional[str]) -> None:
-        kinds = {None: torch.bfloat16, "bfloat16": torch.bfloat16, "float32": torch.float32}
-        if dtype not in kinds:
-            raise ValueError(f"'{self.config.arch}' runs in bfloat16 or float32, not {dtype}")
-        self.act_dtype = kinds[dtype]
 
     # ---- loading --------------------------------------------------------------------------------------
     def _load(self, loader: ZSELoader, progress=None) -> None:
-        c, ops, dev, act = self.config, self.ops, self.device, self.act_dtype
-        if self.plan.tp_size != 1:
-            raise NotImplementedError(f"'{c.arch}' is served by one GPU (no tensor-parallel split of its layers yet)")
-        self.cache_block_size = 64
-        mirror = None
-        if dev.type == "cuda":
-            from ..runtime.weight_stream import open_mirror
-            mirror = open_mirror(loader, dev, self.load_stats)
-
-        def tensor(name: str) -> torch.Tensor:
-            e = loader.weight_index.find(name)
-            if e is None:
-                raise KeyError(name)
-            if mirror is not None:
-                t = mirror.view(e.data_offset, e.data_nbytes, e.dtype).reshape(e.shape)
-            else:
-                a = np.array(loader.view_data(e))
-                t = torch.from_numpy(a.view(np.int16)).view(torch.bfloat16) if e.dtype == "bfloat16" else \
-                    torch.from_numpy(a)
-                t = t.to(dev)
-            return t.to(act)
-
-        def keep(t: torch.Tensor) -> torch.Tensor:
-            """A copy of its own (a mirror's views go away with it)."""
-            t = ops.dense(t.clone(memory_format=torch.contiguous_format), act)
-            self.weight_bytes += t.numel() * t.element_size()
-            return t
-
-        def stack(parts, rows: int, width: int) -> torch.Tensor:
-            """``parts``: (first row, tensor); rows between them are zero."""
-            out = torch.zeros(rows, width, dtype=act, device=dev)
-            for at, t in parts:
-                out[at: at + t.shape[0]] = t
-            return keep(out)
-
+        c, ops, dev = self.config, self.ops, self.device
+        r = self._open(loader)
+        tensor, keep, stack = r.tensor, r.keep, r.stack
         H = c.hidden_size
         self.embed = keep(tensor("embed"))
         self.norm = keep(tensor("final.norm"))
@@ -210,12 +167,11 @@ class LatentMoEModel(DecoderModel):
             if progress:
                 progress(i + 1, c.num_layers)
         self.lm_head = ops.dense_linear(keep(tensor("head")))
-        if mirror is not None:
-            mirror.release()
+        r.release()
         self.embed_scale = float(c.embed_multiplier if c.embed_multiplier is not None else 1.0)
         self.logit_scale = float(c.logit_scale if c.logit_scale is not None else 1.0)
         self.logit_cap = float(c.final_logit_softcapping or 0.0)
-        self.expands = all(ops.latent_expands(L.spec, act) for L in self.layers)
+        self.expands = all(ops.latent_expands(L.spec, self.act_dtype) for L in self.layers)
         self.max_window = c.cache_window
         self._row_views = {}
 

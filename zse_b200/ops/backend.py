@@ -193,16 +193,29 @@ class TorchOps:
         """The routed feed-forward of rows [0, M): returns ``slots`` [M, top (+1), H], to be summed."""
         m, H = L.moe, x.shape[1]
         xs = x[:M].float()
-        ids, w = ref.route_top(xs @ L.router.data.T, m.top)
+        z = xs @ L.router.data.T
+        ids, w = ref.route(z[:, : m.experts], m)
         slots = torch.zeros(M, m.top + (m.shared_ff > 0), H, dtype=torch.float32, device=x.device)
-        up, down = L.up.view(m.experts, m.ff, H), L.down.view(m.experts, H, m.ff)
+
+        def act(t, up, ff, limit, score=None):
+            y = t @ up.T
+            if score is not None and m.weigh == "input":
+                y = score[:, None] * y
+            return (ref.clamped_glu(y[:, :ff], y[:, ff:], limit) if m.gated else ref.gelu_exact(y)).to(x.dtype).float()
+
+        up, down = L.up.view(m.experts, -1, H), L.down.view(m.experts, H, m.ff)
         for e in torch.unique(ids).tolist():
             t, k = torch.where(ids == e)
-            act = ref.gelu_exact(w[t, k, None] * (xs[t] @ up[e].T)).to(x.dtype)
-            slots[t, k] = act.float() @ down[e].T
+            y = act(xs[t], up[e], m.ff, m.limit, w[t, k]) @ down[e].T
+            slots[t, k] = w[t, k, None] * y if m.weigh == "output" else y
         if m.shared_ff:
-            slots[:, m.top] = ref.gelu_exact(xs @ L.shared_up.T).to(x.dtype).float() @ L.shared_down.T
+            y = act(xs, L.shared_up, m.shared_ff, m.shared_limit) @ L.shared_down.T
+            slots[:, m.top] = torch.sigmoid(z[:, m.experts:]) * y if m.shared_gate else y
         return slots
+
+    def moe_up(self, pairs, dtype):
+        """Up products of gated experts from their (gate, up) matrices [ff, H], all experts in one tensor."""
+        return self.dense(torch.cat([t for pair in pairs for t in pair]), dtype)
 
     def latent_expands(self, spec, dtype) -> bool:
         """Whether long chunks of such a layer take ``latent_attn_chunks``."""
@@ -210,6 +223,111 @@ class TorchOps:
 
     def moe_workspace(self, specs, H: int, max_tokens: int, dtype):
         return None
+
+    # ---- designs of attention over heads, matrix memories and post-norms ---------------------------------
+    def embed_design(self, E, ids, positions, row_seq, cu_q, state_rows, last_token, residual, out, M, S, eps):
+        """residual = norm(scaled embedding + what the design adds to it), in fp32, and ``out`` the same for the products.
+        ``cu_q``: first row of every sequence (None: a row each), ``row_seq``: the rows' sequences.  The last token of every
+        sequence goes to ``last_token[state_rows[1, s]]``."""
+        cu = list(range(S + 1)) if cu_q is None else [int(v) for v in cu_q[: S + 1]]
+        t = ids[:M].long()
+        x = E.table[t].float() * E.scale
+        if E.bigram is not None:
+            prev = ref.previous_tokens(t, cu, state_rows, last_token)
+            x = x + E.bigram[torch.where(prev < 0, E.buckets, (prev * E.mul_prev + t * E.mul_cur) % E.buckets)].float()
+            for s in range(S):
+                if int(state_rows[1, s]) >= 0:
+                    last_token[int(state_rows[1, s])] = t[cu[s + 1] - 1].to(last_token.dtype)
+        x = x + ref.sinusoid(positions[:M], x.shape[1], E.base)
+        residual[:M] = ref.rmsnorm_f32(x, E.norm, eps)
+        out[:M] = residual[:M]
+
+    def post_norm(self, residual, partials, n_partials, slots, weight, next_weight, out, M, eps):
+        """residual += RMSNorm(the planes' sum + the sum over a row's ``slots``) * weight; out = residual, or its RMSNorm
+        with ``next_weight``."""
+        H = residual.shape[1]
+        y = torch.zeros(M, H, device=residual.device)
+        if n_partials:
+            y += partials.view(-1)[: n_partials * M * H].view(n_partials, M, H).sum(0)
+        if slots is not None:
+            y += slots[:M].float().sum(1)
+        residual[:M] += ref.rmsnorm_f32(y, weight, eps)
+        out[:M] = residual[:M] if next_weight is None else ref.rmsnorm_f32(residual[:M], next_weight, eps)
+
+    def linear_act(self, w: LinearWeight, x, M, out, activation: str):
+        """out = activation(x W^T) in the activations' type."""
+        out[:M, : w.N] = {"relu2": ref.relu2}[activation](x[:M].float() @ w.data.T)
+
+    def heads_expands(self, spec, dtype) -> bool:
+        """Whether long chunks of such a layer take ``heads_attn_chunks``."""
+        return True
+
+    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M):
+        if n_planes:
+            ld = inp.shape[1]
+            inp[:M] = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
+        ref.heads_prep(inp[:M], kv.k if kv else None, kv.v if kv else None, slots[:M], spec, L.q_norm, L.k_norm, eps)
+
+    def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits):
+        """Rows [0, M) against the cached keys and values; row t belongs to sequence ``row_seq[t]`` (None: t)."""
+        for t in range(M):
+            s = t if row_seq is None else int(row_seq[t])
+            self._heads_rows(inp, kv, block_tables[s], positions, out, t, t + 1, spec)
+
+    def heads_attn_chunks(self, inp, kv, block_tables, cu_q, q_pos0, positions, first, last, max_q, out, spec):
+        """Rows of the sequences ``first .. last - 1``."""
+        for s in range(first, last):
+            self._heads_rows(inp, kv, block_tables[s], positions, out, int(cu_q[s]), int(cu_q[s + 1]), spec)
+
+    @staticmethod
+    def _heads_rows(inp, kv, table, positions, out, a, e, spec):
+        H, w = spec.heads, spec.heads * spec.vdim
+        y = ref.heads_attn(inp[a:e, : H * spec.dim].reshape(e - a, H, spec.dim), positions[a:e].long(), kv.k, kv.v, table,
+                           spec)
+        if spec.gated:
+            y = y * torch.sigmoid(inp[a:e, spec.gate_col: spec.gate_col + H].float())[:, :, None]
+        out[a:e, :w] = y.reshape(e - a, w)
+
+    def memory_expands(self, spec, dtype) -> bool:
+        """Whether long chunks of such a layer take ``memory_chunks``."""
+        return False
+
+    def memory_workspace(self, specs, max_tokens: int):
+        return None
+
+    def memory_prep(self, inp, planes, n_planes, gate_planes, n_gate_planes, gates, L, spec, M):
+        """Sums the split-K planes of the input projection and takes the logarithms of the gates, ``gates`` [M, 2 * heads].
+        With ``n_planes`` 0 ``inp`` is complete and the gates' pre-activations are in ``gate_planes`` [n, M, 2 * heads]."""
+        g = 2 * spec.heads
+        if n_planes:
+            ld = inp.shape[1]
+            full = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
+            inp[:M] = full
+            z = full[:, spec.if_col: spec.if_col + g]
+        else:
+            z = gate_planes.view(-1)[: n_gate_planes * M * g].view(n_gate_planes, M, g).sum(0)
+        gates.view(-1)[: M * g].view(M, g).copy_(ref.memory_gates(z, L.if_bias, spec.gate_cap))
+
+    def memory_tokens(self, inp, gates, states, at, state_rows, cu_q, L, out, S, M, spec, eps):
+        """Sequences [0, S), token by token: memory, read-out, head norm and output gate.  ``states``: the state pool's rows,
+        ``at``: where the layer's part of a row begins; ``cu_q``: first row of every sequence (None: a row each)."""
+        H, d, vd = spec.heads, spec.dim, spec.vdim
+        g = gates.view(-1)[: M * 2 * H].view(M, 2 * H)
+        for s in range(S):
+            a, e = (s, s + 1) if cu_q is None else (int(cu_q[s]), int(cu_q[s + 1]))
+            read, write = int(state_rows[0, s]), int(state_rows[1, s])
+            row = states[read, at: at + spec.state_floats].clone() if read >= 0 else torch.zeros(
+                spec.state_floats, device=inp.device)
+            x = inp[a:e].float()
+            y = ref.memory_tokens(x[:, : H * d].reshape(-1, H, d) * d ** -0.5,
+                                  x[:, spec.k_col: spec.k_col + H * d].reshape(-1, H, d),
+                                  x[:, spec.v_col: spec.v_col + H * vd].reshape(-1, H, vd), g[a:e, :H], g[a:e, H:],
+                                  row[: H * d * vd].view(H, d, vd), row[spec.sum_at: spec.sum_at + H * d].view(H, d),
+                                  row[spec.max_at: spec.max_at + H])
+            if write >= 0:
+                states[write, at: at + spec.state_floats] = row
+            y = ref.rmsnorm_f32(y, L.head_norm.view(H, vd), eps).reshape(e - a, H * vd)
+            out[a:e, : H * vd] = y * torch.sigmoid(x[:, spec.gate_col: spec.gate_col + H * vd])
 
     def logits_finish(self, logits, M, scale, cap):
         """logits <- cap * tanh(scale * logits / cap) in place (cap 0: only scaled)."""

@@ -332,3 +332,98 @@ def route_top(logits: torch.Tensor, top: int):
 def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
     """x / sqrt(mean(x^2) + eps) * w, fp32 in and out."""
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+
+# ---- embedding with what a design adds to it ------------------------------------------------------------------------
+def previous_tokens(ids: torch.Tensor, cu_q, state_rows, last_token: torch.Tensor) -> torch.Tensor:
+    """The token before each of the packed ``ids``; -1 for the first of a sequence.  ``cu_q[s]``: first row of sequence s
+    (and the end); the token before it is ``last_token[state_rows[0, s]]``."""
+    prev = torch.cat([ids.new_zeros(1), ids[:-1]])
+    for s in range(len(cu_q) - 1):
+        read = int(state_rows[0, s])
+        prev[int(cu_q[s])] = int(last_token[read]) if read >= 0 else -1
+    return prev
+
+
+def sinusoid(positions: torch.Tensor, width: int, base: float) -> torch.Tensor:
+    """[T, width]: entry 2i is sin(p * base^(-2i/width)), entry 2i + 1 the cosine of the same angle."""
+    j = torch.arange(width, dtype=torch.float64, device=positions.device)
+    even = j - j % 2
+    ang = positions.double()[:, None] * base ** (-even / width)
+    return torch.where(j % 2 == 0, torch.sin(ang), torch.cos(ang)).float()
+
+
+# ---- attention over heads whose keys and values have their own widths ------------------------------------------------
+def heads_prep(inp: torch.Tensor, k_cache, v_cache, slots, spec, q_norm, k_norm, eps: float) -> None:
+    """Second half of the fused input projection [q | k | v | gate]: query and key norm over a head's dimensions, keys and
+    values into the cache (``k_cache`` [blocks, kv_heads, block_size, dim..]); queries are normed in place."""
+    T, H, G, d, vd = inp.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim
+    inp[:, : H * d] = rmsnorm_f32(inp[:, : H * d].float().view(T, H, d), q_norm, eps).view(T, -1).to(inp.dtype)
+    if not spec.own_kv:
+        return
+    bs = k_cache.shape[2]
+    k = rmsnorm_f32(inp[:, spec.k_col: spec.k_col + G * d].float().reshape(T, G, d), k_norm, eps)
+    v = inp[:, spec.v_col: spec.v_col + G * vd].reshape(T, G, vd)
+    ok = slots >= 0
+    s = slots[ok]
+    k_cache[s // bs, :, s % bs, :d] = k[ok].to(k_cache.dtype)
+    v_cache[s // bs, :, s % bs, :vd] = v[ok]
+
+
+def heads_attn(q: torch.Tensor, positions, k_cache, v_cache, table, spec) -> torch.Tensor:
+    """Queries [T, heads, dim] of one sequence at ``positions`` against its cached keys: [T, heads, vdim] fp32."""
+    bs, rep = k_cache.shape[2], spec.heads // spec.kv_heads
+    first = torch.tensor([spec.first_seen(int(p)) for p in positions], device=q.device)
+    pos = torch.arange(int(first.min()), int(positions.max()) + 1, device=q.device)
+    blk = table[pos // bs].long()
+    k = k_cache[blk.clamp_min(0), :, pos % bs, : spec.dim].float().repeat_interleave(rep, 1)
+    v = v_cache[blk.clamp_min(0), :, pos % bs, : spec.vdim].float().repeat_interleave(rep, 1)
+    see = (pos[None] <= positions[:, None]) & (pos[None] >= first[:, None]) & (blk >= 0)[None]
+    s = torch.einsum("thd,nhd->htn", q.float(), k) * spec.scale
+    return torch.einsum("htn,nhv->thv", torch.softmax(s.masked_fill(~see, float("-inf")), -1).nan_to_num(0.0), v)
+
+
+# ---- matrix memory (mLSTM) --------------------------------------------------------------------------------------------
+def memory_gates(z: torch.Tensor, bias: torch.Tensor, cap: float) -> torch.Tensor:
+    """Pre-activations [T, 2 * heads] of the input and forget gates -> their logarithms, fp32."""
+    H = z.shape[1] // 2
+    g = cap * torch.tanh((z.float() + bias) / cap)
+    return torch.cat([g[:, :H], torch.nn.functional.logsigmoid(g[:, H:])], 1)
+
+
+def memory_tokens(q, k, v, log_i, log_f, S, n, m):
+    """Tokens of one sequence through one layer's memory.  q, k [T, H, d] and v [T, H, vd] fp32, gates [T, H]; S [H, d, vd],
+    n [H, d], m [H] are updated in place.  Returns the read-outs [T, H, vd]."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        new = torch.maximum(log_f[t] + m, log_i[t])
+        keep, add = torch.exp(log_f[t] + m - new), torch.exp(log_i[t] - new)
+        S.mul_(keep[:, None, None]).add_((add[:, None] * k[t])[:, :, None] * v[t][:, None, :])
+        n.mul_(keep[:, None]).add_(add[:, None] * k[t])
+        m.copy_(new)
+        den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        out[t] = torch.einsum("hdv,hd->hv", S, q[t]) / den[:, None]
+    return out
+
+
+# ---- feed-forwards ----------------------------------------------------------------------------------------------------
+def relu2(x: torch.Tensor) -> torch.Tensor:
+    return torch.relu(x).square()
+
+
+def clamped_glu(g: torch.Tensor, u: torch.Tensor, limit: float) -> torch.Tensor:
+    """g sigmoid(1.702 g) (u + 1) with g clamped from above and u from both sides."""
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+
+
+def route(logits: torch.Tensor, moe):
+    """(expert ids [T, top], their weights): largest scores first, the lower id on a tie."""
+    if moe.score == "sigmoid":
+        e, w = route_top(logits, moe.top)
+    else:
+        w, e = torch.sort(torch.softmax(logits.float(), -1), dim=-1, descending=True, stable=True)
+        e, w = e[:, : moe.top], w[:, : moe.top]
+    if moe.normalise:
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    return e, w * moe.scale

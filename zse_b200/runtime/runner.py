@@ -65,6 +65,7 @@ class ModelRunner:
         self.max_attn_splits = attn_splits or (16 if on_gpu else 1)
         logits_rows = max(max_batch_seqs, 64, logits_rows)
         model.cache_block_size = cache.block_size
+        model.states = cache.states
         self.buf = model.make_buffers(self.max_tokens, max_batch_seqs, self.max_blocks, logits_rows,
                                       max_planes=8, attn_splits=self.max_attn_splits)
         self._graphs: Dict[Tuple[int, int, bool], torch.cuda.CUDAGraph] = {}
@@ -88,6 +89,7 @@ class ModelRunner:
         self.h_seed = mk(logits_rows, torch.int64)
         self.h_adapter = mk(self.max_tokens, torch.int32)
         self.h_out = mk(logits_rows, torch.int32)
+        self.h_state = mk((2, max_batch_seqs), torch.int32)      # state rows that a pass's sequences read and write
         # pipelined decode: tokens (and the device status word) of a step are copied out behind the step itself and
         # read after an event, into alternating buffers, while the next step already runs
         self.h_out2 = [mk(logits_rows, torch.int32), mk(logits_rows, torch.int32)]
@@ -117,6 +119,15 @@ class ModelRunner:
             if ev is None:
                 ev = self._staged = torch.cuda.Event()
             ev.record()
+
+    def _stage_states(self, spans, n_pad: int) -> None:
+        """Models with recurrent state: the rows of the state pool that the sequences of the pass read and write."""
+        if self.cache.states is None:
+            return
+        h = self.h_state.numpy()
+        self.cache.stage_states(spans, h[0], h[1])
+        h[:, len(spans): n_pad] = -1
+        self.buf.state_rows[:, :n_pad].copy_(self.h_state[:, :n_pad], non_blocking=True)
 
     def _upload(self, dst: torch.Tensor, src: torch.Tensor, n) -> None:
         dst[:n].copy_(src[:n], non_blocking=True)
@@ -237,6 +248,7 @@ class ModelRunner:
                             (b.logit_rows, self.h_rows, n_rows)):
             self._upload(dst, src, n)
         self._stage_adapters(per_tok_adapter, total, total)
+        self._stage_states([(items[i][0], items[i][2], len(items[i][1])) for i in order], S)
         self.model.stage_prefill(b, [(items[i][2], len(items[i][1])) for i in order])
         greedy = self._stage_sampling(sampling or [GREEDY] * n_rows, n_rows) if select else True
         self._staging_end()
@@ -326,6 +338,8 @@ class ModelRunner:
             self._upload(self._src_rows, self.h_src, Sp)
             torch.index_select(b.out_tokens, 0, self._src_rows[:Sp], out=b.ids[:Sp])
         self._stage_adapters(adapters, S, Sp)
+        if cache.states is not None:
+            self._stage_states([(sid, int(p), 1) for sid, p in zip(seq_ids, n_["pos"][:S])], Sp)
         greedy = self._stage_sampling(sampling or [GREEDY] * S, Sp)
         self._staging_end()
         splits = self._pick_splits(Sp, max_len)

@@ -73,6 +73,7 @@ class SpeculativeRunner:
             toks, _ = runner.prefill(items[i:j], all_logits=True,
                                      adapters=None if adapters is None else list(adapters[i:j]))
             at = 0
+            replay = []
             for idx in range(i, j):
                 r, prop = reqs[idx], drafts[idx]
                 n = 1 + len(prop)
@@ -83,6 +84,8 @@ class SpeculativeRunner:
                 # KV now holds last + all drafts; keep last + accepted drafts
                 keep = items[idx][2] + 1 + res.num_accepted
                 cache.truncate_sequence(r.seq_id, keep)
+                if cache.states is not None and res.num_accepted < len(prop):
+                    replay.append((items[idx][0], items[idx][1][: 1 + res.num_accepted], items[idx][2]))
                 d = self._drafts[r.request_id]
                 for t in res.accepted_tokens:
                     if r.is_finished:
@@ -94,6 +97,9 @@ class SpeculativeRunner:
                     # tokens after a stop are dropped; the cache is freed by the batch runner anyway
                     pass
                 self.seq_steps += 1
+            if replay:
+                # recurrent state has gone past the rejected drafts: run the accepted tokens again from the state before
+                runner.prefill(replay, select=False)
             i = j
         self.tokens_emitted += emitted
         return emitted

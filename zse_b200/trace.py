@@ -35,7 +35,7 @@ class TraceRunner:
         self.engine = ZStreamerEngine(model, config=EngineConfig(
             dtype=dtype, device=device, block_size=block, kv_blocks=tokens // block, max_seq_len=tokens,
             max_batch_seqs=max_live, max_batch_tokens=tokens, prefill_chunk_size=0, logits_rows=tokens,
-            enable_prefix_cache=False))
+            enable_prefix_cache=False, state_slots=max_live))
         self._seq: Dict[str, int] = {}
         self._next = 0
 
