@@ -62,8 +62,8 @@ typedef struct ZseTileGemm {
   int64_t ldb_n, ldb_k, b_batch, b_group;
   void* out;                // row stride ldo, batch stride o_batch; row m goes to out_rows[m] or m * out_row_mul + add
   int64_t ldo, o_batch;
-  int32_t M, N, K, epilogue;   // 0 store, 1 fp32 store, 2 gelu(row_scale * acc), 3 acc * sigmoid(gate)
-  const float* row_scale;
+  int32_t M, N, K, epilogue;   // 0 store, 1 fp32 store, 2 gelu, 3 times sigmoid(gate), 4 square of relu
+  const float* row_scale;      // factor of a row of the product, or null
   const int32_t* out_rows;
   int32_t out_row_mul, out_row_add;
   const void* gate;
@@ -72,6 +72,8 @@ typedef struct ZseTileGemm {
   const int32_t* n_tiles;
 } ZseTileGemm;
 int zse_gemm_tile(int dtype, const ZseTileGemm* a, int batch, int max_tiles, void* stream);
+// in [rows, 2 * ff] (gate, up) -> out [rows, ff] = g sigmoid(1.702 g) (u + 1), g clamped from above and u from both sides
+int zse_clamped_glu(int dtype, const void* in, void* out, int rows, int ff, float limit, void* stream);
 
 int zse_apply_repetition_penalty_f32(void* logits, int ld, const void* rows_i32, const void* tokens_i32,
                                      const void* counts_i32, int n, const void* penalty_f32, int V, void* stream);
@@ -82,6 +84,23 @@ int zse_embedding_typed(int dtype, const void* table, const void* ids, void* out
 // residual += planes [n_planes][M][H] + slots [M][n_slots][H]; out = RMSNorm(residual) * weight
 int zse_add_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes, const void* slots,
                  int n_slots, const void* weight, void* out, int M, int H, float eps, void* stream);
+// y = planes + slots; residual += RMSNorm(y) * weight; out = residual, or (next not null) RMSNorm(residual) * next
+int zse_post_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes, const void* slots,
+                  int n_slots, const void* weight, const void* next, void* out, int M, int H, float eps, void* stream);
+typedef struct ZseEmbed {
+  const void *table, *bigram;   // [vocab, H], [buckets + 1, H] or null
+  const void* norm;
+  const void* turns;            // [ceil(H / 2)] pairs of floats: high and low part of the turns per token
+  const void *ids, *positions;
+  const void *row_seq, *cu_q;   // null: every row is a sequence of its own
+  const void* state_rows;       // [2][state_ld]: rows of last_token that sequences read and write (-1: none)
+  void* last_token;
+  void *residual, *out;
+  int64_t buckets, mul_prev, mul_cur;
+  int32_t H, vocab, state_ld;
+  float scale, eps;
+} ZseEmbed;
+int zse_embed_design(int dtype, const ZseEmbed* a, int M, void* status, void* stream);
 // fp32 logits in place: cap * tanh(scale * x / cap) (cap 0: scale * x)
 int zse_logits_finish(void* logits, int ld, int M, int V, float scale, float cap, void* stream);
 int zse_argmax_f32(const void* logits, int ld, void* out_i32, int M, int V, void* stream);
@@ -121,19 +140,75 @@ int zse_latent_chunk(const void* inp, int ld, const void* kvx, int ldkv, int v_c
 // ---- moe.cu -------------------------------------------------------------------------------------------------
 int zse_moe_tile_rows(int M, int E, int top);
 // router logits (fp32 planes) -> chosen experts, sorted rows, tile table; `counts` [E] must be zero and is zero afterwards
-int zse_moe_route(int dtype, const void* planes, int n_planes, int M, int E, int top, int tile_rows, const void* x, int H,
-                  int out_per_token, void* counts, void* slot_expert, void* slot_rank, void* slot_score,
-                  void* first_row, void* tiles, void* n_tiles, void* xs, void* row_score, void* out_rows, void* stream);
+typedef struct ZseRouter {
+  const void* planes;         // fp32 logits [n_planes][M][cols]; column `experts`, if there is one: the shared expert's gate
+  int32_t n_planes, experts, cols, top;
+  int32_t softmax;            // scores: 0 sigmoid, 1 softmax over the experts
+  int32_t normalise;          // weights: the chosen scores divided by their sum
+  float scale;                // ... times this
+} ZseRouter;
+int zse_moe_route(int dtype, const ZseRouter* r, int M, int tile_rows, const void* x, int H, int out_per_token, void* counts,
+                  void* slot_expert, void* slot_rank, void* slot_score, void* first_row, void* tiles, void* n_tiles,
+                  void* xs, void* row_score, void* out_rows, void* shared_score, void* stream);
 typedef struct ZseMoeGemm {
   const void *routed_w, *routed_x;
   void* routed_out;
   const void *shared_w, *shared_x;
   void* shared_out;
   const void *row_score, *out_rows, *tiles, *n_tiles;
+  const void* shared_score;   // per token, or null
   int32_t routed_n, routed_k, routed_ldo, shared_n, shared_k, shared_ldo, shared_mul, shared_add, shared_x_rows;
+  int32_t routed_cols, shared_cols;     // clamped_glu: output columns (weight rows: tiles of 64 gate rows and 64 up rows)
+  float routed_limit, shared_limit;
 } ZseMoeGemm;
 int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int tile_rows, int max_tiles, int epilogue,
                  void* status, void* stream);
+
+// ---- heads.cu -----------------------------------------------------------------------------------------------
+typedef struct ZseHeads {
+  void *k, *v;                  // cached keys and values: element (block, kv head, token, d) at block * block_stride +
+  int64_t block_stride;         //   (head * block_size + token) * dim_pad + d (values: vdim_pad)
+  int32_t block_size, dim_pad, vdim_pad, max_blocks;
+  const void* tables;           // block tables [sequences][max_blocks], -1: a hole
+  int32_t heads, kv_heads, dim, vdim, chunk, window;
+  float scale;
+} ZseHeads;
+// 1 when the tensor-core kernels take this shape (bfloat16)
+int zse_heads_mma_ok(int dim, int vdim, int block_size);
+// columns of a projected row: q from 0, k from k_col, v from v_col, gate from gate_col (gate_w of them); own_kv 0: no keys
+// and values of its own
+int zse_heads_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, int M, const ZseHeads* h,
+                   const void* slots, const void* q_norm, const void* k_norm, int k_col, int v_col, int gate_col,
+                   int gate_w, int own_kv, float eps, void* stream);
+// rows [0, M) one by one; gate: first element of the gates (row stride ld), or null
+int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads* h, const void* row_seq, const void* positions,
+                   void* out, int ldo, const void* gate, void* scratch, int M, int num_splits, int tensor_cores,
+                   void* stream);
+// rows of the sequences [first, last) in tiles of queries (bfloat16)
+int zse_heads_attn_chunks(const void* inp, int ld, const ZseHeads* h, const void* cu_q, const void* q_pos0, int first,
+                          int last, int max_q, void* out, int ldo, const void* gate, void* stream);
+
+// ---- memory.cu ----------------------------------------------------------------------------------------------
+typedef struct ZseMemory {
+  int32_t heads, dim, vdim;
+  int32_t k_col, v_col, gate_col, if_col;   // columns of a projected row (q from 0); if_col: input gates, then forget gates
+  void* states;                 // state rows, row_floats apart; this layer's part: memory at 0, key sum at sum_at, max at max_at
+  int64_t row_floats;
+  int32_t sum_at, max_at;
+  const void* state_rows;       // [2][state_ld]: rows that sequences read and write (-1: none)
+  int32_t state_ld;
+  float gate_cap, eps;
+  const void* head_norm;        // [heads * vdim], activations' type
+} ZseMemory;
+int zse_memory_chunk_ok(int dim, int vdim);
+int zse_memory_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, const void* gate_planes,
+                    int n_gate_planes, const void* if_bias, void* gates, const ZseMemory* m, int M, void* stream);
+// sequences [0, S), token by token: update, read-out, head norm, output gate; cu_q null: a row each
+int zse_memory_tokens(int dtype, const void* inp, int ld, const void* gates, const ZseMemory* m, const void* cu_q, int S,
+                      void* out, int ldo, void* stream);
+// sequences [first, last) chunkwise (bfloat16): read-outs to o [M, heads * vdim] fp32, then head norm and output gate
+int zse_memory_chunks(const void* inp, int ld, const void* gates, const ZseMemory* m, const void* cu_q, int first, int last,
+                      void* o, int M, int first_row_of_first, void* out, int ldo, void* stream);
 
 // ---- repack.cu ----------------------------------------------------------------------------------------------
 // Row-major INT4 [N, K/2] + scales/zeros [N, K/128] -> tiled chunks.  interleave_rows > 0 builds a fused gate/up

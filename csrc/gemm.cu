@@ -95,7 +95,9 @@ __device__ __forceinline__ void epilogue(const GemmArgs& a, uint32_t tmem_acc, i
       const int t = t0 + col0 + c + i;
       if (t < a.M && n_ok) {
         const float v = __uint_as_float(r[i]);
-        if (EPI == kEpiF16 && BF16) {
+        if (EPI == kEpiRelu2) {
+          reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n] = __float2bfloat16_rn(relu2(v));
+        } else if (EPI == kEpiF16 && BF16) {
           reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n] = __float2bfloat16_rn(v);
         } else if (EPI == kEpiF16) {
           reinterpret_cast<__half*>(a.out)[size_t(t) * a.ldo + n] = __float2half_rn(clamp_f16(v + bias));
@@ -340,6 +342,8 @@ static int gemm_16bit(const void* w, int w_rows_cap, const void* x, int x_rows_c
   int rc = ZSE_ERR_SHAPE;
   if (epilogue == kEpiF16) {
     ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiF16, BF16>(tw, tx, a, grid, st)))
+  } else if (epilogue == kEpiRelu2) {
+    if constexpr (BF16) ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiRelu2, BF16>(tw, tx, a, grid, st)))
   } else {
     ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiPartialF32, BF16>(tw, tx, a, grid, st)))
   }

@@ -12,7 +12,8 @@ constexpr int kW4StageK = 128;       // K per pipeline stage of the INT4 kernel 
 constexpr int kW4ChunkBytes = 8704;  // 8192 nibble bytes + 512 bytes of {scale, zero}
 constexpr int kGemmThreads = 320;    // fp16 kernel: warp 0 producer, warp 1 MMA issuer, warps 2..9 epilogue
 
-enum Epilogue : int { kEpiF16 = 0, kEpiSwiGLU = 1, kEpiPartialF32 = 2, kEpiPushF16 = 3, kEpiScatterF16 = 4 };
+enum Epilogue : int { kEpiF16 = 0, kEpiSwiGLU = 1, kEpiPartialF32 = 2, kEpiPushF16 = 3, kEpiScatterF16 = 4,
+                     kEpiRelu2 = 5 /* bfloat16: store the square of relu */ };
 
 struct GemmArgs {
   const uint8_t* w;        // W4: tiled chunks [n_tiles][k_stages][8704]; F16: unused (tensor map)

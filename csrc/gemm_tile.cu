@@ -1,11 +1,11 @@
 // General matrix product on the CUDA cores, fp32 arithmetic throughout: any sizes, strides and alignments, batched over
 // heads or grouped by expert.
 //
-//   out[m, n] = epilogue( sum_k A[m, k] * B[n, k] )          A, B bfloat16 or float
+//   out[m, n] = epilogue( scale[m] * sum_k A[m, k] * B[n, k] )          A, B bfloat16 or float
 //
 // It is the path of models that run in float, and of bfloat16 shapes whose rows are no multiple of 16 bytes (which TMA
-// cannot address).  Epilogues: 0 store in the activation type, 1 store fp32, 2 gelu(scale[m] * acc), 3 acc *
-// sigmoid(gate[m, n]).
+// cannot address).  Epilogues: 0 store in the activation type, 1 store fp32, 2 gelu, 3 times sigmoid(gate[m, n]), 4 the
+// square of relu.
 #include "api.h"
 #include "moe.cuh"
 #include "typed.cuh"
@@ -76,13 +76,14 @@ __global__ void __launch_bounds__(256) gemm_tile_kernel(const ZseTileGemm a) {
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= a.N) continue;
-      float v = acc[i][j];
+      float v = acc[i][j] * sc;
       const size_t at = om * a.ldo + z * a.o_batch + n;
       if (a.epilogue == 1) {
         reinterpret_cast<float*>(a.out)[at] = v;
         continue;
       }
-      if (a.epilogue == 2) v = gelu_exact(v * sc);
+      if (a.epilogue == 2) v = gelu_exact(v);
+      if (a.epilogue == 4) v = relu2(v);
       if (a.epilogue == 3)
         v *= sigmoid_exact(to_f32(reinterpret_cast<const T*>(a.gate)[size_t(m) * a.ldg + z * a.gate_batch + n]));
       reinterpret_cast<T*>(a.out)[at] = from_f32<T>(v);
@@ -90,10 +91,37 @@ __global__ void __launch_bounds__(256) gemm_tile_kernel(const ZseTileGemm a) {
   }
 }
 
+// in [rows, 2 * ff] (gate, up) -> out [rows, ff]
+template <typename T>
+__global__ void __launch_bounds__(256)
+clamped_glu_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, int ff, float limit) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
+    const T* g = in + i / ff * 2 * ff + i % ff;
+    out[i] = from_f32<T>(clamped_glu(to_f32(g[0]), to_f32(g[ff]), limit));
+  }
+}
+
 }  // namespace
 }  // namespace zse
 
 using namespace zse;
+
+extern "C" int zse_clamped_glu(int dtype, const void* in, void* out, int rows, int ff, float limit, void* stream) {
+  const long long n = (long long)(rows) * ff;
+  if (n <= 0) return 0;
+  const dim3 grid(unsigned(n + 255 < 4096ll * 256 ? (n + 255) / 256 : 4096));
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  cudaError_t e;
+  if (dtype == kBF16)
+    e = launch_pdl(clamped_glu_kernel<bf16>, grid, dim3(256), 0, st, reinterpret_cast<const bf16*>(in),
+                   reinterpret_cast<bf16*>(out), n, ff, limit);
+  else
+    e = launch_pdl(clamped_glu_kernel<float>, grid, dim3(256), 0, st, reinterpret_cast<const float*>(in),
+                   reinterpret_cast<float*>(out), n, ff, limit);
+  return e == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+}
 
 extern "C" int zse_gemm_tile(int dtype, const ZseTileGemm* a, int batch, int max_tiles, void* stream) {
   const int my = a->tiles != nullptr ? max_tiles : (a->M + kBM - 1) / kBM;

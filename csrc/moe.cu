@@ -1,7 +1,7 @@
 // Routed feed-forward: which tokens go to which expert, and the experts' products.
 //
-//   topk      sigmoid scores of the router's fp32 logits, the `top` largest per token (lower id first on a tie), and each
-//             (token, choice) slot's place within its expert
+//   topk      scores of the router's fp32 logits (sigmoid, or softmax over the experts), the `top` largest per token (lower
+//             id first on a tie), their weights, and each (token, choice) slot's place within its expert
 //   plan      one CTA: first row of every expert in the sorted order, table of token tiles for the grouped products
 //   permute   the tokens' rows, copied into sorted order, with the score and the slot of each sorted row
 //   products  grouped GEMM on tcgen05 (moe_gemm_kernel), the shared expert's dense product in the same launch
@@ -19,21 +19,42 @@ namespace {
 
 constexpr int kTopkWarps = 8;
 
+// Router rows are `cols` wide: column E, if there is one, is the shared expert's gate, whose sigmoid goes to shared_score.
 __global__ void __launch_bounds__(kTopkWarps * 32)
-moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, int top, int* __restrict__ counts,
-                int* __restrict__ slot_expert, int* __restrict__ slot_rank, float* __restrict__ slot_score) {
+moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, int cols, int top, int softmax, int normalise,
+                float scale, int* __restrict__ counts, int* __restrict__ slot_expert, int* __restrict__ slot_rank,
+                float* __restrict__ slot_score, float* __restrict__ shared_score) {
   extern __shared__ float scores[];
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kTopkWarps + warp;
   if (t >= M) return;
-  float* s = scores + warp * E;
-  for (int e = lane; e < E; e += 32) {
+  float* s = scores + warp * (E + top);
+  float* chosen = s + E;
+  auto logit = [&](int e) {
     float z = 0.f;
-    for (int p = 0; p < n_planes; ++p) z += planes[(size_t(p) * M + t) * E + e];
-    s[e] = sigmoid_exact(z);
+    for (int p = 0; p < n_planes; ++p) z += planes[(size_t(p) * M + t) * cols + e];
+    return z;
+  };
+  float most = -INFINITY;
+  for (int e = lane; e < E; e += 32) {
+    const float z = logit(e);
+    s[e] = softmax ? z : sigmoid_exact(z);
+    most = fmaxf(most, z);
   }
+  if (cols > E && lane == 0) shared_score[t] = sigmoid_exact(logit(E));
+  if (softmax) {
+    most = warp_max(most);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      s[e] = expf(s[e] - most);
+      sum += s[e];
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) s[e] /= sum;
+  }
+  float total = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -2.f;
     int at = 0x7fffffff;
@@ -57,9 +78,13 @@ moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, in
       const int slot = t * top + k;
       slot_expert[slot] = at;
       slot_rank[slot] = atomicAdd(&counts[at], 1);
-      slot_score[slot] = best;
+      chosen[k] = best;
     }
+    total += best;
   }
+  __syncwarp();
+  const float w = normalise ? scale / (total + 1e-20f) : scale;
+  for (int k = lane; k < top; k += 32) slot_score[t * top + k] = chosen[k] * w;
 }
 
 constexpr int kPlanThreads = 1024;
@@ -149,7 +174,9 @@ struct MoeProduct {
   int N, K;                 // weight rows of a group, reduction length
   void* out;
   int ldo;                  // output row stride
-  const float* row_scale;   // per token row (up) or null
+  int cols;                 // output columns (kMoeGlu: half of N, or less where N is padded)
+  float limit;              // kMoeGlu
+  const float* row_scale;   // per token row, or null: before the activation (up), on the result (down)
   const int* out_rows;      // output row of a token row, or null: row * mul + add
   int mul, add;
 };
@@ -178,7 +205,8 @@ struct MoeBars {
   int abort_flag;
 };
 
-enum MoeEpi { kMoeUp = 0, kMoeDown = 1 };     // gelu(score * acc) -> bf16; acc -> OutT
+// gelu(scale * acc) -> bf16; scale * acc -> OutT; clamped_glu -> bf16 (a tile of W: 64 gate rows, then their 64 up rows)
+enum MoeEpi { kMoeUp = 0, kMoeDown = 1, kMoeGlu = 2 };
 
 template <int NT, int EPI, typename OutT>
 __global__ void __launch_bounds__(kGemmThreads, MoeCfg<NT>::kMinBlocks)
@@ -270,8 +298,46 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
     const int q = warp & 3, ch = (warp - 2) >> 2;
     constexpr int kCols = NT >= 32 ? NT / 2 : NT;
     const bool mine = __all_sync(0xffffffffu, ok && (NT >= 32 || ch == 0));
+    if constexpr (EPI == kMoeGlu) {
+      // warps with up rows (q = 2, 3) park them in shared memory, their partners with the gate rows combine; a warp with
+      // nothing to do still meets its partner
+      float* park = reinterpret_cast<float*>(smem) + ((q & 1) + 2 * ch) * (32 * kCols);
+      const int bar = 1 + (q & 1) + 2 * ch;
+      const bool work = mine && ch * kCols < tile.rows;
+      if (q >= 2) {
+        if (work) {
+#pragma unroll 1
+          for (int c = 0; c < kCols && ch * kCols + c < tile.rows; c += 16) {
+            uint32_t r[16];
+            ZSE_TMEM_LD_X16(r, tmem + (uint32_t(q * 32) << 16) + ch * kCols + c);
+            tc_wait_ld();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) park[(c + i) * 32 + lane] = __uint_as_float(r[i]);
+          }
+        }
+        asm volatile("bar.sync %0, 64;" ::"r"(bar) : "memory");
+      } else {
+        asm volatile("bar.sync %0, 64;" ::"r"(bar) : "memory");
+        const int n = blockIdx.x * 64 + q * 32 + lane;
+        if (work) {
+#pragma unroll 1
+          for (int c = 0; c < kCols && ch * kCols + c < tile.rows; c += 16) {
+            uint32_t r[16];
+            ZSE_TMEM_LD_X16(r, tmem + (uint32_t(q * 32) << 16) + ch * kCols + c);
+            tc_wait_ld();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+              const int col = ch * kCols + c + i;
+              if (col < tile.rows && n < p.cols)
+                reinterpret_cast<OutT*>(p.out)[size_t(tile.row0 + col) * p.ldo + n] =
+                    from_f32<OutT>(clamped_glu(__uint_as_float(r[i]), park[(c + i) * 32 + lane], p.limit));
+            }
+          }
+        }
+      }
+    }
     const int n = n0 + q * 32 + lane;
-    if (mine && ch * kCols < tile.rows) {
+    if (EPI != kMoeGlu && mine && ch * kCols < tile.rows) {
 #pragma unroll 1
       for (int c = 0; c < kCols; c += 16) {
         if (ch * kCols + c >= tile.rows) break;
@@ -284,7 +350,8 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
           if (col < tile.rows && n < p.N) {
             const int row = tile.row0 + col;
             float v = __uint_as_float(r[i]);
-            if (EPI == kMoeUp) v = gelu_exact(p.row_scale != nullptr ? v * p.row_scale[row] : v);
+            if (p.row_scale != nullptr) v *= p.row_scale[row];
+            if (EPI == kMoeUp) v = gelu_exact(v);
             const size_t orow = p.out_rows != nullptr ? p.out_rows[row] : size_t(row) * p.mul + p.add;
             reinterpret_cast<OutT*>(p.out)[orow * p.ldo + n] = from_f32<OutT>(v);
           }
@@ -317,18 +384,20 @@ int launch_moe(const CUtensorMap* m, const MoeGemmArgs& a, dim3 grid, cudaStream
 using namespace zse;
 #define ST(s) reinterpret_cast<cudaStream_t>(s)
 
-extern "C" int zse_moe_route(int dtype, const void* planes, int n_planes, int M, int E, int top, int tile_rows,
-                             const void* x, int H, int out_per_token, void* counts, void* slot_expert, void* slot_rank,
-                             void* slot_score, void* first_row, void* tiles, void* n_tiles, void* xs, void* row_score,
-                             void* out_rows, void* stream) {
+extern "C" int zse_moe_route(int dtype, const ZseRouter* r, int M, int tile_rows, const void* x, int H, int out_per_token,
+                             void* counts, void* slot_expert, void* slot_rank, void* slot_score, void* first_row,
+                             void* tiles, void* n_tiles, void* xs, void* row_score, void* out_rows, void* shared_score,
+                             void* stream) {
+  const int E = r->experts, top = r->top;
   if (M <= 0) return 0;
-  if (E <= 0 || top <= 0 || top > E || tile_rows <= 0 || E > 1024) return ZSE_ERR_SHAPE;
+  if (E <= 0 || top <= 0 || top > E || tile_rows <= 0 || E + top > 1536) return ZSE_ERR_SHAPE;
   cudaStream_t st = ST(stream);
-  const size_t smem = size_t(kTopkWarps) * E * sizeof(float);
+  const size_t smem = size_t(kTopkWarps) * (E + top) * sizeof(float);
   if (launch_pdl(moe_topk_kernel, dim3((M + kTopkWarps - 1) / kTopkWarps), dim3(kTopkWarps * 32), smem, st,
-                 reinterpret_cast<const float*>(planes), n_planes, M, E, top, reinterpret_cast<int*>(counts),
-                 reinterpret_cast<int*>(slot_expert), reinterpret_cast<int*>(slot_rank),
-                 reinterpret_cast<float*>(slot_score)) != cudaSuccess)
+                 reinterpret_cast<const float*>(r->planes), r->n_planes, M, E, r->cols, top, r->softmax, r->normalise,
+                 r->scale, reinterpret_cast<int*>(counts), reinterpret_cast<int*>(slot_expert),
+                 reinterpret_cast<int*>(slot_rank), reinterpret_cast<float*>(slot_score),
+                 reinterpret_cast<float*>(shared_score)) != cudaSuccess)
     return ZSE_ERR_LAUNCH;
   if (launch_pdl(moe_plan_kernel, dim3(1), dim3(kPlanThreads), 0, st, reinterpret_cast<int*>(counts), E, tile_rows,
                  reinterpret_cast<int*>(first_row), reinterpret_cast<MoeTile*>(tiles),
@@ -357,7 +426,8 @@ extern "C" int zse_moe_tile_rows(int M, int E, int top) {
   return want <= 16 ? 16 : want <= 32 ? 32 : want <= 64 ? 64 : want <= 160 ? 128 : 256;
 }
 
-// Up (epilogue 0: gelu(score * acc) in bfloat16) or down (1: bfloat16, 2: fp32 result rows) products of all experts.
+// Up (epilogue 0: gelu(scale * acc) in bfloat16; 3: clamped_glu) or down (1: bfloat16, 2: fp32 result rows) products of all
+// experts.
 extern "C" int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int tile_rows, int max_tiles, int epilogue,
                             void* status, void* stream) {
   if (M <= 0) return 0;
@@ -373,11 +443,12 @@ extern "C" int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int
     if (int rc = get_tmap(g->shared_x, g->shared_x_rows, g->shared_k, tile_rows, &m[3])) return rc;
   }
   MoeGemmArgs a{};
-  a.routed = MoeProduct{g->routed_n, g->routed_k, g->routed_out, g->routed_ldo,
+  if (epilogue == 3 && (g->routed_n % kTileN || (shared && g->shared_n % kTileN))) return ZSE_ERR_SHAPE;
+  a.routed = MoeProduct{g->routed_n, g->routed_k, g->routed_out, g->routed_ldo, g->routed_cols, g->routed_limit,
                         reinterpret_cast<const float*>(g->row_score), reinterpret_cast<const int*>(g->out_rows), 1, 0};
   if (shared)
-    a.shared = MoeProduct{g->shared_n, g->shared_k, g->shared_out, g->shared_ldo, nullptr, nullptr, g->shared_mul,
-                          g->shared_add};
+    a.shared = MoeProduct{g->shared_n, g->shared_k, g->shared_out, g->shared_ldo, g->shared_cols, g->shared_limit,
+                          reinterpret_cast<const float*>(g->shared_score), nullptr, g->shared_mul, g->shared_add};
   a.tiles = reinterpret_cast<const MoeTile*>(g->tiles);
   a.n_tiles = reinterpret_cast<const int*>(g->n_tiles);
   a.dense_tiles = shared ? (M + tile_rows - 1) / tile_rows : 0;
@@ -392,6 +463,8 @@ extern "C" int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int
     ZSE_MOE(kMoeUp, bf16)
   } else if (epilogue == 1) {
     ZSE_MOE(kMoeDown, bf16)
+  } else if (epilogue == 3) {
+    ZSE_MOE(kMoeGlu, bf16)
   } else {
     ZSE_MOE(kMoeDown, float)
   }

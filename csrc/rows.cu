@@ -1,5 +1,7 @@
-// Row kernels for activations of bfloat16 or float: embedding, residual sum + RMSNorm, logits epilogue, arg-max of
-// fp32 logits.  Any row length.
+// Row kernels for activations of bfloat16 or float: embedding (plain, or with a bigram table, a sinusoid and a norm),
+// residual sum + RMSNorm, RMSNorm + residual sum, logits epilogue, arg-max of fp32 logits.  Any row length.
+#include <initializer_list>
+
 #include "api.h"
 #include "typed.cuh"
 
@@ -28,47 +30,23 @@ __global__ void embedding_typed_kernel(const T* __restrict__ table, const int* _
 constexpr int kRowThreads = 256;
 constexpr int kRowRegs = 8;          // accesses per thread: H <= 8 * VEC * 256 * cluster
 
-template <int VEC>
-struct F32Vec {
-  float v[VEC];
-};
-template <int VEC>
-__device__ __forceinline__ F32Vec<VEC> load_vec(const float* p) {
-  F32Vec<VEC> r;
-  if constexpr (VEC == 4) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w;
-  } else {
-    r.v[0] = p[0];
+// Sum of a value over the CTAs of the cluster (every thread of a CTA holds the CTA's value).
+__device__ __forceinline__ float row_cluster_sum(float total, float* slot, int cs) {
+  if (cs == 1) return total;
+  if (threadIdx.x == 0) *slot = total;
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+  total = 0.f;
+  const uint32_t local = smem_u32(slot);
+  for (int r = 0; r < cs; ++r) {                           // same order in every CTA: identical sums
+    uint32_t remote;
+    float t;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(r));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(t) : "r"(remote) : "memory");
+    total += t;
   }
-  return r;
-}
-template <int VEC>
-__device__ __forceinline__ F32Vec<VEC> load_vec(const bf16* p) {
-  F32Vec<VEC> r;
-  if constexpr (VEC == 4) {
-    const uint2 x = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
-    r.v[0] = a.x; r.v[1] = a.y; r.v[2] = b.x; r.v[3] = b.y;
-  } else {
-    r.v[0] = to_f32(p[0]);
-  }
-  return r;
-}
-template <int VEC>
-__device__ __forceinline__ void store_vec(float* p, const F32Vec<VEC>& r) {
-  if constexpr (VEC == 4)
-    *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
-  else
-    p[0] = r.v[0];
-}
-template <int VEC>
-__device__ __forceinline__ void store_vec(bf16* p, const F32Vec<VEC>& r) {
-  if constexpr (VEC == 4)
-    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(r.v[0], r.v[1]), pack_bf16(r.v[2], r.v[3]));
-  else
-    p[0] = from_f32<bf16>(r.v[0]);
+  // nobody exits while its value may still be read
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+  return total;
 }
 
 template <typename T, typename S, int VEC>
@@ -113,21 +91,7 @@ add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, 
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
   __syncthreads();
   float total = warp_sum((threadIdx.x & 31) < (kRowThreads >> 5) ? red[threadIdx.x & 31] : 0.f);
-  if (cs > 1) {
-    if (threadIdx.x == 0) cluster_ss = total;
-    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-    total = 0.f;
-    const uint32_t local = smem_u32(&cluster_ss);
-    for (int r = 0; r < cs; ++r) {                         // same order in every CTA: identical sums
-      uint32_t remote;
-      float t;
-      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(r));
-      asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(t) : "r"(remote) : "memory");
-      total += t;
-    }
-    // nobody exits while its value may still be read
-    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-  }
+  total = row_cluster_sum(total, &cluster_ss, cs);
   const float inv = 1.f / sqrtf(total / float(H) + eps);
 #pragma unroll
   for (int j = 0; j < kRowRegs; ++j) {
@@ -141,11 +105,10 @@ add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, 
   }
 }
 
-template <typename T, typename S>
-int launch_add_norm(void* residual, const void* planes, int n_planes, const void* slots, int n_slots,
-                    const void* weight, void* out, int M, int H, float eps, cudaStream_t st) {
-  const bool vec = H % 4 == 0 && !((reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(out) |
-                                    reinterpret_cast<uintptr_t>(residual)) & 15);
+// Launch over (cluster, rows) with VEC 4 where sizes and addresses allow it.
+template <typename K, typename... Args>
+int launch_rows(K vec_kern, K any_kern, bool aligned, int M, int H, cudaStream_t st, Args... args) {
+  const bool vec = H % 4 == 0 && aligned;
   const int n = vec ? H / 4 : H;
   int cs = 1;
   while (cs < 8 && ((M * cs < 256 && n / (cs * 2) >= 64) || (n + cs - 1) / cs > kRowThreads * kRowRegs)) cs *= 2;
@@ -163,10 +126,187 @@ int launch_add_norm(void* residual, const void* planes, int n_planes, const void
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = pdl_enabled() ? 2 : 1;
-  auto kern = vec ? add_norm_kernel<T, S, 4> : add_norm_kernel<T, S, 1>;
-  return cudaLaunchKernelEx(&cfg, kern, reinterpret_cast<float*>(residual), reinterpret_cast<const float*>(planes),
-                            n_planes, reinterpret_cast<const S*>(slots), n_slots, reinterpret_cast<const T*>(weight),
-                            reinterpret_cast<T*>(out), M, H, eps) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+  return cudaLaunchKernelEx(&cfg, vec ? vec_kern : any_kern, args...) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+}
+
+inline bool aligned16(std::initializer_list<const void*> ps) {
+  for (const void* p : ps)
+    if (reinterpret_cast<uintptr_t>(p) & 15) return false;
+  return true;
+}
+
+template <typename T, typename S>
+int launch_add_norm(void* residual, const void* planes, int n_planes, const void* slots, int n_slots,
+                    const void* weight, void* out, int M, int H, float eps, cudaStream_t st) {
+  return launch_rows(add_norm_kernel<T, S, 4>, add_norm_kernel<T, S, 1>, aligned16({residual, weight, out}), M, H, st,
+                     reinterpret_cast<float*>(residual), reinterpret_cast<const float*>(planes), n_planes,
+                     reinterpret_cast<const S*>(slots), n_slots, reinterpret_cast<const T*>(weight),
+                     reinterpret_cast<T*>(out), M, H, eps);
+}
+
+// y = sum of fp32 planes + sum of the row's slots; residual += RMSNorm(y) * weight; out = residual, or (next != null)
+// RMSNorm(residual) * next.  Rows are split as in add_norm_kernel.
+template <typename T, typename S, int VEC>
+__global__ void __launch_bounds__(kRowThreads)
+post_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, int n_planes,
+                 const S* __restrict__ slots, int n_slots, const T* __restrict__ weight, const T* __restrict__ next,
+                 T* __restrict__ out, int M, int H, float eps) {
+  __shared__ float red[2][32];
+  __shared__ float cluster_ss[2];
+  pdl_launch_dependents();
+  const int row = blockIdx.y, cs = gridDim.x;
+  const int nv = (H / VEC + cs - 1) / cs;
+  const int v0 = blockIdx.x * nv, v1 = min(H / VEC, v0 + nv);
+  const size_t base = size_t(row) * H, plane = size_t(M) * H;
+  pdl_wait();
+  F32Vec<VEC> x[kRowRegs];
+  auto total_of = [&](float ss, int k) {
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[k][threadIdx.x >> 5] = ss;
+    __syncthreads();
+    const float t = warp_sum((threadIdx.x & 31) < (kRowThreads >> 5) ? red[k][threadIdx.x & 31] : 0.f);
+    return row_cluster_sum(t, &cluster_ss[k], cs);
+  };
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < kRowRegs; ++j) {
+    const int i = v0 + threadIdx.x + j * kRowThreads;
+    if (i < v1) {
+      const size_t at = base + size_t(i) * VEC;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[j].v[e] = 0.f;
+#pragma unroll 4
+      for (int p = 0; p < n_planes; ++p) {
+        const F32Vec<VEC> y = load_vec<VEC>(planes + p * plane + at);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[j].v[e] += y.v[e];
+      }
+#pragma unroll 4
+      for (int k = 0; k < n_slots; ++k) {
+        const F32Vec<VEC> y = load_vec<VEC>(slots + (size_t(row) * n_slots + k) * H + size_t(i) * VEC);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[j].v[e] += y.v[e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += x[j].v[e] * x[j].v[e];
+    }
+  }
+  float inv = 1.f / sqrtf(total_of(ss, 0) / float(H) + eps);
+  ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < kRowRegs; ++j) {
+    const int i = v0 + threadIdx.x + j * kRowThreads;
+    if (i < v1) {
+      const size_t at = base + size_t(i) * VEC;
+      const F32Vec<VEC> r = load_vec<VEC>(residual + at), w = load_vec<VEC>(weight + size_t(i) * VEC);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        x[j].v[e] = r.v[e] + x[j].v[e] * inv * w.v[e];
+        ss += x[j].v[e] * x[j].v[e];
+      }
+      store_vec<VEC>(residual + at, x[j]);
+      if (next == nullptr) store_vec<VEC>(out + at, x[j]);
+    }
+  }
+  if (next == nullptr) return;
+  inv = 1.f / sqrtf(total_of(ss, 1) / float(H) + eps);
+#pragma unroll
+  for (int j = 0; j < kRowRegs; ++j) {
+    const int i = v0 + threadIdx.x + j * kRowThreads;
+    if (i < v1) {
+      F32Vec<VEC> w = load_vec<VEC>(next + size_t(i) * VEC);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) w.v[e] *= x[j].v[e] * inv;
+      store_vec<VEC>(out + base + size_t(i) * VEC, w);
+    }
+  }
+}
+
+template <typename T, typename S>
+int launch_post_norm(void* residual, const void* planes, int n_planes, const void* slots, int n_slots,
+                     const void* weight, const void* next, void* out, int M, int H, float eps, cudaStream_t st) {
+  return launch_rows(post_norm_kernel<T, S, 4>, post_norm_kernel<T, S, 1>, aligned16({residual, weight, out, next}), M, H,
+                     st, reinterpret_cast<float*>(residual), reinterpret_cast<const float*>(planes), n_planes,
+                     reinterpret_cast<const S*>(slots), n_slots, reinterpret_cast<const T*>(weight),
+                     reinterpret_cast<const T*>(next), reinterpret_cast<T*>(out), M, H, eps);
+}
+
+// Embedding of a token, scaled, plus the row of a hashed bigram table (null: none), plus a sinusoidal position vector;
+// residual = RMSNorm of the sum, `out` the same in the activations' type.
+//   row of the table: (token before * mul_prev + token * mul_cur) mod buckets; `buckets` itself for a sequence's first token
+//   position vector: entries 2i, 2i + 1 are the sine and cosine of position * turns[i] turns
+// The token before the first one of a pass comes from last_token[state_rows[s]]; the sequence's last one goes to
+// last_token[state_rows[ld + s]].
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_design_kernel(const ZseEmbed a, const T* __restrict__ table, const T* __restrict__ bigram, const T* __restrict__ norm,
+                    const float2* __restrict__ turns, T* __restrict__ out, Status* st) {
+  extern __shared__ float sx[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, H = a.H;
+  const int* ids = reinterpret_cast<const int*>(a.ids);
+  const int* row_seq = reinterpret_cast<const int*>(a.row_seq);
+  const int* cu_q = reinterpret_cast<const int*>(a.cu_q);
+  const int* state_rows = reinterpret_cast<const int*>(a.state_rows);
+  int* last = reinterpret_cast<int*>(a.last_token);
+  int id = ids[t];
+  if (id < 0 || id >= a.vocab) {
+    if (threadIdx.x == 0) report(st, kBadArgument, 62, unsigned(id));
+    id = 0;
+  }
+  const T* src = table + size_t(id) * H;
+  const T* add = nullptr;
+  if (bigram != nullptr) {
+    const int s = row_seq != nullptr ? row_seq[t] : t;
+    long long prev = -1;
+    if (cu_q != nullptr && cu_q[s] != t) {
+      prev = ids[t - 1];
+    } else {
+      const int r = state_rows[s];
+      if (r >= 0) prev = last[r];
+    }
+    long long row = a.buckets;
+    if (prev >= 0) {
+      row = (prev * a.mul_prev + (long long)(id) * a.mul_cur) % a.buckets;
+      if (row < 0) row += a.buckets;
+    }
+    add = bigram + size_t(row) * H;
+    if (threadIdx.x == 0 && (cu_q == nullptr || cu_q[s + 1] == t + 1)) {
+      const int w = state_rows[a.state_ld + s];
+      if (w >= 0) last[w] = id;
+    }
+  }
+  const float p = float(reinterpret_cast<const int*>(a.positions)[t]);
+  float ss = 0.f;
+  for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
+    const float2 f = turns[i];                       // turns per token, as two floats
+    const float hi = p * f.x;
+    const float r = (hi - rintf(hi)) + fmaf(p, f.y, fmaf(p, f.x, -hi));
+    float sc[2];
+    sincospif(2.f * r, &sc[0], &sc[1]);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int c = 2 * i + e;
+      if (c >= H) break;
+      float x = to_f32(src[c]) * a.scale + sc[e];
+      if (add != nullptr) x += to_f32(add[c]);
+      sx[c] = x;
+      ss += x * x;
+    }
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float total = warp_sum((threadIdx.x & 31) < 8 ? red[threadIdx.x & 31] : 0.f);
+  const float inv = 1.f / sqrtf(total / float(H) + a.eps);
+  float* res = reinterpret_cast<float*>(a.residual) + size_t(t) * H;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float y = sx[i] * inv * to_f32(norm[i]);
+    res[i] = y;
+    out[size_t(t) * H + i] = from_f32<T>(y);
+  }
 }
 
 __global__ void logits_finish_kernel(float* __restrict__ x, int ld, int V, float scale, float cap) {
@@ -241,6 +381,35 @@ extern "C" int zse_add_norm(int dtype, int slot_dtype, void* residual, const voi
   if (slot_dtype == kF32)
     return launch_add_norm<bf16, float>(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps, ST(stream));
   return launch_add_norm<bf16, bf16>(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps, ST(stream));
+}
+
+extern "C" int zse_post_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes,
+                             const void* slots, int n_slots, const void* weight, const void* next, void* out, int M, int H,
+                             float eps, void* stream) {
+  if (M <= 0) return 0;
+  auto run = dtype == kF32        ? launch_post_norm<float, float>
+             : slot_dtype == kF32 ? launch_post_norm<bf16, float>
+                                  : launch_post_norm<bf16, bf16>;
+  return run(residual, planes, n_planes, slots, n_slots, weight, next, out, M, H, eps, ST(stream));
+}
+
+extern "C" int zse_embed_design(int dtype, const ZseEmbed* a, int M, void* status, void* stream) {
+  if (M <= 0) return 0;
+  if (a->bigram != nullptr && a->buckets <= 0) return ZSE_ERR_SHAPE;
+  const size_t smem = size_t(a->H) * sizeof(float);
+  if (smem > 48 * 1024) return ZSE_ERR_LIMIT;
+  cudaError_t e;
+  if (dtype == kBF16)
+    e = launch_pdl(embed_design_kernel<bf16>, dim3(M), dim3(256), smem, ST(stream), *a, reinterpret_cast<const bf16*>(a->table),
+                   reinterpret_cast<const bf16*>(a->bigram), reinterpret_cast<const bf16*>(a->norm),
+                   reinterpret_cast<const float2*>(a->turns), reinterpret_cast<bf16*>(a->out),
+                   reinterpret_cast<Status*>(status));
+  else
+    e = launch_pdl(embed_design_kernel<float>, dim3(M), dim3(256), smem, ST(stream), *a,
+                   reinterpret_cast<const float*>(a->table), reinterpret_cast<const float*>(a->bigram),
+                   reinterpret_cast<const float*>(a->norm), reinterpret_cast<const float2*>(a->turns),
+                   reinterpret_cast<float*>(a->out), reinterpret_cast<Status*>(status));
+  return e == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }
 
 extern "C" int zse_logits_finish(void* logits, int ld, int M, int V, float scale, float cap, void* stream) {

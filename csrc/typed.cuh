@@ -21,6 +21,13 @@ __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat1
 __device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float gelu_exact(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
+__device__ __forceinline__ float relu2(float z) { return z > 0.f ? z * z : 0.f; }
+// g sigmoid(1.702 g) (u + 1), g clamped from above, u from both sides
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  return g / (1.f + expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+}
+
 // 2^x on the special-function unit: softmax weights need no more than its fp32 accuracy, and no range handling around it
 __device__ __forceinline__ float ex2(float x) {
   float y;
@@ -35,6 +42,50 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
 // the part of (a, b) that pack_bf16(a, b) lost
 __device__ __forceinline__ uint32_t pack_bf16_rest(float a, float b) {
   return pack_bf16(a - __bfloat162float(__float2bfloat16_rn(a)), b - __bfloat162float(__float2bfloat16_rn(b)));
+}
+
+// VEC consecutive values as fp32 (VEC 4: one access of 16 or 8 bytes)
+template <int VEC>
+struct F32Vec {
+  float v[VEC];
+};
+template <int VEC>
+__device__ __forceinline__ F32Vec<VEC> load_vec(const float* p) {
+  F32Vec<VEC> r;
+  if constexpr (VEC == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w;
+  } else {
+    r.v[0] = p[0];
+  }
+  return r;
+}
+template <int VEC>
+__device__ __forceinline__ F32Vec<VEC> load_vec(const bf16* p) {
+  F32Vec<VEC> r;
+  if constexpr (VEC == 4) {
+    const uint2 x = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
+    r.v[0] = a.x; r.v[1] = a.y; r.v[2] = b.x; r.v[3] = b.y;
+  } else {
+    r.v[0] = to_f32(p[0]);
+  }
+  return r;
+}
+template <int VEC>
+__device__ __forceinline__ void store_vec(float* p, const F32Vec<VEC>& r) {
+  if constexpr (VEC == 4)
+    *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+  else
+    p[0] = r.v[0];
+}
+template <int VEC>
+__device__ __forceinline__ void store_vec(bf16* p, const F32Vec<VEC>& r) {
+  if constexpr (VEC == 4)
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(r.v[0], r.v[1]), pack_bf16(r.v[2], r.v[3]));
+  else
+    p[0] = from_f32<bf16>(r.v[0]);
 }
 
 __device__ __forceinline__ void cpa16(void* smem_dst, const void* gmem_src) {

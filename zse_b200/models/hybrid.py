@@ -174,10 +174,11 @@ class HybridModel(DesignModel):
                 L.router = ops.dense_linear(r.stack(rows, m.router_rows, H))
                 count = lambda w: self._count(w)
                 L.up = count(ops.moe_up([(t(f"mlp.e{e}.gate"), t(f"mlp.e{e}.up")) for e in range(m.experts)],
-                                        self.act_dtype))
+                                        self.act_dtype, m))
                 L.down = r.stack([(e * H, t(f"mlp.e{e}.down")) for e in range(m.experts)], m.experts * H, m.ff)
                 if m.shared_ff:
-                    L.shared_up = count(ops.moe_up([(t("mlp.shared.gate"), t("mlp.shared.up"))], self.act_dtype))
+                    L.shared_up = count(ops.moe_up([(t("mlp.shared.gate"), t("mlp.shared.up"))], self.act_dtype,
+                                                   m))
                     L.shared_down = r.get(p + "mlp.shared.down")
             self.layers.append(L)
             if progress:
@@ -265,8 +266,8 @@ class HybridModel(DesignModel):
                 if seqs:
                     ops.memory_tokens(inp, b.gates, states, L.state_at, b.state_rows, cu_q, L, out, seqs, M, s, eps)
                 if seqs < num_seqs:
-                    ops.memory_chunks(inp, b.gates, states, L.state_at, b.state_rows, b.cu_q, L, out, seqs, num_seqs, M,
-                                      s, eps, b.memory_ws)
+                    ops.memory_chunks(inp, b.gates, states, L.state_at, b.state_rows, b.cu_q, L, out, seqs, num_seqs, rows,
+                                      M, s, eps, b.memory_ws)
             planes = ops.linear_partial(L.o, out, M, partials)
             last = li + 1 == len(self.layers)
             ops.post_norm(b.residual, partials, planes, None, L.norm1, self.norm if last and L.ff is None else None,

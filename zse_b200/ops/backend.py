@@ -7,6 +7,7 @@ Both work in place on caller-owned buffers so that a step allocates nothing and 
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Optional
 
@@ -15,7 +16,7 @@ import torch
 
 from . import reference as ref
 
-EPI_F16, EPI_SWIGLU, EPI_PARTIAL = 0, 1, 2
+EPI_F16, EPI_SWIGLU, EPI_PARTIAL, EPI_RELU2 = 0, 1, 2, 5
 
 
 @dataclass
@@ -213,7 +214,7 @@ class TorchOps:
             slots[:, m.top] = torch.sigmoid(z[:, m.experts:]) * y if m.shared_gate else y
         return slots
 
-    def moe_up(self, pairs, dtype):
+    def moe_up(self, pairs, dtype, m=None):
         """Up products of gated experts from their (gate, up) matrices [ff, H], all experts in one tensor."""
         return self.dense(torch.cat([t for pair in pairs for t in pair]), dtype)
 
@@ -401,6 +402,11 @@ def _dp(t: Optional[torch.Tensor]) -> Optional[int]:
     return None if t is None else t.data_ptr()
 
 
+def moe_tensor_cores(m, H: int, dtype) -> bool:
+    """Whether the experts' products take the grouped tensor-core kernel (rows of whole 16-byte pieces)."""
+    return dtype == torch.bfloat16 and H % 8 == 0 and m.ff % 8 == 0 and m.shared_ff % 8 == 0
+
+
 class MoeWorkspace:
     """Device tables and activations of the routed feed-forward, shared by all layers of a model."""
     F32_ROWS = 1024
@@ -414,15 +420,19 @@ class MoeWorkspace:
         self.counts, self.first_row, self.n_tiles = z(E, i32), z(E, i32), z(1, i32)
         self.slot_expert, self.slot_rank, self.slot_score = z(slots, i32), z(slots, i32), z(slots, f32)
         self.row_score, self.out_rows = z(slots, f32), z(slots, i32)
+        self.shared_score = z(max_tokens, f32)
         self.tiles = z((E + slots // 16 + 1) * 4, i32)
         self.xs = z(slots * H, dtype)
         self.act = z(max_tokens * max(s.top * s.ff for s in specs), dtype)
         self.act_shared = z(max_tokens * max(s.shared_ff for s in specs), dtype)
         self.y = z(max(min(max_tokens, self.F32_ROWS) * 4, max_tokens * dtype.itemsize) * per * H, torch.uint8)
         # router logits in split-K planes: few columns, so the reduction is what fills the GPU
-        self.router = z(8 * max_tokens * E, f32)
-        self.router_views = {s.experts: self.router[: 8 * max_tokens * s.experts].view(8, max_tokens * s.experts)
-                             for s in specs}
+        widths = {s.router_rows for s in specs}
+        self.router = z(8 * max_tokens * max(widths), f32)
+        self.router_views = {w: self.router[: 8 * max_tokens * w].view(8, max_tokens * w) for w in widths}
+        # gate and up products of gated experts that do not take the tensor-core kernel
+        self.glu = z(2 * max_tokens * max([0] + [max(s.top * s.ff, s.shared_ff) for s in specs
+                                                 if s.gated and not moe_tensor_cores(s, H, dtype)]), dtype)
 
 
 class CudaOps(TorchOps):
@@ -706,54 +716,149 @@ class CudaOps(TorchOps):
     def moe_workspace(self, specs, H: int, max_tokens: int, dtype):
         return MoeWorkspace(specs, H, max_tokens, dtype, self.device) if specs else None
 
+    def moe_up(self, pairs, dtype, m=None):
+        """Tensor-core form: tiles of 64 gate rows and their 64 up rows, the experts' rows padded to whole tiles."""
+        ff, H = pairs[0][0].shape
+        if not moe_tensor_cores(m, H, dtype):
+            return super().moe_up(pairs, dtype, m)
+        n = (ff + 63) // 64
+        out = torch.zeros(len(pairs), n, 2, 64, H, dtype=dtype, device=self.device)
+        pad = torch.zeros(n * 64, H, dtype=dtype, device=self.device)
+        for e, pair in enumerate(pairs):
+            for j, w in enumerate(pair):
+                pad[:ff] = w
+                out[e, :, j] = pad.view(n, 64, H)
+        return out.view(-1, H)
+
     def moe(self, L, x, M, ws):
         n, m, H = self.n, L.moe, x.shape[1]
         dt = x.dtype
         per = m.top + (m.shared_ff > 0)
-        planes = self.linear_partial(L.router, x, M, ws.router_views[m.experts])
+        planes = self.linear_partial(L.router, x, M, ws.router_views[m.router_rows])
         slots = M * m.top
         # result rows in fp32 while they are few, in the activations' type for long passes
         y_dt = torch.float32 if M <= ws.F32_ROWS else dt
         y = ws.y[: M * per * H * y_dt.itemsize].view(y_dt).view(M, per, H)
-        if dt == torch.bfloat16 and H % 8 == 0 and m.ff % 8 == 0 and m.shared_ff % 8 == 0:
+        if moe_tensor_cores(m, H, dt):
             tile = n.moe_tile_rows(M, m.experts, m.top)
-            n.moe_route(ws.router, planes, M, m.experts, m.top, tile, x, H, per, ws)
-            self.moe_product_call(L, x, M, ws, 0)()
+            n.moe_route(ws.router, planes, M, m, tile, x, H, per, ws)
+            self.moe_product_call(L, x, M, ws, 3 if m.gated else 0)()
             self.moe_product_call(L, x, M, ws, 2 if y_dt == torch.float32 else 1)()
             return y
         max_tiles = min(slots, m.experts + slots // 64)
-        n.moe_route(ws.router, planes, M, m.experts, m.top, 64, x, H, per, ws)
+        n.moe_route(ws.router, planes, M, m, 64, x, H, per, ws)
         store = n.TILE_F32 if y_dt == torch.float32 else n.TILE_STORE
         group = dict(tiles=ws.tiles, n_tiles=ws.n_tiles, max_tiles=max_tiles)
-        n.gemm_tile(dt, ws.xs, H, L.up, (H, 1), ws.act, m.ff, slots, m.ff, H, n.TILE_GELU, row_scale=ws.row_score,
-                    b_group=m.ff * H, **group)
+        before, after = (None, ws.row_score) if m.weigh == "output" else (ws.row_score, None)
+        shared_after = ws.shared_score if m.shared_gate else None
+        w = 2 if m.gated else 1
+
+        def up(src, weights, act, ff, rows, limit, scale=None, **kw):
+            if m.gated:
+                n.gemm_tile(dt, src, H, weights, (H, 1), ws.glu, 2 * ff, rows, 2 * ff, H, n.TILE_STORE, **kw)
+                n.clamped_glu(ws.glu, act, rows, ff, limit)
+            else:
+                n.gemm_tile(dt, src, H, weights, (H, 1), act, ff, rows, ff, H, n.TILE_GELU, row_scale=scale, **kw)
+
+        up(ws.xs, L.up, ws.act, m.ff, slots, m.limit, before, b_group=w * m.ff * H, **group)
         n.gemm_tile(dt, ws.act, m.ff, L.down, (m.ff, 1), y, H, slots, H, m.ff, store, out_rows=ws.out_rows,
-                    b_group=m.ff * H, **group)
+                    row_scale=after, b_group=m.ff * H, **group)
         if m.shared_ff:
-            n.gemm_tile(dt, x, H, L.shared_up, (H, 1), ws.act_shared, m.shared_ff, M, m.shared_ff, H, n.TILE_GELU)
+            up(x, L.shared_up, ws.act_shared, m.shared_ff, M, m.shared_limit)
             n.gemm_tile(dt, ws.act_shared, m.shared_ff, L.shared_down, (m.shared_ff, 1), y, H, M, H, m.shared_ff, store,
-                        out_row=(per, m.top))
+                        row_scale=shared_after, out_row=(per, m.top))
         return y
 
     def moe_product_call(self, L, x, M, ws, epilogue: int):
-        """The tensor-core launch of one half of the experts (0: up + gelu; 1, 2: down to bfloat16 / fp32 rows), over
-        the tables that ``moe_route`` left in ``ws``."""
+        """The tensor-core launch of one half of the experts (0: up + gelu, 3: gate and up + clamped glu; 1, 2: down to
+        bfloat16 / fp32 rows), over the tables that ``moe_route`` left in ``ws``."""
         n, m, H = self.n, L.moe, x.shape[1]
         tile = n.moe_tile_rows(M, m.experts, m.top)
         max_tiles = min(M * m.top, m.experts + M * m.top // tile)
-        if epilogue == 0:
+        score = ws.row_score.data_ptr()
+        if epilogue in (0, 3):
+            rows_of = lambda ff: (ff + 63) // 64 * 128 if m.gated else ff
             g = n.MoeGemm(L.up.data_ptr(), ws.xs.data_ptr(), ws.act.data_ptr(), _dp(L.shared_up), x.data_ptr(),
-                          ws.act_shared.data_ptr(), ws.row_score.data_ptr(), None, ws.tiles.data_ptr(),
-                          ws.n_tiles.data_ptr(), m.ff, H, m.ff, m.shared_ff, H, m.shared_ff, 1, 0, x.shape[0])
+                          ws.act_shared.data_ptr(), score if m.weigh == "input" else None, None, ws.tiles.data_ptr(),
+                          ws.n_tiles.data_ptr(), None, rows_of(m.ff), H, m.ff, rows_of(m.shared_ff), H, m.shared_ff, 1, 0,
+                          x.shape[0], m.ff, m.shared_ff, m.limit, m.shared_limit)
             rows = ws.xs.numel() // H
         else:
             per = m.top + (m.shared_ff > 0)
             g = n.MoeGemm(L.down.data_ptr(), ws.act.data_ptr(), ws.y.data_ptr(), _dp(L.shared_down),
-                          ws.act_shared.data_ptr(), ws.y.data_ptr(), None, ws.out_rows.data_ptr(), ws.tiles.data_ptr(),
-                          ws.n_tiles.data_ptr(), H, m.ff, H, H if m.shared_ff else 0, m.shared_ff, H, per, m.top,
-                          ws.act_shared.numel() // max(1, m.shared_ff))
+                          ws.act_shared.data_ptr(), ws.y.data_ptr(), score if m.weigh == "output" else None,
+                          ws.out_rows.data_ptr(), ws.tiles.data_ptr(), ws.n_tiles.data_ptr(),
+                          ws.shared_score.data_ptr() if m.shared_gate else None, H, m.ff, H, H if m.shared_ff else 0,
+                          m.shared_ff, H, per, m.top, ws.act_shared.numel() // max(1, m.shared_ff), H, H, 0.0, 0.0)
             rows = ws.act.numel() // m.ff
         return lambda: n.moe_gemm(g, M, m.experts, rows, tile, max_tiles, epilogue, self.status.ptr)
+
+    # ---- designs of attention over heads, matrix memories and post-norms ---------------------------------
+    def embed_design(self, E, ids, positions, row_seq, cu_q, state_rows, last_token, residual, out, M, S, eps):
+        n, H = self.n, E.table.shape[1]
+        if E.turns is None:              # turns per token as two floats: the angle of any position keeps fp32 accuracy
+            j = torch.arange(0, H, 2, dtype=torch.float64)
+            f = E.base ** (-j / H) / (2 * math.pi)
+            hi = f.float()
+            E.turns = torch.stack([hi, (f - hi.double()).float()], 1).contiguous().to(self.device)
+        a = n.Embed(E.table.data_ptr(), _dp(E.bigram), E.norm.data_ptr(), E.turns.data_ptr(), ids.data_ptr(),
+                    positions.data_ptr(), _dp(row_seq), _dp(cu_q), state_rows.data_ptr(), _dp(last_token),
+                    residual.data_ptr(), out.data_ptr(), E.buckets, E.mul_prev, E.mul_cur, H, E.table.shape[0],
+                    state_rows.stride(0), float(E.scale), float(eps))
+        n.embed_design(a, out.dtype, M, self.status.ptr)
+
+    def post_norm(self, residual, partials, n_partials, slots, weight, next_weight, out, M, eps):
+        self.n.post_norm(residual, partials, n_partials, slots, 0 if slots is None else slots.shape[1], weight, next_weight,
+                         out, M, residual.shape[1], float(eps))
+
+    def linear_act(self, w, x, M, out, activation: str):
+        if activation != "relu2":
+            raise NotImplementedError(activation)
+        if w.kind == "bf16" and w.K % 8 == 0:
+            self.n.gemm_bf16(w.data, w.N, x, x.shape[0], out, M, w.N, w.K, out.stride(0), EPI_RELU2, 1, self.status.ptr)
+        else:
+            self.n.gemm_tile(w.data.dtype, x, x.stride(0), w.data, (w.K, 1), out, out.stride(0), M, w.N, w.K,
+                             self.n.TILE_RELU2)
+
+    def heads_expands(self, spec, dtype) -> bool:
+        return dtype == torch.bfloat16 and self.n.heads_mma_ok(spec, 64)
+
+    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M):
+        self.n.heads_prep(inp, planes, n_planes, M, self.n.heads(kv, spec, self._no_tables), slots, L.q_norm, L.k_norm, spec,
+                          eps)
+
+    @staticmethod
+    def _head_gate(inp, spec):
+        return inp.data_ptr() + spec.gate_col * inp.element_size() if spec.gated else None
+
+    def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits):
+        tc = inp.dtype == torch.bfloat16 and self.n.heads_mma_ok(spec, kv.block_size)
+        if not tc or scratch.numel() < M * num_splits * spec.heads * (spec.vdim + 2):
+            num_splits = 1
+        self.n.heads_attn(inp, self.n.heads(kv, spec, block_tables), row_seq, positions, out, self._head_gate(inp, spec),
+                          scratch, M, num_splits, tc)
+
+    def heads_attn_chunks(self, inp, kv, block_tables, cu_q, q_pos0, positions, first, last, max_q, out, spec):
+        self.n.heads_attn_chunks(inp, self.n.heads(kv, spec, block_tables), cu_q, q_pos0, first, last, max_q, out,
+                                 self._head_gate(inp, spec))
+
+    def memory_expands(self, spec, dtype) -> bool:
+        return dtype == torch.bfloat16 and self.n.memory_chunk_ok(spec)
+
+    def memory_workspace(self, specs, max_tokens: int):
+        w = max([0] + [s.heads * s.vdim for s in specs])
+        return torch.zeros(max(1, max_tokens * w), dtype=torch.float32, device=self.device)
+
+    def memory_prep(self, inp, planes, n_planes, gate_planes, n_gate_planes, gates, L, spec, M):
+        self.n.memory_prep(inp, planes, n_planes, gate_planes, n_gate_planes, L.if_bias, gates, spec, M)
+
+    def memory_tokens(self, inp, gates, states, at, state_rows, cu_q, L, out, S, M, spec, eps):
+        self.n.memory_tokens(inp, gates, self.n.memory(states, at, state_rows, L.head_norm, spec, eps), cu_q, S, out)
+
+    def memory_chunks(self, inp, gates, states, at, state_rows, cu_q, L, out, first, last, row0, M, spec, eps, ws):
+        """Sequences ``first .. last - 1`` chunkwise; their rows are [row0, M)."""
+        self.n.memory_chunks(inp, gates, self.n.memory(states, at, state_rows, L.head_norm, spec, eps), cu_q, first, last, ws,
+                             M, row0, out)
 
     def embedding(self, table, ids, out, M, scale=1.0):
         if table.dtype != torch.float16:

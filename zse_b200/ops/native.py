@@ -47,11 +47,37 @@ class Chunks(Structure):
                 ("window", c_int32)]
 
 
+class Router(Structure):
+    _fields_ = [("planes", c_void_p)] + [(n, c_int32) for n in ("n_planes", "experts", "cols", "top", "softmax",
+                                                                "normalise")] + [("scale", c_float)]
+
+
 class MoeGemm(Structure):
     _fields_ = [(n, c_void_p) for n in ("routed_w", "routed_x", "routed_out", "shared_w", "shared_x", "shared_out",
-                                        "row_score", "out_rows", "tiles", "n_tiles")] + \
+                                        "row_score", "out_rows", "tiles", "n_tiles", "shared_score")] + \
                [(n, c_int32) for n in ("routed_n", "routed_k", "routed_ldo", "shared_n", "shared_k", "shared_ldo",
-                                       "shared_mul", "shared_add", "shared_x_rows")]
+                                       "shared_mul", "shared_add", "shared_x_rows", "routed_cols", "shared_cols")] + \
+               [("routed_limit", c_float), ("shared_limit", c_float)]
+
+
+class Embed(Structure):
+    _fields_ = [(n, c_void_p) for n in ("table", "bigram", "norm", "turns", "ids", "positions", "row_seq", "cu_q",
+                                        "state_rows", "last_token", "residual", "out")] + \
+               [(n, c_int64) for n in ("buckets", "mul_prev", "mul_cur")] + \
+               [("H", c_int32), ("vocab", c_int32), ("state_ld", c_int32), ("scale", c_float), ("eps", c_float)]
+
+
+class Heads(Structure):
+    _fields_ = [("k", c_void_p), ("v", c_void_p), ("block_stride", c_int64)] + \
+               [(n, c_int32) for n in ("block_size", "dim_pad", "vdim_pad", "max_blocks")] + [("tables", c_void_p)] + \
+               [(n, c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "chunk", "window")] + [("scale", c_float)]
+
+
+class Memory(Structure):
+    _fields_ = [(n, c_int32) for n in ("heads", "dim", "vdim", "k_col", "v_col", "gate_col", "if_col")] + \
+               [("states", c_void_p), ("row_floats", c_int64), ("sum_at", c_int32), ("max_at", c_int32),
+                ("state_rows", c_void_p), ("state_ld", c_int32), ("gate_cap", c_float), ("eps", c_float),
+                ("head_norm", c_void_p)]
 
 
 _lib: Optional[ctypes.CDLL] = None
@@ -180,7 +206,25 @@ _SIGS = {
     "zse_latent_chunk": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, POINTER(RowCache), POINTER(Chunks),
                                  c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]),
     "zse_moe_tile_rows": (c_int, [c_int, c_int, c_int]),
-    "zse_moe_route": (c_int, [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int] + [c_void_p] * 11),
+    "zse_moe_route": (c_int, [c_int, POINTER(Router), c_int, c_int, c_void_p, c_int, c_int] + [c_void_p] * 12),
+    "zse_post_norm": (c_int, [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                              c_int, c_float, c_void_p]),
+    "zse_embed_design": (c_int, [c_int, POINTER(Embed), c_int, c_void_p, c_void_p]),
+    "zse_clamped_glu": (c_int, [c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p]),
+    "zse_heads_mma_ok": (c_int, [c_int] * 3),
+    "zse_heads_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_int, POINTER(Heads), c_void_p, c_void_p, c_void_p,
+                               c_int, c_int, c_int, c_int, c_int, c_float, c_void_p]),
+    "zse_heads_attn": (c_int, [c_int, c_void_p, c_int, POINTER(Heads), c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                               c_void_p, c_int, c_int, c_int, c_void_p]),
+    "zse_heads_attn_chunks": (c_int, [c_void_p, c_int, POINTER(Heads), c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
+                                      c_int, c_void_p, c_void_p]),
+    "zse_memory_chunk_ok": (c_int, [c_int] * 2),
+    "zse_memory_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                                POINTER(Memory), c_int, c_void_p]),
+    "zse_memory_tokens": (c_int, [c_int, c_void_p, c_int, c_void_p, POINTER(Memory), c_void_p, c_int, c_void_p, c_int,
+                                  c_void_p]),
+    "zse_memory_chunks": (c_int, [c_void_p, c_int, c_void_p, POINTER(Memory), c_void_p, c_int, c_int, c_void_p, c_int, c_int,
+                                  c_void_p, c_int, c_void_p]),
     "zse_moe_gemm": (c_int, [POINTER(MoeGemm), c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
     "zse_read_probe": (c_int, [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p]),
     "zse_tp_gather_rows": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]),
@@ -511,7 +555,7 @@ def gemm_bf16(w, w_rows, x, x_rows_cap, out, M, N, K, ldo, epilogue, k_split, st
                              _stream()), "gemm_bf16")
 
 
-TILE_STORE, TILE_F32, TILE_GELU, TILE_GATE = 0, 1, 2, 3
+TILE_STORE, TILE_F32, TILE_GELU, TILE_GATE, TILE_RELU2 = 0, 1, 2, 3, 4
 
 
 def gemm_tile(dtype, a, lda, b, ldb, out, ldo, M, N, K, epilogue=TILE_STORE, batch=1, a_batch=0, b_batch=0, o_batch=0,
@@ -532,6 +576,76 @@ def add_norm(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps)
     sd = 0 if slots is None else _DTYPE[slots.dtype]
     _ck(load().zse_add_norm(_DTYPE[out.dtype], sd, _p(residual), _p(planes), n_planes, _p(slots), n_slots, _p(weight),
                             _p(out), M, H, eps, _stream()), "add_norm")
+
+
+def post_norm(residual, planes, n_planes, slots, n_slots, weight, next_weight, out, M, H, eps):
+    sd = 0 if slots is None else _DTYPE[slots.dtype]
+    _ck(load().zse_post_norm(_DTYPE[out.dtype], sd, _p(residual), _p(planes), n_planes, _p(slots), n_slots, _p(weight),
+                             _p(next_weight), _p(out), M, H, eps, _stream()), "post_norm")
+
+
+def embed_design(a: Embed, dtype, M, status):
+    _ck(load().zse_embed_design(_DTYPE[dtype], byref(a), M, status, _stream()), "embed_design")
+
+
+def clamped_glu(x, out, rows, ff, limit):
+    _ck(load().zse_clamped_glu(_DTYPE[x.dtype], _p(x), _p(out), rows, ff, float(limit), _stream()), "clamped_glu")
+
+
+def heads(view, spec, block_tables) -> Heads:
+    """``view``: ``models.hybrid.PagedHeads``."""
+    return Heads(view.k.data_ptr(), view.v.data_ptr(), view.block_stride, view.block_size, view.k.shape[3], view.v.shape[3],
+                 block_tables.stride(0), block_tables.data_ptr(), spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.chunk,
+                 spec.window, float(spec.scale))
+
+
+def heads_mma_ok(spec, block_size: int) -> bool:
+    return bool(load().zse_heads_mma_ok(spec.dim, spec.vdim, block_size))
+
+
+def heads_prep(inp, planes, n_planes, M, h, slots, q_norm, k_norm, spec, eps):
+    _ck(load().zse_heads_prep(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, M, byref(h), _p(slots),
+                              _p(q_norm), _p(k_norm), spec.k_col, spec.v_col, spec.gate_col,
+                              spec.heads if spec.gated else 0, int(spec.own_kv), float(eps), _stream()), "heads_prep")
+
+
+def heads_attn(inp, h, row_seq, positions, out, gate, scratch, M, num_splits, tensor_cores):
+    _ck(load().zse_heads_attn(_DTYPE[inp.dtype], _p(inp), inp.stride(0), byref(h), _p(row_seq), _p(positions), _p(out),
+                              out.stride(0), gate, _p(scratch), M, num_splits, int(tensor_cores), _stream()), "heads_attn",
+        2 if num_splits > 1 else 1)
+
+
+def heads_attn_chunks(inp, h, cu_q, q_pos0, first, last, max_q, out, gate):
+    _ck(load().zse_heads_attn_chunks(_p(inp), inp.stride(0), byref(h), _p(cu_q), _p(q_pos0), first, last, max_q, _p(out),
+                                     out.stride(0), gate, _stream()), "heads_attn_chunks")
+
+
+def memory(states, at, state_rows, head_norm, spec, eps) -> Memory:
+    """``states``: the state pool's rows; ``at``: where the layer's part of a row begins."""
+    return Memory(spec.heads, spec.dim, spec.vdim, spec.k_col, spec.v_col, spec.gate_col, spec.if_col,
+                  states.data_ptr() + 4 * at, states.stride(0), spec.sum_at, spec.max_at, _p(state_rows),
+                  state_rows.stride(0), float(spec.gate_cap), float(eps), _p(head_norm))
+
+
+def memory_chunk_ok(spec) -> bool:
+    return bool(load().zse_memory_chunk_ok(spec.dim, spec.vdim))
+
+
+def memory_prep(inp, planes, n_planes, gate_planes, n_gate_planes, if_bias, gates, spec, M):
+    m = Memory(spec.heads, spec.dim, spec.vdim, spec.k_col, spec.v_col, spec.gate_col, spec.if_col, None, 0, 0, 0, None, 0,
+               float(spec.gate_cap), 0.0, None)
+    _ck(load().zse_memory_prep(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, _p(gate_planes),
+                               n_gate_planes, _p(if_bias), _p(gates), byref(m), M, _stream()), "memory_prep")
+
+
+def memory_tokens(inp, gates, m, cu_q, S, out):
+    _ck(load().zse_memory_tokens(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(gates), byref(m), _p(cu_q), S, _p(out),
+                                 out.stride(0), _stream()), "memory_tokens")
+
+
+def memory_chunks(inp, gates, m, cu_q, first, last, o, M, row0, out):
+    _ck(load().zse_memory_chunks(_p(inp), inp.stride(0), _p(gates), byref(m), _p(cu_q), first, last, _p(o), M, row0, _p(out),
+                                 out.stride(0), _stream()), "memory_chunks", 2)
 
 
 def logits_finish(logits, M, scale, cap):
@@ -593,11 +707,14 @@ def moe_tile_rows(M, E, top) -> int:
     return load().zse_moe_tile_rows(M, E, top)
 
 
-def moe_route(planes, n_planes, M, E, top, tile_rows, x, H, out_per_token, ws):
-    _ck(load().zse_moe_route(_DTYPE[x.dtype], _p(planes), n_planes, M, E, top, tile_rows, _p(x), H, out_per_token,
+def moe_route(planes, n_planes, M, moe, tile_rows, x, H, out_per_token, ws):
+    """``moe``: the layer's ``MoESpec``."""
+    r = Router(_p(planes), n_planes, moe.experts, moe.router_rows, moe.top, int(moe.score == "softmax"), int(moe.normalise),
+               float(moe.scale))
+    _ck(load().zse_moe_route(_DTYPE[x.dtype], byref(r), M, tile_rows, _p(x), H, out_per_token,
                              _p(ws.counts), _p(ws.slot_expert), _p(ws.slot_rank), _p(ws.slot_score), _p(ws.first_row),
-                             _p(ws.tiles), _p(ws.n_tiles), _p(ws.xs), _p(ws.row_score), _p(ws.out_rows), _stream()),
-        "moe_route", 3)
+                             _p(ws.tiles), _p(ws.n_tiles), _p(ws.xs), _p(ws.row_score), _p(ws.out_rows),
+                             _p(ws.shared_score), _stream()), "moe_route", 3)
 
 
 def moe_gemm(g, M, E, max_rows, tile_rows, max_tiles, epilogue, status):

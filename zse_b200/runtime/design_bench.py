@@ -253,7 +253,7 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
         add(phase, "router logits", "output projection",
             lambda: ops.linear_partial(L.router, x, M, ws.router_views[m.experts]), *mm(m.experts, H))
         add(phase, "routing + sorted rows", "rotation + cache write",
-            lambda: ops.n.moe_route(ws.router, 1, M, m.experts, m.top, tile, x, H, per, ws), 4.0 * M * m.top * H)
+            lambda: ops.n.moe_route(ws.router, 1, M, m, tile, x, H, per, ws), 4.0 * M * m.top * H)
         add(phase, "feed-forward (all routed kernels)", "gate/up + down projections", lambda: ops.moe(L, x, M, ws),
             2.0 * (touched * 2 * m.ff * H + 2 * m.shared_ff * H + 2 * M * (act + m.top * H)), 4.0 * M * act * H)
         for name, epi in (("experts up + gelu", 0), ("experts down", 2 if y32 else 1)):
