@@ -38,6 +38,7 @@ NUM_REQUESTS = 64
 PROMPT_RANGE = (128, 2048)
 OUTPUT_TOKENS = 256
 # name -> model shape, requests, prompt rule, output tokens, speculative depth, (adapters, rank)
+DESIGNS = ("ruralorn", "nimelorn")      # models of listed layers, beside a dense neighbour
 WORKLOADS = {
     "batch64": dict(model="qwen2.5-14b", requests=64, prompt=("uniform",) + PROMPT_RANGE, out=256, spec_k=0, lora=None,
                     seq_len=f"prompts uniform {PROMPT_RANGE}, 256 output tokens"),
@@ -69,14 +70,15 @@ def parse_args():
     ap.add_argument("--spec-k", type=int, default=None,
                     help="override the workload's number of draft tokens per step (0: plain decoding of the same requests)")
     ap.add_argument("--kernels-file", default=None, metavar="FILE",
-                    help="with --workload ruralorn: also time every kernel alone and write the roofline table to FILE")
-    ap.add_argument("--workload", default="batch64", choices=sorted(WORKLOADS) + ["ruralorn"],
+                    help="with --workload ruralorn or nimelorn: also time every kernel alone and write the roofline table to FILE")
+    ap.add_argument("--workload", default="batch64", choices=sorted(WORKLOADS) + list(DESIGNS),
                     help="batch64: 64 requests, prompts uniform in [128, 2048] (the headline); single: one request "
                          "with a 512-token prompt on the 7B shape (the case the reference publishes); spec32b: n-gram "
                          "speculative decoding on the 32B shape; lora72b: 256 requests over 32 adapters on the 72B shape; ruralorn: prefill and decode of the "
-                         "latent-attention / routed design at two sizes beside a dense model of equal size (one GPU)")
+                         "latent-attention / routed design at two sizes beside a dense model of equal size (one GPU); nimelorn: the "
+                         "same for the design of chunked attention, matrix memories and gated experts")
     a = ap.parse_args()
-    if a.workload not in ("batch64", "ruralorn"):
+    if a.workload not in ("batch64",) + DESIGNS:
         w = WORKLOADS[a.workload]
         a.model = w["model"] if a.model == MODEL_SHAPE else a.model
         a.requests = w["requests"] if a.requests == NUM_REQUESTS else a.requests
@@ -398,16 +400,19 @@ def run_ours(args):
 
 
 def run_designs(args):
-    """bfloat16 Ruralorn shapes beside their dense neighbours (zse_b200/runtime/design_bench.py)."""
-    from zse_b200.runtime import design_bench
+    """bfloat16 shapes of a design beside their dense neighbours (zse_b200/runtime/design_bench.py, hybrid_bench.py)."""
+    if args.workload == "nimelorn":
+        from zse_b200.runtime import hybrid_bench as design_bench
+    else:
+        from zse_b200.runtime import design_bench
     if int(os.environ.get("WORLD_SIZE", "1")) > 1:
-        raise SystemExit("--workload ruralorn runs on one GPU")
+        raise SystemExit(f"--workload {args.workload} runs on one GPU")
     sampler = ClockSampler(0)
     res = design_bench.run(args.steps, args.warmup, kernels_file=args.kernels_file)
     clocks = sampler.stop()
-    first = res[design_bench.SHAPES[0]]["ruralorn"]
+    first = res[design_bench.SHAPES[0]][args.workload]
     print(json.dumps({
-        "metric": "bf16 Ruralorn decode tok/s", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1,
+        "metric": f"bf16 {args.workload.capitalize()} decode tok/s", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1,
         "steps": args.steps, "warmup": args.warmup, "ms_per_step": first["decode_ms_per_step"], "higher_is_better": True,
         "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
         "config": {"model": f"{design_bench.SHAPES[0]} (random weights)", "global_batch": 64,
@@ -439,11 +444,11 @@ def run_reference(args):
 
 if __name__ == "__main__":
     a = parse_args()
-    if a.impl == "reference" and a.workload == "ruralorn":
+    if a.impl == "reference" and a.workload in DESIGNS:
         print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this design"}))
     elif a.impl == "reference":
         run_reference(a)
-    elif a.workload == "ruralorn":
+    elif a.workload in DESIGNS:
         run_designs(a)
     else:
         try:

@@ -150,3 +150,90 @@ def greedy(cfg, weights, prompt, n):
     for _ in range(n):
         seq.append(int(forward(cfg, weights, seq)[-1].argmax()))
     return seq[len(prompt):]
+
+
+# ---- small random models --------------------------------------------------------------------------------------------
+def attention_layer(heads, kv_heads, dim, vdim, chunk, mlp, scale=None, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": chunk},
+         "scale": scale or dim ** -0.5}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def mlstm_layer(heads, dim, vdim, mlp, gate_cap=12.0):
+    return {"type": "mlstm", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": gate_cap}, "mlp": mlp}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts, top, ff, limit, scale=1.0, shared=None, shared_limit=None):
+    m = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top, "scale": scale}}
+    if shared:
+        m["shared"] = {"ff": shared, "limit": shared_limit or limit}
+    return m
+
+
+def config(width, vocab, layers, embed_scale=6.0, eps=1e-5, buckets=61, mul_prev=7, mul_cur=5):
+    return {"architecture": "Nimelorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers,
+            "embedding": {"scale": embed_scale, "bigram": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}}}
+
+
+def shapes(cfg):
+    D = cfg["width"]
+    out = {"embed": (cfg["vocab"], D), "bigram": (cfg["embedding"]["bigram"]["buckets"] + 1, D), "embed.norm": (D,),
+           "final.norm": (D,), "head": (cfg["vocab"], D)}
+    for i, L in enumerate(cfg["layers"]):
+        a, m, p = L["mixer"], L["mlp"], f"l{i}."
+        H, d, v = a["heads"], a["dim"], a["vdim"]
+        out.update({p + "norm1": (D,), p + "mix.q": (H * d, D), p + "mix.o": (D, H * v)})
+        if L["type"] == "mlstm":
+            out.update({p + "mix.k": (H * d, D), p + "mix.v": (H * v, D), p + "mix.g": (H * v, D), p + "mix.norm": (H * v,),
+                        p + "mix.i": (H, D), p + "mix.f": (H, D), p + "mix.i.b": (H,), p + "mix.f.b": (H,)})
+        else:
+            out.update({p + "mix.q.norm": (d,), p + "mix.g": (H, D)})
+            if "kv_from" not in a:
+                out.update({p + "mix.k": (a["kv_heads"] * d, D), p + "mix.v": (a["kv_heads"] * v, D), p + "mix.k.norm": (d,)})
+        if m is None:
+            continue
+        out[p + "norm2"] = (D,)
+        if m["kind"] == "dense":
+            out.update({p + "mlp.up": (m["ff"], D), p + "mlp.down": (D, m["ff"])})
+            continue
+        out[p + "mlp.router"] = (m["router"]["experts"], D)
+        parts = [(f"e{e}", m["expert"]["ff"]) for e in range(m["router"]["experts"])]
+        if m.get("shared"):
+            out[p + "mlp.shared.sg"] = (1, D)
+            parts.append(("shared", m["shared"]["ff"]))
+        for name, ff in parts:
+            out.update({f"{p}mlp.{name}.gate": (ff, D), f"{p}mlp.{name}.up": (ff, D), f"{p}mlp.{name}.down": (D, ff)})
+    return out
+
+
+def random_weights(cfg, seed=0, sharp=2.5):
+    """bfloat16 weights.  Query norms are scaled up by ``sharp`` so that single keys stand out of the softmax; forget gates
+    stay open for some fifty tokens and input gates differ from token to token, so that a lost or misplaced state moves the
+    logits; up products reach the clamps."""
+    g = torch.Generator().manual_seed(seed)
+    W = {}
+    for name, shape in shapes(cfg).items():
+        if name.endswith("i.b"):
+            w = 0.5 * torch.randn(shape, generator=g)
+        elif name.endswith("f.b"):
+            w = 4.0 + torch.randn(shape, generator=g)
+        elif len(shape) == 1:
+            w = 1 + 0.2 * torch.randn(shape, generator=g)
+            if name.endswith("q.norm"):
+                w *= sharp
+        else:
+            w = torch.randn(shape, generator=g) * shape[1] ** -0.5
+            if name in ("embed", "bigram"):
+                w *= shape[1] ** 0.5 * (0.15 if name == "embed" else 0.8)
+            if name.endswith("mix.i"):
+                w *= 2.0
+            if name.endswith("gate") or name.endswith("up"):
+                w *= 1.5
+        W[name] = w.to(torch.bfloat16)
+    return W

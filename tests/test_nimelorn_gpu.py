@@ -1,0 +1,539 @@
+"""Nimelorn on the GPU: every kernel against float64 statements of the same operation, whole models against the plain oracle
+in float32 and bfloat16, generation through the engine."""
+import math
+import os
+import sys
+import types
+
+import numpy as np
+import pytest
+import torch
+
+sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
+from helpers import nimelorn_oracle as oracle                                     # noqa: E402
+from helpers.nimelorn_cases import CASES, Model                                   # noqa: E402
+from helpers.ruralorn_cases import (LENGTHS, MAX_TOKENS, SCHEDULES, assert_close, assert_near, errors, replay,  # noqa: E402
+                                    schedule)
+
+from zse_b200.format.config import HeadsSpec, MatrixMemorySpec, MoESpec           # noqa: E402
+from zse_b200.models.hybrid import EmbedDesign, PagedHeads                        # noqa: E402
+
+pytestmark = pytest.mark.gpu
+BF, F32, F64 = torch.bfloat16, torch.float32, torch.float64
+
+
+@pytest.fixture(scope="module")
+def ops():
+    from zse_b200.ops.backend import CudaOps
+    o = CudaOps("cuda")
+    yield o
+    o.check()
+
+
+def rel(a, b):
+    return ((a.to(F64) - b).abs().max() / b.abs().max()).item()
+
+
+def tol(dt):
+    return 1.5e-2 if dt == BF else 2e-5
+
+
+def i32(v):
+    return torch.tensor(v, dtype=torch.int32, device="cuda")
+
+
+# ---- attention --------------------------------------------------------------------------------------------------------
+SPECS = {
+    "grouped": HeadsSpec(12, 3, 64, 96, 0.25, chunk=150),
+    "one-kv-head": HeadsSpec(20, 1, 128, 128, 0.2, chunk=256),               # two tiles of query heads
+    "wide": HeadsSpec(4, 2, 256, 200, 0.12, chunk=1000),
+    "narrow": HeadsSpec(3, 3, 8, 24, 0.6, chunk=64),
+    "half-steps": HeadsSpec(6, 2, 72, 40, 0.3, chunk=77),                    # widths of half a step of 16
+    "self-only": HeadsSpec(4, 4, 32, 32, 0.4, chunk=1),
+    "window": HeadsSpec(8, 2, 64, 64, 0.25, window=130),
+    "everything": HeadsSpec(8, 2, 64, 128, 0.25),
+    "no-gate": HeadsSpec(4, 2, 48, 80, 0.3, chunk=96, gated=False),
+    "general": HeadsSpec(6, 2, 18, 7, 0.4, chunk=50),
+}
+
+
+class Attention:
+    """Cached keys and values of a layer inside a pool of wider rows; the plain results come from float64 copies."""
+
+    def __init__(self, spec, dt, bs=64, blocks=40, seqs=6, width=12, seed=0, rows=400):
+        g = torch.Generator(device="cuda").manual_seed(seed)
+        rnd = lambda *s: torch.randn(*s, device="cuda", generator=g)
+        self.spec, self.dt, self.bs = spec, dt, bs
+        self.pool = torch.zeros(blocks, 1, 1, bs, spec.row + 16, device="cuda", dtype=dt)
+        self.kv = PagedHeads(self.pool, spec)
+        self.kv.k[..., : spec.dim] = rnd(blocks, spec.kv_heads, bs, spec.dim).to(dt)
+        self.kv.v[..., : spec.vdim] = rnd(blocks, spec.kv_heads, bs, spec.vdim).to(dt)
+        self.tables = torch.stack([torch.randperm(blocks, device="cuda", generator=g)[:width] for _ in range(seqs)]).int()
+        self.inp = rnd(rows, spec.in_width).to(dt)
+
+    def plain(self, t, seq, pos):
+        """Row t of ``inp`` as the query at ``pos`` of sequence ``seq``, float64."""
+        s = self.spec
+        j = torch.arange(s.first_seen(pos), pos + 1, device="cuda")
+        blk = self.tables[seq][j // self.bs].long()
+        j, blk = j[blk >= 0], blk[blk >= 0]
+        rep = s.heads // s.kv_heads
+        k = self.kv.k[blk, :, j % self.bs, : s.dim].to(F64).repeat_interleave(rep, 1)
+        v = self.kv.v[blk, :, j % self.bs, : s.vdim].to(F64).repeat_interleave(rep, 1)
+        q = self.inp[t, : s.heads * s.dim].to(F64).view(s.heads, s.dim)
+        y = torch.einsum("hn,nhv->hv", torch.softmax(torch.einsum("hd,nhd->hn", q, k) * s.scale, -1), v)
+        if s.gated:
+            y = y * torch.sigmoid(self.inp[t, s.gate_col: s.gate_col + s.heads].to(F64))[:, None]
+        return y.reshape(-1)
+
+    def rows(self, ops, seqs, positions, splits=1):
+        s, M = self.spec, len(seqs)
+        out = torch.zeros(M, s.heads * s.vdim, dtype=self.dt, device="cuda")
+        ops.heads_attn(self.inp, self.kv, self.tables, i32(seqs), i32(positions), out, M, s,
+                       torch.zeros(M * splits * s.heads * (s.vdim + 2), device="cuda"), splits)
+        return out
+
+    def chunks(self, ops, spans, first=0):
+        cu = np.cumsum([0] + [n for _, n in spans]).tolist()
+        pos = i32([a + i for a, n in spans for i in range(n)])
+        out = torch.zeros(cu[-1], self.spec.heads * self.spec.vdim, dtype=self.dt, device="cuda")
+        ops.heads_attn_chunks(self.inp, self.kv, self.tables, i32(cu), i32([a for a, _ in spans]), pos, first, len(spans),
+                              max(n for _, n in spans[first:]), out, self.spec)
+        return out, cu
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("name", list(SPECS))
+@pytest.mark.parametrize("bs", [64, 16, 128])
+def test_rows_against_cached_keys(ops, name, dt, bs):
+    A = Attention(SPECS[name], dt, blocks=40 * 64 // bs, bs=bs, width=12 * 64 // bs)
+    A.tables[3, 1] = -1                                 # a hole, inside some chunks
+    seqs, pos = [0, 1, 2, 3, 4, 5, 5, 0, 1], [0, 1, 63, 150, 64, 700, 511, 199, 149]
+    if bs == 16:
+        A.tables[3, 9] = -1
+    want = torch.stack([A.plain(t, s, p) for t, (s, p) in enumerate(zip(seqs, pos))])
+    for splits in (1, 2, 8):
+        assert rel(A.rows(ops, seqs, pos, splits), want) < tol(dt), splits
+    ops.check()
+
+
+@pytest.mark.parametrize("name", [n for n in SPECS if n != "general"])
+@pytest.mark.parametrize("bs", [64, 32])
+def test_tiles_of_queries_against_cached_keys(ops, name, bs):
+    A = Attention(SPECS[name], BF, bs=bs, blocks=40 * 64 // bs, width=12 * 64 // bs)
+    assert ops.heads_expands(A.spec, BF)
+    A.tables[2, 2] = -1
+    spans = [(3, 5), (0, 70), (200, 17), (400, 130), (63, 64)]     # the first sequence is not part of the call
+    out, cu = A.chunks(ops, spans, first=1)
+    assert (out[: cu[1]] == 0).all()
+    for s in range(1, len(spans)):
+        for i in sorted({0, 1, spans[s][1] // 2, 63 % spans[s][1], 64 % spans[s][1], spans[s][1] - 1}):
+            assert rel(out[cu[s] + i], A.plain(cu[s] + i, s, spans[s][0] + i)) < tol(BF), (s, i)
+
+
+@pytest.mark.parametrize("dt,what", [(BF, "rows"), (F32, "rows"), (BF, "tiles")])
+@pytest.mark.parametrize("name", ["grouped", "one-kv-head", "half-steps", "window"])
+def test_one_loud_key_inside_and_outside(ops, name, dt, what):
+    """A key that takes all the weight sits on the first place that is seen, one before it, far away, on block borders, on
+    the token itself and on the next one."""
+    spec = SPECS[name]
+    size = spec.chunk or spec.window
+    g = spec.kv_heads - 1
+    for pos in (size - 1, size, 2 * size - 1, 2 * size, 447, 640):
+        if pos >= 760:
+            continue
+        lo = spec.first_seen(pos)
+        for key in sorted({pos, pos + 1, lo, lo - 1, (lo + pos) // 2, pos // 64 * 64, pos // 64 * 64 - 1, 0}):
+            if not 0 <= key < 760:
+                continue
+            A = Attention(spec, dt, seed=pos)
+            t = 20                                       # a query in the middle of the portion
+            q = A.inp[t, (spec.heads - 1) * spec.dim: spec.heads * spec.dim].float()
+            A.kv.k[A.tables[0, key // 64].long(), g, key % 64, : spec.dim] = (q * (60 / spec.scale / q.pow(2).sum())).to(dt)
+            want = A.plain(t, 0, pos)
+            if what == "rows":
+                A.inp[0] = A.inp[t]
+                got = A.rows(ops, [0], [pos], 2)[0]
+            elif pos < t:
+                continue
+            else:
+                got = A.chunks(ops, [(pos - t, 40)])[0][t]
+            assert rel(got, want) < tol(dt), (pos, key)
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("name", list(SPECS))
+@pytest.mark.parametrize("planes", [0, 1, 4])
+@pytest.mark.parametrize("own", [True, False])
+def test_heads_prep(ops, name, dt, planes, own):
+    import dataclasses
+    spec = SPECS[name] if own else dataclasses.replace(SPECS[name], kv_from=0)
+    A = Attention(spec, dt)
+    s, M, eps = spec, 70, 1e-5
+    H, G, d, vd = s.heads, s.kv_heads, s.dim, s.vdim
+    g = torch.Generator(device="cuda").manual_seed(3)
+    pl = torch.randn(max(1, planes), M, s.in_width, device="cuda", generator=g)
+    full = (pl.sum(0) if planes else A.inp[:M]).to(F64)
+    L = types.SimpleNamespace(q_norm=torch.randn(d, device="cuda", generator=g).to(dt),
+                              k_norm=torch.randn(d, device="cuda", generator=g).to(dt) if own else None)
+    slots = torch.randperm(40 * 64, device="cuda", generator=g)[:M]
+    slots[5] = -1
+    before = A.pool.clone()
+    norm = lambda x, w: x / torch.sqrt((x ** 2).mean(-1, keepdim=True) + eps) * w.to(F64)
+    ops.heads_prep(A.inp, pl, planes, A.kv, slots, L, s, eps, M)
+    q = norm(full[:, : H * d].view(M, H, d), L.q_norm).reshape(M, -1)
+    assert rel(A.inp[:M, : H * d], q) < tol(dt)
+    if s.gated:
+        assert rel(A.inp[:M, s.gate_col: s.gate_col + H], full[:, s.gate_col: s.gate_col + H]) < tol(dt)
+    if not own:
+        assert torch.equal(A.pool, before)
+        return
+    ok = slots >= 0
+    blk, at = slots[ok] // 64, slots[ok] % 64
+    k = norm(full[ok, s.k_col: s.k_col + G * d].view(-1, G, d), L.k_norm)
+    assert rel(A.kv.k[blk, :, at, :d], k) < tol(dt)
+    assert rel(A.kv.v[blk, :, at, :vd], full[ok, s.v_col: s.v_col + G * vd].view(-1, G, vd)) < tol(dt)
+    assert (A.kv.k[..., d:] == 0).all() and (A.kv.v[..., vd:] == 0).all()
+    touched = torch.zeros(40 * 64, dtype=torch.bool, device="cuda")
+    touched[slots[ok]] = True
+    old = PagedHeads(before, s)
+    same = (A.kv.k == old.k).all(-1).all(1).view(-1) & (A.kv.v == old.v).all(-1).all(1).view(-1)
+    assert same[~touched].all()
+
+
+# ---- matrix memory -----------------------------------------------------------------------------------------------------
+MEMORIES = {
+    "small": MatrixMemorySpec(3, 16, 24, 10.0),
+    "usual": MatrixMemorySpec(4, 64, 128, 15.0),
+    "big": MatrixMemorySpec(2, 256, 320, 15.0),
+    "half-steps": MatrixMemorySpec(5, 136, 72, 12.0),
+    "many-columns": MatrixMemorySpec(1, 40, 520, 6.0),
+    "general": MatrixMemorySpec(2, 10, 7, 8.0),
+}
+
+
+class Memory:
+    def __init__(self, spec, dt, rows=420, slots=7, seed=0, slow=True):
+        g = torch.Generator(device="cuda").manual_seed(seed)
+        rnd = lambda *s: torch.randn(*s, device="cuda", generator=g)
+        self.spec, self.dt, self.at = spec, dt, 12
+        self.inp = rnd(rows, spec.in_width).to(dt)
+        i = 3.0 * rnd(rows, spec.heads)
+        f = torch.nn.functional.logsigmoid((3.0 if slow else 0.0) + 2.0 * rnd(rows, spec.heads))
+        self.gates = torch.cat([i, f], 1).contiguous()
+        self.states = torch.zeros(2 * slots, self.at + spec.state_floats + 4, device="cuda")
+        self.L = types.SimpleNamespace(head_norm=rnd(spec.heads * spec.vdim).to(dt))
+        self.eps = 1e-5
+        # starting states that a recursion could have left
+        self.states[:, self.at: self.at + spec.state_floats] = rnd(2 * slots, spec.state_floats)
+
+    def part(self, row):
+        s = self.spec
+        H, d, v = s.heads, s.dim, s.vdim
+        x = self.states[row, self.at: self.at + s.state_floats].to(F64)
+        return (x[: H * d * v].view(H, d, v).clone(), x[s.sum_at: s.sum_at + H * d].view(H, d).clone(),
+                x[s.max_at: s.max_at + H].clone())
+
+    def plain(self, a, e, read):
+        """Rows [a, e) from the state in row ``read`` (-1: none): (outputs, S, n, m) in float64."""
+        from zse_b200.ops import reference as ref
+        s = self.spec
+        H, d, v = s.heads, s.dim, s.vdim
+        x = self.inp[a:e].to(F64)
+        if read >= 0:
+            S, n, m = self.part(read)
+        else:
+            z = lambda *sh: torch.zeros(*sh, dtype=F64, device="cuda")
+            S, n, m = z(H, d, v), z(H, d), z(H)
+        g = self.gates[a:e].to(F64)
+        y = ref.memory_tokens(x[:, : H * d].reshape(-1, H, d) * d ** -0.5, x[:, s.k_col: s.k_col + H * d].reshape(-1, H, d),
+                              x[:, s.v_col: s.v_col + H * v].reshape(-1, H, v), g[:, :H], g[:, H:], S, n, m)
+        y = y / torch.sqrt((y ** 2).mean(-1, keepdim=True) + self.eps)
+        y = y.reshape(e - a, -1) * self.L.head_norm.to(F64) * torch.sigmoid(x[:, s.gate_col: s.gate_col + H * v])
+        return y, S, n, m
+
+    def run(self, ops, cu, rows, chunkwise, first=0):
+        s, M = self.spec, cu[-1] if cu is not None else rows.shape[1]
+        out = torch.zeros(M, s.heads * s.vdim, dtype=self.dt, device="cuda")
+        cu_d = i32(cu) if cu is not None else None
+        S = rows.shape[1]
+        if chunkwise:
+            ws = torch.zeros(M * s.heads * s.vdim, device="cuda")
+            ops.memory_chunks(self.inp, self.gates, self.states, self.at, rows, cu_d, self.L, out, first, S, cu[first], M, s,
+                              self.eps, ws)
+        else:
+            ops.memory_tokens(self.inp, self.gates, self.states, self.at, rows, cu_d, self.L, out, S, M, s, self.eps)
+        return out
+
+
+def check_memory(ops, name, dt, cu, rows, chunkwise, limit, first=0, slow=True):
+    m = Memory(MEMORIES[name], dt, slow=slow)
+    want = [m.plain(cu[i], cu[i + 1], rows[0][i]) for i in range(len(rows[0]))]
+    before = m.states.clone()
+    out = m.run(ops, cu, i32(rows), chunkwise, first)
+    written = torch.zeros(m.states.shape[0], dtype=torch.bool)
+    for i in range(first, len(rows[0])):
+        y, S, n, mx = want[i]
+        a, e = cu[i], cu[i + 1]
+        err = (out[a:e].to(F64) - y).pow(2).mean(1).sqrt() / y.pow(2).mean(1).sqrt()
+        assert err.max() < limit, (i, err.max().item(), int(err.argmax()))
+        w = rows[1][i]
+        if w >= 0:
+            written[w] = True
+            S2, n2, m2 = m.part(w)
+            assert rel(S2, S) < limit and rel(n2, n) < limit and rel(m2, mx) < 1e-5
+    assert torch.equal(m.states[~written], before[~written])
+    assert torch.equal(m.states[:, : m.at], before[:, : m.at])            # other layers' parts
+    assert torch.equal(m.states[:, m.at + m.spec.state_floats:], before[:, m.at + m.spec.state_floats:])
+    ops.check()
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("name", list(MEMORIES))
+def test_memory_token_by_token(ops, name, dt):
+    limit = 1e-2 if dt == BF else 1e-4
+    check_memory(ops, name, dt, [0, 1, 2, 3, 4], [[4, -1, 7, -1], [5, 2, 6, -1]], False, limit)      # a row each
+    check_memory(ops, name, dt, [0, 2, 18, 19, 150], [[4, -1, 7, 0], [5, 2, 6, 1]], False, limit)
+
+
+@pytest.mark.parametrize("slow", [True, False])
+@pytest.mark.parametrize("name", [n for n in MEMORIES if n != "general"])
+def test_memory_in_chunks(ops, name, slow):
+    assert ops.memory_expands(MEMORIES[name], BF)
+    check_memory(ops, name, BF, [0, 64, 147, 160, 400], [[4, -1, 7, 0], [5, 2, 6, 1]], True, 1e-2, slow=slow)
+    check_memory(ops, name, BF, [0, 3, 130, 195], [[4, 2, -1], [5, 3, -1]], True, 1e-2, first=1, slow=slow)
+
+
+def test_memory_decodes_without_row_offsets(ops):
+    m = Memory(MEMORIES["usual"], BF)
+    rows = [[0, 2, -1, -1], [1, 3, 4, -1]]
+    want = torch.cat([m.plain(i, i + 1, rows[0][i])[0] for i in range(4)])
+    assert rel(m.run(ops, None, i32(rows), False), want) < 1e-2
+
+
+@pytest.mark.parametrize("chunkwise", [True, False])
+def test_memory_keeps_a_token_from_long_ago(ops, chunkwise):
+    """Forget gates that stay open: one loud token at the start is what every later token reads; closed for one token, and
+    it is gone."""
+    spec = MatrixMemorySpec(2, 32, 64, 15.0)
+    for closed_at in (None, 200):
+        m = Memory(spec, BF)
+        m.gates[:, :2], m.gates[:, 2:] = -8.0, -1e-4
+        m.gates[3, :2] = 9.0
+        if closed_at is not None:
+            m.gates[closed_at, 2:] = -60.0
+        want = m.plain(0, 400, -1)[0]
+        out = m.run(ops, [0, 400], i32([[-1], [1]]), chunkwise)
+        err = (out.to(F64) - want).pow(2).mean(1).sqrt() / want.pow(2).mean(1).sqrt()
+        assert err.max() < 1.5e-2, (int(err.argmax()), err.max().item())
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("name", list(MEMORIES))
+@pytest.mark.parametrize("planes", [0, 1, 5])
+def test_memory_prep(ops, name, dt, planes):
+    s, M = MEMORIES[name], 37
+    g = torch.Generator(device="cuda").manual_seed(1)
+    pl = 4 * torch.randn(max(1, planes), M, s.in_width, device="cuda", generator=g)
+    gp = 6 * torch.randn(3, M, 2 * s.heads, device="cuda", generator=g)
+    bias = torch.randn(2 * s.heads, device="cuda", generator=g)
+    inp = torch.zeros(M, s.in_width, device="cuda", dtype=dt)
+    gates = torch.zeros(M, 2 * s.heads, device="cuda")
+    ops.memory_prep(inp, pl, planes, gp, 0 if planes else 3, gates, types.SimpleNamespace(if_bias=bias), s, M)
+    z = (pl.to(F64).sum(0)[:, s.if_col: s.if_col + 2 * s.heads] if planes else gp.to(F64).sum(0)) + bias.to(F64)
+    z = s.gate_cap * torch.tanh(z / s.gate_cap)
+    want = torch.cat([z[:, : s.heads], torch.nn.functional.logsigmoid(z[:, s.heads:])], 1)
+    assert ((gates.to(F64) - want).abs() <= 2e-6 + 3e-6 * want.abs()).all()
+    if planes:
+        assert rel(inp[:, : s.if_col], pl.to(F64).sum(0)[:, : s.if_col]) < tol(dt)
+
+
+# ---- rows --------------------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("H", [64, 51, 4096, 10000])
+@pytest.mark.parametrize("planes,slots", [(1, 0), (4, 0), (0, 3), (2, 1)])
+@pytest.mark.parametrize("last", [True, False])
+def test_post_norm(ops, dt, H, planes, slots, last):
+    M, eps = 9, 1e-5
+    g = torch.Generator(device="cuda").manual_seed(H)
+    rnd = lambda *s: torch.randn(*s, device="cuda", generator=g)
+    res, pl, w, nw = rnd(M, H), rnd(max(1, planes), M, H), rnd(H).to(dt), rnd(H).to(dt)
+    for sdt in ({dt, F32} if slots else {F32}):
+        sl = rnd(M, slots, H).to(sdt) if slots else None
+        y = pl.to(F64).sum(0) if planes else torch.zeros(M, H, dtype=F64, device="cuda")
+        if slots:
+            y = y + sl.to(F64).sum(1)
+        norm = lambda x, v: x / torch.sqrt((x ** 2).mean(-1, keepdim=True) + eps) * v.to(F64)
+        r = res.clone()
+        want = r.to(F64) + norm(y, w)
+        out = torch.zeros(M, H, device="cuda", dtype=dt)
+        ops.post_norm(r, pl, planes, sl, w, nw if last else None, out, M, eps)
+        assert rel(r, want) < 1e-5
+        assert rel(out, norm(want, nw) if last else want) < tol(dt)
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("H,positions", [(64, 5), (51, 100000), (2048, 4000)])
+def test_embedding_with_bigrams_and_sinusoid(ops, dt, H, positions):
+    V, B, eps = 900, 499, 1e-5
+    g = torch.Generator(device="cuda").manual_seed(H)
+    rnd = lambda *s: torch.randn(*s, device="cuda", generator=g)
+    E = EmbedDesign(rnd(V, H).to(dt), 1.7, 10000.0, rnd(H).to(dt), rnd(B + 1, H).to(dt), B, 1 << 30, 977)
+    cu, start = [0, 1, 4, 9], [0, positions, positions // 2]
+    ids, M = torch.randint(V, (9,), device="cuda", generator=g, dtype=torch.int32), 9
+    state = i32([[-1, 3, 0], [5, 2, -1]])
+    last = i32([11, 12, 13, 899, 15, 16])
+    pos = i32([start[s] + i for s in range(3) for i in range(cu[s + 1] - cu[s])])
+    seq = i32([s for s in range(3) for _ in range(cu[s + 1] - cu[s])])
+    prev = [-1, 899] + ids[1:3].tolist() + [11] + ids[4:8].tolist()
+    rows = [B if p < 0 else (p * (1 << 30) + t * 977) % B for p, t in zip(prev, ids.tolist())]
+    x = E.table[ids.long()].to(F64) * 1.7 + E.bigram[torch.tensor(rows, device="cuda")].to(F64)
+    j = torch.arange(H, device="cuda")
+    a = pos.to(F64)[:, None] * 10000.0 ** (-(j - j % 2).to(F64) / H)
+    x = x + torch.where(j % 2 == 0, torch.sin(a), torch.cos(a))
+    want = x / torch.sqrt((x ** 2).mean(-1, keepdim=True) + eps) * E.norm.to(F64)
+    res, out = torch.zeros(M, H, device="cuda"), torch.zeros(M, H, device="cuda", dtype=dt)
+    ops.embed_design(E, ids, pos, seq, i32(cu), state, last, res, out, M, 3, eps)
+    assert rel(res, want) < 2e-6 and rel(out, want) < tol(dt)
+    assert last.tolist() == [11, 12, int(ids[3]), 899, 15, int(ids[0])]
+    # decode: every row is a sequence of its own, padding has no state
+    state, last = i32([[0, 4, -1, -1], [1, 5, 3, -1]]), i32([7, 0, 0, 0, 8, 0])
+    ops.embed_design(E, ids, pos, None, None, state, last, res, out, 4, 4, eps)
+    assert last.tolist() == [7, int(ids[0]), 0, int(ids[2]), 8, int(ids[1])]
+    rows = [(7 * (1 << 30) + int(ids[0]) * 977) % B, (8 * (1 << 30) + int(ids[1]) * 977) % B, B, B]
+    x = E.table[ids[:4].long()].to(F64) * 1.7 + E.bigram[torch.tensor(rows, device="cuda")].to(F64)
+    x = x + torch.where(j % 2 == 0, torch.sin(a), torch.cos(a))[:4]
+    want = x / torch.sqrt((x ** 2).mean(-1, keepdim=True) + eps) * E.norm.to(F64)
+    assert rel(res[:4], want) < 2e-6
+    ops.check()
+
+
+# ---- feed-forwards -----------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("M,N,K", [(1, 40, 24), (70, 264, 96), (300, 520, 200), (13, 19, 51)])
+def test_linear_with_squared_relu(ops, dt, M, N, K):
+    g = torch.Generator(device="cuda").manual_seed(N)
+    x = torch.randn(M, K, device="cuda", generator=g).to(dt)
+    w = (torch.randn(N, K, device="cuda", generator=g) * K ** -0.5).to(dt)
+    out = torch.zeros(M, N, device="cuda", dtype=dt)
+    ops.linear_act(ops.dense_linear(w), x, M, out, "relu2")
+    assert rel(out, torch.relu(x.to(F64) @ w.to(F64).T) ** 2) < tol(dt)
+    ops.check()
+
+
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("H,E,top,ff,shared", [(64, 8, 2, 40, 72), (96, 20, 5, 64, 0), (128, 33, 33, 24, 136), (51, 6, 3, 17, 9),
+                                               (256, 64, 6, 200, 320), (64, 1, 1, 64, 64)])
+@pytest.mark.parametrize("M", [1, 7, 90, 700, 1100])
+def test_gated_experts(ops, dt, H, E, top, ff, shared, M):
+    m = MoESpec(E, top, ff, shared, "softmax", "clamped_glu", "output", True, 1.6, 0.9, 0.5, shared > 0)
+    g = torch.Generator(device="cuda").manual_seed(E * 100 + M)
+    rnd = lambda *s, k=1.0: (torch.randn(*s, device="cuda", generator=g) * k).to(dt)
+    x = rnd(M, H)
+    ups = [(rnd(ff, H, k=H ** -0.5), rnd(ff, H, k=H ** -0.5)) for _ in range(E)]
+    down, router = rnd(E * H, ff, k=ff ** -0.5), rnd(m.router_rows, H, k=3 * H ** -0.5)
+    L = types.SimpleNamespace(moe=m, router=ops.dense_linear(router), up=ops.moe_up(ups, dt, m), down=down, shared_up=None,
+                              shared_down=None)
+    if shared:
+        sup = (rnd(shared, H, k=H ** -0.5), rnd(shared, H, k=H ** -0.5))
+        L.shared_up, L.shared_down = ops.moe_up([sup], dt, m), rnd(H, shared, k=shared ** -0.5)
+    z = x.to(F64) @ router.to(F64).T
+    p = torch.softmax(z[:, :E], -1)
+    w, ids = p.sort(-1, descending=True)
+    # rows whose last chosen and first rejected experts are as good as equal may go either way
+    sure = torch.ones(M, dtype=torch.bool, device="cuda") if top == E else (w[:, top - 1] - w[:, top]) > 1e-4 * w[:, top - 1]
+    w = w[:, :top] / (w[:, :top].sum(-1, keepdim=True) + 1e-20) * 1.6
+
+    def expert(pair, dn, limit, t):
+        a, u = (t @ pair[0].to(F64).T).clamp(max=limit), (t @ pair[1].to(F64).T).clamp(-limit, limit)
+        return (a * torch.sigmoid(1.702 * a) * (u + 1)) @ dn.to(F64).T
+
+    want = torch.zeros(M, H, dtype=F64, device="cuda")
+    for e in range(E):
+        t, k = torch.where(ids[:, :top] == e)
+        want.index_add_(0, t, w[t, k, None] * expert(ups[e], down[e * H: (e + 1) * H], 0.9, x[t].to(F64)))
+    if shared:
+        want += torch.sigmoid(z[:, E:]) * expert(sup, L.shared_down, 0.5, x.to(F64))
+    ws = ops.moe_workspace([m], H, max(M, 8), dt)
+    for _ in range(2):
+        got = ops.moe(L, x, M, ws).to(F64).sum(1)
+    assert rel(got[sure], want[sure]) < (2e-2 if dt == BF else 2e-5)
+    ops.check()
+
+
+# ---- whole models ------------------------------------------------------------------------------------------------------
+@pytest.fixture(scope="module", params=list(CASES))
+def model(request, tmp_path_factory):
+    return Model(request.param, tmp_path_factory.mktemp("nimelorn") / request.param)
+
+
+@pytest.fixture(scope="module")
+def small(tmp_path_factory):
+    return Model("layers-differ", tmp_path_factory.mktemp("nimelorn-small"))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_schedules_match_the_oracle(model, dtype):
+    from zse_b200.trace import TraceRunner
+    r = TraceRunner(model.path, dtype, MAX_TOKENS)
+    try:
+        for name in SCHEDULES + ["token-by-token"]:
+            got = replay(r, model, schedule(name))
+            if dtype == "float32":
+                assert_close(model, got, 5e-4)
+            else:
+                assert_near(model, got)
+        assert r.engine.kv_cache.states.num_free == 4
+    finally:
+        r.close()
+
+
+def test_bfloat16_logits_do_not_depend_on_the_schedule(model):
+    from zse_b200.trace import TraceRunner
+    r = TraceRunner(model.path, "bfloat16", MAX_TOKENS)
+    whole = replay(r, model, schedule("whole"))
+    for name in ("portions-2", "mixed", "prompt-then-decode"):
+        for rid, rows in replay(r, model, schedule(name)).items():
+            d = np.sqrt(((rows - whole[rid.split("#")[0]][: len(rows)]) ** 2).mean(1)) / model.want["a"].std()
+            assert np.median(d) < 0.03 and (d < 0.3).mean() > 0.9, (name, rid)
+    r.close()
+
+
+def gpu_engine(path, **kw):
+    from zse_b200.config import EngineConfig
+    from zse_b200.engine import ZStreamerEngine
+    kw = dict(dict(dtype="float32", max_batch_seqs=4, max_batch_tokens=128, kv_blocks=24, max_seq_len=512), **kw)
+    return ZStreamerEngine(path, config=EngineConfig(**kw))
+
+
+@pytest.mark.parametrize("kw", [dict(), dict(pipeline_decode=False), dict(use_cuda_graphs=False, prefill_chunk_size=32),
+                                dict(max_batch_seqs=2, prefill_chunk_size=24, decode_per_prefill=0),
+                                dict(speculative_k=3)])
+def test_greedy_generation_matches_the_oracle(small, kw):
+    eng = gpu_engine(small.path, **kw)
+    prompts = [small.tokens["a"][:75], small.tokens["b"][:5], small.tokens["c"], small.tokens["d"][:40]]
+    rids = [eng.add_request_tokens(p, max_tokens=8, temperature=0.0, stop_tokens=[]) for p in prompts]
+    eng.run_until_done()
+    for p, rid in zip(prompts, rids):
+        assert eng.get_result(rid).output_tokens == oracle.greedy(small.cfg, small.weights, p, 8)
+    eng.destroy()
+
+
+def test_long_decoding(small):
+    """Sixty steps through graphs, over several chunk and block borders, against the oracle's logits."""
+    from zse_b200.trace import TraceRunner
+    r = TraceRunner(small.path, "float32", MAX_TOKENS)
+    assert_close(small, replay(r, small, [[("a", 30)]] + [[("a", 1)] for _ in range(LENGTHS["a"] - 30)]), 5e-4)
+    assert r.engine.runner.timings["graph_replays"] >= 100
+    r.close()
+
+
+def test_synthetic_model_generates_in_bfloat16(tmp_path):
+    from zse_b200.format import synth
+    path = str(tmp_path / "s.zse")
+    synth.write_random_model(path, synth.shape_config("tiny-nimelorn"), seed=3)
+    eng = gpu_engine(path, dtype=None)
+    rids = [eng.add_request_tokens(list(range(k, k + 60)), max_tokens=6, temperature=0.0, stop_tokens=[]) for k in range(6)]
+    eng.run_until_done()
+    assert all(len(eng.get_result(r).output_tokens) == 6 for r in rids)
+    eng.destroy()

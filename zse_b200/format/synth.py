@@ -36,6 +36,28 @@ def ruralorn_design(layers: int, width: int, vocab: int, heads: int, dim: int, r
             "layers": [layer() for _ in range(layers)]}
 
 
+def nimelorn_design(width: int, vocab: int, heads: int, kv_heads: int, dim: int, vdim: int, chunk: int, memory: tuple,
+                    dense_ff: int, experts: int, top: int, ff: int, shared_ff: int, limit: float = 7.0, repeats: int = 1,
+                    buckets: int = 65521, eps: float = 1e-6, gate_cap: float = 15.0) -> dict:
+    """A Nimelorn ``config.json`` of ``repeats`` times four layers: a matrix memory (``memory``: heads, dim, vdim) with a
+    dense feed-forward, attention with experts, attention with a dense one, and attention over the keys and values of the
+    layer before it with experts."""
+    dense = {"kind": "dense", "ff": dense_ff}
+    moe = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top, "scale": 1.0},
+           "shared": {"ff": shared_ff, "limit": limit}}
+
+    def attention(mlp, **kw):
+        return {"type": "attention", "mlp": mlp, "mixer": dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim,
+                                                               scale=dim ** -0.5, mask={"size": chunk}, **kw)}
+    layers = []
+    for r in range(repeats):
+        layers += [{"type": "mlstm", "mlp": dense, "mixer": {"heads": memory[0], "dim": memory[1], "vdim": memory[2],
+                                                             "gate_cap": gate_cap}},
+                   attention(moe), attention(dense), attention(moe, kv_from=4 * r + 2)]
+    return {"architecture": "Nimelorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers,
+            "embedding": {"scale": width ** 0.5, "bigram": {"buckets": buckets, "mul_prev": 31337, "mul_cur": 1009}}}
+
+
 # entries with a "design" hold a config.json of that architecture instead of ``ModelConfig`` fields
 SHAPES = {
     "tiny-ruralorn": dict(arch="ruralorn", design=ruralorn_design(3, 192, 1024, 6, 24, 8, 40, 56, 40, 10, 3, 72, 104)),
@@ -44,6 +66,12 @@ SHAPES = {
                                                                 2816)),
     "ruralorn-4k": dict(arch="ruralorn", design=ruralorn_design(4, 4096, 102400, 32, 128, 64, 128, 512, 4096, 64, 4, 2048,
                                                                 4096)),
+    "tiny-nimelorn": dict(arch="nimelorn", design=nimelorn_design(160, 1024, 6, 2, 32, 24, 48, (3, 40, 56), 224, 10, 3, 72,
+                                                                  104, 1.2, buckets=251)),
+    "nimelorn-2k": dict(arch="nimelorn", design=nimelorn_design(2048, 102400, 16, 4, 128, 128, 4096, (4, 256, 512), 8192, 64,
+                                                                6, 1408, 2816, repeats=2)),
+    "nimelorn-4k": dict(arch="nimelorn", design=nimelorn_design(4096, 102400, 32, 8, 128, 128, 4096, (8, 256, 512), 14336,
+                                                                64, 4, 2048, 4096)),
     "tiny": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64, intermediate_size=688,
                  vocab_size=1024, rms_norm_eps=1e-6, rope_theta=10000.0, arch="llama", max_seq_len=2048),
     "tiny-aligned": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64,
@@ -188,8 +216,10 @@ def write_random_model(path: str, config: ModelConfig, seed: int = 0, std: float
     if with_tokenizer:
         w.set_tokenizer(byte_tokenizer(c.vocab_size).serialize())
     w.begin_weights()
-    if c.is_latent:
-        for name, shape in latent_tensor_shapes(c):
+    if c.is_design:
+        from .arch import get_adapter
+        shapes = latent_tensor_shapes(c) if c.is_latent else get_adapter(c.arch).tensor_shapes(c)
+        for name, shape in shapes:
             w.add_weight_raw_bf16(name, shape, _random_bf16(rng, shape, fast))
         w.finalize()
         return
