@@ -18,11 +18,18 @@ namespace {
 struct Heads {
   long long block_stride;
   int block_size, dp, vp, max_blocks;            // dp, vp: padded widths
+  int block_shift;                               // log2 of the block size, -1: no power of two
   const int* tables;
   int heads, kv_heads, dim, vdim, chunk, window;
   float scale;
   __device__ __forceinline__ int first_seen(int pos) const {
     return chunk > 0 ? pos / chunk * chunk : window > 0 ? max(0, pos + 1 - window) : 0;
+  }
+  __device__ __forceinline__ int block_of(int token) const {
+    return block_shift >= 0 ? token >> block_shift : token / block_size;
+  }
+  __device__ __forceinline__ int in_block(int token) const {
+    return block_shift >= 0 ? token & (block_size - 1) : token % block_size;
   }
   // first element of a token's key (dp) or value (vp)
   __device__ __forceinline__ size_t at(int block, int head, int token, int width) const {
@@ -36,7 +43,7 @@ struct HeadsPrepArgs {
   float eps;
 };
 
-// A warp per (row, section): query heads, then key heads, value heads and - with planes - the gates.
+// A warp per (row, section): query heads, then key heads, value heads and - with planes - the gates.  grid (rows, sections / 8)
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_planes, int M, T* __restrict__ kc,
@@ -46,9 +53,8 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
-  const long long id = blockIdx.x * 8ll + (threadIdx.x >> 5);
-  const int t = int(id / units), u = int(id % units);
-  if (t >= M) return;
+  const int t = blockIdx.x, u = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (u >= units) return;
   T* in = inp + size_t(t) * a.ld;
   const float* pl = planes + size_t(t) * a.ld;
   const size_t plane = size_t(M) * a.ld;
@@ -78,7 +84,7 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
   if (u >= h.heads) {
     const long long slot = slots[t];
     if (slot < 0) return;
-    const int g = (u - h.heads) % G, block = int(slot / h.block_size), token = int(slot % h.block_size);
+    const int g = u - h.heads - (u >= h.heads + G ? G : 0), block = h.block_of(int(slot)), token = h.in_block(int(slot));
     if (u >= h.heads + G) {                      // values: copied
       dst = vc + h.at(block, g, token, h.vp);
       const int c0 = a.v_col + g * h.vdim;
@@ -144,10 +150,10 @@ heads_simple_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ kc,
   const int* table = h.tables + size_t(seq) * h.max_blocks;
   float m = -INFINITY, l = 0.f;
   for (int j = h.first_seen(pos) + warp; j <= pos; j += 4) {
-    const int block = table[j / h.block_size];
+    const int block = table[h.block_of(j)];
     if (block < 0) continue;
-    const T* k = kc + h.at(block, g, j % h.block_size, h.dp);
-    const T* v = vc + h.at(block, g, j % h.block_size, h.vp);
+    const T* k = kc + h.at(block, g, h.in_block(j), h.dp);
+    const T* v = vc + h.at(block, g, h.in_block(j), h.vp);
     float s = 0.f;
     for (int i = lane; i < h.dim; i += 32) s = fmaf(q[i], to_f32(k[i]), s);
     s = warp_sum(s) * h.scale;
@@ -234,25 +240,33 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
         *reinterpret_cast<uint4*>(st + kRowKeys * kp + (r % kRowKeys) * vp + vch * 16) = make_uint4(0, 0, 0, 0);
     }
   }
+  // a tile's rows are contiguous in the cache: piece j * 32 + lane of it goes to this place of the padded tile
+  int k_to[DKS], v_to[DVT / 2];
+#pragma unroll
+  for (int j = 0; j < DKS; ++j) {
+    const int idx = j * 32 + lane;
+    k_to[j] = idx < kRowKeys * kch ? idx / kch * kp + idx % kch * 16 : -1;
+  }
+#pragma unroll
+  for (int j = 0; j < DVT / 2; ++j) {
+    const int idx = j * 32 + lane;
+    v_to[j] = idx < kRowKeys * vch ? idx / vch * vp + idx % vch * 16 : -1;
+  }
   auto issue = [&](int i) {                      // i-th tile of this warp; always commits a group
     if (i < mine) {
       const int tok = (tb + warp + i * kRowWarps) * kRowKeys;
-      const int block = table[tok / h.block_size];
+      const int block = table[h.block_of(tok)];
       if (block >= 0) {
-        const bf16* ks_ = kc + h.at(block, kvh, tok % h.block_size, h.dp);
-        const bf16* vs_ = vc + h.at(block, kvh, tok % h.block_size, h.vp);
+        const bf16* ks_ = kc + h.at(block, kvh, h.in_block(tok), h.dp);
+        const bf16* vs_ = vc + h.at(block, kvh, h.in_block(tok), h.vp);
         uint8_t* kd = ring + (i % kRowStages) * kRowKeys * (kp + vp);
         uint8_t* vd = kd + kRowKeys * kp;
 #pragma unroll
-        for (int j = 0; j < DKS; ++j) {          // a tile's rows are contiguous in the cache
-          const int idx = j * 32 + lane;
-          if (idx < kRowKeys * kch) cpa16(kd + idx / kch * kp + idx % kch * 16, ks_ + idx * 8);
-        }
+        for (int j = 0; j < DKS; ++j)
+          if (k_to[j] >= 0) cpa16(kd + k_to[j], ks_ + (j * 32 + lane) * 8);
 #pragma unroll
-        for (int j = 0; j < DVT / 2; ++j) {
-          const int idx = j * 32 + lane;
-          if (idx < kRowKeys * vch) cpa16(vd + idx / vch * vp + idx % vch * 16, vs_ + idx * 8);
-        }
+        for (int j = 0; j < DVT / 2; ++j)
+          if (v_to[j] >= 0) cpa16(vd + v_to[j], vs_ + (j * 32 + lane) * 8);
       }
     }
     cpa_commit();
@@ -269,7 +283,7 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
     __syncwarp();
     issue(i + kRowStages - 1);
     const int tok = (tb + warp + i * kRowWarps) * kRowKeys;
-    if (table[tok / h.block_size] < 0) continue;
+    if (table[h.block_of(tok)] < 0) continue;
     const uint32_t kb = smem_u32(ring + (i % kRowStages) * kRowKeys * (kp + vp)), vb = kb + kRowKeys * kp;
     float s[2][4] = {};
 #pragma unroll
@@ -465,14 +479,14 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
       uint8_t *kd = sk + st * kChunkKeys * kp, *vd = sv + st * kChunkKeys * vp;
       if (threadIdx.x < kChunkKeys) {
         const int p = key0 + threadIdx.x;
-        const bool v = p < k_end && table[p / h.block_size] >= 0;
+        const bool v = p < k_end && table[h.block_of(p)] >= 0;
         valid[st * kChunkKeys + threadIdx.x] = v;
         if (st == 0) whole[0] = v; else whole[1] = v;
       }
       // runs of 16 keys are contiguous in a block; a warp takes one run
-      const int tok = key0 + warp * 16, block = tok < k_end ? table[tok / h.block_size] : -1;
-      const size_t base_k = h.at(max(block, 0), kvh, tok % h.block_size, h.dp);
-      const size_t base_v = h.at(max(block, 0), kvh, tok % h.block_size, h.vp);
+      const int tok = key0 + warp * 16, block = tok < k_end ? table[h.block_of(tok)] : -1;
+      const size_t base_k = h.at(max(block, 0), kvh, h.in_block(tok), h.dp);
+      const size_t base_v = h.at(max(block, 0), kvh, h.in_block(tok), h.vp);
       const int rows = block < 0 ? 0 : min(16, k_end - tok);
       for (int idx = lane; idx < 16 * kch; idx += 32) {
         const int r = idx / kch, c = idx % kch;
@@ -616,7 +630,10 @@ int raise_smem(K kern, size_t bytes, size_t* done) {      // `done`: per device,
 }
 
 Heads heads_of(const ZseHeads* h) {
-  return Heads{(long long)(h->block_stride), h->block_size, h->dim_pad, h->vdim_pad, h->max_blocks,
+  int shift = -1;
+  for (int i = 0; i < 30; ++i)
+    if (h->block_size == 1 << i) shift = i;
+  return Heads{(long long)(h->block_stride), h->block_size, h->dim_pad, h->vdim_pad, h->max_blocks, shift,
                reinterpret_cast<const int*>(h->tables), h->heads, h->kv_heads, h->dim, h->vdim, h->chunk, h->window,
                h->scale};
 }
@@ -674,7 +691,7 @@ cudaError_t launch_prep(void* inp, const void* planes, int n_planes, int M, cons
                         const void* q_norm, const void* k_norm, const HeadsPrepArgs& a, cudaStream_t st) {
   const Heads h = heads_of(z);
   const int units = h.heads + 2 * (a.own_kv ? h.kv_heads : 0) + (n_planes > 0 && a.gate_w > 0 ? 1 : 0);
-  return launch_pdl(heads_prep_kernel<T, VEC>, dim3(unsigned((size_t(M) * units + 7) / 8)), dim3(256), 0, st,
+  return launch_pdl(heads_prep_kernel<T, VEC>, dim3(M, (units + 7) / 8), dim3(256), 0, st,
                     reinterpret_cast<T*>(inp), reinterpret_cast<const float*>(planes), n_planes, M,
                     reinterpret_cast<T*>(z->k), reinterpret_cast<T*>(z->v), h, reinterpret_cast<const long long*>(slots),
                     reinterpret_cast<const T*>(q_norm), reinterpret_cast<const T*>(k_norm), a, units);

@@ -42,7 +42,8 @@ __device__ __forceinline__ float log_gate(float z, float cap, bool forget) {
   return forget ? fminf(g, 0.f) - log1pf(expf(-fabsf(g))) : g;
 }
 
-// grid (rows, 1 + pieces): piece 0 takes the gates, the others sum kPrepCols columns each.
+// grid (rows, 1 + pieces): piece 0 takes the gates, the others sum kPrepCols columns each.  Without planes: grid (blocks)
+// over all gates.
 template <typename T>
 __global__ void __launch_bounds__(256)
 memory_prep_kernel(T* __restrict__ inp, int ld, const float* __restrict__ planes, int n_planes,
@@ -51,13 +52,19 @@ memory_prep_kernel(T* __restrict__ inp, int ld, const float* __restrict__ planes
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, g = 2 * m.heads;
+  if (n_planes == 0) {
+    const int id = blockIdx.x * blockDim.x + threadIdx.x;
+    if (id >= M * g) return;
+    const int i = id % g;
+    float z = bias[i];
+    for (int p = 0; p < n_gate_planes; ++p) z += gate_planes[size_t(p) * M * g + id];
+    gates[id] = log_gate(z, m.gate_cap, i >= m.heads);
+    return;
+  }
   if (blockIdx.y == 0) {
     for (int i = threadIdx.x; i < g; i += blockDim.x) {
       float z = bias[i];
-      if (n_planes > 0)
-        for (int p = 0; p < n_planes; ++p) z += planes[(size_t(p) * M + t) * ld + m.if_col + i];
-      else
-        for (int p = 0; p < n_gate_planes; ++p) z += gate_planes[(size_t(p) * M + t) * g + i];
+      for (int p = 0; p < n_planes; ++p) z += planes[(size_t(p) * M + t) * ld + m.if_col + i];
       gates[size_t(t) * g + i] = log_gate(z, m.gate_cap, i >= m.heads);
     }
     return;
@@ -642,7 +649,8 @@ extern "C" int zse_memory_prep(int dtype, void* inp, int ld, const void* planes,
   if (M <= 0) return 0;
   if (ld % 8 || z->if_col % 8) return ZSE_ERR_SHAPE;
   const Memory m = memory_of(z);
-  const dim3 grid(M, 1 + (n_planes > 0 ? (m.if_col + kPrepCols - 1) / kPrepCols : 0));
+  const dim3 grid = n_planes > 0 ? dim3(M, 1 + (m.if_col + kPrepCols - 1) / kPrepCols)
+                                 : dim3((M * 2 * m.heads + 255) / 256);
   cudaError_t e;
   if (dtype == kBF16)
     e = launch_pdl(memory_prep_kernel<bf16>, grid, dim3(256), 0, ST(stream), reinterpret_cast<bf16*>(inp), ld,

@@ -105,11 +105,11 @@ add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, 
   }
 }
 
-// Launch over (cluster, rows) with VEC 4 where sizes and addresses allow it.
-template <typename K, typename... Args>
+// Launch over (cluster, rows) with VEC 4 where sizes and addresses allow it, else VEC `ANY`.
+template <int ANY = 1, typename K, typename... Args>
 int launch_rows(K vec_kern, K any_kern, bool aligned, int M, int H, cudaStream_t st, Args... args) {
   const bool vec = H % 4 == 0 && aligned;
-  const int n = vec ? H / 4 : H;
+  const int n = vec ? H / 4 : (H + ANY - 1) / ANY;
   int cs = 1;
   while (cs < 8 && ((M * cs < 256 && n / (cs * 2) >= 64) || (n + cs - 1) / cs > kRowThreads * kRowRegs)) cs *= 2;
   if ((n + cs - 1) / cs > kRowThreads * kRowRegs) return ZSE_ERR_SHAPE;
@@ -237,23 +237,27 @@ int launch_post_norm(void* residual, const void* planes, int n_planes, const voi
 //   position vector: entries 2i, 2i + 1 are the sine and cosine of position * turns[i] turns
 // The token before the first one of a pass comes from last_token[state_rows[s]]; the sequence's last one goes to
 // last_token[state_rows[ld + s]].
-template <typename T>
-__global__ void __launch_bounds__(256)
+template <typename T, int VEC>                       // VEC 4, or 2 with a last column of its own when H is odd
+__global__ void __launch_bounds__(kRowThreads)
 embed_design_kernel(const ZseEmbed a, const T* __restrict__ table, const T* __restrict__ bigram, const T* __restrict__ norm,
-                    const float2* __restrict__ turns, T* __restrict__ out, Status* st) {
-  extern __shared__ float sx[];
+                    const float* __restrict__ turns, T* __restrict__ out, Status* st) {
   __shared__ float red[32];
+  __shared__ float cluster_ss;
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, H = a.H;
+  const int t = blockIdx.y, cs = gridDim.x, H = a.H;
+  const int nv = ((H + VEC - 1) / VEC + cs - 1) / cs;
+  const int v0 = blockIdx.x * nv, v1 = min((H + VEC - 1) / VEC, v0 + nv);
   const int* ids = reinterpret_cast<const int*>(a.ids);
   const int* row_seq = reinterpret_cast<const int*>(a.row_seq);
   const int* cu_q = reinterpret_cast<const int*>(a.cu_q);
   const int* state_rows = reinterpret_cast<const int*>(a.state_rows);
   int* last = reinterpret_cast<int*>(a.last_token);
+  const bool first_cta = blockIdx.x == 0;
   int id = ids[t];
+  const float p = float(reinterpret_cast<const int*>(a.positions)[t]);
   if (id < 0 || id >= a.vocab) {
-    if (threadIdx.x == 0) report(st, kBadArgument, 62, unsigned(id));
+    if (threadIdx.x == 0 && first_cta) report(st, kBadArgument, 62, unsigned(id));
     id = 0;
   }
   const T* src = table + size_t(id) * H;
@@ -273,40 +277,79 @@ embed_design_kernel(const ZseEmbed a, const T* __restrict__ table, const T* __re
       if (row < 0) row += a.buckets;
     }
     add = bigram + size_t(row) * H;
-    if (threadIdx.x == 0 && (cu_q == nullptr || cu_q[s + 1] == t + 1)) {
+    if (threadIdx.x == 0 && first_cta && (cu_q == nullptr || cu_q[s + 1] == t + 1)) {
       const int w = state_rows[a.state_ld + s];
       if (w >= 0) last[w] = id;
     }
   }
-  const float p = float(reinterpret_cast<const int*>(a.positions)[t]);
   float ss = 0.f;
-  for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
-    const float2 f = turns[i];                       // turns per token, as two floats
-    const float hi = p * f.x;
-    const float r = (hi - rintf(hi)) + fmaf(p, f.y, fmaf(p, f.x, -hi));
-    float sc[2];
-    sincospif(2.f * r, &sc[0], &sc[1]);
+  F32Vec<VEC> x[kRowRegs];
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int c = 2 * i + e;
-      if (c >= H) break;
-      float x = to_f32(src[c]) * a.scale + sc[e];
-      if (add != nullptr) x += to_f32(add[c]);
-      sx[c] = x;
-      ss += x * x;
+  for (int j = 0; j < kRowRegs; ++j) {
+    const int i = v0 + threadIdx.x + j * kRowThreads;
+    if (i < v1) {
+      F32Vec<VEC> y{}, z{};
+      if constexpr (VEC == 4) {
+        y = load_vec<4>(src + i * 4);
+        if (add != nullptr) z = load_vec<4>(add + i * 4);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e)
+          if (i * VEC + e < H) {
+            y.v[e] = to_f32(src[i * VEC + e]);
+            if (add != nullptr) z.v[e] = to_f32(add[i * VEC + e]);
+          }
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; e += 2) {
+        const float f = turns[i * VEC + e], lo = turns[i * VEC + e + 1];       // turns per token, as two floats
+        const float hi = p * f;
+        const float r = (hi - rintf(hi)) + fmaf(p, lo, fmaf(p, f, -hi));
+        float sn, cn;
+        sincospif(2.f * r, &sn, &cn);
+        y.v[e] = y.v[e] * a.scale + sn + z.v[e];
+        y.v[e + 1] = i * VEC + e + 1 < H ? y.v[e + 1] * a.scale + cn + z.v[e + 1] : 0.f;
+        ss += y.v[e] * y.v[e] + y.v[e + 1] * y.v[e + 1];
+      }
+      x[j] = y;
     }
   }
   ss = warp_sum(ss);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
   __syncthreads();
-  const float total = warp_sum((threadIdx.x & 31) < 8 ? red[threadIdx.x & 31] : 0.f);
+  float total = warp_sum((threadIdx.x & 31) < (kRowThreads >> 5) ? red[threadIdx.x & 31] : 0.f);
+  total = row_cluster_sum(total, &cluster_ss, cs);
   const float inv = 1.f / sqrtf(total / float(H) + a.eps);
   float* res = reinterpret_cast<float*>(a.residual) + size_t(t) * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    const float y = sx[i] * inv * to_f32(norm[i]);
-    res[i] = y;
-    out[size_t(t) * H + i] = from_f32<T>(y);
+#pragma unroll
+  for (int j = 0; j < kRowRegs; ++j) {
+    const int i = v0 + threadIdx.x + j * kRowThreads;
+    if (i >= v1) continue;
+    if constexpr (VEC == 4) {
+      F32Vec<4> w = load_vec<4>(norm + i * 4);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) w.v[e] *= x[j].v[e] * inv;
+      store_vec<4>(res + i * 4, w);
+      store_vec<4>(out + size_t(t) * H + i * 4, w);
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e)
+        if (i * VEC + e < H) {
+          const float y = x[j].v[e] * inv * to_f32(norm[i * VEC + e]);
+          res[i * VEC + e] = y;
+          out[size_t(t) * H + i * VEC + e] = from_f32<T>(y);
+        }
+    }
   }
+}
+
+template <typename T>
+int launch_embed(const ZseEmbed* a, int M, void* status, cudaStream_t st) {
+  return launch_rows<2>(embed_design_kernel<T, 4>, embed_design_kernel<T, 2>,
+                        aligned16({a->table, a->bigram, a->norm, a->residual, a->out}), M, a->H, st, *a,
+                        reinterpret_cast<const T*>(a->table), reinterpret_cast<const T*>(a->bigram),
+                        reinterpret_cast<const T*>(a->norm), reinterpret_cast<const float*>(a->turns),
+                        reinterpret_cast<T*>(a->out), reinterpret_cast<Status*>(status));
 }
 
 __global__ void logits_finish_kernel(float* __restrict__ x, int ld, int V, float scale, float cap) {
@@ -396,20 +439,7 @@ extern "C" int zse_post_norm(int dtype, int slot_dtype, void* residual, const vo
 extern "C" int zse_embed_design(int dtype, const ZseEmbed* a, int M, void* status, void* stream) {
   if (M <= 0) return 0;
   if (a->bigram != nullptr && a->buckets <= 0) return ZSE_ERR_SHAPE;
-  const size_t smem = size_t(a->H) * sizeof(float);
-  if (smem > 48 * 1024) return ZSE_ERR_LIMIT;
-  cudaError_t e;
-  if (dtype == kBF16)
-    e = launch_pdl(embed_design_kernel<bf16>, dim3(M), dim3(256), smem, ST(stream), *a, reinterpret_cast<const bf16*>(a->table),
-                   reinterpret_cast<const bf16*>(a->bigram), reinterpret_cast<const bf16*>(a->norm),
-                   reinterpret_cast<const float2*>(a->turns), reinterpret_cast<bf16*>(a->out),
-                   reinterpret_cast<Status*>(status));
-  else
-    e = launch_pdl(embed_design_kernel<float>, dim3(M), dim3(256), smem, ST(stream), *a,
-                   reinterpret_cast<const float*>(a->table), reinterpret_cast<const float*>(a->bigram),
-                   reinterpret_cast<const float*>(a->norm), reinterpret_cast<const float2*>(a->turns),
-                   reinterpret_cast<float*>(a->out), reinterpret_cast<Status*>(status));
-  return e == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+  return dtype == kBF16 ? launch_embed<bf16>(a, M, status, ST(stream)) : launch_embed<float>(a, M, status, ST(stream));
 }
 
 extern "C" int zse_logits_finish(void* logits, int ld, int M, int V, float scale, float cap, void* stream) {
