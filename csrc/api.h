@@ -172,6 +172,7 @@ typedef struct ZseHeads {
   const void* tables;           // block tables [sequences][max_blocks], -1: a hole
   int32_t heads, kv_heads, dim, vdim, chunk, window;
   float scale;
+  int32_t num_blocks;           // blocks in the pool
 } ZseHeads;
 // 1 when the tensor-core kernels take this shape (bfloat16)
 int zse_heads_mma_ok(int dim, int vdim, int block_size);
@@ -184,9 +185,11 @@ int zse_heads_prep(int dtype, void* inp, int ld, const void* planes, int n_plane
 int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads* h, const void* row_seq, const void* positions,
                    void* out, int ldo, const void* gate, void* scratch, int M, int num_splits, int tensor_cores,
                    void* stream);
-// rows of the sequences [first, last) in tiles of queries (bfloat16)
-int zse_heads_attn_chunks(const void* inp, int ld, const ZseHeads* h, const void* cu_q, const void* q_pos0, int first,
-                          int last, int max_q, void* out, int ldo, const void* gate, void* stream);
+// rows of the sequences [first, last) in tiles of queries (bfloat16); rows: rows of inp; form: 1 tcgen05 where it takes the
+// shape, 2 mma.sync
+int zse_heads_attn_chunks(const void* inp, int ld, int rows, const ZseHeads* h, const void* cu_q, const void* q_pos0,
+                          int first, int last, int max_q, void* out, int ldo, const void* gate, int form, void* status,
+                          void* stream);
 
 // ---- memory.cu ----------------------------------------------------------------------------------------------
 typedef struct ZseMemory {

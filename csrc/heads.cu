@@ -4,38 +4,17 @@
 //   heads_simple    a row's heads against the cached keys it sees; any shape, bfloat16 or float
 //   heads_rows      the same on bfloat16 tensor cores: the query heads of a kv head are one 16-row tile, each warp streams
 //                   its own tiles of 16 keys; keys may be split over CTAs (heads_combine merges)
-//   heads_chunk     tiles of 64 queries of a sequence against tiles of 64 keys, flash-attention style
+//   heads_chunk     tiles of 64 queries of a sequence against tiles of 64 keys, flash-attention style (widths up to 128 take
+//                   the tcgen05 form, heads_tc.cu)
 //
 // Cached tiles: [block][kv head][token][dim], then the same for values, dims padded to 8 (the padding is zero).  Scores and
 // softmax are fp32; softmax weights enter the product with the values as two bfloat16 terms (value and remainder).  A row
 // sees the positions from first_seen(position) to its own; block -1 of a table is a hole whose tokens do not exist.
 #include "api.h"
-#include "typed.cuh"
+#include "heads.cuh"
 
 namespace zse {
 namespace {
-
-struct Heads {
-  long long block_stride;
-  int block_size, dp, vp, max_blocks;            // dp, vp: padded widths
-  int block_shift;                               // log2 of the block size, -1: no power of two
-  const int* tables;
-  int heads, kv_heads, dim, vdim, chunk, window;
-  float scale;
-  __device__ __forceinline__ int first_seen(int pos) const {
-    return chunk > 0 ? pos / chunk * chunk : window > 0 ? max(0, pos + 1 - window) : 0;
-  }
-  __device__ __forceinline__ int block_of(int token) const {
-    return block_shift >= 0 ? token >> block_shift : token / block_size;
-  }
-  __device__ __forceinline__ int in_block(int token) const {
-    return block_shift >= 0 ? token & (block_size - 1) : token % block_size;
-  }
-  // first element of a token's key (dp) or value (vp)
-  __device__ __forceinline__ size_t at(int block, int head, int token, int width) const {
-    return size_t(block) * block_stride + (size_t(head) * block_size + token) * width;
-  }
-};
 
 // ---- prep -----------------------------------------------------------------------------------------------------------
 struct HeadsPrepArgs {
@@ -760,12 +739,19 @@ extern "C" int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads
   return rc;
 }
 
-extern "C" int zse_heads_attn_chunks(const void* inp, int ld, const ZseHeads* z, const void* cu_q, const void* q_pos0,
-                                     int first, int last, int max_q, void* out, int ldo, const void* gate, void* stream) {
+extern "C" int zse_heads_attn_chunks(const void* inp, int ld, int rows, const ZseHeads* z, const void* cu_q,
+                                     const void* q_pos0, int first, int last, int max_q, void* out, int ldo,
+                                     const void* gate, int form, void* status, void* stream) {
   if (last <= first || max_q <= 0) return 0;
   if (!zse_heads_mma_ok(z->dim, z->vdim, z->block_size) || ld % 8 || ldo % 2 || z->block_stride % 8 ||
       z->heads % z->kv_heads || z->heads > 65535 || last - first > 65535)
     return ZSE_ERR_SHAPE;
+  const Heads h = heads_of(z);
+  if (form == 1 && heads_tc_ok(h, z->num_blocks, ld, ldo))
+    return launch_heads_tc(reinterpret_cast<const bf16*>(inp), ld, rows, z->k, z->v, z->num_blocks, h,
+                           reinterpret_cast<const int*>(cu_q), reinterpret_cast<const int*>(q_pos0), first, last, max_q,
+                           reinterpret_cast<bf16*>(out), ldo, reinterpret_cast<const bf16*>(gate),
+                           reinterpret_cast<Status*>(status), ST(stream));
   auto run = z->vdim <= 64 ? launch_chunks<8> : z->vdim <= 128 ? launch_chunks<16> : launch_chunks<32>;
   return run(z, inp, ld, cu_q, q_pos0, first, last, max_q, out, ldo, gate, ST(stream));
 }

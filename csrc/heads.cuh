@@ -1,0 +1,35 @@
+// Addressing and masks of attention over cached heads (heads.cu, heads_tc.cu).
+#pragma once
+#include "typed.cuh"
+
+namespace zse {
+
+struct Heads {
+  long long block_stride;
+  int block_size, dp, vp, max_blocks;            // dp, vp: padded widths
+  int block_shift;                               // log2 of the block size, -1: no power of two
+  const int* tables;
+  int heads, kv_heads, dim, vdim, chunk, window;
+  float scale;
+  __device__ __forceinline__ int first_seen(int pos) const {
+    return chunk > 0 ? pos / chunk * chunk : window > 0 ? max(0, pos + 1 - window) : 0;
+  }
+  __device__ __forceinline__ int block_of(int token) const {
+    return block_shift >= 0 ? token >> block_shift : token / block_size;
+  }
+  __device__ __forceinline__ int in_block(int token) const {
+    return block_shift >= 0 ? token & (block_size - 1) : token % block_size;
+  }
+  // first element of a token's key (dp) or value (vp)
+  __device__ __forceinline__ size_t at(int block, int head, int token, int width) const {
+    return size_t(block) * block_stride + (size_t(head) * block_size + token) * width;
+  }
+};
+
+bool heads_tc_ok(const Heads& h, int num_blocks, int ld, int ldo);
+// `rows`: rows of inp; num_blocks: blocks of the pool
+int launch_heads_tc(const bf16* inp, int ld, int rows, const void* k, const void* v, int num_blocks, const Heads& h,
+                    const int* cu_q, const int* q_pos0, int first, int last, int max_q, bf16* out, int ldo,
+                    const bf16* gate, Status* status, cudaStream_t st);
+
+}  // namespace zse

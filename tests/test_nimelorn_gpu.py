@@ -102,6 +102,14 @@ class Attention:
         return out, cu
 
 
+@pytest.fixture
+def form(ops, request):
+    """The tensor-core form of attention in tiles of queries that the test runs on."""
+    ops.heads_form, old = request.param, ops.heads_form
+    yield request.param
+    ops.heads_form = old
+
+
 @pytest.mark.parametrize("dt", [BF, F32])
 @pytest.mark.parametrize("name", list(SPECS))
 @pytest.mark.parametrize("bs", [64, 16, 128])
@@ -118,12 +126,13 @@ def test_rows_against_cached_keys(ops, name, dt, bs):
 
 
 @pytest.mark.parametrize("name", [n for n in SPECS if n != "general"])
-@pytest.mark.parametrize("bs", [64, 32])
-def test_tiles_of_queries_against_cached_keys(ops, name, bs):
+@pytest.mark.parametrize("bs", [64, 32, 48])
+@pytest.mark.parametrize("form", [1, 2], indirect=True)
+def test_tiles_of_queries_against_cached_keys(ops, name, bs, form):
     A = Attention(SPECS[name], BF, bs=bs, blocks=40 * 64 // bs, width=12 * 64 // bs)
     assert ops.heads_expands(A.spec, BF)
     A.tables[2, 2] = -1
-    spans = [(3, 5), (0, 70), (200, 17), (400, 130), (63, 64)]     # the first sequence is not part of the call
+    spans = [(3, 5), (0, 70), (200, 17), (390, 130), (63, 64)]     # the first sequence is not part of the call
     out, cu = A.chunks(ops, spans, first=1)
     assert (out[: cu[1]] == 0).all()
     for s in range(1, len(spans)):
@@ -131,9 +140,10 @@ def test_tiles_of_queries_against_cached_keys(ops, name, bs):
             assert rel(out[cu[s] + i], A.plain(cu[s] + i, s, spans[s][0] + i)) < tol(BF), (s, i)
 
 
-@pytest.mark.parametrize("dt,what", [(BF, "rows"), (F32, "rows"), (BF, "tiles")])
+@pytest.mark.parametrize("dt,what,form", [(BF, "rows", 1), (F32, "rows", 1), (BF, "tiles", 1), (BF, "tiles", 2)],
+                         indirect=["form"])
 @pytest.mark.parametrize("name", ["grouped", "one-kv-head", "half-steps", "window"])
-def test_one_loud_key_inside_and_outside(ops, name, dt, what):
+def test_one_loud_key_inside_and_outside(ops, name, dt, what, form):
     """A key that takes all the weight sits on the first place that is seen, one before it, far away, on block borders, on
     the token itself and on the next one."""
     spec = SPECS[name]

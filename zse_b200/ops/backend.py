@@ -459,6 +459,7 @@ class CudaOps(TorchOps):
         self._norm_ctx = None
         self._logits16 = None
         self.latent_form = 1           # decode attention over latent rows: 1 tcgen05 (csrc/latent_tc.cu), 2 mma.sync
+        self.heads_form = 1            # tiles of queries over cached heads: 1 tcgen05 (csrc/heads_tc.cu), 2 mma.sync
         self._no_tables = torch.zeros(1, 1, dtype=torch.int32, device=self.device)
         self.attn_prefill_tc = env.flag("ZSE_ATTN_PREFILL_TC")
 
@@ -840,7 +841,7 @@ class CudaOps(TorchOps):
 
     def heads_attn_chunks(self, inp, kv, block_tables, cu_q, q_pos0, positions, first, last, max_q, out, spec):
         self.n.heads_attn_chunks(inp, self.n.heads(kv, spec, block_tables), cu_q, q_pos0, first, last, max_q, out,
-                                 self._head_gate(inp, spec))
+                                 self._head_gate(inp, spec), self.heads_form, self.status.ptr)
 
     def memory_expands(self, spec, dtype) -> bool:
         return dtype == torch.bfloat16 and self.n.memory_chunk_ok(spec)

@@ -70,7 +70,8 @@ class Embed(Structure):
 class Heads(Structure):
     _fields_ = [("k", c_void_p), ("v", c_void_p), ("block_stride", c_int64)] + \
                [(n, c_int32) for n in ("block_size", "dim_pad", "vdim_pad", "max_blocks")] + [("tables", c_void_p)] + \
-               [(n, c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "chunk", "window")] + [("scale", c_float)]
+               [(n, c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "chunk", "window")] + [("scale", c_float),
+                                                                                               ("num_blocks", c_int32)]
 
 
 class Memory(Structure):
@@ -216,8 +217,8 @@ _SIGS = {
                                c_int, c_int, c_int, c_int, c_int, c_float, c_void_p]),
     "zse_heads_attn": (c_int, [c_int, c_void_p, c_int, POINTER(Heads), c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                c_void_p, c_int, c_int, c_int, c_void_p]),
-    "zse_heads_attn_chunks": (c_int, [c_void_p, c_int, POINTER(Heads), c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
-                                      c_int, c_void_p, c_void_p]),
+    "zse_heads_attn_chunks": (c_int, [c_void_p, c_int, c_int, POINTER(Heads), c_void_p, c_void_p, c_int, c_int, c_int,
+                                      c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p]),
     "zse_memory_chunk_ok": (c_int, [c_int] * 2),
     "zse_memory_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                 POINTER(Memory), c_int, c_void_p]),
@@ -596,7 +597,7 @@ def heads(view, spec, block_tables) -> Heads:
     """``view``: ``models.hybrid.PagedHeads``."""
     return Heads(view.k.data_ptr(), view.v.data_ptr(), view.block_stride, view.block_size, view.k.shape[3], view.v.shape[3],
                  block_tables.stride(0), block_tables.data_ptr(), spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.chunk,
-                 spec.window, float(spec.scale))
+                 spec.window, float(spec.scale), view.k.shape[0])
 
 
 def heads_mma_ok(spec, block_size: int) -> bool:
@@ -615,9 +616,9 @@ def heads_attn(inp, h, row_seq, positions, out, gate, scratch, M, num_splits, te
         2 if num_splits > 1 else 1)
 
 
-def heads_attn_chunks(inp, h, cu_q, q_pos0, first, last, max_q, out, gate):
-    _ck(load().zse_heads_attn_chunks(_p(inp), inp.stride(0), byref(h), _p(cu_q), _p(q_pos0), first, last, max_q, _p(out),
-                                     out.stride(0), gate, _stream()), "heads_attn_chunks")
+def heads_attn_chunks(inp, h, cu_q, q_pos0, first, last, max_q, out, gate, form, status):
+    _ck(load().zse_heads_attn_chunks(_p(inp), inp.stride(0), inp.shape[0], byref(h), _p(cu_q), _p(q_pos0), first, last, max_q,
+                                     _p(out), out.stride(0), gate, form, status, _stream()), "heads_attn_chunks")
 
 
 def memory(states, at, state_rows, head_norm, spec, eps) -> Memory:
