@@ -30,6 +30,10 @@ CASES = {
                               attention_layer(8, 1, 136, 144, 64, None),
                               mlstm_layer(5, 48, 64, moe(9, 8, 16, 0.9, 2.0, 24)),
                               attention_layer(34, 2, 40, 72, 32, None, kv_from=0)], eps=1e-6),
+    # one kind of mixer only: no cached keys at all, no recurrent layer at all
+    "memories-only": config(64, 90, [mlstm_layer(2, 24, 32, None), mlstm_layer(1, 64, 16, dense(24))]),
+    "attention-only": config(64, 90, [attention_layer(4, 2, 16, 24, 30, None),
+                                      attention_layer(2, 1, 32, 16, 200, moe(4, 2, 16, 1.0, 1.3, 16))]),
 }
 
 
