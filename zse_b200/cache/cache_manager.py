@@ -328,7 +328,8 @@ class KVCacheManager:
         keep_from = self._config.first_seen(first_new)
         if e is None or keep_from <= 0:
             return
-        for idx in range(min(keep_from // self._block_size, len(e.blocks))):
+        kept = (self._config.kept_first + self._block_size - 1) // self._block_size
+        for idx in range(kept, min(keep_from // self._block_size, len(e.blocks))):
             if idx not in e.evicted_indices:
                 self._evictor.remove_block(e.blocks[idx].block_id, seq_id)
                 self._page_table.evict_block(seq_id, idx)

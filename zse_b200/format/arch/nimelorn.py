@@ -4,6 +4,7 @@ or routed feed-forward or none; norms sit on the sublayers' outputs.  Tensor nam
 from typing import List
 
 from ..config import HeadsSpec, MatrixMemorySpec, ModelConfig, MoESpec
+from ..layer_specs import mixer_types
 from ..spec import QuantMethod
 from .base import ArchAdapter, register_adapter
 
@@ -21,7 +22,7 @@ class NimelornAdapter(ArchAdapter):
         hf = hf_config
         layers = hf["layers"]
         for i, layer in enumerate(layers):
-            if layer["type"] not in ("attention", "mlstm"):
+            if layer["type"] not in mixer_types(self.ARCH_NAME):
                 raise ValueError(f"layer {i}: unknown mixer '{layer['type']}'")
             mlp = layer.get("mlp")
             if mlp is not None and mlp["kind"] not in ("dense", "moe"):

@@ -11,6 +11,8 @@ from dataclasses import dataclass, field, fields
 from typing import Any, Dict, List, Optional
 
 from . import serializer
+from .layer_specs import (DenseSpec, HeadsSpec, LatentSpec, LayerSpec, MatrixMemorySpec, MoESpec,  # noqa: F401
+                          RECURRENT, StateSpaceSpec, read_ff, read_mixer)
 from .spec import DEFAULT_GROUP_SIZE, DEFAULT_QUANT_BITS, QuantMethod
 
 
@@ -34,189 +36,6 @@ class QuantConfig:
     def from_dict(cls, d: dict) -> "QuantConfig":
         names = {f.name for f in fields(cls)}
         return cls(**{k: v for k, v in d.items() if k in names})
-
-
-@dataclass
-class LayerSpec:
-    head_dim: int
-    num_kv_heads: int
-    rope_theta: float
-    rotary_dim: int          # leading pairs (i, i + head_dim/2), i < rotary_dim/2, rotate; the rest pass through
-    window: int              # 0 = full causal attention
-    k_is_v: bool             # no v_proj: V is the k_proj output before its norm
-    scale: float
-    softcap: float           # 0 = none
-    qk_norm: bool            # per-head RMSNorm of q and k (learned weight) and of v (no weight)
-
-
-def _up8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
-@dataclass(frozen=True)
-class LatentSpec:
-    """Attention over a shared low-rank latent: a token caches its normed latent (``kv_rank``) and one rotated key part
-    (``rot_dim``) that all heads share; a head's key and value are linear images of the latent."""
-    heads: int
-    dim: int                 # query/key dimensions of a head that carry no position
-    rot_dim: int             # ... and those that are rotated
-    vdim: int
-    kv_rank: int
-    window: int              # a position sees itself and the window - 1 before it; 0 = everything before it
-    scale: float
-    rot_dims: int            # leading dimensions of the rot_dim part that rotate (pairs 2i, 2i + 1)
-    rot_base: float
-    gated: bool = True       # heads are multiplied by sigmoid(W_g h) before the output projection
-
-    @property
-    def qk_dim(self) -> int:
-        return self.dim + self.rot_dim
-
-    # columns of the fused input projection [q | latent, rotated key | gate]; every section starts on 8 elements
-    @property
-    def latent_col(self) -> int:
-        return _up8(self.heads * self.qk_dim)
-
-    @property
-    def gate_col(self) -> int:
-        return self.latent_col + _up8(self.kv_rank + self.rot_dim)
-
-    @property
-    def in_width(self) -> int:
-        return self.gate_col + (_up8(self.heads * self.vdim) if self.gated else 0)
-
-    @property
-    def row(self) -> int:
-        """Elements of a cached token: [latent | rotated key part], padded to an odd number of 16-byte pieces (of a
-        16-bit type): consecutive rows then start in different shared-memory banks and can be used where a plain copy
-        puts them."""
-        n = _up8(self.kv_rank + self.rot_dim)
-        return n if n // 8 % 2 else n + 8
-
-
-@dataclass(frozen=True)
-class MoESpec:
-    """Routed feed-forward: ``top`` of ``experts`` per token, chosen and weighted by ``score``.  ``shared_ff`` > 0 adds an
-    expert that every token uses."""
-    experts: int
-    top: int
-    ff: int
-    shared_ff: int = 0
-    score: str = "sigmoid"       # of the router's logits: "sigmoid" (each on its own) or "softmax" (over all experts)
-    activation: str = "gelu"     # exact (erf) gelu, or "clamped_glu": two up products, see ``ops.reference.clamped_glu``
-    weigh: str = "input"         # the weight scales the expert's "input" or "output"
-    normalise: bool = False      # the chosen scores are divided by their sum
-    scale: float = 1.0           # ... and multiplied by this
-    limit: float = 0.0           # clamp of "clamped_glu"
-    shared_limit: float = 0.0
-    shared_gate: bool = False    # the shared expert is multiplied by sigmoid(w . h), one number per token
-
-    @property
-    def gated(self) -> bool:
-        return self.activation == "clamped_glu"
-
-    @property
-    def router_rows(self) -> int:
-        """Columns of the router's product: the experts, and the shared expert's gate behind them."""
-        return self.experts + (1 if self.shared_gate else 0)
-
-
-@dataclass(frozen=True)
-class DenseSpec:
-    """Feed-forward of one up product, an activation and one down product."""
-    ff: int
-    activation: str = "relu2"    # the square of relu
-
-
-@dataclass(frozen=True)
-class HeadsSpec:
-    """Attention of ``heads`` query heads over ``kv_heads`` key/value heads whose widths may differ; no rotation."""
-    heads: int
-    kv_heads: int
-    dim: int
-    vdim: int
-    scale: float
-    chunk: int = 0               # > 0: a position sees the positions of its own chunk of this size only
-    window: int = 0              # > 0: a position sees itself and the window - 1 before it
-    kv_from: int = -1            # >= 0: keys and values are those of that layer
-    gated: bool = True           # a head's result is multiplied by sigmoid(w_h . x)
-
-    @property
-    def own_kv(self) -> bool:
-        return self.kv_from < 0
-
-    # columns of the fused input projection [q | k | v | gate]; every section starts on 8 elements
-    @property
-    def k_col(self) -> int:
-        return _up8(self.heads * self.dim)
-
-    @property
-    def v_col(self) -> int:
-        return self.k_col + (_up8(self.kv_heads * self.dim) if self.own_kv else 0)
-
-    @property
-    def gate_col(self) -> int:
-        return self.v_col + (_up8(self.kv_heads * self.vdim) if self.own_kv else 0)
-
-    @property
-    def in_width(self) -> int:
-        return self.gate_col + (_up8(self.heads) if self.gated else 0)
-
-    @property
-    def row(self) -> int:
-        """Elements of a cached token."""
-        return self.kv_heads * (_up8(self.dim) + _up8(self.vdim))
-
-    def first_seen(self, position: int) -> int:
-        """First position that the token at ``position`` sees."""
-        if self.chunk > 0:
-            return position // self.chunk * self.chunk
-        return max(0, position + 1 - self.window) if self.window > 0 else 0
-
-
-@dataclass(frozen=True)
-class MatrixMemorySpec:
-    """Recurrent mixer whose heads keep a [dim, vdim] matrix memory, a key sum [dim] and a running maximum of the log
-    gates (mLSTM)."""
-    heads: int
-    dim: int
-    vdim: int
-    gate_cap: float
-
-    # columns of the fused input projection [q | k | v | output gate | input and forget gates]
-    @property
-    def k_col(self) -> int:
-        return _up8(self.heads * self.dim)
-
-    @property
-    def v_col(self) -> int:
-        return 2 * self.k_col
-
-    @property
-    def gate_col(self) -> int:
-        return self.v_col + _up8(self.heads * self.vdim)
-
-    @property
-    def if_col(self) -> int:
-        return self.gate_col + _up8(self.heads * self.vdim)
-
-    @property
-    def in_width(self) -> int:
-        return self.if_col + _up8(2 * self.heads)
-
-    # state of one sequence, in 32-bit elements: memory [heads, dim, vdim], key sum [heads, dim], maximum [heads]; every
-    # part starts on 4 elements
-    @property
-    def sum_at(self) -> int:
-        return (self.heads * self.dim * self.vdim + 3) // 4 * 4
-
-    @property
-    def max_at(self) -> int:
-        return self.sum_at + (self.heads * self.dim + 3) // 4 * 4
-
-    @property
-    def state_floats(self) -> int:
-        return self.max_at + (self.heads + 3) // 4 * 4
 
 
 @dataclass
@@ -253,6 +72,8 @@ class ModelConfig:
     embed_multiplier: Optional[float] = None
     # {"bigram": {"buckets", "mul_prev", "mul_cur"}, "sinusoid_base", "norm"}: what is added to a token's embedding
     embed_design: Optional[Dict[str, Any]] = None
+    # {"start", "stop", "times"}: these layers run several times in a row, each pass from [x; embedding]
+    loop: Optional[Dict[str, int]] = None
     logit_scale: Optional[float] = None
     weight_dtype: Optional[str] = None
     multimodal: Optional[Dict[str, Any]] = None
@@ -329,57 +150,60 @@ class ModelConfig:
         return self.is_design and not self.is_latent
 
     def mixer_spec(self, i: int):
-        """``HeadsSpec`` or ``MatrixMemorySpec`` of layer ``i`` of a hybrid design."""
-        L = self.design_layers[i]
-        m = L["mixer"]
-        if L["type"] == "mlstm":
-            return MatrixMemorySpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
-        src = m.get("kv_from")
-        return HeadsSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
-                         chunk=int((m.get("mask") or {}).get("size") or 0), kv_from=-1 if src is None else int(src))
+        """``HeadsSpec`` or one of ``RECURRENT`` of layer ``i`` of a hybrid design."""
+        return read_mixer(self.arch, self.design_layers[i])
 
     def ff_spec(self, i: int):
         """``DenseSpec``, ``MoESpec`` or None of layer ``i`` of a hybrid design."""
-        m = self.design_layers[i].get("mlp")
-        if m is None:
-            return None
-        if m["kind"] == "dense":
-            return DenseSpec(int(m["ff"]))
-        r, e, s = m["router"], m["expert"], m.get("shared")
-        return MoESpec(int(r["experts"]), int(r["top"]), int(e["ff"]), int(s["ff"]) if s else 0, "softmax",
-                       "clamped_glu", "output", True, float(r.get("scale", 1.0)), float(e["limit"]),
-                       float(s["limit"]) if s else 0.0, bool(s))
+        return read_ff(self.arch, self.design_layers[i])
+
+    @property
+    def layer_runs(self) -> List[int]:
+        """The layers in the order in which a token passes them; those of a loop come once per pass.  Every run has its own
+        cache or state."""
+        n, loop = self.num_layers, self.loop
+        if not loop:
+            return list(range(n))
+        body = list(range(loop["start"], loop["stop"]))
+        return list(range(loop["start"])) + body * loop["times"] + list(range(loop["stop"], n))
+
+    def enters_loop(self, run: int) -> bool:
+        """Whether layer run ``run`` is the first of a pass of the loop."""
+        if not self.loop:
+            return False
+        at, body = run - self.loop["start"], self.loop["stop"] - self.loop["start"]
+        return 0 <= at < body * self.loop["times"] and at % body == 0
 
     @property
     def cache_layers(self) -> Dict[int, int]:
-        """Layer -> its layer of the cache pool; layers without keys and values of their own have none."""
+        """Layer run -> its layer of the cache pool; runs without keys and values of their own have none."""
         if not self.is_hybrid:
             return {i: i for i in range(self.num_layers)}
-        own = [i for i in range(self.num_layers) if isinstance(self.mixer_spec(i), HeadsSpec)
+        own = [r for r, i in enumerate(self.layer_runs) if isinstance(self.mixer_spec(i), HeadsSpec)
                and self.mixer_spec(i).own_kv]
-        return {i: n for n, i in enumerate(own)}
+        return {r: n for n, r in enumerate(own)}
 
     @property
     def num_cache_layers(self) -> int:
         return max(1, len(self.cache_layers))
 
+    def _state_layout(self):
+        out, at = {}, 0
+        for r, i in enumerate(self.layer_runs if self.is_hybrid else ()):
+            s = self.mixer_spec(i)
+            if isinstance(s, RECURRENT):
+                out[r] = at
+                at += (s.state_floats + 3) // 4 * 4
+        return out, at
+
     @property
     def state_offsets(self) -> Dict[int, int]:
-        """Recurrent layer -> its first element in a sequence's state."""
-        out, at = {}, 0
-        if self.is_hybrid:
-            for i in range(self.num_layers):
-                s = self.mixer_spec(i)
-                if isinstance(s, MatrixMemorySpec):
-                    out[i] = at
-                    at += s.state_floats
-        return out
+        """Run of a recurrent layer -> its first element in a sequence's state."""
+        return self._state_layout()[0]
 
     @property
     def state_floats(self) -> int:
-        off = self.state_offsets
-        last = max(off, default=-1)
-        return off[last] + self.mixer_spec(last).state_floats if off else 0
+        return self._state_layout()[1]
 
     @property
     def keeps_state(self) -> bool:
@@ -411,14 +235,22 @@ class ModelConfig:
             return max(w) if w and min(w) > 0 else 0
         return int(self.sliding_window) if (self.sliding_window or 0) > 0 and not self.layer_types else 0
 
+    def _masks(self) -> List[HeadsSpec]:
+        if self.__dict__.get("_mask_specs") is None:
+            self.__dict__["_mask_specs"] = list({(s.chunk, s.window, s.keep_first): s for s in (
+                self.mixer_spec(i) for i in range(self.num_layers)) if isinstance(s, HeadsSpec)}.values())
+        return self.__dict__["_mask_specs"]
+
+    @property
+    def kept_first(self) -> int:
+        """First positions that some layer always sees."""
+        return max((s.keep_first for s in self._masks()), default=0) if self.is_hybrid else 0
+
     def first_seen(self, position: int) -> int:
-        """First position that some layer still sees from ``position`` (and from any later one): the cache may give back
-        the blocks before it."""
+        """First position that some layer still sees from ``position`` (and from any later one), apart from the
+        ``kept_first`` ones: the cache may give back the blocks between."""
         if self.is_hybrid:
-            if self.__dict__.get("_masks") is None:
-                self.__dict__["_masks"] = list({(s.chunk, s.window): s for s in (self.mixer_spec(i) for i in range(
-                    self.num_layers)) if isinstance(s, HeadsSpec)}.values())
-            return min((s.first_seen(position) for s in self.__dict__["_masks"]), default=position)
+            return min((s.first_seen(position) for s in self._masks()), default=position)
         w = self.cache_window
         return max(0, position + 1 - w) if w > 0 else 0
 
@@ -429,9 +261,14 @@ class ModelConfig:
 
     @property
     def norm_weight_offset(self) -> float:
-        """Gemma-2 stores RMSNorm weights as ``w - 1`` (the norm multiplies by ``1 + w``); Gemma-4 and everything
+        """Gemma-2 and Movinex store RMSNorm weights as ``w - 1`` (the norm multiplies by ``1 + w``); Gemma-4 and everything
         else multiply by the stored weight (zse-engine/zse_engine/orchestrator/kernels.py:1475-1478)."""
-        return 1.0 if self.arch == "gemma2" else 0.0
+        return 1.0 if self.arch in ("gemma2", "movinex") else 0.0
+
+    @property
+    def norms_outputs(self) -> bool:
+        """Hybrid designs: norms sit on the sublayers' outputs, not on their inputs."""
+        return self.arch == "nimelorn"
 
     def layer_kind(self, i: int) -> str:
         if self.layer_types and i < len(self.layer_types):
@@ -466,7 +303,8 @@ class ModelConfig:
         if self.is_latent:
             return 1, max(self.latent_spec(i).row for i in range(self.num_layers))
         if self.is_hybrid:
-            return 1, max((self.mixer_spec(i).row for i in self.cache_layers), default=8)
+            rows = [self.mixer_spec(i).row for i in range(self.num_layers) if isinstance(self.mixer_spec(i), HeadsSpec)]
+            return 1, max(rows, default=8)
         local = num_kv_heads or self.num_kv_heads
         tp = max(1, self.num_kv_heads // max(1, local))
         specs = {(s.num_kv_heads, s.head_dim) for s in (self.layer_spec(i) for i in range(self.num_layers))}
@@ -483,8 +321,8 @@ class ModelConfig:
                 if isinstance(m, MoESpec):
                     n += self.hidden_size * (m.router_rows + 3 * m.experts * m.ff + 3 * m.shared_ff)
                 elif m is not None:
-                    n += self.hidden_size * 2 * m.ff
-            return n
+                    n += self.hidden_size * (3 if m.gated else 2) * m.ff
+            return n + (2 * self.hidden_size ** 2 if self.loop else 0)
         if self.is_latent:
             n = 0
             for i in range(self.num_layers):

@@ -24,7 +24,7 @@ from typing import Dict, List, Optional, Union
 
 import torch
 
-from ..format.config import DenseSpec, HeadsSpec, MatrixMemorySpec, MoESpec
+from ..format.config import DenseSpec, HeadsSpec, MatrixMemorySpec, MoESpec, StateSpaceSpec
 from ..format.loader import ZSELoader
 from ..ops.backend import LinearWeight
 from .decoder import StepBuffers
@@ -46,7 +46,7 @@ class EmbedDesign:
 
 @dataclass
 class HybridLayer:
-    spec: Union[HeadsSpec, MatrixMemorySpec]
+    spec: Union[HeadsSpec, MatrixMemorySpec, StateSpaceSpec]
     ff: Union[DenseSpec, MoESpec, None]
     norm1: torch.Tensor
     w_in: LinearWeight
@@ -55,12 +55,22 @@ class HybridLayer:
     # attention
     q_norm: Optional[torch.Tensor] = None
     k_norm: Optional[torch.Tensor] = None
-    cache_layer: int = -1
+    bias: Optional[torch.Tensor] = None     # of the columns of w_in before the gates
+    freqs: Optional[torch.Tensor] = None    # of the rotation
     # matrix memory
     w_if: Optional[LinearWeight] = None     # the rows of w_in that make the gates
     if_bias: Optional[torch.Tensor] = None  # fp32 [2 * heads]
     head_norm: Optional[torch.Tensor] = None
-    state_at: int = 0
+    # state space
+    conv_w: Optional[torch.Tensor] = None   # fp32 [taps, channels]
+    conv_b: Optional[torch.Tensor] = None
+    dt_bias: Optional[torch.Tensor] = None  # fp32 [heads], like the next two
+    neg_a: Optional[torch.Tensor] = None    # -exp(A_log)
+    D: Optional[torch.Tensor] = None
+    out_norm: Optional[torch.Tensor] = None
+    # factors of the sublayers' results
+    scale1: Optional[torch.Tensor] = None
+    scale2: Optional[torch.Tensor] = None
     # feed-forward
     up_w: Optional[LinearWeight] = None
     down_w: Optional[LinearWeight] = None
@@ -73,6 +83,30 @@ class HybridLayer:
     @property
     def moe(self) -> Optional[MoESpec]:
         return self.ff if isinstance(self.ff, MoESpec) else None
+
+
+@dataclass
+class LayerRun:
+    """One run of a layer: layers of a loop run several times, each run with its own keys and values or its own state."""
+    layer: HybridLayer
+    cache_layer: int = -1                   # of the cache pool (attention)
+    state_at: int = 0                       # first element of its part of a sequence's state (recurrent mixers)
+    enters_loop: bool = False               # first of a pass of the loop
+
+
+@dataclass
+class Pass:
+    """What a pass's layers need to know about it."""
+    kv: torch.Tensor
+    M: int
+    num_seqs: int
+    max_q_len: int
+    row_seq: Optional[torch.Tensor]         # None: every row is a sequence of its own (decode), like the next
+    cu_q: Optional[torch.Tensor]
+    short: tuple                            # rows and sequences that run token by token
+    planes_ok: bool                         # projections come as split-K planes
+    partials: torch.Tensor
+    splits: int
 
 
 class PagedHeads:
@@ -109,6 +143,10 @@ class HybridStepBuffers(StepBuffers):
 
         self.in_views = views([s.in_width for s in specs], act)
         self.out_views = views([s.heads * s.vdim for s in specs], act)
+        spaces = [s for s in specs if isinstance(s, StateSpaceSpec)]
+        self.xbc_views = views([s.conv_width for s in spaces], act) if spaces else {}
+        self.dt = z(max_tokens * max([1] + [s.heads for s in spaces]), dt=f32)
+        self.dt_side = z(max_tokens * max([1] + [s.in_width - s.dt_col for s in spaces]), dt=f32)
         planes = z(max_planes * self.plane_rows * max(s.in_width for s in specs), dt=f32)
         self.in_plane_views = {w: planes[: max_planes * self.plane_rows * w].view(max_planes, self.plane_rows, w)
                                for w in {s.in_width for s in specs}}
@@ -118,6 +156,9 @@ class HybridStepBuffers(StepBuffers):
                               partials[: max_tokens * H].view(1, max_tokens, H))
         dense = [L.ff.ff for L in model.layers if isinstance(L.ff, DenseSpec)]
         self.act_views = views(dense, act) if dense else {}
+        wide = [L.ff.ff for L in model.layers if isinstance(L.ff, DenseSpec) and L.ff.gated
+                and model.ops.glu_expands(L.ff.ff, H, act)]
+        self.glu = z(max_tokens * 2 * max([0] + wide), dt=act)
         rows_split = min(max_tokens, max(256, max_seqs))      # only decode passes split their keys
         self.attn_scratch = z(rows_split * attn_splits * max([1] + [s.heads * (s.vdim + 2) for s in heads]), dt=f32)
         gate_w = max([1] + [2 * s.heads for s in memories])
@@ -132,6 +173,7 @@ class HybridStepBuffers(StepBuffers):
 
 
 class HybridModel(DesignModel):
+    """Layers whose norms sit on the sublayers' outputs; ``models.looped`` has the other placement."""
     kernel_group = "hybrid"
 
     # ---- loading --------------------------------------------------------------------------------------
@@ -155,7 +197,7 @@ class HybridModel(DesignModel):
                 L = HybridLayer(s, m, r.get(p + "norm1"), ops.dense_linear(w), r.linear(p + "mix.o"))
                 L.w_if = ops.dense_linear(w[s.if_col: s.if_col + 2 * s.heads])
                 L.if_bias = torch.cat([t("mix.i.b"), t("mix.f.b")]).float().contiguous()
-                L.head_norm, L.state_at = r.get(p + "mix.norm"), c.state_offsets[i]
+                L.head_norm = r.get(p + "mix.norm")
             else:
                 parts = [(0, t("mix.q")), (s.gate_col, t("mix.g"))]
                 if s.own_kv:
@@ -164,27 +206,39 @@ class HybridModel(DesignModel):
                                 r.linear(p + "mix.o"), q_norm=r.get(p + "mix.q.norm"))
                 if s.own_kv:
                     L.k_norm = r.get(p + "mix.k.norm")
-                L.cache_layer = c.cache_layers[i if s.own_kv else s.kv_from]
             if m is not None:
                 L.norm2 = r.get(p + "norm2")
             if isinstance(m, DenseSpec):
                 L.up_w, L.down_w = r.linear(p + "mlp.up"), r.linear(p + "mlp.down")
             elif m is not None:
-                rows = [(0, t("mlp.router"))] + ([(m.experts, t("mlp.shared.sg"))] if m.shared_gate else [])
-                L.router = ops.dense_linear(r.stack(rows, m.router_rows, H))
-                count = lambda w: self._count(w)
-                L.up = count(ops.moe_up([(t(f"mlp.e{e}.gate"), t(f"mlp.e{e}.up")) for e in range(m.experts)],
-                                        self.act_dtype, m))
-                L.down = r.stack([(e * H, t(f"mlp.e{e}.down")) for e in range(m.experts)], m.experts * H, m.ff)
-                if m.shared_ff:
-                    L.shared_up = count(ops.moe_up([(t("mlp.shared.gate"), t("mlp.shared.up"))], self.act_dtype,
-                                                   m))
-                    L.shared_down = r.get(p + "mlp.shared.down")
+                self._load_experts(r, L, p, m, H)
             self.layers.append(L)
             if progress:
                 progress(i + 1, c.num_layers)
         self.lm_head = r.linear("head")
         r.release()
+        self._plan_runs()
+
+    def _load_experts(self, r, L: HybridLayer, p: str, m: MoESpec, H: int) -> None:
+        ops, t = self.ops, lambda name: r.tensor(p + name)
+        rows = [(0, t("mlp.router"))] + ([(m.experts, t("mlp.shared.sg"))] if m.shared_gate else [])
+        L.router = ops.dense_linear(r.stack(rows, m.router_rows, H))
+        L.up = self._count(ops.moe_up([(t(f"mlp.e{e}.gate"), t(f"mlp.e{e}.up")) for e in range(m.experts)],
+                                      self.act_dtype, m))
+        L.down = r.stack([(e * H, t(f"mlp.e{e}.down")) for e in range(m.experts)], m.experts * H, m.ff)
+        if m.shared_ff:
+            L.shared_up = self._count(ops.moe_up([(t("mlp.shared.gate"), t("mlp.shared.up"))], self.act_dtype, m))
+            L.shared_down = r.get(p + "mlp.shared.down")
+
+    def _plan_runs(self) -> None:
+        """The order of the layers' runs, and where each keeps its keys and values or its state."""
+        c, caches, states = self.config, self.config.cache_layers, self.config.state_offsets
+        self.runs: List[LayerRun] = []
+        for n, i in enumerate(c.layer_runs):
+            s = self.layers[i].spec
+            own = not isinstance(s, HeadsSpec) or s.own_kv
+            self.runs.append(LayerRun(self.layers[i], caches.get(n if own else s.kv_from, -1), states.get(n, 0),
+                                      c.enters_loop(n)))
         self.heads_specs = [L.spec for L in self.layers if isinstance(L.spec, HeadsSpec)]
         self._views: Dict[tuple, PagedHeads] = {}
 
@@ -197,17 +251,17 @@ class HybridModel(DesignModel):
                      max_planes: int = 8, attn_splits: int = 1) -> HybridStepBuffers:
         return HybridStepBuffers(self, max_tokens, max_seqs, max_blocks, max_planes, logits_rows or max_seqs, attn_splits)
 
-    def _heads_view(self, kv: torch.Tensor, L: HybridLayer) -> PagedHeads:
-        key = (kv.data_ptr(), L.cache_layer)
+    def _heads_view(self, kv: torch.Tensor, run: LayerRun) -> PagedHeads:
+        key = (kv.data_ptr(), run.cache_layer)
         v = self._views.get(key)
         if v is None:
-            v = self._views[key] = PagedHeads(kv[L.cache_layer], L.spec)
+            v = self._views[key] = PagedHeads(kv[run.cache_layer], run.layer.spec)
         return v
 
     def attention_splits(self, seqs: int, max_len: int, most: int, sms: int) -> int:
         if not self.heads_specs:
             return 1
-        span = max(min(max_len, s.chunk or max_len, s.window or max_len) for s in self.heads_specs)
+        span = max(min(max_len, s.chunk or max_len, s.window + s.keep_first if s.window else max_len) for s in self.heads_specs)
         ctas = seqs * min(s.kv_heads * ((s.heads // s.kv_heads + 15) // 16) for s in self.heads_specs)
         want = (2 * sms + ctas - 1) // ctas
         n = int(max(1, min(want, span // 128, most)))
@@ -227,61 +281,91 @@ class HybridModel(DesignModel):
         b.row_seq[:at].copy_(b.h_row_seq[:at], non_blocking=True)
 
     # ---- forward --------------------------------------------------------------------------------------
+    def _pass(self, b: HybridStepBuffers, kv, M: int, mode: str, num_seqs: int, max_q_len: int, attn_splits: int) -> Pass:
+        decode = mode == "decode"
+        planes_ok = M <= b.plane_rows
+        return Pass(kv, M, num_seqs, max_q_len, None if decode else b.row_seq, None if decode else b.cu_q,
+                    (M, num_seqs) if decode else (b.short_rows, b.short_seqs), planes_ok,
+                    b.partial_views[0 if planes_ok else 1], attn_splits)
+
+    def _mix(self, b: HybridStepBuffers, p: Pass, run: LayerRun) -> int:
+        """The layer's mixer on ``b.xnorm``; its result is in the returned number of planes of ``p.partials``."""
+        ops, L, s, M = self.ops, run.layer, run.layer.spec, p.M
+        inp, planes, n_in = b.in_views[s.in_width], b.in_plane_views[s.in_width], 0
+        side = b.dt_side if isinstance(s, StateSpaceSpec) else None      # step sizes stay fp32
+        if p.planes_ok:
+            n_in = ops.linear_partial(L.w_in, b.xnorm, M, planes)
+        else:
+            ops.linear(L.w_in, b.xnorm, M, inp, side=None if side is None else (s.dt_col, side))
+        out = b.out_views[s.heads * s.vdim]
+        mixer = self._attend if isinstance(s, HeadsSpec) else self._space if side is not None else self._remember
+        mixer(b, p, run, inp, planes, n_in, out)
+        return ops.linear_partial(L.o, out, M, p.partials)
+
+    def _attend(self, b, p: Pass, run: LayerRun, inp, planes, n_in: int, out) -> None:
+        ops, L, s, M = self.ops, run.layer, run.layer.spec, p.M
+        view = self._heads_view(p.kv, run)
+        ops.heads_prep(inp, planes, n_in, view, b.slots, L, s, self.config.rms_norm_eps, M, b.positions)
+        rows, seqs = p.short if ops.heads_expands(s, self.act_dtype) else (M, p.num_seqs)
+        if rows:
+            ops.heads_attn(inp, view, b.block_tables, p.row_seq, b.positions, out, rows, s, b.attn_scratch, p.splits)
+        if seqs < p.num_seqs:
+            ops.heads_attn_chunks(inp, view, b.block_tables, b.cu_q, b.q_pos0, b.positions, seqs, p.num_seqs, p.max_q_len,
+                                  out, s)
+
+    def _remember(self, b, p: Pass, run: LayerRun, inp, planes, n_in: int, out) -> None:
+        ops, L, s, M, eps = self.ops, run.layer, run.layer.spec, p.M, self.config.rms_norm_eps
+        n_gate = 0 if n_in else ops.linear_partial(L.w_if, b.xnorm, M, b.gate_planes)
+        ops.memory_prep(inp, planes, n_in, b.gate_planes, n_gate, b.gates, L, s, M)
+        rows, seqs = p.short if ops.memory_expands(s, self.act_dtype) else (M, p.num_seqs)
+        states = self.states.rows
+        if seqs:
+            ops.memory_tokens(inp, b.gates, states, run.state_at, b.state_rows, p.cu_q, L, out, seqs, M, s, eps)
+        if seqs < p.num_seqs:
+            ops.memory_chunks(inp, b.gates, states, run.state_at, b.state_rows, b.cu_q, L, out, seqs, p.num_seqs, rows, M, s,
+                              eps, b.memory_ws)
+
+    def _space(self, b, p: Pass, run: LayerRun, inp, planes, n_in: int, out) -> None:
+        ops, L, s, M, states = self.ops, run.layer, run.layer.spec, p.M, self.states.rows
+        xbc = b.xbc_views[s.conv_width]
+        ops.state_space_prep(inp, planes, n_in, b.dt_side, xbc, b.dt, states, run.state_at, b.state_rows, p.row_seq, p.cu_q,
+                             L, s, M, p.num_seqs)
+        seqs = p.short[1] if ops.state_space_expands(s, self.act_dtype) else p.num_seqs
+        if seqs:
+            ops.state_space_tokens(inp, xbc, b.dt, states, run.state_at, b.state_rows, p.cu_q, L, out, seqs, M, s)
+        if seqs < p.num_seqs:
+            ops.state_space_chunks(inp, xbc, b.dt, states, run.state_at, b.state_rows, b.cu_q, L, out, seqs, p.num_seqs, M, s)
+        ops.group_norm(out, L.out_norm, s.norm_groups, M, self.config.rms_norm_eps)
+
+    def _feed(self, b: HybridStepBuffers, p: Pass, L: HybridLayer):
+        """The layer's feed-forward on ``b.xnorm``: (planes of ``p.partials``, the experts' rows or None)."""
+        if L.moe is not None:
+            return 0, self.ops.moe(L, b.xnorm, p.M, b.moe_ws)
+        act = b.act_views[L.ff.ff]
+        if L.ff.gated:
+            self.ops.linear_glu(L.up_w, b.xnorm, p.M, act, L.ff.activation, b.glu)
+        else:
+            self.ops.linear_act(L.up_w, b.xnorm, p.M, act, L.ff.activation)
+        return self.ops.linear_partial(L.down_w, act, p.M, p.partials), None
+
+    def _logits(self, b: HybridStepBuffers, rows: int) -> None:
+        torch.index_select(b.xnorm, 0, b.logit_rows[:rows], out=b.xsel[:rows])
+        self.ops.linear_f32(self.lm_head, b.xsel, rows, b.logits)
+
     def forward(self, b: HybridStepBuffers, kv: torch.Tensor, M: int, mode: str, num_seqs: int, max_q_len: int = 1,
                 n_logit_rows: int = 0, attn_splits: int = 1) -> None:
-        c, ops, eps = self.config, self.ops, self.config.rms_norm_eps
-        decode = mode == "decode"
-        row_seq, cu_q = (None, None) if decode else (b.row_seq, b.cu_q)
-        short = (M, num_seqs) if decode else (b.short_rows, b.short_seqs)
-        planes_ok = M <= b.plane_rows
-        partials = b.partial_views[0 if planes_ok else 1]
+        ops, eps = self.ops, self.config.rms_norm_eps
+        p = self._pass(b, kv, M, mode, num_seqs, max_q_len, attn_splits)
         last_token = self.states.last_token if self.states is not None else None
-        ops.embed_design(self.embed_design, b.ids, b.positions, row_seq, cu_q, b.state_rows, last_token, b.residual,
+        ops.embed_design(self.embed_design, b.ids, b.positions, p.row_seq, p.cu_q, b.state_rows, last_token, b.residual,
                          b.xnorm, M, num_seqs, eps)
-        for li, L in enumerate(self.layers):
-            s = L.spec
-            inp, in_planes, n_in = b.in_views[s.in_width], b.in_plane_views[s.in_width], 0
-            if planes_ok:
-                n_in = ops.linear_partial(L.w_in, b.xnorm, M, in_planes)
-            else:
-                ops.linear(L.w_in, b.xnorm, M, inp)
-            out = b.out_views[s.heads * s.vdim]
-            if isinstance(s, HeadsSpec):
-                view = self._heads_view(kv, L)
-                ops.heads_prep(inp, in_planes, n_in, view, b.slots, L, s, eps, M)
-                rows, seqs = short if ops.heads_expands(s, self.act_dtype) else (M, num_seqs)
-                if rows:
-                    ops.heads_attn(inp, view, b.block_tables, row_seq, b.positions, out, rows, s, b.attn_scratch,
-                                   attn_splits)
-                if seqs < num_seqs:
-                    ops.heads_attn_chunks(inp, view, b.block_tables, b.cu_q, b.q_pos0, b.positions, seqs, num_seqs,
-                                          max_q_len, out, s)
-            else:
-                n_gate = 0
-                if not n_in:
-                    n_gate = ops.linear_partial(L.w_if, b.xnorm, M, b.gate_planes)
-                ops.memory_prep(inp, in_planes, n_in, b.gate_planes, n_gate, b.gates, L, s, M)
-                rows, seqs = short if ops.memory_expands(s, self.act_dtype) else (M, num_seqs)
-                states = self.states.rows
-                if seqs:
-                    ops.memory_tokens(inp, b.gates, states, L.state_at, b.state_rows, cu_q, L, out, seqs, M, s, eps)
-                if seqs < num_seqs:
-                    ops.memory_chunks(inp, b.gates, states, L.state_at, b.state_rows, b.cu_q, L, out, seqs, num_seqs, rows,
-                                      M, s, eps, b.memory_ws)
-            planes = ops.linear_partial(L.o, out, M, partials)
-            last = li + 1 == len(self.layers)
-            ops.post_norm(b.residual, partials, planes, None, L.norm1, self.norm if last and L.ff is None else None,
+        for run in self.runs:
+            L, last = run.layer, run is self.runs[-1]
+            planes = self._mix(b, p, run)
+            ops.post_norm(b.residual, p.partials, planes, None, L.norm1, self.norm if last and L.ff is None else None,
                           b.xnorm, M, eps)
-            if L.ff is None:
-                continue
-            slots = None
-            if L.moe is not None:
-                slots, planes = ops.moe(L, b.xnorm, M, b.moe_ws), 0
-            else:
-                act = b.act_views[L.ff.ff]
-                ops.linear_act(L.up_w, b.xnorm, M, act, L.ff.activation)
-                planes = ops.linear_partial(L.down_w, act, M, partials)
-            ops.post_norm(b.residual, partials, planes, slots, L.norm2, self.norm if last else None, b.xnorm, M, eps)
+            if L.ff is not None:
+                planes, slots = self._feed(b, p, L)
+                ops.post_norm(b.residual, p.partials, planes, slots, L.norm2, self.norm if last else None, b.xnorm, M, eps)
         if n_logit_rows:
-            torch.index_select(b.xnorm, 0, b.logit_rows[:n_logit_rows], out=b.xsel[:n_logit_rows])
-            ops.linear_f32(self.lm_head, b.xsel, n_logit_rows, b.logits)
+            self._logits(b, n_logit_rows)

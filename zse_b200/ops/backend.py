@@ -67,8 +67,13 @@ class TorchOps:
         pass
 
     # ---- ops ------------------------------------------------------------------------------------------
-    def linear(self, w: LinearWeight, x, M, out, x_cap=None, gather=None):
-        if out.dtype != torch.float16:
+    def linear(self, w: LinearWeight, x, M, out, x_cap=None, gather=None, side=None):
+        """``side``: (first column, fp32 buffer): columns from there on go to the buffer [M, N - first] instead."""
+        if side is not None:
+            y = x[:M].float() @ w.data.T
+            out[:M, : side[0]] = y[:, : side[0]]
+            side[1].view(-1)[: M * (w.N - side[0])].view(M, -1).copy_(y[:, side[0]:])
+        elif out.dtype != torch.float16:
             out[:M, : w.N] = x[:M].float() @ w.data.T
         else:
             out[:M, : w.N] = ref.linear(x[:M], w.data, w.bias)
@@ -83,8 +88,11 @@ class TorchOps:
         partials.view(-1)[: M * w.N].view(M, w.N).copy_(x[:M].float() @ w.data.T)
         return 1
 
-    def embedding(self, table, ids, out, M, scale=1.0):
+    def embedding(self, table, ids, out, M, scale=1.0, copy=None):
+        """out (fp32) = scaled rows of the table; ``copy``: a second place for them, in the activations' type."""
         out[:M] = table[ids[:M].long()].float() * scale
+        if copy is not None:
+            copy[:M] = out[:M]
 
     def add_rmsnorm(self, residual, partials, n_partials, add_f16, weight, out, M, eps):
         H = residual.shape[1]
@@ -139,14 +147,19 @@ class TorchOps:
         """out [M, N] fp32, one plane."""
         out[:M, : w.N] = x[:M].float() @ w.data.T
 
-    def add_norm(self, residual, partials, n_partials, slots, weight, out, M, eps):
-        """residual += the planes' sum + the sum over a row's ``slots`` [M, n, H]; out = RMSNorm(residual) * weight."""
+    def add_norm(self, residual, partials, n_partials, slots, weight, out, M, eps, scale=None, offset=0.0, replace=False):
+        """residual += scale * (the planes' sum + the sum over a row's ``slots`` [M, n, H]), or the sum alone with
+        ``replace``; out = RMSNorm(residual) * (weight + offset), or the residual itself without a weight."""
         H = residual.shape[1]
+        y = torch.zeros(M, H, device=residual.device)
         if n_partials:
-            residual[:M] += partials.view(-1)[: n_partials * M * H].view(n_partials, M, H).sum(0)
+            y += partials.view(-1)[: n_partials * M * H].view(n_partials, M, H).sum(0)
         if slots is not None:
-            residual[:M] += slots[:M].float().sum(1)
-        out[:M] = ref.rmsnorm_f32(residual[:M], weight, eps)
+            y += slots[:M].float().sum(1)
+        if scale is not None:
+            y *= scale.float()
+        residual[:M] = y if replace else residual[:M] + y
+        out[:M] = residual[:M] if weight is None else ref.rmsnorm_f32(residual[:M], weight, eps, offset)
 
     def latent_prep(self, inp, planes, n_planes, rows, positions, slots, freqs, norm_w, spec, eps, M):
         if n_planes:
@@ -202,7 +215,7 @@ class TorchOps:
             y = t @ up.T
             if score is not None and m.weigh == "input":
                 y = score[:, None] * y
-            return (ref.clamped_glu(y[:, :ff], y[:, ff:], limit) if m.gated else ref.gelu_exact(y)).to(x.dtype).float()
+            return (ref.glu(m.activation, y[:, :ff], y[:, ff:], limit) if m.gated else ref.gelu_exact(y)).to(x.dtype).float()
 
         up, down = L.up.view(m.experts, -1, H), L.down.view(m.experts, H, m.ff)
         for e in torch.unique(ids).tolist():
@@ -259,15 +272,33 @@ class TorchOps:
         """out = activation(x W^T) in the activations' type."""
         out[:M, : w.N] = {"relu2": ref.relu2}[activation](x[:M].float() @ w.data.T)
 
+    def glu_linear(self, gate: torch.Tensor, up: torch.Tensor, dtype) -> LinearWeight:
+        """The two up products of a gated dense feed-forward as one weight for ``linear_glu``."""
+        return self.dense_linear(self.dense(torch.cat([gate, up]), dtype))
+
+    def linear_glu(self, w: LinearWeight, x, M, out, activation: str, tmp=None):
+        """out [M, ff] = glu(x W_gate^T, x W_up^T) in the activations' type; ``tmp``: room for both products."""
+        y, ff = x[:M].float() @ w.data.T, out.shape[1]
+        out[:M] = ref.glu(activation, y[:, :ff], y[:, ff:])
+
+    def glu_expands(self, ff: int, H: int, dtype) -> bool:
+        """Whether ``linear_glu`` needs its ``tmp``."""
+        return False
+
     def heads_expands(self, spec, dtype) -> bool:
         """Whether long chunks of such a layer take ``heads_attn_chunks``."""
         return True
 
-    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M):
+    def rotation(self, dims: int, base: float):
+        """Frequencies of the pairs (2i, 2i + 1), base^(-2i / dims) per position, in this back end's form."""
+        return base ** (-torch.arange(0, dims, 2, dtype=torch.float64, device=self.device) / dims) if dims else None
+
+    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M, positions=None):
         if n_planes:
             ld = inp.shape[1]
             inp[:M] = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
-        ref.heads_prep(inp[:M], kv.k if kv else None, kv.v if kv else None, slots[:M], spec, L.q_norm, L.k_norm, eps)
+        ref.heads_prep(inp[:M], kv.k if kv else None, kv.v if kv else None, slots[:M], spec, L.q_norm, L.k_norm, eps,
+                       None if positions is None else positions[:M].long(), L.bias, L.freqs)
 
     def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits):
         """Rows [0, M) against the cached keys and values; row t belongs to sequence ``row_seq[t]`` (None: t)."""
@@ -286,7 +317,7 @@ class TorchOps:
         y = ref.heads_attn(inp[a:e, : H * spec.dim].reshape(e - a, H, spec.dim), positions[a:e].long(), kv.k, kv.v, table,
                            spec)
         if spec.gated:
-            y = y * torch.sigmoid(inp[a:e, spec.gate_col: spec.gate_col + H].float())[:, :, None]
+            y = y * torch.sigmoid(inp[a:e, spec.gate_col: spec.gate_col + spec.gate_width].float()).view(e - a, H, -1)
         out[a:e, :w] = y.reshape(e - a, w)
 
     def memory_expands(self, spec, dtype) -> bool:
@@ -329,6 +360,59 @@ class TorchOps:
                 states[write, at: at + spec.state_floats] = row
             y = ref.rmsnorm_f32(y, L.head_norm.view(H, vd), eps).reshape(e - a, H * vd)
             out[a:e, : H * vd] = y * torch.sigmoid(x[:, spec.gate_col: spec.gate_col + H * vd])
+
+    # ---- state space (Mamba-2) --------------------------------------------------------------------------------------------
+    def state_space_expands(self, spec, dtype) -> bool:
+        """Whether long chunks of such a layer take ``state_space_chunks``."""
+        return False
+
+    def state_space_prep(self, inp, planes, n_planes, side, xbc, dt, states, at, state_rows, row_seq, cu_q, L, spec, M, S):
+        """Sums the split-K planes of the input projection [z | x | B | C | step sizes], passes x, B and C through the
+        convolution and silu into ``xbc`` and takes softplus of the biased step sizes, ``dt`` [M, heads].  Without planes
+        ``inp`` is complete; ``side``: the step sizes before bias and softplus in fp32 (None: those of ``inp``)."""
+        if n_planes:
+            ld = inp.shape[1]
+            full = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
+            inp[:M] = full
+        else:
+            full = inp[:M].float()
+        H, w = spec.heads, spec.conv_width
+        z = full[:, spec.dt_col: spec.dt_col + H]
+        if not n_planes and side is not None:
+            z = side.view(-1)[: M * (spec.in_width - spec.dt_col)].view(M, -1)[:, :H]
+        dt.view(-1)[: M * H].view(M, H).copy_(torch.nn.functional.softplus(z + L.dt_bias, threshold=40))
+        tail = slice(at + spec.conv_at, at + spec.conv_at + (spec.conv - 1) * w)
+        for s in range(S):
+            a, e = (s, s + 1) if cu_q is None else (int(cu_q[s]), int(cu_q[s + 1]))
+            read, write = int(state_rows[0, s]), int(state_rows[1, s])
+            before = states[read, tail].view(spec.conv - 1, w) if read >= 0 else torch.zeros(spec.conv - 1, w,
+                                                                                             device=inp.device)
+            y, last = ref.conv_tokens(full[a:e, spec.x_col: spec.dt_col], before, L.conv_w, L.conv_b)
+            xbc[a:e] = y
+            if write >= 0:
+                states[write, tail] = last.reshape(-1)
+
+    def state_space_tokens(self, inp, xbc, dt, states, at, state_rows, cu_q, L, out, S, M, spec):
+        """Sequences [0, S), token by token: memory, read-out, and the gate silu(z).  ``states``: the state pool's rows,
+        ``at``: where the layer's part of a row begins; ``cu_q``: first row of every sequence (None: a row each)."""
+        H, v, G, n = spec.heads, spec.vdim, spec.groups, spec.state
+        d = dt.view(-1)[: M * H].view(M, H)
+        for s in range(S):
+            a, e = (s, s + 1) if cu_q is None else (int(cu_q[s]), int(cu_q[s + 1]))
+            read, write = int(state_rows[0, s]), int(state_rows[1, s])
+            mem = states[read, at: at + H * n * v].clone() if read >= 0 else torch.zeros(H * n * v, device=inp.device)
+            x = xbc[a:e].float()
+            y = ref.state_space_tokens(x[:, : H * v].view(-1, H, v), x[:, spec.b_at: spec.b_at + G * n].view(-1, G, n),
+                                       x[:, spec.c_at: spec.c_at + G * n].view(-1, G, n), d[a:e], L.neg_a, L.D,
+                                       mem.view(H, n, v))
+            if write >= 0:
+                states[write, at: at + H * n * v] = mem
+            out[a:e, : H * v] = y.reshape(e - a, H * v) * torch.nn.functional.silu(inp[a:e, : H * v].float())
+
+    def group_norm(self, x, weight, parts: int, M, eps):
+        """Rows of ``x`` normed in place in ``parts`` equal parts, times ``weight``."""
+        y = x[:M].float().view(M, parts, -1)
+        x[:M] = ref.rmsnorm_f32(y, None, eps).view(M, -1) * weight.float()
 
     def logits_finish(self, logits, M, scale, cap):
         """logits <- cap * tanh(scale * logits / cap) in place (cap 0: only scaled)."""

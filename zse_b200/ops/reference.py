@@ -322,16 +322,10 @@ def gelu_exact(x: torch.Tensor) -> torch.Tensor:
     return 0.5 * x * (1.0 + torch.erf(x * math.sqrt(0.5)))
 
 
-def route_top(logits: torch.Tensor, top: int):
-    """(expert ids [T, top], their sigmoid scores): largest scores first, the lower id on a tie."""
-    s = torch.sigmoid(logits.float())
-    w, e = torch.sort(s, dim=-1, descending=True, stable=True)
-    return e[:, :top], w[:, :top]
-
-
-def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
-    """x / sqrt(mean(x^2) + eps) * w, fp32 in and out."""
-    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+def rmsnorm_f32(x: torch.Tensor, w: Optional[torch.Tensor], eps: float, offset: float = 0.0) -> torch.Tensor:
+    """x / sqrt(mean(x^2) + eps) * (w + offset), fp32 in and out; without ``w`` the factor is 1."""
+    y = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+    return y if w is None else y * (w.float() + offset)
 
 
 # ---- embedding with what a design adds to it ------------------------------------------------------------------------
@@ -354,16 +348,24 @@ def sinusoid(positions: torch.Tensor, width: int, base: float) -> torch.Tensor:
 
 
 # ---- attention over heads whose keys and values have their own widths ------------------------------------------------
-def heads_prep(inp: torch.Tensor, k_cache, v_cache, slots, spec, q_norm, k_norm, eps: float) -> None:
-    """Second half of the fused input projection [q | k | v | gate]: query and key norm over a head's dimensions, keys and
-    values into the cache (``k_cache`` [blocks, kv_heads, block_size, dim..]); queries are normed in place."""
+def heads_prep(inp: torch.Tensor, k_cache, v_cache, slots, spec, q_norm, k_norm, eps: float, positions=None, bias=None,
+               freqs=None) -> None:
+    """Second half of the fused input projection [q | k | v | gate]: bias, rotation, query and key norm over a head's
+    dimensions, temperature of the queries, keys and values into the cache (``k_cache`` [blocks, kv_heads, block_size,
+    dim..]); queries are finished in place.  ``freqs``: radians per position of every pair that rotates."""
     T, H, G, d, vd = inp.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim
-    inp[:, : H * d] = rmsnorm_f32(inp[:, : H * d].float().view(T, H, d), q_norm, eps).view(T, -1).to(inp.dtype)
+    full = inp.float() if bias is None else inp.float() + bias.float()
+    turn = (lambda x: rotate_pairs(x.double(), positions.double(), freqs).float()) if spec.rot_dims else lambda x: x
+    q = rmsnorm_f32(turn(full[:, : H * d].reshape(T, H, d)), q_norm, eps)
+    if spec.temp_coef:
+        q = q * query_temperature(positions, spec.temp_coef, spec.temp_every)[:, None, None]
+    inp[:, : H * d] = q.view(T, -1).to(inp.dtype)
     if not spec.own_kv:
         return
     bs = k_cache.shape[2]
-    k = rmsnorm_f32(inp[:, spec.k_col: spec.k_col + G * d].float().reshape(T, G, d), k_norm, eps)
-    v = inp[:, spec.v_col: spec.v_col + G * vd].reshape(T, G, vd)
+    raw = full[:, spec.k_col: spec.k_col + G * d].reshape(T, G, d)
+    k = rmsnorm_f32(turn(raw), k_norm, eps)
+    v = (raw if spec.k_as_v else full[:, spec.v_col: spec.v_col + G * vd].reshape(T, G, vd)).to(v_cache.dtype)
     ok = slots >= 0
     s = slots[ok]
     k_cache[s // bs, :, s % bs, :d] = k[ok].to(k_cache.dtype)
@@ -375,12 +377,21 @@ def heads_attn(q: torch.Tensor, positions, k_cache, v_cache, table, spec) -> tor
     bs, rep = k_cache.shape[2], spec.heads // spec.kv_heads
     first = torch.tensor([spec.first_seen(int(p)) for p in positions], device=q.device)
     pos = torch.arange(int(first.min()), int(positions.max()) + 1, device=q.device)
+    if spec.keep_first:
+        pos = torch.cat([torch.arange(min(spec.keep_first, int(first.min())), device=q.device), pos])
     blk = table[pos // bs].long()
     k = k_cache[blk.clamp_min(0), :, pos % bs, : spec.dim].float().repeat_interleave(rep, 1)
     v = v_cache[blk.clamp_min(0), :, pos % bs, : spec.vdim].float().repeat_interleave(rep, 1)
-    see = (pos[None] <= positions[:, None]) & (pos[None] >= first[:, None]) & (blk >= 0)[None]
+    see = (pos[None] <= positions[:, None]) & ((pos[None] >= first[:, None]) | (pos[None] < spec.keep_first)) & (blk >= 0)[None]
     s = torch.einsum("thd,nhd->htn", q.float(), k) * spec.scale
+    if spec.softcap:
+        s = spec.softcap * torch.tanh(s / spec.softcap)
     return torch.einsum("htn,nhv->thv", torch.softmax(s.masked_fill(~see, float("-inf")), -1).nan_to_num(0.0), v)
+
+
+def query_temperature(positions: torch.Tensor, coef: float, every: int) -> torch.Tensor:
+    """Factor of the queries at ``positions``, fp32."""
+    return 1.0 + coef * torch.log((torch.div(positions + 1, every, rounding_mode="floor") + 1).float())
 
 
 # ---- matrix memory (mLSTM) --------------------------------------------------------------------------------------------
@@ -406,24 +417,62 @@ def memory_tokens(q, k, v, log_i, log_f, S, n, m):
     return out
 
 
+# ---- state space (Mamba-2) ---------------------------------------------------------------------------------------------
+def conv_tokens(x: torch.Tensor, before: torch.Tensor, w: torch.Tensor, bias: torch.Tensor):
+    """Causal convolution per channel and silu of one sequence's rows ``x`` [T, C] after its inputs ``before`` [taps - 1, C];
+    ``w`` [taps, C] with the row's own tap last.  Returns the result and the last taps - 1 inputs."""
+    taps, T = w.shape[0], x.shape[0]
+    full = torch.cat([before, x])
+    y = bias + sum(w[j] * full[j: j + T] for j in range(taps))
+    return torch.nn.functional.silu(y), full[T:]
+
+
+def state_space_tokens(x, B, C, dt, neg_a, D, S):
+    """Tokens of one sequence through one layer's memory.  x [T, H, v], B and C [T, G, n], dt [T, H], neg_a [H] = -exp(A_log);
+    S [H, n, v] is updated in place.  Returns the read-outs [T, H, v]."""
+    H, G = x.shape[1], B.shape[1]
+    out = torch.empty_like(x)
+    for t in range(x.shape[0]):
+        b, c = (z[t].repeat_interleave(H // G, 0) for z in (B, C))
+        S.mul_(torch.exp(neg_a * dt[t])[:, None, None]).add_((dt[t][:, None] * b)[:, :, None] * x[t][:, None, :])
+        out[t] = torch.einsum("hnv,hn->hv", S, c) + D[:, None] * x[t]
+    return out
+
+
 # ---- feed-forwards ----------------------------------------------------------------------------------------------------
 def relu2(x: torch.Tensor) -> torch.Tensor:
     return torch.relu(x).square()
 
 
-def clamped_glu(g: torch.Tensor, u: torch.Tensor, limit: float) -> torch.Tensor:
-    """g sigmoid(1.702 g) (u + 1) with g clamped from above and u from both sides."""
-    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
-    return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+def gelu_tanh(x: torch.Tensor) -> torch.Tensor:
+    return 0.5 * x * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (x + 0.044715 * x ** 3)))
+
+
+def glu(kind: str, g: torch.Tensor, u: torch.Tensor, limit: float = 0.0) -> torch.Tensor:
+    """Gated activations: "silu_glu" silu(g) u, "gelu_tanh_glu" gelu(g) u, "clamped_glu" g sigmoid(1.702 g) (u + 1) with g
+    clamped from above and u from both sides."""
+    if kind == "clamped_glu":
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+    return {"silu_glu": torch.nn.functional.silu, "gelu_tanh_glu": gelu_tanh}[kind](g) * u
+
+
+def best_groups(scores: torch.Tensor, groups: int, keep: int) -> torch.Tensor:
+    """[T, experts] bool: experts of the ``keep`` groups whose two largest scores have the largest sum (the lower group on a
+    tie)."""
+    per = scores.view(scores.shape[0], groups, -1)
+    total = torch.topk(per, min(2, per.shape[-1]), dim=-1).values.sum(-1)
+    best = torch.sort(total, dim=-1, descending=True, stable=True).indices[:, :keep]
+    return torch.zeros_like(total, dtype=torch.bool).scatter_(1, best, True)[:, :, None].expand_as(per).reshape(scores.shape)
 
 
 def route(logits: torch.Tensor, moe):
     """(expert ids [T, top], their weights): largest scores first, the lower id on a tie."""
-    if moe.score == "sigmoid":
-        e, w = route_top(logits, moe.top)
-    else:
-        w, e = torch.sort(torch.softmax(logits.float(), -1), dim=-1, descending=True, stable=True)
-        e, w = e[:, : moe.top], w[:, : moe.top]
+    s = torch.sigmoid(logits.float()) if moe.score == "sigmoid" else torch.softmax(logits.float(), -1)
+    if moe.keep_groups < moe.groups:
+        s = s.masked_fill(~best_groups(s, moe.groups, moe.keep_groups), -1.0)
+    w, e = torch.sort(s, dim=-1, descending=True, stable=True)
+    e, w = e[:, : moe.top], w[:, : moe.top]
     if moe.normalise:
         w = w / (w.sum(-1, keepdim=True) + 1e-20)
     return e, w * moe.scale
