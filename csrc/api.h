@@ -50,6 +50,12 @@ int zse_gemm_f16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, c
                  int N, int K, int ldo, int epilogue, int k_split, void* status, void* stream);
 int zse_gemm_f16_splits(int M, int N, int K, int k_split);
 // the same kernel on bfloat16 weights and activations (epilogue 0: bfloat16 store, 2: fp32 planes)
+// gated activation of two up products (tiles of 64 gate rows and their 64 up rows): out [M, cols]; kinds as in zse_glu
+int zse_gemm_bf16_glu(const void* w, const void* x, int x_rows_cap, void* out, int M, int N, int K, int ldo, int cols,
+                      int kind, void* status, void* stream);
+// store in bfloat16, columns from side_col on in fp32 to side [M, N - side_col] instead
+int zse_gemm_bf16_side(const void* w, const void* x, int x_rows_cap, void* out, int M, int N, int K, int ldo, void* side,
+                       int side_col, void* status, void* stream);
 int zse_gemm_bf16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, void* out, int M, int N, int K, int ldo,
                   int epilogue, int k_split, void* status, void* stream);
 
@@ -72,18 +78,21 @@ typedef struct ZseTileGemm {
   const int32_t* n_tiles;
 } ZseTileGemm;
 int zse_gemm_tile(int dtype, const ZseTileGemm* a, int batch, int max_tiles, void* stream);
-// in [rows, 2 * ff] (gate, up) -> out [rows, ff] = g sigmoid(1.702 g) (u + 1), g clamped from above and u from both sides
-int zse_clamped_glu(int dtype, const void* in, void* out, int rows, int ff, float limit, void* stream);
+// in [rows, 2 * ff] (gate, up) -> out [rows, ff]; kind 0: g sigmoid(1.702 g) (u + 1), g clamped from above and u from both
+// sides; 1: silu(g) u; 2: gelu(g) u with the tanh form of gelu
+int zse_glu(int dtype, const void* in, void* out, int rows, int ff, int kind, float limit, void* stream);
 
 int zse_apply_repetition_penalty_f32(void* logits, int ld, const void* rows_i32, const void* tokens_i32,
                                      const void* counts_i32, int n, const void* penalty_f32, int V, void* stream);
 
 // ---- rows.cu ------------------------------------------------------------------------------------------------
 int zse_embedding_typed(int dtype, const void* table, const void* ids, void* out_f32, int M, int H, int vocab,
-                        float scale, void* status, void* stream);
-// residual += planes [n_planes][M][H] + slots [M][n_slots][H]; out = RMSNorm(residual) * weight
+                        float scale, void* copy, int ld_copy, void* status, void* stream);
+// y = planes [n_planes][M][H] + slots [M][n_slots][H], times scale [H] (null: 1); residual += y, or = y with replace;
+// out [M, ldo] = RMSNorm(residual) * (weight + offset), or the residual itself without a weight
 int zse_add_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes, const void* slots,
-                 int n_slots, const void* weight, void* out, int M, int H, float eps, void* stream);
+                 int n_slots, const void* scale, int replace, const void* weight, float offset, void* out, int ldo, int M,
+                 int H, float eps, void* stream);
 // y = planes + slots; residual += RMSNorm(y) * weight; out = residual, or (next not null) RMSNorm(residual) * next
 int zse_post_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes, const void* slots,
                   int n_slots, const void* weight, const void* next, void* out, int M, int H, float eps, void* stream);
@@ -146,6 +155,7 @@ typedef struct ZseRouter {
   int32_t softmax;            // scores: 0 sigmoid, 1 softmax over the experts
   int32_t normalise;          // weights: the chosen scores divided by their sum
   float scale;                // ... times this
+  int32_t groups, keep;       // equal groups of neighbouring experts; experts come from the `keep` best of them
 } ZseRouter;
 int zse_moe_route(int dtype, const ZseRouter* r, int M, int tile_rows, const void* x, int H, int out_per_token, void* counts,
                   void* slot_expert, void* slot_rank, void* slot_score, void* first_row, void* tiles, void* n_tiles,
@@ -158,8 +168,9 @@ typedef struct ZseMoeGemm {
   const void *row_score, *out_rows, *tiles, *n_tiles;
   const void* shared_score;   // per token, or null
   int32_t routed_n, routed_k, routed_ldo, shared_n, shared_k, shared_ldo, shared_mul, shared_add, shared_x_rows;
-  int32_t routed_cols, shared_cols;     // clamped_glu: output columns (weight rows: tiles of 64 gate rows and 64 up rows)
+  int32_t routed_cols, shared_cols;     // gated: output columns (weight rows: tiles of 64 gate rows and 64 up rows)
   float routed_limit, shared_limit;
+  int32_t glu;                // which gated activation, see zse_glu
 } ZseMoeGemm;
 int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int tile_rows, int max_tiles, int epilogue,
                  void* status, void* stream);
@@ -173,14 +184,26 @@ typedef struct ZseHeads {
   int32_t heads, kv_heads, dim, vdim, chunk, window;
   float scale;
   int32_t num_blocks;           // blocks in the pool
+  int32_t keep_first;           // first positions that are seen whatever the window
+  float softcap;                // > 0: scores become softcap * tanh(score / softcap)
+  int32_t gate_each;            // a gate per dimension of a head's result, not per head
 } ZseHeads;
 // 1 when the tensor-core kernels take this shape (bfloat16)
 int zse_heads_mma_ok(int dim, int vdim, int block_size);
-// columns of a projected row: q from 0, k from k_col, v from v_col, gate from gate_col (gate_w of them); own_kv 0: no keys
-// and values of its own
+// columns of a projected row: q from 0, k from k_col, v from v_col (k_col: the values are the keys as projected), gate from
+// gate_col (gate_w of them); own_kv 0: no keys and values of its own
+typedef struct ZseHeadsPrep {
+  const void *q_norm, *k_norm;  // weights of the norms over a head's dimensions, null: 1
+  const void* bias;             // of the columns before gate_col, null: none
+  const void* turns;            // pairs that rotate: [rot_dims / 2] high and low parts of the turns per position
+  const void* positions;
+  int32_t k_col, v_col, gate_col, gate_w, own_kv, rot_dims;
+  float temp_coef;              // queries are multiplied by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)
+  int32_t temp_every;
+  float eps;
+} ZseHeadsPrep;
 int zse_heads_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, int M, const ZseHeads* h,
-                   const void* slots, const void* q_norm, const void* k_norm, int k_col, int v_col, int gate_col,
-                   int gate_w, int own_kv, float eps, void* stream);
+                   const void* slots, const ZseHeadsPrep* p, void* stream);
 // rows [0, M) one by one; gate: first element of the gates (row stride ld), or null
 int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads* h, const void* row_seq, const void* positions,
                    void* out, int ldo, const void* gate, void* scratch, int M, int num_splits, int tensor_cores,
@@ -212,6 +235,34 @@ int zse_memory_tokens(int dtype, const void* inp, int ld, const void* gates, con
 // sequences [first, last) chunkwise (bfloat16): read-outs to o [M, heads * vdim] fp32, then head norm and output gate
 int zse_memory_chunks(const void* inp, int ld, const void* gates, const ZseMemory* m, const void* cu_q, int first, int last,
                       void* o, int M, int first_row_of_first, void* out, int ldo, void* stream);
+
+// ---- state_space.cu -----------------------------------------------------------------------------------------
+typedef struct ZseSpace {
+  int32_t heads, vdim, state, groups, taps;
+  int32_t x_col;                // columns of a projected row: z from 0, the channels x, B, C from x_col, step sizes from dt_col
+  int32_t b_at, c_at, conv_width;   // the channels' layout, in a projected row from x_col on and in the convolution's output
+  int32_t dt_col;
+  void* states;                 // state rows, row_floats apart; this layer's part: S at 0, the convolution's inputs at conv_at
+  int64_t row_floats;
+  int32_t conv_at;
+  const void* state_rows;       // [2][state_ld]: rows that sequences read and write (-1: none)
+  int32_t state_ld;
+  const void *conv_w, *conv_b;  // fp32 [taps][conv_width] (a row's own tap last), [conv_width]
+  const void *dt_bias, *neg_a, *skip;   // fp32 [heads]
+} ZseSpace;
+int zse_space_chunk_ok(int state, int vdim);
+// planes: of the input projection (0: inp is complete; side [M][side_ld]: its step sizes in fp32, or null); xbc
+// [M][conv_width], dt fp32 [M][heads]; row_seq, cu_q null: every row is a sequence of its own
+int zse_space_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, const void* side, int side_ld,
+                   const ZseSpace* m, const void* row_seq, const void* cu_q, void* xbc, void* dt, int M, void* stream);
+// sequences [0, S), token by token: update, read-out, gate silu(z); cu_q null: a row each
+int zse_space_tokens(int dtype, const void* inp, int ld, const void* xbc, const void* dt, const ZseSpace* m,
+                     const void* cu_q, int S, void* out, int ldo, void* stream);
+// sequences [first, last) chunkwise (bfloat16)
+int zse_space_chunks(const void* inp, int ld, const void* xbc, const void* dt, const ZseSpace* m, const void* cu_q, int first,
+                     int last, void* out, int ldo, void* stream);
+// rows [M][ld] in place: `parts` parts of `width` columns, each divided by its root mean square, times weight
+int zse_group_norm(int dtype, void* x, int ld, int M, int parts, int width, const void* weight, float eps, void* stream);
 
 // ---- repack.cu ----------------------------------------------------------------------------------------------
 // Row-major INT4 [N, K/2] + scales/zeros [N, K/128] -> tiled chunks.  interleave_rows > 0 builds a fused gate/up

@@ -37,14 +37,14 @@ __device__ __forceinline__ void epilogue(const GemmArgs& a, uint32_t tmem_acc, i
   constexpr int kColsPerHalf = NT >= 32 ? NT / 2 : NT;
   // A warp with nothing to do (no columns, or an aborted main loop) still meets its partner at the pair barrier.
   if ((NT < 32 && ch != 0) || !valid) {
-    if (EPI == kEpiSwiGLU) asm volatile("bar.sync %0, 64;" ::"r"(1 + ((q & 1) + 2 * ch)) : "memory");
+    if (EPI == kEpiSwiGLU || EPI == kEpiGlu) asm volatile("bar.sync %0, 64;" ::"r"(1 + ((q & 1) + 2 * ch)) : "memory");
     return;
   }
   const int col0 = ch * kColsPerHalf;
   const int n_tile = blockIdx.x, t0 = blockIdx.y * NT;
   const uint32_t taddr = tmem_acc + (uint32_t(q * 32) << 16) + col0;
 
-  if (EPI == kEpiSwiGLU) {
+  if (EPI == kEpiSwiGLU || EPI == kEpiGlu) {
     // up rows (q = 2, 3) park their values in shared memory; gate rows (q = 0, 1) combine.
     float* park = stage_smem + ((q & 1) + 2 * ch) * (32 * kColsPerHalf);
     const int bar_id = 1 + ((q & 1) + 2 * ch);
@@ -70,10 +70,13 @@ __device__ __forceinline__ void epilogue(const GemmArgs& a, uint32_t tmem_acc, i
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           const int t = t0 + col0 + c + i;
-          if (t < a.M && n_out < a.N / 2) {
+          if (t < a.M && n_out < (EPI == kEpiGlu ? a.cols : a.N / 2)) {
             const float g = __uint_as_float(r[i]);
             const float u = park[(c + i) * 32 + lane];
-            out[size_t(t) * a.ldo + n_out] = __float2half_rn(clamp_f16(silu_f(g) * u));
+            if (EPI == kEpiGlu)
+              reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n_out] = __float2bfloat16_rn(glu(a.glu, g, u, 0.f));
+            else
+              out[size_t(t) * a.ldo + n_out] = __float2half_rn(clamp_f16(silu_f(g) * u));
           }
         }
       }
@@ -97,6 +100,8 @@ __device__ __forceinline__ void epilogue(const GemmArgs& a, uint32_t tmem_acc, i
         const float v = __uint_as_float(r[i]);
         if (EPI == kEpiRelu2) {
           reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n] = __float2bfloat16_rn(relu2(v));
+        } else if (EPI == kEpiF16 && BF16 && a.side != nullptr && n >= a.side_col) {
+          a.side[size_t(t) * (a.N - a.side_col) + n - a.side_col] = v;
         } else if (EPI == kEpiF16 && BF16) {
           reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n] = __float2bfloat16_rn(v);
         } else if (EPI == kEpiF16) {
@@ -323,7 +328,8 @@ using namespace zse;
 
 template <bool BF16>
 static int gemm_16bit(const void* w, int w_rows_cap, const void* x, int x_rows_cap, const void* bias, void* out, int M,
-                      int N, int K, int ldo, int epilogue, int k_split, void* status, void* stream) {
+                      int N, int K, int ldo, int epilogue, int k_split, void* status, void* stream, int glu = 0,
+                      int cols = 0, float* side = nullptr, int side_col = 0) {
   if (M <= 0) return 0;
   if (K % 8 != 0 || N <= 0 || epilogue == kEpiSwiGLU) return ZSE_ERR_SHAPE;
   if (epilogue != kEpiPartialF32) k_split = 1;
@@ -336,12 +342,16 @@ static int gemm_16bit(const void* w, int w_rows_cap, const void* x, int x_rows_c
   if (int rc = get_tmap(w, uint64_t(max(w_rows_cap, N)), uint64_t(K), uint32_t(kTileN), &tw)) return rc;
   if (int rc = get_tmap(x, uint64_t(max(x_rows_cap, M)), uint64_t(K), uint32_t(nt), &tx)) return rc;
   GemmArgs a{nullptr, reinterpret_cast<const __half*>(bias), out, M, N, K, ldo, k_stages, spp,
-             reinterpret_cast<Status*>(status)};
+             reinterpret_cast<Status*>(status), glu, cols, side, side_col};
   dim3 grid((N + kTileN - 1) / kTileN, (M + nt - 1) / nt, k_split);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   int rc = ZSE_ERR_SHAPE;
   if (epilogue == kEpiF16) {
     ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiF16, BF16>(tw, tx, a, grid, st)))
+  } else if (epilogue == kEpiGlu) {
+    if (N % kTileN == 0 && cols <= N / 2) {
+      if constexpr (BF16) ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiGlu, BF16>(tw, tx, a, grid, st)))
+    }
   } else if (epilogue == kEpiRelu2) {
     if constexpr (BF16) ZSE_DISPATCH_NT(nt, rc = (launch_f16<NT, kEpiRelu2, BF16>(tw, tx, a, grid, st)))
   } else {
@@ -358,6 +368,19 @@ extern "C" int zse_gemm_f16(const void* w, int w_rows_cap, const void* x, int x_
 extern "C" int zse_gemm_bf16(const void* w, int w_rows_cap, const void* x, int x_rows_cap, void* out, int M, int N, int K,
                              int ldo, int epilogue, int k_split, void* status, void* stream) {
   return gemm_16bit<true>(w, w_rows_cap, x, x_rows_cap, nullptr, out, M, N, K, ldo, epilogue, k_split, status, stream);
+}
+
+// Two up products of a gated feed-forward (tiles of 64 gate rows and their 64 up rows) and the activation: out [M, cols].
+extern "C" int zse_gemm_bf16_glu(const void* w, const void* x, int x_rows_cap, void* out, int M, int N, int K, int ldo,
+                                 int cols, int kind, void* status, void* stream) {
+  return gemm_16bit<true>(w, N, x, x_rows_cap, nullptr, out, M, N, K, ldo, kEpiGlu, 1, status, stream, kind, cols);
+}
+
+// Store in bfloat16, columns from side_col on in fp32 to `side` [M, N - side_col] instead.
+extern "C" int zse_gemm_bf16_side(const void* w, const void* x, int x_rows_cap, void* out, int M, int N, int K, int ldo,
+                                  void* side, int side_col, void* status, void* stream) {
+  return gemm_16bit<true>(w, N, x, x_rows_cap, nullptr, out, M, N, K, ldo, kEpiF16, 1, status, stream, 0, 0,
+                          reinterpret_cast<float*>(side), side_col);
 }
 
 extern "C" int zse_gemm_f16_splits(int M, int N, int K, int k_split) {

@@ -13,7 +13,8 @@ constexpr int kW4ChunkBytes = 8704;  // 8192 nibble bytes + 512 bytes of {scale,
 constexpr int kGemmThreads = 320;    // fp16 kernel: warp 0 producer, warp 1 MMA issuer, warps 2..9 epilogue
 
 enum Epilogue : int { kEpiF16 = 0, kEpiSwiGLU = 1, kEpiPartialF32 = 2, kEpiPushF16 = 3, kEpiScatterF16 = 4,
-                     kEpiRelu2 = 5 /* bfloat16: store the square of relu */ };
+                     kEpiRelu2 = 5 /* bfloat16: store the square of relu */,
+                     kEpiGlu = 6 /* bfloat16: gated activation of 64 gate rows and their 64 up rows per tile */ };
 
 struct GemmArgs {
   const uint8_t* w;        // W4: tiled chunks [n_tiles][k_stages][8704]; F16: unused (tensor map)
@@ -24,6 +25,10 @@ struct GemmArgs {
   int k_stages;            // total K stages
   int stages_per_split;
   Status* status;
+  // bfloat16 only
+  int glu = 0, cols = 0;   // kEpiGlu: which activation (typed.cuh), output columns (N / 2, or less where N is padded)
+  float* side = nullptr;   // kEpiF16: columns from side_col on go here in fp32, [M, N - side_col]
+  int side_col = 0;
 };
 
 

@@ -1,6 +1,7 @@
 // Attention over heads whose keys and values have their own widths, grouped-query, with chunk or window masks.
 //
-//   heads_prep      second half of the fused input projection: split-K sum, query and key norm, cache write
+//   heads_prep      second half of the fused input projection: split-K sum, bias, rotation, query and key norm, temperature
+//                   of the queries, cache write
 //   heads_simple    a row's heads against the cached keys it sees; any shape, bfloat16 or float
 //   heads_rows      the same on bfloat16 tensor cores: the query heads of a kv head are one 16-row tile, each warp streams
 //                   its own tiles of 16 keys; keys may be split over CTAs (heads_combine merges)
@@ -9,7 +10,7 @@
 //
 // Cached tiles: [block][kv head][token][dim], then the same for values, dims padded to 8 (the padding is zero).  Scores and
 // softmax are fp32; softmax weights enter the product with the values as two bfloat16 terms (value and remainder).  A row
-// sees the positions from first_seen(position) to its own; block -1 of a table is a hole whose tokens do not exist.
+// sees the positions from first_seen(position) to its own, and the first `keep` ones; block -1 of a table is a hole whose tokens do not exist.
 #include "api.h"
 #include "heads.cuh"
 
@@ -20,28 +21,54 @@ namespace {
 struct HeadsPrepArgs {
   int ld, k_col, v_col, gate_col, gate_w, own_kv;
   float eps;
+  const float* turns;
+  const int* positions;
+  int rot_dims;
+  float temp_coef;
+  int temp_every;
 };
+constexpr int kPrepPairs = 128;                  // pairs whose sine and cosine a CTA keeps in shared memory
+
+// Sine and cosine of p * (turns per position, as two floats): the reduced angle keeps fp32 accuracy at any position.
+__device__ __forceinline__ float2 pair_turn(const float* turns, int i, float p) {
+  const float f = turns[2 * i], lo = turns[2 * i + 1];
+  const float hi = p * f;
+  const float r = (hi - rintf(hi)) + fmaf(p, lo, fmaf(p, f, -hi));
+  float2 cs;
+  sincospif(2.f * r, &cs.y, &cs.x);
+  return cs;
+}
 
 // A warp per (row, section): query heads, then key heads, value heads and - with planes - the gates.  grid (rows, sections / 8)
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_planes, int M, T* __restrict__ kc,
                   T* __restrict__ vc, Heads h, const long long* __restrict__ slots, const T* __restrict__ q_norm,
-                  const T* __restrict__ k_norm, HeadsPrepArgs a, int units) {
+                  const T* __restrict__ k_norm, const T* __restrict__ bias, HeadsPrepArgs a, int units) {
   constexpr int kKeep = VEC == 4 ? 2 : 8;        // accesses of a head that stay in registers (up to 256 dimensions)
+  __shared__ float2 turned[kPrepPairs];
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x, u = blockIdx.y * 8 + (threadIdx.x >> 5);
+  const float pos = a.positions != nullptr ? float(a.positions[t]) : 0.f;
+  if (a.rot_dims > 0) {
+    for (int i = threadIdx.x; i < min(kPrepPairs, a.rot_dims / 2); i += blockDim.x) turned[i] = pair_turn(a.turns, i, pos);
+    __syncthreads();
+  }
   if (u >= units) return;
   T* in = inp + size_t(t) * a.ld;
   const float* pl = planes + size_t(t) * a.ld;
   const size_t plane = size_t(M) * a.ld;
   auto value = [&](int c) {
-    F32Vec<VEC> v;
-    if (n_planes == 0) return load_vec<VEC>(in + c);
+    F32Vec<VEC> v{};
+    if (bias != nullptr) v = load_vec<VEC>(bias + c);
+    if (n_planes == 0) {
+      const F32Vec<VEC> x = load_vec<VEC>(in + c);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) v.v[e] = 0.f;
+      for (int e = 0; e < VEC; ++e) v.v[e] += x.v[e];
+      return v;
+    }
 #pragma unroll 4
     for (int p = 0; p < n_planes; ++p) {
       const F32Vec<VEC> x = load_vec<VEC>(pl + p * plane + c);
@@ -66,7 +93,7 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
     const int g = u - h.heads - (u >= h.heads + G ? G : 0), block = h.block_of(int(slot)), token = h.in_block(int(slot));
     if (u >= h.heads + G) {                      // values: copied
       dst = vc + h.at(block, g, token, h.vp);
-      const int c0 = a.v_col + g * h.vdim;
+      const int c0 = a.v_col + g * h.vdim;       // with v_col = k_col vdim is dim
       for (int i = lane * VEC; i < h.vdim; i += 32 * VEC) store_vec<VEC>(dst + i, value(c0 + i));
       return;
     }
@@ -75,13 +102,33 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
   const int c0 = u < h.heads ? u * h.dim : a.k_col + (u - h.heads) * h.dim;
   const T* w = u < h.heads ? q_norm : k_norm;
   if (u < h.heads) dst = in + c0;
+  auto turn = [&](int i, float& x, float& y) {   // the pair of dimensions i, i + 1
+    const float2 cs = i / 2 < kPrepPairs ? turned[i / 2] : pair_turn(a.turns, i / 2, pos);
+    const float u0 = x;
+    x = u0 * cs.x - y * cs.y;
+    y = y * cs.x + u0 * cs.y;
+  };
+  auto rotated = [&](int i) {                    // dimensions from i on
+    F32Vec<VEC> v = value(c0 + i);
+    if constexpr (VEC == 4) {
+      if (i < a.rot_dims) turn(i, v.v[0], v.v[1]);
+      if (i + 2 < a.rot_dims) turn(i + 2, v.v[2], v.v[3]);
+    } else if (i < a.rot_dims) {
+      float other = value(c0 + (i ^ 1)).v[0];
+      if (i & 1)
+        turn(i - 1, other, v.v[0]);
+      else
+        turn(i, v.v[0], other);
+    }
+    return v;
+  };
   F32Vec<VEC> x[kKeep];
   float ss = 0.f;
 #pragma unroll
   for (int j = 0; j < kKeep; ++j) {
     const int i = (lane + j * 32) * VEC;
     if (i < h.dim) {
-      x[j] = value(c0 + i);
+      x[j] = rotated(i);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) ss += x[j].v[e] * x[j].v[e];
     }
@@ -91,14 +138,19 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
 #pragma unroll
     for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
   }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / float(h.dim) + a.eps);
+  float inv = 1.f / sqrtf(warp_sum(ss) / float(h.dim) + a.eps);
+  if (u < h.heads && a.temp_coef != 0.f)
+    inv *= 1.f + a.temp_coef * logf(float((a.positions[t] + 1) / a.temp_every + 1));
   auto put = [&](int i, const F32Vec<VEC>& v) {
-    F32Vec<VEC> y = load_vec<VEC>(w + i);
+    F32Vec<VEC> y;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) y.v[e] = 1.f;
+    if (w != nullptr) y = load_vec<VEC>(w + i);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) y.v[e] *= v.v[e] * inv;
     store_vec<VEC>(dst + i, y);
   };
-  for (int i = (lane + kKeep * 32) * VEC; i < h.dim; i += 32 * VEC) put(i, value(c0 + i));
+  for (int i = (lane + kKeep * 32) * VEC; i < h.dim; i += 32 * VEC) put(i, rotated(i));
 #pragma unroll
   for (int j = 0; j < kKeep; ++j) {
     const int i = (lane + j * 32) * VEC;
@@ -128,7 +180,9 @@ heads_simple_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ kc,
   const int seq = row_seq != nullptr ? row_seq[t] : t, pos = positions[t];
   const int* table = h.tables + size_t(seq) * h.max_blocks;
   float m = -INFINITY, l = 0.f;
-  for (int j = h.first_seen(pos) + warp; j <= pos; j += 4) {
+  const int lo = h.first_seen(pos), kept = min(h.keep, lo);
+  for (int n = warp; n < kept + pos + 1 - lo; n += 4) {
+    const int j = n < kept ? n : lo + n - kept;
     const int block = table[h.block_of(j)];
     if (block < 0) continue;
     const T* k = kc + h.at(block, g, h.in_block(j), h.dp);
@@ -136,6 +190,7 @@ heads_simple_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ kc,
     float s = 0.f;
     for (int i = lane; i < h.dim; i += 32) s = fmaf(q[i], to_f32(k[i]), s);
     s = warp_sum(s) * h.scale;
+    if (h.cap > 0.f) s = h.cap * tanhf(s / h.cap);
     const float mn = fmaxf(m, s), corr = expf(m - mn), p = expf(s - mn);
     l = l * corr + p;
     m = mn;
@@ -153,12 +208,12 @@ heads_simple_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ kc,
     f[w] = ml[w] == -INFINITY ? 0.f : expf(ml[w] - most);
     L += ml[4 + w] * f[w];
   }
-  float inv = L > 0.f ? 1.f / L : 0.f;
-  if (gate != nullptr) inv *= sigmoid_exact(to_f32(gate[size_t(t) * ld + head]));
+  const float inv = L > 0.f ? 1.f / L : 0.f;
   for (int i = threadIdx.x; i < h.vdim; i += blockDim.x) {
     float y = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) y += sm[h.dim + w * h.vdim + i] * f[w];
+    if (gate != nullptr) y *= sigmoid_exact(to_f32(gate[size_t(t) * ld + h.gate_at(head, i)]));
     out[size_t(t) * ldo + size_t(head) * h.vdim + i] = from_f32<T>(y * inv);
   }
 }
@@ -174,7 +229,7 @@ inline size_t rows_smem(int dim, int vdim) {
   return ring > merge ? ring : merge;
 }
 
-template <int DKS, int DVT>            // steps of 16 key dimensions, blocks of 8 value dimensions (even)
+template <int DKS, int DVT, bool CAP>  // steps of 16 key dimensions, blocks of 8 value dimensions (even)
 __global__ void __launch_bounds__(kRowWarps * 32)
 heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ kc, const bf16* __restrict__ vc, Heads h,
                   const int* __restrict__ row_seq, const int* __restrict__ positions, bf16* __restrict__ out, int ldo,
@@ -189,9 +244,16 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
   const int seq = row_seq != nullptr ? row_seq[t] : t, pos = positions[t];
   const int* table = h.tables + size_t(seq) * h.max_blocks;
   const int lo = h.first_seen(pos);
-  const int tile0 = lo / kRowKeys, tiles = pos / kRowKeys + 1 - tile0;
+  const int tile0 = lo / kRowKeys;
+  const int kept = min(tile0, (h.keep + kRowKeys - 1) / kRowKeys);  // tiles of kept tokens before the first one of the window
+  const int tiles = kept + pos / kRowKeys + 1 - tile0;
   const int per_split = (tiles + num_splits - 1) / num_splits;
-  const int tb = tile0 + split * per_split, te = min(tile0 + tiles, tb + per_split);
+  const int tb = split * per_split, te = min(tiles, tb + per_split);
+  // first token of the i-th tile of this warp
+  auto token_of = [&](int i) {
+    const int n = tb + warp + i * kRowWarps;
+    return (n < kept ? n : tile0 + n - kept) * kRowKeys;
+  };
   const int mine = te > tb + warp ? (te - tb - warp + kRowWarps - 1) / kRowWarps : 0;
   const int kp = pitch_of(h.dim), vp = pitch_of(h.vdim), ks = (h.dim + 15) / 16;
   const int kch = h.dp / 8, vch = h.vp / 8;
@@ -233,8 +295,7 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
   }
   auto issue = [&](int i) {                      // i-th tile of this warp; always commits a group
     if (i < mine) {
-      const int tok = (tb + warp + i * kRowWarps) * kRowKeys;
-      const int block = table[h.block_of(tok)];
+      const int tok = token_of(i), block = table[h.block_of(tok)];
       if (block >= 0) {
         const bf16* ks_ = kc + h.at(block, kvh, h.in_block(tok), h.dp);
         const bf16* vs_ = vc + h.at(block, kvh, h.in_block(tok), h.vp);
@@ -261,7 +322,7 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
     cpa_wait<kRowStages - 2>();
     __syncwarp();
     issue(i + kRowStages - 1);
-    const int tok = (tb + warp + i * kRowWarps) * kRowKeys;
+    const int tok = token_of(i);
     if (table[h.block_of(tok)] < 0) continue;
     const uint32_t kb = smem_u32(ring + (i % kRowStages) * kRowKeys * (kp + vp)), vb = kb + kRowKeys * kp;
     float s[2][4] = {};
@@ -280,7 +341,7 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int p = tok + j * 8 + (lane & 3) * 2 + (e & 1);
-        s[j][e] = p >= lo && p <= pos ? s[j][e] * scale_log2 : -INFINITY;
+        s[j][e] = h.sees(p, pos, lo) ? (CAP ? h.capped(s[j][e] * h.scale) * kLog2E : s[j][e] * scale_log2) : -INFINITY;
         x[e >> 1] = fmaxf(x[e >> 1], s[j][e]);
       }
     float base[2], corr[2];
@@ -369,7 +430,7 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
     const int head = head0 + g;
     if (num_splits == 1) {
       float inv = L > 0.f ? 1.f / L : 0.f;
-      if (gate != nullptr) inv *= sigmoid_exact(to_f32(gate[size_t(t) * ld + head]));
+      if (gate != nullptr) inv *= sigmoid_exact(to_f32(gate[size_t(t) * ld + h.gate_at(head, d)]));
       out[size_t(t) * ldo + size_t(head) * h.vdim + d] = from_f32<bf16>(acc * inv);
     } else {
       float* dst = scratch + (size_t(t * h.heads + head) * num_splits + split) * (h.vdim + 2);
@@ -385,10 +446,10 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
 // grid (heads, rows)
 __global__ void __launch_bounds__(128)
 heads_combine_kernel(const float* __restrict__ scratch, bf16* __restrict__ out, int ldo, const bf16* __restrict__ gate, int ld,
-                     int heads, int vdim, int num_splits) {
+                     Heads h, int num_splits) {
   pdl_launch_dependents();
   pdl_wait();
-  const int head = blockIdx.x, t = blockIdx.y;
+  const int head = blockIdx.x, t = blockIdx.y, heads = h.heads, vdim = h.vdim;
   const float* src = scratch + size_t(t * heads + head) * num_splits * (vdim + 2);
   float most = -INFINITY, L = 0.f;
   for (int s = 0; s < num_splits; ++s) most = fmaxf(most, src[s * (vdim + 2) + vdim]);
@@ -396,14 +457,14 @@ heads_combine_kernel(const float* __restrict__ scratch, bf16* __restrict__ out, 
     const float ms = src[s * (vdim + 2) + vdim];
     L += src[s * (vdim + 2) + vdim + 1] * (ms == -INFINITY ? 0.f : ex2(ms - most));
   }
-  float inv = L > 0.f ? 1.f / L : 0.f;
-  if (gate != nullptr) inv *= sigmoid_exact(to_f32(gate[size_t(t) * ld + head]));
+  const float inv = L > 0.f ? 1.f / L : 0.f;
   for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < num_splits; ++s) {
       const float ms = src[s * (vdim + 2) + vdim];
       acc += src[s * (vdim + 2) + d] * (ms == -INFINITY ? 0.f : ex2(ms - most));
     }
+    if (gate != nullptr) acc *= sigmoid_exact(to_f32(gate[size_t(t) * ld + h.gate_at(head, d)]));
     out[size_t(t) * ldo + size_t(head) * vdim + d] = from_f32<bf16>(acc * inv);
   }
 }
@@ -415,7 +476,7 @@ inline size_t chunk_smem(int dim, int vdim) {
 }
 
 // CTA = (64 queries of a sequence, head), 4 warps of 16 queries; key tiles of 64 (aligned to 64) through a two-stage ring.
-template <int DVT>
+template <int DVT, bool CAP>
 __global__ void __launch_bounds__(128)
 heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ kc, const bf16* __restrict__ vc, Heads h,
                    const int* __restrict__ cu_q, const int* __restrict__ q_pos0, int first, bf16* __restrict__ out, int ldo,
@@ -438,7 +499,10 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
   const int p_first = q_pos0[s] + q0, p_last = q_pos0[s] + min(q_len, q0 + kChunkQ) - 1;
   const int see_all = h.first_seen(p_last);                        // from here on every query sees what is before it
   const int k_begin = h.first_seen(p_first) / kChunkKeys * kChunkKeys, k_end = p_last + 1;
-  const int count = (k_end - k_begin + kChunkKeys - 1) / kChunkKeys;
+  // tiles of kept tokens, then those from k_begin on
+  const int kept = min(k_begin / kChunkKeys, (h.keep + kChunkKeys - 1) / kChunkKeys);
+  const int count = kept + (k_end - k_begin + kChunkKeys - 1) / kChunkKeys;
+  auto key_of = [&](int i) { return i < kept ? i * kChunkKeys : k_begin + (i - kept) * kChunkKeys; };
 
   for (int i = threadIdx.x; i < kChunkQ * ksteps * 2; i += 128) {
     const int r = i / (ksteps * 2), c = i % (ksteps * 2);
@@ -454,7 +518,7 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
   bool whole[2] = {true, true};                  // this thread's key of the stage exists
   auto issue = [&](int i) {
     if (i < count) {
-      const int st = i & 1, key0 = k_begin + i * kChunkKeys;
+      const int st = i & 1, key0 = key_of(i);
       uint8_t *kd = sk + st * kChunkKeys * kp, *vd = sv + st * kChunkKeys * vp;
       if (threadIdx.x < kChunkKeys) {
         const int p = key0 + threadIdx.x;
@@ -488,7 +552,7 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
   const int pr0 = p_first + warp * 16 + rq;                        // positions of this thread's two query rows
   const int lo[2] = {h.first_seen(pr0), h.first_seen(pr0 + 8)};
   const uint32_t q_addr = smem_u32(sq) + (warp * 16 + (lane & 15)) * kp + (lane >> 4) * 16;
-  const float scale_log2 = h.scale * kLog2E;
+  const float scale_log2 = CAP ? kLog2E : h.scale * kLog2E;
 
   issue(0);
   for (int i = 0; i < count; ++i) {
@@ -511,9 +575,15 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
         mma_bf16(sc[n + 1], a, b[2], b[3]);
       }
     }
-    const int key0 = k_begin + i * kChunkKeys;
+    const int key0 = key_of(i);
     float x[2] = {-INFINITY, -INFINITY};
-    if (all_there && key0 + kChunkKeys - 1 <= p_first && key0 >= see_all) {
+    if constexpr (CAP) {
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[n][e] = h.capped(sc[n][e] * h.scale);
+    }
+    if (all_there && key0 + kChunkKeys - 1 <= p_first && (key0 >= see_all || key0 + kChunkKeys <= h.keep)) {
 #pragma unroll
       for (int n = 0; n < 8; ++n)                // every query sees every key
 #pragma unroll
@@ -527,7 +597,7 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int c = n * 8 + cq + (e & 1), p = key0 + c;
-          const bool see = p <= pr0 + (e >> 1) * 8 && p >= lo[e >> 1] && valid[(i & 1) * kChunkKeys + c] != 0;
+          const bool see = h.sees(p, pr0 + (e >> 1) * 8, lo[e >> 1]) && valid[(i & 1) * kChunkKeys + c] != 0;
           sc[n][e] = see ? sc[n][e] * scale_log2 : -INFINITY;
           x[e >> 1] = fmaxf(x[e >> 1], sc[n][e]);
         }
@@ -585,14 +655,17 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
     const int r = q0 + warp * 16 + rq + half * 8;
     if (r >= q_len) continue;
     const size_t t = size_t(q_begin + r);
-    float inv = L > 0.f ? 1.f / L : 0.f;
-    if (gate != nullptr) inv *= sigmoid_exact(to_f32(gate[t * ld + head]));
+    const float inv = L > 0.f ? 1.f / L : 0.f;
 #pragma unroll
     for (int n = 0; n < DVT; ++n) {
       const int c = n * 8 + cq;
-      if (c < h.vdim)
-        *reinterpret_cast<uint32_t*>(out + t * ldo + size_t(head) * h.vdim + c) =
-            pack_bf16(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
+      if (c >= h.vdim) continue;
+      float y0 = o[n][half * 2] * inv, y1 = o[n][half * 2 + 1] * inv;
+      if (gate != nullptr) {
+        y0 *= sigmoid_exact(to_f32(gate[t * ld + h.gate_at(head, c)]));
+        y1 *= sigmoid_exact(to_f32(gate[t * ld + h.gate_at(head, c + 1)]));
+      }
+      *reinterpret_cast<uint32_t*>(out + t * ldo + size_t(head) * h.vdim + c) = pack_bf16(y0, y1);
     }
   }
 }
@@ -614,7 +687,7 @@ Heads heads_of(const ZseHeads* h) {
     if (h->block_size == 1 << i) shift = i;
   return Heads{(long long)(h->block_stride), h->block_size, h->dim_pad, h->vdim_pad, h->max_blocks, shift,
                reinterpret_cast<const int*>(h->tables), h->heads, h->kv_heads, h->dim, h->vdim, h->chunk, h->window,
-               h->scale};
+               h->scale, h->keep_first, h->softcap, h->gate_each};
 }
 
 struct RowsCall {
@@ -629,10 +702,10 @@ struct RowsCall {
   cudaStream_t st;
 };
 
-template <int DKS, int DVT>
+template <int DKS, int DVT, bool CAP>
 int launch_rows(const ZseHeads* z, const RowsCall& c) {
   static size_t done[kMaxDevices] = {};
-  auto kern = heads_rows_kernel<DKS, DVT>;
+  auto kern = heads_rows_kernel<DKS, DVT, CAP>;
   const Heads h = heads_of(z);
   const size_t smem = rows_smem(h.dim, h.vdim);
   if (int r = raise_smem(kern, smem, done)) return r;
@@ -643,16 +716,24 @@ int launch_rows(const ZseHeads* z, const RowsCall& c) {
              ? 0
              : ZSE_ERR_LAUNCH;
 }
-template <int DKS>
+template <int DKS, bool CAP>
 int launch_rows_v(const ZseHeads* z, const RowsCall& c) {
-  return z->vdim <= 64 ? launch_rows<DKS, 8>(z, c) : z->vdim <= 128 ? launch_rows<DKS, 16>(z, c) : launch_rows<DKS, 32>(z, c);
+  return z->vdim <= 64    ? launch_rows<DKS, 8, CAP>(z, c)
+         : z->vdim <= 128 ? launch_rows<DKS, 16, CAP>(z, c)
+                          : launch_rows<DKS, 32, CAP>(z, c);
+}
+template <bool CAP>
+int launch_rows_k(const ZseHeads* z, const RowsCall& c) {
+  return z->dim <= 64    ? launch_rows_v<4, CAP>(z, c)
+         : z->dim <= 128 ? launch_rows_v<8, CAP>(z, c)
+                         : launch_rows_v<16, CAP>(z, c);
 }
 
-template <int DVT>
+template <int DVT, bool CAP>
 int launch_chunks(const ZseHeads* z, const void* inp, int ld, const void* cu_q, const void* q_pos0, int first, int last,
                   int max_q, void* out, int ldo, const void* gate, cudaStream_t st) {
   static size_t done[kMaxDevices] = {};
-  auto kern = heads_chunk_kernel<DVT>;
+  auto kern = heads_chunk_kernel<DVT, CAP>;
   const Heads h = heads_of(z);
   const size_t smem = chunk_smem(h.dim, h.vdim);
   if (int r = raise_smem(kern, smem, done)) return r;
@@ -667,13 +748,14 @@ int launch_chunks(const ZseHeads* z, const void* inp, int ld, const void* cu_q, 
 
 template <typename T, int VEC>
 cudaError_t launch_prep(void* inp, const void* planes, int n_planes, int M, const ZseHeads* z, const void* slots,
-                        const void* q_norm, const void* k_norm, const HeadsPrepArgs& a, cudaStream_t st) {
+                        const ZseHeadsPrep* p, const HeadsPrepArgs& a, cudaStream_t st) {
   const Heads h = heads_of(z);
   const int units = h.heads + 2 * (a.own_kv ? h.kv_heads : 0) + (n_planes > 0 && a.gate_w > 0 ? 1 : 0);
   return launch_pdl(heads_prep_kernel<T, VEC>, dim3(M, (units + 7) / 8), dim3(256), 0, st,
                     reinterpret_cast<T*>(inp), reinterpret_cast<const float*>(planes), n_planes, M,
                     reinterpret_cast<T*>(z->k), reinterpret_cast<T*>(z->v), h, reinterpret_cast<const long long*>(slots),
-                    reinterpret_cast<const T*>(q_norm), reinterpret_cast<const T*>(k_norm), a, units);
+                    reinterpret_cast<const T*>(p->q_norm), reinterpret_cast<const T*>(p->k_norm),
+                    reinterpret_cast<const T*>(p->bias), a, units);
 }
 
 }  // namespace
@@ -688,19 +770,24 @@ extern "C" int zse_heads_mma_ok(int dim, int vdim, int block_size) {
 }
 
 extern "C" int zse_heads_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, int M, const ZseHeads* h,
-                              const void* slots, const void* q_norm, const void* k_norm, int k_col, int v_col,
-                              int gate_col, int gate_w, int own_kv, float eps, void* stream) {
+                              const void* slots, const ZseHeadsPrep* p, void* stream) {
   if (M <= 0) return 0;
-  if (h->heads <= 0 || h->kv_heads <= 0 || h->heads % h->kv_heads) return ZSE_ERR_SHAPE;
-  const HeadsPrepArgs a{ld, k_col, v_col, gate_col, gate_w, own_kv, eps};
-  const bool vec = h->dim % 4 == 0 && h->vdim % 4 == 0 && ld % 4 == 0 && k_col % 4 == 0 && v_col % 4 == 0 &&
+  if (h->heads <= 0 || h->kv_heads <= 0 || h->heads % h->kv_heads || p->rot_dims % 2 || p->rot_dims > h->dim ||
+      (p->temp_coef != 0.f && p->temp_every <= 0) || (p->own_kv && p->v_col == p->k_col && h->vdim != h->dim) ||
+      ((p->rot_dims > 0 || p->temp_coef != 0.f) && p->positions == nullptr))
+    return ZSE_ERR_SHAPE;
+  const HeadsPrepArgs a{ld, p->k_col, p->v_col, p->gate_col, p->gate_w, p->own_kv, p->eps,
+                        reinterpret_cast<const float*>(p->turns), reinterpret_cast<const int*>(p->positions), p->rot_dims,
+                        p->temp_coef, p->temp_every};
+  const bool vec = h->dim % 4 == 0 && h->vdim % 4 == 0 && ld % 4 == 0 && p->k_col % 4 == 0 && p->v_col % 4 == 0 &&
                    h->block_stride % 4 == 0 &&
                    !((reinterpret_cast<uintptr_t>(inp) | reinterpret_cast<uintptr_t>(planes) |
                       reinterpret_cast<uintptr_t>(h->k) | reinterpret_cast<uintptr_t>(h->v) |
-                      reinterpret_cast<uintptr_t>(q_norm) | reinterpret_cast<uintptr_t>(k_norm)) & 15);
+                      reinterpret_cast<uintptr_t>(p->q_norm) | reinterpret_cast<uintptr_t>(p->k_norm) |
+                      reinterpret_cast<uintptr_t>(p->bias)) & 15);
   auto run = dtype == kBF16 ? (vec ? launch_prep<bf16, 4> : launch_prep<bf16, 1>)
                             : (vec ? launch_prep<float, 4> : launch_prep<float, 1>);
-  return run(inp, planes, n_planes, M, h, slots, q_norm, k_norm, a, ST(stream)) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+  return run(inp, planes, n_planes, M, h, slots, p, a, ST(stream)) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }
 
 extern "C" int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads* z, const void* row_seq,
@@ -731,10 +818,10 @@ extern "C" int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads
   const RowsCall c{reinterpret_cast<const bf16*>(inp), ld, reinterpret_cast<const int*>(row_seq),
                    reinterpret_cast<const int*>(positions), reinterpret_cast<bf16*>(out), ldo,
                    reinterpret_cast<const bf16*>(gate), reinterpret_cast<float*>(scratch), M, num_splits, ST(stream)};
-  int rc = z->dim <= 64 ? launch_rows_v<4>(z, c) : z->dim <= 128 ? launch_rows_v<8>(z, c) : launch_rows_v<16>(z, c);
+  int rc = z->softcap > 0.f ? launch_rows_k<true>(z, c) : launch_rows_k<false>(z, c);
   if (rc == 0 && num_splits > 1 &&
       launch_pdl(heads_combine_kernel, dim3(z->heads, M), dim3(128), 0, ST(stream), reinterpret_cast<const float*>(scratch),
-                 c.out, ldo, c.gate, ld, z->heads, z->vdim, num_splits) != cudaSuccess)
+                 c.out, ldo, c.gate, ld, heads_of(z), num_splits) != cudaSuccess)
     rc = ZSE_ERR_LAUNCH;
   return rc;
 }
@@ -752,6 +839,10 @@ extern "C" int zse_heads_attn_chunks(const void* inp, int ld, int rows, const Zs
                            reinterpret_cast<const int*>(cu_q), reinterpret_cast<const int*>(q_pos0), first, last, max_q,
                            reinterpret_cast<bf16*>(out), ldo, reinterpret_cast<const bf16*>(gate),
                            reinterpret_cast<Status*>(status), ST(stream));
-  auto run = z->vdim <= 64 ? launch_chunks<8> : z->vdim <= 128 ? launch_chunks<16> : launch_chunks<32>;
+  auto run = z->softcap > 0.f
+                 ? (z->vdim <= 64 ? launch_chunks<8, true> : z->vdim <= 128 ? launch_chunks<16, true> : launch_chunks<32, true>)
+                 : (z->vdim <= 64    ? launch_chunks<8, false>
+                    : z->vdim <= 128 ? launch_chunks<16, false>
+                                     : launch_chunks<32, false>);
   return run(z, inp, ld, cu_q, q_pos0, first, last, max_q, out, ldo, gate, ST(stream));
 }

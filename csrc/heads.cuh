@@ -11,6 +11,18 @@ struct Heads {
   const int* tables;
   int heads, kv_heads, dim, vdim, chunk, window;
   float scale;
+  int keep;                                      // first positions that are seen whatever the window
+  float cap;                                     // > 0: scores become cap * tanh(score / cap)
+  int gate_each;                                 // a gate per dimension of a head's result, not per head
+  // whether a row at `pos`, which sees from lo = first_seen(pos) on, sees position p
+  __device__ __forceinline__ bool sees(int p, int pos, int lo) const { return p <= pos && (p >= lo || p < keep); }
+  // cap * tanh(score / cap) of a scaled score; within 2^-22 of cap
+  __device__ __forceinline__ float capped(float s) const {
+    const float e = ex2(s * (2.f * kLog2E / cap));
+    return cap - __fdividef(2.f * cap, 1.f + e);
+  }
+  // place of the gate of a head's dimension d among a row's gates
+  __device__ __forceinline__ int gate_at(int head, int d) const { return gate_each ? head * vdim + d : head; }
   __device__ __forceinline__ int first_seen(int pos) const {
     return chunk > 0 ? pos / chunk * chunk : window > 0 ? max(0, pos + 1 - window) : 0;
   }

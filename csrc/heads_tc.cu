@@ -5,10 +5,11 @@
 // of attention_tc.cu (a loader warp, an MMA issuer, 128 softmax threads that own a row each, two CTAs per SM):
 //   S = Q K^T     both from shared memory (TMA boxes of 64 columns x 16, 32 or 64 tokens through the block table; columns past
 //                 a key's width are the tensor map's zero fill)
-//   softmax       row maximum, then exp2 of the scores; the reference maximum moves only when a row outgrew it by 2^8
+//   softmax       row maximum, then exp2 of the scores (soft-capped first, where a cap is set); the reference maximum moves only when a row outgrew it by 2^8
 //   O += P V      P from TMEM in TWO bfloat16 terms, the weight and what rounding took from it, 64 columns each: together they
 //                 take the place of the 128 columns of scores; V is an MN-major operand as it lies in the cache
-// Tiles start at a multiple of the box, at or before the first key that the tile's first query sees.
+// Tiles start at a multiple of the box, at or before the first key that the tile's first query sees; tiles of the tokens that
+// are always kept come before them.
 // Every wait is bounded; on a failure the loader waits for its copies and the CTA frees its TMEM and leaves.
 #include <cuda.h>
 
@@ -62,6 +63,7 @@ __device__ __forceinline__ uint64_t ht_desc_mn(uint32_t smem_addr) {
   return d;
 }
 
+template <bool CAP>
 __global__ void __launch_bounds__(kHtThreads, 2)
 heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                 const __grid_constant__ CUtensorMap map_v, const HtArgs a) {
@@ -81,7 +83,10 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
   const int p_first = a.q_pos0[seq] + qt * kHtRows, p_last = a.q_pos0[seq] + min(q_len, qt * kHtRows + kHtRows) - 1;
   const int br = a.box_rows;
   const int k_begin = a.h.first_seen(p_first) / br * br, k_end = p_last + 1;
-  const int n_tiles = (k_end - k_begin + kHtKeys - 1) / kHtKeys;
+  const int kept_end = min(k_begin, (a.h.keep + br - 1) / br * br);          // kept tokens before the others, whole boxes
+  const int kept = (kept_end + kHtKeys - 1) / kHtKeys, n_tiles = kept + (k_end - k_begin + kHtKeys - 1) / kHtKeys;
+  auto key_of = [&](int t) { return t < kept ? t * kHtKeys : k_begin + (t - kept) * kHtKeys; };
+  auto end_of = [&](int t) { return t < kept ? kept_end : k_end; };
   const int* table = a.h.tables + size_t(seq) * a.h.max_blocks;
 
   if (threadIdx.x == 0) {
@@ -124,14 +129,14 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
     const int n_groups = kHtKeys / br, g = lane >> 1, panel = lane & 1;
     const uint32_t box_bytes = uint32_t(br) * 128u;
     auto group_block = [&](int t) {              // block of group g of tile t; -1: a hole, or past the end
-      const int tok = k_begin + t * kHtKeys + g * br;
-      return (g < n_groups && t < n_tiles && tok < k_end) ? table[a.h.block_of(tok)] : -1;
+      const int tok = key_of(t) + g * br;
+      return (g < n_groups && t < n_tiles && tok < end_of(t)) ? table[a.h.block_of(tok)] : -1;
     };
     int next = group_block(0), issued_k = 0, issued_v = 0;
     uint32_t ph = 1;                             // "empty" barriers: the first wait passes
     for (int t = 0; t < n_tiles; ++t) {
       const int block = next;
-      const int tok = k_begin + t * kHtKeys + g * br;
+      const int tok = key_of(t) + g * br;
       const int y = kvh * a.h.block_size + a.h.in_block(tok);
       const bool load_k = block >= 0 && panel < a.k_panels, load_v = block >= 0 && panel < a.v_panels;
       const uint32_t n_k = __popc(__ballot_sync(0xffffffffu, load_k)), n_v = __popc(__ballot_sync(0xffffffffu, load_v));
@@ -200,23 +205,25 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
     const int limit = a.q_pos0[seq] + row, lo = a.h.first_seen(limit);
     const uint32_t lane_addr = uint32_t(warp * 32) << 16;
     const float scale_log2 = a.h.scale * kLog2E;
+    auto log2_score = [&](float s) { return CAP ? a.h.capped(s * a.h.scale) * kLog2E : s * scale_log2; };
     const int o_cols = (a.h.vdim + 15) / 16 * 16;
     float m_used = -INFINITY, l = 0.f;
     uint32_t ph = 0;
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t) {
-      const int k0 = k_begin + t * kHtKeys;
+      const int k0 = key_of(t), t_end = end_of(t);
       // which groups of 16 keys of the tile exist; looked up while S is still being computed
       const int g_tok = k0 + (lane & 7) * 16;
       const uint32_t groups =
-          __ballot_sync(0xffffffffu, g_tok < k_end && table[a.h.block_of(g_tok)] >= 0) & 0xFFu;
+          __ballot_sync(0xffffffffu, g_tok < t_end && table[a.h.block_of(g_tok)] >= 0) & 0xFFu;
       // one verdict per warp: the tcgen05.ld / st below are warp-wide
       if (!__all_sync(0xffffffffu, mbar_wait(&bars->s_full, ph, abort_flag, a.status, 98, t))) {
         ok = false;
         break;
       }
       tc_fence_after_sync();
-      const bool full = __all_sync(0xffffffffu, groups == 0xFFu && k0 >= lo && k0 + kHtKeys - 1 <= limit);
+      const bool full = __all_sync(0xffffffffu, groups == 0xFFu && (k0 >= lo || k0 + kHtKeys <= a.h.keep) &&
+                                                    k0 + kHtKeys - 1 <= limit);
       float mx = -INFINITY;
 #pragma unroll 1
       for (int c = 0; c < 4; ++c) {
@@ -236,12 +243,13 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int k = k0 + c * 32 + i;
-            const bool seen = ((groups >> (c * 2 + (i >> 4))) & 1u) && k <= limit && k >= lo;
-            mx = seen ? fmaxf(mx, __uint_as_float(v[i]) * scale_log2) : mx;
+            const bool seen = ((groups >> (c * 2 + (i >> 4))) & 1u) && a.h.sees(k, limit, lo);
+            mx = seen ? fmaxf(mx, __uint_as_float(v[i])) : mx;
           }
         }
       }
-      if (full) mx *= scale_log2;                // scale > 0: the maximum commutes with it
+      // scale > 0 and the cap's tanh is monotone: the maximum commutes with both
+      if (mx != -INFINITY) mx = log2_score(mx);
       // move the reference maximum only when some row of the warp needs it
       if (__any_sync(0xffffffffu, mx > m_used + 8.f)) {
         const float m_new = fmaxf(m_used, mx);
@@ -275,13 +283,19 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
             tc_wait_ld();
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-              float p0 = ex2(fmaf(__uint_as_float(v[2 * i]), scale_log2, -m_ref));
-              float p1 = ex2(fmaf(__uint_as_float(v[2 * i + 1]), scale_log2, -m_ref));
+              float p0, p1;
+              if constexpr (CAP) {
+                p0 = ex2(log2_score(__uint_as_float(v[2 * i])) - m_ref);
+                p1 = ex2(log2_score(__uint_as_float(v[2 * i + 1])) - m_ref);
+              } else {
+                p0 = ex2(fmaf(__uint_as_float(v[2 * i]), scale_log2, -m_ref));
+                p1 = ex2(fmaf(__uint_as_float(v[2 * i + 1]), scale_log2, -m_ref));
+              }
               if constexpr (!decltype(all)::value) {
                 const int k = k0 + c * 32 + b * 16 + 2 * i;
                 const bool there = (groups >> (c * 2 + b)) & 1u;
-                p0 = there && k <= limit && k >= lo ? p0 : 0.f;
-                p1 = there && k + 1 <= limit && k + 1 >= lo ? p1 : 0.f;
+                p0 = there && a.h.sees(k, limit, lo) ? p0 : 0.f;
+                p1 = there && a.h.sees(k + 1, limit, lo) ? p1 : 0.f;
               }
               s0 += p0;
               s1 += p1;
@@ -315,7 +329,8 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
       const bool live = row < q_len;
       const size_t t = size_t(q_begin + (live ? row : 0));
       float inv = l > 0.f ? 1.f / l : 0.f;
-      if (a.gate != nullptr) inv *= sigmoid_exact(to_f32(a.gate[t * a.ld + head]));
+      const bf16* gates = a.gate != nullptr && a.h.gate_each ? a.gate + t * a.ld + size_t(head) * a.h.vdim : nullptr;
+      if (a.gate != nullptr && gates == nullptr) inv *= sigmoid_exact(to_f32(a.gate[t * a.ld + head]));
       bf16* dst = a.out + t * a.ldo + size_t(head) * a.h.vdim;
 #pragma unroll 1
       for (int c = 0; c < o_cols; c += 16) {     // every lane takes part in the warp-wide loads
@@ -326,7 +341,16 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
         for (int b = 0; b < 2; ++b) {
           if (!live || c + b * 8 >= a.h.vdim) continue;
           uint4 w;
-          const uint32_t* x = o + b * 8;
+          uint32_t* x = o + b * 8;
+          if (gates != nullptr) {
+            const uint4 g = *reinterpret_cast<const uint4*>(gates + c + b * 8);
+            const uint32_t two[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              const float z = __uint_as_float(i & 1 ? two[i / 2] & 0xFFFF0000u : two[i / 2] << 16);
+              x[i] = __float_as_uint(__uint_as_float(x[i]) * sigmoid_exact(z));
+            }
+          }
           w.x = pack_bf16(__uint_as_float(x[0]) * inv, __uint_as_float(x[1]) * inv);
           w.y = pack_bf16(__uint_as_float(x[2]) * inv, __uint_as_float(x[3]) * inv);
           w.z = pack_bf16(__uint_as_float(x[4]) * inv, __uint_as_float(x[5]) * inv);
@@ -352,6 +376,7 @@ int launch_heads_tc(const bf16* inp, int ld, int rows, const void* k, const void
                     const int* cu_q, const int* q_pos0, int first, int last, int max_q, bf16* out, int ldo,
                     const bf16* gate, Status* status, cudaStream_t st) {
   if ((reinterpret_cast<uintptr_t>(out) & 15) != 0) return ZSE_ERR_ALIGN;
+  if (gate != nullptr && h.gate_each && (reinterpret_cast<uintptr_t>(gate) & 15) != 0) return ZSE_ERR_ALIGN;
   const int br = h.block_size % 64 == 0 ? 64 : h.block_size % 32 == 0 ? 32 : 16;
   CUtensorMap mq, mk, mv;
   if (int rc = get_tmap(inp, uint64_t(rows), uint64_t(ld), uint32_t(kHtRows), &mq)) return rc;
@@ -361,15 +386,16 @@ int launch_heads_tc(const bf16* inp, int ld, int rows, const void* k, const void
   if (int rc = get_tmap_rows3(v, num_blocks, per_block, h.vp, h.block_stride, br, 0, &mv)) return rc;
   const HtArgs a{h, cu_q, q_pos0, first, out, ldo, gate, ld, br, (h.dim + 63) / 64, (h.vdim + 63) / 64, status};
   const size_t smem = size_t(2 * a.k_panels + a.v_panels) * kHtPanel + 1024 + sizeof(HtBars);
-  static bool done[kMaxDevices] = {};
-  const int slot = current_device_slot();
-  if (!done[slot]) {
-    if (cudaFuncSetAttribute(heads_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+  static bool done[2][kMaxDevices] = {};
+  const int slot = current_device_slot(), cap = h.cap > 0.f;
+  auto kern = cap ? heads_tc_kernel<true> : heads_tc_kernel<false>;
+  if (!done[cap][slot]) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              int(6 * kHtPanel + 1024 + sizeof(HtBars))) != cudaSuccess)
       return ZSE_ERR_LAUNCH;
-    done[slot] = true;
+    done[cap][slot] = true;
   }
-  return launch_pdl(heads_tc_kernel, dim3((max_q + kHtRows - 1) / kHtRows, h.heads, last - first), dim3(kHtThreads), smem, st,
+  return launch_pdl(kern, dim3((max_q + kHtRows - 1) / kHtRows, h.heads, last - first), dim3(kHtThreads), smem, st,
                     mq, mk, mv, a) == cudaSuccess
              ? 0
              : ZSE_ERR_LAUNCH;

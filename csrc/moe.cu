@@ -1,7 +1,8 @@
 // Routed feed-forward: which tokens go to which expert, and the experts' products.
 //
 //   topk      scores of the router's fp32 logits (sigmoid, or softmax over the experts), the `top` largest per token (lower
-//             id first on a tie), their weights, and each (token, choice) slot's place within its expert
+//             id first on a tie) among the experts of the best groups, their weights, and each (token, choice) slot's place
+//             within its expert
 //   plan      one CTA: first row of every expert in the sorted order, table of token tiles for the grouped products
 //   permute   the tokens' rows, copied into sorted order, with the score and the slot of each sorted row
 //   products  grouped GEMM on tcgen05 (moe_gemm_kernel), the shared expert's dense product in the same launch
@@ -22,7 +23,7 @@ constexpr int kTopkWarps = 8;
 // Router rows are `cols` wide: column E, if there is one, is the shared expert's gate, whose sigmoid goes to shared_score.
 __global__ void __launch_bounds__(kTopkWarps * 32)
 moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, int cols, int top, int softmax, int normalise,
-                float scale, int* __restrict__ counts, int* __restrict__ slot_expert, int* __restrict__ slot_rank,
+                float scale, int groups, int keep, int* __restrict__ counts, int* __restrict__ slot_expert, int* __restrict__ slot_rank,
                 float* __restrict__ slot_score, float* __restrict__ shared_score) {
   extern __shared__ float scores[];
   pdl_launch_dependents();
@@ -30,8 +31,9 @@ moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, in
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kTopkWarps + warp;
   if (t >= M) return;
-  float* s = scores + warp * (E + top);
+  float* s = scores + warp * (E + top + groups);
   float* chosen = s + E;
+  float* group = chosen + top;
   auto logit = [&](int e) {
     float z = 0.f;
     for (int p = 0; p < n_planes; ++p) z += planes[(size_t(p) * M + t) * cols + e];
@@ -54,13 +56,13 @@ moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, in
     sum = warp_sum(sum);
     for (int e = lane; e < E; e += 32) s[e] /= sum;
   }
-  float total = 0.f;
-  for (int k = 0; k < top; ++k) {
-    float best = -2.f;
-    int at = 0x7fffffff;
-    for (int e = lane; e < E; e += 32)
-      if (s[e] > best) {
-        best = s[e];
+  // the largest of n values, the lowest index on a tie; every lane gets it
+  auto largest = [&](const float* v, int n, float& best, int& at) {
+    best = -2.f;
+    at = 0x7fffffff;
+    for (int e = lane; e < n; e += 32)
+      if (v[e] > best) {
+        best = v[e];
         at = e;
       }
 #pragma unroll
@@ -72,6 +74,37 @@ moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, in
         at = a2;
       }
     }
+  };
+  if (keep < groups) {                               // only experts of the best groups remain (scores are >= 0)
+    const int per = E / groups;
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      float a = 0.f, b = 0.f;                        // the two largest
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float x = s[e];
+        b = fmaxf(b, fminf(a, x));
+        a = fmaxf(a, x);
+      }
+      group[g] = a + b;
+    }
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {
+      float best;
+      int at;
+      largest(group, groups, best, at);
+      if (at >= groups) at = 0;
+      __syncwarp();
+      if (lane == (at & 31)) group[at] = -1.5f;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (group[e / per] != -1.5f) s[e] = -1.f;
+  }
+  float total = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best;
+    int at;
+    largest(s, E, best, at);
     if (at >= E) at = 0;                              // a row of NaN scores: still a valid expert
     if (lane == (at & 31)) s[at] = -1.f;              // the lane that owns this expert
     if (lane == 0) {
@@ -186,6 +219,7 @@ struct MoeGemmArgs {
   const int* n_tiles;
   int dense_tiles;          // token tiles of the shared expert (0: none)
   int M;                    // tokens
+  int glu;                  // kMoeGlu: which gated activation
   Status* status;
 };
 
@@ -205,7 +239,7 @@ struct MoeBars {
   int abort_flag;
 };
 
-// gelu(scale * acc) -> bf16; scale * acc -> OutT; clamped_glu -> bf16 (a tile of W: 64 gate rows, then their 64 up rows)
+// gelu(scale * acc) -> bf16; scale * acc -> OutT; glu -> bf16 (a tile of W: 64 gate rows, then their 64 up rows)
 enum MoeEpi { kMoeUp = 0, kMoeDown = 1, kMoeGlu = 2 };
 
 template <int NT, int EPI, typename OutT>
@@ -330,7 +364,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
               const int col = ch * kCols + c + i;
               if (col < tile.rows && n < p.cols)
                 reinterpret_cast<OutT*>(p.out)[size_t(tile.row0 + col) * p.ldo + n] =
-                    from_f32<OutT>(clamped_glu(__uint_as_float(r[i]), park[(c + i) * 32 + lane], p.limit));
+                    from_f32<OutT>(glu(a.glu, __uint_as_float(r[i]), park[(c + i) * 32 + lane], p.limit));
             }
           }
         }
@@ -390,12 +424,14 @@ extern "C" int zse_moe_route(int dtype, const ZseRouter* r, int M, int tile_rows
                              void* stream) {
   const int E = r->experts, top = r->top;
   if (M <= 0) return 0;
-  if (E <= 0 || top <= 0 || top > E || tile_rows <= 0 || E + top > 1536) return ZSE_ERR_SHAPE;
+  if (E <= 0 || top <= 0 || top > E || tile_rows <= 0 || E + top + r->groups > 1536) return ZSE_ERR_SHAPE;
+  if (r->groups <= 0 || E % r->groups || r->keep <= 0 || r->keep > r->groups || top > r->keep * (E / r->groups))
+    return ZSE_ERR_SHAPE;
   cudaStream_t st = ST(stream);
-  const size_t smem = size_t(kTopkWarps) * (E + top) * sizeof(float);
+  const size_t smem = size_t(kTopkWarps) * (E + top + r->groups) * sizeof(float);
   if (launch_pdl(moe_topk_kernel, dim3((M + kTopkWarps - 1) / kTopkWarps), dim3(kTopkWarps * 32), smem, st,
                  reinterpret_cast<const float*>(r->planes), r->n_planes, M, E, r->cols, top, r->softmax, r->normalise,
-                 r->scale, reinterpret_cast<int*>(counts), reinterpret_cast<int*>(slot_expert),
+                 r->scale, r->groups, r->keep, reinterpret_cast<int*>(counts), reinterpret_cast<int*>(slot_expert),
                  reinterpret_cast<int*>(slot_rank), reinterpret_cast<float*>(slot_score),
                  reinterpret_cast<float*>(shared_score)) != cudaSuccess)
     return ZSE_ERR_LAUNCH;
@@ -426,7 +462,7 @@ extern "C" int zse_moe_tile_rows(int M, int E, int top) {
   return want <= 16 ? 16 : want <= 32 ? 32 : want <= 64 ? 64 : want <= 160 ? 128 : 256;
 }
 
-// Up (epilogue 0: gelu(scale * acc) in bfloat16; 3: clamped_glu) or down (1: bfloat16, 2: fp32 result rows) products of all
+// Up (epilogue 0: gelu(scale * acc) in bfloat16; 3: gated) or down (1: bfloat16, 2: fp32 result rows) products of all
 // experts.
 extern "C" int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int tile_rows, int max_tiles, int epilogue,
                             void* status, void* stream) {
@@ -453,6 +489,7 @@ extern "C" int zse_moe_gemm(const ZseMoeGemm* g, int M, int E, int max_rows, int
   a.n_tiles = reinterpret_cast<const int*>(g->n_tiles);
   a.dense_tiles = shared ? (M + tile_rows - 1) / tile_rows : 0;
   a.M = M;
+  a.glu = g->glu;
   a.status = reinterpret_cast<Status*>(status);
   const int nmax = shared && g->shared_n > g->routed_n ? g->shared_n : g->routed_n;
   if (a.dense_tiles + max_tiles > 65535) return ZSE_ERR_LIMIT;

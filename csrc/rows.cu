@@ -10,7 +10,8 @@ namespace {
 
 template <typename T>
 __global__ void embedding_typed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                       float* __restrict__ out, int H, int vocab, float scale, Status* st) {
+                                       float* __restrict__ out, int H, int vocab, float scale, T* __restrict__ copy,
+                                       int ld_copy, Status* st) {
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x;
@@ -21,11 +22,16 @@ __global__ void embedding_typed_kernel(const T* __restrict__ table, const int* _
   }
   const T* src = table + size_t(id) * H;
   float* dst = out + size_t(row) * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = to_f32(src[i]) * scale;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float x = to_f32(src[i]) * scale;
+    dst[i] = x;
+    if (copy != nullptr) copy[size_t(row) * ld_copy + i] = from_f32<T>(x);
+  }
 }
 
-// residual += sum of fp32 planes [n_planes][M][H] + sum of the row's slots [M][n_slots][H];
-// out = RMSNorm(residual) * weight.  A row is split over the CTAs of a cluster (gridDim.x), each thread keeps its
+// y = sum of fp32 planes [n_planes][M][H] + sum of the row's slots [M][n_slots][H], times scale [H] if there is one;
+// residual += y, or residual = y (replace); out [M, ldo] = RMSNorm(residual) * (weight + offset), or the residual itself
+// without a weight.  A row is split over the CTAs of a cluster (gridDim.x), each thread keeps its
 // columns in registers between the sum and the norm; VEC consecutive columns per access (4 when H % 4 == 0).
 constexpr int kRowThreads = 256;
 constexpr int kRowRegs = 8;          // accesses per thread: H <= 8 * VEC * 256 * cluster
@@ -52,8 +58,8 @@ __device__ __forceinline__ float row_cluster_sum(float total, float* slot, int c
 template <typename T, typename S, int VEC>
 __global__ void __launch_bounds__(kRowThreads)
 add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, int n_planes,
-                const S* __restrict__ slots, int n_slots, const T* __restrict__ weight, T* __restrict__ out, int M,
-                int H, float eps) {
+                const S* __restrict__ slots, int n_slots, const T* __restrict__ scale, int replace,
+                const T* __restrict__ weight, float offset, T* __restrict__ out, int ldo, int M, int H, float eps) {
   __shared__ float red[32];
   __shared__ float cluster_ss;
   pdl_launch_dependents();
@@ -69,7 +75,11 @@ add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, 
     const int i = v0 + threadIdx.x + j * kRowThreads;
     if (i < v1) {
       const size_t at = base + size_t(i) * VEC;
-      x[j] = load_vec<VEC>(residual + at);
+      F32Vec<VEC> old{}, f;
+      if (!replace) old = load_vec<VEC>(residual + at);
+      if (scale != nullptr) f = load_vec<VEC>(scale + size_t(i) * VEC);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[j].v[e] = scale == nullptr ? old.v[e] : 0.f;
 #pragma unroll 4
       for (int p = 0; p < n_planes; ++p) {
         const F32Vec<VEC> y = load_vec<VEC>(planes + p * plane + at);
@@ -82,11 +92,17 @@ add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, 
 #pragma unroll
         for (int e = 0; e < VEC; ++e) x[j].v[e] += y.v[e];
       }
+      if (scale != nullptr) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[j].v[e] = fmaf(x[j].v[e], f.v[e], old.v[e]);
+      }
       if (n_planes + n_slots > 0) store_vec<VEC>(residual + at, x[j]);
+      if (weight == nullptr) store_vec<VEC>(out + size_t(row) * ldo + size_t(i) * VEC, x[j]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) ss += x[j].v[e] * x[j].v[e];
     }
   }
+  if (weight == nullptr) return;                           // the same for every CTA of the cluster
   ss = warp_sum(ss);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
   __syncthreads();
@@ -99,8 +115,8 @@ add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, 
     if (i < v1) {
       F32Vec<VEC> w = load_vec<VEC>(weight + size_t(i) * VEC);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) w.v[e] *= x[j].v[e] * inv;
-      store_vec<VEC>(out + base + size_t(i) * VEC, w);
+      for (int e = 0; e < VEC; ++e) w.v[e] = (w.v[e] + offset) * (x[j].v[e] * inv);
+      store_vec<VEC>(out + size_t(row) * ldo + size_t(i) * VEC, w);
     }
   }
 }
@@ -136,12 +152,14 @@ inline bool aligned16(std::initializer_list<const void*> ps) {
 }
 
 template <typename T, typename S>
-int launch_add_norm(void* residual, const void* planes, int n_planes, const void* slots, int n_slots,
-                    const void* weight, void* out, int M, int H, float eps, cudaStream_t st) {
-  return launch_rows(add_norm_kernel<T, S, 4>, add_norm_kernel<T, S, 1>, aligned16({residual, weight, out}), M, H, st,
+int launch_add_norm(void* residual, const void* planes, int n_planes, const void* slots, int n_slots, const void* scale,
+                    int replace, const void* weight, float offset, void* out, int ldo, int M, int H, float eps,
+                    cudaStream_t st) {
+  return launch_rows(add_norm_kernel<T, S, 4>, add_norm_kernel<T, S, 1>,
+                     aligned16({residual, weight, out, scale}) && ldo % 4 == 0, M, H, st,
                      reinterpret_cast<float*>(residual), reinterpret_cast<const float*>(planes), n_planes,
-                     reinterpret_cast<const S*>(slots), n_slots, reinterpret_cast<const T*>(weight),
-                     reinterpret_cast<T*>(out), M, H, eps);
+                     reinterpret_cast<const S*>(slots), n_slots, reinterpret_cast<const T*>(scale), replace,
+                     reinterpret_cast<const T*>(weight), offset, reinterpret_cast<T*>(out), ldo, M, H, eps);
 }
 
 // y = sum of fp32 planes + sum of the row's slots; residual += RMSNorm(y) * weight; out = residual, or (next != null)
@@ -401,29 +419,29 @@ using namespace zse;
 #define ST(s) reinterpret_cast<cudaStream_t>(s)
 
 extern "C" int zse_embedding_typed(int dtype, const void* table, const void* ids, void* out, int M, int H, int vocab,
-                                   float scale, void* status, void* stream) {
+                                   float scale, void* copy, int ld_copy, void* status, void* stream) {
   if (M <= 0) return 0;
   cudaError_t e;
   if (dtype == kBF16)
     e = launch_pdl(embedding_typed_kernel<bf16>, dim3(M), dim3(128), 0, ST(stream), reinterpret_cast<const bf16*>(table),
                    reinterpret_cast<const int*>(ids), reinterpret_cast<float*>(out), H, vocab, scale,
-                   reinterpret_cast<Status*>(status));
+                   reinterpret_cast<bf16*>(copy), ld_copy, reinterpret_cast<Status*>(status));
   else
     e = launch_pdl(embedding_typed_kernel<float>, dim3(M), dim3(128), 0, ST(stream),
                    reinterpret_cast<const float*>(table), reinterpret_cast<const int*>(ids),
-                   reinterpret_cast<float*>(out), H, vocab, scale, reinterpret_cast<Status*>(status));
+                   reinterpret_cast<float*>(out), H, vocab, scale, reinterpret_cast<float*>(copy), ld_copy,
+                   reinterpret_cast<Status*>(status));
   return e == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }
 
 extern "C" int zse_add_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes,
-                            const void* slots, int n_slots, const void* weight, void* out, int M, int H, float eps,
-                            void* stream) {
+                            const void* slots, int n_slots, const void* scale, int replace, const void* weight,
+                            float offset, void* out, int ldo, int M, int H, float eps, void* stream) {
   if (M <= 0) return 0;
-  if (dtype == kF32)
-    return launch_add_norm<float, float>(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps, ST(stream));
-  if (slot_dtype == kF32)
-    return launch_add_norm<bf16, float>(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps, ST(stream));
-  return launch_add_norm<bf16, bf16>(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps, ST(stream));
+  auto run = dtype == kF32        ? launch_add_norm<float, float>
+             : slot_dtype == kF32 ? launch_add_norm<bf16, float>
+                                  : launch_add_norm<bf16, bf16>;
+  return run(residual, planes, n_planes, slots, n_slots, scale, replace, weight, offset, out, ldo, M, H, eps, ST(stream));
 }
 
 extern "C" int zse_post_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes,

@@ -28,6 +28,15 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
   return g / (1.f + expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
 }
 
+__device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh(float z) {
+  return 0.5f * z * (1.f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z)));
+}
+// gated activations of two products: kinds 0 clamped_glu, 1 silu(g) u, 2 gelu_tanh(g) u
+__device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
+  return kind == 0 ? clamped_glu(g, u, limit) : (kind == 1 ? silu_exact(g) : gelu_tanh(g)) * u;
+}
+
 // 2^x on the special-function unit: softmax weights need no more than its fp32 accuracy, and no range handling around it
 __device__ __forceinline__ float ex2(float x) {
   float y;

@@ -20,6 +20,8 @@ from .hybrid import HybridLayer, HybridModel, HybridStepBuffers
 
 
 class LoopedModel(HybridModel):
+    kernel_group = "looped"
+
     # ---- loading --------------------------------------------------------------------------------------
     def _load(self, loader: ZSELoader, progress=None) -> None:
         c, ops = self.config, self.ops

@@ -14,6 +14,7 @@ from typing import Optional
 import numpy as np
 import torch
 
+from ..format.layer_specs import GLU
 from . import reference as ref
 
 EPI_F16, EPI_SWIGLU, EPI_PARTIAL, EPI_RELU2 = 0, 1, 2, 5
@@ -298,7 +299,8 @@ class TorchOps:
             ld = inp.shape[1]
             inp[:M] = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
         ref.heads_prep(inp[:M], kv.k if kv else None, kv.v if kv else None, slots[:M], spec, L.q_norm, L.k_norm, eps,
-                       None if positions is None else positions[:M].long(), L.bias, L.freqs)
+                       None if positions is None else positions[:M].long(), getattr(L, "bias", None),
+                       getattr(L, "freqs", None))
 
     def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits):
         """Rows [0, M) against the cached keys and values; row t belongs to sequence ``row_seq[t]`` (None: t)."""
@@ -634,7 +636,7 @@ class CudaOps(TorchOps):
         return LinearWeight("f16", w.shape[0], K, w, b, swiglu, w.numel() * 2)
 
     # ---- ops ------------------------------------------------------------------------------------------
-    def linear(self, w, x, M, out, x_cap=None, gather=None):
+    def linear(self, w, x, M, out, x_cap=None, gather=None, side=None):
         """``gather``: a tensor-parallel context whose gathered activation buffer ``x`` is - the GEMM then waits, tile
         by tile, for the rows to arrive from the ranks that own them (INT4 weights, more than 64 rows)."""
         cap = x.shape[0] if x_cap is None else x_cap
@@ -656,6 +658,8 @@ class CudaOps(TorchOps):
                                self.status.ptr)
         elif w.kind == "w4t":
             self.n.gemm_w4(w.data, x, cap, w.bias, out, M, w.N, w.K, out.stride(0), EPI_F16, 0, self.status.ptr)
+        elif side is not None and self.linear_has_side(w):
+            self.n.gemm_bf16_side(w.data, x, cap, out, M, w.N, w.K, out.stride(0), side[1], side[0], self.status.ptr)
         elif w.kind in ("bf16", "f32"):
             self._typed_linear(w, x, M, out, out.stride(0), EPI_F16, 1, cap)
         else:
@@ -742,15 +746,20 @@ class CudaOps(TorchOps):
                          self.n.TILE_STORE if epilogue == EPI_F16 else self.n.TILE_F32)
         return 1
 
+    @staticmethod
+    def linear_has_side(w) -> bool:
+        """Whether ``linear`` puts columns into its ``side`` (the general kernel leaves them among the others)."""
+        return w.kind == "bf16" and w.K % 8 == 0
+
     def dense(self, t: torch.Tensor, dtype) -> torch.Tensor:
         return t.to(self.device, dtype)
 
     def linear_f32(self, w, x, M, out):
         self._typed_linear(w, x, M, out, out.stride(0), EPI_PARTIAL, 1, x.shape[0])
 
-    def add_norm(self, residual, partials, n_partials, slots, weight, out, M, eps):
+    def add_norm(self, residual, partials, n_partials, slots, weight, out, M, eps, scale=None, offset=0.0, replace=False):
         self.n.add_norm(residual, partials, n_partials, slots, 0 if slots is None else slots.shape[1], weight, out, M,
-                        residual.shape[1], float(eps))
+                        residual.shape[1], float(eps), scale, offset, replace)
 
     def logits_finish(self, logits, M, scale, cap):
         self.n.logits_finish(logits, M, scale, cap)
@@ -803,9 +812,12 @@ class CudaOps(TorchOps):
 
     def moe_up(self, pairs, dtype, m=None):
         """Tensor-core form: tiles of 64 gate rows and their 64 up rows, the experts' rows padded to whole tiles."""
-        ff, H = pairs[0][0].shape
-        if not moe_tensor_cores(m, H, dtype):
+        if not moe_tensor_cores(m, pairs[0][0].shape[1], dtype):
             return super().moe_up(pairs, dtype, m)
+        return self._interleaved(pairs, dtype)
+
+    def _interleaved(self, pairs, dtype) -> torch.Tensor:
+        ff, H = pairs[0][0].shape
         n = (ff + 63) // 64
         out = torch.zeros(len(pairs), n, 2, 64, H, dtype=dtype, device=self.device)
         pad = torch.zeros(n * 64, H, dtype=dtype, device=self.device)
@@ -841,7 +853,7 @@ class CudaOps(TorchOps):
         def up(src, weights, act, ff, rows, limit, scale=None, **kw):
             if m.gated:
                 n.gemm_tile(dt, src, H, weights, (H, 1), ws.glu, 2 * ff, rows, 2 * ff, H, n.TILE_STORE, **kw)
-                n.clamped_glu(ws.glu, act, rows, ff, limit)
+                n.glu(ws.glu, act, rows, ff, GLU[m.activation], limit)
             else:
                 n.gemm_tile(dt, src, H, weights, (H, 1), act, ff, rows, ff, H, n.TILE_GELU, row_scale=scale, **kw)
 
@@ -855,7 +867,7 @@ class CudaOps(TorchOps):
         return y
 
     def moe_product_call(self, L, x, M, ws, epilogue: int):
-        """The tensor-core launch of one half of the experts (0: up + gelu, 3: gate and up + clamped glu; 1, 2: down to
+        """The tensor-core launch of one half of the experts (0: up + gelu, 3: gate and up + glu; 1, 2: down to
         bfloat16 / fp32 rows), over the tables that ``moe_route`` left in ``ws``."""
         n, m, H = self.n, L.moe, x.shape[1]
         tile = n.moe_tile_rows(M, m.experts, m.top)
@@ -866,7 +878,7 @@ class CudaOps(TorchOps):
             g = n.MoeGemm(L.up.data_ptr(), ws.xs.data_ptr(), ws.act.data_ptr(), _dp(L.shared_up), x.data_ptr(),
                           ws.act_shared.data_ptr(), score if m.weigh == "input" else None, None, ws.tiles.data_ptr(),
                           ws.n_tiles.data_ptr(), None, rows_of(m.ff), H, m.ff, rows_of(m.shared_ff), H, m.shared_ff, 1, 0,
-                          x.shape[0], m.ff, m.shared_ff, m.limit, m.shared_limit)
+                          x.shape[0], m.ff, m.shared_ff, m.limit, m.shared_limit, GLU.get(m.activation, 0))
             rows = ws.xs.numel() // H
         else:
             per = m.top + (m.shared_ff > 0)
@@ -874,7 +886,7 @@ class CudaOps(TorchOps):
                           ws.act_shared.data_ptr(), ws.y.data_ptr(), score if m.weigh == "output" else None,
                           ws.out_rows.data_ptr(), ws.tiles.data_ptr(), ws.n_tiles.data_ptr(),
                           ws.shared_score.data_ptr() if m.shared_gate else None, H, m.ff, H, H if m.shared_ff else 0,
-                          m.shared_ff, H, per, m.top, ws.act_shared.numel() // max(1, m.shared_ff), H, H, 0.0, 0.0)
+                          m.shared_ff, H, per, m.top, ws.act_shared.numel() // max(1, m.shared_ff), H, H, 0.0, 0.0, 0)
             rows = ws.act.numel() // m.ff
         return lambda: n.moe_gemm(g, M, m.experts, rows, tile, max_tiles, epilogue, self.status.ptr)
 
@@ -882,10 +894,7 @@ class CudaOps(TorchOps):
     def embed_design(self, E, ids, positions, row_seq, cu_q, state_rows, last_token, residual, out, M, S, eps):
         n, H = self.n, E.table.shape[1]
         if E.turns is None:              # turns per token as two floats: the angle of any position keeps fp32 accuracy
-            j = torch.arange(0, H, 2, dtype=torch.float64)
-            f = E.base ** (-j / H) / (2 * math.pi)
-            hi = f.float()
-            E.turns = torch.stack([hi, (f - hi.double()).float()], 1).contiguous().to(self.device)
+            E.turns = self._turns(E.base ** (-torch.arange(0, H, 2, dtype=torch.float64) / H)).to(self.device)
         a = n.Embed(E.table.data_ptr(), _dp(E.bigram), E.norm.data_ptr(), E.turns.data_ptr(), ids.data_ptr(),
                     positions.data_ptr(), _dp(row_seq), _dp(cu_q), state_rows.data_ptr(), _dp(last_token),
                     residual.data_ptr(), out.data_ptr(), E.buckets, E.mul_prev, E.mul_cur, H, E.table.shape[0],
@@ -905,12 +914,41 @@ class CudaOps(TorchOps):
             self.n.gemm_tile(w.data.dtype, x, x.stride(0), w.data, (w.K, 1), out, out.stride(0), M, w.N, w.K,
                              self.n.TILE_RELU2)
 
+    def glu_expands(self, ff: int, H: int, dtype) -> bool:
+        return not (dtype == torch.bfloat16 and H % 8 == 0)
+
+    def glu_linear(self, gate, up, dtype):
+        """Tensor-core form: tiles of 64 gate rows and their 64 up rows."""
+        if self.glu_expands(gate.shape[0], gate.shape[1], dtype):
+            return super().glu_linear(gate, up, dtype)
+        return self.dense_linear(self._interleaved([(gate, up)], dtype))
+
+    def linear_glu(self, w, x, M, out, activation: str, tmp=None):
+        n, ff = self.n, out.shape[1]
+        if not self.glu_expands(ff, w.K, x.dtype):
+            n.gemm_bf16_glu(w.data, x, x.shape[0], out, M, w.N, w.K, out.stride(0), ff, GLU[activation], self.status.ptr)
+            return
+        n.gemm_tile(x.dtype, x, x.stride(0), w.data, (w.K, 1), tmp, 2 * ff, M, 2 * ff, w.K)
+        n.glu(tmp, out, M, ff, GLU[activation], 0.0)
+
     def heads_expands(self, spec, dtype) -> bool:
         return dtype == torch.bfloat16 and self.n.heads_mma_ok(spec, 64)
 
-    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M):
-        self.n.heads_prep(inp, planes, n_planes, M, self.n.heads(kv, spec, self._no_tables), slots, L.q_norm, L.k_norm, spec,
-                          eps)
+    @staticmethod
+    def _turns(f: torch.Tensor) -> torch.Tensor:
+        """Frequencies (radians per token, float64) as turns per token in two floats [n, 2]: the angle of any position keeps
+        fp32 accuracy."""
+        f = f / (2 * math.pi)
+        hi = f.float()
+        return torch.stack([hi, (f - hi.double()).float()], 1).contiguous()
+
+    def rotation(self, dims: int, base: float):
+        f = super().rotation(dims, base)
+        return None if f is None else self._turns(f)
+
+    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M, positions=None):
+        self.n.heads_prep(inp, planes, n_planes, M, self.n.heads(kv, spec, self._no_tables), slots, L.q_norm, L.k_norm,
+                          getattr(L, "bias", None), getattr(L, "freqs", None), positions, spec, eps)
 
     @staticmethod
     def _head_gate(inp, spec):
@@ -945,9 +983,28 @@ class CudaOps(TorchOps):
         self.n.memory_chunks(inp, gates, self.n.memory(states, at, state_rows, L.head_norm, spec, eps), cu_q, first, last, ws,
                              M, row0, out)
 
-    def embedding(self, table, ids, out, M, scale=1.0):
+    def state_space_expands(self, spec, dtype) -> bool:
+        return dtype == torch.bfloat16 and self.n.space_chunk_ok(spec)
+
+    def state_space_prep(self, inp, planes, n_planes, side, xbc, dt, states, at, state_rows, row_seq, cu_q, L, spec, M, S):
+        if not self.linear_has_side(L.w_in):
+            side = None
+        self.n.space_prep(inp, planes, n_planes, side, spec.in_width - spec.dt_col,
+                          self.n.space(states, at, state_rows, L, spec), row_seq, cu_q, xbc, dt, M)
+
+    def state_space_tokens(self, inp, xbc, dt, states, at, state_rows, cu_q, L, out, S, M, spec):
+        self.n.space_tokens(inp, xbc, dt, self.n.space(states, at, state_rows, L, spec), cu_q, S, out)
+
+    def state_space_chunks(self, inp, xbc, dt, states, at, state_rows, cu_q, L, out, first, last, M, spec):
+        """Sequences ``first .. last - 1`` chunkwise."""
+        self.n.space_chunks(inp, xbc, dt, self.n.space(states, at, state_rows, L, spec), cu_q, first, last, out)
+
+    def group_norm(self, x, weight, parts: int, M, eps):
+        self.n.group_norm(x, weight, parts, M, eps)
+
+    def embedding(self, table, ids, out, M, scale=1.0, copy=None):
         if table.dtype != torch.float16:
-            self.n.embedding_typed(table, ids, out, M, table.shape[1], table.shape[0], float(scale), self.status.ptr)
+            self.n.embedding_typed(table, ids, out, M, table.shape[1], table.shape[0], float(scale), copy, self.status.ptr)
             return
         self.n.embedding(table, ids, out, M, table.shape[1], table.shape[0], float(scale), self.status.ptr)
 

@@ -158,7 +158,10 @@ def _build_named(out: str, srcs: List[str], extra: tuple, verbose: bool) -> str:
 # first start then waits for these sources only).  The ordinary build contains all of them and is preferred.
 GROUPS = {
     "latent": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "latent.cu", "latent_tc.cu", "moe.cu", "sampling.cu"),
-    "hybrid": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "heads.cu", "heads_tc.cu", "memory.cu", "moe.cu", "sampling.cu"),
+    "hybrid": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "heads.cu", "heads_tc.cu", "memory.cu", "moe.cu",
+               "sampling.cu"),
+    "looped": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "heads.cu", "heads_tc.cu", "state_space.cu", "moe.cu",
+               "sampling.cu"),
 }
 
 

@@ -49,7 +49,8 @@ class Chunks(Structure):
 
 class Router(Structure):
     _fields_ = [("planes", c_void_p)] + [(n, c_int32) for n in ("n_planes", "experts", "cols", "top", "softmax",
-                                                                "normalise")] + [("scale", c_float)]
+                                                                "normalise")] + [("scale", c_float), ("groups", c_int32),
+                                                                                 ("keep", c_int32)]
 
 
 class MoeGemm(Structure):
@@ -57,7 +58,7 @@ class MoeGemm(Structure):
                                         "row_score", "out_rows", "tiles", "n_tiles", "shared_score")] + \
                [(n, c_int32) for n in ("routed_n", "routed_k", "routed_ldo", "shared_n", "shared_k", "shared_ldo",
                                        "shared_mul", "shared_add", "shared_x_rows", "routed_cols", "shared_cols")] + \
-               [("routed_limit", c_float), ("shared_limit", c_float)]
+               [("routed_limit", c_float), ("shared_limit", c_float), ("glu", c_int32)]
 
 
 class Embed(Structure):
@@ -71,7 +72,13 @@ class Heads(Structure):
     _fields_ = [("k", c_void_p), ("v", c_void_p), ("block_stride", c_int64)] + \
                [(n, c_int32) for n in ("block_size", "dim_pad", "vdim_pad", "max_blocks")] + [("tables", c_void_p)] + \
                [(n, c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "chunk", "window")] + [("scale", c_float),
-                                                                                               ("num_blocks", c_int32)]
+                   ("num_blocks", c_int32), ("keep_first", c_int32), ("softcap", c_float), ("gate_each", c_int32)]
+
+
+class HeadsPrep(Structure):
+    _fields_ = [(n, c_void_p) for n in ("q_norm", "k_norm", "bias", "turns", "positions")] + \
+               [(n, c_int32) for n in ("k_col", "v_col", "gate_col", "gate_w", "own_kv", "rot_dims")] + \
+               [("temp_coef", c_float), ("temp_every", c_int32), ("eps", c_float)]
 
 
 class Memory(Structure):
@@ -79,6 +86,13 @@ class Memory(Structure):
                [("states", c_void_p), ("row_floats", c_int64), ("sum_at", c_int32), ("max_at", c_int32),
                 ("state_rows", c_void_p), ("state_ld", c_int32), ("gate_cap", c_float), ("eps", c_float),
                 ("head_norm", c_void_p)]
+
+
+class Space(Structure):
+    _fields_ = [(n, c_int32) for n in ("heads", "vdim", "state", "groups", "taps", "x_col", "b_at", "c_at", "conv_width",
+                                       "dt_col")] + \
+               [("states", c_void_p), ("row_floats", c_int64), ("conv_at", c_int32), ("state_rows", c_void_p),
+                ("state_ld", c_int32)] + [(n, c_void_p) for n in ("conv_w", "conv_b", "dt_bias", "neg_a", "skip")]
 
 
 _lib: Optional[ctypes.CDLL] = None
@@ -190,10 +204,15 @@ _SIGS = {
     "zse_tp_ctx_set_gather": (c_int, [c_void_p, c_int, c_int, POINTER(c_uint64), POINTER(c_uint64)]),
     "zse_gemm_bf16": (c_int, [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                               c_void_p, c_void_p]),
+    "zse_gemm_bf16_glu": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                                  c_void_p]),
+    "zse_gemm_bf16_side": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
+                                   c_void_p]),
     "zse_gemm_tile": (c_int, [c_int, POINTER(TileGemm), c_int, c_int, c_void_p]),
-    "zse_embedding_typed": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p]),
-    "zse_add_norm": (c_int, [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-                             c_float, c_void_p]),
+    "zse_embedding_typed": (c_int, [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_int,
+                                    c_void_p, c_void_p]),
+    "zse_add_norm": (c_int, [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float,
+                             c_void_p, c_int, c_int, c_int, c_float, c_void_p]),
     "zse_logits_finish": (c_int, [c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p]),
     "zse_argmax_f32": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p]),
     "zse_latent_mma_ok": (c_int, [c_int] * 6),
@@ -211,10 +230,10 @@ _SIGS = {
     "zse_post_norm": (c_int, [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                               c_int, c_float, c_void_p]),
     "zse_embed_design": (c_int, [c_int, POINTER(Embed), c_int, c_void_p, c_void_p]),
-    "zse_clamped_glu": (c_int, [c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p]),
+    "zse_glu": (c_int, [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p]),
     "zse_heads_mma_ok": (c_int, [c_int] * 3),
-    "zse_heads_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_int, POINTER(Heads), c_void_p, c_void_p, c_void_p,
-                               c_int, c_int, c_int, c_int, c_int, c_float, c_void_p]),
+    "zse_heads_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_int, POINTER(Heads), c_void_p, POINTER(HeadsPrep),
+                               c_void_p]),
     "zse_heads_attn": (c_int, [c_int, c_void_p, c_int, POINTER(Heads), c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                c_void_p, c_int, c_int, c_int, c_void_p]),
     "zse_heads_attn_chunks": (c_int, [c_void_p, c_int, c_int, POINTER(Heads), c_void_p, c_void_p, c_int, c_int, c_int,
@@ -226,6 +245,14 @@ _SIGS = {
                                   c_void_p]),
     "zse_memory_chunks": (c_int, [c_void_p, c_int, c_void_p, POINTER(Memory), c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                                   c_void_p, c_int, c_void_p]),
+    "zse_space_chunk_ok": (c_int, [c_int] * 2),
+    "zse_space_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, POINTER(Space), c_void_p, c_void_p,
+                               c_void_p, c_void_p, c_int, c_void_p]),
+    "zse_space_tokens": (c_int, [c_int, c_void_p, c_int, c_void_p, c_void_p, POINTER(Space), c_void_p, c_int, c_void_p, c_int,
+                                 c_void_p]),
+    "zse_space_chunks": (c_int, [c_void_p, c_int, c_void_p, c_void_p, POINTER(Space), c_void_p, c_int, c_int, c_void_p, c_int,
+                                 c_void_p]),
+    "zse_group_norm": (c_int, [c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p]),
     "zse_moe_gemm": (c_int, [POINTER(MoeGemm), c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
     "zse_read_probe": (c_int, [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p]),
     "zse_tp_gather_rows": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]),
@@ -556,6 +583,16 @@ def gemm_bf16(w, w_rows, x, x_rows_cap, out, M, N, K, ldo, epilogue, k_split, st
                              _stream()), "gemm_bf16")
 
 
+def gemm_bf16_glu(w, x, x_rows_cap, out, M, N, K, ldo, cols, kind, status):
+    _ck(load().zse_gemm_bf16_glu(_p(w), _p(x), x_rows_cap, _p(out), M, N, K, ldo, cols, kind, status, _stream()),
+        "gemm_bf16_glu")
+
+
+def gemm_bf16_side(w, x, x_rows_cap, out, M, N, K, ldo, side, side_col, status):
+    _ck(load().zse_gemm_bf16_side(_p(w), _p(x), x_rows_cap, _p(out), M, N, K, ldo, _p(side), side_col, status, _stream()),
+        "gemm_bf16_side")
+
+
 TILE_STORE, TILE_F32, TILE_GELU, TILE_GATE, TILE_RELU2 = 0, 1, 2, 3, 4
 
 
@@ -568,15 +605,16 @@ def gemm_tile(dtype, a, lda, b, ldb, out, ldo, M, N, K, epilogue=TILE_STORE, bat
     _ck(load().zse_gemm_tile(_DTYPE[dtype], byref(g), batch, max_tiles, _stream()), "gemm_tile")
 
 
-def embedding_typed(table, ids, out, M, H, vocab, scale, status):
-    _ck(load().zse_embedding_typed(_DTYPE[table.dtype], _p(table), _p(ids), _p(out), M, H, vocab, scale, status,
-                                   _stream()), "embedding_typed")
+def embedding_typed(table, ids, out, M, H, vocab, scale, copy, status):
+    _ck(load().zse_embedding_typed(_DTYPE[table.dtype], _p(table), _p(ids), _p(out), M, H, vocab, scale, _p(copy),
+                                   0 if copy is None else copy.stride(0), status, _stream()), "embedding_typed")
 
 
-def add_norm(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps):
+def add_norm(residual, planes, n_planes, slots, n_slots, weight, out, M, H, eps, scale=None, offset=0.0, replace=False):
     sd = 0 if slots is None else _DTYPE[slots.dtype]
-    _ck(load().zse_add_norm(_DTYPE[out.dtype], sd, _p(residual), _p(planes), n_planes, _p(slots), n_slots, _p(weight),
-                            _p(out), M, H, eps, _stream()), "add_norm")
+    _ck(load().zse_add_norm(_DTYPE[out.dtype], sd, _p(residual), _p(planes), n_planes, _p(slots), n_slots, _p(scale),
+                            int(replace), _p(weight), float(offset), _p(out), out.stride(0), M, H, eps, _stream()),
+        "add_norm")
 
 
 def post_norm(residual, planes, n_planes, slots, n_slots, weight, next_weight, out, M, H, eps):
@@ -589,25 +627,27 @@ def embed_design(a: Embed, dtype, M, status):
     _ck(load().zse_embed_design(_DTYPE[dtype], byref(a), M, status, _stream()), "embed_design")
 
 
-def clamped_glu(x, out, rows, ff, limit):
-    _ck(load().zse_clamped_glu(_DTYPE[x.dtype], _p(x), _p(out), rows, ff, float(limit), _stream()), "clamped_glu")
+def glu(x, out, rows, ff, kind, limit):
+    _ck(load().zse_glu(_DTYPE[x.dtype], _p(x), _p(out), rows, ff, kind, float(limit), _stream()), "glu")
 
 
 def heads(view, spec, block_tables) -> Heads:
     """``view``: ``models.hybrid.PagedHeads``."""
     return Heads(view.k.data_ptr(), view.v.data_ptr(), view.block_stride, view.block_size, view.k.shape[3], view.v.shape[3],
                  block_tables.stride(0), block_tables.data_ptr(), spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.chunk,
-                 spec.window, float(spec.scale), view.k.shape[0])
+                 spec.window, float(spec.scale), view.k.shape[0], spec.keep_first, float(spec.softcap), int(spec.gate_each))
 
 
 def heads_mma_ok(spec, block_size: int) -> bool:
     return bool(load().zse_heads_mma_ok(spec.dim, spec.vdim, block_size))
 
 
-def heads_prep(inp, planes, n_planes, M, h, slots, q_norm, k_norm, spec, eps):
+def heads_prep(inp, planes, n_planes, M, h, slots, q_norm, k_norm, bias, turns, positions, spec, eps):
+    p = HeadsPrep(_p(q_norm), _p(k_norm), _p(bias), _p(turns), _p(positions), spec.k_col,
+                  spec.k_col if spec.k_as_v else spec.v_col, spec.gate_col, spec.gate_width, int(spec.own_kv), spec.rot_dims,
+                  float(spec.temp_coef), int(spec.temp_every), float(eps))
     _ck(load().zse_heads_prep(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, M, byref(h), _p(slots),
-                              _p(q_norm), _p(k_norm), spec.k_col, spec.v_col, spec.gate_col,
-                              spec.heads if spec.gated else 0, int(spec.own_kv), float(eps), _stream()), "heads_prep")
+                              byref(p), _stream()), "heads_prep")
 
 
 def heads_attn(inp, h, row_seq, positions, out, gate, scratch, M, num_splits, tensor_cores):
@@ -647,6 +687,37 @@ def memory_tokens(inp, gates, m, cu_q, S, out):
 def memory_chunks(inp, gates, m, cu_q, first, last, o, M, row0, out):
     _ck(load().zse_memory_chunks(_p(inp), inp.stride(0), _p(gates), byref(m), _p(cu_q), first, last, _p(o), M, row0, _p(out),
                                  out.stride(0), _stream()), "memory_chunks", 2)
+
+
+def space(states, at, state_rows, L, spec) -> Space:
+    """``states``: the state pool's rows; ``at``: where the layer's part of a row begins; ``L``: the layer's weights."""
+    return Space(spec.heads, spec.vdim, spec.state, spec.groups, spec.conv, spec.x_col, spec.b_at, spec.c_at, spec.conv_width,
+                 spec.dt_col, states.data_ptr() + 4 * at, states.stride(0), spec.conv_at, _p(state_rows),
+                 state_rows.stride(0), _p(L.conv_w), _p(L.conv_b), _p(L.dt_bias), _p(L.neg_a), _p(L.D))
+
+
+def space_chunk_ok(spec) -> bool:
+    return bool(load().zse_space_chunk_ok(spec.state, spec.vdim))
+
+
+def space_prep(inp, planes, n_planes, side, side_ld, m, row_seq, cu_q, xbc, dt, M):
+    _ck(load().zse_space_prep(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, _p(side), side_ld, byref(m),
+                              _p(row_seq), _p(cu_q), _p(xbc), _p(dt), M, _stream()), "space_prep")
+
+
+def space_tokens(inp, xbc, dt, m, cu_q, S, out):
+    _ck(load().zse_space_tokens(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(xbc), _p(dt), byref(m), _p(cu_q), S, _p(out),
+                                out.stride(0), _stream()), "space_tokens")
+
+
+def space_chunks(inp, xbc, dt, m, cu_q, first, last, out):
+    _ck(load().zse_space_chunks(_p(inp), inp.stride(0), _p(xbc), _p(dt), byref(m), _p(cu_q), first, last, _p(out),
+                                out.stride(0), _stream()), "space_chunks")
+
+
+def group_norm(x, weight, parts, M, eps):
+    _ck(load().zse_group_norm(_DTYPE[x.dtype], _p(x), x.stride(0), M, parts, x.shape[1] // parts, _p(weight), float(eps),
+                              _stream()), "group_norm")
 
 
 def logits_finish(logits, M, scale, cap):
@@ -711,7 +782,7 @@ def moe_tile_rows(M, E, top) -> int:
 def moe_route(planes, n_planes, M, moe, tile_rows, x, H, out_per_token, ws):
     """``moe``: the layer's ``MoESpec``."""
     r = Router(_p(planes), n_planes, moe.experts, moe.router_rows, moe.top, int(moe.score == "softmax"), int(moe.normalise),
-               float(moe.scale))
+               float(moe.scale), moe.groups, moe.keep_groups)
     _ck(load().zse_moe_route(_DTYPE[x.dtype], byref(r), M, tile_rows, _p(x), H, out_per_token,
                              _p(ws.counts), _p(ws.slot_expert), _p(ws.slot_rank), _p(ws.slot_score), _p(ws.first_row),
                              _p(ws.tiles), _p(ws.n_tiles), _p(ws.xs), _p(ws.row_score), _p(ws.out_rows),
