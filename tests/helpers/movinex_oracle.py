@@ -201,13 +201,13 @@ def greedy(cfg, weights, prompt, n):
 # ---- small random models --------------------------------------------------------------------------------------------
 def attention_layer(heads, kv_heads, dim, vdim, mlp, coef=0.4, every=11, scale=None):
     return {"type": "attention", "mlp": mlp,
-            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or dim ** -0.5,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or 2 * dim ** -0.5,
                       "q_temp": {"coef": coef, "every": every}}}
 
 
 def window_layer(heads, kv_heads, dim, size, keep, mlp, rot=None, base=1e4, softcap=8.0, scale=None):
     return {"type": "attention_2", "mlp": mlp,
-            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale or dim ** -0.5,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale or 2 * dim ** -0.5,
                       "softcap": softcap, "mask": {"size": size, "keep_first": keep},
                       "rot": {"dims": dim if rot is None else rot, "base": base}}}
 
@@ -269,7 +269,7 @@ def shapes(cfg):
     return out
 
 
-def random_weights(cfg, seed=0, sharp=1.0):
+def random_weights(cfg, seed=0):
     """bfloat16 weights.  Every mechanism has a share in the logits: biases of the size of the projections, layer scales that
     differ by channel, memories of some tens of tokens beside short ones, step sizes that differ from token to token."""
     g = torch.Generator().manual_seed(seed)
@@ -295,7 +295,5 @@ def random_weights(cfg, seed=0, sharp=1.0):
             w = rnd(shape) * shape[1] ** -0.5
             if name == "embed":
                 w *= shape[1] ** 0.5
-            if last in ("q", "k"):
-                w *= sharp
         W[name] = w.to(torch.bfloat16)
     return W
