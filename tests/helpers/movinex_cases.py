@@ -24,14 +24,14 @@ CASES = {
                                  mamba_layer(3, 5, 19, None, groups=3, conv=6, norm_groups=5)], loop=(0, 2, 3),
                         logit_scale=1.9),
     # more query heads on a kv head than one tile of 16, heads wider than a tensor-core tile of columns, states wider than one
-    # tile of rows, a window of the token alone beside kept ones, groups of one expert, taps of 1 and 5
+    # tile of rows, a window of the token alone beside kept ones, taps of 1 and 5
     "wide": config(128, 200, [window_layer(34, 2, 40, 65, 64, moe(20, 4, 32, 5, 2), rot=0),
                               mamba_layer(2, 72, 136, dense(136), conv=1, norm_groups=2),
-                              attention_layer(8, 1, 136, 144, moe(9, 4, 16, 9, 5), every=1),
+                              attention_layer(8, 1, 136, 144, dense(64), every=1),
                               window_layer(5, 1, 8, 1, 9, None),
                               mamba_layer(5, 64, 256, None, groups=5, conv=5)], loop=(2, 5, 2), eps=1e-6),
-    # no layer sees everything: blocks leave, those of the kept tokens stay
-    "windows-only": config(64, 90, [window_layer(4, 2, 16, 30, 3, None), window_layer(2, 1, 32, 17, 66, moe(4, 2, 16))],
+    # no layer sees everything: blocks leave, those of the kept tokens stay; groups of one expert
+    "windows-only": config(64, 90, [window_layer(4, 2, 16, 30, 3, None), window_layer(2, 1, 32, 17, 66, moe(9, 4, 16, 9, 5))],
                            loop=(0, 2, 1)),
     # no cached keys at all, no loop
     "states-only": config(64, 90, [mamba_layer(2, 32, 24, None), mamba_layer(4, 16, 64, dense(24), conv=3, norm_groups=4)]),
