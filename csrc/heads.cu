@@ -27,6 +27,7 @@ struct HeadsPrepArgs {
   float temp_coef;
   int temp_every;
 };
+constexpr int kPrepGates = 256;                  // gates of a warp
 constexpr int kPrepPairs = 128;                  // pairs whose sine and cosine a CTA keeps in shared memory
 
 // Sine and cosine of p * (turns per position, as two floats): the reduced angle keeps fp32 accuracy at any position.
@@ -78,12 +79,10 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
     return v;
   };
   const int G = a.own_kv ? h.kv_heads : 0;
-  if (u >= h.heads + 2 * G) {                    // gates
-    for (int i = lane; i < a.gate_w; i += 32) {
-      float v = 0.f;
-      for (int p = 0; p < n_planes; ++p) v += pl[p * plane + a.gate_col + i];
-      in[a.gate_col + i] = from_f32<T>(v);
-    }
+  if (u >= h.heads + 2 * G) {                    // gates; their section is padded to 8 columns
+    const int g0 = (u - h.heads - 2 * G) * kPrepGates, g1 = min(a.gate_w, g0 + kPrepGates);
+#pragma unroll 2
+    for (int i = g0 + lane * VEC; i < g1; i += 32 * VEC) store_vec<VEC>(in + a.gate_col + i, value(a.gate_col + i));
     return;
   }
   T* dst = nullptr;
@@ -750,7 +749,7 @@ template <typename T, int VEC>
 cudaError_t launch_prep(void* inp, const void* planes, int n_planes, int M, const ZseHeads* z, const void* slots,
                         const ZseHeadsPrep* p, const HeadsPrepArgs& a, cudaStream_t st) {
   const Heads h = heads_of(z);
-  const int units = h.heads + 2 * (a.own_kv ? h.kv_heads : 0) + (n_planes > 0 && a.gate_w > 0 ? 1 : 0);
+  const int units = h.heads + 2 * (a.own_kv ? h.kv_heads : 0) + (n_planes > 0 ? (a.gate_w + kPrepGates - 1) / kPrepGates : 0);
   return launch_pdl(heads_prep_kernel<T, VEC>, dim3(M, (units + 7) / 8), dim3(256), 0, st,
                     reinterpret_cast<T*>(inp), reinterpret_cast<const float*>(planes), n_planes, M,
                     reinterpret_cast<T*>(z->k), reinterpret_cast<T*>(z->v), h, reinterpret_cast<const long long*>(slots),
@@ -780,6 +779,7 @@ extern "C" int zse_heads_prep(int dtype, void* inp, int ld, const void* planes, 
                         reinterpret_cast<const float*>(p->turns), reinterpret_cast<const int*>(p->positions), p->rot_dims,
                         p->temp_coef, p->temp_every};
   const bool vec = h->dim % 4 == 0 && h->vdim % 4 == 0 && ld % 4 == 0 && p->k_col % 4 == 0 && p->v_col % 4 == 0 &&
+                   p->gate_col % 4 == 0 && p->gate_col + (p->gate_w + 3) / 4 * 4 <= ld &&
                    h->block_stride % 4 == 0 &&
                    !((reinterpret_cast<uintptr_t>(inp) | reinterpret_cast<uintptr_t>(planes) |
                       reinterpret_cast<uintptr_t>(h->k) | reinterpret_cast<uintptr_t>(h->v) |

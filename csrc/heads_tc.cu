@@ -63,7 +63,12 @@ __device__ __forceinline__ uint64_t ht_desc_mn(uint32_t smem_addr) {
   return d;
 }
 
-template <bool CAP>
+// A cap bounds the scores: with one of up to kHtFixedCap the cap itself is the reference maximum of every row (weights down to
+// exp(-2 cap) are ordinary fp32 numbers), and a tile is read once.
+enum HtCap { kHtNoCap = 0, kHtCap = 1, kHtFixed = 2 };
+constexpr float kHtFixedCap = 40.f;
+
+template <int CAP>
 __global__ void __launch_bounds__(kHtThreads, 2)
 heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                 const __grid_constant__ CUtensorMap map_v, const HtArgs a) {
@@ -205,8 +210,9 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
     const int limit = a.q_pos0[seq] + row, lo = a.h.first_seen(limit);
     const uint32_t lane_addr = uint32_t(warp * 32) << 16;
     const float scale_log2 = a.h.scale * kLog2E;
-    auto log2_score = [&](float s) { return CAP ? a.h.capped(s * a.h.scale) * kLog2E : s * scale_log2; };
+    auto log2_score = [&](float s) { return CAP != kHtNoCap ? a.h.capped(s * a.h.scale) * kLog2E : s * scale_log2; };
     const int o_cols = (a.h.vdim + 15) / 16 * 16;
+    const float cap_in = 2.f * a.h.scale * kLog2E / a.h.cap, cap_out = -2.f * a.h.cap * kLog2E;        // kHtFixed
     float m_used = -INFINITY, l = 0.f;
     uint32_t ph = 0;
     bool ok = true;
@@ -226,7 +232,7 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
                                                     k0 + kHtKeys - 1 <= limit);
       float mx = -INFINITY;
 #pragma unroll 1
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; CAP != kHtFixed && c < 4; ++c) {
         uint32_t v[32];
         ZSE_TMEM_LD_X16(v, tm_s + lane_addr + c * 32);
         ZSE_TMEM_LD_X16((v + 16), tm_s + lane_addr + c * 32 + 16);
@@ -284,7 +290,10 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               float p0, p1;
-              if constexpr (CAP) {
+              if constexpr (CAP == kHtFixed) {     // cap tanh(s / cap) - cap = -2 cap / (1 + exp(2 s / cap))
+                p0 = ex2(__fdividef(cap_out, 1.f + ex2(__uint_as_float(v[2 * i]) * cap_in)));
+                p1 = ex2(__fdividef(cap_out, 1.f + ex2(__uint_as_float(v[2 * i + 1]) * cap_in)));
+              } else if constexpr (CAP == kHtCap) {
                 p0 = ex2(log2_score(__uint_as_float(v[2 * i])) - m_ref);
                 p1 = ex2(log2_score(__uint_as_float(v[2 * i + 1])) - m_ref);
               } else {
@@ -386,9 +395,9 @@ int launch_heads_tc(const bf16* inp, int ld, int rows, const void* k, const void
   if (int rc = get_tmap_rows3(v, num_blocks, per_block, h.vp, h.block_stride, br, 0, &mv)) return rc;
   const HtArgs a{h, cu_q, q_pos0, first, out, ldo, gate, ld, br, (h.dim + 63) / 64, (h.vdim + 63) / 64, status};
   const size_t smem = size_t(2 * a.k_panels + a.v_panels) * kHtPanel + 1024 + sizeof(HtBars);
-  static bool done[2][kMaxDevices] = {};
-  const int slot = current_device_slot(), cap = h.cap > 0.f;
-  auto kern = cap ? heads_tc_kernel<true> : heads_tc_kernel<false>;
+  static bool done[3][kMaxDevices] = {};
+  const int slot = current_device_slot(), cap = h.cap <= 0.f ? kHtNoCap : h.cap <= kHtFixedCap ? kHtFixed : kHtCap;
+  auto kern = cap == kHtNoCap ? heads_tc_kernel<kHtNoCap> : cap == kHtCap ? heads_tc_kernel<kHtCap> : heads_tc_kernel<kHtFixed>;
   if (!done[cap][slot]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              int(6 * kHtPanel + 1024 + sizeof(HtBars))) != cudaSuccess)

@@ -8,8 +8,8 @@
 namespace zse {
 namespace {
 
-template <typename T>
-__global__ void embedding_typed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) embedding_typed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
                                        float* __restrict__ out, int H, int vocab, float scale, T* __restrict__ copy,
                                        int ld_copy, Status* st) {
   pdl_launch_dependents();
@@ -22,10 +22,13 @@ __global__ void embedding_typed_kernel(const T* __restrict__ table, const int* _
   }
   const T* src = table + size_t(id) * H;
   float* dst = out + size_t(row) * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    const float x = to_f32(src[i]) * scale;
-    dst[i] = x;
-    if (copy != nullptr) copy[size_t(row) * ld_copy + i] = from_f32<T>(x);
+#pragma unroll 4
+  for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
+    F32Vec<VEC> x = load_vec<VEC>(src + i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x.v[e] *= scale;
+    store_vec<VEC>(dst + i, x);
+    if (copy != nullptr) store_vec<VEC>(copy + size_t(row) * ld_copy + i, x);
   }
 }
 
@@ -418,20 +421,21 @@ __global__ void __launch_bounds__(1024) argmax_f32_kernel(const float* __restric
 using namespace zse;
 #define ST(s) reinterpret_cast<cudaStream_t>(s)
 
+template <typename T>
+static cudaError_t launch_embedding_typed(const void* table, const void* ids, void* out, int M, int H, int vocab, float scale,
+                                          void* copy, int ld_copy, void* status, cudaStream_t st) {
+  const bool vec = H % 4 == 0 && ld_copy % 4 == 0 && aligned16({table, out}) && !(reinterpret_cast<uintptr_t>(copy) & 7) &&
+                   (sizeof(T) == 2 || aligned16({copy}));
+  return launch_pdl(vec ? embedding_typed_kernel<T, 4> : embedding_typed_kernel<T, 1>, dim3(M), dim3(256), 0, st,
+                    reinterpret_cast<const T*>(table), reinterpret_cast<const int*>(ids), reinterpret_cast<float*>(out), H,
+                    vocab, scale, reinterpret_cast<T*>(copy), ld_copy, reinterpret_cast<Status*>(status));
+}
+
 extern "C" int zse_embedding_typed(int dtype, const void* table, const void* ids, void* out, int M, int H, int vocab,
                                    float scale, void* copy, int ld_copy, void* status, void* stream) {
   if (M <= 0) return 0;
-  cudaError_t e;
-  if (dtype == kBF16)
-    e = launch_pdl(embedding_typed_kernel<bf16>, dim3(M), dim3(128), 0, ST(stream), reinterpret_cast<const bf16*>(table),
-                   reinterpret_cast<const int*>(ids), reinterpret_cast<float*>(out), H, vocab, scale,
-                   reinterpret_cast<bf16*>(copy), ld_copy, reinterpret_cast<Status*>(status));
-  else
-    e = launch_pdl(embedding_typed_kernel<float>, dim3(M), dim3(128), 0, ST(stream),
-                   reinterpret_cast<const float*>(table), reinterpret_cast<const int*>(ids),
-                   reinterpret_cast<float*>(out), H, vocab, scale, reinterpret_cast<float*>(copy), ld_copy,
-                   reinterpret_cast<Status*>(status));
-  return e == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+  auto run = dtype == kBF16 ? launch_embedding_typed<bf16> : launch_embedding_typed<float>;
+  return run(table, ids, out, M, H, vocab, scale, copy, ld_copy, status, ST(stream)) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }
 
 extern "C" int zse_add_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes,

@@ -107,49 +107,59 @@ ss_prep_kernel(T* __restrict__ inp, T* __restrict__ xbc, const Space m, const Sp
     return load_vec<4>(m.states + size_t(read) * m.row_floats + m.conv_at +
                        size_t(taps - 1 + t - back - begin) * m.conv_width + c);
   };
-  for (int t = t0; t < t1; ++t) {
-    if (t >= end) {                              // the block's first row, or a sequence's
-      s = a.row_seq != nullptr ? a.row_seq[t] : t;
-      begin = a.cu_q != nullptr ? a.cu_q[s] : t;
-      end = a.cu_q != nullptr ? a.cu_q[s + 1] : t + 1;
-      read = m.state_rows[s];
-      write = m.state_rows[m.state_ld + s];
-      if constexpr (TAPS > 1) {
+  constexpr int kAhead = 4;                      // rows whose loads are under way together
+  for (int tb = t0; tb < t1; tb += kAhead) {
+    F32Vec<4> rows_in[kAhead];
 #pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) win[j] = before(t, TAPS - 1 - j);
+    for (int j = 0; j < kAhead; ++j)
+      if (tb + j < t1) rows_in[j] = raw(tb + j, col);
+#pragma unroll
+    for (int jr = 0; jr < kAhead; ++jr) {
+      const int t = tb + jr;
+      if (t >= t1) break;
+      if (t >= end) {                              // the block's first row, or a sequence's
+        s = a.row_seq != nullptr ? a.row_seq[t] : t;
+        begin = a.cu_q != nullptr ? a.cu_q[s] : t;
+        end = a.cu_q != nullptr ? a.cu_q[s + 1] : t + 1;
+        read = m.state_rows[s];
+        write = m.state_rows[m.state_ld + s];
+        if constexpr (TAPS > 1) {
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) win[j] = before(t, TAPS - 1 - j);
+        }
       }
+      float* last = write >= 0 ? m.states + size_t(write) * m.row_floats + m.conv_at + c : nullptr;
+      if (last != nullptr && t == begin && end - begin < taps - 1)   // what stays of the inputs before a short portion
+        for (int j = 0; j + end - begin < taps - 1; ++j)
+          store_vec<4>(last + size_t(j) * m.conv_width, before(t, taps - 1 - j - (end - begin)));
+      const F32Vec<4> x = rows_in[jr];
+      F32Vec<4> y = bias;
+      if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[j].v[e], win[j].v[e], y.v[e]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[TAPS - 1].v[e], x.v[e], y.v[e]);
+        if constexpr (TAPS > 1) {
+#pragma unroll
+          for (int j = 0; j + 1 < TAPS - 1; ++j) win[j] = win[j + 1];
+          win[TAPS - 2] = x;
+        }
+      } else {
+        for (int j = 0; j < taps; ++j) {
+          const F32Vec<4> f = load_vec<4>(a.conv_w + size_t(j) * m.conv_width + c);
+          const F32Vec<4> v = j + 1 == taps ? x : before(t, taps - 1 - j);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y.v[e] = fmaf(f.v[e], v.v[e], y.v[e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y.v[e] = silu_exact(y.v[e]);
+      store_vec<4>(xbc + size_t(t) * m.conv_width + c, y);
+      const int place = t - (end - (taps - 1));
+      if (last != nullptr && place >= 0) store_vec<4>(last + size_t(place) * m.conv_width, x);
     }
-    float* last = write >= 0 ? m.states + size_t(write) * m.row_floats + m.conv_at + c : nullptr;
-    if (last != nullptr && t == begin && end - begin < taps - 1)   // what stays of the inputs before a short portion
-      for (int j = 0; j + end - begin < taps - 1; ++j)
-        store_vec<4>(last + size_t(j) * m.conv_width, before(t, taps - 1 - j - (end - begin)));
-    const F32Vec<4> x = raw(t, col);
-    F32Vec<4> y = bias;
-    if constexpr (TAPS > 0) {
-#pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[j].v[e], win[j].v[e], y.v[e]);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[TAPS - 1].v[e], x.v[e], y.v[e]);
-      if constexpr (TAPS > 1) {
-#pragma unroll
-        for (int j = 0; j + 1 < TAPS - 1; ++j) win[j] = win[j + 1];
-        win[TAPS - 2] = x;
-      }
-    } else {
-      for (int j = 0; j < taps; ++j) {
-        const F32Vec<4> f = load_vec<4>(a.conv_w + size_t(j) * m.conv_width + c);
-        const F32Vec<4> v = j + 1 == taps ? x : before(t, taps - 1 - j);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) y.v[e] = fmaf(f.v[e], v.v[e], y.v[e]);
-      }
-    }
-#pragma unroll
-    for (int e = 0; e < 4; ++e) y.v[e] = silu_exact(y.v[e]);
-    store_vec<4>(xbc + size_t(t) * m.conv_width + c, y);
-    const int place = t - (end - (taps - 1));
-    if (last != nullptr && place >= 0) store_vec<4>(last + size_t(place) * m.conv_width, x);
   }
 }
 
@@ -158,7 +168,7 @@ constexpr int kSpTokThreads = 256, kSpTokRows = 8;       // rows of S that a thr
 
 // grid (columns / (cw * VEC), heads, sequences); cw: column vectors side by side, a power of two up to 32
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kSpTokThreads)
+__global__ void __launch_bounds__(kSpTokThreads, 3)
 ss_tokens_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ xbc, const float* __restrict__ dt,
                  const Space m, const float* __restrict__ neg_a, const float* __restrict__ skip, const int* __restrict__ cu_q,
                  T* __restrict__ out, int ldo, int cw) {

@@ -41,10 +41,15 @@ CASES = {
 }
 
 
+# of the weights and tokens: one with which no early token's choice of experts is a close call, which rounding would decide
+SEEDS = {"wide": 2}
+
+
 class Model:
     """A case on disk with its oracle logits; ``tokens[r]`` / ``want[r]`` per request."""
 
-    def __init__(self, name, folder, seed=1):
+    def __init__(self, name, folder, seed=None):
+        seed = seed or SEEDS.get(name, 1)
         self.cfg = CASES[name]
         self.weights = oracle.random_weights(self.cfg, seed)
         self.path = write_model(folder, self.cfg, self.weights)

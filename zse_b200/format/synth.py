@@ -59,22 +59,22 @@ def nimelorn_design(width: int, vocab: int, heads: int, kv_heads: int, dim: int,
 
 
 def movinex_design(width: int, vocab: int, heads: int, kv_heads: int, dim: int, window: int, keep: int, space: tuple,
-                   dense_ff: int, experts: int, top: int, ff: int, groups: tuple, repeats: int = 1, times: int = 2,
+                   dense_ff: int, experts: int, top: int, ff: int, groups: tuple, times: int = 2, tail: tuple = (2,),
                    rot: int = 0, eps: float = 1e-6) -> dict:
-    """A Movinex ``config.json`` of ``repeats`` times three layers - attention with a dense feed-forward, windowed attention
-    with experts, a state space (``space``: heads, vdim, state, groups) with experts - and a last such state space; the first
-    three layers are a loop of ``times`` passes.  ``groups``: count and keep of the router."""
+    """A Movinex ``config.json`` of three kinds of layers - attention with a dense feed-forward, windowed attention with
+    experts, a state space (``space``: heads, vdim, state, groups) with experts -, one of each in a loop of ``times`` passes,
+    and behind the loop those that ``tail`` names.  ``groups``: count and keep of the router."""
     dense = {"kind": "dense", "ff": dense_ff}
     moe = {"kind": "moe", "expert": {"ff": ff},
            "router": {"experts": experts, "top": top, "groups": dict(zip(("count", "keep"), groups))}}
     m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
-    state = {"type": "mamba2", "mlp": moe, "mixer": dict(zip(("heads", "vdim", "state", "groups"), space), conv=4,
-                                                         norm_groups=1)}
-    layers = [{"type": "attention", "mlp": dense, "mixer": dict(m, q_temp={"coef": 0.1, "every": 8192})},
-              {"type": "attention_2", "mlp": moe, "mixer": dict(m, softcap=30.0, mask={"size": window, "keep_first": keep},
-                                                                rot={"dims": rot or dim, "base": 10000.0})}, state] * repeats
-    return {"architecture": "Movinex", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers + [state],
-            "logit_scale": 1.0, "loop": {"start": 0, "stop": 3, "times": times}}
+    kinds = [{"type": "attention", "mlp": dense, "mixer": dict(m, q_temp={"coef": 0.1, "every": 8192})},
+             {"type": "attention_2", "mlp": moe, "mixer": dict(m, softcap=30.0, mask={"size": window, "keep_first": keep},
+                                                               rot={"dims": rot or dim, "base": 10000.0})},
+             {"type": "mamba2", "mlp": moe, "mixer": dict(zip(("heads", "vdim", "state", "groups"), space), conv=4,
+                                                          norm_groups=1)}]
+    return {"architecture": "Movinex", "vocab": vocab, "width": width, "norm": {"eps": eps},
+            "layers": kinds + [kinds[i] for i in tail], "logit_scale": 1.0, "loop": {"start": 0, "stop": 3, "times": times}}
 
 
 # entries with a "design" hold a config.json of that architecture instead of ``ModelConfig`` fields
@@ -93,10 +93,10 @@ SHAPES = {
                                                                 64, 4, 2048, 4096)),
     "tiny-movinex": dict(arch="movinex", design=movinex_design(160, 1024, 6, 2, 32, 48, 6, (5, 32, 40, 1), 224, 10, 3, 72,
                                                                (5, 3), rot=16)),
-    "movinex-2k": dict(arch="movinex", design=movinex_design(2048, 102400, 16, 4, 128, 4096, 64, (64, 64, 128, 1), 8192, 64, 6,
-                                                             1408, (8, 4), repeats=2, rot=64)),
-    "movinex-4k": dict(arch="movinex", design=movinex_design(4096, 102400, 32, 8, 128, 4096, 64, (128, 64, 128, 8), 14336, 64,
-                                                             4, 2048, (8, 4), rot=64)),
+    "movinex-2k": dict(arch="movinex", design=movinex_design(2048, 102400, 16, 4, 128, 2048, 64, (64, 64, 128, 1), 8192, 64, 6,
+                                                             1408, (8, 4), tail=(1, 2), rot=64)),
+    "movinex-4k": dict(arch="movinex", design=movinex_design(4096, 102400, 32, 8, 128, 2048, 64, (128, 64, 128, 8), 14336, 64,
+                                                             4, 2048, (8, 4), times=1, rot=64)),
     "tiny": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64, intermediate_size=688,
                  vocab_size=1024, rms_norm_eps=1e-6, rope_theta=10000.0, arch="llama", max_seq_len=2048),
     "tiny-aligned": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64,

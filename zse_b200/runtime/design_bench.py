@@ -279,8 +279,8 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
     return T.rows
 
 
-def markdown(rows: List[dict]) -> str:
-    out = ["| phase | kernel | us | roofline us | fraction | bound | like kernel (dense) | its us | its fraction |",
+def markdown(rows: List[dict], neighbour: str = "dense") -> str:
+    out = [f"| phase | kernel | us | roofline us | fraction | bound | like kernel ({neighbour}) | its us | its fraction |",
            "|---|---|---|---|---|---|---|---|---|"]
     by = {(r["phase"], r["kernel"]): r for r in rows}
     for r in rows:
