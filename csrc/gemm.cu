@@ -74,7 +74,7 @@ __device__ __forceinline__ void epilogue(const GemmArgs& a, uint32_t tmem_acc, i
             const float g = __uint_as_float(r[i]);
             const float u = park[(c + i) * 32 + lane];
             if (EPI == kEpiGlu)
-              reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n_out] = __float2bfloat16_rn(glu(a.glu, g, u, 0.f));
+              reinterpret_cast<bf16*>(a.out)[size_t(t) * a.ldo + n_out] = __float2bfloat16_rn(glu<true>(a.glu, g, u, 0.f));
             else
               out[size_t(t) * a.ldo + n_out] = __float2half_rn(clamp_f16(silu_f(g) * u));
           }

@@ -99,7 +99,7 @@ glu_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, int ff, i
   pdl_wait();
   for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
     const T* g = in + i / ff * 2 * ff + i % ff;
-    out[i] = from_f32<T>(glu(kind, to_f32(g[0]), to_f32(g[ff]), limit));
+    out[i] = from_f32<T>(glu<false>(kind, to_f32(g[0]), to_f32(g[ff]), limit));
   }
 }
 

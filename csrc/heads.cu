@@ -10,7 +10,8 @@
 //
 // Cached tiles: [block][kv head][token][dim], then the same for values, dims padded to 8 (the padding is zero).  Scores and
 // softmax are fp32; softmax weights enter the product with the values as two bfloat16 terms (value and remainder).  A row
-// sees the positions from first_seen(position) to its own, and the first `keep` ones; block -1 of a table is a hole whose tokens do not exist.
+// sees the positions from first_seen(position) to its own, and the first `keep` ones; block -1 of a table is a hole whose
+// tokens do not exist.
 #include "api.h"
 #include "heads.cuh"
 
@@ -41,19 +42,20 @@ __device__ __forceinline__ float2 pair_turn(const float* turns, int i, float p) 
 }
 
 // A warp per (row, section): query heads, then key heads, value heads and - with planes - the gates.  grid (rows, sections / 8)
-template <typename T, int VEC>
+// MORE: with bias, rotation or temperature.
+template <typename T, int VEC, bool MORE>
 __global__ void __launch_bounds__(256)
 heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_planes, int M, T* __restrict__ kc,
                   T* __restrict__ vc, Heads h, const long long* __restrict__ slots, const T* __restrict__ q_norm,
                   const T* __restrict__ k_norm, const T* __restrict__ bias, HeadsPrepArgs a, int units) {
   constexpr int kKeep = VEC == 4 ? 2 : 8;        // accesses of a head that stay in registers (up to 256 dimensions)
-  __shared__ float2 turned[kPrepPairs];
+  __shared__ float2 turned[MORE ? kPrepPairs : 1];
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x, u = blockIdx.y * 8 + (threadIdx.x >> 5);
-  const float pos = a.positions != nullptr ? float(a.positions[t]) : 0.f;
-  if (a.rot_dims > 0) {
+  const float pos = MORE && a.positions != nullptr ? float(a.positions[t]) : 0.f;
+  if (MORE && a.rot_dims > 0) {
     for (int i = threadIdx.x; i < min(kPrepPairs, a.rot_dims / 2); i += blockDim.x) turned[i] = pair_turn(a.turns, i, pos);
     __syncthreads();
   }
@@ -63,7 +65,8 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
   const size_t plane = size_t(M) * a.ld;
   auto value = [&](int c) {
     F32Vec<VEC> v{};
-    if (bias != nullptr) v = load_vec<VEC>(bias + c);
+    if (n_planes == 0 && !MORE) return load_vec<VEC>(in + c);
+    if (MORE && bias != nullptr) v = load_vec<VEC>(bias + c);
     if (n_planes == 0) {
       const F32Vec<VEC> x = load_vec<VEC>(in + c);
 #pragma unroll
@@ -109,6 +112,7 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
   };
   auto rotated = [&](int i) {                    // dimensions from i on
     F32Vec<VEC> v = value(c0 + i);
+    if constexpr (!MORE) return v;
     if constexpr (VEC == 4) {
       if (i < a.rot_dims) turn(i, v.v[0], v.v[1]);
       if (i + 2 < a.rot_dims) turn(i + 2, v.v[2], v.v[3]);
@@ -138,7 +142,7 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
     for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
   }
   float inv = 1.f / sqrtf(warp_sum(ss) / float(h.dim) + a.eps);
-  if (u < h.heads && a.temp_coef != 0.f)
+  if (MORE && u < h.heads && a.temp_coef != 0.f)
     inv *= 1.f + a.temp_coef * logf(float((a.positions[t] + 1) / a.temp_every + 1));
   auto put = [&](int i, const F32Vec<VEC>& v) {
     F32Vec<VEC> y;
@@ -661,8 +665,8 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
       if (c >= h.vdim) continue;
       float y0 = o[n][half * 2] * inv, y1 = o[n][half * 2 + 1] * inv;
       if (gate != nullptr) {
-        y0 *= sigmoid_exact(to_f32(gate[t * ld + h.gate_at(head, c)]));
-        y1 *= sigmoid_exact(to_f32(gate[t * ld + h.gate_at(head, c + 1)]));
+        y0 *= sigmoid_fast(to_f32(gate[t * ld + h.gate_at(head, c)]));
+        y1 *= sigmoid_fast(to_f32(gate[t * ld + h.gate_at(head, c + 1)]));
       }
       *reinterpret_cast<uint32_t*>(out + t * ldo + size_t(head) * h.vdim + c) = pack_bf16(y0, y1);
     }
@@ -750,7 +754,9 @@ cudaError_t launch_prep(void* inp, const void* planes, int n_planes, int M, cons
                         const ZseHeadsPrep* p, const HeadsPrepArgs& a, cudaStream_t st) {
   const Heads h = heads_of(z);
   const int units = h.heads + 2 * (a.own_kv ? h.kv_heads : 0) + (n_planes > 0 ? (a.gate_w + kPrepGates - 1) / kPrepGates : 0);
-  return launch_pdl(heads_prep_kernel<T, VEC>, dim3(M, (units + 7) / 8), dim3(256), 0, st,
+  const bool more = p->bias != nullptr || p->rot_dims > 0 || p->temp_coef != 0.f;
+  return launch_pdl(more ? heads_prep_kernel<T, VEC, true> : heads_prep_kernel<T, VEC, false>, dim3(M, (units + 7) / 8),
+                    dim3(256), 0, st,
                     reinterpret_cast<T*>(inp), reinterpret_cast<const float*>(planes), n_planes, M,
                     reinterpret_cast<T*>(z->k), reinterpret_cast<T*>(z->v), h, reinterpret_cast<const long long*>(slots),
                     reinterpret_cast<const T*>(p->q_norm), reinterpret_cast<const T*>(p->k_norm),

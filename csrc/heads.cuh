@@ -19,7 +19,7 @@ struct Heads {
   // cap * tanh(score / cap) of a scaled score; within 2^-22 of cap
   __device__ __forceinline__ float capped(float s) const {
     const float e = ex2(s * (2.f * kLog2E / cap));
-    return cap - __fdividef(2.f * cap, 1.f + e);
+    return fmaf(-2.f * cap, rcp(1.f + e), cap);
   }
   // place of the gate of a head's dimension d among a row's gates
   __device__ __forceinline__ int gate_at(int head, int d) const { return gate_each ? head * vdim + d : head; }

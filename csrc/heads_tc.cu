@@ -5,7 +5,8 @@
 // of attention_tc.cu (a loader warp, an MMA issuer, 128 softmax threads that own a row each, two CTAs per SM):
 //   S = Q K^T     both from shared memory (TMA boxes of 64 columns x 16, 32 or 64 tokens through the block table; columns past
 //                 a key's width are the tensor map's zero fill)
-//   softmax       row maximum, then exp2 of the scores (soft-capped first, where a cap is set); the reference maximum moves only when a row outgrew it by 2^8
+//   softmax       row maximum, then exp2 of the scores (soft-capped first, where a cap is set); the reference maximum moves
+//                 only when a row outgrew it by 2^8
 //   O += P V      P from TMEM in TWO bfloat16 terms, the weight and what rounding took from it, 64 columns each: together they
 //                 take the place of the 128 columns of scores; V is an MN-major operand as it lies in the cache
 // Tiles start at a multiple of the box, at or before the first key that the tile's first query sees; tiles of the tokens that
@@ -65,10 +66,10 @@ __device__ __forceinline__ uint64_t ht_desc_mn(uint32_t smem_addr) {
 
 // A cap bounds the scores: with one of up to kHtFixedCap the cap itself is the reference maximum of every row (weights down to
 // exp(-2 cap) are ordinary fp32 numbers), and a tile is read once.
-enum HtCap { kHtNoCap = 0, kHtCap = 1, kHtFixed = 2 };
+enum HtMode { kHtPlain = 0 /* no kept tokens, no cap */, kHtNoCap = 1, kHtCap = 2, kHtFixed = 3 };
 constexpr float kHtFixedCap = 40.f;
 
-template <int CAP>
+template <int MODE>
 __global__ void __launch_bounds__(kHtThreads, 2)
 heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                 const __grid_constant__ CUtensorMap map_v, const HtArgs a) {
@@ -88,10 +89,11 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
   const int p_first = a.q_pos0[seq] + qt * kHtRows, p_last = a.q_pos0[seq] + min(q_len, qt * kHtRows + kHtRows) - 1;
   const int br = a.box_rows;
   const int k_begin = a.h.first_seen(p_first) / br * br, k_end = p_last + 1;
-  const int kept_end = min(k_begin, (a.h.keep + br - 1) / br * br);          // kept tokens before the others, whole boxes
+  // kept tokens before the others, in whole boxes
+  const int kept_end = MODE == kHtPlain ? 0 : min(k_begin, (a.h.keep + br - 1) / br * br);
   const int kept = (kept_end + kHtKeys - 1) / kHtKeys, n_tiles = kept + (k_end - k_begin + kHtKeys - 1) / kHtKeys;
-  auto key_of = [&](int t) { return t < kept ? t * kHtKeys : k_begin + (t - kept) * kHtKeys; };
-  auto end_of = [&](int t) { return t < kept ? kept_end : k_end; };
+  auto key_of = [&](int t) { return MODE != kHtPlain && t < kept ? t * kHtKeys : k_begin + (t - kept) * kHtKeys; };
+  auto end_of = [&](int t) { return MODE != kHtPlain && t < kept ? kept_end : k_end; };
   const int* table = a.h.tables + size_t(seq) * a.h.max_blocks;
 
   if (threadIdx.x == 0) {
@@ -210,7 +212,10 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
     const int limit = a.q_pos0[seq] + row, lo = a.h.first_seen(limit);
     const uint32_t lane_addr = uint32_t(warp * 32) << 16;
     const float scale_log2 = a.h.scale * kLog2E;
-    auto log2_score = [&](float s) { return CAP != kHtNoCap ? a.h.capped(s * a.h.scale) * kLog2E : s * scale_log2; };
+    auto sees = [&](int k) { return MODE == kHtPlain ? k <= limit && k >= lo : a.h.sees(k, limit, lo); };
+    auto log2_score = [&](float s) {
+      return MODE == kHtCap || MODE == kHtFixed ? a.h.capped(s * a.h.scale) * kLog2E : s * scale_log2;
+    };
     const int o_cols = (a.h.vdim + 15) / 16 * 16;
     const float cap_in = 2.f * a.h.scale * kLog2E / a.h.cap, cap_out = -2.f * a.h.cap * kLog2E;        // kHtFixed
     float m_used = -INFINITY, l = 0.f;
@@ -228,11 +233,11 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
         break;
       }
       tc_fence_after_sync();
-      const bool full = __all_sync(0xffffffffu, groups == 0xFFu && (k0 >= lo || k0 + kHtKeys <= a.h.keep) &&
-                                                    k0 + kHtKeys - 1 <= limit);
+      const bool from_lo = k0 >= lo || (MODE != kHtPlain && k0 + kHtKeys <= a.h.keep);
+      const bool full = __all_sync(0xffffffffu, groups == 0xFFu && from_lo && k0 + kHtKeys - 1 <= limit);
       float mx = -INFINITY;
 #pragma unroll 1
-      for (int c = 0; CAP != kHtFixed && c < 4; ++c) {
+      for (int c = 0; MODE != kHtFixed && c < 4; ++c) {
         uint32_t v[32];
         ZSE_TMEM_LD_X16(v, tm_s + lane_addr + c * 32);
         ZSE_TMEM_LD_X16((v + 16), tm_s + lane_addr + c * 32 + 16);
@@ -249,7 +254,7 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int k = k0 + c * 32 + i;
-            const bool seen = ((groups >> (c * 2 + (i >> 4))) & 1u) && a.h.sees(k, limit, lo);
+            const bool seen = ((groups >> (c * 2 + (i >> 4))) & 1u) && sees(k);
             mx = seen ? fmaxf(mx, __uint_as_float(v[i])) : mx;
           }
         }
@@ -290,10 +295,10 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               float p0, p1;
-              if constexpr (CAP == kHtFixed) {     // cap tanh(s / cap) - cap = -2 cap / (1 + exp(2 s / cap))
-                p0 = ex2(__fdividef(cap_out, 1.f + ex2(__uint_as_float(v[2 * i]) * cap_in)));
-                p1 = ex2(__fdividef(cap_out, 1.f + ex2(__uint_as_float(v[2 * i + 1]) * cap_in)));
-              } else if constexpr (CAP == kHtCap) {
+              if constexpr (MODE == kHtFixed) {     // cap tanh(s / cap) - cap = -2 cap / (1 + exp(2 s / cap))
+                p0 = ex2(cap_out * rcp(1.f + ex2(__uint_as_float(v[2 * i]) * cap_in)));
+                p1 = ex2(cap_out * rcp(1.f + ex2(__uint_as_float(v[2 * i + 1]) * cap_in)));
+              } else if constexpr (MODE == kHtCap) {
                 p0 = ex2(log2_score(__uint_as_float(v[2 * i])) - m_ref);
                 p1 = ex2(log2_score(__uint_as_float(v[2 * i + 1])) - m_ref);
               } else {
@@ -303,8 +308,8 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
               if constexpr (!decltype(all)::value) {
                 const int k = k0 + c * 32 + b * 16 + 2 * i;
                 const bool there = (groups >> (c * 2 + b)) & 1u;
-                p0 = there && a.h.sees(k, limit, lo) ? p0 : 0.f;
-                p1 = there && a.h.sees(k + 1, limit, lo) ? p1 : 0.f;
+                p0 = there && sees(k) ? p0 : 0.f;
+                p1 = there && sees(k + 1) ? p1 : 0.f;
               }
               s0 += p0;
               s1 += p1;
@@ -357,7 +362,7 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               const float z = __uint_as_float(i & 1 ? two[i / 2] & 0xFFFF0000u : two[i / 2] << 16);
-              x[i] = __float_as_uint(__uint_as_float(x[i]) * sigmoid_exact(z));
+              x[i] = __float_as_uint(__uint_as_float(x[i]) * sigmoid_fast(z));
             }
           }
           w.x = pack_bf16(__uint_as_float(x[0]) * inv, __uint_as_float(x[1]) * inv);
@@ -395,14 +400,18 @@ int launch_heads_tc(const bf16* inp, int ld, int rows, const void* k, const void
   if (int rc = get_tmap_rows3(v, num_blocks, per_block, h.vp, h.block_stride, br, 0, &mv)) return rc;
   const HtArgs a{h, cu_q, q_pos0, first, out, ldo, gate, ld, br, (h.dim + 63) / 64, (h.vdim + 63) / 64, status};
   const size_t smem = size_t(2 * a.k_panels + a.v_panels) * kHtPanel + 1024 + sizeof(HtBars);
-  static bool done[3][kMaxDevices] = {};
-  const int slot = current_device_slot(), cap = h.cap <= 0.f ? kHtNoCap : h.cap <= kHtFixedCap ? kHtFixed : kHtCap;
-  auto kern = cap == kHtNoCap ? heads_tc_kernel<kHtNoCap> : cap == kHtCap ? heads_tc_kernel<kHtCap> : heads_tc_kernel<kHtFixed>;
-  if (!done[cap][slot]) {
+  static bool done[4][kMaxDevices] = {};
+  const int slot = current_device_slot();
+  const int mode = h.cap <= 0.f ? (h.keep > 0 ? kHtNoCap : kHtPlain) : h.cap <= kHtFixedCap ? kHtFixed : kHtCap;
+  auto kern = mode == kHtPlain   ? heads_tc_kernel<kHtPlain>
+              : mode == kHtNoCap ? heads_tc_kernel<kHtNoCap>
+              : mode == kHtCap   ? heads_tc_kernel<kHtCap>
+                                 : heads_tc_kernel<kHtFixed>;
+  if (!done[mode][slot]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              int(6 * kHtPanel + 1024 + sizeof(HtBars))) != cudaSuccess)
       return ZSE_ERR_LAUNCH;
-    done[cap][slot] = true;
+    done[mode][slot] = true;
   }
   return launch_pdl(kern, dim3((max_q + kHtRows - 1) / kHtRows, h.heads, last - first), dim3(kHtThreads), smem, st,
                     mq, mk, mv, a) == cudaSuccess

@@ -23,8 +23,8 @@ constexpr int kTopkWarps = 8;
 // Router rows are `cols` wide: column E, if there is one, is the shared expert's gate, whose sigmoid goes to shared_score.
 __global__ void __launch_bounds__(kTopkWarps * 32)
 moe_topk_kernel(const float* __restrict__ planes, int n_planes, int M, int E, int cols, int top, int softmax, int normalise,
-                float scale, int groups, int keep, int* __restrict__ counts, int* __restrict__ slot_expert, int* __restrict__ slot_rank,
-                float* __restrict__ slot_score, float* __restrict__ shared_score) {
+                float scale, int groups, int keep, int* __restrict__ counts, int* __restrict__ slot_expert,
+                int* __restrict__ slot_rank, float* __restrict__ slot_score, float* __restrict__ shared_score) {
   extern __shared__ float scores[];
   pdl_launch_dependents();
   pdl_wait();
@@ -364,7 +364,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
               const int col = ch * kCols + c + i;
               if (col < tile.rows && n < p.cols)
                 reinterpret_cast<OutT*>(p.out)[size_t(tile.row0 + col) * p.ldo + n] =
-                    from_f32<OutT>(glu(a.glu, __uint_as_float(r[i]), park[(c + i) * 32 + lane], p.limit));
+                    from_f32<OutT>(glu<true>(a.glu, __uint_as_float(r[i]), park[(c + i) * 32 + lane], p.limit));
             }
           }
         }

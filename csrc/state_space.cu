@@ -6,8 +6,8 @@
 // head; heads of a group share B and C.  The gated result is RMS-normed in equal parts (group_norm).
 //
 //   ss_prep     second half of the fused input projection [z | x | B | C | dt]: split-K sum, convolution, step sizes
-//   ss_tokens   token by token (decode, short portions, any shape, any type): a CTA per (columns of S, head, sequence) keeps its
-//               part of S in registers
+//   ss_tokens   token by token (decode, short portions, any shape, any type): a CTA per (columns of S, head, sequence) keeps
+//               its part of S in registers
 //   ss_chunk    chunks of 64 tokens (bfloat16): a CTA per (64 columns of S, head, sequence) keeps its part of S in accumulators
 //               and walks through the sequence
 //   group_norm  norm in parts and weight, in place
@@ -155,7 +155,7 @@ ss_prep_kernel(T* __restrict__ inp, T* __restrict__ xbc, const Space m, const Sp
         }
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) y.v[e] = silu_exact(y.v[e]);
+      for (int e = 0; e < 4; ++e) y.v[e] = sizeof(T) == 2 ? y.v[e] * sigmoid_fast(y.v[e]) : silu_exact(y.v[e]);
       store_vec<4>(xbc + size_t(t) * m.conv_width + c, y);
       const int place = t - (end - (taps - 1));
       if (last != nullptr && place >= 0) store_vec<4>(last + size_t(place) * m.conv_width, x);
@@ -278,7 +278,7 @@ ss_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ x
   uint8_t* ssl = ssh + ksteps * 16 * kCkPitch;
   uint8_t* sph = ssh;                            // in the same place: weighted scores, two terms
   uint8_t* spl = sph + kCkT * kCkPitch;
-  float* gb = reinterpret_cast<float*>(ssh + overlay_bytes(N));    // b_t
+  float* gb = reinterpret_cast<float*>(ssh + overlay_bytes(N));    // b_t, in units of ln 2
   float* gd = gb + kCkT;                         // dt_t
   float* ge = gd + kCkT;                         // exp(b_t)
   float* gw = ge + kCkT;                         // exp(b_end - b_t) dt_t
@@ -351,7 +351,7 @@ ss_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ x
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int t = lane * 2 + j;
-        gb[t] = bt[j];
+        gb[t] = bt[j] * kLog2E;
         gd[t] = d[j];
         ge[t] = expf(bt[j]);
         gw[t] = expf(bend - bt[j]) * d[j];
@@ -419,8 +419,8 @@ ss_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ x
 #pragma unroll
       for (int n = 0; n < 4; ++n) {
         const int c = pc * 32 + n * 8 + c2;
-        const float x = c <= t ? sc[n][h * 2] * gd[c] * expf(bt - gb[c]) : 0.f;
-        const float y = c + 1 <= t ? sc[n][h * 2 + 1] * gd[c + 1] * expf(bt - gb[c + 1]) : 0.f;
+        const float x = c <= t ? sc[n][h * 2] * gd[c] * ex2(bt - gb[c]) : 0.f;
+        const float y = c + 1 <= t ? sc[n][h * 2 + 1] * gd[c + 1] * ex2(bt - gb[c + 1]) : 0.f;
         *reinterpret_cast<uint32_t*>(sph + t * kCkPitch + c * 2) = pack_bf16(x, y);
         *reinterpret_cast<uint32_t*>(spl + t * kCkPitch + c * 2) = pack_bf16_rest(x, y);
         acc[n][h * 2] *= wi;
@@ -485,8 +485,8 @@ ss_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ x
         if (c >= nc) continue;
         const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sx + t * kCkPitch + c * 2));
         const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sz + t * kCkPitch + c * 2));
-        *reinterpret_cast<uint32_t*>(o + c) = pack_bf16(fmaf(D, x.x, acc[n][h * 2]) * silu_exact(z.x),
-                                                        fmaf(D, x.y, acc[n][h * 2 + 1]) * silu_exact(z.y));
+        *reinterpret_cast<uint32_t*>(o + c) = pack_bf16(fmaf(D, x.x, acc[n][h * 2]) * (z.x * sigmoid_fast(z.x)),
+                                                        fmaf(D, x.y, acc[n][h * 2 + 1]) * (z.y * sigmoid_fast(z.y)));
       }
     }
     __syncthreads();                             // everyone is done with the chunk's tiles

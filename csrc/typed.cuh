@@ -29,19 +29,35 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
 }
 
 __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
-__device__ __forceinline__ float gelu_tanh(float z) {
-  return 0.5f * z * (1.f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z)));
-}
-// gated activations of two products: kinds 0 clamped_glu, 1 silu(g) u, 2 gelu_tanh(g) u
-__device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
-  return kind == 0 ? clamped_glu(g, u, limit) : (kind == 1 ? silu_exact(g) : gelu_tanh(g)) * u;
-}
 
 // 2^x on the special-function unit: softmax weights need no more than its fp32 accuracy, and no range handling around it
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// 1 / x on the special-function unit, for normal x (infinity gives zero)
+__device__ __forceinline__ float rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// sigmoid on the special-function unit, within a few units in the last place of fp32
+__device__ __forceinline__ float sigmoid_fast(float z) { return rcp(1.f + ex2(z * -1.4426950408889634f)); }
+
+// Gated activations of two products: kinds 0 clamped_glu, 1 silu(g) u, 2 gelu(g) u with the tanh form of gelu, which is
+// z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3)).  FAST: the special-function unit's sigmoid, for results in bfloat16.
+template <bool FAST>
+__device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
+  if (kind == 0 && !FAST) return clamped_glu(g, u, limit);
+  if (kind == 0) {
+    g = fminf(g, limit);
+    return g * sigmoid_fast(1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  }
+  const float z = kind == 1 ? g : 1.5957691216057308f * (g + 0.044715f * g * g * g);
+  return g * (FAST ? sigmoid_fast(z) : sigmoid_exact(z)) * u;
 }
 
 __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {

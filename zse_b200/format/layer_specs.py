@@ -288,8 +288,8 @@ def _windowed_attention(m: dict) -> HeadsSpec:
     mask, rot = m.get("mask") or {}, m.get("rot") or {}
     return HeadsSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
                      window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0), gate_each=True,
-                     softcap=float(m.get("softcap") or 0.0), k_as_v=True, learned_norm=False, rot_dims=int(rot.get("dims") or 0),
-                     rot_base=float(rot.get("base", 10000.0)))
+                     softcap=float(m.get("softcap") or 0.0), k_as_v=True, learned_norm=False,
+                     rot_dims=int(rot.get("dims") or 0), rot_base=float(rot.get("base", 10000.0)))
 
 
 def _state_space(m: dict) -> StateSpaceSpec:

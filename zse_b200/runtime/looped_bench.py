@@ -115,8 +115,9 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
         for name, key, s, L, like in (("norms, bias, temperature, cache write", "full", full, L_full, "norms, cache write"),
                                       ("norms, rotation, cache write", "win", win, L_win, "norms, cache write"),
                                       ("norms, cache write", "at", n_at, L_at, None)):
-            add(phase, name, like, lambda k=key, s=s, L=L: ops.heads_prep(inp[k], pv(s.in_width), n_pl, kv[k], slots, L, s, 1e-6,
-                                                                          M, positions), moved(s))
+            add(phase, name, like,
+                lambda k=key, s=s, L=L: ops.heads_prep(inp[k], pv(s.in_width), n_pl, kv[k], slots, L, s, 1e-6, M, positions),
+                moved(s))
         xbc, dt = rnd(M, sp.conv_width), zeros(M, sp.heads)
         add(phase, "convolution, step sizes", "norms, cache write",
             lambda: ops.state_space_prep(inp["sp"], pv(sp.in_width), n_pl, side, xbc, dt, state, 0, rows, row_seq, cu, L_sp, sp,
@@ -126,7 +127,8 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
         gates, gp = zeros(M * 2 * n_mem.heads), zeros(8, M * 2 * n_mem.heads)
         out = {k: rnd(M, s.heads * s.vdim) for k, s in (("full", full), ("win", win), ("sp", sp), ("at", n_at), ("mem", n_mem))}
         seen = lambda s, p: min(p + 1, s.window + s.keep_first) if s.window else p + 1
-        sp_io, mem_io = 2.0 * M * (sp.conv_width + 2 * sp.inner) + 4.0 * M * sp.heads, 2.0 * M * (n_mem.if_col + n_mem.heads * n_mem.vdim)
+        sp_io = 2.0 * M * (sp.conv_width + 2 * sp.inner) + 4.0 * M * sp.heads
+        mem_io = 2.0 * M * (n_mem.if_col + n_mem.heads * n_mem.vdim)
         if dec:
             for name, key, s, like in (("attention rows", "full", full, "chunked attention rows"),
                                        ("windowed attention rows", "win", win, "chunked attention rows"),
@@ -135,8 +137,8 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
                 scratch = zeros(M * splits * s.heads * (s.vdim + 2))
                 n = seen(s, ctx - 1)
                 add(phase, name, like,
-                    lambda k=key, s=s, sc=scratch, n=splits: ops.heads_attn(inp[k], kv[k], tables, None, positions, out[k], M, s,
-                                                                            sc, n),
+                    lambda k=key, s=s, sc=scratch, sp_=splits: ops.heads_attn(inp[k], kv[k], tables, None, positions, out[k],
+                                                                              M, s, sc, sp_),
                     2.0 * M * (n * s.row + s.heads * (s.dim + s.vdim) + s.gate_width),
                     2.0 * M * n * s.heads * (s.dim + s.vdim))
             add(phase, "state space step", "memory step",
@@ -152,18 +154,19 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
                                        ("chunked attention tiles", "at", n_at, None)):
                 pairs = chunks * sum(seen(s, p) for p in range(chunk))
                 add(phase, name, like,
-                    lambda k=key, s=s: ops.heads_attn_chunks(inp[k], kv[k], ctab, cu, p0, positions, 0, chunks, chunk, out[k], s),
+                    lambda k=key, s=s: ops.heads_attn_chunks(inp[k], kv[k], ctab, cu, p0, positions, 0, chunks, chunk, out[k],
+                                                             s),
                     2.0 * M * (s.in_width + s.heads * s.vdim), 2.0 * pairs * s.heads * (s.dim + s.vdim))
             ws = ops.memory_workspace([n_mem], M)
             add(phase, "state space in chunks", "memory in chunks",
                 lambda: ops.state_space_chunks(inp["sp"], xbc, dt, state, 0, rows, cu, L_sp, out["sp"], 0, chunks, M, sp),
                 sp_io + 8.0 * S * sp.heads * sp.state * sp.vdim, 4.0 * M * sp.heads * sp.state * sp.vdim)
             add(phase, "memory in chunks", None,
-                lambda: ops.memory_chunks(inp["mem"], gates, state, 0, rows, cu, L_mem, out["mem"], 0, chunks, 0, M, n_mem, 1e-6,
-                                          ws), mem_io + 8.0 * S * n_mem.state_floats,
+                lambda: ops.memory_chunks(inp["mem"], gates, state, 0, rows, cu, L_mem, out["mem"], 0, chunks, 0, M, n_mem,
+                                          1e-6, ws), mem_io + 8.0 * S * n_mem.state_floats,
                 4.0 * M * n_mem.heads * n_mem.dim * n_mem.vdim)
-        add(phase, "norm in parts", "norm + residual", lambda: ops.group_norm(out["sp"], L_sp.out_norm, sp.norm_groups, M, 1e-6),
-            4.0 * M * sp.inner)
+        add(phase, "norm in parts", "norm + residual",
+            lambda: ops.group_norm(out["sp"], L_sp.out_norm, sp.norm_groups, M, 1e-6), 4.0 * M * sp.inner)
         add(phase, "output projection (state space)", "output projection",
             lambda: ops.linear_partial(o["sp"], out["sp"], M, pv(H)), *mm(H, sp.inner))
         add(phase, "output projection", None, lambda: ops.linear_partial(o["at"], out["at"], M, pv(H)),
@@ -199,7 +202,8 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
             ops.moe(L, x, M, ws)                           # tables for the single kernels below
             tile = ops.n.moe_tile_rows(M, e.experts, e.top)
             add(phase, "router logits" + sfx, like("router logits"),
-                lambda L=L, e=e, ws=ws: ops.linear_partial(L.router, x, M, ws.router_views[e.router_rows]), *mm(e.router_rows, H))
+                lambda L=L, e=e, ws=ws: ops.linear_partial(L.router, x, M, ws.router_views[e.router_rows]),
+                *mm(e.router_rows, H))
             add(phase, "routing, sorted rows" + sfx, like("routing, sorted rows"),
                 lambda e=e, ws=ws, tile=tile, per=per: ops.n.moe_route(ws.router, 1, M, e, tile, x, H, per, ws),
                 4.0 * M * e.top * H)
@@ -214,7 +218,8 @@ def kernel_table(shape: str, iters: int = 20, seqs: int = 64, ctx: int = 4096, c
         del planes, inp, out
         torch.cuda.empty_cache()
     logits = zeros(seqs, c.vocab_size)
-    add("decode", "logit scale", "norm + residual", lambda: ops.logits_finish(logits, seqs, 0.5, 0.0), 8.0 * seqs * c.vocab_size)
+    add("decode", "logit scale", "norm + residual", lambda: ops.logits_finish(logits, seqs, 0.5, 0.0),
+        8.0 * seqs * c.vocab_size)
     ops.check()
     by = {(x["phase"], x["kernel"]): x for x in T.rows}
     for x in T.rows:
