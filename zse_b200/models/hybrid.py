@@ -1,5 +1,6 @@
-"""Decoders whose layers mix attention over heads and recurrent matrix memories, with norms on the sublayers' outputs
-(Nimelorn), over the paged cache and the state slots.
+"""Decoders whose layers mix attention over heads and recurrent mixers (matrix memories, state spaces), over the paged cache
+and the state slots: layer runs, mixers, feed-forwards, and the placement of norms on the sublayers' outputs (Nimelorn).
+``looped`` has the other placement.
 
 Same pass contract as ``DecoderModel``.  The residual x is fp32; sublayers read x itself (rounded to the activations' type):
 
@@ -12,7 +13,8 @@ Attention caches normed keys and values as [kv head][token][dim] tiles of a bloc
 and values projects queries only.  Rows that decode, and chunks of at most ``SHORT_CHUNK`` tokens, run a row at a time with
 the keys split over CTAs; longer chunks run in tiles of queries.  A matrix memory does the same: short chunks step through
 the state token by token, with read-out, head norm and output gate in the step's kernel; longer ones run chunkwise, with the
-decays inside a chunk as a lower-triangular matrix.  A packed pass may hold both kinds: short ones are laid out first.
+decays inside a chunk as a lower-triangular matrix.  A state space passes its inputs through a short convolution first, whose
+last inputs are part of its state, and does the same.  A packed pass may hold both kinds: short ones are laid out first.
 
 A sequence's recurrent state and its last token live in ``cache.state_slots``; ``state_rows`` names the rows that a pass's
 sequences read and write.
