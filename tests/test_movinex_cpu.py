@@ -238,7 +238,7 @@ def test_choice_of_experts():
     for experts, top, groups, keep in ((15, 3, 5, 2), (8, 4, 2, 1), (9, 3, 9, 4), (10, 3, 1, 1), (6, 2, 3, 3)):
         m = MoESpec(experts, top, 8, activation="silu_glu", weigh="output", groups=groups, keep_groups=keep)
         z = torch.randn(200, experts, generator=g)
-        z[:50] = z[:50].round()                        # ties
+        z[:50] = z[:50].round().abs()                  # ties
         ids, w = ref.route(z, m)
         s = torch.sigmoid(z)
         for t in range(200):
