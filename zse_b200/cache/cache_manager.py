@@ -81,7 +81,7 @@ class KVCacheManager:
         if config.keeps_state:
             self.states = StateSlots(state_slots or 64, config.state_floats, device)
             enable_dedup = False         # a shared prefix has no recurrent state to start from
-        self._page_table = PageTable(self._pool)
+        self._page_table = PageTable(self._pool, config.pool_step)
         self._evictor = Evictor(eviction_policy)
         self._dedup = BlockDedup(self._pool) if enable_dedup else None
         self._prompt_lengths: Dict[int, int] = {}
@@ -127,7 +127,7 @@ class KVCacheManager:
                     shared.append(bid)
                     prev = h
             fresh_tokens = n - len(shared) * bs
-            need = (fresh_tokens + bs - 1) // bs
+            need = (fresh_tokens + bs - 1) // bs + self._page_table.mean_blocks(n)
             if need > self._pool.num_free and not self._evict_locked(need):
                 raise RuntimeError(f"cannot allocate {need} KV blocks for sequence {seq_id}: "
                                    f"{self._pool.num_free} free and eviction did not help")
@@ -209,13 +209,14 @@ class KVCacheManager:
         neither the pool nor the evictor."""
         errs = [None] * len(seq_ids)
         bs, limit = self._block_size, self._config.max_seq_len
-        windowed = self._windowed
+        windowed, step = self._windowed, self._config.pool_step
         with self._lock:
             for i, sid in enumerate(seq_ids):
                 e = self._page_table.get_entry_or_none(sid)
                 n = e.num_tokens if e is not None else 0
-                # (the step that moves the first position seen over a block border gives blocks back: ordinary path)
-                if e is not None and (not windowed or self._config.first_seen(n) // bs
+                # (the step that moves the first position seen over a block border gives blocks back, one that completes the
+                # tokens of a mean may need a block for it: ordinary path)
+                if e is not None and (not step or (n + 1) % step) and (not windowed or self._config.first_seen(n) // bs
                                       == self._config.first_seen(max(0, n - 1)) // bs):
                     fill = n % bs
                     if fill and n < limit and e.blocks:
@@ -280,6 +281,7 @@ class KVCacheManager:
                     tail.num_tokens = keep_tokens - (keep_blocks - 1) * bs
                     if self._dedup is not None and tail.num_tokens < bs:
                         self._dedup.deregister_block(tail.block_id)
+            self._page_table.truncate_means(e, keep_tokens)
             e.num_tokens = keep_tokens
             self._registered_upto[seq_id] = min(self._registered_upto.get(seq_id, 0), keep_tokens // bs)
 
@@ -343,16 +345,26 @@ class KVCacheManager:
         with self._lock:
             return self._page_table.block_ids_np(seq_id)
 
+    def mean_block_ids(self, seq_id: int) -> List[int]:
+        """The blocks that hold the sequence's block means, in order."""
+        with self._lock:
+            return [b.block_id for b in self._page_table.get_entry(seq_id).means]
+
+    def mean_blocks(self, num_tokens: int) -> int:
+        """Blocks that the means of a sequence of ``num_tokens`` tokens fill."""
+        return self._page_table.mean_blocks(num_tokens)
+
     def stage_states(self, spans, read, write) -> None:
         """``spans``: (seq_id, start, tokens) of a pass's sequences; fills the rows of ``states`` they read and write."""
         with self._lock:
             for s, (sid, start, n) in enumerate(spans):
                 read[s], write[s] = self.states.advance(sid, start, n)
 
-    def stage_decode(self, seq_ids, block_tables, seq_lens, positions, slots) -> int:
+    def stage_decode(self, seq_ids, block_tables, seq_lens, positions, slots, means_at: int = 0) -> int:
         """Fills the decode-step arrays (numpy views of the runner's pinned staging buffers) for ``seq_ids`` in one
-        pass: block table rows (-1 padded), lengths, the position of each sequence's newest token and the cache slot
-        that token is written to (-1 when its block was evicted).  Returns the longest sequence length."""
+        pass: block table rows (-1 padded; the blocks of means from column ``means_at`` on), lengths, the position of
+        each sequence's newest token and the cache slot that token is written to (-1 when its block was evicted).
+        Returns the longest sequence length."""
         S = len(seq_ids)
         bs = self._block_size
         with self._lock:
@@ -364,6 +376,8 @@ class KVCacheManager:
             for s, e in enumerate(entries):
                 ids = e.block_ids_np()
                 block_tables[s, :ids.shape[0]] = ids
+                if e.means:
+                    block_tables[s, means_at: means_at + len(e.means)] = [b.block_id for b in e.means]
             seq_lens[:S] = [e.num_tokens for e in entries]
         n = seq_lens[:S]
         last = n - 1

@@ -3,6 +3,9 @@
 
 An evicted block leaves a hole: its index stays in the sequence (the block table carries -1 there and attention
 skips it) and the tokens it held no longer count as cached.
+
+Sequences of models that also attend to means of blocks of tokens own further blocks of the pool whose rows hold those
+means, one per ``pool_step`` whole tokens; they stay when the tokens' blocks leave.
 """
 from __future__ import annotations
 
@@ -21,6 +24,7 @@ class SequenceEntry:
     num_tokens: int = 0                      # logical length (positions 0..num_tokens-1), holes included
     evicted_indices: Set[int] = field(default_factory=set)
     tokens_evicted: int = 0
+    means: List[Block] = field(default_factory=list)     # blocks that hold means of tokens
     version: int = 0                         # bumped by every change of `blocks` / `evicted_indices`
     _ids_np: Optional[np.ndarray] = field(default=None, repr=False, compare=False)
     _ids_version: int = field(default=-1, repr=False, compare=False)
@@ -47,8 +51,9 @@ class SequenceEntry:
 
 
 class PageTable:
-    def __init__(self, pool: BlockPool):
+    def __init__(self, pool: BlockPool, pool_step: int = 0):
         self._pool = pool
+        self._step = pool_step
         self._seqs: Dict[int, SequenceEntry] = {}
 
     def create_sequence(self, seq_id: int) -> SequenceEntry:
@@ -67,13 +72,40 @@ class PageTable:
     def get_entry_or_none(self, seq_id: int) -> Optional[SequenceEntry]:
         return self._seqs.get(seq_id)
 
+    def mean_blocks(self, num_tokens: int) -> int:
+        """Blocks that the means of ``num_tokens`` tokens fill."""
+        bs = self._pool.block_size_tokens
+        return (num_tokens // self._step + bs - 1) // bs if self._step else 0
+
+    def _copies_mean_tail(self, e: SequenceEntry, num_tokens: int) -> bool:
+        """Whether growing to ``num_tokens`` writes into a block of means that another sequence shares."""
+        if not e.means or not e.means[-1].is_shared:
+            return False
+        rows = e.num_tokens // self._step
+        return num_tokens // self._step > rows and len(e.means) * self._pool.block_size_tokens > rows
+
+    def _grow_means(self, e: SequenceEntry, num_tokens: int) -> None:
+        if self._copies_mean_tail(e, num_tokens):
+            fresh, tail = self._pool.alloc(e.seq_id), e.means[-1]
+            self._pool.copy_block(tail, fresh)
+            self._pool.free(tail)
+            e.means[-1] = fresh
+        while len(e.means) < self.mean_blocks(num_tokens):
+            e.means.append(self._pool.alloc(e.seq_id))
+
+    def truncate_means(self, e: SequenceEntry, num_tokens: int) -> None:
+        while len(e.means) > self.mean_blocks(num_tokens):
+            self._pool.free(e.means.pop())
+
     def blocks_needed(self, seq_id: int, num_new_tokens: int) -> int:
         e = self._seqs[seq_id]
         bs = self._pool.block_size_tokens
+        total = e.num_tokens + num_new_tokens
         need = (e.num_tokens + num_new_tokens + bs - 1) // bs - len(e.blocks)
         tail_shared = bool(e.blocks) and e.num_tokens % bs != 0 and (len(e.blocks) - 1) not in e.evicted_indices \
             and e.blocks[-1].is_shared
-        return max(0, need) + int(tail_shared)
+        means = max(0, self.mean_blocks(total) - len(e.means)) + int(self._copies_mean_tail(e, total))
+        return max(0, need) + int(tail_shared) + means
 
     def append_tokens(self, seq_id: int, num_tokens: int) -> List[int]:
         """Grows the sequence; returns ids of newly allocated blocks.  A partly filled shared tail block is copied
@@ -81,6 +113,8 @@ class PageTable:
         e = self._seqs[seq_id]
         bs = self._pool.block_size_tokens
         new_ids: List[int] = []
+        if self._step:
+            self._grow_means(e, e.num_tokens + num_tokens)
         remaining = num_tokens
         while remaining > 0:
             if len(e.blocks) * bs <= e.num_tokens:          # every block so far is full
@@ -131,6 +165,7 @@ class PageTable:
         for i, b in enumerate(e.blocks):
             if i not in e.evicted_indices and self._pool.free(b):
                 released.append(b)
+        released += [b for b in e.means if self._pool.free(b)]
         return released
 
     def fork_sequence(self, src_id: int, dst_id: int) -> SequenceEntry:
@@ -140,6 +175,9 @@ class PageTable:
             if i not in src.evicted_indices:
                 self._pool.increment_ref(b)
             dst.blocks.append(b)
+        for b in src.means:
+            self._pool.increment_ref(b)
+        dst.means = list(src.means)
         dst.num_tokens = src.num_tokens
         dst.evicted_indices = set(src.evicted_indices)
         dst.touch()

@@ -41,6 +41,7 @@ class EngineConfig:
     headroom_ratio: float = 0.5
     kv_fraction: Optional[float] = None   # share of free memory for the KV cache (None = demand rule)
     kv_blocks: int = 0                    # explicit KV block count (tests)
+    kv_tokens: int = 0                    # or: tokens the cache holds, whole blocks counted, with what a model keeps beside them
     state_slots: int = 0                  # sequences with recurrent state at a time (0 = the batch, and one for retrieval)
     eviction_policy: str = "smart"
     enable_prefix_cache: bool = True

@@ -118,6 +118,8 @@ class ZStreamerEngine:
         slots = cfg.state_slots or cfg.max_batch_seqs + 1
         if cfg.kv_blocks > 0:
             blocks = cfg.kv_blocks
+        elif cfg.kv_tokens > 0:
+            blocks = mc.cache_blocks(cfg.kv_tokens, cfg.max_batch_seqs, block_size)
         elif on_gpu:
             scratch_est = cfg.max_batch_tokens * (mc.hidden_size * 40 + mc.intermediate_size * 2) + (256 << 20)
             if mc.keeps_state:
@@ -137,7 +139,7 @@ class ZStreamerEngine:
                                    logits_rows=cfg.logits_rows)
         from .lora.manager import LoRAManager
         self._lora_manager = LoRAManager(self._model, self.device)
-        self._budget = MemoryBudget(blocks, block_size, cfg.headroom_ratio)
+        self._budget = MemoryBudget(blocks, block_size, cfg.headroom_ratio, mean_step=mc.pool_step)
         self._sched_config = SchedulerConfig(cfg.max_batch_tokens, cfg.max_batch_seqs, cfg.max_prefill_per_step,
                                              cfg.prefill_chunk_size, cfg.decode_per_prefill, cfg.enable_preemption,
                                              cfg.speculative_k, cfg.max_queue_size, cfg.speculative_mode)

@@ -6,7 +6,7 @@ keep-list, name-sorted load order and basic shape sanity warnings.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Type
+from typing import Dict, List, Tuple, Type
 
 from ..config import ModelConfig
 from ..spec import should_quantize as _default_should_quantize
@@ -78,6 +78,9 @@ class ArchAdapter:
     def config_from_hf(self, hf_config: dict) -> ModelConfig:
         hf = hf_config
         raise NotImplementedError
+
+    def sizes_of_tensors(self, config: ModelConfig, shapes: Dict[str, Tuple[int, ...]]) -> None:
+        """Completes ``config`` by sizes that only the tensors' shapes give."""
 
     def _common(self, hf: dict, arch: str, *, max_seq: int, theta: float, eps: float, tie: bool,
                 explicit_head_dim: bool) -> ModelConfig:

@@ -11,8 +11,8 @@ from dataclasses import dataclass, field, fields
 from typing import Any, Dict, List, Optional
 
 from . import serializer
-from .layer_specs import (DenseSpec, HeadsSpec, LatentSpec, LayerSpec, MatrixMemorySpec, MoESpec,  # noqa: F401
-                          RECURRENT, StateSpaceSpec, read_ff, read_mixer)
+from .layer_specs import (DenseSpec, GatedLinearSpec, HeadsSpec, LatentSpec, LayerSpec, MatrixMemorySpec,  # noqa: F401
+                          MoESpec, StateSpaceSpec, TwinSpec, attention_of, read_ff, read_mixer, recurrent_of)
 from .spec import DEFAULT_GROUP_SIZE, DEFAULT_QUANT_BITS, QuantMethod
 
 
@@ -72,8 +72,10 @@ class ModelConfig:
     embed_multiplier: Optional[float] = None
     # {"bigram": {"buckets", "mul_prev", "mul_cur"}, "sinusoid_base", "norm"}: what is added to a token's embedding
     embed_design: Optional[Dict[str, Any]] = None
-    # {"start", "stop", "times"}: these layers run several times in a row, each pass from [x; embedding]
+    # {"start", "stop", "times"}: these layers run several times in a row
     loop: Optional[Dict[str, int]] = None
+    # taps of a causal convolution over what the mixers read, whose last inputs are part of a sequence's state
+    input_conv: Optional[int] = None
     logit_scale: Optional[float] = None
     weight_dtype: Optional[str] = None
     multimodal: Optional[Dict[str, Any]] = None
@@ -150,7 +152,7 @@ class ModelConfig:
         return self.is_design and not self.is_latent
 
     def mixer_spec(self, i: int):
-        """``HeadsSpec`` or one of ``RECURRENT`` of layer ``i`` of a hybrid design."""
+        """``HeadsSpec``, ``TwinSpec`` or a recurrent mixer's of layer ``i`` of a hybrid design."""
         return read_mixer(self.arch, self.design_layers[i])
 
     def ff_spec(self, i: int):
@@ -168,8 +170,8 @@ class ModelConfig:
         return list(range(loop["start"])) + body * loop["times"] + list(range(loop["stop"], n))
 
     def enters_loop(self, run: int) -> bool:
-        """Whether layer run ``run`` is the first of a pass of the loop."""
-        if not self.loop:
+        """Whether layer run ``run`` is the first of a pass of a loop whose passes start from [x; embedding]."""
+        if not self.loop or not self.loop_rejoins:
             return False
         at, body = run - self.loop["start"], self.loop["stop"] - self.loop["start"]
         return 0 <= at < body * self.loop["times"] and at % body == 0
@@ -179,22 +181,25 @@ class ModelConfig:
         """Layer run -> its layer of the cache pool; runs without keys and values of their own have none."""
         if not self.is_hybrid:
             return {i: i for i in range(self.num_layers)}
-        own = [r for r, i in enumerate(self.layer_runs) if isinstance(self.mixer_spec(i), HeadsSpec)
-               and self.mixer_spec(i).own_kv]
-        return {r: n for n, r in enumerate(own)}
+        specs = [attention_of(self.mixer_spec(i)) for i in self.layer_runs]
+        return {r: n for n, r in enumerate(r for r, s in enumerate(specs) if s is not None and s.own_kv)}
 
     @property
     def num_cache_layers(self) -> int:
         return max(1, len(self.cache_layers))
 
     def _state_layout(self):
-        out, at = {}, 0
+        out, inputs, at = {}, {}, 0
+        kept = max(0, (self.input_conv or 1) - 1) * self.hidden_size
         for r, i in enumerate(self.layer_runs if self.is_hybrid else ()):
-            s = self.mixer_spec(i)
-            if isinstance(s, RECURRENT):
+            s = recurrent_of(self.mixer_spec(i))
+            if s is not None:
                 out[r] = at
                 at += (s.state_floats + 3) // 4 * 4
-        return out, at
+            if kept:
+                inputs[r] = at
+                at += (kept + 3) // 4 * 4
+        return out, inputs, at
 
     @property
     def state_offsets(self) -> Dict[int, int]:
@@ -202,8 +207,13 @@ class ModelConfig:
         return self._state_layout()[0]
 
     @property
-    def state_floats(self) -> int:
+    def input_offsets(self) -> Dict[int, int]:
+        """Layer run -> where a sequence's state holds the last inputs of its ``input_conv``, the oldest first."""
         return self._state_layout()[1]
+
+    @property
+    def state_floats(self) -> int:
+        return self._state_layout()[2]
 
     @property
     def keeps_state(self) -> bool:
@@ -237,8 +247,8 @@ class ModelConfig:
 
     def _masks(self) -> List[HeadsSpec]:
         if self.__dict__.get("_mask_specs") is None:
-            self.__dict__["_mask_specs"] = list({(s.chunk, s.window, s.keep_first): s for s in (
-                self.mixer_spec(i) for i in range(self.num_layers)) if isinstance(s, HeadsSpec)}.values())
+            self.__dict__["_mask_specs"] = list({(s.chunk, s.window, s.keep_first, s.pool): s for s in (
+                attention_of(self.mixer_spec(i)) for i in range(self.num_layers)) if s is not None}.values())
         return self.__dict__["_mask_specs"]
 
     @property
@@ -247,12 +257,29 @@ class ModelConfig:
         return max((s.keep_first for s in self._masks()), default=0) if self.is_hybrid else 0
 
     def first_seen(self, position: int) -> int:
-        """First position that some layer still sees from ``position`` (and from any later one), apart from the
-        ``kept_first`` ones: the cache may give back the blocks between."""
+        """First position that some layer still sees from ``position`` (and from any later one), or needs for the mean of a
+        block, apart from the ``kept_first`` ones: the cache may give back the blocks between."""
         if self.is_hybrid:
-            return min((s.first_seen(position) for s in self._masks()), default=position)
+            return min((s.first_needed(position) for s in self._masks()), default=position)
         w = self.cache_window
         return max(0, position + 1 - w) if w > 0 else 0
+
+    @property
+    def pool_step(self) -> int:
+        """Tokens of the smallest block whose mean some layer caches; 0: no layer does."""
+        return min((s.pool for s in self._masks() if s.pool > 0), default=0) if self.is_hybrid else 0
+
+    def mean_rows(self, tokens: int) -> int:
+        """Rows of block means that a sequence of ``tokens`` tokens has in the cache."""
+        return tokens // self.pool_step if self.pool_step else 0
+
+    def cache_blocks(self, tokens: int, sequences: int, block_size: int) -> int:
+        """Blocks of a cache pool for up to ``tokens`` tokens (whole blocks of every sequence counted) of up to ``sequences``
+        sequences, with their block means."""
+        n = (tokens + block_size - 1) // block_size
+        if self.pool_step:
+            n += self.mean_rows(tokens) // block_size + sequences
+        return n
 
     # ---- per-layer attention geometry (Gemma-family models mix layer kinds) -----------------------
     @property
@@ -269,6 +296,16 @@ class ModelConfig:
     def norms_outputs(self) -> bool:
         """Hybrid designs: norms sit on the sublayers' outputs, not on their inputs."""
         return self.arch == "nimelorn"
+
+    @property
+    def side_by_side(self) -> bool:
+        """Hybrid designs: a layer's sublayers read one norm and their results are added together."""
+        return self.arch == "vobisun"
+
+    @property
+    def loop_rejoins(self) -> bool:
+        """Hybrid designs: a pass of the loop starts from a product of x and the embedding."""
+        return self.arch == "movinex"
 
     def layer_kind(self, i: int) -> str:
         if self.layer_types and i < len(self.layer_types):
@@ -303,7 +340,7 @@ class ModelConfig:
         if self.is_latent:
             return 1, max(self.latent_spec(i).row for i in range(self.num_layers))
         if self.is_hybrid:
-            rows = [self.mixer_spec(i).row for i in range(self.num_layers) if isinstance(self.mixer_spec(i), HeadsSpec)]
+            rows = [s.row for s in (attention_of(self.mixer_spec(i)) for i in range(self.num_layers)) if s is not None]
             return 1, max(rows, default=8)
         local = num_kv_heads or self.num_kv_heads
         tp = max(1, self.num_kv_heads // max(1, local))
@@ -317,12 +354,12 @@ class ModelConfig:
             n = 0
             for i in range(self.num_layers):
                 a, m = self.mixer_spec(i), self.ff_spec(i)
-                n += self.hidden_size * (a.in_width + a.heads * a.vdim)
+                n += self.hidden_size * (a.in_width + a.out_width)
                 if isinstance(m, MoESpec):
                     n += self.hidden_size * (m.router_rows + 3 * m.experts * m.ff + 3 * m.shared_ff)
                 elif m is not None:
                     n += self.hidden_size * (3 if m.gated else 2) * m.ff
-            return n + (2 * self.hidden_size ** 2 if self.loop else 0)
+            return n + (2 * self.hidden_size ** 2 if self.loop and self.loop_rejoins else 0)
         if self.is_latent:
             n = 0
             for i in range(self.num_layers):

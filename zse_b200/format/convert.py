@@ -194,6 +194,7 @@ def convert_hf_to_zse(model_dir: str, output_path: str,
         if not quiet:
             print(f"WARNING: {warning}")
     tensor_map = build_tensor_map(find_safetensor_files(model_dir))
+    adapter.sizes_of_tensors(cfg, {adapter.map_tensor_name(n): tuple(t[1]["shape"]) for n, t in tensor_map.items()})
     tok_bytes = None
     if not skip_tokenizer and os.path.exists(os.path.join(model_dir, "tokenizer.json")):
         tok_bytes = BPETokenizer.from_hf_dir(model_dir).serialize()

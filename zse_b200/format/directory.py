@@ -49,6 +49,7 @@ class DirectoryLoader(ZSELoader):
             n = int(np.prod(shape, dtype=np.int64)) if shape else 1
             self._weight_index.add(WeightEntry(stored, shape, dtype, data_nbytes=n * _WIDTH[dtype]))
             self._source[stored] = src
+        adapter.sizes_of_tensors(self._config, {e.name: e.shape for e in self._weight_index})
         missing = [t for t in adapter.expected_tensors(self._config) if t not in self._weight_index] \
             if self._config.is_design else []
         if missing:

@@ -2,7 +2,7 @@
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Dict, Optional
+from typing import Dict, Optional, Union
 
 
 @dataclass
@@ -110,7 +110,7 @@ class DenseSpec:
 @dataclass(frozen=True)
 class HeadsSpec:
     """Attention of ``heads`` query heads over ``kv_heads`` key/value heads whose widths may differ.  Queries and keys are
-    normed per head."""
+    normed, per head after a rotation or all heads together before it."""
     heads: int
     kv_heads: int
     dim: int
@@ -130,6 +130,13 @@ class HeadsSpec:
     rot_base: float = 10000.0
     temp_coef: float = 0.0       # a query at p is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
     temp_every: int = 1
+    pool: int = 0                # > 0, with a window: what left it is seen as means of blocks of that many tokens, once all
+    #                              of a block has left
+    sink: bool = False           # the softmax has one more score per head, learned, without a value
+    head_temp: bool = False      # a learned factor of the scores per head
+    whole_norm: bool = False     # one query (key) norm over the rows of all heads, before the rotation
+    rot_factor: float = 1.0      # the rotation is slower by this factor
+    out_scale: float = 1.0       # factor of the result
 
     @property
     def own_kv(self) -> bool:
@@ -167,6 +174,21 @@ class HeadsSpec:
             return position // self.chunk * self.chunk
         return max(0, position + 1 - self.window) if self.window > 0 else 0
 
+    def blocks_seen(self, position: int) -> int:
+        """Blocks of ``pool`` tokens whose means the token at ``position`` sees: the first ones, all of whose tokens lie
+        before its window."""
+        return max(0, position + 1 - self.window) // self.pool if self.pool > 0 else 0
+
+    def first_needed(self, position: int) -> int:
+        """First position whose key and value a pass from ``position`` on reads: a block that is not complete yet still
+        needs its tokens for the mean, wherever the window begins."""
+        first = self.first_seen(position)
+        return min(first, position // self.pool * self.pool) if self.pool > 0 else first
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
 
 @dataclass(frozen=True)
 class MatrixMemorySpec:
@@ -176,6 +198,10 @@ class MatrixMemorySpec:
     dim: int
     vdim: int
     gate_cap: float
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
 
     # columns of the fused input projection [q | k | v | output gate | input and forget gates]
     @property
@@ -228,6 +254,10 @@ class StateSpaceSpec:
     def inner(self) -> int:
         return self.heads * self.vdim
 
+    @property
+    def out_width(self) -> int:
+        return self.inner
+
     # columns of the fused input projection [z | x | B | C | step sizes]; x, B and C are the channels of the convolution,
     # whose output keeps their layout from column 0 on
     @property
@@ -264,7 +294,89 @@ class StateSpaceSpec:
         return self.conv_at + (self.conv - 1) * self.conv_width
 
 
-RECURRENT = (MatrixMemorySpec, StateSpaceSpec)
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    """Recurrent mixer whose heads keep a [dim, vdim] matrix whose rows, one per key channel, decay each at its own rate
+    (gated linear attention).  The decays' logarithms come from a projection of low rank, divided by ``tau``."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int                    # of the projection that makes the decays
+    col: int = 0                 # first column of its part of the input projection
+    out_scale: float = 1.0       # factor of the result
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    # columns of the fused input projection [q | k | v | output gate | inner vector of the decays]
+    @property
+    def k_col(self) -> int:
+        return self.col + _up8(self.heads * self.dim)
+
+    @property
+    def v_col(self) -> int:
+        return self.k_col + _up8(self.heads * self.dim)
+
+    @property
+    def gate_col(self) -> int:
+        return self.v_col + _up8(self.heads * self.vdim)
+
+    @property
+    def rank_col(self) -> int:
+        return self.gate_col + _up8(self.heads * self.vdim)
+
+    @property
+    def in_width(self) -> int:
+        """Columns up to the end of its part."""
+        return self.rank_col + _up8(self.rank)
+
+    @property
+    def state_floats(self) -> int:
+        return (self.heads * self.dim * self.vdim + 3) // 4 * 4
+
+
+@dataclass(frozen=True)
+class TwinSpec:
+    """Two mixers that read the same input and whose results are added: attention over heads and gated linear attention.
+    Their projections are one, [left | right], and so are their results."""
+    left: HeadsSpec
+    right: GatedLinearSpec
+
+    @property
+    def heads(self) -> int:
+        return max(self.left.heads, self.right.heads)
+
+    @property
+    def in_width(self) -> int:
+        return self.right.in_width
+
+    @property
+    def right_at(self) -> int:
+        """Column of the right mixer's result."""
+        return _up8(self.left.out_width)
+
+    @property
+    def out_width(self) -> int:
+        """Both results; what comes behind them starts on 8 elements."""
+        return self.right_at + _up8(self.right.out_width)
+
+
+RECURRENT = (MatrixMemorySpec, StateSpaceSpec, GatedLinearSpec)
+MixerSpec = Union[HeadsSpec, MatrixMemorySpec, StateSpaceSpec, TwinSpec]
+
+
+def attention_of(s: MixerSpec) -> Optional[HeadsSpec]:
+    """The part of a mixer that caches keys and values."""
+    s = s.left if isinstance(s, TwinSpec) else s
+    return s if isinstance(s, HeadsSpec) else None
+
+
+def recurrent_of(s: MixerSpec):
+    """The part of a mixer that keeps recurrent state."""
+    s = s.right if isinstance(s, TwinSpec) else s
+    return s if isinstance(s, RECURRENT) else None
 
 
 # ---- entries of a design's ``layers`` list -------------------------------------------------------------------------------
@@ -292,14 +404,31 @@ def _windowed_attention(m: dict) -> HeadsSpec:
                      rot_dims=int(rot.get("dims") or 0), rot_base=float(rot.get("base", 10000.0)))
 
 
+# rank of the decays' projection where nothing says another (a model's own tensors do, see ``ArchAdapter.sizes_of_tensors``)
+DECAY_RANK = 16
+
+
 def _state_space(m: dict) -> StateSpaceSpec:
     return StateSpaceSpec(int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"]), int(m["conv"]),
                           int(m["norm_groups"]))
 
 
+def _twin(m: dict) -> TwinSpec:
+    a, r = m["left"], m["right"]
+    mask, rot = a.get("mask") or {}, a.get("rot") or {}
+    left = HeadsSpec(int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), int(a["vdim"]), float(a["scale"]),
+                     window=int(mask.get("size") or 0), pool=int(mask.get("pool") or 0), bias=True, whole_norm=True,
+                     rot_dims=int(rot.get("dims") or 0), rot_base=float(rot.get("base", 10000.0)),
+                     rot_factor=float((rot.get("scaling") or {}).get("factor", 1.0)), sink=True, head_temp=True,
+                     out_scale=float(m.get("left_scale", 1.0)))
+    return TwinSpec(left, GatedLinearSpec(int(r["heads"]), int(r["dim"]), int(r["vdim"]), float(r["tau"]),
+                                          int(r.get("rank") or DECAY_RANK), left.in_width, float(m.get("right_scale", 1.0))))
+
+
 _MIXERS = {
     "nimelorn": {"attention": _chunked_attention, "mlstm": _matrix_memory},
     "movinex": {"attention": _tempered_attention, "attention_2": _windowed_attention, "mamba2": _state_space},
+    "vobisun": {"parallel": _twin},
 }
 
 
@@ -316,6 +445,8 @@ def read_ff(arch: str, layer: dict):
     m = layer.get("mlp")
     if m is None:
         return None
+    if arch == "vobisun":
+        return DenseSpec(int(m["ff"]), "silu_glu")
     if arch == "movinex":
         if m["kind"] == "dense":
             return DenseSpec(int(m["ff"]), "gelu_tanh_glu")

@@ -28,7 +28,7 @@ from ..ops import reference as ref
 from ..ops.backend import LinearWeight, TorchOps, make_ops, np_to_dev
 from ..parallel.shard_plan import ShardPlan, make_plan
 
-SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "phi3", "gemma2", "gemma4", "ruralorn", "nimelorn", "movinex")
+SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "phi3", "gemma2", "gemma4", "ruralorn", "nimelorn", "movinex", "vobisun")
 
 
 def _entry_part(loader: ZSELoader, name: str, rows=None, cols=None, mirror=None) -> dict:
@@ -186,7 +186,8 @@ class DecoderModel:
         elif c.is_hybrid and cls is DecoderModel:
             from .hybrid import HybridModel
             from .looped import LoopedModel
-            cls = HybridModel if c.norms_outputs else LoopedModel
+            from .twin import TwinModel
+            cls = TwinModel if c.side_by_side else HybridModel if c.norms_outputs else LoopedModel
         m = cls(c, plan, ops or make_ops(device, cls.kernel_group))
         m.set_dtype(dtype)
         m._load(loader, progress)

@@ -26,7 +26,8 @@ from typing import Dict, List, Optional, Union
 
 import torch
 
-from ..format.config import DenseSpec, HeadsSpec, MatrixMemorySpec, MoESpec, StateSpaceSpec
+from ..format.config import (DenseSpec, GatedLinearSpec, HeadsSpec, MatrixMemorySpec, MoESpec, StateSpaceSpec, TwinSpec,
+                             attention_of, recurrent_of)
 from ..format.loader import ZSELoader
 from ..ops.backend import LinearWeight
 from .decoder import StepBuffers
@@ -48,7 +49,7 @@ class EmbedDesign:
 
 @dataclass
 class HybridLayer:
-    spec: Union[HeadsSpec, MatrixMemorySpec, StateSpaceSpec]
+    spec: Union[HeadsSpec, MatrixMemorySpec, StateSpaceSpec, TwinSpec]
     ff: Union[DenseSpec, MoESpec, None]
     norm1: torch.Tensor
     w_in: LinearWeight
@@ -59,11 +60,16 @@ class HybridLayer:
     k_norm: Optional[torch.Tensor] = None
     bias: Optional[torch.Tensor] = None     # of the columns of w_in before the gates
     freqs: Optional[torch.Tensor] = None    # of the rotation
+    temp: Optional[torch.Tensor] = None     # fp32 [heads], factor of a head's scores
+    sink: Optional[torch.Tensor] = None     # fp32 [heads], score without a value
     # matrix memory
     w_if: Optional[LinearWeight] = None     # the rows of w_in that make the gates
     if_bias: Optional[torch.Tensor] = None  # fp32 [2 * heads]
-    head_norm: Optional[torch.Tensor] = None
-    # state space
+    head_norm: Optional[torch.Tensor] = None  # also of gated linear attention: [vdim], shared by the heads
+    # gated linear attention
+    decay_w: Optional[torch.Tensor] = None  # fp32 [heads * dim, rank]
+    decay_b: Optional[torch.Tensor] = None  # fp32 [heads * dim]
+    # state space; of what a twin layer's mixers read
     conv_w: Optional[torch.Tensor] = None   # fp32 [taps, channels]
     conv_b: Optional[torch.Tensor] = None
     dt_bias: Optional[torch.Tensor] = None  # fp32 [heads], like the next two
@@ -86,6 +92,12 @@ class HybridLayer:
     def moe(self) -> Optional[MoESpec]:
         return self.ff if isinstance(self.ff, MoESpec) else None
 
+    @property
+    def out_width(self) -> int:
+        """Columns that the mixer's last product reads; of a twin layer that of the feed-forward reads them too."""
+        w = self.spec.out_width
+        return w + (self.ff.ff + 7) // 8 * 8 if isinstance(self.spec, TwinSpec) and self.ff is not None else w
+
 
 @dataclass
 class LayerRun:
@@ -93,6 +105,7 @@ class LayerRun:
     layer: HybridLayer
     cache_layer: int = -1                   # of the cache pool (attention)
     state_at: int = 0                       # first element of its part of a sequence's state (recurrent mixers)
+    inputs_at: int = 0                      # ... of the last inputs of the convolution ahead of its mixer
     enters_loop: bool = False               # first of a pass of the loop
 
 
@@ -113,9 +126,10 @@ class Pass:
 
 class PagedHeads:
     """One layer's cached keys [blocks, kv_heads, block_size, dim] and values inside the pool, whose rows are as wide as the
-    widest layer's; dims are padded to 8."""
+    widest layer's; dims are padded to 8.  ``means_at``: where the blocks of means begin in a row of the block tables."""
 
-    def __init__(self, layer: torch.Tensor, spec: HeadsSpec):
+    def __init__(self, layer: torch.Tensor, spec: HeadsSpec, means_at: int = 0):
+        self.means_at = means_at
         # layer: [blocks, 1, 1, block_size, pool row]
         bs, G = layer.shape[3], spec.kv_heads
         d, v = (spec.dim + 7) // 8 * 8, (spec.vdim + 7) // 8 * 8
@@ -135,7 +149,7 @@ class HybridStepBuffers(StepBuffers):
         self._common(dev, H, c.vocab_size, max_tokens, max_seqs, max_blocks, logits_rows, attn_splits, act=act,
                      logits=f32)
         specs = [L.spec for L in model.layers]
-        heads = [s for s in specs if isinstance(s, HeadsSpec)]
+        heads = [a for a in map(attention_of, specs) if a is not None]
         memories = [s for s in specs if isinstance(s, MatrixMemorySpec)]
         self.plane_rows = min(max_tokens, PLANE_ROWS)
 
@@ -144,11 +158,15 @@ class HybridStepBuffers(StepBuffers):
             return {w: flat[: max_tokens * w].view(max_tokens, w) for w in set(widths)}
 
         self.in_views = views([s.in_width for s in specs], act)
-        self.out_views = views([s.heads * s.vdim for s in specs], act)
+        self.out_views = views([L.out_width for L in model.layers], act)
         spaces = [s for s in specs if isinstance(s, StateSpaceSpec)]
         self.xbc_views = views([s.conv_width for s in spaces], act) if spaces else {}
         self.dt = z(max_tokens * max([1] + [s.heads for s in spaces]), dt=f32)
-        self.dt_side = z(max_tokens * max([1] + [s.in_width - s.dt_col for s in spaces]), dt=f32)
+        linears = [s for s in map(recurrent_of, specs) if isinstance(s, GatedLinearSpec)]
+        self.dt_side = z(max_tokens * max([1] + [s.in_width - s.dt_col for s in spaces]
+                                          + [s.in_width - s.rank_col for s in linears]), dt=f32)
+        self.decays = z(max_tokens * max([1] + [s.heads * s.dim for s in linears]), dt=f32)
+        self.linear_ws = model.ops.gated_linear_workspace(linears, max_tokens) if linears else None
         planes = z(max_planes * self.plane_rows * max(s.in_width for s in specs), dt=f32)
         self.in_plane_views = {w: planes[: max_planes * self.plane_rows * w].view(max_planes, self.plane_rows, w)
                                for w in {s.in_width for s in specs}}
@@ -177,6 +195,7 @@ class HybridStepBuffers(StepBuffers):
 class HybridModel(DesignModel):
     """Layers whose norms sit on the sublayers' outputs; ``models.looped`` has the other placement."""
     kernel_group = "hybrid"
+    means_at = 0                # column of the block tables from which on the blocks of means stand; set by the runner
 
     # ---- loading --------------------------------------------------------------------------------------
     def _load(self, loader: ZSELoader, progress=None) -> None:
@@ -235,13 +254,14 @@ class HybridModel(DesignModel):
     def _plan_runs(self) -> None:
         """The order of the layers' runs, and where each keeps its keys and values or its state."""
         c, caches, states = self.config, self.config.cache_layers, self.config.state_offsets
+        inputs = c.input_offsets
         self.runs: List[LayerRun] = []
         for n, i in enumerate(c.layer_runs):
-            s = self.layers[i].spec
-            own = not isinstance(s, HeadsSpec) or s.own_kv
+            s = attention_of(self.layers[i].spec)
+            own = s is None or s.own_kv
             self.runs.append(LayerRun(self.layers[i], caches.get(n if own else s.kv_from, -1), states.get(n, 0),
-                                      c.enters_loop(n)))
-        self.heads_specs = [L.spec for L in self.layers if isinstance(L.spec, HeadsSpec)]
+                                      inputs.get(n, 0), c.enters_loop(n)))
+        self.heads_specs = [a for a in (attention_of(L.spec) for L in self.layers) if a is not None]
         self._views: Dict[tuple, PagedHeads] = {}
 
     def _count(self, w: torch.Tensor) -> torch.Tensor:
@@ -257,13 +277,14 @@ class HybridModel(DesignModel):
         key = (kv.data_ptr(), run.cache_layer)
         v = self._views.get(key)
         if v is None:
-            v = self._views[key] = PagedHeads(kv[run.cache_layer], run.layer.spec)
+            v = self._views[key] = PagedHeads(kv[run.cache_layer], attention_of(run.layer.spec), self.means_at)
         return v
 
     def attention_splits(self, seqs: int, max_len: int, most: int, sms: int) -> int:
         if not self.heads_specs:
             return 1
-        span = max(min(max_len, s.chunk or max_len, s.window + s.keep_first if s.window else max_len) for s in self.heads_specs)
+        span = max(min(max_len, s.chunk or max_len, s.window + s.keep_first if s.window else max_len)
+                   + (max_len // s.pool if s.pool else 0) for s in self.heads_specs)
         ctas = seqs * min(s.kv_heads * ((s.heads // s.kv_heads + 15) // 16) for s in self.heads_specs)
         want = (2 * sms + ctas - 1) // ctas
         n = int(max(1, min(want, span // 128, most)))
@@ -299,24 +320,27 @@ class HybridModel(DesignModel):
             n_in = ops.linear_partial(L.w_in, b.xnorm, M, planes)
         else:
             ops.linear(L.w_in, b.xnorm, M, inp, side=None if side is None else (s.dt_col, side))
-        out = b.out_views[s.heads * s.vdim]
+        out = b.out_views[L.out_width]
         mixer = self._attend if isinstance(s, HeadsSpec) else self._space if side is not None else self._remember
-        mixer(b, p, run, inp, planes, n_in, out)
+        mixer(b, p, run, s, inp, planes, n_in, out)
         return ops.linear_partial(L.o, out, M, p.partials)
 
-    def _attend(self, b, p: Pass, run: LayerRun, inp, planes, n_in: int, out) -> None:
-        ops, L, s, M = self.ops, run.layer, run.layer.spec, p.M
+    def _attend(self, b, p: Pass, run: LayerRun, s: HeadsSpec, inp, planes, n_in: int, out) -> None:
+        ops, L, M = self.ops, run.layer, p.M
         view = self._heads_view(p.kv, run)
         ops.heads_prep(inp, planes, n_in, view, b.slots, L, s, self.config.rms_norm_eps, M, b.positions)
+        if s.pool:
+            ops.heads_pool(view, b.block_tables, p.row_seq, b.positions, s, M)
         rows, seqs = p.short if ops.heads_expands(s, self.act_dtype) else (M, p.num_seqs)
         if rows:
-            ops.heads_attn(inp, view, b.block_tables, p.row_seq, b.positions, out, rows, s, b.attn_scratch, p.splits)
+            ops.heads_attn(inp, view, b.block_tables, p.row_seq, b.positions, out, rows, s, b.attn_scratch, p.splits,
+                           L.sink)
         if seqs < p.num_seqs:
             ops.heads_attn_chunks(inp, view, b.block_tables, b.cu_q, b.q_pos0, b.positions, seqs, p.num_seqs, p.max_q_len,
-                                  out, s)
+                                  out, s, L.sink)
 
-    def _remember(self, b, p: Pass, run: LayerRun, inp, planes, n_in: int, out) -> None:
-        ops, L, s, M, eps = self.ops, run.layer, run.layer.spec, p.M, self.config.rms_norm_eps
+    def _remember(self, b, p: Pass, run: LayerRun, s: MatrixMemorySpec, inp, planes, n_in: int, out) -> None:
+        ops, L, M, eps = self.ops, run.layer, p.M, self.config.rms_norm_eps
         n_gate = 0 if n_in else ops.linear_partial(L.w_if, b.xnorm, M, b.gate_planes)
         ops.memory_prep(inp, planes, n_in, b.gate_planes, n_gate, b.gates, L, s, M)
         rows, seqs = p.short if ops.memory_expands(s, self.act_dtype) else (M, p.num_seqs)
@@ -327,8 +351,23 @@ class HybridModel(DesignModel):
             ops.memory_chunks(inp, b.gates, states, run.state_at, b.state_rows, b.cu_q, L, out, seqs, p.num_seqs, rows, M, s,
                               eps, b.memory_ws)
 
-    def _space(self, b, p: Pass, run: LayerRun, inp, planes, n_in: int, out) -> None:
-        ops, L, s, M, states = self.ops, run.layer, run.layer.spec, p.M, self.states.rows
+    def _recall(self, b, p: Pass, run: LayerRun, s: GatedLinearSpec, inp, planes, n_in: int, out) -> None:
+        ops, L, M, eps, states = self.ops, run.layer, p.M, self.config.rms_norm_eps, self.states.rows
+        seqs = p.short[1] if ops.gated_linear_expands(s, self.act_dtype) else p.num_seqs
+        decays = b.decays
+        if n_in and seqs == p.num_seqs:
+            decays = None                    # token by token only: the step's kernel reads the planes
+        else:
+            ops.gated_linear_prep(inp, planes, n_in, b.dt_side, decays, L, s, M)
+        if seqs:
+            ops.gated_linear_tokens(inp, planes, n_in, decays, states, run.state_at, b.state_rows, p.cu_q, L, out, seqs, M, s,
+                                    eps)
+        if seqs < p.num_seqs:
+            ops.gated_linear_chunks(inp, decays, states, run.state_at, b.state_rows, b.cu_q, L, out, seqs, p.num_seqs, M, s,
+                                    eps, b.linear_ws)
+
+    def _space(self, b, p: Pass, run: LayerRun, s: StateSpaceSpec, inp, planes, n_in: int, out) -> None:
+        ops, L, M, states = self.ops, run.layer, p.M, self.states.rows
         xbc = b.xbc_views[s.conv_width]
         ops.state_space_prep(inp, planes, n_in, b.dt_side, xbc, b.dt, states, run.state_at, b.state_rows, p.row_seq, p.cu_q,
                              L, s, M, p.num_seqs)
@@ -338,6 +377,18 @@ class HybridModel(DesignModel):
         if seqs < p.num_seqs:
             ops.state_space_chunks(inp, xbc, b.dt, states, run.state_at, b.state_rows, b.cu_q, L, out, seqs, p.num_seqs, M, s)
         ops.group_norm(out, L.out_norm, s.norm_groups, M, self.config.rms_norm_eps)
+
+    def _mix_both(self, b: HybridStepBuffers, p: Pass, run: LayerRun, x: torch.Tensor) -> None:
+        """Both mixers of a twin layer on ``x``, their results side by side in the layer's output buffer."""
+        ops, L, s, M = self.ops, run.layer, run.layer.spec, p.M
+        inp, planes, n_in = b.in_views[s.in_width], b.in_plane_views[s.in_width], 0
+        if p.planes_ok:
+            n_in = ops.linear_partial(L.w_in, x, M, planes)
+        else:
+            ops.linear(L.w_in, x, M, inp, side=(s.right.rank_col, b.dt_side))
+        out = b.out_views[L.out_width]
+        self._attend(b, p, run, s.left, inp, planes, n_in, out)
+        self._recall(b, p, run, s.right, inp, planes, n_in, out[:, s.right_at:])
 
     def _feed(self, b: HybridStepBuffers, p: Pass, L: HybridLayer):
         """The layer's feed-forward on ``b.xnorm``: (planes of ``p.partials``, the experts' rows or None)."""

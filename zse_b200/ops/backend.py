@@ -290,37 +290,48 @@ class TorchOps:
         """Whether long chunks of such a layer take ``heads_attn_chunks``."""
         return True
 
-    def rotation(self, dims: int, base: float):
-        """Frequencies of the pairs (2i, 2i + 1), base^(-2i / dims) per position, in this back end's form."""
-        return base ** (-torch.arange(0, dims, 2, dtype=torch.float64, device=self.device) / dims) if dims else None
+    def rotation(self, dims: int, base: float, factor: float = 1.0):
+        """Frequencies of the pairs (2i, 2i + 1), base^(-2i / dims) / factor per position, in this back end's form."""
+        if not dims:
+            return None
+        return base ** (-torch.arange(0, dims, 2, dtype=torch.float64, device=self.device) / dims) / factor
 
     def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M, positions=None):
         if n_planes:
-            ld = inp.shape[1]
-            inp[:M] = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
+            ld, w = inp.shape[1], spec.in_width
+            inp[:M, :w] = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld)[..., :w].sum(0)
         ref.heads_prep(inp[:M], kv.k if kv else None, kv.v if kv else None, slots[:M], spec, L.q_norm, L.k_norm, eps,
                        None if positions is None else positions[:M].long(), getattr(L, "bias", None),
-                       getattr(L, "freqs", None))
+                       getattr(L, "freqs", None), getattr(L, "temp", None))
 
-    def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits):
+    def heads_pool(self, kv, block_tables, row_seq, positions, spec, M):
+        """Means of the blocks of ``spec.pool`` tokens that rows [0, M) complete, from the cached keys and values into the cache.
+        Row t belongs to sequence ``row_seq[t]`` (None: t)."""
+        for t in range(M):
+            p, s = int(positions[t]), t if row_seq is None else int(row_seq[t])
+            if (p + 1) % spec.pool == 0:
+                for cache in (kv.k, kv.v):
+                    ref.pool_rows(cache, block_tables[s], kv.means_at, p // spec.pool, spec.pool)
+
+    def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits, sink=None):
         """Rows [0, M) against the cached keys and values; row t belongs to sequence ``row_seq[t]`` (None: t)."""
         for t in range(M):
             s = t if row_seq is None else int(row_seq[t])
-            self._heads_rows(inp, kv, block_tables[s], positions, out, t, t + 1, spec)
+            self._heads_rows(inp, kv, block_tables[s], positions, out, t, t + 1, spec, sink)
 
-    def heads_attn_chunks(self, inp, kv, block_tables, cu_q, q_pos0, positions, first, last, max_q, out, spec):
+    def heads_attn_chunks(self, inp, kv, block_tables, cu_q, q_pos0, positions, first, last, max_q, out, spec, sink=None):
         """Rows of the sequences ``first .. last - 1``."""
         for s in range(first, last):
-            self._heads_rows(inp, kv, block_tables[s], positions, out, int(cu_q[s]), int(cu_q[s + 1]), spec)
+            self._heads_rows(inp, kv, block_tables[s], positions, out, int(cu_q[s]), int(cu_q[s + 1]), spec, sink)
 
     @staticmethod
-    def _heads_rows(inp, kv, table, positions, out, a, e, spec):
+    def _heads_rows(inp, kv, table, positions, out, a, e, spec, sink=None):
         H, w = spec.heads, spec.heads * spec.vdim
         y = ref.heads_attn(inp[a:e, : H * spec.dim].reshape(e - a, H, spec.dim), positions[a:e].long(), kv.k, kv.v, table,
-                           spec)
+                           spec, sink, getattr(kv, "means_at", 0))
         if spec.gated:
             y = y * torch.sigmoid(inp[a:e, spec.gate_col: spec.gate_col + spec.gate_width].float()).view(e - a, H, -1)
-        out[a:e, :w] = y.reshape(e - a, w)
+        out[a:e, :w] = (spec.out_scale * y).reshape(e - a, w)
 
     def memory_expands(self, spec, dtype) -> bool:
         """Whether long chunks of such a layer take ``memory_chunks``."""
@@ -410,6 +421,70 @@ class TorchOps:
             if write >= 0:
                 states[write, at: at + H * n * v] = mem
             out[a:e, : H * v] = y.reshape(e - a, H * v) * torch.nn.functional.silu(inp[a:e, : H * v].float())
+
+    # ---- gated linear attention -------------------------------------------------------------------------------------------
+    def gated_linear_expands(self, spec, dtype) -> bool:
+        """Whether long chunks of such a layer take ``gated_linear_chunks``."""
+        return False
+
+    def gated_linear_workspace(self, specs, max_tokens: int):
+        return None
+
+    def gated_linear_prep(self, inp, planes, n_planes, side, decays, L, spec, M):
+        """Sums the split-K planes of its part of the input projection and makes the logarithms of the decays, ``decays``
+        [M, heads * dim].  Without planes ``inp`` is complete; ``side``: the decays' inner vectors in fp32 (None: those of
+        ``inp``)."""
+        ld = inp.shape[1]
+        if n_planes:
+            full = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld).sum(0)
+            inp[:M, spec.col: spec.in_width] = full[:, spec.col: spec.in_width]
+            u = full[:, spec.rank_col: spec.rank_col + spec.rank]
+        elif side is not None:
+            u = side.view(-1)[: M * (ld - spec.rank_col)].view(M, -1)[:, : spec.rank]
+        else:
+            u = inp[:M, spec.rank_col: spec.rank_col + spec.rank]
+        w = spec.heads * spec.dim
+        decays.view(-1)[: M * w].view(M, w).copy_(ref.log_decays(u, L.decay_w, L.decay_b, spec.tau))
+
+    def gated_linear_tokens(self, inp, planes, n_planes, decays, states, at, state_rows, cu_q, L, out, S, M, spec, eps):
+        """Sequences [0, S), token by token: memory, read-out, head norm and output gate.  ``states``: the state pool's rows,
+        ``at``: where the layer's part of a row begins; ``cu_q``: first row of every sequence (None: a row each).  With
+        ``decays`` None the rows of ``inp`` are still in the planes and the decays are made on the way."""
+        if decays is None:
+            decays = torch.empty(M * spec.heads * spec.dim, device=inp.device)
+            self.gated_linear_prep(inp, planes, n_planes, None, decays, L, spec, M)
+        H, d, vd = spec.heads, spec.dim, spec.vdim
+        g = decays.view(-1)[: M * H * d].view(M, H, d)
+        n = H * d * vd
+        for s in range(S):
+            a, e = (s, s + 1) if cu_q is None else (int(cu_q[s]), int(cu_q[s + 1]))
+            read, write = int(state_rows[0, s]), int(state_rows[1, s])
+            mem = states[read, at: at + n].clone() if read >= 0 else torch.zeros(n, device=inp.device)
+            x = inp[a:e].float()
+            y = ref.gated_linear_tokens(x[:, spec.col: spec.col + H * d].reshape(-1, H, d) * d ** -0.5,
+                                        x[:, spec.k_col: spec.k_col + H * d].reshape(-1, H, d),
+                                        x[:, spec.v_col: spec.v_col + H * vd].reshape(-1, H, vd), g[a:e], mem.view(H, d, vd))
+            if write >= 0:
+                states[write, at: at + n] = mem
+            y = ref.rmsnorm_f32(y, L.head_norm, eps).reshape(e - a, H * vd) * spec.out_scale
+            out[a:e, : H * vd] = y * torch.nn.functional.silu(x[:, spec.gate_col: spec.gate_col + H * vd])
+
+    def add_norm_conv(self, residual, partials, n_partials, weight, out, conv_w, conv_out, states, at, state_rows, row_seq,
+                      cu_q, M, S, eps):
+        """residual += the planes' sum; out = RMSNorm(residual) * weight; conv_out = out plus its causal convolution along the
+        sequence, ``conv_w`` [taps, H].  ``states``: the state pool's rows, which hold a sequence's last taps - 1 rows of
+        ``out`` from ``at`` on."""
+        H, taps = residual.shape[1], conv_w.shape[0]
+        self.add_norm(residual, partials, n_partials, None, weight, out, M, eps)
+        tail = slice(at, at + (taps - 1) * H)
+        for s in range(S):
+            a, e = (s, s + 1) if cu_q is None else (int(cu_q[s]), int(cu_q[s + 1]))
+            read, write = int(state_rows[0, s]), int(state_rows[1, s])
+            before = states[read, tail].view(taps - 1, H) if read >= 0 else torch.zeros(taps - 1, H, device=out.device)
+            y, last = ref.conv_inputs(out[a:e].float(), before, conv_w)
+            conv_out[a:e] = y
+            if write >= 0:
+                states[write, tail] = last.reshape(-1)
 
     def group_norm(self, x, weight, parts: int, M, eps):
         """Rows of ``x`` normed in place in ``parts`` equal parts, times ``weight``."""

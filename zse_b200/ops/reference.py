@@ -349,44 +349,79 @@ def sinusoid(positions: torch.Tensor, width: int, base: float) -> torch.Tensor:
 
 # ---- attention over heads whose keys and values have their own widths ------------------------------------------------
 def heads_prep(inp: torch.Tensor, k_cache, v_cache, slots, spec, q_norm, k_norm, eps: float, positions=None, bias=None,
-               freqs=None) -> None:
-    """Second half of the fused input projection [q | k | v | gate]: bias, rotation, query and key norm over a head's
-    dimensions, temperature of the queries, keys and values into the cache (``k_cache`` [blocks, kv_heads, block_size,
-    dim..]); queries are finished in place.  ``freqs``: radians per position of every pair that rotates."""
+               freqs=None, temp=None) -> None:
+    """Second half of the fused input projection [q | k | v | gate]: bias, query and key norm (over a head's dimensions after
+    the rotation, or over all heads' before it), rotation, factors of the queries (by position, or ``temp`` [heads]), keys and
+    values into the cache (``k_cache`` [blocks, kv_heads, block_size, dim..]); queries are finished in place.  ``freqs``:
+    radians per position of every pair that rotates."""
     T, H, G, d, vd = inp.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim
-    full = inp.float() if bias is None else inp.float() + bias.float()
+    full = inp.float()
+    if bias is not None:
+        full = full.clone()
+        full[:, : bias.numel()] += bias.float()
     turn = (lambda x: rotate_pairs(x.double(), positions.double(), freqs).float()) if spec.rot_dims else lambda x: x
-    q = rmsnorm_f32(turn(full[:, : H * d].reshape(T, H, d)), q_norm, eps)
+
+    def normed(x, n, w):
+        if spec.whole_norm:
+            return turn(rmsnorm_f32(x, w, eps).reshape(T, n, d))
+        return rmsnorm_f32(turn(x.reshape(T, n, d)), w, eps)
+
+    q = normed(full[:, : H * d], H, q_norm)
     if spec.temp_coef:
         q = q * query_temperature(positions, spec.temp_coef, spec.temp_every)[:, None, None]
-    inp[:, : H * d] = q.view(T, -1).to(inp.dtype)
+    if temp is not None:
+        q = q * temp.float()[:, None]
+    inp[:, : H * d] = q.reshape(T, -1).to(inp.dtype)
     if not spec.own_kv:
         return
     bs = k_cache.shape[2]
-    raw = full[:, spec.k_col: spec.k_col + G * d].reshape(T, G, d)
-    k = rmsnorm_f32(turn(raw), k_norm, eps)
-    v = (raw if spec.k_as_v else full[:, spec.v_col: spec.v_col + G * vd].reshape(T, G, vd)).to(v_cache.dtype)
+    raw = full[:, spec.k_col: spec.k_col + G * d]
+    k = normed(raw, G, k_norm)
+    v = (raw.reshape(T, G, d) if spec.k_as_v else full[:, spec.v_col: spec.v_col + G * vd].reshape(T, G, vd)).to(v_cache.dtype)
     ok = slots >= 0
     s = slots[ok]
     k_cache[s // bs, :, s % bs, :d] = k[ok].to(k_cache.dtype)
     v_cache[s // bs, :, s % bs, :vd] = v[ok]
 
 
-def heads_attn(q: torch.Tensor, positions, k_cache, v_cache, table, spec) -> torch.Tensor:
-    """Queries [T, heads, dim] of one sequence at ``positions`` against its cached keys: [T, heads, vdim] fp32."""
+def pool_rows(cache: torch.Tensor, table: torch.Tensor, means_at: int, block: int, size: int) -> None:
+    """Writes the mean of the cached rows of block ``block`` of ``size`` tokens (``cache`` [blocks, kv_heads, block_size, d]) to
+    its place behind ``means_at`` in the sequence's block table."""
+    bs = cache.shape[2]
+    pos = torch.arange(block * size, block * size + size, device=cache.device)
+    blk = table[pos // bs].long()
+    rows = cache[blk.clamp_min(0), :, pos % bs].float() * (blk >= 0)[:, None, None]
+    to = int(table[means_at + block // bs])
+    if to >= 0:
+        cache[to, :, block % bs] = (rows.sum(0) / size).to(cache.dtype)
+
+
+def heads_attn(q: torch.Tensor, positions, k_cache, v_cache, table, spec, sink=None, means_at: int = 0) -> torch.Tensor:
+    """Queries [T, heads, dim] of one sequence at ``positions`` against its cached keys: [T, heads, vdim] fp32.  ``sink``
+    [heads]: one more score of every row, without a value; ``means_at``: where the blocks of means begin in ``table``."""
     bs, rep = k_cache.shape[2], spec.heads // spec.kv_heads
     first = torch.tensor([spec.first_seen(int(p)) for p in positions], device=q.device)
     pos = torch.arange(int(first.min()), int(positions.max()) + 1, device=q.device)
     if spec.keep_first:
         pos = torch.cat([torch.arange(min(spec.keep_first, int(first.min())), device=q.device), pos])
-    blk = table[pos // bs].long()
-    k = k_cache[blk.clamp_min(0), :, pos % bs, : spec.dim].float().repeat_interleave(rep, 1)
-    v = v_cache[blk.clamp_min(0), :, pos % bs, : spec.vdim].float().repeat_interleave(rep, 1)
-    see = (pos[None] <= positions[:, None]) & ((pos[None] >= first[:, None]) | (pos[None] < spec.keep_first)) & (blk >= 0)[None]
+    blk, at = table[pos // bs].long(), pos % bs
+    see = (pos[None] <= positions[:, None]) & ((pos[None] >= first[:, None]) | (pos[None] < spec.keep_first))
+    if spec.pool:
+        seen = torch.tensor([spec.blocks_seen(int(p)) for p in positions], device=q.device)
+        b = torch.arange(int(seen.max()), device=q.device)
+        blk, at = torch.cat([table[means_at + b // bs].long(), blk]), torch.cat([b % bs, at])
+        see = torch.cat([b[None] < seen[:, None], see], 1)
+    k = k_cache[blk.clamp_min(0), :, at, : spec.dim].float().repeat_interleave(rep, 1)
+    v = v_cache[blk.clamp_min(0), :, at, : spec.vdim].float().repeat_interleave(rep, 1)
+    see = see & (blk >= 0)[None]
     s = torch.einsum("thd,nhd->htn", q.float(), k) * spec.scale
     if spec.softcap:
         s = spec.softcap * torch.tanh(s / spec.softcap)
-    return torch.einsum("htn,nhv->thv", torch.softmax(s.masked_fill(~see, float("-inf")), -1).nan_to_num(0.0), v)
+    s = s.masked_fill(~see, float("-inf"))
+    if sink is not None:
+        s = torch.cat([s, sink.float()[:, None, None].expand(-1, s.shape[1], 1)], -1)
+    w = torch.softmax(s, -1).nan_to_num(0.0)[..., : k.shape[0]]
+    return torch.einsum("htn,nhv->thv", w, v)
 
 
 def query_temperature(positions: torch.Tensor, coef: float, every: int) -> torch.Tensor:
@@ -437,6 +472,30 @@ def state_space_tokens(x, B, C, dt, neg_a, D, S):
         S.mul_(torch.exp(neg_a * dt[t])[:, None, None]).add_((dt[t][:, None] * b)[:, :, None] * x[t][:, None, :])
         out[t] = torch.einsum("hnv,hn->hv", S, c) + D[:, None] * x[t]
     return out
+
+
+# ---- gated linear attention -------------------------------------------------------------------------------------------
+def log_decays(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
+    """Logarithms of the decays [T, heads * dim] from their inner vectors ``u`` [T, rank], fp32."""
+    return torch.nn.functional.logsigmoid(u.float() @ w.float().T + bias) / tau
+
+
+def gated_linear_tokens(q, k, v, log_alpha, S):
+    """Tokens of one sequence through one layer's memory.  q, k, log_alpha [T, H, d] and v [T, H, vd] fp32; S [H, d, vd] is
+    updated in place.  Returns the read-outs [T, H, vd]."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        S.mul_(torch.exp(log_alpha[t])[:, :, None]).add_(k[t][:, :, None] * v[t][:, None, :])
+        out[t] = torch.einsum("hdv,hd->hv", S, q[t])
+    return out
+
+
+def conv_inputs(h: torch.Tensor, before: torch.Tensor, w: torch.Tensor):
+    """One sequence's rows ``h`` [T, C] plus their causal convolution per channel, after the inputs ``before`` [taps - 1, C];
+    ``w`` [taps, C] with the row's own tap last.  Returns the result and the last taps - 1 inputs."""
+    taps, T = w.shape[0], h.shape[0]
+    full = torch.cat([before, h])
+    return h + sum(w[j] * full[j: j + T] for j in range(taps)), full[T:]
 
 
 # ---- feed-forwards ----------------------------------------------------------------------------------------------------

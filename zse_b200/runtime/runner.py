@@ -57,7 +57,9 @@ class ModelRunner:
         self.max_seq_len = min(max_seq_len or c.max_seq_len, c.max_seq_len)
         self.max_batch_seqs = max_batch_seqs
         self.max_tokens = max(max_tokens_per_pass, max_batch_seqs)
-        self.max_blocks = (self.max_seq_len + cache.block_size - 1) // cache.block_size
+        # columns of a sequence's row of the block tables: blocks of tokens, then those of their means
+        self.means_at = (self.max_seq_len + cache.block_size - 1) // cache.block_size
+        self.max_blocks = self.means_at + cache.mean_blocks(self.max_seq_len)
         on_gpu = self.device.type == "cuda"
         self.use_graphs = on_gpu if use_graphs is None else (use_graphs and on_gpu)
         sm = torch.cuda.get_device_properties(self.device).multi_processor_count if on_gpu else 1
@@ -66,6 +68,7 @@ class ModelRunner:
         logits_rows = max(max_batch_seqs, 64, logits_rows)
         model.cache_block_size = cache.block_size
         model.states = cache.states
+        model.means_at = self.means_at
         self.buf = model.make_buffers(self.max_tokens, max_batch_seqs, self.max_blocks, logits_rows,
                                       max_planes=8, attn_splits=self.max_attn_splits)
         self._graphs: Dict[Tuple[int, int, bool], torch.cuda.CUDAGraph] = {}
@@ -227,6 +230,9 @@ class ModelRunner:
             self.h_slots[at:at + n] = torch.from_numpy(cache.slots_for_range(sid, start, n))
             ids = cache.get_block_ids(sid)
             self.h_bt[s, :len(ids)] = torch.as_tensor(ids, dtype=torch.int32)
+            if self.max_blocks > self.means_at:
+                ids = cache.mean_block_ids(sid)
+                self.h_bt[s, self.means_at: self.means_at + len(ids)] = torch.as_tensor(ids, dtype=torch.int32)
             self.h_cu[s] = at
             self.h_pos0[s] = start
             if per_tok_adapter is not None:
@@ -314,7 +320,8 @@ class ModelRunner:
         bs = cache.block_size
         n_ = self._np
         self._staging_begin()
-        max_len = max(1, cache.stage_decode(seq_ids, n_["bt"], n_["lens"], n_["pos"], n_["slots"]))
+        max_len = max(1, cache.stage_decode(seq_ids, n_["bt"], n_["lens"], n_["pos"], n_["slots"],
+                                              self.means_at))
         if ids_rows is None:
             n_["ids"][:S] = last_tokens
         else:

@@ -28,7 +28,10 @@ MemoryReservation = _Commit      # the reference's name for the per-request reco
 
 
 class MemoryBudget:
-    def __init__(self, total_blocks: int, block_size: int, headroom_ratio: float = 0.5, reserve_blocks: int = 2):
+    def __init__(self, total_blocks: int, block_size: int, headroom_ratio: float = 0.5, reserve_blocks: int = 2,
+                 mean_step: int = 0):
+        """``mean_step``: tokens per row of block means, which take blocks of their own (0: the model caches none)."""
+        self._step = mean_step
         self._total = total_blocks
         self._bs = block_size
         self._ratio = headroom_ratio
@@ -37,7 +40,10 @@ class MemoryBudget:
         self._lock = threading.Lock()
 
     def _tokens_to_blocks(self, tokens: int) -> int:
-        return (tokens + self._bs - 1) // self._bs if tokens > 0 else 0
+        if tokens <= 0:
+            return 0
+        means = (tokens // self._step + self._bs - 1) // self._bs if self._step else 0
+        return (tokens + self._bs - 1) // self._bs + means
 
     def _estimate(self, req: InferenceRequest) -> _Commit:
         prompt = self._tokens_to_blocks(req.prompt_len + req.num_generated)

@@ -33,7 +33,7 @@ class TraceRunner:
         block = 64
         tokens = (max(1, max_tokens) + block - 1) // block * block
         self.engine = ZStreamerEngine(model, config=EngineConfig(
-            dtype=dtype, device=device, block_size=block, kv_blocks=tokens // block, max_seq_len=tokens,
+            dtype=dtype, device=device, block_size=block, kv_tokens=tokens, max_seq_len=tokens,
             max_batch_seqs=max_live, max_batch_tokens=tokens, prefill_chunk_size=0, logits_rows=tokens,
             enable_prefix_cache=False, state_slots=max_live))
         self._seq: Dict[str, int] = {}
