@@ -80,7 +80,7 @@ typedef struct ZseTileGemm {
 int zse_gemm_tile(int dtype, const ZseTileGemm* a, int batch, int max_tiles, void* stream);
 // in [rows, 2 * ff] (gate, up) -> out [rows, ff]; kind 0: g sigmoid(1.702 g) (u + 1), g clamped from above and u from both
 // sides; 1: silu(g) u; 2: gelu(g) u with the tanh form of gelu
-int zse_glu(int dtype, const void* in, void* out, int rows, int ff, int kind, float limit, void* stream);
+int zse_glu(int dtype, const void* in, void* out, int ldo, int rows, int ff, int kind, float limit, void* stream);
 
 int zse_apply_repetition_penalty_f32(void* logits, int ld, const void* rows_i32, const void* tokens_i32,
                                      const void* counts_i32, int n, const void* penalty_f32, int V, void* stream);
@@ -88,6 +88,22 @@ int zse_apply_repetition_penalty_f32(void* logits, int ld, const void* rows_i32,
 // ---- rows.cu ------------------------------------------------------------------------------------------------
 int zse_embedding_typed(int dtype, const void* table, const void* ids, void* out_f32, int M, int H, int vocab,
                         float scale, void* copy, int ld_copy, void* status, void* stream);
+// causal convolution along every sequence, per channel, of normed rows
+typedef struct ZseRowConv {
+  const void* w;                // fp32 [taps][H], a row's own tap last
+  int32_t taps;
+  void* states;                 // state rows, row_floats apart; this layer's part: the last taps - 1 rows, the oldest first
+  int64_t row_floats;
+  const void* state_rows;       // [2][state_ld]: rows that sequences read and write (-1: none)
+  int32_t state_ld;
+} ZseRowConv;
+// residual += planes; out [M, H] = RMSNorm(residual) * weight; conv_out = out plus its convolution; every row is a sequence of
+// its own
+int zse_add_norm_conv(int dtype, void* residual, const void* planes, int n_planes, const void* weight, void* out,
+                      const ZseRowConv* z, void* conv_out, int M, int H, float eps, void* stream);
+// out = h plus its convolution, packed sequences: cu_q their first rows, row_seq the rows' sequences
+int zse_row_conv(int dtype, const void* h, void* out, const ZseRowConv* z, const void* row_seq, const void* cu_q, int M, int H,
+                 void* stream);
 // y = planes [n_planes][M][H] + slots [M][n_slots][H], times scale [H] (null: 1); residual += y, or = y with replace;
 // out [M, ldo] = RMSNorm(residual) * (weight + offset), or the residual itself without a weight
 int zse_add_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes, const void* slots,
@@ -187,13 +203,17 @@ typedef struct ZseHeads {
   int32_t keep_first;           // first positions that are seen whatever the window
   float softcap;                // > 0: scores become softcap * tanh(score / softcap)
   int32_t gate_each;            // a gate per dimension of a head's result, not per head
+  int32_t pool;                 // > 0, with a window: blocks of that many tokens that lie before it are seen as their means,
+  int32_t means_at;             //   rows of the cache whose blocks stand from this column on in a row of the tables
+  const void* sink;             // fp32 [heads]: one more score without a value, null: none
+  float out_scale;              // factor of the result
 } ZseHeads;
 // 1 when the tensor-core kernels take this shape (bfloat16)
 int zse_heads_mma_ok(int dim, int vdim, int block_size);
 // columns of a projected row: q from 0, k from k_col, v from v_col (k_col: the values are the keys as projected), gate from
 // gate_col (gate_w of them); own_kv 0: no keys and values of its own
 typedef struct ZseHeadsPrep {
-  const void *q_norm, *k_norm;  // weights of the norms over a head's dimensions, null: 1
+  const void *q_norm, *k_norm;  // weights of the norms over a head's dimensions, null: 1; `whole`: over all heads'
   const void* bias;             // of the columns before gate_col, null: none
   const void* turns;            // pairs that rotate: [rot_dims / 2] high and low parts of the turns per position
   const void* positions;
@@ -201,9 +221,16 @@ typedef struct ZseHeadsPrep {
   float temp_coef;              // queries are multiplied by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)
   int32_t temp_every;
   float eps;
+  int32_t whole;                // one norm over all query (key) heads, before the rotation
+  const void* head_temp;        // `whole`: fp32 [heads], factor of a head's queries, null: 1
+  int32_t pool_rows;            // `whole`: rows are sequences of their own, and one that completes a block of tokens leaves
+                                //   its mean in the cache
 } ZseHeadsPrep;
 int zse_heads_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, int M, const ZseHeads* h,
                    const void* slots, const ZseHeadsPrep* p, void* stream);
+// means of the blocks of h->pool tokens that rows [0, M) complete, from the cache into the cache; row_seq null: row t is
+// sequence t
+int zse_heads_pool(int dtype, const ZseHeads* h, const void* row_seq, const void* positions, int M, void* stream);
 // rows [0, M) one by one; gate: first element of the gates (row stride ld), or null
 int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads* h, const void* row_seq, const void* positions,
                    void* out, int ldo, const void* gate, void* scratch, int M, int num_splits, int tensor_cores,
@@ -263,6 +290,31 @@ int zse_space_chunks(const void* inp, int ld, const void* xbc, const void* dt, c
                      int last, void* out, int ldo, void* stream);
 // rows [M][ld] in place: `parts` parts of `width` columns, each divided by its root mean square, times weight
 int zse_group_norm(int dtype, void* x, int ld, int M, int parts, int width, const void* weight, float eps, void* stream);
+
+// ---- gated_linear.cu ----------------------------------------------------------------------------------------
+typedef struct ZseGatedLinear {
+  int32_t heads, dim, vdim, rank;
+  int32_t q_col, k_col, v_col, gate_col, rank_col;   // columns of a projected row; rank_col: the decays' inner vector
+  void* states;                 // state rows, row_floats apart; this layer's part: [heads][dim][vdim]
+  int64_t row_floats;
+  const void* state_rows;       // [2][state_ld]: rows that sequences read and write (-1: none)
+  int32_t state_ld;
+  float tau, eps, out_scale;
+  const void* head_norm;        // [vdim], shared by the heads
+  const void *decay_w, *decay_b;   // fp32 [heads * dim][rank], [heads * dim]
+} ZseGatedLinear;
+int zse_gated_linear_chunk_ok(int dim, int vdim);
+// split-K planes of its columns -> inp (n_planes 0: inp is complete; side [M][side_ld]: its inner vectors in fp32, or null);
+// decays: fp32 [M][heads * dim], logarithms
+int zse_gated_linear_prep(int dtype, void* inp, int ld, const void* planes, int n_planes, const void* side, int side_ld,
+                          const ZseGatedLinear* z, void* decays, int M, void* stream);
+// sequences [0, S), token by token: update, read-out, head norm, output gate; cu_q null: a row each; decays null: inp and the
+// decays' inner vectors are in the planes
+int zse_gated_linear_tokens(int dtype, const void* inp, int ld, const void* planes, int n_planes, int M, const void* decays,
+                            const ZseGatedLinear* z, const void* cu_q, int S, void* out, int ldo, void* stream);
+// sequences [first, last) chunkwise (bfloat16), whose rows are [row0, M); o: fp32 [M][heads * vdim] scratch
+int zse_gated_linear_chunks(const void* inp, int ld, const void* decays, const ZseGatedLinear* z, const void* cu_q, int first,
+                            int last, void* o, int M, int row0, void* out, int ldo, void* stream);
 
 // ---- repack.cu ----------------------------------------------------------------------------------------------
 // Row-major INT4 [N, K/2] + scales/zeros [N, K/128] -> tiled chunks.  interleave_rows > 0 builds a fused gate/up

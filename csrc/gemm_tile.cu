@@ -94,12 +94,12 @@ __global__ void __launch_bounds__(256) gemm_tile_kernel(const ZseTileGemm a) {
 // in [rows, 2 * ff] (gate, up) -> out [rows, ff]
 template <typename T>
 __global__ void __launch_bounds__(256)
-glu_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, int ff, int kind, float limit) {
+glu_kernel(const T* __restrict__ in, T* __restrict__ out, int ldo, long long n, int ff, int kind, float limit) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
     const T* g = in + i / ff * 2 * ff + i % ff;
-    out[i] = from_f32<T>(glu<false>(kind, to_f32(g[0]), to_f32(g[ff]), limit));
+    out[i / ff * ldo + i % ff] = from_f32<T>(glu<false>(kind, to_f32(g[0]), to_f32(g[ff]), limit));
   }
 }
 
@@ -108,7 +108,7 @@ glu_kernel(const T* __restrict__ in, T* __restrict__ out, long long n, int ff, i
 
 using namespace zse;
 
-extern "C" int zse_glu(int dtype, const void* in, void* out, int rows, int ff, int kind, float limit, void* stream) {
+extern "C" int zse_glu(int dtype, const void* in, void* out, int ldo, int rows, int ff, int kind, float limit, void* stream) {
   const long long n = (long long)(rows) * ff;
   if (n <= 0) return 0;
   const dim3 grid(unsigned(n + 255 < 4096ll * 256 ? (n + 255) / 256 : 4096));
@@ -116,10 +116,10 @@ extern "C" int zse_glu(int dtype, const void* in, void* out, int rows, int ff, i
   cudaError_t e;
   if (dtype == kBF16)
     e = launch_pdl(glu_kernel<bf16>, grid, dim3(256), 0, st, reinterpret_cast<const bf16*>(in),
-                   reinterpret_cast<bf16*>(out), n, ff, kind, limit);
+                   reinterpret_cast<bf16*>(out), ldo, n, ff, kind, limit);
   else
     e = launch_pdl(glu_kernel<float>, grid, dim3(256), 0, st, reinterpret_cast<const float*>(in),
-                   reinterpret_cast<float*>(out), n, ff, kind, limit);
+                   reinterpret_cast<float*>(out), ldo, n, ff, kind, limit);
   return e == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }
 

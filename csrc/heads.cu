@@ -2,6 +2,7 @@
 //
 //   heads_prep      second half of the fused input projection: split-K sum, bias, rotation, query and key norm, temperature
 //                   of the queries, cache write
+//   heads_prep_whole  the same where one norm covers all query (key) heads and comes before the rotation
 //   heads_simple    a row's heads against the cached keys it sees; any shape, bfloat16 or float
 //   heads_rows      the same on bfloat16 tensor cores: the query heads of a kv head are one 16-row tile, each warp streams
 //                   its own tiles of 16 keys; keys may be split over CTAs (heads_combine merges)
@@ -11,7 +12,8 @@
 // Cached tiles: [block][kv head][token][dim], then the same for values, dims padded to 8 (the padding is zero).  Scores and
 // softmax are fp32; softmax weights enter the product with the values as two bfloat16 terms (value and remainder).  A row
 // sees the positions from first_seen(position) to its own, and the first `keep` ones; block -1 of a table is a hole whose
-// tokens do not exist.
+// tokens do not exist.  With `pool` > 0 the means of blocks of tokens come before the window's tokens as further keys and values:
+// rows of cache blocks of their own, which heads_prep_whole (decode) or heads_pool leave there.
 #include "api.h"
 #include "heads.cuh"
 
@@ -161,6 +163,188 @@ heads_prep_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_p
   }
 }
 
+// The sum of a value over the block; `red`: one place per warp.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  return warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
+}
+
+// Means over the `pool` tokens up to position `pos` of a sequence's cached keys and values (VEC columns per access), from the
+// calling threads tid, tid + step, ...; blocks that are gone count as zeros.
+template <typename T, int VEC>
+__device__ __forceinline__ void pool_means(T* kc, T* vc, const Heads& h, const int* table, int pos, int tid, int step) {
+  const int b = pos / h.pool, first = b * h.pool;
+  const int to = table[h.means_at + h.block_of(b)], at = h.in_block(b);
+  if (to < 0) return;
+  const int kv = h.dim / VEC, vv = h.vdim / VEC, n = h.kv_heads * (kv + vv);
+  const float inv = 1.f / float(h.pool);
+  for (int i = tid; i < n; i += step) {
+    const bool key = i < h.kv_heads * kv;
+    const int j = key ? i : i - h.kv_heads * kv, per = key ? kv : vv;
+    const int g = j / per, c = j % per * VEC, width = key ? h.dp : h.vp;
+    T* cache = key ? kc : vc;
+    F32Vec<VEC> sum{};
+#pragma unroll 8
+    for (int p = first; p <= pos; ++p) {
+      const int block = table[h.block_of(p)];
+      if (block < 0) continue;
+      const F32Vec<VEC> x = load_vec<VEC>(cache + h.at(block, g, h.in_block(p), width) + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) sum.v[e] += x.v[e];
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) sum.v[e] *= inv;
+    store_vec<VEC>(cache + h.at(to, g, at, width) + c, sum);
+  }
+}
+
+// grid (blocks of kPoolRows rows)
+constexpr int kPoolRows = 16;
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+heads_pool_kernel(T* kc, T* vc, const Heads h, const int* __restrict__ row_seq, const int* __restrict__ positions, int M) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = blockIdx.x * kPoolRows;
+  for (int t = t0; t < min(M, t0 + kPoolRows); ++t) {
+    const int pos = positions[t];
+    if ((pos + 1) % h.pool) continue;
+    const int s = row_seq != nullptr ? row_seq[t] : t;
+    pool_means<T, VEC>(kc, vc, h, h.tables + size_t(s) * h.max_blocks, pos, threadIdx.x, 256);
+  }
+}
+
+// A CTA per row: split-K sum and bias of queries, keys, values and (with planes) gates; one norm over all queries and one over
+// all keys, weights, rotation, factors of the heads' queries, cache write.  POOL: a row that completes a block of tokens leaves
+// its mean in the cache as well; rows are sequences of their own.
+template <typename T, int VEC, int THREADS>
+__global__ void __launch_bounds__(THREADS)
+heads_prep_whole_kernel(T* __restrict__ inp, const float* __restrict__ planes, int n_planes, int M, T* kc, T* vc, const Heads h,
+                        const long long* __restrict__ slots, const T* __restrict__ q_norm, const T* __restrict__ k_norm,
+                        const T* __restrict__ bias, const HeadsPrepArgs a, const float* __restrict__ head_temp, int pool_rows) {
+  constexpr int kKeep = VEC == 4 ? 4 : 8;        // accesses of the queries that stay in registers
+  __shared__ float2 turned[kPrepPairs];
+  __shared__ float red[2][32];
+  extern __shared__ float row[];                 // VEC 1: the queries with their bias (pairs lie in two threads)
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int pos_i = a.positions != nullptr ? a.positions[t] : 0;
+  const float pos = float(pos_i);
+  for (int i = threadIdx.x; i < min(kPrepPairs, a.rot_dims / 2); i += THREADS) turned[i] = pair_turn(a.turns, i, pos);
+  T* in = inp + size_t(t) * a.ld;
+  const float* pl = planes + size_t(t) * a.ld;
+  const size_t plane = size_t(M) * a.ld;
+  auto raw = [&](int c) {
+    if (n_planes == 0) return load_vec<VEC>(in + c);
+    F32Vec<VEC> v{};
+#pragma unroll 4
+    for (int p = 0; p < n_planes; ++p) {
+      const F32Vec<VEC> x = load_vec<VEC>(pl + p * plane + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] += x.v[e];
+    }
+    return v;
+  };
+  auto value = [&](int c) {
+    F32Vec<VEC> v = raw(c);
+    if (bias != nullptr) {
+      const F32Vec<VEC> x = load_vec<VEC>(bias + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] += x.v[e];
+    }
+    return v;
+  };
+  const int nq = h.heads * h.dim, nk = a.own_kv ? h.kv_heads * h.dim : 0, nv = a.own_kv ? h.kv_heads * h.vdim : 0;
+  const int step = THREADS * VEC, far = kKeep * step, i0 = threadIdx.x * VEC;
+  F32Vec<VEC> q[kKeep], k0{};
+  float qs = 0.f, ks = 0.f;
+#pragma unroll
+  for (int j = 0; j < kKeep; ++j)
+    if (i0 + j * step < nq) {
+      q[j] = value(i0 + j * step);
+      if constexpr (VEC == 1) row[i0 + j * step] = q[j].v[0];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) qs += q[j].v[e] * q[j].v[e];
+    }
+  for (int i = far + i0; i < nq; i += step) {
+    const F32Vec<VEC> x = value(i);
+    if constexpr (VEC == 1) row[i] = x.v[0];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) qs += x.v[e] * x.v[e];
+  }
+  for (int i = i0; i < nk; i += step) {
+    const F32Vec<VEC> x = value(a.k_col + i);
+    if (i == i0) k0 = x;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ks += x.v[e] * x.v[e];
+  }
+  const long long slot = a.own_kv ? slots[t] : -1;
+  const int block = slot >= 0 ? h.block_of(int(slot)) : 0, token = slot >= 0 ? h.in_block(int(slot)) : 0;
+  if (slot >= 0) {
+    for (int i = i0; i < nv; i += step)
+      store_vec<VEC>(vc + h.at(block, i / h.vdim, token, h.vp) + i % h.vdim, value(a.v_col + i));
+  }
+  if (n_planes > 0)
+    for (int i = i0; i < a.gate_w; i += step) store_vec<VEC>(in + a.gate_col + i, raw(a.gate_col + i));
+  const float q_inv = 1.f / sqrtf(block_sum(qs, red[0]) / float(nq) + a.eps);
+  const float k_inv = nk > 0 ? 1.f / sqrtf(block_sum(ks, red[1]) / float(nk) + a.eps) : 0.f;
+  auto turn = [&](int i, float& x, float& y) {   // the pair of a head's dimensions i, i + 1
+    const float2 cs = i / 2 < kPrepPairs ? turned[i / 2] : pair_turn(a.turns, i / 2, pos);
+    const float u0 = x;
+    x = u0 * cs.x - y * cs.y;
+    y = y * cs.x + u0 * cs.y;
+  };
+  // columns i.. of the queries (or keys), normed, weighted and turned; `other_of`: one column of the same row, for VEC 1
+  auto finished = [&](F32Vec<VEC> v, int i, float inv, const T* w, float factor, auto other_of) {
+    const int d = i % h.dim;
+    const F32Vec<VEC> f = load_vec<VEC>(w + i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v.v[e] *= inv * f.v[e];
+    if constexpr (VEC == 4) {
+      if (d < a.rot_dims) turn(d, v.v[0], v.v[1]);
+      if (d + 2 < a.rot_dims) turn(d + 2, v.v[2], v.v[3]);
+    } else if (d < a.rot_dims) {
+      const int o = d & 1 ? i - 1 : i + 1;
+      float other = other_of(o) * (inv * to_f32(w[o]));
+      if (d & 1)
+        turn(d - 1, other, v.v[0]);
+      else
+        turn(d, v.v[0], other);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v.v[e] *= factor;
+    return v;
+  };
+  auto put_q = [&](int i, const F32Vec<VEC>& x) {
+    const float factor = head_temp != nullptr ? head_temp[i / h.dim] : 1.f;
+    store_vec<VEC>(in + i, finished(x, i, q_inv, q_norm, factor, [&](int o) { return row[o]; }));
+  };
+#pragma unroll
+  for (int j = 0; j < kKeep; ++j)
+    if (i0 + j * step < nq) put_q(i0 + j * step, q[j]);
+  for (int i = far + i0; i < nq; i += step) {
+    F32Vec<VEC> x;
+    if constexpr (VEC == 1)
+      x.v[0] = row[i];
+    else
+      x = value(i);
+    put_q(i, x);
+  }
+  if (slot < 0) return;                          // the same for the whole block
+  for (int i = i0; i < nk; i += step) {
+    const F32Vec<VEC> x = i == i0 ? k0 : value(a.k_col + i);
+    store_vec<VEC>(kc + h.at(block, i / h.dim, token, h.dp) + i % h.dim,
+                   finished(x, i, k_inv, k_norm, 1.f, [&](int o) { return value(a.k_col + o).v[0]; }));
+  }
+  if (pool_rows && h.pool > 0 && (pos_i + 1) % h.pool == 0) {
+    __syncthreads();                             // this token's key and value are in the cache
+    pool_means<T, VEC>(kc, vc, h, h.tables + size_t(t) * h.max_blocks, pos_i, threadIdx.x, THREADS);
+  }
+}
+
 // ---- any shape, any type -----------------------------------------------------------------------------------------------
 // grid (heads, rows), 4 warps that take every fourth key.
 template <typename T>
@@ -183,10 +367,10 @@ heads_simple_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ kc,
   const int seq = row_seq != nullptr ? row_seq[t] : t, pos = positions[t];
   const int* table = h.tables + size_t(seq) * h.max_blocks;
   float m = -INFINITY, l = 0.f;
-  const int lo = h.first_seen(pos), kept = min(h.keep, lo);
+  const int lo = h.first_seen(pos), kept = h.pool > 0 ? h.means_seen(pos) : min(h.keep, lo);
   for (int n = warp; n < kept + pos + 1 - lo; n += 4) {
     const int j = n < kept ? n : lo + n - kept;
-    const int block = table[h.block_of(j)];
+    const int block = table[(n < kept && h.pool > 0 ? h.means_at : 0) + h.block_of(j)];
     if (block < 0) continue;
     const T* k = kc + h.at(block, g, h.in_block(j), h.dp);
     const T* v = vc + h.at(block, g, h.in_block(j), h.vp);
@@ -204,14 +388,18 @@ heads_simple_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ kc,
     ml[4 + warp] = l;
   }
   __syncthreads();
-  const float most = fmaxf(fmaxf(ml[0], ml[1]), fmaxf(ml[2], ml[3]));
+  float most = fmaxf(fmaxf(ml[0], ml[1]), fmaxf(ml[2], ml[3]));
   float f[4], L = 0.f;
+  if (h.sink != nullptr) {
+    most = fmaxf(most, h.sink[head]);
+    L = expf(h.sink[head] - most);
+  }
 #pragma unroll
   for (int w = 0; w < 4; ++w) {
     f[w] = ml[w] == -INFINITY ? 0.f : expf(ml[w] - most);
     L += ml[4 + w] * f[w];
   }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
+  const float inv = L > 0.f ? h.out_scale / L : 0.f;
   for (int i = threadIdx.x; i < h.vdim; i += blockDim.x) {
     float y = 0.f;
 #pragma unroll
@@ -220,6 +408,9 @@ heads_simple_kernel(const T* __restrict__ inp, int ld, const T* __restrict__ kc,
     out[size_t(t) * ldo + size_t(head) * h.vdim + i] = from_f32<T>(y * inv);
   }
 }
+
+// What is special about a layer's scores: nothing, a soft cap, means of blocks as further keys.
+enum ScoreKind { kPlainScores = 0, kCapped = 1, kPooled = 2 };
 
 // ---- rows on tensor cores ----------------------------------------------------------------------------------------------
 // An odd number of 16-byte pieces: consecutive rows start in different banks for ldmatrix.  Widths are whole steps of 16.
@@ -232,7 +423,7 @@ inline size_t rows_smem(int dim, int vdim) {
   return ring > merge ? ring : merge;
 }
 
-template <int DKS, int DVT, bool CAP>  // steps of 16 key dimensions, blocks of 8 value dimensions (even)
+template <int DKS, int DVT, int KIND>  // steps of 16 key dimensions, blocks of 8 value dimensions (even)
 __global__ void __launch_bounds__(kRowWarps * 32)
 heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ kc, const bf16* __restrict__ vc, Heads h,
                   const int* __restrict__ row_seq, const int* __restrict__ positions, bf16* __restrict__ out, int ldo,
@@ -248,7 +439,9 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
   const int* table = h.tables + size_t(seq) * h.max_blocks;
   const int lo = h.first_seen(pos);
   const int tile0 = lo / kRowKeys;
-  const int kept = min(tile0, (h.keep + kRowKeys - 1) / kRowKeys);  // tiles of kept tokens before the first one of the window
+  const int means = KIND == kPooled ? h.means_seen(pos) : 0;
+  // tiles of kept tokens, or of means, before the first one of the window
+  const int kept = KIND == kPooled ? (means + kRowKeys - 1) / kRowKeys : min(tile0, (h.keep + kRowKeys - 1) / kRowKeys);
   const int tiles = kept + pos / kRowKeys + 1 - tile0;
   const int per_split = (tiles + num_splits - 1) / num_splits;
   const int tb = split * per_split, te = min(tiles, tb + per_split);
@@ -257,6 +450,8 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
     const int n = tb + warp + i * kRowWarps;
     return (n < kept ? n : tile0 + n - kept) * kRowKeys;
   };
+  auto of_means = [&](int i) { return KIND == kPooled && tb + warp + i * kRowWarps < kept; };
+  auto block_at = [&](int i, int tok) { return table[(of_means(i) ? h.means_at : 0) + h.block_of(tok)]; };
   const int mine = te > tb + warp ? (te - tb - warp + kRowWarps - 1) / kRowWarps : 0;
   const int kp = pitch_of(h.dim), vp = pitch_of(h.vdim), ks = (h.dim + 15) / 16;
   const int kch = h.dp / 8, vch = h.vp / 8;
@@ -298,7 +493,7 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
   }
   auto issue = [&](int i) {                      // i-th tile of this warp; always commits a group
     if (i < mine) {
-      const int tok = token_of(i), block = table[h.block_of(tok)];
+      const int tok = token_of(i), block = block_at(i, tok);
       if (block >= 0) {
         const bf16* ks_ = kc + h.at(block, kvh, h.in_block(tok), h.dp);
         const bf16* vs_ = vc + h.at(block, kvh, h.in_block(tok), h.vp);
@@ -326,7 +521,8 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
     __syncwarp();
     issue(i + kRowStages - 1);
     const int tok = token_of(i);
-    if (table[h.block_of(tok)] < 0) continue;
+    if (block_at(i, tok) < 0) continue;
+    const bool mean = of_means(i);
     const uint32_t kb = smem_u32(ring + (i % kRowStages) * kRowKeys * (kp + vp)), vb = kb + kRowKeys * kp;
     float s[2][4] = {};
 #pragma unroll
@@ -344,7 +540,8 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int p = tok + j * 8 + (lane & 3) * 2 + (e & 1);
-        s[j][e] = h.sees(p, pos, lo) ? (CAP ? h.capped(s[j][e] * h.scale) * kLog2E : s[j][e] * scale_log2) : -INFINITY;
+        const bool seen = KIND == kPooled ? (mean ? p < means : p <= pos && p >= lo) : h.sees(p, pos, lo);
+        s[j][e] = seen ? (KIND == kCapped ? h.capped(s[j][e] * h.scale) * kLog2E : s[j][e] * scale_log2) : -INFINITY;
         x[e >> 1] = fmaxf(x[e >> 1], s[j][e]);
       }
     float base[2], corr[2];
@@ -432,7 +629,12 @@ heads_rows_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__
     }
     const int head = head0 + g;
     if (num_splits == 1) {
-      float inv = L > 0.f ? 1.f / L : 0.f;
+      if (h.sink != nullptr) {
+        const float sink = h.sink_log2(head), top = fmaxf(most, sink), f = ex2(most - top);
+        L = L * f + ex2(sink - top);
+        acc *= f;
+      }
+      float inv = L > 0.f ? h.out_scale / L : 0.f;
       if (gate != nullptr) inv *= sigmoid_exact(to_f32(gate[size_t(t) * ld + h.gate_at(head, d)]));
       out[size_t(t) * ldo + size_t(head) * h.vdim + d] = from_f32<bf16>(acc * inv);
     } else {
@@ -454,13 +656,14 @@ heads_combine_kernel(const float* __restrict__ scratch, bf16* __restrict__ out, 
   pdl_wait();
   const int head = blockIdx.x, t = blockIdx.y, heads = h.heads, vdim = h.vdim;
   const float* src = scratch + size_t(t * heads + head) * num_splits * (vdim + 2);
-  float most = -INFINITY, L = 0.f;
+  float most = h.sink != nullptr ? h.sink_log2(head) : -INFINITY, L = 0.f;
   for (int s = 0; s < num_splits; ++s) most = fmaxf(most, src[s * (vdim + 2) + vdim]);
+  if (h.sink != nullptr) L = ex2(h.sink_log2(head) - most);
   for (int s = 0; s < num_splits; ++s) {
     const float ms = src[s * (vdim + 2) + vdim];
     L += src[s * (vdim + 2) + vdim + 1] * (ms == -INFINITY ? 0.f : ex2(ms - most));
   }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
+  const float inv = L > 0.f ? h.out_scale / L : 0.f;
   for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < num_splits; ++s) {
@@ -479,7 +682,7 @@ inline size_t chunk_smem(int dim, int vdim) {
 }
 
 // CTA = (64 queries of a sequence, head), 4 warps of 16 queries; key tiles of 64 (aligned to 64) through a two-stage ring.
-template <int DVT, bool CAP>
+template <int DVT, int KIND>
 __global__ void __launch_bounds__(128)
 heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict__ kc, const bf16* __restrict__ vc, Heads h,
                    const int* __restrict__ cu_q, const int* __restrict__ q_pos0, int first, bf16* __restrict__ out, int ldo,
@@ -502,10 +705,13 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
   const int p_first = q_pos0[s] + q0, p_last = q_pos0[s] + min(q_len, q0 + kChunkQ) - 1;
   const int see_all = h.first_seen(p_last);                        // from here on every query sees what is before it
   const int k_begin = h.first_seen(p_first) / kChunkKeys * kChunkKeys, k_end = p_last + 1;
-  // tiles of kept tokens, then those from k_begin on
-  const int kept = min(k_begin / kChunkKeys, (h.keep + kChunkKeys - 1) / kChunkKeys);
+  const int means = KIND == kPooled ? h.means_seen(p_last) : 0;
+  // tiles of kept tokens or of means, then those from k_begin on
+  const int kept = KIND == kPooled ? (means + kChunkKeys - 1) / kChunkKeys
+                                   : min(k_begin / kChunkKeys, (h.keep + kChunkKeys - 1) / kChunkKeys);
   const int count = kept + (k_end - k_begin + kChunkKeys - 1) / kChunkKeys;
   auto key_of = [&](int i) { return i < kept ? i * kChunkKeys : k_begin + (i - kept) * kChunkKeys; };
+  auto of_means = [&](int i) { return KIND == kPooled && i < kept; };
 
   for (int i = threadIdx.x; i < kChunkQ * ksteps * 2; i += 128) {
     const int r = i / (ksteps * 2), c = i % (ksteps * 2);
@@ -521,19 +727,20 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
   bool whole[2] = {true, true};                  // this thread's key of the stage exists
   auto issue = [&](int i) {
     if (i < count) {
-      const int st = i & 1, key0 = key_of(i);
+      const int st = i & 1, key0 = key_of(i), end = of_means(i) ? means : k_end;
+      const int* row = table + (of_means(i) ? h.means_at : 0);
       uint8_t *kd = sk + st * kChunkKeys * kp, *vd = sv + st * kChunkKeys * vp;
       if (threadIdx.x < kChunkKeys) {
         const int p = key0 + threadIdx.x;
-        const bool v = p < k_end && table[h.block_of(p)] >= 0;
+        const bool v = p < end && row[h.block_of(p)] >= 0;
         valid[st * kChunkKeys + threadIdx.x] = v;
         if (st == 0) whole[0] = v; else whole[1] = v;
       }
       // runs of 16 keys are contiguous in a block; a warp takes one run
-      const int tok = key0 + warp * 16, block = tok < k_end ? table[h.block_of(tok)] : -1;
+      const int tok = key0 + warp * 16, block = tok < end ? row[h.block_of(tok)] : -1;
       const size_t base_k = h.at(max(block, 0), kvh, h.in_block(tok), h.dp);
       const size_t base_v = h.at(max(block, 0), kvh, h.in_block(tok), h.vp);
-      const int rows = block < 0 ? 0 : min(16, k_end - tok);
+      const int rows = block < 0 ? 0 : min(16, end - tok);
       for (int idx = lane; idx < 16 * kch; idx += 32) {
         const int r = idx / kch, c = idx % kch;
         uint8_t* d = kd + (warp * 16 + r) * kp + c * 16;
@@ -554,8 +761,9 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
   const int rq = lane >> 2, cq = (lane & 3) * 2;
   const int pr0 = p_first + warp * 16 + rq;                        // positions of this thread's two query rows
   const int lo[2] = {h.first_seen(pr0), h.first_seen(pr0 + 8)};
+  const int seen_means[2] = {KIND == kPooled ? h.means_seen(pr0) : 0, KIND == kPooled ? h.means_seen(pr0 + 8) : 0};
   const uint32_t q_addr = smem_u32(sq) + (warp * 16 + (lane & 15)) * kp + (lane >> 4) * 16;
-  const float scale_log2 = CAP ? kLog2E : h.scale * kLog2E;
+  const float scale_log2 = KIND == kCapped ? kLog2E : h.scale * kLog2E;
 
   issue(0);
   for (int i = 0; i < count; ++i) {
@@ -580,13 +788,16 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
     }
     const int key0 = key_of(i);
     float x[2] = {-INFINITY, -INFINITY};
-    if constexpr (CAP) {
+    if constexpr (KIND == kCapped) {
 #pragma unroll
       for (int n = 0; n < 8; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) sc[n][e] = h.capped(sc[n][e] * h.scale);
     }
-    if (all_there && key0 + kChunkKeys - 1 <= p_first && (key0 >= see_all || key0 + kChunkKeys <= h.keep)) {
+    const bool mean = of_means(i);
+    const bool all_seen = mean ? key0 + kChunkKeys <= h.means_seen(p_first)
+                               : key0 + kChunkKeys - 1 <= p_first && (key0 >= see_all || key0 + kChunkKeys <= h.keep);
+    if (all_there && all_seen) {
 #pragma unroll
       for (int n = 0; n < 8; ++n)                // every query sees every key
 #pragma unroll
@@ -600,7 +811,9 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int c = n * 8 + cq + (e & 1), p = key0 + c;
-          const bool see = h.sees(p, pr0 + (e >> 1) * 8, lo[e >> 1]) && valid[(i & 1) * kChunkKeys + c] != 0;
+          const bool in_reach = KIND == kPooled ? (mean ? p < seen_means[e >> 1] : p <= pr0 + (e >> 1) * 8 && p >= lo[e >> 1])
+                                                : h.sees(p, pr0 + (e >> 1) * 8, lo[e >> 1]);
+          const bool see = in_reach && valid[(i & 1) * kChunkKeys + c] != 0;
           sc[n][e] = see ? sc[n][e] * scale_log2 : -INFINITY;
           x[e >> 1] = fmaxf(x[e >> 1], sc[n][e]);
         }
@@ -658,7 +871,13 @@ heads_chunk_kernel(const bf16* __restrict__ inp, int ld, const bf16* __restrict_
     const int r = q0 + warp * 16 + rq + half * 8;
     if (r >= q_len) continue;
     const size_t t = size_t(q_begin + r);
-    const float inv = L > 0.f ? 1.f / L : 0.f;
+    float inv;
+    if (h.sink != nullptr) {
+      const float sink = h.sink_log2(head), top = fmaxf(m[half], sink), f = ex2(m[half] - top);
+      inv = h.out_scale * f / (L * f + ex2(sink - top));
+    } else {
+      inv = L > 0.f ? h.out_scale / L : 0.f;
+    }
 #pragma unroll
     for (int n = 0; n < DVT; ++n) {
       const int c = n * 8 + cq;
@@ -690,7 +909,8 @@ Heads heads_of(const ZseHeads* h) {
     if (h->block_size == 1 << i) shift = i;
   return Heads{(long long)(h->block_stride), h->block_size, h->dim_pad, h->vdim_pad, h->max_blocks, shift,
                reinterpret_cast<const int*>(h->tables), h->heads, h->kv_heads, h->dim, h->vdim, h->chunk, h->window,
-               h->scale, h->keep_first, h->softcap, h->gate_each};
+               h->scale, h->keep_first, h->softcap, h->gate_each, h->pool, h->means_at,
+               reinterpret_cast<const float*>(h->sink), h->out_scale};
 }
 
 struct RowsCall {
@@ -705,10 +925,10 @@ struct RowsCall {
   cudaStream_t st;
 };
 
-template <int DKS, int DVT, bool CAP>
+template <int DKS, int DVT, int KIND>
 int launch_rows(const ZseHeads* z, const RowsCall& c) {
   static size_t done[kMaxDevices] = {};
-  auto kern = heads_rows_kernel<DKS, DVT, CAP>;
+  auto kern = heads_rows_kernel<DKS, DVT, KIND>;
   const Heads h = heads_of(z);
   const size_t smem = rows_smem(h.dim, h.vdim);
   if (int r = raise_smem(kern, smem, done)) return r;
@@ -719,24 +939,24 @@ int launch_rows(const ZseHeads* z, const RowsCall& c) {
              ? 0
              : ZSE_ERR_LAUNCH;
 }
-template <int DKS, bool CAP>
+template <int DKS, int KIND>
 int launch_rows_v(const ZseHeads* z, const RowsCall& c) {
-  return z->vdim <= 64    ? launch_rows<DKS, 8, CAP>(z, c)
-         : z->vdim <= 128 ? launch_rows<DKS, 16, CAP>(z, c)
-                          : launch_rows<DKS, 32, CAP>(z, c);
+  return z->vdim <= 64    ? launch_rows<DKS, 8, KIND>(z, c)
+         : z->vdim <= 128 ? launch_rows<DKS, 16, KIND>(z, c)
+                          : launch_rows<DKS, 32, KIND>(z, c);
 }
-template <bool CAP>
+template <int KIND>
 int launch_rows_k(const ZseHeads* z, const RowsCall& c) {
-  return z->dim <= 64    ? launch_rows_v<4, CAP>(z, c)
-         : z->dim <= 128 ? launch_rows_v<8, CAP>(z, c)
-                         : launch_rows_v<16, CAP>(z, c);
+  return z->dim <= 64    ? launch_rows_v<4, KIND>(z, c)
+         : z->dim <= 128 ? launch_rows_v<8, KIND>(z, c)
+                         : launch_rows_v<16, KIND>(z, c);
 }
 
-template <int DVT, bool CAP>
+template <int DVT, int KIND>
 int launch_chunks(const ZseHeads* z, const void* inp, int ld, const void* cu_q, const void* q_pos0, int first, int last,
                   int max_q, void* out, int ldo, const void* gate, cudaStream_t st) {
   static size_t done[kMaxDevices] = {};
-  auto kern = heads_chunk_kernel<DVT, CAP>;
+  auto kern = heads_chunk_kernel<DVT, KIND>;
   const Heads h = heads_of(z);
   const size_t smem = chunk_smem(h.dim, h.vdim);
   if (int r = raise_smem(kern, smem, done)) return r;
@@ -761,6 +981,37 @@ cudaError_t launch_prep(void* inp, const void* planes, int n_planes, int M, cons
                     reinterpret_cast<T*>(z->k), reinterpret_cast<T*>(z->v), h, reinterpret_cast<const long long*>(slots),
                     reinterpret_cast<const T*>(p->q_norm), reinterpret_cast<const T*>(p->k_norm),
                     reinterpret_cast<const T*>(p->bias), a, units);
+}
+
+template <typename T, int VEC>
+int launch_prep_whole(void* inp, const void* planes, int n_planes, int M, const ZseHeads* z, const void* slots,
+                      const ZseHeadsPrep* p, const HeadsPrepArgs& a, cudaStream_t st) {
+  static size_t done[2][kMaxDevices] = {};
+  const Heads h = heads_of(z);
+  const size_t smem = VEC == 1 ? size_t(h.heads) * h.dim * sizeof(float) : 0;
+  const bool few = M < 4 * 148;                  // as many threads as a row has work for
+  auto kern = few ? heads_prep_whole_kernel<T, VEC, 512> : heads_prep_whole_kernel<T, VEC, 256>;
+  if (smem > 40 * 1024)
+    if (int r = raise_smem(kern, smem, done[few])) return r;
+  return launch_pdl(kern, dim3(M), dim3(few ? 512 : 256), smem, st, reinterpret_cast<T*>(inp),
+                    reinterpret_cast<const float*>(planes), n_planes, M, reinterpret_cast<T*>(z->k),
+                    reinterpret_cast<T*>(z->v), h, reinterpret_cast<const long long*>(slots),
+                    reinterpret_cast<const T*>(p->q_norm), reinterpret_cast<const T*>(p->k_norm),
+                    reinterpret_cast<const T*>(p->bias), a, reinterpret_cast<const float*>(p->head_temp),
+                    p->pool_rows) == cudaSuccess
+             ? 0
+             : ZSE_ERR_LAUNCH;
+}
+
+// Vectors of four columns in every cached row.
+bool cache_vec(const ZseHeads* h) {
+  return h->dim % 4 == 0 && h->vdim % 4 == 0 && h->block_stride % 4 == 0 &&
+         !((reinterpret_cast<uintptr_t>(h->k) | reinterpret_cast<uintptr_t>(h->v)) & 15);
+}
+
+bool pool_ok(const ZseHeads* h) {
+  return h->pool >= 0 && (h->pool == 0 || (h->window > 0 && h->chunk == 0 && h->keep_first == 0 && h->softcap <= 0.f &&
+                                           h->means_at > 0 && h->means_at <= h->max_blocks));
 }
 
 }  // namespace
@@ -791,16 +1042,40 @@ extern "C" int zse_heads_prep(int dtype, void* inp, int ld, const void* planes, 
                       reinterpret_cast<uintptr_t>(h->k) | reinterpret_cast<uintptr_t>(h->v) |
                       reinterpret_cast<uintptr_t>(p->q_norm) | reinterpret_cast<uintptr_t>(p->k_norm) |
                       reinterpret_cast<uintptr_t>(p->bias)) & 15);
+  if (p->whole) {
+    if (p->temp_coef != 0.f || p->v_col == p->k_col || p->q_norm == nullptr || (p->own_kv && p->k_norm == nullptr) ||
+        (p->pool_rows && (!pool_ok(h) || p->positions == nullptr)))
+      return ZSE_ERR_SHAPE;
+    auto whole = dtype == kBF16 ? (vec ? launch_prep_whole<bf16, 4> : launch_prep_whole<bf16, 1>)
+                                : (vec ? launch_prep_whole<float, 4> : launch_prep_whole<float, 1>);
+    return whole(inp, planes, n_planes, M, h, slots, p, a, ST(stream));
+  }
   auto run = dtype == kBF16 ? (vec ? launch_prep<bf16, 4> : launch_prep<bf16, 1>)
                             : (vec ? launch_prep<float, 4> : launch_prep<float, 1>);
   return run(inp, planes, n_planes, M, h, slots, p, a, ST(stream)) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
+}
+
+extern "C" int zse_heads_pool(int dtype, const ZseHeads* z, const void* row_seq, const void* positions, int M, void* stream) {
+  if (M <= 0) return 0;
+  if (!pool_ok(z) || z->pool <= 0) return ZSE_ERR_SHAPE;
+  const Heads h = heads_of(z);
+  const dim3 grid((M + kPoolRows - 1) / kPoolRows);
+  const bool vec = cache_vec(z);
+  const int* seq = reinterpret_cast<const int*>(row_seq);
+  const int* pos = reinterpret_cast<const int*>(positions);
+  const cudaError_t e =
+      dtype == kBF16 ? launch_pdl(vec ? heads_pool_kernel<bf16, 4> : heads_pool_kernel<bf16, 1>, grid, dim3(256), 0, ST(stream),
+                                  reinterpret_cast<bf16*>(z->k), reinterpret_cast<bf16*>(z->v), h, seq, pos, M)
+                     : launch_pdl(vec ? heads_pool_kernel<float, 4> : heads_pool_kernel<float, 1>, grid, dim3(256), 0,
+                                  ST(stream), reinterpret_cast<float*>(z->k), reinterpret_cast<float*>(z->v), h, seq, pos, M);
+  return e == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }
 
 extern "C" int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads* z, const void* row_seq,
                               const void* positions, void* out, int ldo, const void* gate, void* scratch, int M,
                               int num_splits, int tensor_cores, void* stream) {
   if (M <= 0) return 0;
-  if (z->heads <= 0 || z->kv_heads <= 0 || z->heads % z->kv_heads || M > 65535) return ZSE_ERR_SHAPE;
+  if (z->heads <= 0 || z->kv_heads <= 0 || z->heads % z->kv_heads || M > 65535 || !pool_ok(z)) return ZSE_ERR_SHAPE;
   if (!tensor_cores || dtype != kBF16) {
     const Heads h = heads_of(z);
     const size_t smem = size_t(h.dim + 4 * h.vdim + 8) * sizeof(float);
@@ -824,7 +1099,9 @@ extern "C" int zse_heads_attn(int dtype, const void* inp, int ld, const ZseHeads
   const RowsCall c{reinterpret_cast<const bf16*>(inp), ld, reinterpret_cast<const int*>(row_seq),
                    reinterpret_cast<const int*>(positions), reinterpret_cast<bf16*>(out), ldo,
                    reinterpret_cast<const bf16*>(gate), reinterpret_cast<float*>(scratch), M, num_splits, ST(stream)};
-  int rc = z->softcap > 0.f ? launch_rows_k<true>(z, c) : launch_rows_k<false>(z, c);
+  int rc = z->pool > 0        ? launch_rows_k<kPooled>(z, c)
+           : z->softcap > 0.f ? launch_rows_k<kCapped>(z, c)
+                              : launch_rows_k<kPlainScores>(z, c);
   if (rc == 0 && num_splits > 1 &&
       launch_pdl(heads_combine_kernel, dim3(z->heads, M), dim3(128), 0, ST(stream), reinterpret_cast<const float*>(scratch),
                  c.out, ldo, c.gate, ld, heads_of(z), num_splits) != cudaSuccess)
@@ -837,7 +1114,7 @@ extern "C" int zse_heads_attn_chunks(const void* inp, int ld, int rows, const Zs
                                      const void* gate, int form, void* status, void* stream) {
   if (last <= first || max_q <= 0) return 0;
   if (!zse_heads_mma_ok(z->dim, z->vdim, z->block_size) || ld % 8 || ldo % 2 || z->block_stride % 8 ||
-      z->heads % z->kv_heads || z->heads > 65535 || last - first > 65535)
+      z->heads % z->kv_heads || z->heads > 65535 || last - first > 65535 || !pool_ok(z))
     return ZSE_ERR_SHAPE;
   const Heads h = heads_of(z);
   if (form == 1 && heads_tc_ok(h, z->num_blocks, ld, ldo))
@@ -845,10 +1122,16 @@ extern "C" int zse_heads_attn_chunks(const void* inp, int ld, int rows, const Zs
                            reinterpret_cast<const int*>(cu_q), reinterpret_cast<const int*>(q_pos0), first, last, max_q,
                            reinterpret_cast<bf16*>(out), ldo, reinterpret_cast<const bf16*>(gate),
                            reinterpret_cast<Status*>(status), ST(stream));
-  auto run = z->softcap > 0.f
-                 ? (z->vdim <= 64 ? launch_chunks<8, true> : z->vdim <= 128 ? launch_chunks<16, true> : launch_chunks<32, true>)
-                 : (z->vdim <= 64    ? launch_chunks<8, false>
-                    : z->vdim <= 128 ? launch_chunks<16, false>
-                                     : launch_chunks<32, false>);
+  auto run = z->pool > 0
+                 ? (z->vdim <= 64    ? launch_chunks<8, kPooled>
+                    : z->vdim <= 128 ? launch_chunks<16, kPooled>
+                                     : launch_chunks<32, kPooled>)
+             : z->softcap > 0.f
+                 ? (z->vdim <= 64    ? launch_chunks<8, kCapped>
+                    : z->vdim <= 128 ? launch_chunks<16, kCapped>
+                                     : launch_chunks<32, kCapped>)
+                 : (z->vdim <= 64    ? launch_chunks<8, kPlainScores>
+                    : z->vdim <= 128 ? launch_chunks<16, kPlainScores>
+                                     : launch_chunks<32, kPlainScores>);
   return run(z, inp, ld, cu_q, q_pos0, first, last, max_q, out, ldo, gate, ST(stream));
 }

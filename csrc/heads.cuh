@@ -14,6 +14,14 @@ struct Heads {
   int keep;                                      // first positions that are seen whatever the window
   float cap;                                     // > 0: scores become cap * tanh(score / cap)
   int gate_each;                                 // a gate per dimension of a head's result, not per head
+  int pool, means_at;                            // > 0: what lies before the window is seen as means of blocks of `pool` tokens;
+                                                 // rows of the cache whose blocks stand from column means_at on in the tables
+  const float* sink;                             // a score per head without a value, null: none
+  float out_scale;                               // factor of the result
+  // means that a row at `pos` sees: those of the blocks that lie wholly before its window
+  __device__ __forceinline__ int means_seen(int pos) const { return max(0, pos + 1 - window) / pool; }
+  // a head's sink as a score in units of ln 2
+  __device__ __forceinline__ float sink_log2(int head) const { return sink[head] * kLog2E; }
   // whether a row at `pos`, which sees from lo = first_seen(pos) on, sees position p
   __device__ __forceinline__ bool sees(int p, int pos, int lo) const { return p <= pos && (p >= lo || p < keep); }
   // cap * tanh(score / cap) of a scaled score; within 2^-22 of cap

@@ -10,7 +10,7 @@
 //   O += P V      P from TMEM in TWO bfloat16 terms, the weight and what rounding took from it, 64 columns each: together they
 //                 take the place of the 128 columns of scores; V is an MN-major operand as it lies in the cache
 // Tiles start at a multiple of the box, at or before the first key that the tile's first query sees; tiles of the tokens that
-// are always kept come before them.
+// are always kept, or of the means of older blocks of tokens, come before them.
 // Every wait is bounded; on a failure the loader waits for its copies and the CTA frees its TMEM and leaves.
 #include <cuda.h>
 
@@ -66,7 +66,7 @@ __device__ __forceinline__ uint64_t ht_desc_mn(uint32_t smem_addr) {
 
 // A cap bounds the scores: with one of up to kHtFixedCap the cap itself is the reference maximum of every row (weights down to
 // exp(-2 cap) are ordinary fp32 numbers), and a tile is read once.
-enum HtMode { kHtPlain = 0 /* no kept tokens, no cap */, kHtNoCap = 1, kHtCap = 2, kHtFixed = 3 };
+enum HtMode { kHtPlain = 0 /* no kept tokens, no cap */, kHtNoCap = 1, kHtCap = 2, kHtFixed = 3, kHtPooled = 4 };
 constexpr float kHtFixedCap = 40.f;
 
 template <int MODE>
@@ -89,12 +89,15 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
   const int p_first = a.q_pos0[seq] + qt * kHtRows, p_last = a.q_pos0[seq] + min(q_len, qt * kHtRows + kHtRows) - 1;
   const int br = a.box_rows;
   const int k_begin = a.h.first_seen(p_first) / br * br, k_end = p_last + 1;
-  // kept tokens before the others, in whole boxes
-  const int kept_end = MODE == kHtPlain ? 0 : min(k_begin, (a.h.keep + br - 1) / br * br);
+  // kept tokens before the others, in whole boxes; or the means that the tile's last query sees
+  const int kept_end = MODE == kHtPlain    ? 0
+                       : MODE == kHtPooled ? a.h.means_seen(p_last)
+                                           : min(k_begin, (a.h.keep + br - 1) / br * br);
   const int kept = (kept_end + kHtKeys - 1) / kHtKeys, n_tiles = kept + (k_end - k_begin + kHtKeys - 1) / kHtKeys;
   auto key_of = [&](int t) { return MODE != kHtPlain && t < kept ? t * kHtKeys : k_begin + (t - kept) * kHtKeys; };
   auto end_of = [&](int t) { return MODE != kHtPlain && t < kept ? kept_end : k_end; };
   const int* table = a.h.tables + size_t(seq) * a.h.max_blocks;
+  auto block_at = [&](int t, int tok) { return table[(MODE == kHtPooled && t < kept ? a.h.means_at : 0) + a.h.block_of(tok)]; };
 
   if (threadIdx.x == 0) {
     mbar_init(&bars->q_full, 1);
@@ -137,7 +140,7 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
     const uint32_t box_bytes = uint32_t(br) * 128u;
     auto group_block = [&](int t) {              // block of group g of tile t; -1: a hole, or past the end
       const int tok = key_of(t) + g * br;
-      return (g < n_groups && t < n_tiles && tok < end_of(t)) ? table[a.h.block_of(tok)] : -1;
+      return (g < n_groups && t < n_tiles && tok < end_of(t)) ? block_at(t, tok) : -1;
     };
     int next = group_block(0), issued_k = 0, issued_v = 0;
     uint32_t ph = 1;                             // "empty" barriers: the first wait passes
@@ -212,29 +215,36 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
     const int limit = a.q_pos0[seq] + row, lo = a.h.first_seen(limit);
     const uint32_t lane_addr = uint32_t(warp * 32) << 16;
     const float scale_log2 = a.h.scale * kLog2E;
-    auto sees = [&](int k) { return MODE == kHtPlain ? k <= limit && k >= lo : a.h.sees(k, limit, lo); };
+    const int means = MODE == kHtPooled ? a.h.means_seen(limit) : 0;
+    bool of_means = false;                       // the tile at hand
+    auto sees = [&](int k) {
+      if (MODE == kHtPooled && of_means) return k < means;
+      return MODE == kHtPlain || MODE == kHtPooled ? k <= limit && k >= lo : a.h.sees(k, limit, lo);
+    };
     auto log2_score = [&](float s) {
       return MODE == kHtCap || MODE == kHtFixed ? a.h.capped(s * a.h.scale) * kLog2E : s * scale_log2;
     };
     const int o_cols = (a.h.vdim + 15) / 16 * 16;
     const float cap_in = 2.f * a.h.scale * kLog2E / a.h.cap, cap_out = -2.f * a.h.cap * kLog2E;        // kHtFixed
-    float m_used = -INFINITY, l = 0.f;
+    // a sink is one more key of every row, with a value of zero
+    float m_used = a.h.sink != nullptr ? a.h.sink_log2(head) : -INFINITY, l = a.h.sink != nullptr ? 1.f : 0.f;
     uint32_t ph = 0;
     bool ok = true;
     for (int t = 0; t < n_tiles; ++t) {
       const int k0 = key_of(t), t_end = end_of(t);
       // which groups of 16 keys of the tile exist; looked up while S is still being computed
       const int g_tok = k0 + (lane & 7) * 16;
-      const uint32_t groups =
-          __ballot_sync(0xffffffffu, g_tok < t_end && table[a.h.block_of(g_tok)] >= 0) & 0xFFu;
+      const uint32_t groups = __ballot_sync(0xffffffffu, g_tok < t_end && block_at(t, g_tok) >= 0) & 0xFFu;
+      if constexpr (MODE == kHtPooled) of_means = t < kept;
       // one verdict per warp: the tcgen05.ld / st below are warp-wide
       if (!__all_sync(0xffffffffu, mbar_wait(&bars->s_full, ph, abort_flag, a.status, 98, t))) {
         ok = false;
         break;
       }
       tc_fence_after_sync();
-      const bool from_lo = k0 >= lo || (MODE != kHtPlain && k0 + kHtKeys <= a.h.keep);
-      const bool full = __all_sync(0xffffffffu, groups == 0xFFu && from_lo && k0 + kHtKeys - 1 <= limit);
+      const bool from_lo = k0 >= lo || (MODE != kHtPlain && MODE != kHtPooled && k0 + kHtKeys <= a.h.keep);
+      const bool whole = MODE == kHtPooled && of_means ? k0 + kHtKeys <= means : from_lo && k0 + kHtKeys - 1 <= limit;
+      const bool full = __all_sync(0xffffffffu, groups == 0xFFu && whole);
       float mx = -INFINITY;
 #pragma unroll 1
       for (int c = 0; MODE != kHtFixed && c < 4; ++c) {
@@ -342,7 +352,7 @@ heads_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
     if (ok) {
       const bool live = row < q_len;
       const size_t t = size_t(q_begin + (live ? row : 0));
-      float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? a.h.out_scale / l : 0.f;
       const bf16* gates = a.gate != nullptr && a.h.gate_each ? a.gate + t * a.ld + size_t(head) * a.h.vdim : nullptr;
       if (a.gate != nullptr && gates == nullptr) inv *= sigmoid_exact(to_f32(a.gate[t * a.ld + head]));
       bf16* dst = a.out + t * a.ldo + size_t(head) * a.h.vdim;
@@ -400,13 +410,14 @@ int launch_heads_tc(const bf16* inp, int ld, int rows, const void* k, const void
   if (int rc = get_tmap_rows3(v, num_blocks, per_block, h.vp, h.block_stride, br, 0, &mv)) return rc;
   const HtArgs a{h, cu_q, q_pos0, first, out, ldo, gate, ld, br, (h.dim + 63) / 64, (h.vdim + 63) / 64, status};
   const size_t smem = size_t(2 * a.k_panels + a.v_panels) * kHtPanel + 1024 + sizeof(HtBars);
-  static bool done[4][kMaxDevices] = {};
+  static bool done[5][kMaxDevices] = {};
   const int slot = current_device_slot();
-  const int mode = h.cap <= 0.f ? (h.keep > 0 ? kHtNoCap : kHtPlain) : h.cap <= kHtFixedCap ? kHtFixed : kHtCap;
-  auto kern = mode == kHtPlain   ? heads_tc_kernel<kHtPlain>
-              : mode == kHtNoCap ? heads_tc_kernel<kHtNoCap>
-              : mode == kHtCap   ? heads_tc_kernel<kHtCap>
-                                 : heads_tc_kernel<kHtFixed>;
+  const int mode = h.pool > 0 ? kHtPooled : h.cap <= 0.f ? (h.keep > 0 ? kHtNoCap : kHtPlain) : h.cap <= kHtFixedCap ? kHtFixed : kHtCap;
+  auto kern = mode == kHtPlain    ? heads_tc_kernel<kHtPlain>
+              : mode == kHtNoCap  ? heads_tc_kernel<kHtNoCap>
+              : mode == kHtCap    ? heads_tc_kernel<kHtCap>
+              : mode == kHtPooled ? heads_tc_kernel<kHtPooled>
+                                  : heads_tc_kernel<kHtFixed>;
   if (!done[mode][slot]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              int(6 * kHtPanel + 1024 + sizeof(HtBars))) != cudaSuccess)

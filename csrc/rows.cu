@@ -1,5 +1,6 @@
 // Row kernels for activations of bfloat16 or float: embedding (plain, or with a bigram table, a sinusoid and a norm),
-// residual sum + RMSNorm, RMSNorm + residual sum, logits epilogue, arg-max of fp32 logits.  Any row length.
+// residual sum + RMSNorm (+ a causal convolution over the normed rows), RMSNorm + residual sum, logits epilogue, arg-max of
+// fp32 logits.  Any row length.
 #include <initializer_list>
 
 #include "api.h"
@@ -58,11 +59,25 @@ __device__ __forceinline__ float row_cluster_sum(float total, float* slot, int c
   return total;
 }
 
-template <typename T, typename S, int VEC>
+// A causal convolution along every sequence, per channel, of rows h [M, H]: y = h + sum_j w[j] h_(t - taps + 1 + j).  State rows
+// hold a sequence's last taps - 1 rows of h, the oldest first: a pass reads them in one row of the pool (-1: zeros) and leaves
+// its own last ones in another.
+struct RowConv {
+  const float* w;                     // [taps][H], the row's own tap last
+  int taps;
+  float* states;
+  long long row_floats;
+  const int* state_rows;              // [2][state_ld]
+  int state_ld;
+};
+
+// CONV: every row is a sequence of its own; conv_out [M, H] = the row (as rounded into `out`) plus its convolution.
+template <typename T, typename S, int VEC, bool CONV>
 __global__ void __launch_bounds__(kRowThreads)
 add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, int n_planes,
                 const S* __restrict__ slots, int n_slots, const T* __restrict__ scale, int replace,
-                const T* __restrict__ weight, float offset, T* __restrict__ out, int ldo, int M, int H, float eps) {
+                const T* __restrict__ weight, float offset, T* __restrict__ out, int ldo, int M, int H, float eps,
+                const RowConv cv, T* __restrict__ conv_out) {
   __shared__ float red[32];
   __shared__ float cluster_ss;
   pdl_launch_dependents();
@@ -120,6 +135,105 @@ add_norm_kernel(float* __restrict__ residual, const float* __restrict__ planes, 
 #pragma unroll
       for (int e = 0; e < VEC; ++e) w.v[e] = (w.v[e] + offset) * (x[j].v[e] * inv);
       store_vec<VEC>(out + size_t(row) * ldo + size_t(i) * VEC, w);
+      if constexpr (CONV) {
+        const int read = cv.state_rows[row], write = cv.state_rows[cv.state_ld + row];
+        const int c = i * VEC;
+        const F32Vec<VEC> own = load_vec<VEC>(cv.w + size_t(cv.taps - 1) * H + c);
+        F32Vec<VEC> y;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          w.v[e] = to_f32(from_f32<T>(w.v[e]));
+          y.v[e] = fmaf(own.v[e], w.v[e], w.v[e]);
+        }
+        for (int k = 0; k + 1 < cv.taps; ++k) {
+          F32Vec<VEC> b{};
+          if (read >= 0) b = load_vec<VEC>(cv.states + size_t(read) * cv.row_floats + size_t(k) * H + c);
+          const F32Vec<VEC> f = load_vec<VEC>(cv.w + size_t(k) * H + c);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) y.v[e] = fmaf(f.v[e], b.v[e], y.v[e]);
+          if (write >= 0 && k > 0) store_vec<VEC>(cv.states + size_t(write) * cv.row_floats + size_t(k - 1) * H + c, b);
+        }
+        if (write >= 0 && cv.taps > 1)
+          store_vec<VEC>(cv.states + size_t(write) * cv.row_floats + size_t(cv.taps - 2) * H + c, w);
+        store_vec<VEC>(conv_out + size_t(row) * H + c, y);
+      }
+    }
+  }
+}
+
+// The convolution alone, over packed sequences.  A thread takes VEC columns of `rows` rows; TAPS 0: any number of taps.
+template <typename T, int VEC, int TAPS>
+__global__ void __launch_bounds__(kRowThreads)
+row_conv_kernel(const T* __restrict__ h, T* __restrict__ out, const RowConv cv, const int* __restrict__ row_seq,
+                const int* __restrict__ cu_q, int M, int H, int rows) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = (blockIdx.x * kRowThreads + threadIdx.x) * VEC, t0 = blockIdx.y * rows, t1 = min(M, t0 + rows);
+  if (c >= H) return;
+  const int taps = TAPS > 0 ? TAPS : cv.taps;
+  constexpr int kWin = TAPS > 1 ? TAPS - 1 : 1;
+  F32Vec<VEC> w[TAPS > 0 ? TAPS : 1], win[kWin];
+  if constexpr (TAPS > 0) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = load_vec<VEC>(cv.w + size_t(j) * H + c);
+  }
+  int begin = 0, end = -1, read = -1, write = -1;
+  // the row `back` rows before row t (back < taps): of this pass, of the state, or zero
+  auto before = [&](int t, int back) {
+    if (t - back >= begin) return load_vec<VEC>(h + size_t(t - back) * H + c);
+    if (read < 0) return F32Vec<VEC>{};
+    return load_vec<VEC>(cv.states + size_t(read) * cv.row_floats + size_t(taps - 1 + t - back - begin) * H + c);
+  };
+  constexpr int kAhead = 4;                      // rows whose loads are under way together
+  for (int tb = t0; tb < t1; tb += kAhead) {
+    F32Vec<VEC> in[kAhead];
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j)
+      if (tb + j < t1) in[j] = load_vec<VEC>(h + size_t(tb + j) * H + c);
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      const int t = tb + j;
+      if (t >= t1) break;
+      if (t >= end) {                            // the block's first row, or a sequence's
+        const int s = row_seq[t];
+        begin = cu_q[s];
+        end = cu_q[s + 1];
+        read = cv.state_rows[s];
+        write = cv.state_rows[cv.state_ld + s];
+        if constexpr (TAPS > 1) {
+#pragma unroll
+          for (int k = 0; k < TAPS - 1; ++k) win[k] = before(t, TAPS - 1 - k);
+        }
+      }
+      float* last = write >= 0 ? cv.states + size_t(write) * cv.row_floats + c : nullptr;
+      if (last != nullptr && t == begin && end - begin < taps - 1)   // what stays of the rows before a short portion
+        for (int k = 0; k + end - begin < taps - 1; ++k)
+          store_vec<VEC>(last + size_t(k) * H, before(t, taps - 1 - k - (end - begin)));
+      const F32Vec<VEC> x = in[j];
+      F32Vec<VEC> y = x;
+      if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y.v[e] = fmaf(w[TAPS - 1].v[e], x.v[e], y.v[e]);
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) y.v[e] = fmaf(w[k].v[e], win[k].v[e], y.v[e]);
+        if constexpr (TAPS > 1) {
+#pragma unroll
+          for (int k = 0; k + 1 < TAPS - 1; ++k) win[k] = win[k + 1];
+          win[TAPS - 2] = x;
+        }
+      } else {
+        for (int k = 0; k < taps; ++k) {
+          const F32Vec<VEC> f = load_vec<VEC>(cv.w + size_t(k) * H + c);
+          const F32Vec<VEC> v = k + 1 == taps ? x : before(t, taps - 1 - k);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) y.v[e] = fmaf(f.v[e], v.v[e], y.v[e]);
+        }
+      }
+      store_vec<VEC>(out + size_t(t) * H + c, y);
+      const int place = t - (end - (taps - 1));
+      if (last != nullptr && place >= 0) store_vec<VEC>(last + size_t(place) * H, x);
     }
   }
 }
@@ -158,11 +272,41 @@ template <typename T, typename S>
 int launch_add_norm(void* residual, const void* planes, int n_planes, const void* slots, int n_slots, const void* scale,
                     int replace, const void* weight, float offset, void* out, int ldo, int M, int H, float eps,
                     cudaStream_t st) {
-  return launch_rows(add_norm_kernel<T, S, 4>, add_norm_kernel<T, S, 1>,
+  return launch_rows(add_norm_kernel<T, S, 4, false>, add_norm_kernel<T, S, 1, false>,
                      aligned16({residual, weight, out, scale}) && ldo % 4 == 0, M, H, st,
                      reinterpret_cast<float*>(residual), reinterpret_cast<const float*>(planes), n_planes,
                      reinterpret_cast<const S*>(slots), n_slots, reinterpret_cast<const T*>(scale), replace,
-                     reinterpret_cast<const T*>(weight), offset, reinterpret_cast<T*>(out), ldo, M, H, eps);
+                     reinterpret_cast<const T*>(weight), offset, reinterpret_cast<T*>(out), ldo, M, H, eps, RowConv{},
+                     static_cast<T*>(nullptr));
+}
+
+RowConv conv_of(const ZseRowConv* z) {
+  return RowConv{reinterpret_cast<const float*>(z->w), z->taps, reinterpret_cast<float*>(z->states),
+                 (long long)(z->row_floats), reinterpret_cast<const int*>(z->state_rows), z->state_ld};
+}
+
+template <typename T>
+int launch_add_norm_conv(void* residual, const void* planes, int n_planes, const void* weight, void* out, const ZseRowConv* z,
+                         void* conv_out, int M, int H, float eps, cudaStream_t st) {
+  return launch_rows(add_norm_kernel<T, float, 4, true>, add_norm_kernel<T, float, 1, true>,
+                     aligned16({residual, weight, out, z->w, z->states, conv_out}) && z->row_floats % 4 == 0, M, H, st,
+                     reinterpret_cast<float*>(residual), reinterpret_cast<const float*>(planes), n_planes,
+                     static_cast<const float*>(nullptr), 0, static_cast<const T*>(nullptr), 0,
+                     reinterpret_cast<const T*>(weight), 0.f, reinterpret_cast<T*>(out), H, M, H, eps, conv_of(z),
+                     reinterpret_cast<T*>(conv_out));
+}
+
+template <typename T, int VEC>
+cudaError_t launch_row_conv(const void* h, void* out, const ZseRowConv* z, const void* row_seq, const void* cu_q, int M, int H,
+                            cudaStream_t st) {
+  const int rows = M >= 4096 ? 32 : M >= 512 ? 8 : 4;
+  const dim3 grid((H / VEC + kRowThreads - 1) / kRowThreads, (M + rows - 1) / rows);
+  auto kern = z->taps == 2   ? row_conv_kernel<T, VEC, 2>
+              : z->taps == 3 ? row_conv_kernel<T, VEC, 3>
+              : z->taps == 4 ? row_conv_kernel<T, VEC, 4>
+                             : row_conv_kernel<T, VEC, 0>;
+  return launch_pdl(kern, grid, dim3(kRowThreads), 0, st, reinterpret_cast<const T*>(h), reinterpret_cast<T*>(out), conv_of(z),
+                    reinterpret_cast<const int*>(row_seq), reinterpret_cast<const int*>(cu_q), M, H, rows);
 }
 
 // y = sum of fp32 planes + sum of the row's slots; residual += RMSNorm(y) * weight; out = residual, or (next != null)
@@ -446,6 +590,24 @@ extern "C" int zse_add_norm(int dtype, int slot_dtype, void* residual, const voi
              : slot_dtype == kF32 ? launch_add_norm<bf16, float>
                                   : launch_add_norm<bf16, bf16>;
   return run(residual, planes, n_planes, slots, n_slots, scale, replace, weight, offset, out, ldo, M, H, eps, ST(stream));
+}
+
+extern "C" int zse_add_norm_conv(int dtype, void* residual, const void* planes, int n_planes, const void* weight, void* out,
+                                 const ZseRowConv* z, void* conv_out, int M, int H, float eps, void* stream) {
+  if (M <= 0) return 0;
+  if (z->taps < 1) return ZSE_ERR_SHAPE;
+  auto run = dtype == kF32 ? launch_add_norm_conv<float> : launch_add_norm_conv<bf16>;
+  return run(residual, planes, n_planes, weight, out, z, conv_out, M, H, eps, ST(stream));
+}
+
+extern "C" int zse_row_conv(int dtype, const void* h, void* out, const ZseRowConv* z, const void* row_seq, const void* cu_q,
+                            int M, int H, void* stream) {
+  if (M <= 0) return 0;
+  if (z->taps < 1 || M > 65535 * 4) return ZSE_ERR_SHAPE;
+  const bool vec = H % 4 == 0 && z->row_floats % 4 == 0 && aligned16({h, out, z->w, z->states});
+  auto run = dtype == kF32 ? (vec ? launch_row_conv<float, 4> : launch_row_conv<float, 1>)
+                           : (vec ? launch_row_conv<bf16, 4> : launch_row_conv<bf16, 1>);
+  return run(h, out, z, row_seq, cu_q, M, H, ST(stream)) == cudaSuccess ? 0 : ZSE_ERR_LAUNCH;
 }
 
 extern "C" int zse_post_norm(int dtype, int slot_dtype, void* residual, const void* planes, int n_planes,

@@ -328,8 +328,10 @@ class HybridModel(DesignModel):
     def _attend(self, b, p: Pass, run: LayerRun, s: HeadsSpec, inp, planes, n_in: int, out) -> None:
         ops, L, M = self.ops, run.layer, p.M
         view = self._heads_view(p.kv, run)
-        ops.heads_prep(inp, planes, n_in, view, b.slots, L, s, self.config.rms_norm_eps, M, b.positions)
-        if s.pool:
+        alone = s.pool > 0 and p.row_seq is None           # a decode step's rows leave the means of blocks themselves
+        ops.heads_prep(inp, planes, n_in, view, b.slots, L, s, self.config.rms_norm_eps, M, b.positions,
+                       b.block_tables if alone else None)
+        if s.pool and not alone:
             ops.heads_pool(view, b.block_tables, p.row_seq, b.positions, s, M)
         rows, seqs = p.short if ops.heads_expands(s, self.act_dtype) else (M, p.num_seqs)
         if rows:
@@ -353,7 +355,7 @@ class HybridModel(DesignModel):
 
     def _recall(self, b, p: Pass, run: LayerRun, s: GatedLinearSpec, inp, planes, n_in: int, out) -> None:
         ops, L, M, eps, states = self.ops, run.layer, p.M, self.config.rms_norm_eps, self.states.rows
-        seqs = p.short[1] if ops.gated_linear_expands(s, self.act_dtype) else p.num_seqs
+        rows, seqs = p.short if ops.gated_linear_expands(s, self.act_dtype) else (M, p.num_seqs)
         decays = b.decays
         if n_in and seqs == p.num_seqs:
             decays = None                    # token by token only: the step's kernel reads the planes
@@ -363,8 +365,8 @@ class HybridModel(DesignModel):
             ops.gated_linear_tokens(inp, planes, n_in, decays, states, run.state_at, b.state_rows, p.cu_q, L, out, seqs, M, s,
                                     eps)
         if seqs < p.num_seqs:
-            ops.gated_linear_chunks(inp, decays, states, run.state_at, b.state_rows, b.cu_q, L, out, seqs, p.num_seqs, M, s,
-                                    eps, b.linear_ws)
+            ops.gated_linear_chunks(inp, decays, states, run.state_at, b.state_rows, b.cu_q, L, out, seqs, p.num_seqs,
+                                    rows, M, s, eps, b.linear_ws)
 
     def _space(self, b, p: Pass, run: LayerRun, s: StateSpaceSpec, inp, planes, n_in: int, out) -> None:
         ops, L, M, states = self.ops, run.layer, p.M, self.states.rows

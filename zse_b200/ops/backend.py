@@ -296,13 +296,15 @@ class TorchOps:
             return None
         return base ** (-torch.arange(0, dims, 2, dtype=torch.float64, device=self.device) / dims) / factor
 
-    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M, positions=None):
+    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M, positions=None, block_tables=None):
         if n_planes:
             ld, w = inp.shape[1], spec.in_width
             inp[:M, :w] = planes.view(-1)[: n_planes * M * ld].view(n_planes, M, ld)[..., :w].sum(0)
         ref.heads_prep(inp[:M], kv.k if kv else None, kv.v if kv else None, slots[:M], spec, L.q_norm, L.k_norm, eps,
                        None if positions is None else positions[:M].long(), getattr(L, "bias", None),
                        getattr(L, "freqs", None), getattr(L, "temp", None))
+        if spec.pool and block_tables is not None:
+            self.heads_pool(kv, block_tables, None, positions, spec, M)
 
     def heads_pool(self, kv, block_tables, row_seq, positions, spec, M):
         """Means of the blocks of ``spec.pool`` tokens that rows [0, M) complete, from the cached keys and values into the cache.
@@ -1017,27 +1019,33 @@ class CudaOps(TorchOps):
         hi = f.float()
         return torch.stack([hi, (f - hi.double()).float()], 1).contiguous()
 
-    def rotation(self, dims: int, base: float):
-        f = super().rotation(dims, base)
+    def rotation(self, dims: int, base: float, factor: float = 1.0):
+        f = super().rotation(dims, base, factor)
         return None if f is None else self._turns(f)
 
-    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M, positions=None):
-        self.n.heads_prep(inp, planes, n_planes, M, self.n.heads(kv, spec, self._no_tables), slots, L.q_norm, L.k_norm,
-                          getattr(L, "bias", None), getattr(L, "freqs", None), positions, spec, eps)
+    def heads_prep(self, inp, planes, n_planes, kv, slots, L, spec, eps, M, positions=None, block_tables=None):
+        """``block_tables``: of a pass whose rows are sequences of their own, which leaves the means of blocks as well."""
+        tables = self._no_tables if block_tables is None else block_tables
+        self.n.heads_prep(inp, planes, n_planes, M, self.n.heads(kv, spec, tables), slots, L.q_norm, L.k_norm,
+                          getattr(L, "bias", None), getattr(L, "freqs", None), positions, spec, eps,
+                          getattr(L, "temp", None), block_tables is not None)
+
+    def heads_pool(self, kv, block_tables, row_seq, positions, spec, M):
+        self.n.heads_pool(self.n.heads(kv, spec, block_tables), kv.k.dtype, row_seq, positions, M)
 
     @staticmethod
     def _head_gate(inp, spec):
         return inp.data_ptr() + spec.gate_col * inp.element_size() if spec.gated else None
 
-    def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits):
+    def heads_attn(self, inp, kv, block_tables, row_seq, positions, out, M, spec, scratch, num_splits, sink=None):
         tc = inp.dtype == torch.bfloat16 and self.n.heads_mma_ok(spec, kv.block_size)
         if not tc or scratch.numel() < M * num_splits * spec.heads * (spec.vdim + 2):
             num_splits = 1
-        self.n.heads_attn(inp, self.n.heads(kv, spec, block_tables), row_seq, positions, out, self._head_gate(inp, spec),
-                          scratch, M, num_splits, tc)
+        self.n.heads_attn(inp, self.n.heads(kv, spec, block_tables, sink), row_seq, positions, out,
+                          self._head_gate(inp, spec), scratch, M, num_splits, tc)
 
-    def heads_attn_chunks(self, inp, kv, block_tables, cu_q, q_pos0, positions, first, last, max_q, out, spec):
-        self.n.heads_attn_chunks(inp, self.n.heads(kv, spec, block_tables), cu_q, q_pos0, first, last, max_q, out,
+    def heads_attn_chunks(self, inp, kv, block_tables, cu_q, q_pos0, positions, first, last, max_q, out, spec, sink=None):
+        self.n.heads_attn_chunks(inp, self.n.heads(kv, spec, block_tables, sink), cu_q, q_pos0, first, last, max_q, out,
                                  self._head_gate(inp, spec), self.heads_form, self.status.ptr)
 
     def memory_expands(self, spec, dtype) -> bool:
@@ -1073,6 +1081,37 @@ class CudaOps(TorchOps):
     def state_space_chunks(self, inp, xbc, dt, states, at, state_rows, cu_q, L, out, first, last, M, spec):
         """Sequences ``first .. last - 1`` chunkwise."""
         self.n.space_chunks(inp, xbc, dt, self.n.space(states, at, state_rows, L, spec), cu_q, first, last, out)
+
+    def gated_linear_expands(self, spec, dtype) -> bool:
+        return dtype == torch.bfloat16 and self.n.gated_linear_chunk_ok(spec)
+
+    def gated_linear_workspace(self, specs, max_tokens: int):
+        return torch.zeros(max_tokens * max(s.heads * s.vdim for s in specs), dtype=torch.float32, device=self.device)
+
+    def gated_linear_prep(self, inp, planes, n_planes, side, decays, L, spec, M):
+        if not self.linear_has_side(L.w_in):
+            side = None
+        self.n.gated_linear_prep(inp, planes, n_planes, side, spec.in_width - spec.rank_col,
+                                 self.n.gated_linear(None, 0, None, L, spec, 0.0), decays, M)
+
+    def gated_linear_tokens(self, inp, planes, n_planes, decays, states, at, state_rows, cu_q, L, out, S, M, spec, eps):
+        self.n.gated_linear_tokens(inp, planes, n_planes, M, decays,
+                                   self.n.gated_linear(states, at, state_rows, L, spec, eps), cu_q, S, out)
+
+    def gated_linear_chunks(self, inp, decays, states, at, state_rows, cu_q, L, out, first, last, row0, M, spec, eps, ws):
+        """Sequences ``first .. last - 1`` chunkwise; their rows are [row0, M)."""
+        self.n.gated_linear_chunks(inp, decays, self.n.gated_linear(states, at, state_rows, L, spec, eps), cu_q, first, last,
+                                   ws, M, row0, out)
+
+    def add_norm_conv(self, residual, partials, n_partials, weight, out, conv_w, conv_out, states, at, state_rows, row_seq,
+                      cu_q, M, S, eps):
+        n, H = self.n, residual.shape[1]
+        cv = n.row_conv_args(conv_w, states, at, state_rows)
+        if cu_q is None:                     # every row is a sequence of its own: one kernel
+            n.add_norm_conv(residual, partials, n_partials, weight, out, cv, conv_out, M, H, float(eps))
+            return
+        self.add_norm(residual, partials, n_partials, None, weight, out, M, eps)
+        n.row_conv(out, conv_out, cv, row_seq, cu_q, M, H)
 
     def group_norm(self, x, weight, parts: int, M, eps):
         self.n.group_norm(x, weight, parts, M, eps)

@@ -162,6 +162,7 @@ GROUPS = {
                "sampling.cu"),
     "looped": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "heads.cu", "heads_tc.cu", "state_space.cu", "moe.cu",
                "sampling.cu"),
+    "twin": ("runtime.cu", "rows.cu", "gemm.cu", "gemm_tile.cu", "heads.cu", "heads_tc.cu", "gated_linear.cu", "sampling.cu"),
 }
 
 

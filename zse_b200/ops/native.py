@@ -72,13 +72,27 @@ class Heads(Structure):
     _fields_ = [("k", c_void_p), ("v", c_void_p), ("block_stride", c_int64)] + \
                [(n, c_int32) for n in ("block_size", "dim_pad", "vdim_pad", "max_blocks")] + [("tables", c_void_p)] + \
                [(n, c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "chunk", "window")] + [("scale", c_float),
-                   ("num_blocks", c_int32), ("keep_first", c_int32), ("softcap", c_float), ("gate_each", c_int32)]
+                   ("num_blocks", c_int32), ("keep_first", c_int32), ("softcap", c_float), ("gate_each", c_int32),
+                   ("pool", c_int32), ("means_at", c_int32), ("sink", c_void_p), ("out_scale", c_float)]
 
 
 class HeadsPrep(Structure):
     _fields_ = [(n, c_void_p) for n in ("q_norm", "k_norm", "bias", "turns", "positions")] + \
                [(n, c_int32) for n in ("k_col", "v_col", "gate_col", "gate_w", "own_kv", "rot_dims")] + \
-               [("temp_coef", c_float), ("temp_every", c_int32), ("eps", c_float)]
+               [("temp_coef", c_float), ("temp_every", c_int32), ("eps", c_float), ("whole", c_int32),
+                ("head_temp", c_void_p), ("pool_rows", c_int32)]
+
+
+class RowConv(Structure):
+    _fields_ = [("w", c_void_p), ("taps", c_int32), ("states", c_void_p), ("row_floats", c_int64), ("state_rows", c_void_p),
+                ("state_ld", c_int32)]
+
+
+class GatedLinear(Structure):
+    _fields_ = [(n, c_int32) for n in ("heads", "dim", "vdim", "rank", "q_col", "k_col", "v_col", "gate_col", "rank_col")] + \
+               [("states", c_void_p), ("row_floats", c_int64), ("state_rows", c_void_p), ("state_ld", c_int32),
+                ("tau", c_float), ("eps", c_float), ("out_scale", c_float)] + \
+               [(n, c_void_p) for n in ("head_norm", "decay_w", "decay_b")]
 
 
 class Memory(Structure):
@@ -213,6 +227,9 @@ _SIGS = {
                                     c_void_p, c_void_p]),
     "zse_add_norm": (c_int, [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float,
                              c_void_p, c_int, c_int, c_int, c_float, c_void_p]),
+    "zse_add_norm_conv": (c_int, [c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, POINTER(RowConv), c_void_p, c_int,
+                                  c_int, c_float, c_void_p]),
+    "zse_row_conv": (c_int, [c_int, c_void_p, c_void_p, POINTER(RowConv), c_void_p, c_void_p, c_int, c_int, c_void_p]),
     "zse_logits_finish": (c_int, [c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p]),
     "zse_argmax_f32": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p]),
     "zse_latent_mma_ok": (c_int, [c_int] * 6),
@@ -230,10 +247,11 @@ _SIGS = {
     "zse_post_norm": (c_int, [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                               c_int, c_float, c_void_p]),
     "zse_embed_design": (c_int, [c_int, POINTER(Embed), c_int, c_void_p, c_void_p]),
-    "zse_glu": (c_int, [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p]),
+    "zse_glu": (c_int, [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]),
     "zse_heads_mma_ok": (c_int, [c_int] * 3),
     "zse_heads_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_int, POINTER(Heads), c_void_p, POINTER(HeadsPrep),
                                c_void_p]),
+    "zse_heads_pool": (c_int, [c_int, POINTER(Heads), c_void_p, c_void_p, c_int, c_void_p]),
     "zse_heads_attn": (c_int, [c_int, c_void_p, c_int, POINTER(Heads), c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                c_void_p, c_int, c_int, c_int, c_void_p]),
     "zse_heads_attn_chunks": (c_int, [c_void_p, c_int, c_int, POINTER(Heads), c_void_p, c_void_p, c_int, c_int, c_int,
@@ -252,6 +270,13 @@ _SIGS = {
                                  c_void_p]),
     "zse_space_chunks": (c_int, [c_void_p, c_int, c_void_p, c_void_p, POINTER(Space), c_void_p, c_int, c_int, c_void_p, c_int,
                                  c_void_p]),
+    "zse_gated_linear_chunk_ok": (c_int, [c_int] * 2),
+    "zse_gated_linear_prep": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, POINTER(GatedLinear), c_void_p,
+                                      c_int, c_void_p]),
+    "zse_gated_linear_tokens": (c_int, [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, POINTER(GatedLinear),
+                                        c_void_p, c_int, c_void_p, c_int, c_void_p]),
+    "zse_gated_linear_chunks": (c_int, [c_void_p, c_int, c_void_p, POINTER(GatedLinear), c_void_p, c_int, c_int, c_void_p,
+                                        c_int, c_int, c_void_p, c_int, c_void_p]),
     "zse_group_norm": (c_int, [c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p]),
     "zse_moe_gemm": (c_int, [POINTER(MoeGemm), c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
     "zse_read_probe": (c_int, [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p]),
@@ -628,26 +653,48 @@ def embed_design(a: Embed, dtype, M, status):
 
 
 def glu(x, out, rows, ff, kind, limit):
-    _ck(load().zse_glu(_DTYPE[x.dtype], _p(x), _p(out), rows, ff, kind, float(limit), _stream()), "glu")
+    _ck(load().zse_glu(_DTYPE[x.dtype], _p(x), _p(out), out.stride(0) if out.dim() > 1 else ff, rows, ff, kind, float(limit),
+                       _stream()), "glu")
 
 
-def heads(view, spec, block_tables) -> Heads:
+def row_conv_args(w, states, at, state_rows) -> RowConv:
+    """``w`` [taps, H]; ``states``: the state pool's rows; ``at``: where the layer's part of a row begins."""
+    return RowConv(_p(w), w.shape[0], states.data_ptr() + 4 * at, states.stride(0), _p(state_rows), state_rows.stride(0))
+
+
+def add_norm_conv(residual, planes, n_planes, weight, out, cv, conv_out, M, H, eps):
+    _ck(load().zse_add_norm_conv(_DTYPE[out.dtype], _p(residual), _p(planes), n_planes, _p(weight), _p(out), byref(cv),
+                                 _p(conv_out), M, H, eps, _stream()), "add_norm_conv")
+
+
+def row_conv(h, out, cv, row_seq, cu_q, M, H):
+    _ck(load().zse_row_conv(_DTYPE[h.dtype], _p(h), _p(out), byref(cv), _p(row_seq), _p(cu_q), M, H, _stream()), "row_conv")
+
+
+def heads(view, spec, block_tables, sink=None) -> Heads:
     """``view``: ``models.hybrid.PagedHeads``."""
     return Heads(view.k.data_ptr(), view.v.data_ptr(), view.block_stride, view.block_size, view.k.shape[3], view.v.shape[3],
                  block_tables.stride(0), block_tables.data_ptr(), spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.chunk,
-                 spec.window, float(spec.scale), view.k.shape[0], spec.keep_first, float(spec.softcap), int(spec.gate_each))
+                 spec.window, float(spec.scale), view.k.shape[0], spec.keep_first, float(spec.softcap), int(spec.gate_each),
+                 spec.pool, getattr(view, "means_at", 0), _p(sink), float(spec.out_scale))
 
 
 def heads_mma_ok(spec, block_size: int) -> bool:
     return bool(load().zse_heads_mma_ok(spec.dim, spec.vdim, block_size))
 
 
-def heads_prep(inp, planes, n_planes, M, h, slots, q_norm, k_norm, bias, turns, positions, spec, eps):
+def heads_prep(inp, planes, n_planes, M, h, slots, q_norm, k_norm, bias, turns, positions, spec, eps, head_temp=None,
+               pool_rows=False):
     p = HeadsPrep(_p(q_norm), _p(k_norm), _p(bias), _p(turns), _p(positions), spec.k_col,
                   spec.k_col if spec.k_as_v else spec.v_col, spec.gate_col, spec.gate_width, int(spec.own_kv), spec.rot_dims,
-                  float(spec.temp_coef), int(spec.temp_every), float(eps))
+                  float(spec.temp_coef), int(spec.temp_every), float(eps), int(spec.whole_norm), _p(head_temp),
+                  int(pool_rows))
     _ck(load().zse_heads_prep(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, M, byref(h), _p(slots),
                               byref(p), _stream()), "heads_prep")
+
+
+def heads_pool(h, dtype, row_seq, positions, M):
+    _ck(load().zse_heads_pool(_DTYPE[dtype], byref(h), _p(row_seq), _p(positions), M, _stream()), "heads_pool")
 
 
 def heads_attn(inp, h, row_seq, positions, out, gate, scratch, M, num_splits, tensor_cores):
@@ -713,6 +760,34 @@ def space_tokens(inp, xbc, dt, m, cu_q, S, out):
 def space_chunks(inp, xbc, dt, m, cu_q, first, last, out):
     _ck(load().zse_space_chunks(_p(inp), inp.stride(0), _p(xbc), _p(dt), byref(m), _p(cu_q), first, last, _p(out),
                                 out.stride(0), _stream()), "space_chunks")
+
+
+def gated_linear(states, at, state_rows, L, spec, eps) -> GatedLinear:
+    """``states``: the state pool's rows (None: of a call that needs none); ``at``: where the layer's part of a row begins."""
+    return GatedLinear(spec.heads, spec.dim, spec.vdim, spec.rank, spec.col, spec.k_col, spec.v_col, spec.gate_col,
+                       spec.rank_col, None if states is None else states.data_ptr() + 4 * at,
+                       0 if states is None else states.stride(0), _p(state_rows),
+                       0 if state_rows is None else state_rows.stride(0), float(spec.tau), float(eps), float(spec.out_scale),
+                       _p(L.head_norm), _p(L.decay_w), _p(L.decay_b))
+
+
+def gated_linear_chunk_ok(spec) -> bool:
+    return bool(load().zse_gated_linear_chunk_ok(spec.dim, spec.vdim))
+
+
+def gated_linear_prep(inp, planes, n_planes, side, side_ld, m, decays, M):
+    _ck(load().zse_gated_linear_prep(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, _p(side), side_ld,
+                                     byref(m), _p(decays), M, _stream()), "gated_linear_prep")
+
+
+def gated_linear_tokens(inp, planes, n_planes, M, decays, m, cu_q, S, out):
+    _ck(load().zse_gated_linear_tokens(_DTYPE[inp.dtype], _p(inp), inp.stride(0), _p(planes), n_planes, M, _p(decays),
+                                       byref(m), _p(cu_q), S, _p(out), out.stride(0), _stream()), "gated_linear_tokens")
+
+
+def gated_linear_chunks(inp, decays, m, cu_q, first, last, o, M, row0, out):
+    _ck(load().zse_gated_linear_chunks(_p(inp), inp.stride(0), _p(decays), byref(m), _p(cu_q), first, last, _p(o), M, row0,
+                                       _p(out), out.stride(0), _stream()), "gated_linear_chunks", 2)
 
 
 def group_norm(x, weight, parts, M, eps):
