@@ -77,6 +77,21 @@ def movinex_design(width: int, vocab: int, heads: int, kv_heads: int, dim: int, 
             "layers": kinds + [kinds[i] for i in tail], "logit_scale": 1.0, "loop": {"start": 0, "stop": 3, "times": times}}
 
 
+def vobisun_design(width: int, vocab: int, heads: int, kv_heads: int, dim: int, window: int, pool: int, memory: tuple, ff: int,
+                   layers: int, loop: tuple = (), rot: int = 0, taps: int = 4, eps: float = 1e-6) -> dict:
+    """A Vobisun ``config.json`` of equal layers; ``memory``: heads, dim, vdim of the gated linear attention, ``loop``: start,
+    stop, times."""
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+            "mask": {"size": window, "pool": pool},
+            "rot": {"dims": rot or dim, "base": 10000.0, "scaling": {"factor": 1.0}}}
+    layer = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff},
+             "mixer": {"left": left, "right": dict(zip(("heads", "dim", "vdim"), memory), tau=16.0), "left_scale": 1.0,
+                       "right_scale": 1.0}}
+    c = {"architecture": "Vobisun", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": [layer] * layers,
+         "canon": {"taps": taps}, "embedding": {"scale": width ** 0.5}}
+    return dict(c, loop=dict(zip(("start", "stop", "times"), loop))) if loop else c
+
+
 # entries with a "design" hold a config.json of that architecture instead of ``ModelConfig`` fields
 SHAPES = {
     "tiny-ruralorn": dict(arch="ruralorn", design=ruralorn_design(3, 192, 1024, 6, 24, 8, 40, 56, 40, 10, 3, 72, 104)),
@@ -97,6 +112,12 @@ SHAPES = {
                                                              1408, (8, 4), tail=(1, 2), rot=64)),
     "movinex-4k": dict(arch="movinex", design=movinex_design(4096, 102400, 32, 8, 128, 2048, 64, (128, 64, 128, 8), 14336, 64,
                                                              4, 2048, (8, 4), times=1, rot=64)),
+    "tiny-vobisun": dict(arch="vobisun", design=vobisun_design(160, 1024, 6, 2, 32, 48, 6, (3, 40, 56), 224, 3, (0, 2, 2),
+                                                               rot=16)),
+    "vobisun-2k": dict(arch="vobisun", design=vobisun_design(2048, 102400, 16, 4, 128, 2048, 16, (16, 128, 256), 8192, 6,
+                                                             (1, 3, 2), rot=64)),
+    "vobisun-4k": dict(arch="vobisun", design=vobisun_design(4096, 102400, 32, 8, 128, 2048, 16, (32, 128, 256), 14336, 4,
+                                                             rot=64)),
     "tiny": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64, intermediate_size=688,
                  vocab_size=1024, rms_norm_eps=1e-6, rope_theta=10000.0, arch="llama", max_seq_len=2048),
     "tiny-aligned": dict(num_layers=2, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64,
