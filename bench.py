@@ -38,7 +38,7 @@ NUM_REQUESTS = 64
 PROMPT_RANGE = (128, 2048)
 OUTPUT_TOKENS = 256
 # name -> model shape, requests, prompt rule, output tokens, speculative depth, (adapters, rank)
-DESIGNS = ("ruralorn", "nimelorn", "movinex")      # models of listed layers, beside a neighbour of equal size
+DESIGNS = ("ruralorn", "nimelorn", "movinex", "vobisun")      # models of listed layers, beside a neighbour of equal size
 WORKLOADS = {
     "batch64": dict(model="qwen2.5-14b", requests=64, prompt=("uniform",) + PROMPT_RANGE, out=256, spec_k=0, lora=None,
                     seq_len=f"prompts uniform {PROMPT_RANGE}, 256 output tokens"),
@@ -70,14 +70,15 @@ def parse_args():
     ap.add_argument("--spec-k", type=int, default=None,
                     help="override the workload's number of draft tokens per step (0: plain decoding of the same requests)")
     ap.add_argument("--kernels-file", default=None, metavar="FILE",
-                    help="with --workload ruralorn, nimelorn or movinex: also time every kernel alone and write the roofline table to FILE")
+                    help="with --workload ruralorn, nimelorn, movinex or vobisun: also time every kernel alone and write the roofline table to FILE")
     ap.add_argument("--workload", default="batch64", choices=sorted(WORKLOADS) + list(DESIGNS),
                     help="batch64: 64 requests, prompts uniform in [128, 2048] (the headline); single: one request "
                          "with a 512-token prompt on the 7B shape (the case the reference publishes); spec32b: n-gram "
                          "speculative decoding on the 32B shape; lora72b: 256 requests over 32 adapters on the 72B shape; ruralorn: prefill and decode of the "
                          "latent-attention / routed design at two sizes beside a dense model of equal size (one GPU); nimelorn: the "
                          "same for the design of chunked attention, matrix memories and gated experts; movinex: looped layers of "
-                         "attention, windowed attention and state spaces beside a Nimelorn model of equal size")
+                         "attention, windowed attention and state spaces beside a Nimelorn model of equal size; vobisun: windowed "
+                         "attention over tokens and block means beside gated linear attention, next to a Movinex model")
     a = ap.parse_args()
     if a.workload not in ("batch64",) + DESIGNS:
         w = WORKLOADS[a.workload]
@@ -402,11 +403,13 @@ def run_ours(args):
 
 def run_designs(args):
     """bfloat16 shapes of a design beside their neighbours (zse_b200/runtime/design_bench.py, hybrid_bench.py,
-    looped_bench.py)."""
+    looped_bench.py, twin_bench.py)."""
     if args.workload == "nimelorn":
         from zse_b200.runtime import hybrid_bench as design_bench
     elif args.workload == "movinex":
         from zse_b200.runtime import looped_bench as design_bench
+    elif args.workload == "vobisun":
+        from zse_b200.runtime import twin_bench as design_bench
     else:
         from zse_b200.runtime import design_bench
     if int(os.environ.get("WORLD_SIZE", "1")) > 1:
