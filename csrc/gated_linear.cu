@@ -18,7 +18,8 @@
 // A is made in blocks of 16 tokens: with r the b before the first token of t's block, the product of q_t exp(b_t - r) and
 // k_s exp(r - b_s).  Only keys of t's own block have positive exponents; where a channel decays so fast that those could leave
 // fp32, the blocks on the diagonal are summed element by element instead, whose exponents b_t - b_s are never positive.
-// S, A and the keys of the update enter the tensor-core products as two bfloat16 terms, value and remainder.
+// All that a decay has touched - S, A, weighted queries and keys - enters the tensor-core products as two bfloat16 terms, value
+// and remainder (of the product of two such factors the remainders' own is left out).
 //
 // State rows come in pairs: a pass reads one row (-1: zero) and writes another, see cache/state_slots.py.
 #include "api.h"
@@ -37,21 +38,33 @@ struct Gl {
   const float *decay_w, *decay_b;
 };
 
-// log(sigmoid(z)) without overflow
-__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// log(sigmoid(z)) = min(z, 0) - log(1 + e), e = exp(-|z|) in (0, 1].  log(1 + e) = 2 artanh(s) with s = e / (2 + e) <= 1/3, by
+// the series of artanh, whose first terms left out are below 2^-27 of it.
+__device__ __forceinline__ float log_sigmoid(float z) {
+  const float e = ex2(fabsf(z) * -kLog2E), s = e * rcp(2.f + e), q = s * s;
+  float p = 1.f / 15.f;
+  p = fmaf(p, q, 1.f / 13.f);
+  p = fmaf(p, q, 1.f / 11.f);
+  p = fmaf(p, q, 1.f / 9.f);
+  p = fmaf(p, q, 1.f / 7.f);
+  p = fmaf(p, q, 1.f / 5.f);
+  p = fmaf(p, q, 1.f / 3.f);
+  p = fmaf(p, q, 1.f);
+  return fminf(z, 0.f) - 2.f * s * p;
+}
 
 // ---- prep -----------------------------------------------------------------------------------------------------------
-constexpr int kGpThreads = 256, kGpRows = 16, kGpCols = kGpThreads * 4;
+constexpr int kGpThreads = 256, kGpGroup = 16, kGpCols = kGpThreads * 4;      // rows that share a reading of the weights
 
 // grid (blocks of rows, pieces of channels + pieces of columns); u rows in shared memory, padded to 4 floats
 template <typename T>
 __global__ void __launch_bounds__(kGpThreads)
 gl_prep_kernel(T* __restrict__ inp, int ld, const float* __restrict__ planes, int n_planes, const float* __restrict__ side,
-               int side_ld, const Gl m, float* __restrict__ decays, int M, int channel_pieces) {
+               int side_ld, const Gl m, float* __restrict__ decays, int M, int channel_pieces, int rows) {
   extern __shared__ __align__(16) float us[];
   pdl_launch_dependents();
   pdl_wait();
-  const int t0 = blockIdx.x * kGpRows, n = min(M - t0, kGpRows);
+  const int t0 = blockIdx.x * rows, n = min(M - t0, rows);
   const size_t plane = size_t(M) * ld;
   if (blockIdx.y >= channel_pieces) {            // with planes: the columns before the inner vectors
     const int c = m.q_col + (blockIdx.y - channel_pieces) * kGpCols + threadIdx.x * 4;
@@ -71,10 +84,10 @@ gl_prep_kernel(T* __restrict__ inp, int ld, const float* __restrict__ planes, in
     return;
   }
   const int rp = (m.rank + 3) / 4 * 4, width = m.heads * m.dim;
-  for (int i = threadIdx.x; i < kGpRows * rp; i += kGpThreads) {
+  for (int i = threadIdx.x; i < n * rp; i += kGpThreads) {
     const int j = i / rp, r = i % rp, t = t0 + j;
     float x = 0.f;
-    if (j < n && r < m.rank) {
+    if (r < m.rank) {
       if (n_planes > 0) {
         for (int p = 0; p < n_planes; ++p) x += planes[p * plane + size_t(t) * ld + m.rank_col + r];
       } else {
@@ -86,23 +99,43 @@ gl_prep_kernel(T* __restrict__ inp, int ld, const float* __restrict__ planes, in
   __syncthreads();
   const int c = blockIdx.y * kGpThreads + threadIdx.x;
   if (c >= width) return;
-  float z[kGpRows];
   const float bias = m.decay_b[c], inv = 1.f / m.tau;
-#pragma unroll
-  for (int j = 0; j < kGpRows; ++j) z[j] = bias;
-  for (int r = 0; r < rp; r += 4) {
-    float w[4];
+  auto weights = [&](int r, float (&w)[4]) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) w[e] = r + e < m.rank ? m.decay_w[size_t(c) * m.rank + r + e] : 0.f;
+  };
+  auto add = [&](float z, const float (&w)[4], const float* at) {
+    const float4 u = *reinterpret_cast<const float4*>(at);
+    return fmaf(w[0], u.x, fmaf(w[1], u.y, fmaf(w[2], u.z, fmaf(w[3], u.w, z))));
+  };
+  float* dst = decays + size_t(t0) * width + c;
+  if (rp == 16) {                                // the weights stay in registers
+    float w[4][4];
 #pragma unroll
-    for (int j = 0; j < kGpRows; ++j) {
-      const float4 u = *reinterpret_cast<const float4*>(us + j * rp + r);
-      z[j] = fmaf(w[0], u.x, fmaf(w[1], u.y, fmaf(w[2], u.z, fmaf(w[3], u.w, z[j]))));
+    for (int r = 0; r < 4; ++r) weights(r * 4, w[r]);
+#pragma unroll 4
+    for (int j = 0; j < n; ++j) {
+      float z = bias;
+#pragma unroll
+      for (int r = 0; r < 4; ++r) z = add(z, w[r], us + j * 16 + r * 4);
+      dst[size_t(j) * width] = log_sigmoid(z) * inv;
     }
+    return;
   }
+  for (int j0 = 0; j0 < n; j0 += kGpGroup) {
+    float z[kGpGroup];
 #pragma unroll
-  for (int j = 0; j < kGpRows; ++j)
-    if (j < n) decays[size_t(t0 + j) * width + c] = log_sigmoid(z[j]) * inv;
+    for (int j = 0; j < kGpGroup; ++j) z[j] = bias;
+    for (int r = 0; r < rp; r += 4) {
+      float w[4];
+      weights(r, w);
+#pragma unroll
+      for (int j = 0; j < kGpGroup; ++j) z[j] = add(z[j], w, us + min(j0 + j, n - 1) * rp + r);
+    }
+#pragma unroll
+    for (int j = 0; j < kGpGroup; ++j)
+      if (j0 + j < n) dst[size_t(j0 + j) * width] = log_sigmoid(z[j]) * inv;
+  }
 }
 
 // ---- token by token ----------------------------------------------------------------------------------------------------
@@ -266,6 +299,13 @@ __device__ __forceinline__ float2 unpack_bf16(uint32_t x) {
   return make_float2(__uint_as_float(x << 16), __uint_as_float(x & 0xFFFF0000u));
 }
 
+// value and remainder of two numbers
+__device__ __forceinline__ void two_terms(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(x, y);
+  const float2 v = unpack_bf16(hi);
+  lo = pack_bf16(x - v.x, y - v.y);
+}
+
 // MT: 16-row tiles of S per warp (8 warps: dim <= 128 * MT).  grid (column blocks, heads, sequences)
 template <int MT>
 __global__ void __launch_bounds__(kGcThreads, MT == 1 ? 2 : 1)
@@ -316,7 +356,8 @@ gl_chunk_kernel(const bf16* __restrict__ inp, int ld, const float* __restrict__ 
     for (int c = N; c < bp; ++c) sb[i * bp + c] = 0.f;
   }
 
-  const int pr = warp & 3, pc = warp >> 2;       // 16 tokens and half of the columns in the read-out
+  // 16 tokens and half of the columns in the read-out; later tokens have more work, so a scheduler's two warps share it
+  const int pc = warp >> 2, pr = pc ? 3 - (warp & 3) : warp & 3;
   for (int t0 = begin; t0 < end; t0 += kGcT) {
     const int len = min(kGcT, end - t0);
     for (int i = threadIdx.x; i < kGcT * dch; i += kGcThreads) {
@@ -355,8 +396,8 @@ gl_chunk_kernel(const bf16* __restrict__ inp, int ld, const float* __restrict__ 
 #pragma unroll
           for (int h = 0; h < 2; ++h) {
             const int at = ((warp * MT + i) * 16 + r4 + h * 8) * kGcPitch + (n * 8 + c2) * 2;
-            *reinterpret_cast<uint32_t*>(ssh + at) = pack_bf16(S[i][n][h * 2], S[i][n][h * 2 + 1]);
-            *reinterpret_cast<uint32_t*>(ssl + at) = pack_bf16_rest(S[i][n][h * 2], S[i][n][h * 2 + 1]);
+            two_terms(S[i][n][h * 2], S[i][n][h * 2 + 1], *reinterpret_cast<uint32_t*>(ssh + at),
+                      *reinterpret_cast<uint32_t*>(ssl + at));
           }
       }
     cpa_wait<0>();
@@ -394,8 +435,8 @@ gl_chunk_kernel(const bf16* __restrict__ inp, int ld, const float* __restrict__ 
     const float* b_ref = sb + (pr * 16 - 1) * bp + c2;             // not read for pr 0
     const float* b_k = sb + (pc * 32 + r4) * bp + c2;
     for (int kk = 0; kk < ksteps; ++kk) {
-      uint32_t a[4], b[4], ah[4], as[4];
-      ldm_x4(q_addr + kk * 32, a);
+      uint32_t b[4], qh[4], ql[4], sh[4], sl[4];   // queries towards their block's start, and towards the chunk's
+      ldm_x4(q_addr + kk * 32, qh);
       float2 ref[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
       if (pr > 0) {
         ref[0] = *reinterpret_cast<const float2*>(b_ref + kk * 16);
@@ -407,15 +448,27 @@ gl_chunk_kernel(const bf16* __restrict__ inp, int ld, const float* __restrict__ 
 #pragma unroll
         for (int h = 0; h < 2; ++h) {            // rows r4 and r4 + 8
           const float2 bt = *reinterpret_cast<const float2*>(b_q + h * 8 * bp + kk * 16 + x * 8);
-          const float2 q = unpack_bf16(a[x * 2 + h]);
+          const float2 q = unpack_bf16(qh[x * 2 + h]);
           const float qx = q.x * q_scale * ex2(bt.x - ref[x].x), qy = q.y * q_scale * ex2(bt.y - ref[x].y);
-          ah[x * 2 + h] = pack_bf16(qx, qy);
-          as[x * 2 + h] = pack_bf16(qx * ex, qy * ey);
+          two_terms(qx, qy, qh[x * 2 + h], ql[x * 2 + h]);
+          two_terms(qx * ex, qy * ey, sh[x * 2 + h], sl[x * 2 + h]);
         }
+      }
+#pragma unroll
+      for (int n = 0; n < 4; n += 2) {
+        ldm_x4_t(sh_addr + kk * 16 * kGcPitch + n * 16, b);
+        mma_bf16(acc[n], sh, b[0], b[1]);
+        mma_bf16(acc[n + 1], sh, b[2], b[3]);
+        mma_bf16(acc[n], sl, b[0], b[1]);
+        mma_bf16(acc[n + 1], sl, b[2], b[3]);
+        ldm_x4_t(sl_addr + kk * 16 * kGcPitch + n * 16, b);
+        mma_bf16(acc[n], sh, b[0], b[1]);
+        mma_bf16(acc[n + 1], sh, b[2], b[3]);
       }
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         if (j >= blocks || (slow && pc * 2 + j == pr)) continue;
+        uint32_t bl[4];
         ldm_x4(k_addr + j * 16 * qp + kk * 32, b);
 #pragma unroll
         for (int h = 0; h < 2; ++h)              // keys r4 and r4 + 8 of the block
@@ -423,19 +476,14 @@ gl_chunk_kernel(const bf16* __restrict__ inp, int ld, const float* __restrict__ 
           for (int x = 0; x < 2; ++x) {
             const float2 bs = *reinterpret_cast<const float2*>(b_k + (j * 16 + h * 8) * bp + kk * 16 + x * 8);
             const float2 key = unpack_bf16(b[h * 2 + x]);
-            b[h * 2 + x] = pack_bf16(key.x * ex2(ref[x].x - bs.x), key.y * ex2(ref[x].y - bs.y));
+            two_terms(key.x * ex2(ref[x].x - bs.x), key.y * ex2(ref[x].y - bs.y), b[h * 2 + x], bl[h * 2 + x]);
           }
-        mma_bf16(sc[j * 2], ah, b[0], b[1]);
-        mma_bf16(sc[j * 2 + 1], ah, b[2], b[3]);
-      }
-#pragma unroll
-      for (int n = 0; n < 4; n += 2) {
-        ldm_x4_t(sh_addr + kk * 16 * kGcPitch + n * 16, b);
-        mma_bf16(acc[n], as, b[0], b[1]);
-        mma_bf16(acc[n + 1], as, b[2], b[3]);
-        ldm_x4_t(sl_addr + kk * 16 * kGcPitch + n * 16, b);
-        mma_bf16(acc[n], as, b[0], b[1]);
-        mma_bf16(acc[n + 1], as, b[2], b[3]);
+        mma_bf16(sc[j * 2], qh, b[0], b[1]);
+        mma_bf16(sc[j * 2 + 1], qh, b[2], b[3]);
+        mma_bf16(sc[j * 2], ql, b[0], b[1]);
+        mma_bf16(sc[j * 2 + 1], ql, b[2], b[3]);
+        mma_bf16(sc[j * 2], qh, bl[0], bl[1]);
+        mma_bf16(sc[j * 2 + 1], qh, bl[2], bl[3]);
       }
     }
     if (slow && (pr >> 1) == pc) {               // the block on the diagonal, element by element
@@ -470,8 +518,8 @@ gl_chunk_kernel(const bf16* __restrict__ inp, int ld, const float* __restrict__ 
       for (int n = 0; n < 4; ++n) {
         const int c = pc * 32 + n * 8 + c2;
         const float x = c <= t ? sc[n][h * 2] : 0.f, y = c + 1 <= t ? sc[n][h * 2 + 1] : 0.f;
-        *reinterpret_cast<uint32_t*>(sph + t * kGcPitch + c * 2) = pack_bf16(x, y);
-        *reinterpret_cast<uint32_t*>(spl + t * kGcPitch + c * 2) = pack_bf16_rest(x, y);
+        two_terms(x, y, *reinterpret_cast<uint32_t*>(sph + t * kGcPitch + c * 2),
+                  *reinterpret_cast<uint32_t*>(spl + t * kGcPitch + c * 2));
       }
     }
     __syncthreads();
@@ -535,8 +583,7 @@ gl_chunk_kernel(const bf16* __restrict__ inp, int ld, const float* __restrict__ 
             const float* at = b_s + (kk * 16 + x * 8) * bp + h * 8;
             const float2 key = unpack_bf16(a[x * 2 + h]);
             const float k0 = key.x * ex2(b_end[h] - at[0]), k1 = key.y * ex2(b_end[h] - at[bp]);
-            a[x * 2 + h] = pack_bf16(k0, k1);
-            al[x * 2 + h] = pack_bf16_rest(k0, k1);
+            two_terms(k0, k1, a[x * 2 + h], al[x * 2 + h]);
           }
         const uint32_t w = smem_u32(sv) + v_row + kk * 16 * kGcPitch;
 #pragma unroll
@@ -622,11 +669,15 @@ int launch_gl_prep(void* inp, int ld, const void* planes, int n_planes, const vo
   const Gl m = gl_of(z);
   const int pieces = (m.heads * m.dim + kGpThreads - 1) / kGpThreads;
   const int copies = n_planes > 0 ? (m.rank_col - m.q_col + kGpCols - 1) / kGpCols : 0;
-  const size_t smem = size_t(kGpRows) * ((m.rank + 3) / 4 * 4) * sizeof(float);
+  const int rp = (m.rank + 3) / 4 * 4;
+  int rows = M >= 4096 ? 64 : 16;
+  while (rows > 1 && size_t(rows) * rp * sizeof(float) > 48 * 1024) rows /= 2;
+  const size_t smem = size_t(rows) * rp * sizeof(float);
   if (smem > 48 * 1024) return ZSE_ERR_LIMIT;
-  return launch_pdl(gl_prep_kernel<T>, dim3((M + kGpRows - 1) / kGpRows, pieces + copies), dim3(kGpThreads), smem, st,
+  return launch_pdl(gl_prep_kernel<T>, dim3((M + rows - 1) / rows, pieces + copies), dim3(kGpThreads), smem, st,
                     reinterpret_cast<T*>(inp), ld, reinterpret_cast<const float*>(planes), n_planes,
-                    reinterpret_cast<const float*>(side), side_ld, m, reinterpret_cast<float*>(decays), M, pieces) == cudaSuccess
+                    reinterpret_cast<const float*>(side), side_ld, m, reinterpret_cast<float*>(decays), M, pieces,
+                    rows) == cudaSuccess
              ? 0
              : ZSE_ERR_LAUNCH;
 }

@@ -171,33 +171,53 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
 }
 
-// Means over the `pool` tokens up to position `pos` of a sequence's cached keys and values (VEC columns per access), from the
-// calling threads tid, tid + step, ...; blocks that are gone count as zeros.
+// Pieces of VEC columns of a cached token, keys first, then values.
+template <int VEC>
+__device__ __forceinline__ int cached_pieces(const Heads& h) { return h.kv_heads * (h.dim / VEC + h.vdim / VEC); }
+
+// Piece i of a cached token: a place in its row of `kc` or `vc`.
 template <typename T, int VEC>
-__device__ __forceinline__ void pool_means(T* kc, T* vc, const Heads& h, const int* table, int pos, int tid, int step) {
-  const int b = pos / h.pool, first = b * h.pool;
-  const int to = table[h.means_at + h.block_of(b)], at = h.in_block(b);
-  if (to < 0) return;
-  const int kv = h.dim / VEC, vv = h.vdim / VEC, n = h.kv_heads * (kv + vv);
-  const float inv = 1.f / float(h.pool);
-  for (int i = tid; i < n; i += step) {
-    const bool key = i < h.kv_heads * kv;
-    const int j = key ? i : i - h.kv_heads * kv, per = key ? kv : vv;
-    const int g = j / per, c = j % per * VEC, width = key ? h.dp : h.vp;
-    T* cache = key ? kc : vc;
-    F32Vec<VEC> sum{};
-#pragma unroll 8
-    for (int p = first; p <= pos; ++p) {
-      const int block = table[h.block_of(p)];
-      if (block < 0) continue;
-      const F32Vec<VEC> x = load_vec<VEC>(cache + h.at(block, g, h.in_block(p), width) + c);
+__device__ __forceinline__ T* cached_piece(T* kc, T* vc, const Heads& h, int block, int token, int i) {
+  const int kv = h.dim / VEC, n = h.kv_heads * kv;
+  if (i < n) return kc + h.at(block, i / kv, token, h.dp) + i % kv * VEC;
+  const int vv = h.vdim / VEC;
+  return vc + h.at(block, (i - n) / vv, token, h.vp) + (i - n) % vv * VEC;
+}
+
+// Sum of piece i over the cached tokens [from, to) of a sequence; blocks that are gone count as zeros.
+template <typename T, int VEC>
+__device__ __forceinline__ F32Vec<VEC> pool_sum(T* kc, T* vc, const Heads& h, const int* table, int i, int from, int to) {
+  constexpr int kAhead = 8;                      // tokens whose loads are under way together
+  F32Vec<VEC> sum{};
+  const T* base = cached_piece<T, VEC>(kc, vc, h, 0, 0, i);
+  const int width = i < h.kv_heads * (h.dim / VEC) ? h.dp : h.vp;
+  for (int p0 = from; p0 < to; p0 += kAhead) {
+    int block[kAhead];
+    F32Vec<VEC> x[kAhead];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) sum.v[e] += x.v[e];
+    for (int u = 0; u < kAhead; ++u) block[u] = p0 + u < to ? table[h.block_of(p0 + u)] : -1;
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+      x[u] = F32Vec<VEC>{};
+      if (block[u] >= 0) x[u] = load_vec<VEC>(base + size_t(block[u]) * h.block_stride + size_t(h.in_block(p0 + u)) * width);
     }
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) sum.v[e] *= inv;
-    store_vec<VEC>(cache + h.at(to, g, at, width) + c, sum);
+    for (int u = 0; u < kAhead; ++u)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) sum.v[e] += x[u].v[e];
   }
+  return sum;
+}
+
+// Stores a sum over a block of tokens as the mean of the sequence's block b.
+template <typename T, int VEC>
+__device__ __forceinline__ void put_mean(T* kc, T* vc, const Heads& h, const int* table, int i, int b, F32Vec<VEC> sum) {
+  const int to = table[h.means_at + h.block_of(b)];
+  if (to < 0) return;
+  const float inv = 1.f / float(h.pool);
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) sum.v[e] *= inv;
+  store_vec<VEC>(cached_piece<T, VEC>(kc, vc, h, to, h.in_block(b), i), sum);
 }
 
 // grid (blocks of kPoolRows rows)
@@ -212,7 +232,9 @@ heads_pool_kernel(T* kc, T* vc, const Heads h, const int* __restrict__ row_seq, 
     const int pos = positions[t];
     if ((pos + 1) % h.pool) continue;
     const int s = row_seq != nullptr ? row_seq[t] : t;
-    pool_means<T, VEC>(kc, vc, h, h.tables + size_t(s) * h.max_blocks, pos, threadIdx.x, 256);
+    const int* table = h.tables + size_t(s) * h.max_blocks;
+    for (int i = threadIdx.x; i < cached_pieces<VEC>(h); i += 256)
+      put_mean<T, VEC>(kc, vc, h, table, i, pos / h.pool, pool_sum<T, VEC>(kc, vc, h, table, i, pos + 1 - h.pool, pos + 1));
   }
 }
 
@@ -259,11 +281,21 @@ heads_prep_whole_kernel(T* __restrict__ inp, const float* __restrict__ planes, i
   };
   const int nq = h.heads * h.dim, nk = a.own_kv ? h.kv_heads * h.dim : 0, nv = a.own_kv ? h.kv_heads * h.vdim : 0;
   const int step = THREADS * VEC, far = kKeep * step, i0 = threadIdx.x * VEC;
-  F32Vec<VEC> q[kKeep], k0{};
+  constexpr bool kEarly = THREADS > 256;         // few rows: latency counts, not registers
+  F32Vec<VEC> q[kKeep], qw[kEarly ? kKeep : 1], k0{}, kw{};
   float qs = 0.f, ks = 0.f;
+  const long long slot = a.own_kv ? slots[t] : -1;
+  // what does not depend on the row's values is under way before they are summed
+  const int* table = h.tables + size_t(pool_rows ? t : 0) * h.max_blocks;
+  const bool due = pool_rows && slot >= 0 && h.pool > 0 && (pos_i + 1) % h.pool == 0;
+  const int pieces = cached_pieces<VEC>(h);
+  F32Vec<VEC> before{};
+  if (due && threadIdx.x < pieces) before = pool_sum<T, VEC>(kc, vc, h, table, threadIdx.x, pos_i + 1 - h.pool, pos_i);
+  if (kEarly && i0 < nk) kw = load_vec<VEC>(k_norm + i0);
 #pragma unroll
   for (int j = 0; j < kKeep; ++j)
     if (i0 + j * step < nq) {
+      if constexpr (kEarly) qw[j] = load_vec<VEC>(q_norm + i0 + j * step);
       q[j] = value(i0 + j * step);
       if constexpr (VEC == 1) row[i0 + j * step] = q[j].v[0];
 #pragma unroll
@@ -281,7 +313,6 @@ heads_prep_whole_kernel(T* __restrict__ inp, const float* __restrict__ planes, i
 #pragma unroll
     for (int e = 0; e < VEC; ++e) ks += x.v[e] * x.v[e];
   }
-  const long long slot = a.own_kv ? slots[t] : -1;
   const int block = slot >= 0 ? h.block_of(int(slot)) : 0, token = slot >= 0 ? h.in_block(int(slot)) : 0;
   if (slot >= 0) {
     for (int i = i0; i < nv; i += step)
@@ -298,9 +329,8 @@ heads_prep_whole_kernel(T* __restrict__ inp, const float* __restrict__ planes, i
     y = y * cs.x + u0 * cs.y;
   };
   // columns i.. of the queries (or keys), normed, weighted and turned; `other_of`: one column of the same row, for VEC 1
-  auto finished = [&](F32Vec<VEC> v, int i, float inv, const T* w, float factor, auto other_of) {
+  auto finished = [&](F32Vec<VEC> v, int i, float inv, const F32Vec<VEC>& f, const T* w, float factor, auto other_of) {
     const int d = i % h.dim;
-    const F32Vec<VEC> f = load_vec<VEC>(w + i);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) v.v[e] *= inv * f.v[e];
     if constexpr (VEC == 4) {
@@ -318,30 +348,37 @@ heads_prep_whole_kernel(T* __restrict__ inp, const float* __restrict__ planes, i
     for (int e = 0; e < VEC; ++e) v.v[e] *= factor;
     return v;
   };
-  auto put_q = [&](int i, const F32Vec<VEC>& x) {
+  auto put_q = [&](int i, const F32Vec<VEC>& x, const F32Vec<VEC>& w) {
     const float factor = head_temp != nullptr ? head_temp[i / h.dim] : 1.f;
-    store_vec<VEC>(in + i, finished(x, i, q_inv, q_norm, factor, [&](int o) { return row[o]; }));
+    store_vec<VEC>(in + i, finished(x, i, q_inv, w, q_norm, factor, [&](int o) { return row[o]; }));
   };
 #pragma unroll
   for (int j = 0; j < kKeep; ++j)
-    if (i0 + j * step < nq) put_q(i0 + j * step, q[j]);
+    if (i0 + j * step < nq) put_q(i0 + j * step, q[j], kEarly ? qw[kEarly ? j : 0] : load_vec<VEC>(q_norm + i0 + j * step));
   for (int i = far + i0; i < nq; i += step) {
     F32Vec<VEC> x;
     if constexpr (VEC == 1)
       x.v[0] = row[i];
     else
       x = value(i);
-    put_q(i, x);
+    put_q(i, x, load_vec<VEC>(q_norm + i));
   }
   if (slot < 0) return;                          // the same for the whole block
   for (int i = i0; i < nk; i += step) {
     const F32Vec<VEC> x = i == i0 ? k0 : value(a.k_col + i);
     store_vec<VEC>(kc + h.at(block, i / h.dim, token, h.dp) + i % h.dim,
-                   finished(x, i, k_inv, k_norm, 1.f, [&](int o) { return value(a.k_col + o).v[0]; }));
+                   finished(x, i, k_inv, kEarly && i == i0 ? kw : load_vec<VEC>(k_norm + i), k_norm, 1.f,
+                            [&](int o) { return value(a.k_col + o).v[0]; }));
   }
-  if (pool_rows && h.pool > 0 && (pos_i + 1) % h.pool == 0) {
+  if (due) {
     __syncthreads();                             // this token's key and value are in the cache
-    pool_means<T, VEC>(kc, vc, h, h.tables + size_t(t) * h.max_blocks, pos_i, threadIdx.x, THREADS);
+    for (int i = threadIdx.x; i < pieces; i += THREADS) {
+      F32Vec<VEC> sum = i == threadIdx.x ? before : pool_sum<T, VEC>(kc, vc, h, table, i, pos_i + 1 - h.pool, pos_i);
+      const F32Vec<VEC> own = load_vec<VEC>(cached_piece<T, VEC>(kc, vc, h, block, token, i));
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) sum.v[e] += own.v[e];
+      put_mean<T, VEC>(kc, vc, h, table, i, pos_i / h.pool, sum);
+    }
   }
 }
 
