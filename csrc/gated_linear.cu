@@ -153,7 +153,7 @@ __device__ __forceinline__ float gt_sum(float v, float* red) {
 
 // grid (cluster, heads, sequences)
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kGtThreads)
+__global__ void __launch_bounds__(kGtThreads, 3)
 gl_tokens_kernel(const T* __restrict__ inp, int ld, const float* __restrict__ planes, int n_planes, int M,
                  const float* __restrict__ decays, const Gl m, const int* __restrict__ cu_q, const T* __restrict__ head_norm,
                  T* __restrict__ out, int ldo) {

@@ -1,6 +1,6 @@
 """Decoders whose layers mix attention over heads and recurrent mixers (matrix memories, state spaces), over the paged cache
 and the state slots: layer runs, mixers, feed-forwards, and the placement of norms on the sublayers' outputs (Nimelorn).
-``looped`` has the other placement.
+``looped`` and ``twin`` have the other placements.
 
 Same pass contract as ``DecoderModel``.  The residual x is fp32; sublayers read x itself (rounded to the activations' type):
 
@@ -14,7 +14,9 @@ and values projects queries only.  Rows that decode, and chunks of at most ``SHO
 the keys split over CTAs; longer chunks run in tiles of queries.  A matrix memory does the same: short chunks step through
 the state token by token, with read-out, head norm and output gate in the step's kernel; longer ones run chunkwise, with the
 decays inside a chunk as a lower-triangular matrix.  A state space passes its inputs through a short convolution first, whose
-last inputs are part of its state, and does the same.  A packed pass may hold both kinds: short ones are laid out first.
+last inputs are part of its state, and does the same; so does gated linear attention.  Attention that sees older tokens as means
+of blocks keeps those in blocks of the cache of their own, behind the tokens' in the block tables; the kernel that writes a
+block's last key and value writes the mean in a decode step, one more kernel in any other pass.  A packed pass may hold both kinds: short ones are laid out first.
 
 A sequence's recurrent state and its last token live in ``cache.state_slots``; ``state_rows`` names the rows that a pass's
 sequences read and write.
@@ -193,7 +195,7 @@ class HybridStepBuffers(StepBuffers):
 
 
 class HybridModel(DesignModel):
-    """Layers whose norms sit on the sublayers' outputs; ``models.looped`` has the other placement."""
+    """Layers whose norms sit on the sublayers' outputs; ``models.looped`` and ``models.twin`` have the other placements."""
     kernel_group = "hybrid"
     means_at = 0                # column of the block tables from which on the blocks of means stand; set by the runner
 
